@@ -193,6 +193,8 @@ class AdapterManager:
             self.stats["host_hits"] += 1
             return hb
         self.stats["host_misses"] += 1
+        if not self.layout.groups:
+            raise ValueError(f"{self.model.config.model_type} models take no adapters")
         check_architecture(cfg, mm, self.model.config)
         blob, rp = self.layout.pack(cfg, mm, dtype=self.dtype, pin=self.is_cuda)
         hb = HostBlob(key, blob, rp, blob.numel() * blob.element_size())

@@ -16,7 +16,7 @@ import dataclasses
 import json
 import os
 from dataclasses import dataclass, field
-from typing import Any, Dict, List, Optional
+from typing import Any, Dict, List, Optional, Tuple
 
 # Architectures handled by the single config-driven decoder (models/decoder.py).
 DECODER_MODEL_TYPES = (
@@ -24,6 +24,19 @@ DECODER_MODEL_TYPES = (
     "cohere", "solar", "granite", "gpt2", "gpt_neox", "falcon", "RefinedWeb",
     "RefinedWebModel", "gpt_bigcode", "dbrx",
 )
+
+
+# Designs whose config.json lists its layers one by one, each with a mixer of its own (models/mixers.py).
+MIXER_MODEL_TYPES = ("vabunex",)
+
+
+@dataclass
+class LayerSpec:
+    """One layer of a design whose layers differ: the kind of mixer, the mixer's sizes and constants, and the width of the
+    gated feed-forward beside it (0: none)."""
+    mixer: str
+    params: Dict[str, Any]
+    ff: int = 0
 
 
 @dataclass
@@ -75,6 +88,9 @@ class ModelConfig:
     embed_norm: bool = False
     # clamp of the fused QKV projection's output (mpt, dbrx)
     clip_qkv: Optional[float] = None
+    # layer-by-layer designs: the layers, and (start, stop, times): layers start .. stop-1 run `times` times in a row
+    layer_specs: Optional[List[LayerSpec]] = None
+    layer_loop: Optional[Tuple[int, int, int]] = None
     eos_token_id: Any = None
     bos_token_id: Any = None
     pad_token_id: Any = None
@@ -102,6 +118,15 @@ class ModelConfig:
         return int(self.head_dim * self.partial_rotary_factor)
 
     @property
+    def layer_schedule(self) -> List[int]:
+        """Layer indices in the order they run (a looped range counts every pass)."""
+        n = self.num_hidden_layers
+        if self.layer_loop is None:
+            return list(range(n))
+        a, b, k = self.layer_loop
+        return list(range(a)) + list(range(a, b)) * k + list(range(b, n))
+
+    @property
     def is_moe(self) -> bool:
         return self.num_local_experts > 0
 
@@ -117,7 +142,9 @@ class ModelConfig:
     @classmethod
     def from_dict(cls, d: Dict[str, Any]) -> "ModelConfig":
         d = dict(d)
-        mt = d.get("model_type", "llama")
+        mt = d.get("model_type") or str(d.get("architecture", "")).lower() or "llama"
+        if mt in MIXER_MODEL_TYPES:
+            return cls(**_mixer_model_kwargs(mt, d))
         known = {f.name for f in dataclasses.fields(cls)}
         kw: Dict[str, Any] = {k: v for k, v in d.items() if k in known}
         extra = {k: v for k, v in d.items() if k not in known}
@@ -221,6 +248,28 @@ class ModelConfig:
         d = dataclasses.asdict(self)
         d.update(d.pop("extra"))
         return d
+
+
+def _mixer_model_kwargs(mt: str, d: Dict[str, Any]) -> Dict[str, Any]:
+    """ModelConfig fields of a config.json that lists its layers (`layers`, `loop`, `norm`, `embedding`, `vocab`, `width`)."""
+    specs = []
+    for i, layer in enumerate(d["layers"]):
+        mlp = layer.get("mlp")
+        if mlp is not None and mlp.get("kind", "dense") != "dense":
+            raise NotImplementedError(f"layer {i}: feed-forward kind {mlp['kind']!r}")
+        specs.append(LayerSpec(layer["type"], dict(layer["mixer"]), int(mlp["ff"]) if mlp is not None else 0))
+    loop = d.get("loop")
+    if loop is not None:
+        loop = (int(loop["start"]), int(loop["stop"]), int(loop["times"]))
+        if not (0 <= loop[0] <= loop[1] <= len(specs)) or loop[2] < 0:
+            raise ValueError(f"loop {loop} does not fit {len(specs)} layers")
+    heads = max([int(s.params["heads"]) for s in specs] + [1])
+    return dict(model_type=mt, vocab_size=int(d["vocab"]), hidden_size=int(d["width"]), intermediate_size=max([s.ff for s in specs] + [1]),
+                num_hidden_layers=len(specs), num_attention_heads=heads, head_dim=max([int(s.params["dim"]) for s in specs] + [1]),
+                rms_norm_eps=float(d["norm"]["eps"]), max_position_embeddings=int(d.get("max_position_embeddings", 1 << 20)),
+                hidden_act="gelu_tanh", norm_weight_offset=1.0, embedding_multiplier=float(d["embedding"]["scale"]), parallel_residual=True,
+                layer_specs=specs, layer_loop=loop, eos_token_id=d.get("eos_token_id"), bos_token_id=d.get("bos_token_id"),
+                torch_dtype=d.get("torch_dtype", "bfloat16"), extra={})
 
 
 def mistral_7b() -> ModelConfig:

@@ -107,6 +107,20 @@ class StepInputs:
     # vision-language prompts: rows of the embedded sequence that are replaced by projected image features
     embed_rows: Optional[torch.Tensor] = None
     embed_values: Optional[torch.Tensor] = None
+    # Models with per-request state: the state slot of every sequence (prefill: [B], decode: [T]; mixed: the decode rows' slots
+    # apart), and the prompt tokens cut into segments of `seg_len` for the recurrence kernels (sequence, first token within it)
+    state_slots: Optional[torch.Tensor] = None
+    dec_state_slots: Optional[torch.Tensor] = None
+    seg_seq: Optional[torch.Tensor] = None
+    seg_q0: Optional[torch.Tensor] = None
+    seg_len: int = 0
+    max_ctx: int = 0                                 # longest context of the prefill sequences (host knowledge; 0: unknown)
+
+    def decode_view(self, T: int):
+        """(decode rows, their block tables, state slots, context lengths) of a step over T rows."""
+        if not self.is_prefill:
+            return T, self.block_tables, self.state_slots, self.ctx_lens
+        return self.n_decode, self.dec_block_tables, self.dec_state_slots, self.ctx_lens
 
 
 class DecoderModel:
@@ -125,12 +139,19 @@ class DecoderModel:
         self.nkv = max(c.num_key_value_heads // ws, 1)
         self.kv_replicas = max(ws // c.num_key_value_heads, 1)
         self.d = c.head_dim
+        self.eps = c.rms_norm_eps
+        self.schedule = c.layer_schedule         # layer of every run (a looped layer runs several times, each with its own cache)
+        self.mixed = c.layer_specs is not None   # layers with mixers of their own (models/mixers.py) on an fp32 residual stream
+        self.recurrent = False
+        if self.mixed:
+            from .mixers import MIXERS
+            self.recurrent = any(getattr(MIXERS.get(sp.mixer), "recurrent", False) for sp in c.layer_specs)
         self.inter = c.intermediate_size // ws if not c.is_moe else c.intermediate_size
         self.hidden = c.hidden_size
         self.vocab = c.vocab_size
         self.vocab_local = (c.vocab_size + ws - 1) // ws
         self.vocab_start = self.tp.rank * self.vocab_local
-        self.ops = get_ops(self.device, dtype)
+        self.ops = get_ops(self.device, dtype, fp32=self.mixed)
         self.layers: List[LayerWeights] = []
         self.embed: Optional[torch.Tensor] = None
         self.pos_embed: Optional[torch.Tensor] = None
@@ -146,7 +167,8 @@ class DecoderModel:
         if scaling and scaling.get("rope_type", scaling.get("type")) == "dynamic" and "original_max_position_embeddings" not in scaling:
             # dynamic NTK stretches the base once the table is longer than the length the model was trained at
             scaling = dict(scaling, original_max_position_embeddings=c.max_position_embeddings)
-        self.cos_sin = reference.rope_cache(c.rotary_dim, self.max_positions, c.rope_theta, scaling, device=self.device)
+        self._rope_tables: Dict[tuple, torch.Tensor] = {}
+        self.cos_sin = None if self.mixed else reference.rope_cache(c.rotary_dim, self.max_positions, c.rope_theta, scaling, device=self.device)
         self.adapters = None     # AdapterManager, attached by the runtime
         self.quantized: Optional[str] = None
         self.keep_hidden = False                 # keep the head's input rows of the last eager forward pass in `last_hidden`
@@ -167,6 +189,17 @@ class DecoderModel:
             full = alibi_slopes(c.num_attention_heads, c.alibi_bias_max, interleave=c.model_type == "mpt")
             self.alibi_slopes = full[self.tp.rank * self.nh:(self.tp.rank + 1) * self.nh].to(self.device).contiguous()
 
+    def rope_table(self, rot: int, base: float) -> torch.Tensor:
+        """cos / sin of a layer's own rotation, shared by the layers that have the same one."""
+        key = (rot, base)
+        if key not in self._rope_tables:
+            self._rope_tables[key] = reference.rope_table(rot, self.max_positions, base, self.device)
+        return self._rope_tables[key]
+
+    def cache_shapes(self) -> Optional[List[dict]]:
+        """What every layer run keeps (`Mixer.cache_shape`), or None for the uniform key/value cache."""
+        return [self.layers[li].mixer.cache_shape(self) for li in self.schedule] if self.mixed else None
+
     # ------------------------------------------------------------------ shapes
     @property
     def q_size(self):
@@ -183,6 +216,8 @@ class DecoderModel:
     def group_shapes(self) -> Dict[str, dict]:
         """Per projection group: K (input features on this rank), N (outputs on this rank), output part sizes,
         and which side is sharded (column groups shard N, row groups shard K)."""
+        if self.mixed:
+            return {}                            # the fused projections of these layers take no adapters
         g = {
             "qkv": dict(K=self.hidden, parts=[self.q_size, self.kv_size, self.kv_size], shard="col",
                         names=["q_proj", "k_proj", "v_proj"]),
@@ -205,6 +240,10 @@ class DecoderModel:
         """Random weights of the right shapes.  Every rank draws the FULL tensors from the same seed and keeps its
         shard, so TP=k and TP=1 hold the same model (needed for the rank-consistency tests)."""
         m = cls(config, device, dtype, tp, max_positions)
+        if m.mixed:
+            from .mixers import RandomWeights, load_mixer_layers
+            load_mixer_layers(m, RandomWeights(config, "cpu", seed))
+            return m
         c, ws, rk = config, m.tp.world_size, m.tp.rank
         gen = torch.Generator(device="cpu").manual_seed(seed)
 
@@ -297,6 +336,10 @@ class DecoderModel:
         drawing the full tensors on the host as `random_init` does would take minutes).  Ranks use different
         seeds, so this is a statistically equivalent model per TP degree, not the same model."""
         m = cls(config, device, dtype, tp, max_positions)
+        if m.mixed:
+            from .mixers import RandomWeights, load_mixer_layers
+            load_mixer_layers(m, RandomWeights(config, m.device, seed))
+            return m
         c, ws = config, m.tp.world_size
         gen = torch.Generator(device=m.device).manual_seed(seed * 1000 + m.tp.rank)
 
@@ -347,6 +390,8 @@ class DecoderModel:
         """Replace the dense projection matrices of every layer by block-scaled fp8 (e4m3, 128 x 128 scales) for the
         fp8 tensor-core GEMM; embeddings, norms, the lm_head, MoE experts and every LoRA adapter stay as they are.
         The reference's `--quantize fp8` does the same on load with per-tensor scales (layers/fp8.py:14-45)."""
+        if self.mixed:
+            raise ValueError(f"quantisation of {self.config.model_type} is not supported")
         for lw in self.layers:
             for name in ("qkv_w", "o_w", "gate_up_w", "down_w"):
                 w = getattr(lw, name)
@@ -363,6 +408,8 @@ class DecoderModel:
         holds in packed form are left as loaded."""
         if method == "fp8":
             return self.quantize_fp8()
+        if self.mixed:
+            raise ValueError(f"quantisation of {self.config.model_type} is not supported")
         from ..utils.quant_formats import quantize_weight
         for lw in self.layers:
             for name in ("qkv_w", "o_w", "gate_up_w", "down_w"):
@@ -438,7 +485,7 @@ class DecoderModel:
     def _native_executor(self, inp: StepInputs, kv_cache: List[torch.Tensor]):
         """The C++ layer executor for eager steps (prefill, mixed prefill + decode) of the architectures it covers;
         None keeps the per-kernel Python path (decode steps are CUDA graphs, where host time does not matter)."""
-        if not inp.is_prefill or not self.use_native_layers or torch.cuda.is_current_stream_capturing():
+        if self.mixed or not inp.is_prefill or not self.use_native_layers or torch.cuda.is_current_stream_capturing():
             return None
         from . import native_exec
         ex = self._native
@@ -452,6 +499,13 @@ class DecoderModel:
     def forward(self, inp: StepInputs, kv_cache: List[torch.Tensor]) -> torch.Tensor:
         """-> logits [n_out, vocab] (full vocabulary on every rank)."""
         c, ops = self.config, self.ops
+        if self.mixed:
+            # fp32 residual stream; every layer hands its contribution to the norm that reads the stream next
+            residual, pending = ops.embed_stream(inp.input_ids, self.embed, c.embedding_multiplier), None
+            for run, li in enumerate(self.schedule):
+                pending = self.layers[li].forward(self, residual, pending, inp, kv_cache[run])
+            hidden = ops.norm_stream(residual, pending, self.final_norm, self.eps, c.norm_weight_offset, self.hidden, self.dtype)
+            return self._score(hidden, inp)
         fused = self.tp.fused if self.tp.world_size > 1 else None
         if fused is not None and fused.embed_ptrs is not None and inp.input_ids.is_cuda:
             h = fused.embed(inp.input_ids, c.embedding_multiplier)       # peer reads, no collective
@@ -492,6 +546,10 @@ class DecoderModel:
             normed2 = self._norm(attn_out, residual, lw.post_norm, lw.post_norm_b, x_scale=rm)
             pending = self._moe(normed2, lw, li, inp) if c.is_moe else self._mlp(normed2, lw, li, inp)
         hidden = self._norm(pending, residual, self.final_norm, self.final_norm_b, x_scale=rm)
+        return self._score(hidden, inp)
+
+    def _score(self, hidden: torch.Tensor, inp: StepInputs) -> torch.Tensor:
+        """Logits of the rows the step asks for."""
         if inp.lm_head_indices is not None:
             hidden = hidden.index_select(0, inp.lm_head_indices.long()) if hidden.device.type == "cpu" else hidden[inp.lm_head_indices.long()]
         if self.keep_hidden:

@@ -129,6 +129,9 @@ def _shard_qkv(m: DecoderModel, q, k, v):
 
 def load_decoder_weights(m: DecoderModel, w: AbstractWeights):
     c = m.config
+    if m.mixed:
+        from .mixers import load_mixer_layers
+        return load_mixer_layers(m, w)
     nm = NAME_MAPS.get(c.model_type)
     if nm is None:
         raise NotImplementedError(f"no weight map for model_type={c.model_type}")

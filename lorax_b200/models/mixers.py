@@ -1,0 +1,335 @@
+"""Layers of designs that list their layers one by one: a token mixer and an optional gated feed-forward in parallel, both reading
+one RMS norm of the fp32 residual stream.
+
+A mixer declares its tensors (`shapes`), what it keeps per token or per request (`cache_shape`), which of its projections read the
+layer's norm (`in_parts`, fused with the feed-forward's gate and up projections into one GEMM) and its output projection (`out_parts`,
+fused with the down projection into one GEMM: the sum of both sublayers is formed in the accumulator).  All sizes are padded to
+multiples of 16 with zero weights when the layer is loaded, so the kernels see aligned heads whatever the configuration says; a padded
+channel stays exactly zero through every operation.
+
+  lightning         linear attention, one constant decay per head, state [heads, dim, vdim] per request
+  wkv               token-shifted linear recurrence with a data-dependent decay per key channel, state [heads, dim, dim] per request
+                    plus the previous token's input
+  latent_attention  softmax attention over a low-rank latent and one shared rotated key part per token, both paged
+"""
+
+from __future__ import annotations
+
+from dataclasses import dataclass, field
+from typing import Dict, List, Optional, Tuple
+
+import torch
+
+PAD = 16
+
+
+def pad16(n: int) -> int:
+    return (n + PAD - 1) // PAD * PAD
+
+
+def _pad_to(t: torch.Tensor, *shape: int) -> torch.Tensor:
+    """Zero-pad every dimension at its end."""
+    if tuple(t.shape) == tuple(shape):
+        return t
+    out = torch.zeros(*shape, dtype=t.dtype, device=t.device)
+    out[tuple(slice(0, n) for n in t.shape)] = t
+    return out
+
+
+def pad_heads_rows(w: torch.Tensor, heads: int, d: int, K: int) -> torch.Tensor:
+    """[heads * d, k] -> [heads * pad16(d), K]: every head's rows padded on their own."""
+    return _pad_to(w.view(heads, d, -1), heads, pad16(d), K).reshape(heads * pad16(d), K)
+
+
+def pad_heads_cols(w: torch.Tensor, heads: int, d: int, N: int) -> torch.Tensor:
+    """[n, heads * d] -> [N, heads * pad16(d)]."""
+    return _pad_to(w.view(w.shape[0], heads, d), N, heads, pad16(d)).reshape(N, heads * pad16(d))
+
+
+def pad_heads_vec(v: torch.Tensor, heads: int, d: int) -> torch.Tensor:
+    return _pad_to(v.reshape(heads, d), heads, pad16(d)).reshape(-1)
+
+
+class Mixer:
+    """Common part.  `get(name)` passed to `load` returns the checkpoint tensor of this mixer in fp32; `fin` brings a matrix to the
+    model's dtype and device, `vec` a vector to fp32 on the device."""
+
+    recurrent = False
+
+    def __init__(self, params: dict, width: int):
+        self.width, self.W = width, pad16(width)
+
+    def shapes(self) -> Dict[str, Tuple[int, ...]]:
+        raise NotImplementedError
+
+    def in_parts(self, get) -> List[Tuple[str, torch.Tensor]]:
+        """(name, [rows, W]) of the projections that read the layer's norm."""
+        raise NotImplementedError
+
+    def out_part(self, get) -> torch.Tensor:
+        """Output projection [W, out_dim]."""
+        raise NotImplementedError
+
+    def load(self, get, fin, vec, model):
+        raise NotImplementedError
+
+    def cache_shape(self, model) -> dict:
+        """{"paged": width per token} or {"state": {name: (shape per request, dtype)}}."""
+        raise NotImplementedError
+
+    def run(self, model, h, proj, y, inp, cache):
+        """Mixes the step's rows: h [T, W] the layer's norm, proj name -> view of the fused projection, y [T, out_dim] the result."""
+        raise NotImplementedError
+
+
+class LightningMixer(Mixer):
+    recurrent = True
+
+    def __init__(self, params: dict, width: int):
+        super().__init__(params, width)
+        self.H, self.d, self.dv = int(params["heads"]), int(params["dim"]), int(params["vdim"])
+        self.decay_values = [float(x) for x in params["decay"]]
+        if len(self.decay_values) != self.H:
+            raise ValueError(f"{len(self.decay_values)} decays for {self.H} heads")
+        self.dp, self.dvp = pad16(self.d), pad16(self.dv)
+        self.out_dim = self.H * self.dvp
+
+    def shapes(self):
+        H, d, dv, w = self.H, self.d, self.dv, self.width
+        return {"q": (H * d, w), "k": (H * d, w), "v": (H * dv, w), "g": (H * dv, w), "o": (w, H * dv), "norm": (H * dv,)}
+
+    def in_parts(self, get):
+        H, d, dv, W = self.H, self.d, self.dv, self.W
+        return [(n, pad_heads_rows(get(n), H, dd, W)) for n, dd in (("q", d), ("k", d), ("v", dv), ("g", dv))]
+
+    def out_part(self, get):
+        return pad_heads_cols(get("o"), self.H, self.dv, self.W)
+
+    def load(self, get, fin, vec, model):
+        self.norm = vec(pad_heads_vec(get("norm"), self.H, self.dv))
+        self.decay = vec(torch.tensor(self.decay_values, dtype=torch.float64))
+
+    def cache_shape(self, model):
+        return {"state": {"S": ((self.H, self.dp, self.dvp), torch.float32)}}
+
+    def run(self, model, h, proj, y, inp, cache):
+        ops = model.ops
+        o = ops.linear_attn(proj["q"], proj["k"], proj["v"], self.H, self.dp, self.dvp, self.decay, cache["S"], inp)
+        ops.norm_gate(o, self.out_dim, self.H * self.dv, self.norm, proj["g"], "sigmoid", model.eps, y)
+
+
+class WkvMixer(Mixer):
+    recurrent = True
+    STREAMS = ("r", "k", "v", "g", "w")
+
+    def __init__(self, params: dict, width: int):
+        super().__init__(params, width)
+        self.H, self.d = int(params["heads"]), int(params["dim"])
+        self.dp = pad16(self.d)
+        self.out_dim = self.H * self.dp
+        self.rank: Optional[int] = params.get("rank")      # of the decay's low-rank map; the checkpoint's own shape decides
+
+    def shapes(self):
+        hd, w, r = self.H * self.d, self.width, int(self.rank or max(16, self.width // 64))
+        out = {"mu." + s: (w,) for s in self.STREAMS}
+        out.update({s: (hd, w) for s in "rkvg"})
+        out.update({"w1": (r, w), "w2": (hd, r), "w0": (hd,), "u": (self.H, self.d), "norm": (hd,), "o": (w, hd)})
+        return out
+
+    def in_parts(self, get):
+        return []                                           # every projection reads a shifted mix of its own
+
+    def out_part(self, get):
+        return pad_heads_cols(get("o"), self.H, self.d, self.W)
+
+    def load(self, get, fin, vec, model):
+        H, d, W = self.H, self.d, self.W
+        self.mu = vec(torch.stack([_pad_to(get("mu." + s), W) for s in self.STREAMS]))
+        self.rkvg = fin(torch.stack([pad_heads_rows(get(s), H, d, W) for s in "rkvg"]))          # [4, H * dp, W]
+        w1, w2 = get("w1"), get("w2")
+        rp = pad16(w1.shape[0])
+        self.w1 = fin(_pad_to(w1, rp, W))
+        self.w2 = fin(pad_heads_rows(w2, H, d, rp))
+        self.w0 = vec(pad_heads_vec(get("w0"), H, d))
+        self.u = vec(pad_heads_vec(get("u"), H, d))
+        self.norm = vec(pad_heads_vec(get("norm"), H, d))
+
+    def cache_shape(self, model):
+        return {"state": {"S": ((self.H, self.dp, self.dp), torch.float32), "shift": ((self.W,), model.dtype)}}
+
+    def run(self, model, h, proj, y, inp, cache):
+        ops = model.ops
+        mix = ops.token_shift(h, self.mu, cache["shift"], inp)                 # [5, T, W]
+        r, k, v, g = ops.gemm_stack(mix[:4], self.rkvg)
+        z = ops.gemm(ops.tanh_(ops.gemm(mix[4], self.w1)), self.w2)
+        o = ops.wkv(r, k, v, z, self.w0, self.u, self.H, self.dp, cache["S"], inp)
+        ops.norm_gate(o, self.dp, self.d, self.norm, g, "silu", model.eps, y)
+
+
+class LatentAttentionMixer(Mixer):
+    def __init__(self, params: dict, width: int):
+        super().__init__(params, width)
+        p = params
+        self.H, self.d, self.rot, self.dv = int(p["heads"]), int(p["dim"]), int(p["rot_dim"]), int(p["vdim"])
+        self.q_rank, self.kv_rank, self.scale = int(p["q_rank"]), int(p["kv_rank"]), float(p["scale"])
+        self.rot_base = float(p["rot"]["base"])
+        if int(p["rot"].get("dims", self.rot)) != self.rot:
+            raise NotImplementedError("latent attention rotates the whole rotated key part")
+        self.dp, self.rp, self.dvp = pad16(self.d), pad16(self.rot), pad16(self.dv)
+        self.qrp, self.kvp, self.gp = pad16(self.q_rank), pad16(self.kv_rank), pad16(self.H)
+        self.out_dim = self.H * self.dvp
+
+    def shapes(self):
+        H, d, r, dv, w = self.H, self.d, self.rot, self.dv, self.width
+        return {"dq": (self.q_rank, w), "dq.norm": (self.q_rank,), "uq": (H * (d + r), self.q_rank), "dkv": (self.kv_rank + r, w),
+                "dkv.norm": (self.kv_rank,), "uk": (H * d, self.kv_rank), "uv": (H * dv, self.kv_rank), "g": (H, w), "o": (w, H * dv)}
+
+    def in_parts(self, get):
+        dkv, W = get("dkv"), self.W
+        dkv = torch.cat([_pad_to(dkv[: self.kv_rank], self.kvp, W), _pad_to(dkv[self.kv_rank:], self.rp, W)])
+        return [("dq", _pad_to(get("dq"), self.qrp, W)), ("dkv", dkv), ("g", _pad_to(get("g"), self.gp, W))]
+
+    def out_part(self, get):
+        return pad_heads_cols(get("o"), self.H, self.dv, self.W)
+
+    def load(self, get, fin, vec, model):
+        H, d, r, dv = self.H, self.d, self.rot, self.dv
+        uq = get("uq").view(H, d + r, self.q_rank)
+        self.uq = fin(torch.cat([_pad_to(uq[:, :d], H, self.dp, self.qrp), _pad_to(uq[:, d:], H, self.rp, self.qrp)], 1)
+                      .reshape(H * (self.dp + self.rp), self.qrp))
+        self.uk_t = fin(_pad_to(get("uk").view(H, d, self.kv_rank).transpose(1, 2), H, self.kvp, self.dp))     # [H, kv_rank, dim]
+        self.uv = fin(_pad_to(get("uv").view(H, dv, self.kv_rank), H, self.dvp, self.kvp))                     # [H, vdim, kv_rank]
+        self.dq_norm = vec(_pad_to(get("dq.norm"), self.qrp))
+        self.dkv_norm = vec(_pad_to(get("dkv.norm"), self.kvp))
+        self.cos_sin = model.rope_table(self.rot, self.rot_base)
+
+    def cache_shape(self, model):
+        return {"paged": self.kvp + self.rp}
+
+    def run(self, model, h, proj, y, inp, cache):
+        ops = model.ops
+        head = self.dp + self.rp
+        cq = ops.latent_prep(proj["dq"], proj["dkv"], self.dq_norm, self.dkv_norm, self.q_rank, self.kv_rank, self.rot, model.eps,
+                             self.cos_sin, inp.positions, inp.slots, cache)
+        q = ops.gemm(cq, self.uq)
+        ops.rope_pairs(q, inp.positions, self.cos_sin, self.H, head, self.dp, self.rot)
+        q_lat = torch.empty(q.shape[0], self.H * self.kvp, dtype=q.dtype, device=q.device)
+        ops.gemm_heads(q, self.uk_t, q_lat, head)
+        o_lat = ops.latent_attn(q_lat, q, cache, self.H, self.kvp, head, self.dp, self.rp, self.scale, inp)
+        ops.gemm_heads(o_lat, self.uv, y, self.kvp, gate=proj["g"])
+
+
+MIXERS = {"lightning": LightningMixer, "wkv": WkvMixer, "latent_attention": LatentAttentionMixer}
+
+
+def make_mixer(spec, width: int) -> Mixer:
+    cls = MIXERS.get(spec.mixer)
+    if cls is None:
+        raise NotImplementedError(f"no mixer {spec.mixer!r}; known: {sorted(MIXERS)}")
+    return cls(spec.params, width)
+
+
+@dataclass
+class MixerLayer:
+    """One layer: its norm, its mixer and the two fused projections."""
+    mixer: Mixer
+    ff: int                                                  # padded width of the feed-forward (0: none)
+    norm: Optional[torch.Tensor] = None                      # fp32 [W], stored around zero
+    in_w: Optional[torch.Tensor] = None                      # [rows, W]: the mixer's input projections, then gate and up
+    out_w: Optional[torch.Tensor] = None                     # [W, mixer out_dim + ff]
+    parts: Dict[str, Tuple[int, int]] = field(default_factory=dict)
+
+    def forward(self, model, residual, pending, inp, cache):
+        """residual (fp32) += pending; returns this layer's contribution, to be added by whoever norms the residual next."""
+        ops, m = model.ops, self.mixer
+        h = ops.norm_stream(residual, pending, self.norm, model.eps, model.config.norm_weight_offset, model.hidden, model.dtype)
+        T = h.shape[0]
+        proj = ops.gemm(h, self.in_w) if self.in_w is not None else None
+        views = {n: proj[:, a:b] for n, (a, b) in self.parts.items()}
+        y = torch.empty(T, m.out_dim + self.ff, dtype=h.dtype, device=h.device)
+        m.run(model, h, views, y, inp, cache)
+        if self.ff:
+            ops.act_mul(views["mlp"], self.ff, model.config.hidden_act, gated=True, out=y[:, m.out_dim:])
+        return ops.gemm(y, self.out_w)
+
+
+def load_mixer_layers(m, w):
+    """Tensors of a layer-by-layer checkpoint -> `m` (a DecoderModel): `embed`, `l<i>.norm1`, `l<i>.mix.*`, `l<i>.mlp.*`,
+    `final.norm`, `head`."""
+    c, dt, dev = m.config, m.dtype, m.device
+    if m.tp.world_size > 1:
+        raise ValueError(f"{c.model_type} is served on one shard")
+    W = pad16(c.hidden_size)
+
+    def get(name):
+        return w.get_tensor(name).float()
+
+    def fin(t):
+        return t.to(dt).to(dev).contiguous()
+
+    def vec(t):
+        return t.to(torch.float32).to(dev).contiguous()
+
+    m.embed = fin(_pad_to(get("embed"), c.vocab_size, W))
+    m.lm_head = fin(_pad_to(get("head"), pad16(c.vocab_size), W))
+    m.final_norm = vec(_pad_to(get("final.norm"), W))
+    m.layers = []
+    for i, spec in enumerate(c.layer_specs):
+        mx = make_mixer(spec, c.hidden_size)
+        ff = pad16(spec.ff) if spec.ff else 0
+        layer = MixerLayer(mx, ff, norm=vec(_pad_to(get(f"l{i}.norm1"), W)))
+        sub = lambda name, i=i: get(f"l{i}.mix.{name}")
+        rows = mx.in_parts(sub)
+        out = [mx.out_part(sub)]
+        if ff:
+            rows.append(("mlp", torch.cat([_pad_to(get(f"l{i}.mlp.{n}"), ff, W) for n in ("gate", "up")])))
+            out.append(_pad_to(get(f"l{i}.mlp.down"), W, ff))
+        o = 0
+        for name, t in rows:
+            layer.parts[name] = (o, o + t.shape[0])
+            o += t.shape[0]
+        layer.in_w = fin(torch.cat([t for _, t in rows])) if rows else None
+        layer.out_w = fin(torch.cat(out, 1))
+        mx.load(sub, fin, vec, m)
+        m.layers.append(layer)
+
+
+def tensor_shapes(c) -> Dict[str, Tuple[int, ...]]:
+    """Name -> shape of every tensor of a layer-by-layer checkpoint of this configuration."""
+    w = c.hidden_size
+    out = {"embed": (c.vocab_size, w), "head": (c.vocab_size, w), "final.norm": (w,)}
+    for i, spec in enumerate(c.layer_specs):
+        out[f"l{i}.norm1"] = (w,)
+        out.update({f"l{i}.mix.{n}": s for n, s in make_mixer(spec, w).shapes().items()})
+        if spec.ff:
+            out.update({f"l{i}.mlp.gate": (spec.ff, w), f"l{i}.mlp.up": (spec.ff, w), f"l{i}.mlp.down": (w, spec.ff)})
+    return out
+
+
+class RandomWeights:
+    """Random tensors of `tensor_shapes`, drawn one at a time on `device` when the loader asks for them (benchmarks, tests)."""
+    quant = None
+
+    def __init__(self, c, device="cpu", seed: int = 0):
+        self.shapes, self.device, self.seed = tensor_shapes(c), device, seed
+        self.order = {n: i for i, n in enumerate(self.shapes)}
+
+    def has_tensor(self, name):
+        return name in self.shapes
+
+    def get_tensor(self, name):
+        shape = self.shapes[name]
+        g = torch.Generator(device=self.device).manual_seed(self.seed * 100003 + self.order[name])
+        t = torch.randn(*shape, generator=g, device=self.device, dtype=torch.float32)
+        leaf = name.rsplit(".", 1)[-1]
+        if ".mu." in name:
+            return torch.sigmoid(t)
+        if name.endswith(("dq.norm", "dkv.norm", "mix.norm")):
+            return 1.0 + 0.1 * t
+        if leaf == "w0":
+            return -2.0 + 1.5 * t
+        if leaf in ("norm1", "norm"):
+            return 0.1 * t
+        if leaf == "u":
+            return 0.5 * t
+        return t if name == "embed" else t * shape[-1] ** -0.5

@@ -13,10 +13,11 @@ import torch
 from . import reference
 
 
-def get_ops(device, dtype=torch.bfloat16):
+def get_ops(device, dtype=torch.bfloat16, fp32: bool = False):
+    """`fp32`: the caller's operators also exist as 32-bit kernels (the layer-by-layer designs)."""
     device = torch.device(device)
     if device.type == "cuda":
-        if dtype != torch.bfloat16:
+        if dtype != torch.bfloat16 and not (fp32 and dtype == torch.float32):
             raise ValueError("the CUDA kernels are bf16; got %s" % dtype)
         from . import native
         native.load()

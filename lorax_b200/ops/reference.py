@@ -453,3 +453,181 @@ def rope_cache(rot: int, max_pos: int, theta: float, scaling: Optional[dict] = N
             mscale = 1.0 if sc <= 1 else math.sqrt(1 + math.log(sc) / math.log(orig))
     freqs = torch.outer(t, inv_freq)
     return torch.cat([freqs.cos() * mscale, freqs.sin() * mscale], dim=-1).to(device)
+
+
+# ------------------------------------------------------------------------------------------------
+# Layer-by-layer designs (models/mixers.py): fp32 residual stream, linear recurrences with per-request state, latent attention.
+# `inp` is the StepInputs of the step: rows [0, nd) are decode rows, the rows after them ragged prompt tokens.
+# ------------------------------------------------------------------------------------------------
+def rope_table(rot: int, max_pos: int, base: float, device="cpu") -> torch.Tensor:
+    """[max_pos, rot] fp32: cos of position * base^(-2i / rot) in the first half, sin in the second; angles formed in fp64."""
+    f = torch.pow(torch.tensor(float(base), dtype=torch.float64), -torch.arange(0, rot, 2, dtype=torch.float64) / rot)
+    a = torch.outer(torch.arange(max_pos, dtype=torch.float64), f)
+    return torch.cat([a.cos(), a.sin()], -1).float().to(device)
+
+
+def embed_stream(ids, table, mult=1.0):
+    return table[ids.long().clamp(0, table.shape[0] - 1)].float() * mult
+
+
+def norm_stream(residual, pending, weight, eps, weight_offset: float, n: int, dtype):
+    """residual (fp32, in place) += pending; returns its RMS norm (mean over the first `n` columns) in `dtype`."""
+    if pending is not None:
+        residual += pending.float()
+    y = residual * torch.rsqrt((residual * residual).sum(-1, keepdim=True) / n + eps)
+    return (y * (weight + weight_offset)).to(dtype)
+
+
+def norm_gate(x, group: int, n: int, weight, gate, act: str, eps, out):
+    """x [T, G * group] fp32: every group of columns divided by its root mean square (over `n` real columns), times `weight`
+    [G * group], times act(gate); written to `out` in its dtype."""
+    T, C = x.shape
+    g = x.view(T, C // group, group)
+    y = (g * torch.rsqrt((g * g).sum(-1, keepdim=True) / n + eps)).view(T, C) * weight
+    z = gate[:, :C].float()
+    y = y * (torch.sigmoid(z) if act == "sigmoid" else F.silu(z))
+    out[:, :C] = y.to(out.dtype)
+    return out
+
+
+def _sequences(inp, T: int):
+    """(first row, rows, state slot, tokens before the step) of every live sequence of the step."""
+    nd, _, slots, ctx = inp.decode_view(T)
+    out = [(i, 1, int(slots[i]), int(ctx[i]) - 1) for i in range(nd) if int(ctx[i]) > 0]
+    if inp.is_prefill:
+        cu = [int(c) for c in inp.cu_q]
+        out += [(nd + cu[b], cu[b + 1] - cu[b], int(inp.state_slots[b]), int(inp.cache_lens[b])) for b in range(len(cu) - 1)
+                if cu[b + 1] > cu[b]]
+    return out
+
+
+def linear_attn(q, k, v, H: int, d: int, dv: int, decay, state, inp):
+    """Linear attention with one decay per head over silu(q), silu(k), silu(v) (row-strided views [T, H * d / dv]):
+    S <- decay S + k v^T, o = S^T q.  `state` [slots, H, d, dv] fp32 is read and updated.  -> o [T, H * dv] fp32."""
+    T = q.shape[0]
+    qf, kf = F.silu(q.float()).view(T, H, d), F.silu(k.float()).view(T, H, d)
+    vf = F.silu(v.float()).view(T, H, dv)
+    if q.dtype != torch.float32:
+        qf, kf, vf = (x.to(q.dtype).float() for x in (qf, kf, vf))
+    out = torch.zeros(T, H * dv, dtype=torch.float32, device=q.device)
+    for r0, n, slot, before in _sequences(inp, T):
+        S = state[slot].clone() if before > 0 else torch.zeros_like(state[slot])
+        for t in range(r0, r0 + n):
+            S = decay[:, None, None] * S + kf[t][:, :, None] * vf[t][:, None, :]
+            out[t] = torch.einsum("hij,hi->hj", S, qf[t]).reshape(-1)
+        state[slot] = S
+    return out
+
+
+def token_shift(h, mu, shift, inp):
+    """Interpolation with the previous token's input: row s of the result [n, T, W] is h + (h' - h) * mu[s]; h' of a sequence's
+    first token comes from `shift` [slots, W] (zeros at position 0), which then takes the sequence's last row."""
+    T = h.shape[0]
+    prev = torch.zeros_like(h)
+    last = []
+    for r0, n, slot, before in _sequences(inp, T):
+        prev[r0 + 1: r0 + n] = h[r0: r0 + n - 1]
+        if before > 0:
+            prev[r0] = shift[slot]
+        last.append((slot, r0 + n - 1))
+    for slot, r in last:
+        shift[slot] = h[r]
+    hf, pf = h.float(), prev.float()
+    return torch.stack([(hf + (pf - hf) * mu[s]).to(h.dtype) for s in range(mu.shape[0])])
+
+
+def gemm_stack(x, w):
+    """x [n, T, K], w [n, N, K] -> [n, T, N]: one product per stacked pair."""
+    return torch.stack([gemm(x[i], w[i]) for i in range(w.shape[0])])
+
+
+def tanh_(x):
+    x.copy_(torch.tanh(x.float()).to(x.dtype))
+    return x
+
+
+def wkv(r, k, v, z, w0, u, H: int, d: int, state, inp):
+    """WKV recurrence with data-dependent decay w = exp(-exp(z + w0)) per key channel and a bonus u for the current token:
+    o = (S + diag(u) k v^T)^T r, then S <- diag(w) S + k v^T.  -> o [T, H * d] fp32; `state` [slots, H, d, d] is updated."""
+    T = r.shape[0]
+    rf, kf, vf = (x.float().reshape(T, H, d) for x in (r, k, v))
+    w = torch.exp(-torch.exp(z.float() + w0)).view(T, H, d)
+    out = torch.zeros(T, H * d, dtype=torch.float32, device=r.device)
+    for r0, n, slot, before in _sequences(inp, T):
+        S = state[slot].clone() if before > 0 else torch.zeros_like(state[slot])
+        for t in range(r0, r0 + n):
+            kv = kf[t][:, :, None] * vf[t][:, None, :]
+            out[t] = torch.einsum("hij,hi->hj", S + u.view(H, d)[:, :, None] * kv, rf[t]).reshape(-1)
+            S = w[t][:, :, None] * S + kv
+        state[slot] = S
+    return out
+
+
+def _rotate_pairs(x, cos, sin):
+    """x [..., rot] with interleaved pairs; cos / sin broadcastable [..., rot / 2]."""
+    u, v = x[..., 0::2].float(), x[..., 1::2].float()
+    return torch.stack([u * cos - v * sin, v * cos + u * sin], -1).flatten(-2)
+
+
+def latent_prep(dq, dkv, dq_norm, dkv_norm, q_rank: int, kv_rank: int, rot: int, eps, cos_sin, positions, slots, cache):
+    """Down-projections of latent attention -> normalised query latent [T, q_rank padded] (returned) and cache rows
+    [normalised key/value latent | rotated key part] (scattered into `cache` [blocks, page, kv_rank padded + rot padded])."""
+    dt = dq.dtype
+    qr, kr = dq_norm.shape[0], dkv_norm.shape[0]
+    page = cache.shape[1]
+
+    def rms(x, n, w):
+        x = x.float()
+        return (x * torch.rsqrt((x * x).sum(-1, keepdim=True) / n + eps) * w).to(dt)
+    cq = rms(dq[:, :qr], q_rank, dq_norm)
+    row = torch.zeros(dq.shape[0], cache.shape[2], dtype=dt, device=dq.device)
+    row[:, :kr] = rms(dkv[:, :kr], kv_rank, dkv_norm)
+    cs = cos_sin[positions.long()]
+    row[:, kr: kr + rot] = _rotate_pairs(dkv[:, kr: kr + rot], cs[:, : rot // 2], cs[:, rot // 2:]).to(dt)
+    ok = slots >= 0
+    s = slots[ok].long()
+    cache[s // page, s % page] = row[ok]
+    return cq
+
+
+def rope_pairs(x, positions, cos_sin, H: int, head: int, off: int, rot: int):
+    """Rotates columns [off, off + rot) of every head (width `head`) of x [T, H * head] in place, interleaved pairs."""
+    T = x.shape[0]
+    cs = cos_sin[positions.long()]
+    part = x.view(T, H, head)[:, :, off: off + rot]
+    part.copy_(_rotate_pairs(part, cs[:, None, : rot // 2], cs[:, None, rot // 2:]).to(x.dtype))
+
+
+def gemm_heads(x, w, out, x_head: int, gate=None):
+    """Per-head products: head h of `out` (width N) = columns [h * x_head, h * x_head + K) of x times w[h]^T (w [H, N, K]),
+    optionally times sigmoid(gate[:, h])."""
+    H, N, K = w.shape
+    T = x.shape[0]
+    xs = torch.stack([x[:, h * x_head: h * x_head + K] for h in range(H)], 1).float()
+    y = torch.einsum("thk,hnk->thn", xs, w.float())
+    if gate is not None:
+        y = y * torch.sigmoid(gate[:, :H].float())[:, :, None]
+    out[:, : H * N] = y.reshape(T, H * N).to(out.dtype)
+    return out
+
+
+def latent_attn(q_lat, q, cache, H: int, kv_rank: int, head: int, rot_off: int, rot: int, scale: float, inp, w_uk=None, w_uv=None):
+    """Causal softmax attention in the latent space: head h's query is [q_lat[h] | q[h, rot_off : rot_off + rot]] against the
+    cached rows [latent | rotated key].  -> weighted latents [T, H * kv_rank]."""
+    T = q.shape[0]
+    page = cache.shape[1]
+    nd, dbt, _, ctx = inp.decode_view(T)
+    ql, qr = q_lat.view(T, H, kv_rank).float(), q.view(T, H, head)[:, :, rot_off: rot_off + rot].float()
+    out = torch.zeros(T, H, kv_rank, dtype=q.dtype, device=q.device)
+    spans = [(i, 1, dbt[i], int(ctx[i]) - 1) for i in range(nd) if int(ctx[i]) > 0]
+    if inp.is_prefill:
+        cu = [int(c) for c in inp.cu_q]
+        spans += [(nd + cu[b], cu[b + 1] - cu[b], inp.block_tables[b], int(inp.cache_lens[b])) for b in range(len(cu) - 1) if cu[b + 1] > cu[b]]
+    for r0, n, bt, before in spans:
+        keys = before + n
+        rows = cache[bt[: (keys + page - 1) // page].long()].reshape(-1, cache.shape[2])[:keys].float()
+        s = torch.einsum("thc,sc->hts", ql[r0: r0 + n], rows[:, :kv_rank]) + torch.einsum("thc,sc->hts", qr[r0: r0 + n], rows[:, kv_rank: kv_rank + rot])
+        pos = torch.arange(before, keys, device=q.device)
+        s = (s * scale).masked_fill(torch.arange(keys, device=q.device)[None, None, :] > pos[None, :, None], float("-inf"))
+        out[r0: r0 + n] = torch.einsum("hts,sc->thc", torch.softmax(s, -1), rows[:, :kv_rank]).to(q.dtype)
+    return out.view(T, H * kv_rank)

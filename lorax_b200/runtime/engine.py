@@ -29,7 +29,7 @@ from ..sampling.chooser import (FINISH_EOS, FINISH_LENGTH, FINISH_STOP, Heteroge
                                 StoppingCriteria)
 from ..sampling.device import RowSampler, has_penalties, needs_device_step, tp_eligible
 from ..sampling.device import supported as device_sampling_supported
-from .kv_cache import BlockAllocator, KVCache
+from .kv_cache import BlockAllocator, make_cache
 from .runner import ModelRunner, PrefillItem
 
 
@@ -63,6 +63,7 @@ class _Seq:
     req: GenRequest
     blocks: List[int]
     row: int = -1
+    state_slot: int = 0
     output_ids: List[int] = field(default_factory=list)
     launched: int = 0                    # tokens whose computation has been launched (incl. the prefill token)
     finished: bool = False
@@ -82,8 +83,7 @@ class Engine:
         self._max_batch = max_batch
         if num_blocks is None:
             num_blocks = self._auto_blocks(page)
-        from .kv_cache import kv_dtype_of
-        self.kv = KVCache(c.num_hidden_layers, num_blocks, model.nkv, model.d, kv_dtype_of(model, self.cfg), model.device, page)
+        self.kv = make_cache(model, self.cfg, num_blocks, max_batch, page)
         self.alloc = BlockAllocator(num_blocks, page, c.sliding_window)
         self.runner = ModelRunner(model, self.kv, max_batch=max_batch, max_seq_tokens=self.cfg.max_total_tokens,
                                   max_prefill_tokens=self.cfg.max_batch_prefill_tokens,
@@ -107,8 +107,7 @@ class Engine:
         self.mixed_steps = os.environ.get("LORAX_MIXED_STEPS", "1") != "0"   # prefills ride along with the decode batch
 
     def _auto_blocks(self, page: int) -> int:
-        m, c = self.model, self.model.config
-        per_block = KVCache.bytes_per_block(c.num_hidden_layers, m.nkv, m.d, m.dtype, page)
+        m = self.model
         if m.device.type == "cuda":
             from .kv_cache import plan_kv_blocks
             return plan_kv_blocks(m, self.cfg, self._max_batch, page, reserve_bytes=2 << 30)
@@ -231,9 +230,14 @@ class Engine:
             if not self._adapter_ready(req.adapter_index):
                 skipped.append(self.waiting.popleft())
                 continue
+            slots = self.kv.state_slots
+            if slots is not None and not slots.free:
+                break
             blocks = self.alloc.allocate(n + req.max_new_tokens + 1)
             if blocks is None:
                 break
+            if slots is not None:
+                slots.acquire(req.request_id)
             self.waiting.popleft()
             picked.append((req, blocks))
             self._picking.add(req.adapter_index)
@@ -241,6 +245,10 @@ class Engine:
         for r in reversed(skipped):
             self.waiting.appendleft(r)
         return picked
+
+    def _state_slot(self, req: GenRequest) -> int:
+        slots = self.kv.state_slots
+        return slots.acquire(req.request_id) if slots is not None else 0
 
     def _finish(self, seq: _Seq, reason: int):
         seq.finished = True
@@ -250,6 +258,8 @@ class Engine:
         if seq.row >= 0:
             self.runner.state.drop_row(seq.row)
         self.alloc.release(seq.blocks)
+        if self.kv.state_slots is not None:
+            self.kv.state_slots.release(seq.req.request_id)
         self.running.pop(seq.req.request_id, None)
         self.draining.pop(seq.req.request_id, None)
         self.finished[seq.req.request_id] = seq
@@ -274,23 +284,25 @@ class Engine:
         """Give freshly prefilled requests their decode rows.  The first tokens stay on the device: they are scattered
         into the rows there and reach the host through the pinned ring like every later token, so the host never waits
         for a prefill to finish."""
-        rows, sel, poss, blks, ads, rids = [], [], [], [], [], []
+        rows, sel, poss, blks, ads, sts, rids = [], [], [], [], [], [], []
         for i, (req, blocks) in enumerate(picked):
             seq = _Seq(req, blocks, stopping=StoppingCriteria(req.max_new_tokens, req.eos_token_ids, list(req.stop_sequences),
                                                               req.ignore_eos_token))
             seq.launched = 1
+            seq.state_slot = self._state_slot(req)
             rids.append(req.request_id)
             if req.max_new_tokens > 1:
                 seq.row = self.runner.state.take_row(req.request_id)
                 self.running[req.request_id] = seq
                 rows.append(seq.row); sel.append(i); poss.append(len(req.prompt_ids)); blks.append(blocks)
                 ads.append(req.adapter_index)
+                sts.append(seq.state_slot)
             else:                       # only the prefill token is wanted: no decode row
                 seq.retired = True
                 self.draining[req.request_id] = seq
         if rows:
             first = next_ids if len(sel) == len(picked) else next_ids[torch.tensor(sel, device=next_ids.device)]
-            self.runner.install(rows, first, poss, blks, ads)
+            self.runner.install(rows, first, poss, blks, ads, sts)
         mapping = self.runner.resort()
         for s_ in list(self.running.values()) + list(self.draining.values()):
             if s_.row in mapping:
@@ -370,7 +382,7 @@ class Engine:
         picked = self._select_prefill()
         launched = False
         if picked:
-            items = [PrefillItem(r.prompt_ids, 0, b, r.adapter_index) for r, b in picked]
+            items = [PrefillItem(r.prompt_ids, 0, b, r.adapter_index, state_slot=self._state_slot(r)) for r, b in picked]
             snapshot = {s.row: rid for rid, s in self.running.items() if not s.retired}
             sampling = any(needs_device_step(r.params) for r, _ in picked) or any(needs_device_step(s.req.params) for s in self.running.values())
             if self.mixed_steps and snapshot and self.runner.can_mix() and not sampling:

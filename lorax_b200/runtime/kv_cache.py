@@ -12,7 +12,7 @@ needs more than ceil(window / PAGE) + 1 blocks per request because old pages are
 
 from __future__ import annotations
 
-from typing import List, Optional
+from typing import Dict, List, Optional
 
 import torch
 
@@ -45,9 +45,86 @@ class KVCache:
     def bytes_per_block(num_layers: int, kv_heads: int, head_dim: int, dtype, page: int = PAGE_SIZE) -> int:
         return num_layers * kv_heads * 2 * page * head_dim * torch.empty(0, dtype=dtype).element_size()
 
+    state_slots: Optional["StateSlots"] = None       # the layers of a uniform cache keep nothing per request
+
     @property
     def max_tokens(self) -> int:
         return (self.num_blocks - 1) * self.page
+
+
+class StateSlots:
+    """Slots of the per-request state (recurrent layers), one per live request.  Slot 0 belongs to no request (health probes run
+    in it).  Nothing is cleared when a slot changes hands: a request's first tokens start from zeros by position."""
+
+    def __init__(self, num_slots: int):
+        self.num_slots = num_slots
+        self.free: List[int] = list(range(num_slots - 1, 0, -1))
+        self.of_request: Dict[int, int] = {}
+
+    def acquire(self, request_id) -> Optional[int]:
+        """The request's slot, taken now if it has none; None when all are in use."""
+        slot = self.of_request.get(request_id)
+        if slot is None and self.free:
+            slot = self.of_request[request_id] = self.free.pop()
+        return slot
+
+    def release(self, request_id):
+        slot = self.of_request.pop(request_id, None)
+        if slot is not None:
+            self.free.append(slot)
+
+
+class LayeredCache:
+    """Cache of a model whose layer runs keep different things (`DecoderModel.cache_shapes`): a run's entry in `layers` is either a
+    paged tensor [num_blocks, page, width] in the model's dtype, addressed by the requests' block tables like a key/value cache, or a
+    dict of state tensors [slots, ...], addressed by the requests' state slot."""
+
+    def __init__(self, shapes: List[dict], num_blocks: int, num_slots: int, dtype, device, page: int = PAGE_SIZE):
+        self.page = page
+        self.num_blocks = num_blocks
+        self.layers: List[object] = []
+        for sh in shapes:
+            if "paged" in sh:
+                self.layers.append(torch.zeros(num_blocks, page, sh["paged"], dtype=dtype, device=device))
+            else:
+                self.layers.append({n: torch.zeros(num_slots, *dims, dtype=dt, device=device) for n, (dims, dt) in sh["state"].items()})
+        self.state_slots = StateSlots(num_slots) if any("state" in sh for sh in shapes) else None
+
+    @property
+    def max_tokens(self) -> int:
+        return (self.num_blocks - 1) * self.page
+
+
+def num_state_slots(max_batch: int) -> int:
+    """Running requests, a few whose prompts are still arriving in portions, and the reserved slot."""
+    return max_batch + max(4, max_batch // 8) + 1
+
+
+def make_cache(model, cfg, num_blocks: int, max_batch: int, page: int = PAGE_SIZE, num_slots: Optional[int] = None):
+    """The cache a model's layers ask for."""
+    shapes = model.cache_shapes()
+    if shapes is None:
+        return KVCache(model.config.num_hidden_layers, num_blocks, model.nkv, model.d, kv_dtype_of(model, cfg), model.device, page)
+    if getattr(cfg, "kv_cache_dtype", None) not in (None, "", "auto"):
+        raise ValueError(f"{model.config.model_type} keeps its cache in the model's dtype (kv_cache_dtype {cfg.kv_cache_dtype!r})")
+    return LayeredCache(shapes, num_blocks, num_slots or num_state_slots(max_batch), model.dtype, model.device, page)
+
+
+def cache_bytes(model, cfg, max_batch: int, page: int = PAGE_SIZE):
+    """(bytes per block, bytes that do not grow with the blocks) of a model's cache."""
+    shapes = model.cache_shapes()
+    if shapes is None:
+        return KVCache.bytes_per_block(model.config.num_hidden_layers, model.nkv, model.d, kv_dtype_of(model, cfg), page), 0
+    size = lambda dt: torch.empty(0, dtype=dt).element_size()
+    paged = sum(sh["paged"] for sh in shapes if "paged" in sh) * page * size(model.dtype)
+    fixed = 0
+    for sh in shapes:
+        for dims, dt in sh.get("state", {}).values():
+            n = size(dt) * num_state_slots(max_batch)
+            for x in dims:
+                n *= x
+            fixed += n
+    return paged, fixed
 
 
 class BlockAllocator:
@@ -70,6 +147,15 @@ class BlockAllocator:
         del self.free[-n:]
         return out
 
+    def extend(self, blocks: List[int], tokens: int) -> bool:
+        """Grow a request's blocks in place until they hold `tokens` tokens; False (nothing taken) when they do not fit."""
+        n = self.blocks_needed(tokens) - len(blocks)
+        if n > len(self.free):
+            return False
+        for _ in range(n):
+            blocks.append(self.free.pop())
+        return True
+
     def release(self, blocks: List[int]):
         self.free.extend(reversed(blocks))
 
@@ -86,8 +172,7 @@ def plan_kv_blocks(model, cfg, max_batch: int, page: int = PAGE_SIZE, reserve_by
     the same time (the prefill contains collectives) and the ranks agree on the minimum."""
     from .runner import ModelRunner, PrefillItem
     c, dev = model.config, model.device
-    kv_dtype = kv_dtype_of(model, cfg)
-    per_block = KVCache.bytes_per_block(c.num_hidden_layers, model.nkv, model.d, kv_dtype, page)
+    per_block, fixed = cache_bytes(model, cfg, max_batch, page)
     if dev.type != "cuda":
         return 1024
     tokens = max(int(cfg.max_batch_prefill_tokens), 16)
@@ -95,14 +180,14 @@ def plan_kv_blocks(model, cfg, max_batch: int, page: int = PAGE_SIZE, reserve_by
     lens = [seq] * (tokens // seq) + ([tokens % seq] if tokens % seq else [])
     window = c.sliding_window
     blocks_per = [min((n + page - 1) // page, (window + page - 1) // page + 1) if window else (n + page - 1) // page for n in lens]
-    tmp = KVCache(c.num_hidden_layers, sum(blocks_per) + 2, model.nkv, model.d, kv_dtype, dev, page)
+    tmp = make_cache(model, cfg, sum(blocks_per) + 2, max_batch, page, num_slots=len(lens) + 2)
     runner = ModelRunner(model, tmp, max_batch=max_batch, max_seq_tokens=cfg.max_total_tokens, max_prefill_tokens=tokens, use_graphs=False)
     torch.cuda.synchronize(dev)
     torch.cuda.reset_peak_memory_stats(dev)
     base = torch.cuda.memory_allocated(dev)
     items, nxt = [], 1
     for n, nb in zip(lens, blocks_per):
-        items.append(PrefillItem([1] * n, 0, list(range(nxt, nxt + nb))))
+        items.append(PrefillItem([1] * n, 0, list(range(nxt, nxt + nb)), state_slot=len(items) + 1))
         nxt += nb
     runner.prefill(items)
     torch.cuda.synchronize(dev)
@@ -110,8 +195,11 @@ def plan_kv_blocks(model, cfg, max_batch: int, page: int = PAGE_SIZE, reserve_by
     del runner, tmp, items
     torch.cuda.empty_cache()
     free, _ = torch.cuda.mem_get_info(dev)
-    budget = int(free * cfg.memory_wiggle_room) - int(peak * 1.1) - reserve_bytes
-    blocks = max(int(budget // per_block), 64)
+    budget = int(free * cfg.memory_wiggle_room) - int(peak * 1.1) - reserve_bytes - fixed
+    if budget <= 0 and fixed:
+        raise ValueError(f"the state of {max_batch} requests ({fixed >> 20} MiB) does not fit: lower the maximum batch size")
+    most = max_batch * ((cfg.max_total_tokens + page - 1) // page + 1) + 1       # no step can address more
+    blocks = max(int(budget // per_block), 64) if per_block else most
     tp = model.tp
     if tp.world_size > 1:
         import torch.distributed as dist

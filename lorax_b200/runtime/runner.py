@@ -44,6 +44,8 @@ class PrefillItem:
     # of the embedding of their (placeholder) token id
     embed_index: Optional[Sequence[int]] = None
     embeds: Optional[torch.Tensor] = None
+    state_slot: int = 0             # slot of the request's recurrent state (models that have one; `KVCache.state_slots`)
+    logit_rows: Optional[Sequence[int]] = None      # score these places of the chunk instead of its last token
 
 
 class DecodeState:
@@ -56,6 +58,7 @@ class DecodeState:
         self.slots = torch.full((max_batch,), -1, **i32)
         self.block_tables = torch.zeros(max_batch, max_blocks, **i32)
         self.tok_slot = torch.full((max_batch,), -1, **i32)
+        self.state_slots = torch.zeros(max_batch, **i32)       # slot of the row's recurrent state
         self.next_ids = torch.zeros(max_batch, **i32)
         self.logprobs = torch.zeros(max_batch, dtype=torch.float32, device=device)
         # LoRA tile table of the decode batch (rows are kept sorted by adapter slot): [max_batch, 4], unused = slot -1
@@ -128,6 +131,8 @@ class ModelRunner:
         self.h2d_bytes = 0
         self.d2h_bytes = 0
         self.graph_kernels: Dict[Tuple[int, bool], int] = {}
+        self.keep_logits = False                             # callers that read the logits of mixed steps
+        self.last_logits: Optional[torch.Tensor] = None      # of the last mixed step (decode rows, then the prefill's scored rows)
         self.tiles_valid = False
         self.replayed_launches = 0
 
@@ -177,6 +182,7 @@ class ModelRunner:
         cache_lens, tables, head_idx, head_slot, q_lens, seq_slot = [], [], [], [], [], []
         tl: List[Tuple[int, int, int, int]] = list(lead_tiles)
         any_lora = False
+        state_slots: List[int] = []
         over_rows: List[int] = []
         over_vals: List[torch.Tensor] = []
         for it in items:
@@ -193,11 +199,15 @@ class ModelRunner:
             tables.append(self._table_row(it.blocks))
             q_lens.append(n)
             seq_slot.append(slot_id)
+            state_slots.append(it.state_slot)
             if slot_id >= 0:
                 # rows of one adapter in tiles of at most 32 (a run that continues the previous sequence's adapter starts a new tile)
                 tl += [(slot_id, base + a + row_offset, min(32, n - a), 0) for a in range(0, n, 32)]
             if it.want_logits:
-                if it.all_logprobs:
+                if it.logit_rows is not None:
+                    head_idx += [base + int(r) for r in it.logit_rows]
+                    head_slot += [slot_id] * len(it.logit_rows)
+                elif it.all_logprobs:
                     head_idx += list(range(base, base + n))
                     head_slot += [slot_id] * n
                 else:
@@ -209,9 +219,15 @@ class ModelRunner:
         ts, tq = reference.prefill_tiles(q_lens)
         if not any_lora:
             tl = list(lead_tiles)
+        seg_len, sgs, sgq = 0, [], []
+        if self.model.recurrent:
+            # the recurrence kernels carry the state through segments of this many tokens: long enough that the states between
+            # segments stay a small part of the traffic, short enough that a lone prompt fills the GPU
+            seg_len = min(512, max(64, (T // 16 + 63) // 64 * 64))
+            sgs, sgq = reference.prefill_tiles(q_lens, seg_len)
         i32 = lambda v: np.asarray(v, dtype=np.int32).reshape(-1)
         segs = [np.concatenate(id_parts) if id_parts else i32([]), i32(cu), i32(cache_lens), i32(seq_slot), i32(ts), i32(tq), i32(head_idx),
-                i32(head_slot), i32(tl), i32(tables)]
+                i32(head_slot), i32(tl), i32(tables), i32(state_slots), i32(sgs), i32(sgq)]
         flat = torch.from_numpy(np.concatenate(segs))
         if self.is_cuda:
             flat = flat.pin_memory().to(self.device, non_blocking=True)
@@ -220,7 +236,7 @@ class ModelRunner:
         for sgm in segs:
             views.append(flat[o:o + sgm.shape[0]])
             o += sgm.shape[0]
-        d_ids, d_cu, d_cl, d_seqslot, d_ts, d_tq, d_head, d_headslot, d_tiles, d_bt = views
+        d_ids, d_cu, d_cl, d_seqslot, d_ts, d_tq, d_head, d_headslot, d_tiles, d_bt, d_state, d_sgs, d_sgq = views
         bt = d_bt.view(len(items), self.max_blocks)
         d_pos, d_slots, d_tokslot = self.model.ops.prefill_metadata(d_cu, d_cl, d_seqslot, bt, page, T)
         if any_lora and self.model.adapters is not None:
@@ -229,7 +245,8 @@ class ModelRunner:
         inp = StepInputs(input_ids=d_ids, positions=d_pos, slots=d_slots, is_prefill=True, block_tables=bt, cu_q=d_cu,
                          cache_lens=d_cl, tile_seq=d_ts, tile_q0=d_tq, lm_head_indices=d_head if len(head_idx) else d_ids[:0],
                          tok_slot=d_tokslot if any_lora else None, head_tok_slot=d_headslot if any_lora else None,
-                         lora_tiles=tiles)
+                         lora_tiles=tiles, state_slots=d_state, seg_seq=d_sgs, seg_q0=d_sgq, seg_len=seg_len,
+                         max_ctx=max([c + n for c, n in zip(cache_lens, q_lens)] + [0]))
         if over_rows:
             inp.embed_rows = torch.tensor(over_rows, dtype=torch.long, device=self.model.device)
             inp.embed_values = torch.cat(over_vals, 0).to(self.model.dtype).to(self.model.device)
@@ -292,8 +309,10 @@ class ModelRunner:
                          cache_lens=pin.cache_lens, tile_seq=pin.tile_seq, tile_q0=pin.tile_q0, lm_head_indices=head,
                          tok_slot=tok_slot, head_tok_slot=head_slot, lora_tiles=tiles, attn_nsplit=nsplit, n_decode=nd,
                          dec_block_tables=st.block_tables[:nd], ctx_lens=st.ctx_lens[:nd], embed_rows=pin.embed_rows,
-                         embed_values=pin.embed_values)
+                         embed_values=pin.embed_values, state_slots=pin.state_slots, dec_state_slots=st.state_slots[:nd],
+                         seg_seq=pin.seg_seq, seg_q0=pin.seg_q0, seg_len=pin.seg_len, max_ctx=pin.max_ctx)
         logits = self.model.forward(inp, self.kv.layers)
+        self.last_logits = self._cap(logits) if self.keep_logits else None
         ids, lps = self.model.ops.argmax_logprob(logits, softcap=self.model.config.final_logit_softcapping or 0.0)
         st.next_ids[:nd].copy_(ids[:nd])
         st.logprobs[:nd].copy_(lps[:nd])
@@ -304,8 +323,8 @@ class ModelRunner:
 
     # ------------------------------------------------------------------ decode rows
     def install(self, rows: Sequence[int], first_tokens, positions: Sequence[int], blocks: Sequence[Sequence[int]],
-                adapter_indices: Sequence[int]):
-        """Write freshly prefilled sequences into their decode rows (one packed H2D + six scatters).  `first_tokens` is a
+                adapter_indices: Sequence[int], state_slots: Optional[Sequence[int]] = None):
+        """Write freshly prefilled sequences into their decode rows (one packed H2D + seven scatters).  `first_tokens` is a
         host list or the device tensor the prefill's argmax left behind (the host then never waits for the prefill)."""
         if not rows:
             return
@@ -319,7 +338,8 @@ class ModelRunner:
         ctx = [p + 1 for p in positions]
         tslot = [self._slot_of(a) for a in adapter_indices]
         n = len(rows)
-        flat = list(rows) + list(first_tokens) + list(positions) + ctx + slots + tslot + [x for t in tabs for x in t]
+        sslot = list(state_slots) if state_slots is not None else [0] * n
+        flat = list(rows) + list(first_tokens) + list(positions) + ctx + slots + tslot + sslot + [x for t in tabs for x in t]
         dev = self._to_dev(flat)
         r = dev[:n].long()
         st.input_ids.index_copy_(0, r, dev[n:2 * n] if dev_first is None else dev_first.to(torch.int32))
@@ -327,7 +347,8 @@ class ModelRunner:
         st.ctx_lens.index_copy_(0, r, dev[3 * n:4 * n])
         st.slots.index_copy_(0, r, dev[4 * n:5 * n])
         st.tok_slot.index_copy_(0, r, dev[5 * n:6 * n])
-        st.block_tables.index_copy_(0, r, dev[6 * n:].view(n, self.max_blocks))
+        st.state_slots.index_copy_(0, r, dev[6 * n:7 * n])
+        st.block_tables.index_copy_(0, r, dev[7 * n:].view(n, self.max_blocks))
         for row, sl in zip(rows, tslot):
             st.row_slot[row] = sl
         self.tiles_valid = False        # rows are no longer grouped by adapter until resort() runs
@@ -342,7 +363,7 @@ class ModelRunner:
         mapping = {old: new for new, old in enumerate(old_rows)}
         if n and any(o != nw for o, nw in mapping.items()):
             perm = self._to_dev(old_rows).long()
-            for t in (st.input_ids, st.positions, st.ctx_lens, st.slots, st.tok_slot, st.block_tables):
+            for t in (st.input_ids, st.positions, st.ctx_lens, st.slots, st.tok_slot, st.state_slots, st.block_tables):
                 t[:n] = t.index_select(0, perm)
         hw = st.high_water
         if hw > n:
@@ -412,7 +433,8 @@ class ModelRunner:
                       and not (self.model.config.final_logit_softcapping or 0.0))
         inp = StepInputs(input_ids=st.input_ids[:b], positions=st.positions[:b], slots=st.slots[:b], is_prefill=False,
                          block_tables=st.block_tables[:b], ctx_lens=st.ctx_lens[:b], tok_slot=st.tok_slot[:b] if lora else None,
-                         head_tok_slot=st.tok_slot[:b] if lora else None, attn_nsplit=nsplit, lora_tiles=tiles, local_logits=fused_head)
+                         head_tok_slot=st.tok_slot[:b] if lora else None, attn_nsplit=nsplit, lora_tiles=tiles, local_logits=fused_head,
+                         state_slots=st.state_slots[:b])
         logits = self.model.forward(inp, self.kv.layers)
         if fused_head:
             # vocabulary-parallel greedy head: 16 bytes per row and rank cross NVLink instead of the logits
@@ -438,6 +460,8 @@ class ModelRunner:
             return
         # warm up outside capture (lazy cudaFuncSetAttribute calls, workspace allocation)
         saved = [t.clone() for t in (self.state.input_ids, self.state.positions, self.state.ctx_lens, self.state.slots)]
+        if self.model.recurrent:
+            self.state.ctx_lens[:b] = 0          # the warm-up must not advance the state of live requests: every row is padding
         self._decode_body(b, lora, need_logits)
         torch.cuda.synchronize(self.device)
         g = torch.cuda.CUDAGraph()

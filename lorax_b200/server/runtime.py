@@ -28,7 +28,7 @@ from ..adapters.merges import merge_adapters
 from ..config import EngineConfig, ModelConfig
 from ..models.decoder import DecoderModel
 from ..parallel.tp import TensorParallel
-from ..runtime.kv_cache import KVCache
+from ..runtime.kv_cache import make_cache
 from ..runtime.runner import ModelRunner, PrefillItem
 from ..sampling.chooser import (FINISH_EOS, FINISH_LENGTH, FINISH_STOP, HeterogeneousNextTokenChooser, NextTokenParams, ngram_speculate,
                                 StoppingCriteria)
@@ -92,6 +92,8 @@ class ShardRuntime:
         self.tp = model.tp
         c = model.config
         dev = model.device
+        if adapter_arena_bytes is None and model.mixed:
+            adapter_arena_bytes = 0                          # its projections take no adapters
         if adapter_arena_bytes is None:
             if dev.type == "cuda":
                 total = torch.cuda.get_device_properties(dev).total_memory
@@ -107,8 +109,10 @@ class ShardRuntime:
                 num_blocks = plan_kv_blocks(model, self.cfg, max_batch, page)      # a maximum prefill runs first: its peak is measured
             else:
                 num_blocks = 1024
-        from ..runtime.kv_cache import kv_dtype_of
-        self.kv = KVCache(c.num_hidden_layers, num_blocks, model.nkv, model.d, kv_dtype_of(model, self.cfg), dev, page)
+        self.kv = make_cache(model, self.cfg, num_blocks, max_batch, page)
+        if model.recurrent and (self.cfg.prefix_caching or self.cfg.speculative_tokens > 0):
+            raise ValueError(f"{c.model_type} carries a recurrent state: a cached prefix has none to go on from and a rejected guess cannot be "
+                             "taken back, so --prefix-caching and --speculative-tokens are not available")
         self.runner = ModelRunner(model, self.kv, max_batch=max_batch, max_seq_tokens=self.cfg.max_total_tokens,
                                   max_prefill_tokens=max(self.cfg.max_batch_prefill_tokens, 16), use_graphs=self.cfg.compile)
         self.seqs: Dict[int, SeqState] = {}
@@ -299,6 +303,9 @@ class ShardRuntime:
         """Put Medusa heads on the device under `adapter_index` (0 = default heads for every request).  As in the reference
         (adapters/medusa.py:52-71) heads loaded at request time need speculation to be on and must not have more heads than
         the configured number of speculative tokens; the first heads loaded as index 0 turn speculation on."""
+        if self.model.recurrent:
+            raise ValueError(f"{self.model.config.model_type} carries a recurrent state: a rejected guess cannot be taken back, so Medusa heads "
+                             "are not available")
         heads = MedusaHeads(config, tensors, self.model.device, self.model.dtype)
         if adapter_index == 0 and self.cfg.speculative_tokens == 0:
             self.cfg.speculative_tokens = heads.num_heads
@@ -335,6 +342,9 @@ class ShardRuntime:
         for bid in ids:
             for rid in self.batches.pop(bid, []):
                 self._drop(rid)
+        if not req.HasField("id") and self.kv.state_slots is not None:
+            for rid in [r for r in self.kv.state_slots.of_request if r not in self.seqs]:
+                self._release_state(rid)
         if self.seqs:
             self._resort()
         return self.pb.ClearCacheResponse()
@@ -344,6 +354,27 @@ class ShardRuntime:
         if s is not None and s.row >= 0:
             self.runner.retire([s.row])
             self.runner.state.drop_row(s.row)
+        self._release_state(rid)
+
+    def _release_state(self, rid: int):
+        if self.kv.state_slots is not None:
+            self.kv.state_slots.release(rid)
+
+    def _state_slot(self, rid: int, cache_len: int, batch_ids) -> int:
+        """The state slot of a request whose prompt (or the portion from `cache_len` on) is about to run; 0 for models without."""
+        slots = self.kv.state_slots
+        if slots is None:
+            return 0
+        if cache_len > 0 and rid not in slots.of_request:
+            raise RuntimeError(f"request {rid} goes on at token {cache_len} but its state is not on this shard")
+        slot = slots.acquire(rid)
+        if slot is None:                                     # requests that went away between two portions of their prompt
+            for other in [r for r in slots.of_request if r not in self.seqs and r not in batch_ids]:
+                slots.release(other)
+            slot = slots.acquire(rid)
+        if slot is None:
+            raise RuntimeError("no state slot is free")
+        return slot
 
     def _resort(self):
         mapping = self.runner.resort()
@@ -522,14 +553,16 @@ class ShardRuntime:
         (chunked prefill: reference `server.py:93-123`, `flash_causal_lm.py:171-389`)."""
         items, seqs, chunks = [], [], []
         max_in = self.cfg.max_input_length
+        batch_ids = {r.id for r in batch.requests}
         for r in batch.requests:
             ids = list(r.tokenized_inputs.ids) if r.HasField("tokenized_inputs") and len(r.tokenized_inputs.ids) else self.tokenize(r.inputs)
             trunc = r.truncate or max_in
             ids = ids[-trunc:]
+            state_slot = self._state_slot(r.id, r.cache_len, batch_ids)
             if r.HasField("chunk_len") and r.cache_len + r.chunk_len < len(ids):
                 lora_index = r.adapter_index if (r.adapter_index == 0 or self.adapters.is_loaded(r.adapter_index)) else 0
                 chunks.append(PrefillItem(ids[r.cache_len: r.cache_len + r.chunk_len], r.cache_len, list(r.blocks), lora_index,
-                                          want_logits=False))
+                                          want_logits=False, state_slot=state_slot))
                 continue
             params = self._params_from_pb(r.parameters)
             stopping = StoppingCriteria(r.stopping_parameters.max_new_tokens or 1, self.eos_ids, list(r.stopping_parameters.stop_sequences),
@@ -545,7 +578,7 @@ class ShardRuntime:
                 s.grammar = compile_schema(params.schema, self.tokenizer, self.eos_ids)
             seqs.append(s)
             items.append(PrefillItem(ids[r.cache_len:] if r.cache_len else ids, r.cache_len, list(r.blocks), lora_index,
-                                     all_logprobs=r.prefill_logprobs))
+                                     all_logprobs=r.prefill_logprobs, state_slot=state_slot))
         return seqs, items, chunks
 
     def _finish_prefill(self, batch, seqs, items, next_ids, lps, logits, merge_with: Optional[List[int]] = None, merged_id: Optional[int] = None,
@@ -566,7 +599,7 @@ class ShardRuntime:
         ids_l, lps_l, alts = self._sample_rows(seqs, logits.index_select(0, last_rows) if logits is not None else None, gid, glp)
         if self.medusa and self.model.last_hidden is not None and self.model.last_hidden.shape[0] == next_ids.shape[0]:
             self._medusa_guess(seqs, self.model.last_hidden.index_select(0, last_rows))
-        gens, live, rows, firsts, poss, blks, ads = [], [], [], [], [], [], []
+        gens, live, rows, firsts, poss, blks, ads, sts = [], [], [], [], [], [], [], []
         o = 0
         for s, it, tok, lp, alt in zip(seqs, items, ids_l, lps_l, alts):
             gen, stop = self._emit(s, int(tok), float(lp), alt)
@@ -585,9 +618,12 @@ class ShardRuntime:
                 s.row = self.runner.state.take_row(s.request_id)
                 live.append(s.request_id)
                 rows.append(s.row); firsts.append(int(tok)); poss.append(len(s.prompt_ids)); blks.append(s.blocks); ads.append(s.adapter_index)
+                sts.append(it.state_slot)
+            else:
+                self._release_state(s.request_id)
         resp = pb.PrefillResponse(generations=list(extra_generations) + gens)
         if live:
-            self.runner.install(rows, firsts, poss, blks, ads)
+            self.runner.install(rows, firsts, poss, blks, ads, sts)
             self._resort()
         bid = batch.id if merged_id is None else merged_id
         members = list(merge_with or []) + live

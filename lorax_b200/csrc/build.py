@@ -64,14 +64,23 @@ def _run(cmd, verbose: bool, log_path: Path | None = None, quiet: bool = False) 
     return proc.stdout
 
 
-def build_kernels(force: bool = False, verbose: bool = False) -> Path:
+# Sources a program needs that only ever runs one kind of model (`ops.native.use_subset`).
+SUBSETS = {"mixers": ("gemm_bf16", "elementwise", "stream", "recurrent", "latent_attn")}
+
+
+def build_kernels(force: bool = False, verbose: bool = False, subset: str | None = None) -> Path:
+    """All kernels -> `_lx_kernels.so`; with `subset`, the sources of that subset -> `_lx_kernels_<subset>.so`."""
     sources = sorted(KERNEL_DIR.glob("*.cu"))
+    target, stamp_name = KERNELS_SO, "kernels.sha256"
+    if subset is not None:
+        sources = [s for s in sources if s.stem in SUBSETS[subset]]
+        target, stamp_name = PKG / f"_lx_kernels_{subset}.so", f"kernels_{subset}.sha256"
     headers = sorted(KERNEL_DIR.glob("*.cuh")) + sorted(KERNEL_DIR.glob("*.h"))
     BUILD_DIR.mkdir(exist_ok=True)
-    stamp = BUILD_DIR / "kernels.sha256"
+    stamp = BUILD_DIR / stamp_name
     digest = _digest(sources + headers + [Path(__file__)])
-    if not force and KERNELS_SO.exists() and stamp.exists() and stamp.read_text() == digest:
-        return KERNELS_SO
+    if not force and target.exists() and stamp.exists() and stamp.read_text() == digest:
+        return target
     nvcc = _nvcc()
     hdr_digest = _digest(headers)
 
@@ -88,10 +97,10 @@ def build_kernels(force: bool = False, verbose: bool = False) -> Path:
 
     with cf.ThreadPoolExecutor(max_workers=min(8, len(sources) or 1)) as ex:
         objs = list(ex.map(compile_one, sources))
-    _run([nvcc, "-shared", "-o", str(KERNELS_SO), *map(str, objs), "-gencode", "arch=compute_100a,code=sm_100a",
+    _run([nvcc, "-shared", "-o", str(target), *map(str, objs), "-gencode", "arch=compute_100a,code=sm_100a",
           "-Xcompiler", "-fPIC", "-lcudart_static", "-ldl", "-lrt", "-lpthread"], verbose)
     stamp.write_text(digest)
-    return KERNELS_SO
+    return target
 
 
 def _unicode_tables():

@@ -1,0 +1,416 @@
+// Token-wise kernels of the layer-by-layer designs: fp32 residual stream (embedding, norm), gated RMS norms of mixer outputs,
+// per-head products, and the 32-bit forms of the matrix product, gated activation and greedy head.
+#include "stream.cuh"
+
+namespace lx {
+
+// ------------------------------------------------------------------------------------------------
+// Residual stream: x[t] = table[ids[t]] * mult in fp32.
+// ------------------------------------------------------------------------------------------------
+template <typename T>
+__global__ void __launch_bounds__(128) embed_stream_kernel(const int* __restrict__ ids, const T* __restrict__ table, float* __restrict__ out,
+                                                           int W, int V, float mult) {
+  pdl_trigger();
+  pdl_wait();
+  const int t = blockIdx.x;
+  const int id = min(max(ids[t], 0), V - 1);
+  for (int c = threadIdx.x * 8; c < W; c += blockDim.x * 8) {
+    float f[8];
+    load8(table + (long long)id * W + c, f);
+#pragma unroll
+    for (int q = 0; q < 8; ++q) f[q] *= mult;
+    store8(out + (long long)t * W + c, f);
+  }
+}
+
+// ------------------------------------------------------------------------------------------------
+// residual += pending (fp32); out = residual / sqrt(sum / n + eps) * (w + w_offset).  One CTA per row.
+// ------------------------------------------------------------------------------------------------
+constexpr int kNsThreads = 256, kNsMaxVec = 8;      // 16384 columns at most
+
+template <typename T>
+__global__ void __launch_bounds__(kNsThreads) norm_stream_kernel(float* __restrict__ residual, const T* __restrict__ pending,
+                                                                 const float* __restrict__ w, T* __restrict__ out, int W, float inv_n,
+                                                                 float eps, float w_offset) {
+  pdl_trigger();
+  pdl_wait();
+  __shared__ float red[kNsThreads / 32];
+  const long long row = (long long)blockIdx.x * W;
+  float v[kNsMaxVec][8];
+  float ss = 0.f;
+#pragma unroll
+  for (int it = 0; it < kNsMaxVec; ++it) {
+    const int c = (threadIdx.x + it * blockDim.x) * 8;
+    if (c < W) {
+      load8(residual + row + c, v[it]);
+      if (pending != nullptr) {
+        float p[8];
+        load8(pending + row + c, p);
+#pragma unroll
+        for (int q = 0; q < 8; ++q) v[it][q] += p[q];
+        store8(residual + row + c, v[it]);
+      }
+#pragma unroll
+      for (int q = 0; q < 8; ++q) ss += v[it][q] * v[it][q];
+    }
+  }
+  const float r = rsqrtf(block_sum(ss, red) * inv_n + eps);
+#pragma unroll
+  for (int it = 0; it < kNsMaxVec; ++it) {
+    const int c = (threadIdx.x + it * blockDim.x) * 8;
+    if (c < W) {
+      float g[8];
+      load8(w + c, g);
+#pragma unroll
+      for (int q = 0; q < 8; ++q) g[q] = v[it][q] * r * (g[q] + w_offset);
+      store8(out + row + c, g);
+    }
+  }
+}
+
+// ------------------------------------------------------------------------------------------------
+// Gated RMS norm: every `group` columns of x (fp32) divided by their root mean square (over n columns), times weight, times
+// sigmoid(gate) or silu(gate).  WARP: one warp per group (up to 512 columns), else one CTA per group.
+// ------------------------------------------------------------------------------------------------
+template <typename T, bool WARP>
+__global__ void __launch_bounds__(256) norm_gate_kernel(const float* __restrict__ x, const float* __restrict__ w, const T* __restrict__ gate,
+                                                        long long ldg, T* __restrict__ out, long long ldo, int groups, int group, float inv_n,
+                                                        float eps, int silu) {
+  pdl_trigger();
+  pdl_wait();
+  __shared__ float red[8];
+  const int t = blockIdx.x;
+  const int lane = WARP ? (threadIdx.x & 31) : threadIdx.x;
+  const int width = WARP ? 32 : blockDim.x;
+  const int g = WARP ? blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5) : blockIdx.y;
+  if (WARP && g >= groups) return;
+  const long long base = (long long)t * groups * group + (long long)g * group;
+  float ss = 0.f;
+  for (int c = lane * 4; c < group; c += width * 4) {
+    const float4 a = load4(x + base + c);
+    ss += a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w;
+  }
+  ss = WARP ? warp_sum(ss) : block_sum(ss, red);
+  const float r = rsqrtf(ss * inv_n + eps);
+  for (int c = lane * 4; c < group; c += width * 4) {
+    float4 a = load4(x + base + c);
+    const int col = g * group + c;
+    const float4 ww = load4(w + col);
+    const float4 z = load4(gate + (long long)t * ldg + col);
+    if (silu) {
+      a.x *= r * ww.x * silu_f(z.x); a.y *= r * ww.y * silu_f(z.y); a.z *= r * ww.z * silu_f(z.z); a.w *= r * ww.w * silu_f(z.w);
+    } else {
+      a.x *= r * ww.x * sigmoid_f(z.x); a.y *= r * ww.y * sigmoid_f(z.y); a.z *= r * ww.z * sigmoid_f(z.z); a.w *= r * ww.w * sigmoid_f(z.w);
+    }
+    store4(out + (long long)t * ldo + col, a);
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) tanh_kernel(T* __restrict__ x, long long n8) {
+  pdl_trigger();
+  pdl_wait();
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < n8; i += (long long)gridDim.x * blockDim.x) {
+    float f[8];
+    load8(x + i * 8, f);
+#pragma unroll
+    for (int q = 0; q < 8; ++q) f[q] = tanhf(f[q]);
+    store8(x + i * 8, f);
+  }
+}
+
+// out[t, i] = gelu_tanh(x[t, i]) * x[t, I + i] (or silu) for fp32 rows
+__global__ void __launch_bounds__(256) act_mul_f32_kernel(const float* __restrict__ x, float* __restrict__ out, int I, long long ldx,
+                                                          long long ldo, long long total4, int act, int gated) {
+  pdl_trigger();
+  pdl_wait();
+  const int per_row = I / 4;
+  for (long long v = blockIdx.x * (long long)blockDim.x + threadIdx.x; v < total4; v += (long long)gridDim.x * blockDim.x) {
+    const long long t = v / per_row;
+    const int c = (int)(v % per_row) * 4;
+    float4 a = load4(x + t * ldx + c);
+    float* e = reinterpret_cast<float*>(&a);
+#pragma unroll
+    for (int q = 0; q < 4; ++q) {
+      const float z = e[q];
+      if (act == 0) e[q] = silu_f(z);
+      else if (act == 1) e[q] = 0.5f * z * (1.f + erff(z * 0.70710678118654752f));
+      else if (act == 2) e[q] = 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+      else e[q] = fmaxf(z, 0.f);
+    }
+    if (gated) {
+      const float4 u = load4(x + t * ldx + I + c);
+      a.x *= u.x; a.y *= u.y; a.z *= u.z; a.w *= u.w;
+    }
+    store4(out + t * ldo + c, a);
+  }
+}
+
+// Greedy head over fp32 logits: arg-max (lowest index on ties) and its log-probability.
+__global__ void __launch_bounds__(512) argmax_f32_kernel(const float* __restrict__ logits, long long ld, int V, int* __restrict__ ids,
+                                                         float* __restrict__ lps, float softcap) {
+  pdl_trigger();
+  pdl_wait();
+  const float* row = logits + (long long)blockIdx.x * ld;
+  __shared__ float sm[16], red[16];
+  __shared__ int si[16];
+  float best = -INFINITY;
+  int bi = 0x7fffffff;
+  for (int i = threadIdx.x; i < V; i += blockDim.x) {
+    float x = row[i];
+    if (softcap > 0.f) x = softcap * tanhf(x / softcap);
+    if (x > best) { best = x; bi = i; }
+  }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+    const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+    if (ob > best || (ob == best && oi < bi)) { best = ob; bi = oi; }
+  }
+  if ((threadIdx.x & 31) == 0) { sm[threadIdx.x >> 5] = best; si[threadIdx.x >> 5] = bi; }
+  __syncthreads();
+  best = sm[0]; bi = si[0];
+  for (int i = 1; i < (int)(blockDim.x >> 5); ++i)
+    if (sm[i] > best || (sm[i] == best && si[i] < bi)) { best = sm[i]; bi = si[i]; }
+  float s = 0.f;
+  for (int i = threadIdx.x; i < V; i += blockDim.x) {
+    float x = row[i];
+    if (softcap > 0.f) x = softcap * tanhf(x / softcap);
+    s += expf(x - best);
+  }
+  s = block_sum(s, red);
+  if (threadIdx.x == 0) {
+    ids[blockIdx.x] = bi;
+    if (lps) lps[blockIdx.x] = -logf(s);
+  }
+}
+
+// ------------------------------------------------------------------------------------------------
+// Batched product in true fp32: out[b][t, n] = sum_k x[b][t, k] * w[b][n, k] (* sigmoid(gate[t, b])).  64 x 64 tiles.
+// ------------------------------------------------------------------------------------------------
+struct BatchedGemmParams {
+  const void* x; const void* w; void* out; const void* gate;
+  long long ldx, sx, ldw, sw, ldo, so, ldg;
+  int T, N, K;
+  float out_scale;
+};
+
+__global__ void __launch_bounds__(256) gemm_f32_kernel(const BatchedGemmParams p) {
+  pdl_trigger();
+  pdl_wait();
+  __shared__ float xs[16][68], ws[16][68];
+  const int b = blockIdx.z, t0 = blockIdx.y * 64, n0 = blockIdx.x * 64;
+  const float* x = reinterpret_cast<const float*>(p.x) + b * p.sx;
+  const float* w = reinterpret_cast<const float*>(p.w) + b * p.sw;
+  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+  const int lr = threadIdx.x >> 2, lk = (threadIdx.x & 3) * 4;
+  float acc[4][4] = {};
+  for (int k0 = 0; k0 < p.K; k0 += 16) {
+#pragma unroll
+    for (int q = 0; q < 4; ++q) {
+      const int k = k0 + lk + q;
+      xs[lk + q][lr] = (t0 + lr < p.T && k < p.K) ? x[(long long)(t0 + lr) * p.ldx + k] : 0.f;
+      ws[lk + q][lr] = (n0 + lr < p.N && k < p.K) ? w[(long long)(n0 + lr) * p.ldw + k] : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < 16; ++k) {
+      float a[4], c[4];
+#pragma unroll
+      for (int q = 0; q < 4; ++q) { a[q] = xs[k][ty * 4 + q]; c[q] = ws[k][tx * 4 + q]; }
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(a[i], c[j], acc[i][j]);
+    }
+    __syncthreads();
+  }
+  float* out = reinterpret_cast<float*>(p.out) + b * p.so;
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int t = t0 + ty * 4 + i;
+    if (t >= p.T) continue;
+    const float s = p.gate ? p.out_scale * sigmoid_f(reinterpret_cast<const float*>(p.gate)[(long long)t * p.ldg + b]) : p.out_scale;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int n = n0 + tx * 4 + j;
+      if (n < p.N) out[(long long)t * p.ldo + n] = acc[i][j] * s;
+    }
+  }
+}
+
+// ------------------------------------------------------------------------------------------------
+// The same product per head in bf16 on mma.sync (K and N of a head are small: the work is a batch of skinny products).  64 tokens x
+// 64 columns per CTA of four warps, K in steps of 32 through a double-buffered shared-memory ring.
+// ------------------------------------------------------------------------------------------------
+LX_DEVICE void mma16816(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+LX_DEVICE void ldsm4(uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3, uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
+}
+
+constexpr int kGhK = 64, kGhLd = kGhK + 8;      // row pitch 144 bytes: eight rows of one ldmatrix hit different banks
+
+__global__ void __launch_bounds__(128) gemm_heads_kernel(const BatchedGemmParams p) {
+  pdl_trigger();
+  pdl_wait();
+  __shared__ __align__(16) __nv_bfloat16 xs[2][64 * kGhLd], ws[2][64 * kGhLd];
+  const int b = blockIdx.z, t0 = blockIdx.y * 64, n0 = blockIdx.x * 64;
+  const __nv_bfloat16* x = reinterpret_cast<const __nv_bfloat16*>(p.x) + b * p.sx;
+  const __nv_bfloat16* w = reinterpret_cast<const __nv_bfloat16*>(p.w) + b * p.sw;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  auto load = [&](int st, int k0) {
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int c = threadIdx.x + i * 128, r = c >> 3, k = k0 + (c & 7) * 8;
+      const bool okx = t0 + r < p.T && k < p.K, okw = n0 + r < p.N && k < p.K;
+      cp_async_16(&xs[st][r * kGhLd + (c & 7) * 8], okx ? x + (long long)(t0 + r) * p.ldx + k : x, okx);
+      cp_async_16(&ws[st][r * kGhLd + (c & 7) * 8], okw ? w + (long long)(n0 + r) * p.ldw + k : w, okw);
+    }
+    cp_async_commit();
+  };
+  const int nk = (p.K + kGhK - 1) / kGhK;
+  float acc[8][4];
+#pragma unroll
+  for (int i = 0; i < 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+  load(0, 0);
+  for (int s = 0; s < nk; ++s) {
+    if (s + 1 < nk) load((s + 1) & 1, (s + 1) * kGhK); else cp_async_commit();
+    cp_async_wait<1>();
+    __syncthreads();
+    const uint32_t xa = smem_u32(xs[s & 1]) + ((warp * 16 + (lane & 15)) * kGhLd + (lane >> 4) * 8) * 2;
+    const uint32_t wa = smem_u32(ws[s & 1]) + (((lane & 7) + (lane >> 4) * 8) * kGhLd + ((lane >> 3) & 1) * 8) * 2;
+#pragma unroll
+    for (int ks = 0; ks < kGhK / 16; ++ks) {
+      uint32_t a[4];
+      ldsm4(a[0], a[1], a[2], a[3], xa + ks * 32);
+#pragma unroll
+      for (int nt = 0; nt < 4; ++nt) {
+        uint32_t b0, b1, b2, b3;
+        ldsm4(b0, b1, b2, b3, wa + nt * 16 * kGhLd * 2 + ks * 32);
+        mma16816(acc[2 * nt], a, b0, b1);
+        mma16816(acc[2 * nt + 1], a, b2, b3);
+      }
+    }
+    __syncthreads();
+  }
+  __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(p.out) + b * p.so;
+#pragma unroll
+  for (int hr = 0; hr < 2; ++hr) {
+    const int t = t0 + warp * 16 + (lane >> 2) + hr * 8;
+    if (t >= p.T) continue;
+    const float s = p.gate ? sigmoid_f(to_f(reinterpret_cast<const __nv_bfloat16*>(p.gate)[(long long)t * p.ldg + b])) : 1.f;
+#pragma unroll
+    for (int nt = 0; nt < 8; ++nt) {
+      const int n = n0 + nt * 8 + (lane & 3) * 2;
+      if (n < p.N) *reinterpret_cast<uint32_t*>(out + (long long)t * p.ldo + n) = pack_bf16x2(acc[nt][2 * hr] * s, acc[nt][2 * hr + 1] * s);
+    }
+  }
+}
+
+}  // namespace lx
+
+extern "C" {
+
+// `f32` selects the element type of activations and weights everywhere below (0: bf16, 1: fp32).
+int lx_embed_stream(const int* ids, const void* table, void* out, int T, int W, int V, float mult, int f32, void* stream) {
+  using namespace lx;
+  if (T <= 0) return 0;
+  if (W % 8 != 0 || V <= 0) return -1;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  float* o = reinterpret_cast<float*>(out);
+  if (f32) launch_pdl(embed_stream_kernel<float>, dim3(T), dim3(128), 0, s, ids, reinterpret_cast<const float*>(table), o, W, V, mult);
+  else launch_pdl(embed_stream_kernel<__nv_bfloat16>, dim3(T), dim3(128), 0, s, ids, reinterpret_cast<const __nv_bfloat16*>(table), o, W, V, mult);
+  return -(int)cudaGetLastError();
+}
+
+int lx_norm_stream(void* residual, const void* pending, const void* w, void* out, int T, int W, int n, float eps, float w_offset, int f32,
+                   void* stream) {
+  using namespace lx;
+  if (T <= 0) return 0;
+  if (W % 8 != 0 || W > kNsThreads * kNsMaxVec * 8 || n <= 0) return -1;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  const int threads = W / 8 >= kNsThreads ? kNsThreads : (W / 8 + 31) / 32 * 32;
+  float* r = reinterpret_cast<float*>(residual);
+  const float* wp = reinterpret_cast<const float*>(w);
+  if (f32)
+    launch_pdl(norm_stream_kernel<float>, dim3(T), dim3(threads), 0, s, r, reinterpret_cast<const float*>(pending), wp, reinterpret_cast<float*>(out), W,
+               1.f / n, eps, w_offset);
+  else
+    launch_pdl(norm_stream_kernel<__nv_bfloat16>, dim3(T), dim3(threads), 0, s, r, reinterpret_cast<const __nv_bfloat16*>(pending), wp,
+               reinterpret_cast<__nv_bfloat16*>(out), W, 1.f / n, eps, w_offset);
+  return -(int)cudaGetLastError();
+}
+
+int lx_norm_gate(const void* x, const void* w, const void* gate, long long ldg, void* out, long long ldo, int T, int groups, int group, int n,
+                 float eps, int silu, int f32, void* stream) {
+  using namespace lx;
+  if (T <= 0) return 0;
+  if (group % 4 != 0 || ldg % 4 != 0 || ldo % 4 != 0 || n <= 0) return -1;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  const bool warp = group <= 512;
+  const int wpb = groups < 8 ? groups : 8;
+  const dim3 grid(T, warp ? (groups + wpb - 1) / wpb : groups), block(warp ? 32 * wpb : 256);
+  const float* xp = reinterpret_cast<const float*>(x);
+  const float* wp = reinterpret_cast<const float*>(w);
+#define LX_NG(TY, WP)                                                                                                                  \
+  launch_pdl(norm_gate_kernel<TY, WP>, grid, block, 0, s, xp, wp, reinterpret_cast<const TY*>(gate), ldg, reinterpret_cast<TY*>(out), ldo, \
+             groups, group, 1.f / n, eps, silu)
+  if (f32) { if (warp) LX_NG(float, true); else LX_NG(float, false); }
+  else { if (warp) LX_NG(__nv_bfloat16, true); else LX_NG(__nv_bfloat16, false); }
+#undef LX_NG
+  return -(int)cudaGetLastError();
+}
+
+int lx_tanh(void* x, long long n, int f32, void* stream) {
+  using namespace lx;
+  if (n <= 0) return 0;
+  if (n % 8 != 0) return -1;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  const long long n8 = n / 8;
+  const int grid = (int)((n8 + 255) / 256 < 148 * 8 ? (n8 + 255) / 256 : 148 * 8);
+  if (f32) launch_pdl(tanh_kernel<float>, dim3(grid), dim3(256), 0, s, reinterpret_cast<float*>(x), n8);
+  else launch_pdl(tanh_kernel<__nv_bfloat16>, dim3(grid), dim3(256), 0, s, reinterpret_cast<__nv_bfloat16*>(x), n8);
+  return -(int)cudaGetLastError();
+}
+
+int lx_act_mul_f32(const void* x, void* out, int T, int I, long long ldx, long long ldo, int act, int gated, void* stream) {
+  using namespace lx;
+  if (T <= 0) return 0;
+  if (I % 4 != 0 || ldx % 4 != 0 || ldo % 4 != 0) return -1;
+  const long long total = (long long)T * (I / 4);
+  const int grid = (int)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16);
+  launch_pdl(act_mul_f32_kernel, dim3(grid), dim3(256), 0, reinterpret_cast<cudaStream_t>(stream), reinterpret_cast<const float*>(x),
+             reinterpret_cast<float*>(out), I, ldx, ldo, total, act, gated);
+  return -(int)cudaGetLastError();
+}
+
+int lx_argmax_f32(const void* logits, long long ld, int T, int V, int* ids, float* logprobs, float softcap, void* stream) {
+  using namespace lx;
+  if (T <= 0) return 0;
+  launch_pdl(argmax_f32_kernel, dim3(T), dim3(512), 0, reinterpret_cast<cudaStream_t>(stream), reinterpret_cast<const float*>(logits), ld, V, ids,
+             logprobs, softcap);
+  return -(int)cudaGetLastError();
+}
+
+// out[b][t, n] = x[b][t, :] . w[b][n, :] over `batch` products with element strides sx / sw / so; gate [T, ldg]: column b.
+int lx_gemm_batched(const void* x, long long ldx, long long sx, const void* w, long long ldw, long long sw, void* out, long long ldo,
+                    long long so, const void* gate, long long ldg, int T, int N, int K, int batch, float out_scale, int f32, void* stream) {
+  using namespace lx;
+  if (T <= 0 || N <= 0 || batch <= 0) return 0;
+  BatchedGemmParams p{x, w, out, gate, ldx, sx, ldw, sw, ldo, so, ldg, T, N, K, out_scale};
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  const dim3 grid((N + 63) / 64, (T + 63) / 64, batch);
+  if (f32) {
+    launch_pdl(gemm_f32_kernel, grid, dim3(256), 0, s, p);
+  } else {
+    if (K % 8 != 0 || N % 2 != 0 || ldx % 8 != 0 || sx % 8 != 0 || ldw % 8 != 0 || sw % 8 != 0 || ldo % 2 != 0 || so % 2 != 0) return -1;
+    launch_pdl(gemm_heads_kernel, grid, dim3(128), 0, s, p);
+  }
+  return -(int)cudaGetLastError();
+}
+
+}  // extern "C"

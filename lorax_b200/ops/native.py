@@ -37,17 +37,28 @@ def available() -> bool:
     return _LIB_PATH.exists()
 
 
+_subset: Optional[str] = None
+
+
+def use_subset(name: str):
+    """For programs that run one kind of model: when the full library has not been built yet, `load()` builds and loads only the
+    sources this kind needs (`csrc.build.SUBSETS`).  An existing full library is used as it is."""
+    global _subset
+    _subset = name
+
+
 def load() -> ctypes.CDLL:
     global _lib
     if _lib is not None:
         return _lib
-    if not _LIB_PATH.exists():
+    path = _LIB_PATH
+    if not path.exists():
         if os.environ.get("LORAX_B200_NO_BUILD") != "1":
             from lorax_b200.csrc import build as _build
-            _build.build_kernels()
-        if not _LIB_PATH.exists():
-            raise NativeError(f"{_LIB_PATH} is missing; run `python -m lorax_b200.csrc.build`")
-    lib = ctypes.CDLL(str(_LIB_PATH))
+            path = _build.build_kernels(subset=_subset)
+        if not path.exists():
+            raise NativeError(f"{path} is missing; run `python -m lorax_b200.csrc.build`")
+    lib = ctypes.CDLL(str(path))
     P, I, L, F = c_void_p, c_int, c_longlong, c_float
     sigs = {
         "lx_gemm_ws_bytes": ([], L),
@@ -92,10 +103,17 @@ def load() -> ctypes.CDLL:
         "lx_moe_combine": ([P, L, P, P, I, P, L, I, I, P], I),
         "lx_moe_grouped_gemm": ([P, L, P, L, P, L, P, I, I, I, I, I, P, I, P], I),
     }
+    from . import native_mixers
+    sigs.update(native_mixers.SIGNATURES)
     for name, (argtypes, restype) in sigs.items():
-        fn = getattr(lib, name)
+        fn = getattr(lib, name, None)
+        if fn is None:
+            if path == _LIB_PATH:
+                raise NativeError(f"{path} does not export {name}: it is older than the package, run `python -m lorax_b200.csrc.build`")
+            continue
         fn.argtypes = argtypes
         fn.restype = restype
+    native_mixers.check_layouts(lib)
     _lib = lib
     return lib
 
@@ -247,7 +265,9 @@ def lora_fused_desc(ws: "Workspace", lf: LoraFused, K: int) -> LxLoraFused:
 
 def gemm(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None,
          out_scale: float = 1.0, mode: int = 0, force_split: int = 0) -> torch.Tensor:
-    """out[T, N] = x[T, K] @ w[N, K]^T (+ bias).  bf16 in, fp32 accumulate on tcgen05, bf16 out."""
+    """out[T, N] = x[T, K] @ w[N, K]^T (+ bias).  bf16 in, fp32 accumulate on tcgen05, bf16 out (fp32 in: true fp32 throughout)."""
+    if x.dtype == torch.float32 and bias is None:
+        return gemm_f32(x, w, out=out, out_scale=out_scale)
     assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and x.dim() == 2 and w.dim() == 2
     assert x.stride(1) == 1 and w.stride(1) == 1
     T, K = x.shape
@@ -478,6 +498,9 @@ def act_mul(x: torch.Tensor, inter: int, act: str = "silu", gated: bool = True, 
     T = x.shape[0]
     if out is None:
         out = torch.empty(T, inter, dtype=x.dtype, device=x.device)
+    if x.dtype == torch.float32:
+        _check(load().lx_act_mul_f32(_ptr(x), _ptr(out), T, inter, x.stride(0), out.stride(0), _ACTS[act], int(gated), _stream()), "lx_act_mul_f32")
+        return out
     rc = load().lx_act_mul(_ptr(x), _ptr(out), T, inter, x.stride(0), out.stride(0), _ACTS[act], int(gated), _stream())
     _check(rc, "lx_act_mul")
     return out
@@ -503,6 +526,9 @@ def argmax_logprob(logits: torch.Tensor, ids: Optional[torch.Tensor] = None, log
         ids = torch.empty(T, dtype=torch.int32, device=logits.device)
     if logprobs is None:
         logprobs = torch.empty(T, dtype=torch.float32, device=logits.device)
+    if logits.dtype == torch.float32:
+        _check(load().lx_argmax_f32(_ptr(logits), logits.stride(0), T, V, _ptr(ids), _ptr(logprobs), softcap, _stream()), "lx_argmax_f32")
+        return ids, logprobs
     rc = load().lx_argmax_logprob(_ptr(logits), logits.stride(0), T, V, _ptr(ids), _ptr(logprobs), softcap, _stream())
     _check(rc, "lx_argmax_logprob")
     return ids, logprobs
@@ -656,9 +682,16 @@ def lora_expand_tiles(v, tiles: torch.Tensor, num_tiles: int, max_tile_rows: int
                                      _ptr(ws.status), _stream())
     _check(rc, "lx_lora_expand_tiled")
 
+
+# ------------------------------------------------------------------------------------------------ layer-by-layer designs
+from .native_mixers import (embed_stream, gemm_f32, gemm_heads, gemm_stack, latent_attn, latent_prep, linear_attn, norm_gate,  # noqa: E402
+                            norm_stream, rope_pairs, tanh_, token_shift, wkv)
+
 # ------------------------------------------------------------------------------------------------ per-op timing
 _TIMED_OPS = ("gemm", "gemm_fp8", "norm_residual", "rope_kvwrite", "act_mul", "embed", "argmax_logprob", "advance_decode", "attn_decode",
-              "attn_prefill", "lora_shrink", "lora_expand", "lora_shrink_tiles", "lora_expand_tiles")
+              "attn_prefill", "lora_shrink", "lora_expand", "lora_shrink_tiles", "lora_expand_tiles",
+              "embed_stream", "norm_stream", "norm_gate", "tanh_", "gemm_heads", "linear_attn", "wkv", "token_shift", "latent_prep", "rope_pairs",
+              "latent_attn")
 _timing_records = None
 _timing_originals = {}
 

@@ -1,0 +1,204 @@
+"""Bindings of the kernels of the layer-by-layer designs (`models/mixers.py`): `csrc/kernels/stream.cu`, `recurrent.cu` and
+`latent_attn.cu`.  Every operator exists for bf16 and for fp32 activations.  Imported into :mod:`lorax_b200.ops.native`."""
+
+from __future__ import annotations
+
+import ctypes
+from ctypes import POINTER, Structure, c_float, c_int, c_longlong, c_void_p
+from typing import Optional
+
+import torch
+
+from . import native as nv
+
+P, I, L, F = c_void_p, c_int, c_longlong, c_float
+
+
+class StepRows(Structure):
+    _fields_ = [("nd", I), ("dec_slots", P), ("ctx_lens", P), ("dec_bt", P), ("B", I), ("cu_q", P), ("cache_lens", P), ("slots", P),
+                ("bt", P), ("max_blocks", I), ("dec_max_blocks", I)]
+
+
+class RecParams(Structure):
+    _fields_ = [("q", P), ("k", P), ("v", P), ("z", P), ("ldq", L), ("ldk", L), ("ldv", L), ("ldz", L), ("decay", P), ("w0", P), ("u", P),
+                ("state", P), ("out", P), ("H", I), ("d", I), ("dv", I), ("rows", StepRows), ("seg_seq", P), ("seg_q0", P), ("nseg", I),
+                ("seg_len", I), ("seg_state", P), ("seg_decay", P)]
+
+
+class LatentPrepParams(Structure):
+    _fields_ = [("dq", P), ("dkv", P), ("ld_dq", L), ("ld_dkv", L), ("dq_norm", P), ("dkv_norm", P), ("cq", P), ("cache", P),
+                ("positions", P), ("slots", P), ("cos_sin", P), ("QR", I), ("KR", I), ("R", I), ("q_rank", I), ("kv_rank", I), ("rot", I),
+                ("eps", F)]
+
+
+class LatentAttnParams(Structure):
+    _fields_ = [("q_lat", P), ("ld_ql", L), ("q", P), ("ldq", L), ("head", I), ("rot_off", I), ("cache", P), ("out", P), ("ldo", L),
+                ("rows", StepRows), ("H", I), ("KR", I), ("R", I), ("page", I), ("scale", F)]
+
+
+SIGNATURES = {
+    "lx_embed_stream": ([P, P, P, I, I, I, F, I, P], I),
+    "lx_norm_stream": ([P, P, P, P, I, I, I, F, F, I, P], I),
+    "lx_norm_gate": ([P, P, P, L, P, L, I, I, I, I, F, I, I, P], I),
+    "lx_tanh": ([P, L, I, P], I),
+    "lx_act_mul_f32": ([P, P, I, I, L, L, I, I, P], I),
+    "lx_argmax_f32": ([P, L, I, I, P, P, F, P], I),
+    "lx_gemm_batched": ([P, L, L, P, L, L, P, L, L, P, L, I, I, I, I, F, I, P], I),
+    "lx_step_rows_bytes": ([], I),
+    "lx_rec_params_bytes": ([], I),
+    "lx_recurrence": ([P, I, I, I, P], I),
+    "lx_token_shift": ([P, P, P, P, I, I, I, P, I, P], I),
+    "lx_latent_prep_bytes": ([], I),
+    "lx_latent_attn_bytes": ([], I),
+    "lx_latent_prep": ([P, I, I, P], I),
+    "lx_rope_pairs": ([P, L, P, P, I, I, I, I, I, I, P], I),
+    "lx_latent_attn": ([P, I, I, P], I),
+}
+
+
+def check_layouts(lib):
+    for name, st in (("lx_step_rows_bytes", StepRows), ("lx_rec_params_bytes", RecParams), ("lx_latent_prep_bytes", LatentPrepParams),
+                     ("lx_latent_attn_bytes", LatentAttnParams)):
+        if getattr(lib, name)() != ctypes.sizeof(st):
+            raise nv.NativeError(f"{name}: C++ says {getattr(lib, name)()} bytes, ctypes says {ctypes.sizeof(st)}")
+
+
+def _f32(t: torch.Tensor) -> int:
+    return int(t.dtype == torch.float32)
+
+
+def _p(t: Optional[torch.Tensor]):
+    return None if t is None else t.data_ptr()
+
+
+def step_rows(inp, T: int) -> StepRows:
+    nd, dbt, slots, ctx = inp.decode_view(T)
+    r = StepRows()
+    r.nd = nd
+    if nd:
+        r.dec_slots, r.ctx_lens, r.dec_bt, r.dec_max_blocks = _p(slots), _p(ctx), _p(dbt), dbt.shape[1]
+    if inp.is_prefill:
+        r.B, r.cu_q, r.cache_lens, r.slots = inp.cache_lens.shape[0], _p(inp.cu_q), _p(inp.cache_lens), _p(inp.state_slots)
+        r.bt, r.max_blocks = _p(inp.block_tables), inp.block_tables.shape[1]
+    return r
+
+
+def embed_stream(ids, table, mult: float = 1.0):
+    T, W = ids.shape[0], table.shape[1]
+    out = torch.empty(T, W, dtype=torch.float32, device=table.device)
+    nv._check(nv.load().lx_embed_stream(_p(ids), _p(table), _p(out), T, W, table.shape[0], mult, _f32(table), nv._stream()), "lx_embed_stream")
+    return out
+
+
+def norm_stream(residual, pending, weight, eps: float, weight_offset: float, n: int, dtype):
+    T, W = residual.shape
+    out = torch.empty(T, W, dtype=dtype, device=residual.device)
+    assert pending is None or pending.is_contiguous()
+    nv._check(nv.load().lx_norm_stream(_p(residual), _p(pending), _p(weight), _p(out), T, W, n, eps, weight_offset, _f32(out), nv._stream()),
+              "lx_norm_stream")
+    return out
+
+
+def norm_gate(x, group: int, n: int, weight, gate, act: str, eps: float, out):
+    T, C = x.shape
+    nv._check(nv.load().lx_norm_gate(_p(x), _p(weight), _p(gate), gate.stride(0), _p(out), out.stride(0), T, C // group, group, n, eps,
+                                     int(act == "silu"), _f32(out), nv._stream()), "lx_norm_gate")
+    return out
+
+
+def tanh_(x):
+    assert x.is_contiguous()
+    nv._check(nv.load().lx_tanh(_p(x), x.numel(), _f32(x), nv._stream()), "lx_tanh")
+    return x
+
+
+def gemm_f32(x, w, out=None, out_scale: float = 1.0):
+    T, K = x.shape
+    N = w.shape[0]
+    if out is None:
+        out = torch.empty(T, N, dtype=torch.float32, device=x.device)
+    nv._check(nv.load().lx_gemm_batched(_p(x), x.stride(0), 0, _p(w), w.stride(0), 0, _p(out), out.stride(0), 0, None, 0, T, N, K, 1, out_scale, 1,
+                                        nv._stream()), "lx_gemm_batched")
+    return out
+
+
+def gemm_stack(x, w):
+    """x [n, T, K], w [n, N, K] -> [n, T, N]: one product per stacked pair."""
+    n, T, _ = x.shape
+    out = torch.empty(n, T, w.shape[1], dtype=x.dtype, device=x.device)
+    for i in range(n):
+        nv.gemm(x[i], w[i], out=out[i])
+    return out
+
+
+def gemm_heads(x, w, out, x_head: int, gate=None):
+    """out[:, h * N : (h + 1) * N] = x[:, h * x_head : h * x_head + K] @ w[h]^T (* sigmoid(gate[:, h]))."""
+    H, N, K = w.shape
+    T = x.shape[0]
+    nv._check(nv.load().lx_gemm_batched(_p(x), x.stride(0), x_head, _p(w), K, N * K, _p(out), out.stride(0), N, _p(gate),
+                                        gate.stride(0) if gate is not None else 0, T, N, K, H, 1.0, _f32(x), nv._stream()), "lx_gemm_batched")
+    return out
+
+
+def _recurrence(mode: int, q, k, v, z, decay, w0, u, H: int, d: int, dv: int, state, inp):
+    T = q.shape[0]
+    out = torch.empty(T, H * dv, dtype=torch.float32, device=q.device)
+    p = RecParams()
+    p.q, p.k, p.v, p.z = _p(q), _p(k), _p(v), _p(z)
+    p.ldq, p.ldk, p.ldv, p.ldz = q.stride(0), k.stride(0), v.stride(0), z.stride(0) if z is not None else 0
+    p.decay, p.w0, p.u, p.state, p.out = _p(decay), _p(w0), _p(u), _p(state), _p(out)
+    p.H, p.d, p.dv, p.rows = H, d, dv, step_rows(inp, T)
+    multi = 0
+    hold = None
+    if inp.is_prefill:
+        p.seg_seq, p.seg_q0, p.nseg, p.seg_len = _p(inp.seg_seq), _p(inp.seg_q0), inp.seg_seq.shape[0], inp.seg_len
+        multi = int(p.nseg > p.rows.B)
+        if multi:
+            hold = torch.empty(p.nseg * H * d * (dv + 1), dtype=torch.float32, device=q.device)
+            p.seg_state, p.seg_decay = _p(hold), hold.data_ptr() + 4 * p.nseg * H * d * dv
+    nv._check(nv.load().lx_recurrence(ctypes.byref(p), mode, multi, _f32(q), nv._stream()), "lx_recurrence")
+    nv.launch_count += (1 if p.rows.nd and p.rows.B else 0) + 2 * multi
+    return out
+
+
+def linear_attn(q, k, v, H: int, d: int, dv: int, decay, state, inp):
+    return _recurrence(0, q, k, v, None, decay, None, None, H, d, dv, state, inp)
+
+
+def wkv(r, k, v, z, w0, u, H: int, d: int, state, inp):
+    return _recurrence(1, r, k, v, z, None, w0, u, H, d, d, state, inp)
+
+
+def token_shift(h, mu, shift, inp):
+    T, W = h.shape
+    out = torch.empty(mu.shape[0], T, W, dtype=h.dtype, device=h.device)
+    rows = step_rows(inp, T)
+    nv._check(nv.load().lx_token_shift(_p(h), _p(mu), _p(shift), _p(out), mu.shape[0], W, T, ctypes.byref(rows), _f32(h), nv._stream()),
+              "lx_token_shift")
+    nv.launch_count += int(rows.B > 0)
+    return out
+
+
+def latent_prep(dq, dkv, dq_norm, dkv_norm, q_rank: int, kv_rank: int, rot: int, eps: float, cos_sin, positions, slots, cache):
+    T, QR, KR = dq.shape[0], dq_norm.shape[0], dkv_norm.shape[0]
+    cq = torch.empty(T, QR, dtype=dq.dtype, device=dq.device)
+    p = LatentPrepParams(_p(dq), _p(dkv), dq.stride(0), dkv.stride(0), _p(dq_norm), _p(dkv_norm), _p(cq), _p(cache), _p(positions), _p(slots),
+                         _p(cos_sin), QR, KR, cache.shape[2], q_rank, kv_rank, rot, eps)
+    nv._check(nv.load().lx_latent_prep(ctypes.byref(p), T, _f32(dq), nv._stream()), "lx_latent_prep")
+    return cq
+
+
+def rope_pairs(x, positions, cos_sin, H: int, head: int, off: int, rot: int):
+    nv._check(nv.load().lx_rope_pairs(_p(x), x.stride(0), _p(positions), _p(cos_sin), x.shape[0], H, head, off, rot, _f32(x), nv._stream()),
+              "lx_rope_pairs")
+
+
+def latent_attn(q_lat, q, cache, H: int, kv_rank: int, head: int, rot_off: int, rot: int, scale: float, inp):
+    T = q.shape[0]
+    out = torch.empty(T, H * kv_rank, dtype=q.dtype, device=q.device)
+    p = LatentAttnParams()
+    p.q_lat, p.ld_ql, p.q, p.ldq, p.head, p.rot_off = _p(q_lat), q_lat.stride(0), _p(q), q.stride(0), head, rot_off
+    p.cache, p.out, p.ldo, p.rows = _p(cache), _p(out), out.stride(0), step_rows(inp, T)
+    p.H, p.KR, p.R, p.page, p.scale = H, kv_rank, kv_rank + rot, cache.shape[1], scale
+    nv._check(nv.load().lx_latent_attn(ctypes.byref(p), T, _f32(q), nv._stream()), "lx_latent_attn")
+    return out

@@ -200,7 +200,14 @@ def main():
     ap.add_argument("--no-graphs", action="store_true")
     ap.add_argument("--waiting-served-ratio", type=float, default=None, help="scheduler knob (default: the engine's)")
     ap.add_argument("--baseline-mode", action="store_true", help="NCCL collectives instead of the fused NVLink kernels")
+    ap.add_argument("--design", default=None, choices=[None, "vabunex"],
+                    help="instead of the serving benchmark: prefill / decode throughput and kernel times of this design beside the closest "
+                         "uniform decoder (benchmarks/bench_design.py; one JSON line per case)")
+    ap.add_argument("--design-size", default="small,base")
     args = ap.parse_args()
+    if args.design is not None:
+        from benchmarks import bench_design
+        return bench_design.main(args)
     if args.impl == "reference":
         return reference_arm(args)
 

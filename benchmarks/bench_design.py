@@ -1,0 +1,243 @@
+"""Prefill and decode throughput of a layer-by-layer design (random weights, layers of a real model's size) beside the closest
+uniform decoder of this framework at equal size, and the device time of every kernel of both with its share of the roofline.
+
+    python bench.py --design vabunex [--design-size small,base] [--steps K] [--warmup W]
+
+"Equal size": a llama-style decoder with the same width, feed-forward width, number of layer runs and attention heads of 128.
+Throughput: prefill is one eager forward pass over ragged prompts, decode one CUDA-graph replay per token, both through
+`ModelRunner`, timed with CUDA events.  Kernel times: CUDA events around every operator of an eager pass, L2 flushed in front of it,
+median of the passes.  Rooflines: the measured copy bandwidth and bf16 rate of MEASURED_PEAKS.json, whichever bounds the operator.
+"""
+
+from __future__ import annotations
+
+import json
+import os
+import statistics
+
+REPO = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+
+SIZES = {
+    # width, ff, recurrent heads x dim, wkv heads x dim, latent heads, q rank, kv rank, rot
+    "small": dict(width=2048, ff=8192, lin=(16, 128), wkv=(32, 64), heads=16, q_rank=1024, kv_rank=512, rot=64),
+    "base": dict(width=4096, ff=14336, lin=(32, 128), wkv=(64, 64), heads=32, q_rank=1536, kv_rank=512, rot=64),
+}
+PREFILL = [(1, 4096), (4, 2048), (1, 16384)]           # (prompts, tokens each)
+DECODE = [(16, 2048), (64, 2048), (256, 2048)]         # (rows, tokens of context)
+
+
+def vabunex_config(s, vocab=32000):
+    H, d = s["lin"]
+    wh, wd = s["wkv"]
+    decay = [1.0 - 2.0 ** (-3 - 7 * h / max(H - 1, 1)) for h in range(H)]
+    lin = dict(type="lightning", mixer=dict(heads=H, dim=d, vdim=d, decay=decay), mlp=dict(kind="dense", ff=s["ff"]))
+    wkv = dict(type="wkv", mixer=dict(heads=wh, dim=wd), mlp=dict(kind="dense", ff=s["ff"]))
+    lat = dict(type="latent_attention", mlp=dict(kind="dense", ff=s["ff"]),
+               mixer=dict(heads=s["heads"], dim=128, rot_dim=s["rot"], vdim=128, q_rank=s["q_rank"], kv_rank=s["kv_rank"],
+                          scale=(128 + s["rot"]) ** -0.5, rot=dict(base=10000.0, dims=s["rot"])))
+    return dict(architecture="Vabunex", vocab=vocab, width=s["width"], norm=dict(eps=1e-5), embedding=dict(scale=1.0),
+                layers=[lin, wkv, lat, wkv], loop=dict(start=1, stop=3, times=2))
+
+
+def llama_like(s, runs, vocab=32000):
+    from lorax_b200.config import ModelConfig
+    heads = s["width"] // 128
+    return ModelConfig(model_type="llama", vocab_size=vocab, hidden_size=s["width"], intermediate_size=s["ff"], num_hidden_layers=runs,
+                       num_attention_heads=heads, num_key_value_heads=max(heads // 4, 1), head_dim=128, max_position_embeddings=32768)
+
+
+def peaks():
+    try:
+        with open(os.path.join(REPO, "MEASURED_PEAKS.json")) as f:
+            p = json.load(f)
+        return p["hbm_gbs"] * 1e9, p["bf16_tflops"] * 1e12, "of measured"
+    except (OSError, KeyError, ValueError):
+        return 6.65e12, 1.59e15, "of fallback"
+
+
+class OpTimer:
+    """Wraps the operators of `ops.native` for eager passes: flush L2, event, call, event; knows each operator's algorithmic bytes
+    and FLOPs."""
+
+    FLUSH_BYTES = 256 << 20
+
+    def __init__(self, native, names, inp_info):
+        import torch
+        self.nv, self.names, self.info = native, names, inp_info
+        self.flush = torch.empty(self.FLUSH_BYTES, dtype=torch.uint8, device="cuda")
+        self.records, self.saved = [], {}
+
+    def __enter__(self):
+        import torch
+
+        def wrap(name, fn):
+            def timed(*a, **kw):
+                self.flush.zero_()
+                s, e = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+                s.record()
+                out = fn(*a, **kw)
+                e.record()
+                self.records.append((name, self.cost(name, a, kw), s, e))
+                return out
+            return timed
+        for n in self.names:
+            self.saved[n] = getattr(self.nv, n)
+            setattr(self.nv, n, wrap(n, self.saved[n]))
+        return self
+
+    def __exit__(self, *exc):
+        for n, fn in self.saved.items():
+            setattr(self.nv, n, fn)
+
+    def cost(self, name, a, kw):
+        """(label, bytes, flops) of one call."""
+        nb = lambda *ts: sum(t.numel() * t.element_size() for t in ts if t is not None)
+        q = self.info                                       # rows, causal (query, key) pairs, cached tokens read, sequences, decode?
+        if name == "gemm":
+            x, w = a[0], a[1]
+            return (f"gemm [{x.shape[0]}, {w.shape[1]}] x [{w.shape[0]}]", nb(x, w) + x.shape[0] * w.shape[0] * 2, 2 * x.shape[0] * w.numel())
+        if name == "gemm_stack":
+            x, w = a
+            return ("gemm_stack", nb(x, w) + x.shape[0] * x.shape[1] * w.shape[1] * 2, 2 * x.shape[1] * w.numel())
+        if name == "gemm_heads":
+            x, w, out = a[:3]
+            H, N, K = w.shape
+            return (f"gemm_heads {N}x{K}", nb(w) + x.shape[0] * H * (N + K) * 2, 2 * x.shape[0] * w.numel())
+        if name in ("linear_attn", "wkv"):
+            H, d = (a[3], a[4]) if name == "linear_attn" else (a[6], a[7])
+            dv = a[5] if name == "linear_attn" else d
+            T = a[0].shape[0]
+            io = T * H * (2 * d + dv) * 2 + T * H * dv * 4 + (T * H * d * 2 if name == "wkv" else 0)
+            st = q["seqs"] * H * d * dv * 4 * (2 if q["decode"] else 1)
+            return (name, io + st, 0)
+        if name == "latent_attn":
+            H, kv, rot = a[3], a[4], a[7]
+            T = a[0].shape[0]
+            if q["decode"]:                                 # absorbed: rows of the cache against every head
+                return (name, q["ctx"] * (kv + rot) * 2 + T * H * (2 * kv + rot) * 2, 2 * q["ctx"] * H * (2 * kv + rot))
+            return (name, 0, 2 * q["pairs"] * H * (128 + rot + 128))       # the products of plain multi-head attention
+        if name == "attn_decode":
+            nh, nkv, d = a[4], a[5], a[6]
+            return (name, q["ctx"] * nkv * 2 * d * 2 + a[0].shape[0] * nh * d * 4, 4 * q["ctx"] * nh * d)
+        if name == "attn_prefill":
+            nh, d = a[7], a[9]
+            return (name, 0, 4 * q["pairs"] * nh * d)
+        if name == "norm_stream":
+            r, pend = a[0], a[1]
+            return (name, nb(r) * (2 if pend is not None else 1) + nb(pend) + r.numel() * 2, 0)
+        if name == "norm_residual":
+            return (name, nb(a[0]) * 2 + nb(a[1]) * 2, 0)
+        if name == "norm_gate":
+            return (name, nb(a[0]) + a[0].numel() * 4, 0)
+        if name == "token_shift":
+            return (name, nb(a[0]) * (1 + a[1].shape[0]), 0)
+        if name == "act_mul":
+            return (name, a[0].shape[0] * a[1] * 6, 0)
+        if name == "rope_kvwrite":
+            T, nh, nkv, d = a[0].shape[0], a[5], a[6], a[7]
+            return (name, T * (2 * (nh + nkv) * d + 3 * nkv * d) * 2, 0)
+        if name == "latent_prep":
+            return (name, a[0].shape[0] * (a[2].shape[0] * 2 + a[3].shape[0] * 2) * 2, 0)
+        if name == "rope_pairs":
+            return (name, a[0].shape[0] * a[3] * a[6] * 4, 0)
+        if name in ("embed", "embed_stream"):
+            return (name, a[0].shape[0] * a[1].shape[1] * (6 if name == "embed_stream" else 4), 0)
+        return (name, nb(*[t for t in a if hasattr(t, "numel")]), 0)
+
+    def report(self, bw, fl):
+        import torch
+        torch.cuda.synchronize()
+        agg = {}
+        for name, (label, nbytes, flops), s, e in self.records:
+            agg.setdefault(label, []).append((s.elapsed_time(e) * 1e3, nbytes, flops))
+        rows = []
+        for label, xs in agg.items():
+            us = statistics.median(x[0] for x in xs)
+            best = max(xs[0][1] / bw, xs[0][2] / fl) * 1e6
+            rows.append((label, len(xs), round(us, 1), round(best / us, 3)))
+        return sorted(rows, key=lambda r: -r[1] * r[2])
+
+
+OPS = ("gemm", "norm_residual", "rope_kvwrite", "act_mul", "embed", "attn_decode", "attn_prefill", "embed_stream", "norm_stream", "norm_gate",
+       "tanh_", "gemm_heads", "gemm_stack", "linear_attn", "wkv", "token_shift", "latent_prep", "rope_pairs", "latent_attn", "argmax_logprob")
+
+
+def main(args):
+    import torch
+    from lorax_b200.config import EngineConfig, ModelConfig
+    from lorax_b200.models.decoder import DecoderModel
+    from lorax_b200.ops import native
+    from lorax_b200.runtime.kv_cache import make_cache
+    from lorax_b200.runtime.runner import ModelRunner, PrefillItem
+    if not torch.cuda.is_available():
+        print(json.dumps({"error": "bench.py needs a CUDA device"}))
+        return 1
+    dev = torch.device("cuda", 0)
+    bw, fl, of = peaks()
+    steps, warm = min(args.steps, 50), max(3, min(args.warmup, 10))
+    from bench import ClockSampler
+    results = []
+    with torch.inference_mode():
+        for size in args.design_size.split(","):
+            s = SIZES[size]
+            ours = ModelConfig.from_dict(vabunex_config(s))
+            for name, cfg in ((args.design, ours), ("llama-like", llama_like(s, len(ours.layer_schedule)))):
+                model = DecoderModel.random_init_on_device(cfg, dev, torch.bfloat16, seed=0, max_positions=20000)
+                model.use_native_layers = True
+                for kind, cases in (("prefill", PREFILL), ("decode", DECODE)):
+                    for n, length in cases:
+                        total = length + (8 + 2 * (steps + warm) if kind == "decode" else 0)
+                        pages = (total + 31) // 32 + 1
+                        kv = make_cache(model, EngineConfig(), n * pages + 1, n, num_slots=n + 1)
+                        run = ModelRunner(model, kv, max_batch=n, max_seq_tokens=total + 32, max_prefill_tokens=max(n * length, 64))
+                        blocks = [list(range(1 + i * pages, 1 + (i + 1) * pages)) for i in range(n)]
+                        g = torch.Generator().manual_seed(1)
+                        items = [PrefillItem(torch.randint(0, cfg.vocab_size, (length,), generator=g).tolist(), 0, blocks[i], state_slot=i + 1)
+                                 for i in range(n)]
+                        if kind == "decode":
+                            # (the contents of caches and states do not matter for the time: no prompt is run)
+                            rows = [run.state.take_row(i) for i in range(n)]
+                            run.install(rows, [5] * n, [length] * n, blocks, [0] * n, list(range(1, n + 1)))
+                            run.resort()
+                            step = lambda: run.decode()
+                            info = dict(decode=True, seqs=n, ctx=n * length, pairs=n * length)
+                            toks = n
+                        else:
+                            inp, _ = run._prefill_inputs(items)
+                            step = lambda: model.forward(inp, kv.layers)
+                            info = dict(decode=False, seqs=n, ctx=n * length, pairs=n * length * (length + 1) // 2)
+                            toks = n * length
+                        for _ in range(warm):
+                            step()
+                        torch.cuda.synchronize()
+                        clk = ClockSampler(0, 0.05)
+                        clk.start()
+                        k = steps if kind == "decode" else max(3, min(steps, 10))
+                        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+                        e0.record()
+                        for _ in range(k):
+                            step()
+                        e1.record()
+                        torch.cuda.synchronize()
+                        clocks = clk.stop()
+                        ms = e0.elapsed_time(e1) / k
+                        # per operator, eager, one launch at a time
+                        model.use_native_layers = False
+                        graphs, run.use_graphs = run.use_graphs, False
+                        with OpTimer(native, OPS, info) as tm:
+                            for _ in range(3):
+                                step()
+                            kernels = tm.report(bw, fl)
+                        run.use_graphs, model.use_native_layers = graphs, True
+                        native.workspace(dev).check_status()
+                        r = {"design": name, "size": size, "kind": kind, "sequences": n, "tokens": length, "ms": round(ms, 3),
+                             "tok_s": round(toks / ms * 1e3, 1), "layer_runs": len(model.schedule), "roofline": of,
+                             "clocks": {c: clocks[c] for c in ("sm_mhz", "sm_max_mhz", "reasons")},
+                             "kernels": [dict(op=a, calls=b // 3, us=c, roofline=d) for a, b, c, d in kernels]}
+                        results.append(r)
+                        print(json.dumps(r), flush=True)
+                        del run, kv, step
+                        torch.cuda.empty_cache()
+                del model
+                torch.cuda.empty_cache()
+    return 0

@@ -114,13 +114,24 @@ class StepInputs:
     seg_seq: Optional[torch.Tensor] = None
     seg_q0: Optional[torch.Tensor] = None
     seg_len: int = 0
-    max_ctx: int = 0                                 # longest context of the prefill sequences (host knowledge; 0: unknown)
+    # latent attention over prompts: 128-query tiles (sequence, first query), and the contexts of the prefill sequences laid end to end
+    q128_seq: Optional[torch.Tensor] = None
+    q128_q0: Optional[torch.Tensor] = None
+    ctx_off: Optional[torch.Tensor] = None           # [B + 1]
+    ctx_total: int = 0
 
     def decode_view(self, T: int):
         """(decode rows, their block tables, state slots, context lengths) of a step over T rows."""
         if not self.is_prefill:
             return T, self.block_tables, self.state_slots, self.ctx_lens
         return self.n_decode, self.dec_block_tables, self.dec_state_slots, self.ctx_lens
+
+    def decode_rows(self) -> "StepInputs":
+        """The decode rows of a mixed step as a step of their own."""
+        n = self.n_decode
+        return StepInputs(input_ids=self.input_ids[:n], positions=self.positions[:n], slots=self.slots[:n], is_prefill=False,
+                          block_tables=self.dec_block_tables, ctx_lens=self.ctx_lens, attn_nsplit=self.attn_nsplit,
+                          state_slots=self.dec_state_slots)
 
 
 class DecoderModel:

@@ -199,6 +199,10 @@ class LatentAttentionMixer(Mixer):
                       .reshape(H * (self.dp + self.rp), self.qrp))
         self.uk_t = fin(_pad_to(get("uk").view(H, d, self.kv_rank).transpose(1, 2), H, self.kvp, self.dp))     # [H, kv_rank, dim]
         self.uv = fin(_pad_to(get("uv").view(H, dv, self.kv_rank), H, self.dvp, self.kvp))                     # [H, vdim, kv_rank]
+        # the expansion of prompts: every head's key rows, then its value rows
+        self.ukv = fin(torch.cat([_pad_to(get("uk").view(H, d, self.kv_rank), H, self.dp, self.kvp),
+                                  _pad_to(get("uv").view(H, dv, self.kv_rank), H, self.dvp, self.kvp)], 1)
+                       .reshape(H * (self.dp + self.dvp), self.kvp))
         self.dq_norm = vec(_pad_to(get("dq.norm"), self.qrp))
         self.dkv_norm = vec(_pad_to(get("dkv.norm"), self.kvp))
         self.cos_sin = model.rope_table(self.rot, self.rot_base)
@@ -213,10 +217,17 @@ class LatentAttentionMixer(Mixer):
                              self.cos_sin, inp.positions, inp.slots, cache)
         q = ops.gemm(cq, self.uq)
         ops.rope_pairs(q, inp.positions, self.cos_sin, self.H, head, self.dp, self.rot)
+        gate = proj["g"]
+        if inp.is_prefill and ops.latent_prefill(q, cache, self.ukv, gate, y, self.H, self.dp, self.rp, self.dvp, self.scale, inp, inp.n_decode):
+            if inp.n_decode == 0:
+                return
+            inp = inp.decode_rows()                          # the decode rows of a mixed step are left
+            n = inp.input_ids.shape[0]
+            q, gate, y = q[:n], gate[:n], y[:n]
         q_lat = torch.empty(q.shape[0], self.H * self.kvp, dtype=q.dtype, device=q.device)
         ops.gemm_heads(q, self.uk_t, q_lat, head)
         o_lat = ops.latent_attn(q_lat, q, cache, self.H, self.kvp, head, self.dp, self.rp, self.scale, inp)
-        ops.gemm_heads(o_lat, self.uv, y, self.kvp, gate=proj["g"])
+        ops.gemm_heads(o_lat, self.uv, y, self.kvp, gate=gate)
 
 
 MIXERS = {"lightning": LightningMixer, "wkv": WkvMixer, "latent_attention": LatentAttentionMixer}

@@ -685,13 +685,13 @@ def lora_expand_tiles(v, tiles: torch.Tensor, num_tiles: int, max_tile_rows: int
 
 # ------------------------------------------------------------------------------------------------ layer-by-layer designs
 from .native_mixers import (embed_stream, gemm_f32, gemm_heads, gemm_stack, latent_attn, latent_prep, linear_attn, norm_gate,  # noqa: E402
-                            norm_stream, rope_pairs, tanh_, token_shift, wkv)
+                            latent_prefill, norm_stream, rope_pairs, tanh_, token_shift, wkv)
 
 # ------------------------------------------------------------------------------------------------ per-op timing
 _TIMED_OPS = ("gemm", "gemm_fp8", "norm_residual", "rope_kvwrite", "act_mul", "embed", "argmax_logprob", "advance_decode", "attn_decode",
               "attn_prefill", "lora_shrink", "lora_expand", "lora_shrink_tiles", "lora_expand_tiles",
               "embed_stream", "norm_stream", "norm_gate", "tanh_", "gemm_heads", "linear_attn", "wkv", "token_shift", "latent_prep", "rope_pairs",
-              "latent_attn")
+              "latent_attn", "latent_prefill")
 _timing_records = None
 _timing_originals = {}
 

@@ -53,6 +53,9 @@ SIGNATURES = {
     "lx_latent_prep": ([P, I, I, P], I),
     "lx_rope_pairs": ([P, L, P, P, I, I, I, I, I, I, P], I),
     "lx_latent_attn": ([P, I, I, P], I),
+    "lx_latent_gather": ([P, P, I, P, I, I, I, I, I, P, P, P], I),
+    "lx_latent_prefill_supported": ([I, I, I], I),
+    "lx_latent_prefill": ([P, L, I, P, P, I, P, P, P, P, P, I, P, L, P, L, I, I, I, I, F, P, P], I),
 }
 
 
@@ -202,3 +205,29 @@ def latent_attn(q_lat, q, cache, H: int, kv_rank: int, head: int, rot_off: int, 
     p.H, p.KR, p.R, p.page, p.scale = H, kv_rank, kv_rank + rot, cache.shape[1], scale
     nv._check(nv.load().lx_latent_attn(ctypes.byref(p), T, _f32(q), nv._stream()), "lx_latent_attn")
     return out
+
+
+# mean prompt tokens per sequence from which a prompt expands its latents to keys and values instead of being carried into the
+# latent space row by row (the expansion costs a row of the context about as much as twenty queries save on it)
+LATENT_EXPAND_MIN_ROWS = 24
+
+
+def latent_prefill(q, cache, w_ukv, gate, out, H: int, dk: int, rot: int, dv: int, scale: float, inp, nd: int) -> bool:
+    """Gated attention outputs of the prompt rows [nd, T) into out[nd:, : H * dv] on the tensor-core kernel; False when this step is
+    better (or only) served by the absorbed form."""
+    T, B = q.shape[0] - nd, inp.cache_lens.shape[0]
+    lib = nv.load()
+    if q.dtype != torch.bfloat16 or T < LATENT_EXPAND_MIN_ROWS * B or not lib.lx_latent_prefill_supported(dk, rot, dv):
+        return False
+    rows, KR, dev = inp.ctx_total, cache.shape[2] - rot, q.device
+    lat = torch.empty(rows, KR, dtype=q.dtype, device=dev)
+    keys = torch.empty(rows, rot, dtype=q.dtype, device=dev)
+    nv._check(lib.lx_latent_gather(_p(cache), _p(inp.block_tables), inp.block_tables.shape[1], _p(inp.ctx_off), B, rows, cache.shape[1], KR, rot,
+                                   _p(lat), _p(keys), nv._stream()), "lx_latent_gather")
+    kv = nv.gemm(lat, w_ukv)
+    y, g = out[nd:], gate[nd:]
+    qp = q[nd:]
+    nv._check(lib.lx_latent_prefill(_p(qp), qp.stride(0), T, _p(kv), _p(keys), rows, _p(inp.ctx_off), _p(inp.cu_q), _p(inp.cache_lens),
+                                    _p(inp.q128_seq), _p(inp.q128_q0), inp.q128_seq.shape[0], _p(g), g.stride(0), _p(y), y.stride(0), H, dk, rot,
+                                    dv, scale, _p(nv.workspace(dev).status), nv._stream()), "lx_latent_prefill")
+    return True

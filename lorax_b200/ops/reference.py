@@ -611,7 +611,12 @@ def gemm_heads(x, w, out, x_head: int, gate=None):
     return out
 
 
-def latent_attn(q_lat, q, cache, H: int, kv_rank: int, head: int, rot_off: int, rot: int, scale: float, inp, w_uk=None, w_uv=None):
+def latent_prefill(q, cache, w_ukv, gate, out, H: int, dk: int, rot: int, dv: int, scale: float, inp, nd: int) -> bool:
+    """The expanded form of prompt attention exists on the device only; False sends the rows through `latent_attn`."""
+    return False
+
+
+def latent_attn(q_lat, q, cache, H: int, kv_rank: int, head: int, rot_off: int, rot: int, scale: float, inp):
     """Causal softmax attention in the latent space: head h's query is [q_lat[h] | q[h, rot_off : rot_off + rot]] against the
     cached rows [latent | rotated key].  -> weighted latents [T, H * kv_rank]."""
     T = q.shape[0]

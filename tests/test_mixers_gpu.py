@@ -1,0 +1,259 @@
+"""Kernels of the layer-by-layer designs against the PyTorch statement of the same operator (`ops.reference`), in bf16 and in fp32."""
+
+import pytest
+import torch
+
+pytestmark = pytest.mark.gpu
+PAGE = 32
+DTYPES = (torch.bfloat16, torch.float32)
+
+
+def make_step(dec, pre, slots=None, seg_len=64, seed=0, pages_per_seq=None):
+    """StepInputs (on the CPU) of decode rows with contexts `dec` and prompt portions `pre` = [(tokens before, tokens)], over shuffled
+    pages and state slots.  -> (inp, number of blocks, number of state slots)"""
+    from lorax_b200.models.decoder import StepInputs
+    from lorax_b200.ops import reference
+    g = torch.Generator().manual_seed(seed)
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32)
+    spans = [(max(c - 1, 0), 1) for c in dec] + list(pre)
+    width = pages_per_seq or max((b + n + PAGE - 1) // PAGE for b, n in spans) + 1
+    blocks = (1 + torch.randperm(width * len(spans), generator=g)).view(len(spans), width).to(torch.int32)
+    sl = (1 + torch.randperm(len(spans), generator=g)).to(torch.int32)
+    nd = len(dec)
+    pos, slot = [], []
+    for i, (b, n) in enumerate(spans):
+        for t in range(b, b + n):
+            pos.append(t)
+            dead = i < nd and dec[i] <= 0
+            slot.append(-1 if dead else int(blocks[i, t // PAGE]) * PAGE + t % PAGE)
+    T = len(pos)
+    kw = dict(input_ids=torch.zeros(T, dtype=torch.int32), positions=i32(pos), slots=i32(slot))
+    if not pre:
+        inp = StepInputs(is_prefill=False, block_tables=blocks, ctx_lens=i32(dec), state_slots=sl, **kw)
+    else:
+        q = [n for _, n in pre]
+        cu, off = [0], [0]
+        for b, n in pre:
+            cu.append(cu[-1] + n)
+            off.append(off[-1] + b + n)
+        ss, s0 = reference.prefill_tiles(q, seg_len)
+        ts, t0 = reference.prefill_tiles(q, 128)
+        inp = StepInputs(is_prefill=True, block_tables=blocks[nd:].contiguous(), cu_q=i32(cu), cache_lens=i32([b for b, _ in pre]),
+                         state_slots=sl[nd:].contiguous(), n_decode=nd, dec_block_tables=blocks[:nd].contiguous(), ctx_lens=i32(dec),
+                         dec_state_slots=sl[:nd].contiguous(), seg_seq=i32(ss), seg_q0=i32(s0), seg_len=seg_len, q128_seq=i32(ts),
+                         q128_q0=i32(t0), ctx_off=i32(off), ctx_total=off[-1], **kw)
+    return inp, width * len(spans) + 1, len(spans) + 1
+
+
+def to_dev(x):
+    import dataclasses
+    if isinstance(x, torch.Tensor):
+        return x.cuda()
+    return dataclasses.replace(x, **{f.name: getattr(x, f.name).cuda() for f in dataclasses.fields(x)
+                                     if isinstance(getattr(x, f.name), torch.Tensor)})
+
+
+def close(got, want, dtype, rows=None, tol16=2e-2, tol32=2e-5):
+    got, want = got.float().cpu(), want.float()
+    if rows is not None:
+        got, want = got[rows], want[rows]
+    assert torch.isfinite(got).all()
+    err = (got - want).norm() / want.norm().clamp_min(1e-6)
+    worst = (got - want).abs().max() / want.abs().max().clamp_min(1e-6)
+    tol = tol32 if dtype == torch.float32 else tol16
+    assert err < tol and worst < 4 * tol, (float(err), float(worst))
+
+
+STEPS = {
+    "decode": ([1, 2, 33, 0, 700], []),
+    "prompts": ([], [(0, 1), (0, 64), (0, 65), (0, 300), (31, 2), (64, 130)]),
+    "mixed": ([5, 0, 64, 1], [(0, 129), (70, 3), (200, 64), (1, 2)]),
+}
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("step", list(STEPS))
+@pytest.mark.parametrize("H,d,dv", [(3, 16, 48), (2, 64, 32), (4, 128, 128), (1, 256, 80), (2, 48, 144)])
+def test_linear_attention_recurrence(dtype, step, H, d, dv):
+    from lorax_b200.ops import native, reference
+    inp, _, ns = make_step(*STEPS[step])
+    T = inp.positions.shape[0]
+    g = torch.Generator().manual_seed(1)
+    x = torch.randn(T, H * (2 * d + dv), generator=g).to(dtype)
+    decay = torch.linspace(0.3, 0.9995, H)
+    if H > 2:
+        decay[0], decay[1] = 0.0, 1.0
+    state = torch.randn(ns, H, d, dv, generator=g)
+    q, k, v = x[:, : H * d], x[:, H * d: 2 * H * d], x[:, 2 * H * d:]
+    st = state.clone()
+    want = reference.linear_attn(q.float(), k.float(), v.float(), H, d, dv, decay, st, inp)
+    xd, sd = x.cuda(), state.cuda()
+    got = native.linear_attn(xd[:, : H * d], xd[:, H * d: 2 * H * d], xd[:, 2 * H * d:], H, d, dv, decay.cuda(), sd, to_dev(inp))
+    live = [i for i in range(T) if i >= len(STEPS[step][0]) or STEPS[step][0][i] > 0]
+    close(got, want, dtype, live, tol16=6e-3)
+    close(sd, st, dtype, tol16=6e-3)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("step", list(STEPS))
+@pytest.mark.parametrize("H,d,strong", [(3, 16, False), (2, 64, False), (2, 64, True), (1, 128, False), (2, 80, True), (1, 256, False)])
+def test_wkv_recurrence(dtype, step, H, d, strong):
+    """`strong`: decays so strong (and so weak) that products over a few tokens under- and overflow unless they are formed safely."""
+    from lorax_b200.ops import native, reference
+    inp, _, ns = make_step(*STEPS[step], seed=3)
+    T, C = inp.positions.shape[0], H * d
+    g = torch.Generator().manual_seed(2)
+    r, k, v, z = (torch.randn(T, C, generator=g).to(dtype) for _ in range(4))
+    w0 = torch.randn(C, generator=g) * (3.0 if strong else 1.0) + (1.0 if strong else -2.0)
+    u = torch.randn(C, generator=g)
+    state = torch.randn(ns, H, d, d, generator=g)
+    st = state.clone()
+    want = reference.wkv(r.float(), k.float(), v.float(), z.float(), w0, u, H, d, st, inp)
+    sd = state.cuda()
+    got = native.wkv(r.cuda(), k.cuda(), v.cuda(), z.cuda(), w0.cuda(), u.cuda(), H, d, sd, to_dev(inp))
+    live = [i for i in range(T) if i >= len(STEPS[step][0]) or STEPS[step][0][i] > 0]
+    close(got, want, dtype, live, tol16=2e-4)
+    close(sd, st, dtype, tol16=2e-4)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("step", list(STEPS))
+def test_token_shift(dtype, step):
+    from lorax_b200.ops import native, reference
+    inp, _, ns = make_step(*STEPS[step], seed=4)
+    T, W = inp.positions.shape[0], 112
+    g = torch.Generator().manual_seed(2)
+    h, mu, shift = torch.randn(T, W, generator=g).to(dtype), torch.rand(5, W, generator=g), torch.randn(ns, W, generator=g).to(dtype)
+    sh = shift.clone()
+    want = reference.token_shift(h, mu, sh, inp)
+    sd = shift.cuda()
+    got = native.token_shift(h.cuda(), mu.cuda(), sd, to_dev(inp))
+    live = [i for i in range(T) if i >= len(STEPS[step][0]) or STEPS[step][0][i] > 0]
+    assert torch.equal(sd.cpu(), sh)
+    assert torch.allclose(got.cpu().float()[:, live], want.float()[:, live], atol=2e-2 if dtype == torch.bfloat16 else 1e-6)
+
+
+def latent_case(H, dk, rot, dv, kv, inp, nb, dtype, peak, seed=5):
+    """Random queries, cache and expansion weights.  `peak`: every query matches one far key of its own context far better than all
+    others, so a key that is lost or misplaced shows."""
+    g = torch.Generator().manual_seed(seed)
+    T = inp.positions.shape[0]
+    q = torch.randn(T, H * (dk + rot), generator=g).to(dtype)
+    cache = torch.randn(nb, PAGE, kv + rot, generator=g).to(dtype)
+    uk, uv = torch.randn(H, dk, kv, generator=g) * kv ** -0.5, torch.randn(H, dv, kv, generator=g) * kv ** -0.5
+    if peak:
+        nd, dbt, _, ctx = inp.decode_view(T)
+        for t in range(T):
+            if t < nd:
+                bt, keys = dbt[t], int(ctx[t])
+            else:
+                b = int(torch.searchsorted(inp.cu_q[1:], torch.tensor(t - nd), right=True))
+                bt, keys = inp.block_tables[b], int(inp.cache_lens[b]) + (t - nd - int(inp.cu_q[b])) + 1
+            if keys <= 0:
+                continue
+            j = (0, keys - 1, keys // 3, keys // 32 * 32, max(keys // 32 * 32 - 1, 0))[t % 5]
+            j = min(j, keys - 1)
+            kr = cache[int(bt[j // PAGE]), j % PAGE, kv:].float()
+            q.view(T, H, dk + rot)[t, :, dk:] = (kr * 2.0).to(dtype)
+    return q, cache, uk.to(dtype), uv.to(dtype)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("peak", [False, True])
+@pytest.mark.parametrize("step", list(STEPS) + ["long"])
+@pytest.mark.parametrize("H,dk,rot,dv,kv", [(3, 32, 16, 48, 80), (2, 128, 64, 128, 512), (5, 64, 64, 64, 256), (17, 64, 64, 128, 128)])
+def test_latent_attention(dtype, peak, step, H, dk, rot, dv, kv):
+    """Absorbed and expanded form, decode rows, portions and whole prompts: gated outputs against the fp32 statement."""
+    from lorax_b200.ops import native, reference
+    dec, pre = STEPS[step] if step in STEPS else ([1000, 1500], [(1000, 300), (0, 500), (129, 40)])
+    inp, nb, _ = make_step(dec, pre, seed=6)
+    T = inp.positions.shape[0]
+    q, cache, uk, uv = latent_case(H, dk, rot, dv, kv, inp, nb, dtype, peak)
+    gate = torch.randn(T, 32, generator=torch.Generator().manual_seed(9)).to(dtype)
+    scale = (dk + rot) ** -0.5
+    head = dk + rot
+    ql = torch.empty(T, H * kv)
+    reference.gemm_heads(q.float(), uk.float().transpose(1, 2).contiguous(), ql, head)
+    o = reference.latent_attn(ql, q.float(), cache.float(), H, kv, head, dk, rot, scale, inp)
+    want = torch.zeros(T, H * dv)
+    reference.gemm_heads(o, uv.float(), want, kv, gate=gate.float())
+    live = [i for i in range(T) if i >= len(dec) or dec[i] > 0]
+
+    d = to_dev(inp)
+    qd, cd, gd = q.cuda(), cache.cuda(), gate.cuda()
+    qld = torch.empty(T, H * kv, dtype=dtype, device="cuda")
+    native.gemm_heads(qd, uk.transpose(1, 2).contiguous().cuda(), qld, head)
+    od = native.latent_attn(qld, qd, cd, H, kv, head, dk, rot, scale, d)
+    got = torch.zeros(T, H * dv, dtype=dtype, device="cuda")
+    native.gemm_heads(od, uv.cuda(), got, kv, gate=gd)
+    close(got, want, dtype, live)
+    if pre:
+        ukv = torch.cat([uk, uv], 1).reshape(H * (dk + dv), kv).contiguous().cuda()
+        out = torch.zeros(T, H * dv, dtype=dtype, device="cuda")
+        if native.latent_prefill(qd, cd, ukv, gd, out, H, dk, rot, dv, scale, d, len(dec)):
+            native.workspace(out.device).check_status()
+            close(out, want, dtype, list(range(len(dec), T)))
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_latent_preparation_and_rotation(dtype):
+    from lorax_b200.ops import native, reference
+    inp, nb, _ = make_step([7, 0, 40], [(0, 50), (33, 5)], seed=8)
+    T = inp.positions.shape[0]
+    g = torch.Generator().manual_seed(3)
+    qr, kr, rot, rp, H, dk = 96, 80, 10, 16, 3, 32
+    x = torch.randn(T, qr + kr + rp, generator=g).to(dtype)
+    qn, kn = torch.rand(qr, generator=g) + 0.5, torch.rand(kr, generator=g) + 0.5
+    cs = reference.rope_table(rot, 128, 10000.0)
+    cache = torch.zeros(nb, PAGE, kr + rp)
+    want = reference.latent_prep(x[:, :qr].float(), x[:, qr:].float(), qn, kn, 90, 75, rot, 1e-5, cs, inp.positions, inp.slots, cache)
+    xd, cd = x.cuda(), torch.zeros(nb, PAGE, kr + rp, dtype=dtype, device="cuda")
+    got = native.latent_prep(xd[:, :qr], xd[:, qr:], qn.cuda(), kn.cuda(), 90, 75, rot, 1e-5, cs.cuda(), inp.positions.cuda(), inp.slots.cuda(), cd)
+    close(got, want, dtype, tol16=5e-3)
+    close(cd, cache, dtype, tol16=5e-3)
+    q = torch.randn(T, H * (dk + rp), generator=g).to(dtype)
+    qf, qd = q.float(), q.cuda()
+    reference.rope_pairs(qf, inp.positions, cs, H, dk + rp, dk, rot)
+    native.rope_pairs(qd, inp.positions.cuda(), cs.cuda(), H, dk + rp, dk, rot)
+    close(qd, qf, dtype, tol16=5e-3)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("T,W,n", [(1, 16, 9), (5, 208, 200), (67, 4096, 4096), (3, 5120, 5100)])
+def test_stream_norms_and_products(dtype, T, W, n):
+    from lorax_b200.ops import native, reference
+    g = torch.Generator().manual_seed(T)
+    res, pend, w = torch.randn(T, W, generator=g), torch.randn(T, W, generator=g).to(dtype), torch.randn(W, generator=g) * 0.2
+    rd, rf = res.cuda(), res.clone()
+    for p in (None, pend):
+        want = reference.norm_stream(rf, None if p is None else p.float(), w, 1e-5, 1.0, n, torch.float32)
+        got = native.norm_stream(rd, None if p is None else p.cuda(), w.cuda(), 1e-5, 1.0, n, dtype)
+        close(got, want, dtype, tol16=4e-3)
+        assert torch.allclose(rd.cpu(), rf, atol=1e-6)              # the stream itself stays fp32
+    table = torch.randn(50, W, generator=g).to(dtype)
+    ids = torch.randint(0, 50, (T,), generator=g, dtype=torch.int32)
+    assert torch.equal(native.embed_stream(ids.cuda(), table.cuda(), 0.75).cpu(), reference.embed_stream(ids, table, 0.75))
+    for group, act in ((16, "silu"), (W, "sigmoid")):
+        x, gate = torch.randn(T, W, generator=g), torch.randn(T, W, generator=g).to(dtype)
+        out = torch.zeros(T, W + 16, dtype=dtype, device="cuda")
+        want = reference.norm_gate(x, group, group - 3, w, gate.float(), act, 1e-5, torch.zeros(T, W))
+        native.norm_gate(x.cuda(), group, group - 3, w.cuda(), gate.cuda(), act, 1e-5, out[:, :W])
+        close(out[:, :W], want, dtype, tol16=4e-3)
+        assert not out[:, W:].any()
+
+
+@pytest.mark.parametrize("T,N,K", [(1, 640, 192), (7, 48, 16), (130, 200, 96)])
+def test_32_bit_products_and_head(T, N, K):
+    """The fp32 operators: no reduced-precision multiply anywhere."""
+    from lorax_b200.ops import native, reference
+    g = torch.Generator().manual_seed(T)
+    x, w = torch.randn(T, K, generator=g), torch.randn(N, K, generator=g)
+    want = (x.double() @ w.double().t()).float()
+    close(native.gemm(x.cuda(), w.cuda()), want, torch.float32, tol32=2e-6)
+    inter = N // 2 // 4 * 4
+    close(native.act_mul(want.cuda(), inter, "gelu_tanh"), reference.act_mul(want, inter, "gelu_tanh"), torch.float32, tol32=2e-6)
+    ids, lps = native.argmax_logprob(want.cuda())
+    ri, rl = reference.argmax_logprob(want)
+    assert torch.equal(ids.cpu(), ri) and torch.allclose(lps.cpu(), rl, atol=1e-4)
+    t = torch.randn(8, 16, generator=g)
+    assert torch.allclose(native.tanh_(t.cuda()).cpu(), torch.tanh(t), atol=1e-6)

@@ -69,14 +69,21 @@ class OpTimer:
 
     def __enter__(self):
         import torch
+        self.inside = False
 
         def wrap(name, fn):
             def timed(*a, **kw):
+                if self.inside:                             # an operator inside another one belongs to that one's time
+                    return fn(*a, **kw)
+                self.inside = True
                 self.flush.zero_()
                 s, e = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
                 s.record()
                 out = fn(*a, **kw)
                 e.record()
+                self.inside = False
+                if out is False:                            # (the operator declined; nothing was launched)
+                    return out
                 self.records.append((name, self.cost(name, a, kw), s, e))
                 return out
             return timed
@@ -116,6 +123,9 @@ class OpTimer:
             if q["decode"]:                                 # absorbed: rows of the cache against every head
                 return (name, q["ctx"] * (kv + rot) * 2 + T * H * (2 * kv + rot) * 2, 2 * q["ctx"] * H * (2 * kv + rot))
             return (name, 0, 2 * q["pairs"] * H * (128 + rot + 128))       # the products of plain multi-head attention
+        if name == "latent_prefill":                        # expansion of the contexts, then multi-head attention
+            w, H, dk, rot, dv = a[2], *a[5:9]
+            return (name, 0, 2 * q["ctx"] * w.numel() + 2 * q["pairs"] * H * (dk + rot + dv))
         if name == "attn_decode":
             nh, nkv, d = a[4], a[5], a[6]
             return (name, q["ctx"] * nkv * 2 * d * 2 + a[0].shape[0] * nh * d * 4, 4 * q["ctx"] * nh * d)
@@ -159,7 +169,7 @@ class OpTimer:
 
 
 OPS = ("gemm", "norm_residual", "rope_kvwrite", "act_mul", "embed", "attn_decode", "attn_prefill", "embed_stream", "norm_stream", "norm_gate",
-       "tanh_", "gemm_heads", "gemm_stack", "linear_attn", "wkv", "token_shift", "latent_prep", "rope_pairs", "latent_attn", "argmax_logprob")
+       "tanh_", "gemm_heads", "gemm_stack", "linear_attn", "wkv", "token_shift", "latent_prep", "rope_pairs", "latent_attn", "latent_prefill", "argmax_logprob")
 
 
 def main(args):

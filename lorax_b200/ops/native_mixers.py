@@ -36,6 +36,11 @@ class LatentAttnParams(Structure):
                 ("rows", StepRows), ("H", I), ("KR", I), ("R", I), ("page", I), ("scale", F)]
 
 
+class LatentDecodeParams(Structure):
+    _fields_ = [("q_lat", P), ("ld_ql", L), ("q", P), ("ldq", L), ("head", I), ("rot_off", I), ("cache", P), ("out", P), ("ldo", L),
+                ("rows", StepRows), ("H", I), ("R", I), ("page", I), ("nsplit", I), ("scale", F), ("part_o", P), ("part_ml", P)]
+
+
 SIGNATURES = {
     "lx_embed_stream": ([P, P, P, I, I, I, F, I, P], I),
     "lx_norm_stream": ([P, P, P, P, I, I, I, F, F, I, P], I),
@@ -53,6 +58,9 @@ SIGNATURES = {
     "lx_latent_prep": ([P, I, I, P], I),
     "lx_rope_pairs": ([P, L, P, P, I, I, I, I, I, I, P], I),
     "lx_latent_attn": ([P, I, I, P], I),
+    "lx_latent_decode_bytes": ([], I),
+    "lx_latent_decode_supported": ([I, I], I),
+    "lx_latent_decode": ([P, I, I, P], I),
     "lx_latent_gather": ([P, P, I, P, I, I, I, I, I, P, P, P], I),
     "lx_latent_prefill_supported": ([I, I, I], I),
     "lx_latent_prefill": ([P, L, I, P, P, I, P, P, P, P, P, I, P, L, P, L, I, I, I, I, F, P, P], I),
@@ -61,7 +69,7 @@ SIGNATURES = {
 
 def check_layouts(lib):
     for name, st in (("lx_step_rows_bytes", StepRows), ("lx_rec_params_bytes", RecParams), ("lx_latent_prep_bytes", LatentPrepParams),
-                     ("lx_latent_attn_bytes", LatentAttnParams)):
+                     ("lx_latent_attn_bytes", LatentAttnParams), ("lx_latent_decode_bytes", LatentDecodeParams)):
         if getattr(lib, name)() != ctypes.sizeof(st):
             raise nv.NativeError(f"{name}: C++ says {getattr(lib, name)()} bytes, ctypes says {ctypes.sizeof(st)}")
 
@@ -199,6 +207,23 @@ def rope_pairs(x, positions, cos_sin, H: int, head: int, off: int, rot: int):
 def latent_attn(q_lat, q, cache, H: int, kv_rank: int, head: int, rot_off: int, rot: int, scale: float, inp):
     T = q.shape[0]
     out = torch.empty(T, H * kv_rank, dtype=q.dtype, device=q.device)
+    lib = nv.load()
+    if q.dtype == torch.bfloat16 and lib.lx_latent_decode_supported(kv_rank, kv_rank + rot):
+        d = LatentDecodeParams()
+        d.q_lat, d.ld_ql, d.q, d.ldq, d.head, d.rot_off = _p(q_lat), q_lat.stride(0), _p(q), q.stride(0), head, rot_off
+        d.cache, d.out, d.ldo, d.rows = _p(cache), _p(out), out.stride(0), step_rows(inp, T)
+        d.H, d.R, d.page, d.scale = H, kv_rank + rot, cache.shape[1], scale
+        # the keys of a row are shared out until the grid fills the GPU once (one CTA per SM)
+        groups = (H + 31) // 32 if H > 16 else 1
+        d.nsplit = max(1, min(32, nv.workspace(q.device).num_sms // (T * groups)))
+        hold = None
+        if d.nsplit > 1:
+            n = T * H * d.nsplit
+            hold = torch.empty(n * (kv_rank + 2), dtype=torch.float32, device=q.device)
+            d.part_o, d.part_ml = _p(hold), hold.data_ptr() + 4 * n * kv_rank
+        nv._check(lib.lx_latent_decode(ctypes.byref(d), kv_rank, T, nv._stream()), "lx_latent_decode")
+        nv.launch_count += int(d.nsplit > 1)
+        return out
     p = LatentAttnParams()
     p.q_lat, p.ld_ql, p.q, p.ldq, p.head, p.rot_off = _p(q_lat), q_lat.stride(0), _p(q), q.stride(0), head, rot_off
     p.cache, p.out, p.ldo, p.rows = _p(cache), _p(out), out.stride(0), step_rows(inp, T)

@@ -1,0 +1,284 @@
+// Linear attention over prompt segments in chunks of 64 tokens on the tensor cores (bf16 activations, fp32 state).
+//
+// One CTA of four warps = one segment x one head x 64 value columns.  Within a chunk of tokens i, j with decay c:
+//   o_i  = c^(i+1) q_i S + sum_{j <= i} c^(i-j) (q_i . k_j) v_j        S: the state in front of the chunk
+//   S    = c^n S + sum_j c^(n-1-j) k_j v_j^T
+// The state lives in fp32 accumulators.  Whatever is fp32 and enters a product (the state, the decayed weights, the decayed keys) is
+// split into two bf16 terms, value and remainder, and multiplied as two operands; q, k and v are bf16 after their silu anyway.
+// STATES: the segment's own contribution to the state only.
+#include "stream.cuh"
+
+namespace lx {
+
+struct LinTcParams {
+  const __nv_bfloat16* q; const __nv_bfloat16* k; const __nv_bfloat16* v;
+  long long ldq, ldk, ldv;
+  const float* decay;
+  float* state;            // [slots, H, d, dv]
+  float* seg_state;        // [nseg, H, d, dv]
+  float* out;              // [T, H * dv]
+  int H, dv;
+  StepRows rows;
+  const int* seg_seq; const int* seg_q0;
+  int seg_len;
+};
+
+constexpr int kLtC = 64;                        // tokens per chunk
+constexpr int kLtV = 64;                        // value columns per CTA
+constexpr int kLtVLd = kLtV + 8;
+
+LX_DEVICE void lt_mma(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+LX_DEVICE void lt_ldsm(uint32_t (&r)[4], uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+LX_DEVICE void lt_ldsm_t(uint32_t (&r)[4], uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+LX_DEVICE void lt_split(float a, float b, uint32_t& hi, uint32_t& lo) {
+  hi = pack_bf16x2(a, b);
+  const float2 back = unpack_bf16x2(hi);
+  lo = pack_bf16x2(a - back.x, b - back.y);
+}
+LX_DEVICE float lt_silu(float z) { return __fdividef(z, 1.f + __expf(-z)); }
+
+// rows [0, n) of a [64, COLS] tile: silu(global) -> shared (row pitch COLS + 8), zeros behind
+template <int COLS>
+LX_DEVICE void lt_load(__nv_bfloat16* dst, const __nv_bfloat16* src, long long ld, int n) {
+#pragma unroll
+  for (int e = threadIdx.x; e < kLtC * COLS / 8; e += 128) {
+    const int r = e / (COLS / 8), c = e % (COLS / 8) * 8;
+    float f[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+    if (r < n) {
+      load8(src + r * ld + c, f);
+#pragma unroll
+      for (int q = 0; q < 8; ++q) f[q] = lt_silu(f[q]);
+    }
+    store8(dst + r * (COLS + 8) + c, f);
+  }
+}
+
+template <int D, bool STATES>
+struct LtSmem {
+  static constexpr int kQ = STATES ? 0 : kLtC * (D + 8) * 2;
+  static constexpr int kK = kLtC * (D + 8) * 2;
+  static constexpr int kV = kLtC * kLtVLd * 2;
+  static constexpr int kS = STATES ? 0 : 2 * D * kLtVLd * 2;
+  static constexpr int kTotal = kQ + kK + kV + kS + (kLtC + 1) * 4 + 16;
+};
+
+template <int D, bool STATES>
+__global__ void __launch_bounds__(128, 2) linear_attn_tc_kernel(const LinTcParams p) {
+  pdl_trigger();
+  pdl_wait();
+  using M = LtSmem<D, STATES>;
+  constexpr int LD = D + 8, MT = D / 64;         // 16-row tiles of the state per warp
+  extern __shared__ __align__(16) uint8_t lt_sm[];
+  __nv_bfloat16* sq = reinterpret_cast<__nv_bfloat16*>(lt_sm);
+  __nv_bfloat16* sk = reinterpret_cast<__nv_bfloat16*>(lt_sm + M::kQ);
+  __nv_bfloat16* sv = reinterpret_cast<__nv_bfloat16*>(lt_sm + M::kQ + M::kK);
+  __nv_bfloat16* ss = reinterpret_cast<__nv_bfloat16*>(lt_sm + M::kQ + M::kK + M::kV);      // [2 terms][D][kLtVLd]
+  float* pw = reinterpret_cast<float*>(lt_sm + M::kQ + M::kK + M::kV + M::kS);             // decay^e, e = 0 .. 64
+  const int seg = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * kLtV;
+  const int b = p.seg_seq[seg], q0 = p.seg_q0[seg];
+  const int r0 = p.rows.cu_q[b], qlen = p.rows.cu_q[b + 1] - r0;
+  const int n = min(p.seg_len, qlen - q0);
+  const bool last = q0 + p.seg_len >= qlen;
+  if (STATES && last) return;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const float lam = p.decay[h];
+  for (int e = threadIdx.x; e <= kLtC; e += 128) pw[e] = powf(lam, (float)e);
+
+  // state rows warp * D / 4 + m * 16 + lane / 4 (+ 8), columns c0 + nt * 8 + 2 (lane % 4)
+  float S[MT][8][4];
+  const float* init = nullptr;
+  if (!STATES) {
+    if (qlen > p.seg_len) init = p.seg_state + ((long long)seg * p.H + h) * D * p.dv;
+    else if (p.rows.cache_lens[b] > 0) init = p.state + ((long long)p.rows.slots[b] * p.H + h) * D * p.dv;
+  }
+  const long long s_at = (long long)(warp * (D / 4) + (lane >> 2)) * p.dv + c0 + (lane & 3) * 2;
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int nt = 0; nt < 8; ++nt)
+#pragma unroll
+      for (int hr = 0; hr < 2; ++hr) {
+        float2 v = make_float2(0.f, 0.f);
+        if (init != nullptr) v = *reinterpret_cast<const float2*>(init + s_at + (long long)(m * 16 + hr * 8) * p.dv + nt * 8);
+        S[m][nt][2 * hr] = v.x;
+        S[m][nt][2 * hr + 1] = v.y;
+      }
+  const long long tok0 = (long long)p.rows.nd + r0 + q0;
+  const uint32_t q_a = smem_u32(sq) + ((warp * 16 + (lane & 15)) * LD + (lane >> 4) * 8) * 2;
+  const uint32_t k_b = smem_u32(sk) + (((lane & 7) + (lane >> 4) * 8) * LD + ((lane >> 3) & 1) * 8) * 2;
+  const uint32_t kt_a = smem_u32(sk) + (((lane & 7) + (lane >> 4) * 8) * LD + warp * (D / 4) + ((lane >> 3) & 1) * 8) * 2;
+  const uint32_t v_b = smem_u32(sv) + (((lane & 7) + ((lane >> 3) & 1) * 8) * kLtVLd + (lane >> 4) * 8) * 2;
+  const uint32_t s_b = smem_u32(ss) + (((lane & 7) + ((lane >> 3) & 1) * 8) * kLtVLd + (lane >> 4) * 8) * 2;
+
+  for (int t0 = 0; t0 < n; t0 += kLtC) {
+    const int m_tok = min(kLtC, n - t0);
+    __syncthreads();
+    if (!STATES) lt_load<D>(sq, p.q + (tok0 + t0) * p.ldq + h * D, p.ldq, m_tok);
+    lt_load<D>(sk, p.k + (tok0 + t0) * p.ldk + h * D, p.ldk, m_tok);
+    lt_load<kLtV>(sv, p.v + (tok0 + t0) * p.ldv + h * p.dv + c0, p.ldv, m_tok);
+    if (!STATES) {
+#pragma unroll
+      for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int nt = 0; nt < 8; ++nt)
+#pragma unroll
+          for (int hr = 0; hr < 2; ++hr) {
+            uint32_t hi, lo;
+            lt_split(S[m][nt][2 * hr], S[m][nt][2 * hr + 1], hi, lo);
+            __nv_bfloat16* d = ss + (warp * (D / 4) + m * 16 + (lane >> 2) + hr * 8) * kLtVLd + nt * 8 + (lane & 3) * 2;
+            *reinterpret_cast<uint32_t*>(d) = hi;
+            *reinterpret_cast<uint32_t*>(d + D * kLtVLd) = lo;
+          }
+    }
+    __syncthreads();
+    if (!STATES && warp * 16 < m_tok) {
+      float o[8][4], s[8][4];
+#pragma unroll
+      for (int nt = 0; nt < 8; ++nt) {
+        o[nt][0] = o[nt][1] = o[nt][2] = o[nt][3] = 0.f;
+        s[nt][0] = s[nt][1] = s[nt][2] = s[nt][3] = 0.f;
+      }
+#pragma unroll
+      for (int ks = 0; ks < D / 16; ++ks) {
+        uint32_t a[4];
+        lt_ldsm(a, q_a + ks * 32);
+#pragma unroll
+        for (int n2 = 0; n2 < 4; ++n2) {
+          if (n2 <= warp) {                        // keys behind the rows of this warp do not count
+            uint32_t kb[4];
+            lt_ldsm(kb, k_b + n2 * 16 * LD * 2 + ks * 32);
+            lt_mma(s[2 * n2], a, kb[0], kb[1]);
+            lt_mma(s[2 * n2 + 1], a, kb[2], kb[3]);
+          }
+          uint32_t sb[4];
+          lt_ldsm_t(sb, s_b + ks * 16 * kLtVLd * 2 + n2 * 32);
+          lt_mma(o[2 * n2], a, sb[0], sb[1]);
+          lt_mma(o[2 * n2 + 1], a, sb[2], sb[3]);
+          lt_ldsm_t(sb, s_b + (D + ks * 16) * kLtVLd * 2 + n2 * 32);
+          lt_mma(o[2 * n2], a, sb[0], sb[1]);
+          lt_mma(o[2 * n2 + 1], a, sb[2], sb[3]);
+        }
+      }
+      const int i0 = warp * 16 + (lane >> 2), i1 = i0 + 8;
+      const float f0 = pw[i0 + 1], f1 = pw[i1 + 1];
+#pragma unroll
+      for (int nt = 0; nt < 8; ++nt) { o[nt][0] *= f0; o[nt][1] *= f0; o[nt][2] *= f1; o[nt][3] *= f1; }
+#pragma unroll
+      for (int kk = 0; kk < 4; ++kk) {
+        if (kk > warp) continue;
+        uint32_t ph[4], pl[4];
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+          const int j = kk * 16 + u * 8 + (lane & 3) * 2;
+          const float* x = s[2 * kk + u];
+          lt_split(j <= i0 ? x[0] * pw[i0 - j] : 0.f, j + 1 <= i0 ? x[1] * pw[i0 - j - 1] : 0.f, ph[2 * u], pl[2 * u]);
+          lt_split(j <= i1 ? x[2] * pw[i1 - j] : 0.f, j + 1 <= i1 ? x[3] * pw[i1 - j - 1] : 0.f, ph[2 * u + 1], pl[2 * u + 1]);
+        }
+#pragma unroll
+        for (int n2 = 0; n2 < 4; ++n2) {
+          uint32_t vb[4];
+          lt_ldsm_t(vb, v_b + kk * 16 * kLtVLd * 2 + n2 * 32);
+          lt_mma(o[2 * n2], ph, vb[0], vb[1]);
+          lt_mma(o[2 * n2 + 1], ph, vb[2], vb[3]);
+          lt_mma(o[2 * n2], pl, vb[0], vb[1]);
+          lt_mma(o[2 * n2 + 1], pl, vb[2], vb[3]);
+        }
+      }
+      const long long ldo = (long long)p.H * p.dv;
+      float* orow = p.out + (tok0 + t0 + i0) * ldo + (long long)h * p.dv + c0 + (lane & 3) * 2;
+#pragma unroll
+      for (int nt = 0; nt < 8; ++nt) {
+        if (i0 < m_tok) *reinterpret_cast<float2*>(orow + nt * 8) = make_float2(o[nt][0], o[nt][1]);
+        if (i1 < m_tok) *reinterpret_cast<float2*>(orow + 8 * ldo + nt * 8) = make_float2(o[nt][2], o[nt][3]);
+      }
+    }
+    // ---- state
+    const float fs = pw[m_tok];
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+      for (int nt = 0; nt < 8; ++nt) { S[m][nt][0] *= fs; S[m][nt][1] *= fs; S[m][nt][2] *= fs; S[m][nt][3] *= fs; }
+#pragma unroll
+    for (int kk = 0; kk < 4; ++kk) {
+      uint32_t kh[MT][4], kl[MT][4];
+      const int j = kk * 16 + (lane & 3) * 2;
+      // (rows behind the chunk's last token are zero: their factor only has to exist)
+      const float g0 = pw[max(m_tok - 1 - j, 0)], g1 = pw[max(m_tok - 2 - j, 0)], g8 = pw[max(m_tok - 9 - j, 0)], g9 = pw[max(m_tok - 10 - j, 0)];
+#pragma unroll
+      for (int m = 0; m < MT; ++m) {
+        uint32_t a[4];
+        lt_ldsm_t(a, kt_a + kk * 16 * LD * 2 + m * 32);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float2 x = unpack_bf16x2(a[e]);
+          lt_split(x.x * (e < 2 ? g0 : g8), x.y * (e < 2 ? g1 : g9), kh[m][e], kl[m][e]);
+        }
+      }
+#pragma unroll
+      for (int n2 = 0; n2 < 4; ++n2) {
+        uint32_t vb[4];
+        lt_ldsm_t(vb, v_b + kk * 16 * kLtVLd * 2 + n2 * 32);
+#pragma unroll
+        for (int m = 0; m < MT; ++m) {
+          lt_mma(S[m][2 * n2], kh[m], vb[0], vb[1]);
+          lt_mma(S[m][2 * n2 + 1], kh[m], vb[2], vb[3]);
+          lt_mma(S[m][2 * n2], kl[m], vb[0], vb[1]);
+          lt_mma(S[m][2 * n2 + 1], kl[m], vb[2], vb[3]);
+        }
+      }
+    }
+  }
+  float* dst = nullptr;
+  if (STATES) dst = p.seg_state + ((long long)seg * p.H + h) * D * p.dv;
+  else if (last) dst = p.state + ((long long)p.rows.slots[b] * p.H + h) * D * p.dv;
+  if (dst != nullptr) {
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+      for (int nt = 0; nt < 8; ++nt)
+#pragma unroll
+        for (int hr = 0; hr < 2; ++hr)
+          *reinterpret_cast<float2*>(dst + s_at + (long long)(m * 16 + hr * 8) * p.dv + nt * 8) = make_float2(S[m][nt][2 * hr], S[m][nt][2 * hr + 1]);
+  }
+}
+
+template <int D>
+static int lt_launch(const LinTcParams& p, int nseg, bool states, cudaStream_t s) {
+  const dim3 grid(nseg, p.H, p.dv / kLtV);
+  if (states) {
+    cudaFuncSetAttribute(linear_attn_tc_kernel<D, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, LtSmem<D, true>::kTotal);
+    launch_pdl(linear_attn_tc_kernel<D, true>, grid, dim3(128), (size_t)LtSmem<D, true>::kTotal, s, p);
+  } else {
+    cudaFuncSetAttribute(linear_attn_tc_kernel<D, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, LtSmem<D, false>::kTotal);
+    launch_pdl(linear_attn_tc_kernel<D, false>, grid, dim3(128), (size_t)LtSmem<D, false>::kTotal, s, p);
+  }
+  return -(int)cudaGetLastError();
+}
+
+}  // namespace lx
+
+extern "C" {
+
+int lx_linear_attn_tc_bytes() { return (int)sizeof(lx::LinTcParams); }
+int lx_linear_attn_tc_supported(int d, int dv) { return ((d == 64 || d == 128) && dv % 64 == 0) ? 1 : 0; }
+
+// One pass over the segments: states != 0 the segments' contributions, else outputs and final states (the carry pass in between is
+// lx_recurrence's).
+int lx_linear_attn_tc(const void* params, int d, int nseg, int states, void* stream) {
+  using namespace lx;
+  if (nseg <= 0) return 0;
+  const LinTcParams& p = *reinterpret_cast<const LinTcParams*>(params);
+  if (!lx_linear_attn_tc_supported(d, p.dv) || p.ldq % 8 != 0 || p.ldk % 8 != 0 || p.ldv % 8 != 0) return -1;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  return d == 64 ? lt_launch<64>(p, nseg, states != 0, s) : lt_launch<128>(p, nseg, states != 0, s);
+}
+
+}  // extern "C"

@@ -289,20 +289,22 @@ __global__ void __launch_bounds__(256) rec_carry_kernel(const RecParams p) {
   }
 }
 
+enum RecPass : int { kRecStep = 1, kRecStates = 2, kRecCarry = 4, kRecOutputs = 8 };
+
 template <typename T, int MODE>
-static int rec_launch(const RecParams& p, int multi, cudaStream_t s) {
-  if (p.rows.nd > 0) {
+static int rec_launch(const RecParams& p, int what, cudaStream_t s) {
+  if ((what & kRecStep) && p.rows.nd > 0) {
     const int nc = p.dv / 4;
     const size_t smem = sizeof(float) * (3 * p.d + p.dv + (kRecStepThreads / nc) * p.dv);
     launch_pdl(rec_step_kernel<T, MODE>, dim3(p.rows.nd, p.H), dim3(kRecStepThreads), smem, s, p);
   }
-  if (p.rows.B > 0 && p.nseg > 0) {
+  if ((what & ~kRecStep) && p.rows.B > 0 && p.nseg > 0) {
     const int rpt = p.d <= 128 ? 16 : 32;
     const int nw = (p.d + rpt - 1) / rpt;
     const int tc = p.d <= 128 ? 16 : 8;
     const size_t smem = sizeof(float) * ((MODE == kWkv ? 3 : 2) * tc * p.d + tc * 64 + tc * nw * 64 + tc);
     const dim3 grid(p.nseg, p.H, (p.dv + 63) / 64), block(32 * nw);
-    if (multi) {
+    if (what & kRecStates) {
       if (rpt == 16) {
         cudaFuncSetAttribute(rec_scan_kernel<T, MODE, 16, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         launch_pdl(rec_scan_kernel<T, MODE, 16, true>, grid, block, smem, s, p, tc);
@@ -310,8 +312,10 @@ static int rec_launch(const RecParams& p, int multi, cudaStream_t s) {
         cudaFuncSetAttribute(rec_scan_kernel<T, MODE, 32, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         launch_pdl(rec_scan_kernel<T, MODE, 32, true>, grid, block, smem, s, p, tc);
       }
-      launch_pdl(rec_carry_kernel<MODE>, dim3(p.rows.B, p.H, (p.d * p.dv / 4 + 255) / 256), dim3(256), 0, s, p);
     }
+    if (what & kRecCarry)
+      launch_pdl(rec_carry_kernel<MODE>, dim3(p.rows.B, p.H, (p.d * p.dv / 4 + 255) / 256), dim3(256), 0, s, p);
+    if (!(what & kRecOutputs)) return -(int)cudaGetLastError();
     if (rpt == 16) {
       cudaFuncSetAttribute(rec_scan_kernel<T, MODE, 16, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
       launch_pdl(rec_scan_kernel<T, MODE, 16, false>, grid, block, smem, s, p, tc);
@@ -387,16 +391,17 @@ extern "C" {
 int lx_step_rows_bytes() { return (int)sizeof(lx::StepRows); }
 int lx_rec_params_bytes() { return (int)sizeof(lx::RecParams); }
 
-// mode 0: linear attention, 1: WKV.  multi: some sequence has more than one segment (seg_state / seg_decay are needed then).
-int lx_recurrence(const void* params, int mode, int multi, int f32, void* stream) {
+// mode 0: linear attention, 1: WKV.  what: the passes to launch (1 decode rows, 2 the segments' contributions, 4 the carry over the
+// segments, 8 outputs and final states); 2 and 4 are needed, with seg_state / seg_decay, when some sequence has more than one segment.
+int lx_recurrence(const void* params, int mode, int what, int f32, void* stream) {
   using namespace lx;
   const RecParams& p = *reinterpret_cast<const RecParams*>(params);
   if (p.d % 16 != 0 || p.dv % 16 != 0 || p.d > 256 || p.dv > 1024 || p.H <= 0) return -1;
   if (p.ldq % 4 != 0 || p.ldk % 4 != 0 || p.ldv % 4 != 0 || (mode == kWkv && p.ldz % 4 != 0)) return -2;
-  if (multi && (p.seg_state == nullptr || (mode == kWkv && p.seg_decay == nullptr))) return -3;
+  if ((what & (kRecStates | kRecCarry)) && (p.seg_state == nullptr || (mode == kWkv && p.seg_decay == nullptr))) return -3;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  if (f32) return mode == kLinAttn ? rec_launch<float, kLinAttn>(p, multi, s) : rec_launch<float, kWkv>(p, multi, s);
-  return mode == kLinAttn ? rec_launch<__nv_bfloat16, kLinAttn>(p, multi, s) : rec_launch<__nv_bfloat16, kWkv>(p, multi, s);
+  if (f32) return mode == kLinAttn ? rec_launch<float, kLinAttn>(p, what, s) : rec_launch<float, kWkv>(p, what, s);
+  return mode == kLinAttn ? rec_launch<__nv_bfloat16, kLinAttn>(p, what, s) : rec_launch<__nv_bfloat16, kWkv>(p, what, s);
 }
 
 int lx_token_shift(const void* h, const void* mu, void* shift, void* out, int n_mix, int W, int T, const void* rows_, int f32, void* stream) {

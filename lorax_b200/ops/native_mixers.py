@@ -25,6 +25,11 @@ class RecParams(Structure):
                 ("seg_len", I), ("seg_state", P), ("seg_decay", P)]
 
 
+class LinTcParams(Structure):
+    _fields_ = [("q", P), ("k", P), ("v", P), ("ldq", L), ("ldk", L), ("ldv", L), ("decay", P), ("state", P), ("seg_state", P), ("out", P),
+                ("H", I), ("dv", I), ("rows", StepRows), ("seg_seq", P), ("seg_q0", P), ("seg_len", I)]
+
+
 class LatentPrepParams(Structure):
     _fields_ = [("dq", P), ("dkv", P), ("ld_dq", L), ("ld_dkv", L), ("dq_norm", P), ("dkv_norm", P), ("cq", P), ("cache", P),
                 ("positions", P), ("slots", P), ("cos_sin", P), ("QR", I), ("KR", I), ("R", I), ("q_rank", I), ("kv_rank", I), ("rot", I),
@@ -52,6 +57,9 @@ SIGNATURES = {
     "lx_step_rows_bytes": ([], I),
     "lx_rec_params_bytes": ([], I),
     "lx_recurrence": ([P, I, I, I, P], I),
+    "lx_linear_attn_tc_bytes": ([], I),
+    "lx_linear_attn_tc_supported": ([I, I], I),
+    "lx_linear_attn_tc": ([P, I, I, I, P], I),
     "lx_token_shift": ([P, P, P, P, I, I, I, P, I, P], I),
     "lx_latent_prep_bytes": ([], I),
     "lx_latent_attn_bytes": ([], I),
@@ -69,7 +77,8 @@ SIGNATURES = {
 
 def check_layouts(lib):
     for name, st in (("lx_step_rows_bytes", StepRows), ("lx_rec_params_bytes", RecParams), ("lx_latent_prep_bytes", LatentPrepParams),
-                     ("lx_latent_attn_bytes", LatentAttnParams), ("lx_latent_decode_bytes", LatentDecodeParams)):
+                     ("lx_latent_attn_bytes", LatentAttnParams), ("lx_latent_decode_bytes", LatentDecodeParams),
+                     ("lx_linear_attn_tc_bytes", LinTcParams)):
         if getattr(lib, name)() != ctypes.sizeof(st):
             raise nv.NativeError(f"{name}: C++ says {getattr(lib, name)()} bytes, ctypes says {ctypes.sizeof(st)}")
 
@@ -167,8 +176,26 @@ def _recurrence(mode: int, q, k, v, z, decay, w0, u, H: int, d: int, dv: int, st
         if multi:
             hold = torch.empty(p.nseg * H * d * (dv + 1), dtype=torch.float32, device=q.device)
             p.seg_state, p.seg_decay = _p(hold), hold.data_ptr() + 4 * p.nseg * H * d * dv
-    nv._check(nv.load().lx_recurrence(ctypes.byref(p), mode, multi, _f32(q), nv._stream()), "lx_recurrence")
-    nv.launch_count += (1 if p.rows.nd and p.rows.B else 0) + 2 * multi
+    lib = nv.load()
+    step, prompts = (1 if p.rows.nd else 0), p.rows.B > 0
+
+    def passes(what):
+        if what:
+            nv._check(lib.lx_recurrence(ctypes.byref(p), mode, what, _f32(q), nv._stream()), "lx_recurrence")
+            nv.launch_count += bin(what).count("1") - 1
+
+    if mode == 0 and prompts and q.dtype == torch.bfloat16 and lib.lx_linear_attn_tc_supported(d, dv):
+        t = LinTcParams(p.q, p.k, p.v, p.ldq, p.ldk, p.ldv, p.decay, p.state, p.seg_state, p.out, H, dv, p.rows, p.seg_seq, p.seg_q0, p.seg_len)
+
+        def chunks(states):
+            nv._check(lib.lx_linear_attn_tc(ctypes.byref(t), d, p.nseg, states, nv._stream()), "lx_linear_attn_tc")
+        passes(step)
+        if multi:
+            chunks(1)
+            passes(4)
+        chunks(0)
+        return out
+    passes(step | (6 if multi else 0) | (8 if prompts else 0))
     return out
 
 

@@ -73,7 +73,7 @@ STEPS = {
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("step", list(STEPS))
-@pytest.mark.parametrize("H,d,dv", [(3, 16, 48), (2, 64, 32), (4, 128, 128), (1, 256, 80), (2, 48, 144)])
+@pytest.mark.parametrize("H,d,dv", [(3, 16, 48), (2, 64, 32), (4, 128, 128), (3, 64, 64), (2, 128, 192), (1, 256, 80), (2, 48, 144)])
 def test_linear_attention_recurrence(dtype, step, H, d, dv):
     from lorax_b200.ops import native, reference
     inp, _, ns = make_step(*STEPS[step])

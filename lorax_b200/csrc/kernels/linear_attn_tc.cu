@@ -1,11 +1,13 @@
 // Linear attention over prompt segments in chunks of 64 tokens on the tensor cores (bf16 activations, fp32 state).
 //
-// One CTA of four warps = one segment x one head x 64 value columns.  Within a chunk of tokens i, j with decay c:
+// One CTA of eight warps = one segment x one head x 64 value columns: four warps form the outputs of a chunk while the other four
+// advance the state past it.  Within a chunk of tokens i, j with decay c:
 //   o_i  = c^(i+1) q_i S + sum_{j <= i} c^(i-j) (q_i . k_j) v_j        S: the state in front of the chunk
 //   S    = c^n S + sum_j c^(n-1-j) k_j v_j^T
 // The state lives in fp32 accumulators.  Whatever is fp32 and enters a product (the state, the decayed weights, the decayed keys) is
-// split into two bf16 terms, value and remainder, and multiplied as two operands; q, k and v are bf16 after their silu anyway.
-// STATES: the segment's own contribution to the state only.
+// split into two bf16 terms, value and remainder, and multiplied as two operands; q, k and v arrive as bf16 with their silu applied
+// (silu_cols_kernel: they are read by two passes and two column halves).
+// STATES: the segment's own contribution to the state only (each group of four warps takes half of the columns).
 #include "stream.cuh"
 
 namespace lx {
@@ -26,6 +28,7 @@ struct LinTcParams {
 constexpr int kLtC = 64;                        // tokens per chunk
 constexpr int kLtV = 64;                        // value columns per CTA
 constexpr int kLtVLd = kLtV + 8;
+constexpr int kLtThreads = 256;
 
 LX_DEVICE void lt_mma(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
   asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
@@ -43,21 +46,28 @@ LX_DEVICE void lt_split(float a, float b, uint32_t& hi, uint32_t& lo) {
   const float2 back = unpack_bf16x2(hi);
   lo = pack_bf16x2(a - back.x, b - back.y);
 }
-LX_DEVICE float lt_silu(float z) { return __fdividef(z, 1.f + __expf(-z)); }
-
-// rows [0, n) of a [64, COLS] tile: silu(global) -> shared (row pitch COLS + 8), zeros behind
+// rows [0, n) of a [64, COLS] tile -> shared (row pitch COLS + 8), zeros behind
 template <int COLS>
-LX_DEVICE void lt_load(__nv_bfloat16* dst, const __nv_bfloat16* src, long long ld, int n) {
+LX_DEVICE void lt_fetch(__nv_bfloat16* dst, const __nv_bfloat16* src, long long ld, int n) {
 #pragma unroll
-  for (int e = threadIdx.x; e < kLtC * COLS / 8; e += 128) {
-    const int r = e / (COLS / 8), c = e % (COLS / 8) * 8;
-    float f[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-    if (r < n) {
-      load8(src + r * ld + c, f);
+  for (int i = 0; i < COLS / 32; ++i) {
+    const int e = threadIdx.x + i * kLtThreads, r = e / (COLS / 8), c = e % (COLS / 8) * 8;
+    cp_async_16(dst + r * (COLS + 8) + c, r < n ? src + r * ld + c : src, r < n);
+  }
+}
+
+// silu in place over the columns [0, cols) of a row-strided matrix (the projections of prompt rows, read several times below)
+__global__ void __launch_bounds__(256) silu_cols_kernel(__nv_bfloat16* __restrict__ x, long long ld, int cols, long long total) {
+  pdl_trigger();
+  pdl_wait();
+  const int per_row = cols / 8;
+  for (long long e = blockIdx.x * (long long)blockDim.x + threadIdx.x; e < total; e += (long long)gridDim.x * blockDim.x) {
+    __nv_bfloat16* at = x + (e / per_row) * ld + (e % per_row) * 8;
+    float f[8];
+    load8(at, f);
 #pragma unroll
-      for (int q = 0; q < 8; ++q) f[q] = lt_silu(f[q]);
-    }
-    store8(dst + r * (COLS + 8) + c, f);
+    for (int q = 0; q < 8; ++q) f[q] = __fdividef(f[q], 1.f + __expf(-f[q]));
+    store8(at, f);
   }
 }
 
@@ -71,7 +81,7 @@ struct LtSmem {
 };
 
 template <int D, bool STATES>
-__global__ void __launch_bounds__(128, 2) linear_attn_tc_kernel(const LinTcParams p) {
+__global__ void __launch_bounds__(kLtThreads, 2) linear_attn_tc_kernel(const LinTcParams p) {
   pdl_trigger();
   pdl_wait();
   using M = LtSmem<D, STATES>;
@@ -88,26 +98,29 @@ __global__ void __launch_bounds__(128, 2) linear_attn_tc_kernel(const LinTcParam
   const int n = min(p.seg_len, qlen - q0);
   const bool last = q0 + p.seg_len >= qlen;
   if (STATES && last) return;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int warp = (threadIdx.x >> 5) & 3, group = threadIdx.x >> 7, lane = threadIdx.x & 31;
+  const bool for_state = STATES || group == 1;
+  constexpr int NS = STATES ? 4 : 8;             // 8-wide column tiles of a state warp
+  const int cs = STATES ? group * 32 : 0;        // its first column
   const float lam = p.decay[h];
-  for (int e = threadIdx.x; e <= kLtC; e += 128) pw[e] = powf(lam, (float)e);
+  for (int e = threadIdx.x; e <= kLtC; e += kLtThreads) pw[e] = powf(lam, (float)e);
 
-  // state rows warp * D / 4 + m * 16 + lane / 4 (+ 8), columns c0 + nt * 8 + 2 (lane % 4)
-  float S[MT][8][4];
+  // state warps: rows warp * D / 4 + m * 16 + lane / 4 (+ 8), columns c0 + cs + nt * 8 + 2 (lane % 4)
+  float S[MT][NS][4];
   const float* init = nullptr;
   if (!STATES) {
     if (qlen > p.seg_len) init = p.seg_state + ((long long)seg * p.H + h) * D * p.dv;
     else if (p.rows.cache_lens[b] > 0) init = p.state + ((long long)p.rows.slots[b] * p.H + h) * D * p.dv;
   }
-  const long long s_at = (long long)(warp * (D / 4) + (lane >> 2)) * p.dv + c0 + (lane & 3) * 2;
+  const long long s_at = (long long)(warp * (D / 4) + (lane >> 2)) * p.dv + c0 + cs + (lane & 3) * 2;
 #pragma unroll
   for (int m = 0; m < MT; ++m)
 #pragma unroll
-    for (int nt = 0; nt < 8; ++nt)
+    for (int nt = 0; nt < NS; ++nt)
 #pragma unroll
       for (int hr = 0; hr < 2; ++hr) {
         float2 v = make_float2(0.f, 0.f);
-        if (init != nullptr) v = *reinterpret_cast<const float2*>(init + s_at + (long long)(m * 16 + hr * 8) * p.dv + nt * 8);
+        if (init != nullptr && for_state) v = *reinterpret_cast<const float2*>(init + s_at + (long long)(m * 16 + hr * 8) * p.dv + nt * 8);
         S[m][nt][2 * hr] = v.x;
         S[m][nt][2 * hr + 1] = v.y;
       }
@@ -121,14 +134,15 @@ __global__ void __launch_bounds__(128, 2) linear_attn_tc_kernel(const LinTcParam
   for (int t0 = 0; t0 < n; t0 += kLtC) {
     const int m_tok = min(kLtC, n - t0);
     __syncthreads();
-    if (!STATES) lt_load<D>(sq, p.q + (tok0 + t0) * p.ldq + h * D, p.ldq, m_tok);
-    lt_load<D>(sk, p.k + (tok0 + t0) * p.ldk + h * D, p.ldk, m_tok);
-    lt_load<kLtV>(sv, p.v + (tok0 + t0) * p.ldv + h * p.dv + c0, p.ldv, m_tok);
-    if (!STATES) {
+    if (!STATES) lt_fetch<D>(sq, p.q + (tok0 + t0) * p.ldq + h * D, p.ldq, m_tok);
+    lt_fetch<D>(sk, p.k + (tok0 + t0) * p.ldk + h * D, p.ldk, m_tok);
+    lt_fetch<kLtV>(sv, p.v + (tok0 + t0) * p.ldv + h * p.dv + c0, p.ldv, m_tok);
+    cp_async_commit();
+    if (!STATES && for_state) {
 #pragma unroll
       for (int m = 0; m < MT; ++m)
 #pragma unroll
-        for (int nt = 0; nt < 8; ++nt)
+        for (int nt = 0; nt < NS; ++nt)
 #pragma unroll
           for (int hr = 0; hr < 2; ++hr) {
             uint32_t hi, lo;
@@ -138,8 +152,9 @@ __global__ void __launch_bounds__(128, 2) linear_attn_tc_kernel(const LinTcParam
             *reinterpret_cast<uint32_t*>(d + D * kLtVLd) = lo;
           }
     }
+    cp_async_wait<0>();
     __syncthreads();
-    if (!STATES && warp * 16 < m_tok) {
+    if (!for_state && warp * 16 < m_tok) {
       float o[8][4], s[8][4];
 #pragma unroll
       for (int nt = 0; nt < 8; ++nt) {
@@ -193,19 +208,20 @@ __global__ void __launch_bounds__(128, 2) linear_attn_tc_kernel(const LinTcParam
         }
       }
       const long long ldo = (long long)p.H * p.dv;
-      float* orow = p.out + (tok0 + t0 + i0) * ldo + (long long)h * p.dv + c0 + (lane & 3) * 2;
+      float* orow = p.out + (tok0 + t0 + i0) * ldo + (long long)h * p.dv + c0 + cs + (lane & 3) * 2;
 #pragma unroll
       for (int nt = 0; nt < 8; ++nt) {
         if (i0 < m_tok) *reinterpret_cast<float2*>(orow + nt * 8) = make_float2(o[nt][0], o[nt][1]);
         if (i1 < m_tok) *reinterpret_cast<float2*>(orow + 8 * ldo + nt * 8) = make_float2(o[nt][2], o[nt][3]);
       }
     }
+    if (!for_state) continue;
     // ---- state
     const float fs = pw[m_tok];
 #pragma unroll
     for (int m = 0; m < MT; ++m)
 #pragma unroll
-      for (int nt = 0; nt < 8; ++nt) { S[m][nt][0] *= fs; S[m][nt][1] *= fs; S[m][nt][2] *= fs; S[m][nt][3] *= fs; }
+      for (int nt = 0; nt < NS; ++nt) { S[m][nt][0] *= fs; S[m][nt][1] *= fs; S[m][nt][2] *= fs; S[m][nt][3] *= fs; }
 #pragma unroll
     for (int kk = 0; kk < 4; ++kk) {
       uint32_t kh[MT][4], kl[MT][4];
@@ -223,9 +239,9 @@ __global__ void __launch_bounds__(128, 2) linear_attn_tc_kernel(const LinTcParam
         }
       }
 #pragma unroll
-      for (int n2 = 0; n2 < 4; ++n2) {
+      for (int n2 = 0; n2 < NS / 2; ++n2) {
         uint32_t vb[4];
-        lt_ldsm_t(vb, v_b + kk * 16 * kLtVLd * 2 + n2 * 32);
+        lt_ldsm_t(vb, v_b + kk * 16 * kLtVLd * 2 + (cs + n2 * 16) * 2);
 #pragma unroll
         for (int m = 0; m < MT; ++m) {
           lt_mma(S[m][2 * n2], kh[m], vb[0], vb[1]);
@@ -239,11 +255,11 @@ __global__ void __launch_bounds__(128, 2) linear_attn_tc_kernel(const LinTcParam
   float* dst = nullptr;
   if (STATES) dst = p.seg_state + ((long long)seg * p.H + h) * D * p.dv;
   else if (last) dst = p.state + ((long long)p.rows.slots[b] * p.H + h) * D * p.dv;
-  if (dst != nullptr) {
+  if (dst != nullptr && for_state) {
 #pragma unroll
     for (int m = 0; m < MT; ++m)
 #pragma unroll
-      for (int nt = 0; nt < 8; ++nt)
+      for (int nt = 0; nt < NS; ++nt)
 #pragma unroll
         for (int hr = 0; hr < 2; ++hr)
           *reinterpret_cast<float2*>(dst + s_at + (long long)(m * 16 + hr * 8) * p.dv + nt * 8) = make_float2(S[m][nt][2 * hr], S[m][nt][2 * hr + 1]);
@@ -255,10 +271,10 @@ static int lt_launch(const LinTcParams& p, int nseg, bool states, cudaStream_t s
   const dim3 grid(nseg, p.H, p.dv / kLtV);
   if (states) {
     cudaFuncSetAttribute(linear_attn_tc_kernel<D, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, LtSmem<D, true>::kTotal);
-    launch_pdl(linear_attn_tc_kernel<D, true>, grid, dim3(128), (size_t)LtSmem<D, true>::kTotal, s, p);
+    launch_pdl(linear_attn_tc_kernel<D, true>, grid, dim3(kLtThreads), (size_t)LtSmem<D, true>::kTotal, s, p);
   } else {
     cudaFuncSetAttribute(linear_attn_tc_kernel<D, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, LtSmem<D, false>::kTotal);
-    launch_pdl(linear_attn_tc_kernel<D, false>, grid, dim3(128), (size_t)LtSmem<D, false>::kTotal, s, p);
+    launch_pdl(linear_attn_tc_kernel<D, false>, grid, dim3(kLtThreads), (size_t)LtSmem<D, false>::kTotal, s, p);
   }
   return -(int)cudaGetLastError();
 }
@@ -270,7 +286,18 @@ extern "C" {
 int lx_linear_attn_tc_bytes() { return (int)sizeof(lx::LinTcParams); }
 int lx_linear_attn_tc_supported(int d, int dv) { return ((d == 64 || d == 128) && dv % 64 == 0) ? 1 : 0; }
 
-// One pass over the segments: states != 0 the segments' contributions, else outputs and final states (the carry pass in between is
+// silu in place over columns [0, cols) of T rows.
+int lx_silu_cols(void* x, long long ld, int T, int cols, void* stream) {
+  using namespace lx;
+  if (T <= 0 || cols <= 0) return 0;
+  if (cols % 8 != 0 || ld % 8 != 0) return -1;
+  const long long total = (long long)T * (cols / 8);
+  const int grid = (int)((total + 255) / 256 < 148 * 8 ? (total + 255) / 256 : 148 * 8);
+  launch_pdl(silu_cols_kernel, dim3(grid), dim3(256), 0, reinterpret_cast<cudaStream_t>(stream), reinterpret_cast<__nv_bfloat16*>(x), ld, cols, total);
+  return -(int)cudaGetLastError();
+}
+
+// q, k, v with their silu applied.  One pass over the segments: states != 0 the segments' contributions, else outputs and final states (the carry pass in between is
 // lx_recurrence's).
 int lx_linear_attn_tc(const void* params, int d, int nseg, int states, void* stream) {
   using namespace lx;

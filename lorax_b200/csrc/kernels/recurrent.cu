@@ -277,14 +277,25 @@ __global__ void __launch_bounds__(256) rec_carry_kernel(const RecParams p) {
   float4 run = make_float4(0.f, 0.f, 0.f, 0.f);
   if (p.rows.cache_lens[b] > 0) run = load4(p.state + ((long long)p.rows.slots[b] * p.H + h) * dd + e);
   const float lam = MODE == kLinAttn ? powf(p.decay[h], (float)p.seg_len) : 0.f;
-  for (int j = 0; j < ns; ++j) {
-    const long long at = ((long long)(lo + j) * p.H + h);
-    float4 own = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (j + 1 < ns) own = load4(p.seg_state + at * dd + e);
-    store4(p.seg_state + at * dd + e, run);
-    if (j + 1 < ns) {
-      const float w = MODE == kLinAttn ? lam : p.seg_decay[at * p.d + row];
-      run.x = w * run.x + own.x; run.y = w * run.y + own.y; run.z = w * run.z + own.z; run.w = w * run.w + own.w;
+  for (int j0 = 0; j0 < ns; j0 += 8) {            // eight segments' loads in flight: only the sums are a chain
+    float4 own[8];
+    float w[8];
+#pragma unroll
+    for (int u = 0; u < 8; ++u) {
+      const long long at = (long long)(lo + j0 + u) * p.H + h;
+      own[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+      w[u] = lam;
+      if (j0 + u + 1 < ns) {
+        own[u] = load4(p.seg_state + at * dd + e);
+        if (MODE == kWkv) w[u] = p.seg_decay[at * p.d + row];
+      }
+    }
+#pragma unroll
+    for (int u = 0; u < 8; ++u) {
+      if (j0 + u >= ns) break;
+      store4(p.seg_state + ((long long)(lo + j0 + u) * p.H + h) * dd + e, run);
+      run.x = w[u] * run.x + own[u].x; run.y = w[u] * run.y + own[u].y;
+      run.z = w[u] * run.z + own[u].z; run.w = w[u] * run.w + own[u].w;
     }
   }
 }

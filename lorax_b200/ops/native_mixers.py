@@ -60,6 +60,7 @@ SIGNATURES = {
     "lx_linear_attn_tc_bytes": ([], I),
     "lx_linear_attn_tc_supported": ([I, I], I),
     "lx_linear_attn_tc": ([P, I, I, I, P], I),
+    "lx_silu_cols": ([P, L, I, I, P], I),
     "lx_token_shift": ([P, P, P, P, I, I, I, P, I, P], I),
     "lx_latent_prep_bytes": ([], I),
     "lx_latent_attn_bytes": ([], I),
@@ -190,6 +191,10 @@ def _recurrence(mode: int, q, k, v, z, decay, w0, u, H: int, d: int, dv: int, st
         def chunks(states):
             nv._check(lib.lx_linear_attn_tc(ctypes.byref(t), d, p.nseg, states, nv._stream()), "lx_linear_attn_tc")
         passes(step)
+        nd = p.rows.nd
+        for x, cols in (((q, 2 * H * d + H * dv),) if k.data_ptr() == q.data_ptr() + 2 * H * d and v.data_ptr() == k.data_ptr() + 2 * H * d
+                        else ((q, H * d), (k, H * d), (v, H * dv))):
+            nv._check(lib.lx_silu_cols(_p(x[nd:]), x.stride(0), T - nd, cols, nv._stream()), "lx_silu_cols")
         if multi:
             chunks(1)
             passes(4)
@@ -200,6 +205,7 @@ def _recurrence(mode: int, q, k, v, z, decay, w0, u, H: int, d: int, dv: int, st
 
 
 def linear_attn(q, k, v, H: int, d: int, dv: int, decay, state, inp):
+    """(q, k and v are consumed: prompt rows may be overwritten by their silu)"""
     return _recurrence(0, q, k, v, None, decay, None, None, H, d, dv, state, inp)
 
 

@@ -30,6 +30,11 @@ class LinTcParams(Structure):
                 ("H", I), ("dv", I), ("rows", StepRows), ("seg_seq", P), ("seg_q0", P), ("seg_len", I)]
 
 
+class WkvTcParams(Structure):
+    _fields_ = [("r", P), ("k", P), ("v", P), ("z", P), ("ldr", L), ("ldk", L), ("ldv", L), ("ldz", L), ("w0", P), ("u", P), ("state", P),
+                ("seg_state", P), ("seg_decay", P), ("out", P), ("H", I), ("rows", StepRows), ("seg_seq", P), ("seg_q0", P), ("seg_len", I)]
+
+
 class LatentPrepParams(Structure):
     _fields_ = [("dq", P), ("dkv", P), ("ld_dq", L), ("ld_dkv", L), ("dq_norm", P), ("dkv_norm", P), ("cq", P), ("cache", P),
                 ("positions", P), ("slots", P), ("cos_sin", P), ("QR", I), ("KR", I), ("R", I), ("q_rank", I), ("kv_rank", I), ("rot", I),
@@ -60,6 +65,9 @@ SIGNATURES = {
     "lx_linear_attn_tc_bytes": ([], I),
     "lx_linear_attn_tc_supported": ([I, I], I),
     "lx_linear_attn_tc": ([P, I, I, I, P], I),
+    "lx_wkv_tc_bytes": ([], I),
+    "lx_wkv_tc_supported": ([I], I),
+    "lx_wkv_tc": ([P, I, I, P], I),
     "lx_silu_cols": ([P, L, I, I, P], I),
     "lx_token_shift": ([P, P, P, P, I, I, I, P, I, P], I),
     "lx_latent_prep_bytes": ([], I),
@@ -79,7 +87,7 @@ SIGNATURES = {
 def check_layouts(lib):
     for name, st in (("lx_step_rows_bytes", StepRows), ("lx_rec_params_bytes", RecParams), ("lx_latent_prep_bytes", LatentPrepParams),
                      ("lx_latent_attn_bytes", LatentAttnParams), ("lx_latent_decode_bytes", LatentDecodeParams),
-                     ("lx_linear_attn_tc_bytes", LinTcParams)):
+                     ("lx_linear_attn_tc_bytes", LinTcParams), ("lx_wkv_tc_bytes", WkvTcParams)):
         if getattr(lib, name)() != ctypes.sizeof(st):
             raise nv.NativeError(f"{name}: C++ says {getattr(lib, name)()} bytes, ctypes says {ctypes.sizeof(st)}")
 
@@ -199,6 +207,18 @@ def _recurrence(mode: int, q, k, v, z, decay, w0, u, H: int, d: int, dv: int, st
             chunks(1)
             passes(4)
         chunks(0)
+        return out
+    if mode == 1 and prompts and q.dtype == torch.bfloat16 and lib.lx_wkv_tc_supported(d):
+        t = WkvTcParams(p.q, p.k, p.v, p.z, p.ldq, p.ldk, p.ldv, p.ldz, p.w0, p.u, p.state, p.seg_state, p.seg_decay, p.out, H, p.rows,
+                        p.seg_seq, p.seg_q0, p.seg_len)
+
+        def blocks(states):
+            nv._check(lib.lx_wkv_tc(ctypes.byref(t), p.nseg, states, nv._stream()), "lx_wkv_tc")
+        passes(step)
+        if multi:
+            blocks(1)
+            passes(4)
+        blocks(0)
         return out
     passes(step | (6 if multi else 0) | (8 if prompts else 0))
     return out

@@ -65,7 +65,7 @@ def _run(cmd, verbose: bool, log_path: Path | None = None, quiet: bool = False) 
 
 
 # Sources a program needs that only ever runs one kind of model (`ops.native.use_subset`).
-SUBSETS = {"mixers": ("gemm_bf16", "elementwise", "stream", "recurrent", "latent_attn", "latent_prefill_tc", "latent_decode_tc", "linear_attn_tc",
+SUBSETS = {"mixers": ("gemm_bf16", "moe", "elementwise", "stream", "recurrent", "latent_attn", "latent_prefill_tc", "latent_decode_tc", "linear_attn_tc",
                       "wkv_tc")}
 
 

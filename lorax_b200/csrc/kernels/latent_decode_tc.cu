@@ -1,7 +1,7 @@
 // Absorbed latent attention for single query rows (decode rows, and portions too short to be worth an expansion): every cached row
 // [latent | shared key part] is read once and serves as key and value of 16 or 32 heads at a time.
 //
-// One CTA of eight warps = one row x MT * 16 heads x one share of the keys, in tiles of 64 keys through a two-stage cp.async ring:
+// One CTA of eight warps = one row x MT * 16 heads x one share of the keys, in tiles of 32 or 64 keys through a two-stage cp.async ring:
 //   scores   four K slices x two key halves over the warps; the query fragments stay in registers, the slices' partial sums meet in
 //            shared memory
 //   softmax  fp32, eight or sixteen threads per head; the weights are split into two bf16 terms (value + remainder)
@@ -11,7 +11,6 @@
 
 namespace lx {
 
-constexpr int kLdKeys = 64, kLdThreads = 256;
 
 struct LatentDecodeParams {
   const __nv_bfloat16* q_lat; long long ld_ql;    // [T, H * KR]
@@ -43,28 +42,30 @@ LX_DEVICE float ld_ex2(float x) {
   return y;
 }
 
-template <int MT>
+template <int MT, int KEYS, int WARPS>
 struct LdSmem {
   static constexpr int kRows = MT * 16;
-  static constexpr int kPartLd = kLdKeys + 4;
-  static constexpr int kPLd = kLdKeys + 8;
-  static constexpr int kPart = 4 * kRows * kPartLd * 4;
+  static constexpr int kPartLd = KEYS + 4;
+  static constexpr int kPLd = KEYS + 8;
+  static constexpr int kPart = WARPS / 2 * kRows * kPartLd * 4;
   static constexpr int kP = 2 * kRows * kPLd * 2;
   static constexpr int kVec = 3 * kRows * 4;
-  static int total(int R) { return 2 * kLdKeys * (R + 8) * 2 + kPart + kP + kVec; }
+  static int total(int R) { return 2 * KEYS * (R + 8) * 2 + kPart + kP + kVec; }
 };
 
-// KS: 16-wide K steps per slice; KR: latent columns.
-template <int MT, int KS, int KR>
-__global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const LatentDecodeParams p) {
+// KS: 16-wide K steps per slice; KR: latent columns; KEYS: keys per tile; WARPS: per CTA; OCC: CTAs per SM.
+template <int MT, int KS, int KR, int KEYS, int WARPS, int OCC>
+__global__ void __launch_bounds__(32 * WARPS, OCC) latent_decode_kernel(const LatentDecodeParams p) {
   pdl_trigger();
   pdl_wait();
-  using S = LdSmem<MT>;
-  constexpr int NT = KR / 64;                      // 8-wide column tiles per warp
+  using S = LdSmem<MT, KEYS, WARPS>;
+  constexpr int kLdThreads = 32 * WARPS, KG = WARPS / 2;      // K slices of the score products
+  constexpr int NK2 = KEYS / 32;                   // 16-key steps of a warp's half of the tile
+  constexpr int NT = KR / (8 * WARPS);                    // 8-wide column tiles per warp
   extern __shared__ __align__(16) uint8_t ld_sm[];
   const int pitch = (p.R + 8) * 2;                 // bytes; an odd multiple of 16: ldmatrix rows fall into different banks
   uint8_t* sk = ld_sm;
-  float* part = reinterpret_cast<float*>(ld_sm + 2 * kLdKeys * pitch);
+  float* part = reinterpret_cast<float*>(ld_sm + 2 * KEYS * pitch);
   __nv_bfloat16* sp = reinterpret_cast<__nv_bfloat16*>(reinterpret_cast<uint8_t*>(part) + S::kPart);
   float* s_alpha = reinterpret_cast<float*>(reinterpret_cast<uint8_t*>(sp) + S::kP);
   float* s_m = s_alpha + S::kRows;
@@ -82,11 +83,11 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
     bt = p.rows.bt + (long long)b * p.rows.max_blocks;
   }
   keys = max(keys, 0);
-  const int tiles = (keys + kLdKeys - 1) / kLdKeys;
+  const int tiles = (keys + KEYS - 1) / KEYS;
   const int per = (tiles + p.nsplit - 1) / p.nsplit;
   const int t_lo = split * per, t_hi = min(t_lo + per, tiles);
 
-  const int kg = warp & 3, kh = warp >> 2;         // K slice, key half of the score products
+  const int kg = warp % KG, kh = warp / KG;         // K slice, key half of the score products
   const int nk = p.R / 16;
   uint32_t qf[MT][KS][4];
 #pragma unroll
@@ -112,17 +113,19 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
     for (int n = 0; n < NT; ++n) o[m][n][0] = o[m][n][1] = o[m][n][2] = o[m][n][3] = 0.f;
 
   auto load = [&](int tile, int st) {
-    const int r = threadIdx.x >> 2, key = tile * kLdKeys + r;
+    constexpr int TPK = kLdThreads / KEYS;          // threads per key
+    const int r = threadIdx.x / TPK, key = tile * KEYS + r;
     const bool ok = key < keys;
     const __nv_bfloat16* src = p.cache;
     if (ok) src += ((long long)bt[key / p.page] * p.page + key % p.page) * p.R;
-    uint8_t* dst = sk + (st * kLdKeys + r) * pitch;
-    for (int c = threadIdx.x & 3; c < p.R / 8; c += 4) cp_async_16(dst + c * 16, ok ? src + c * 8 : src, ok);
+    uint8_t* dst = sk + (st * KEYS + r) * pitch;
+    for (int c = threadIdx.x % TPK; c < p.R / 8; c += TPK) cp_async_16(dst + c * 16, ok ? src + c * 8 : src, ok);
     cp_async_commit();
   };
 
   constexpr int TPR = kLdThreads / S::kRows;       // softmax threads per head
-  constexpr int KPT = kLdKeys / TPR;               // keys of each
+  constexpr int KPT = KEYS / TPR;                  // keys of each
+  static_assert(KPT % 2 == 0, "a softmax thread reads its keys' scores in pairs");
   const int srow = threadIdx.x / TPR, sk0 = (threadIdx.x % TPR) * KPT;
   const float scale_l2 = p.scale * 1.4426950408889634f;
   float mx = -INFINITY, sum = 0.f;                 // of head srow; sum: this thread's keys only
@@ -133,21 +136,21 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
     cp_async_wait<0>();
     __syncthreads();
     if (i + 1 < t_hi) load(i + 1, st ^ 1);
-    const uint32_t kb = smem_u32(sk) + (uint32_t)(st * kLdKeys * pitch);
+    const uint32_t kb = smem_u32(sk) + (uint32_t)(st * KEYS * pitch);
     // ---- scores
     {
-      float acc[MT][4][4];
+      float acc[MT][2 * NK2][4];
 #pragma unroll
       for (int m = 0; m < MT; ++m)
 #pragma unroll
-        for (int n = 0; n < 4; ++n) acc[m][n][0] = acc[m][n][1] = acc[m][n][2] = acc[m][n][3] = 0.f;
-      const uint32_t a0 = kb + (uint32_t)((kh * 32 + (lane & 7) + (lane >> 4) * 8) * pitch + ((lane >> 3) & 1) * 16);
+        for (int n = 0; n < 2 * NK2; ++n) acc[m][n][0] = acc[m][n][1] = acc[m][n][2] = acc[m][n][3] = 0.f;
+      const uint32_t a0 = kb + (uint32_t)((kh * (KEYS / 2) + (lane & 7) + (lane >> 4) * 8) * pitch + ((lane >> 3) & 1) * 16);
 #pragma unroll
       for (int s = 0; s < KS; ++s) {
         const int ks = kg * KS + s;
         if (ks < nk) {
 #pragma unroll
-          for (int n2 = 0; n2 < 2; ++n2) {
+          for (int n2 = 0; n2 < NK2; ++n2) {
             uint32_t b[4];
             ld_ldsm(b, a0 + (uint32_t)(n2 * 16 * pitch + ks * 32));
 #pragma unroll
@@ -161,8 +164,8 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
 #pragma unroll
       for (int m = 0; m < MT; ++m)
 #pragma unroll
-        for (int n = 0; n < 4; ++n) {
-          float* d = part + (kg * S::kRows + m * 16 + (lane >> 2)) * S::kPartLd + kh * 32 + n * 8 + (lane & 3) * 2;
+        for (int n = 0; n < 2 * NK2; ++n) {
+          float* d = part + (kg * S::kRows + m * 16 + (lane >> 2)) * S::kPartLd + kh * (KEYS / 2) + n * 8 + (lane & 3) * 2;
           *reinterpret_cast<float2*>(d) = make_float2(acc[m][n][0], acc[m][n][1]);
           *reinterpret_cast<float2*>(d + 8 * S::kPartLd) = make_float2(acc[m][n][2], acc[m][n][3]);
         }
@@ -172,18 +175,18 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
     {
       float s[KPT], bm = -INFINITY;
 #pragma unroll
-      for (int q = 0; q < KPT; q += 4) {
-        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+      for (int q = 0; q < KPT; q += 2) {
+        float2 v = make_float2(0.f, 0.f);
 #pragma unroll
-        for (int g = 0; g < 4; ++g) {
-          const float4 a = *reinterpret_cast<const float4*>(part + (g * S::kRows + srow) * S::kPartLd + sk0 + q);
-          v.x += a.x; v.y += a.y; v.z += a.z; v.w += a.w;
+        for (int g = 0; g < KG; ++g) {
+          const float2 a = *reinterpret_cast<const float2*>(part + (g * S::kRows + srow) * S::kPartLd + sk0 + q);
+          v.x += a.x; v.y += a.y;
         }
-        s[q] = v.x; s[q + 1] = v.y; s[q + 2] = v.z; s[q + 3] = v.w;
+        s[q] = v.x; s[q + 1] = v.y;
       }
 #pragma unroll
       for (int q = 0; q < KPT; ++q) {
-        s[q] = (i * kLdKeys + sk0 + q < keys) ? s[q] * scale_l2 : -INFINITY;
+        s[q] = (i * KEYS + sk0 + q < keys) ? s[q] * scale_l2 : -INFINITY;
         bm = fmaxf(bm, s[q]);
       }
 #pragma unroll
@@ -215,9 +218,9 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
         for (int n = 0; n < NT; ++n) { o[m][n][0] *= f0; o[m][n][1] *= f0; o[m][n][2] *= f1; o[m][n][3] *= f1; }
       }
       const uint32_t pa = smem_u32(sp) + (uint32_t)(((lane & 15) * S::kPLd + (lane >> 4) * 8) * 2);
-      const uint32_t vb = kb + (uint32_t)(((lane & 7) + ((lane >> 3) & 1) * 8) * pitch + (warp * (KR / 8) + (lane >> 4) * 8) * 2);
+      const uint32_t vb = kb + (uint32_t)(((lane & 7) + ((lane >> 3) & 1) * 8) * pitch + (warp * (KR / WARPS) + (lane >> 4) * 8) * 2);
 #pragma unroll
-      for (int ks = 0; ks < kLdKeys / 16; ++ks) {
+      for (int ks = 0; ks < KEYS / 16; ++ks) {
         uint32_t ah[MT][4], al[MT][4];
 #pragma unroll
         for (int m = 0; m < MT; ++m) {
@@ -250,7 +253,7 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
       const int r = m * 16 + (lane >> 2) + hr * 8, hd = h0 + r;
       if (hd >= p.H) continue;
       const float l = s_l[r], inv = l > 0.f ? 1.f / l : 0.f;
-      const int c0 = warp * (KR / 8) + (lane & 3) * 2;
+      const int c0 = warp * (KR / WARPS) + (lane & 3) * 2;
       if (p.nsplit == 1) {
         __nv_bfloat16* d = p.out + (long long)t * p.ldo + (long long)hd * KR + c0;
 #pragma unroll
@@ -291,14 +294,14 @@ __global__ void __launch_bounds__(128) latent_combine_kernel(const float* __rest
   }
 }
 
-template <int MT, int KS, int KR>
+template <int MT, int KS, int KR, int KEYS, int WARPS, int OCC>
 static int ld_launch(const LatentDecodeParams& p, int T, cudaStream_t s) {
-  const int smem = LdSmem<MT>::total(p.R);
+  const int smem = LdSmem<MT, KEYS, WARPS>::total(p.R);
   if (smem > 227 * 1024) return -4;
-  cudaError_t e = cudaFuncSetAttribute(latent_decode_kernel<MT, KS, KR>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  cudaError_t e = cudaFuncSetAttribute(latent_decode_kernel<MT, KS, KR, KEYS, WARPS, OCC>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   if (e != cudaSuccess) return -(int)e;
   const int groups = (p.H + MT * 16 - 1) / (MT * 16);
-  launch_pdl(latent_decode_kernel<MT, KS, KR>, dim3(T, groups, p.nsplit), dim3(kLdThreads), (size_t)smem, s, p);
+  launch_pdl(latent_decode_kernel<MT, KS, KR, KEYS, WARPS, OCC>, dim3(T, groups, p.nsplit), dim3(32 * WARPS), (size_t)smem, s, p);
   if (p.nsplit > 1)
     launch_pdl(latent_combine_kernel, dim3(T, p.H), dim3(128), 0, s, (const float*)p.part_o, (const float*)p.part_ml, p.out, p.ldo, p.H, KR, p.nsplit);
   return -(int)cudaGetLastError();
@@ -320,10 +323,11 @@ int lx_latent_decode(const void* params, int KR, int T, void* stream) {
   if (!lx_latent_decode_supported(KR, p.R) || p.nsplit < 1 || (p.nsplit > 1 && (p.part_o == nullptr || p.part_ml == nullptr))) return -1;
   if (p.head % 2 != 0 || p.rot_off % 2 != 0 || p.ldq % 2 != 0 || p.ld_ql % 2 != 0 || p.ldo % 4 != 0) return -2;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  // up to 16 heads: 32-key tiles, two CTAs per SM hide each other's barriers; more: 32 heads share a 64-key tile
   const bool two = p.H > 16;
-  if (KR == 512) return two ? ld_launch<2, 9, 512>(p, T, s) : ld_launch<1, 9, 512>(p, T, s);
-  if (KR == 256) return two ? ld_launch<2, 5, 256>(p, T, s) : ld_launch<1, 5, 256>(p, T, s);
-  return two ? ld_launch<2, 3, 128>(p, T, s) : ld_launch<1, 3, 128>(p, T, s);
+  if (KR == 512) return two ? ld_launch<2, 9, 512, 64, 8, 1>(p, T, s) : ld_launch<1, 9, 512, 32, 8, 2>(p, T, s);
+  if (KR == 256) return two ? ld_launch<2, 5, 256, 64, 8, 1>(p, T, s) : ld_launch<1, 5, 256, 32, 8, 2>(p, T, s);
+  return two ? ld_launch<2, 3, 128, 64, 8, 1>(p, T, s) : ld_launch<1, 3, 128, 32, 8, 2>(p, T, s);
 }
 
 }  // extern "C"

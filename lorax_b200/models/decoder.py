@@ -207,6 +207,11 @@ class DecoderModel:
             self._rope_tables[key] = reference.rope_table(rot, self.max_positions, base, self.device)
         return self._rope_tables[key]
 
+    @property
+    def state_parallelism(self) -> int:
+        """Thread blocks one sequence gives the recurrence kernels (the least of the layers)."""
+        return min([lw.mixer.parallelism for lw in self.layers if lw.mixer.recurrent] + [1 << 20])
+
     def cache_shapes(self) -> Optional[List[dict]]:
         """What every layer run keeps (`Mixer.cache_shape`), or None for the uniform key/value cache."""
         return [self.layers[li].mixer.cache_shape(self) for li in self.schedule] if self.mixed else None

@@ -93,6 +93,7 @@ class LightningMixer(Mixer):
             raise ValueError(f"{len(self.decay_values)} decays for {self.H} heads")
         self.dp, self.dvp = pad16(self.d), pad16(self.dv)
         self.out_dim = self.H * self.dvp
+        self.parallelism = self.H * ((self.dvp + 63) // 64)
 
     def shapes(self):
         H, d, dv, w = self.H, self.d, self.dv, self.width
@@ -127,6 +128,7 @@ class WkvMixer(Mixer):
         self.H, self.d = int(params["heads"]), int(params["dim"])
         self.dp = pad16(self.d)
         self.out_dim = self.H * self.dp
+        self.parallelism = self.H * ((self.dp + 63) // 64)
         self.rank: Optional[int] = params.get("rank")      # of the decay's low-rank map; the checkpoint's own shape decides
 
     def shapes(self):

@@ -151,10 +151,26 @@ def gemm_f32(x, w, out=None, out_scale: float = 1.0):
     return out
 
 
+STACK_GROUPED_MAX_ROWS = 256
+_segments = {}
+
+
+def _stack_segments(n: int, T: int, device) -> torch.Tensor:
+    key = (n, T, device)
+    if key not in _segments:
+        _segments[key] = torch.arange(0, (n + 1) * T, T, dtype=torch.int32, device=device)
+    return _segments[key]
+
+
 def gemm_stack(x, w):
     """x [n, T, K], w [n, N, K] -> [n, T, N]: one product per stacked pair."""
-    n, T, _ = x.shape
-    out = torch.empty(n, T, w.shape[1], dtype=x.dtype, device=x.device)
+    n, T, K = x.shape
+    N = w.shape[1]
+    out = torch.empty(n, T, N, dtype=x.dtype, device=x.device)
+    if x.dtype == torch.bfloat16 and T <= STACK_GROUPED_MAX_ROWS and N % 128 == 0 and x.is_contiguous():
+        # few rows: all products stream their weights in one launch (the grouped GEMM of the expert layers, one group per pair)
+        nv.moe_grouped_gemm(x.view(n * T, K), w, _stack_segments(n, T, x.device), T, out.view(n * T, N))
+        return out
     for i in range(n):
         nv.gemm(x[i], w[i], out=out[i])
     return out
@@ -266,9 +282,9 @@ def latent_attn(q_lat, q, cache, H: int, kv_rank: int, head: int, rot_off: int, 
         d.q_lat, d.ld_ql, d.q, d.ldq, d.head, d.rot_off = _p(q_lat), q_lat.stride(0), _p(q), q.stride(0), head, rot_off
         d.cache, d.out, d.ldo, d.rows = _p(cache), _p(out), out.stride(0), step_rows(inp, T)
         d.H, d.R, d.page, d.scale = H, kv_rank + rot, cache.shape[1], scale
-        # the keys of a row are shared out until the grid fills the GPU once (one CTA per SM)
-        groups = (H + 31) // 32 if H > 16 else 1
-        d.nsplit = max(1, min(32, nv.workspace(q.device).num_sms // (T * groups)))
+        # the keys of a row are shared out until the grid fills the GPU once (one CTA per SM, two for up to 16 heads)
+        groups, per_sm = ((H + 31) // 32, 1) if H > 16 else (1, 2)
+        d.nsplit = max(1, min(32, nv.workspace(q.device).num_sms * per_sm // (T * groups)))
         hold = None
         if d.nsplit > 1:
             n = T * H * d.nsplit

@@ -227,8 +227,12 @@ class ModelRunner:
                 ctx_off.append(ctx_off[-1] + c + n)
         if self.model.recurrent:
             # the recurrence kernels carry the state through segments of this many tokens: long enough that the states between
-            # segments stay a small part of the traffic, short enough that a lone prompt fills the GPU
+            # segments stay a small part of the traffic, short enough that a lone prompt fills the GPU.  Prompts that fill it by
+            # themselves take one segment each, which saves the pass over the segments' states.
             seg_len = min(512, max(64, (T // 16 + 63) // 64 * 64))
+            longest = max(q_lens + [1])
+            if T // longest * self.model.state_parallelism >= 224:
+                seg_len = (longest + 63) // 64 * 64
             sgs, sgq = reference.prefill_tiles(q_lens, seg_len)
         i32 = lambda v: np.asarray(v, dtype=np.int32).reshape(-1)
         segs = [np.concatenate(id_parts) if id_parts else i32([]), i32(cu), i32(cache_lens), i32(seq_slot), i32(ts), i32(tq), i32(head_idx),

@@ -382,3 +382,37 @@ def test_cuda_graphs_do_not_advance_the_state():
             outs.append([eng.finished[i + 1].output_ids for i in range(5)])
     assert outs[0] == outs[1]
     assert outs[0][2] == oracle.greedy(cfg, w, tokens(17, cfg["vocab"], 2), 16)
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("name", ["aligned", "recurrent"])
+def test_cache_is_sized_from_free_memory(name):
+    """No block count given: a maximum prefill is measured and the pool takes its share of what is left beside the states."""
+    from lorax_b200.runtime.engine import Engine
+    cfg = CONFIGS[name]
+    w = weights_of(cfg, seed=9)
+    m = build(cfg, w, "cuda", torch.float32)
+    with torch.inference_mode():
+        eng = Engine(m, EngineConfig(max_total_tokens=128, max_batch_prefill_tokens=256, max_input_length=100, memory_wiggle_room=0.04), max_batch=4)
+        p = tokens(21, cfg["vocab"], 3)
+        assert eng.kv.num_blocks >= 16
+        assert eng.generate([p, p[:5]], 6) == [oracle.greedy(cfg, w, p, 6), oracle.greedy(cfg, w, p[:5], 6)]
+
+
+@pytest.mark.gpu
+def test_prompts_that_fill_the_gpu_take_one_segment_each():
+    """Many heads and several prompts: the recurrences run without the pass over segment states; same results as alone."""
+    cfg = config([wkv(heads=64, dim=64, ff=0), lightning(heads=60, dim=64, vdim=128, ff=0)], width=64, vocab=100)
+    w = weights_of(cfg, seed=10)
+    m = build(cfg, w, "cuda", torch.bfloat16)
+    from lorax_b200.runtime.runner import PrefillItem
+    seqs = [tokens(n, 100, n) for n in (150, 149, 131, 90)]
+    with torch.inference_mode():
+        r = TraceReplay(m, 640)
+        for i in range(4):
+            r.alloc.extend(r.held.setdefault(str(i), []), len(seqs[i]))
+        items = [PrefillItem(s, 0, r.held[str(i)], state_slot=i + 1, logit_rows=[0, 63, 64, len(s) - 1]) for i, s in enumerate(seqs)]
+        assert r.runner._prefill_inputs(items)[0].seg_len == 192
+        _, _, logits = r.runner.prefill(items)
+        for i, s in enumerate(seqs):
+            check(logits[4 * i: 4 * i + 4].float().cpu(), oracle.forward(cfg, w, s)[[0, 63, 64, len(s) - 1]], torch.bfloat16)

@@ -231,7 +231,7 @@ class ModelRunner:
             # themselves take one segment each, which saves the pass over the segments' states.
             seg_len = min(512, max(64, (T // 16 + 63) // 64 * 64))
             longest = max(q_lens + [1])
-            if T // longest * self.model.state_parallelism >= 224:
+            if T * self.model.state_parallelism >= 200 * longest:
                 seg_len = (longest + 63) // 64 * 64
             sgs, sgq = reference.prefill_tiles(q_lens, seg_len)
         i32 = lambda v: np.asarray(v, dtype=np.int32).reshape(-1)

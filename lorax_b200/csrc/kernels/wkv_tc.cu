@@ -49,6 +49,32 @@ LX_DEVICE void wk_split1(float a, __nv_bfloat16& hi, __nv_bfloat16& lo) {
   lo = __float2bfloat16(a - __bfloat162float(hi));
 }
 
+// two fp32 numbers in one 64-bit register: one instruction multiplies or accumulates both
+LX_DEVICE unsigned long long wk_pair(float a, float b) {
+  unsigned long long r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+  return r;
+}
+LX_DEVICE float2 wk_unpair(unsigned long long v) {
+  float2 f;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(f.x), "=f"(f.y) : "l"(v));
+  return f;
+}
+LX_DEVICE unsigned long long wk_mul2(unsigned long long a, unsigned long long b) {
+  unsigned long long r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+LX_DEVICE unsigned long long wk_fma2(unsigned long long a, unsigned long long b, unsigned long long c) {
+  unsigned long long r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+LX_DEVICE void wk_load4(unsigned long long (&x)[4], const float* p) {
+  const ulonglong2 a = reinterpret_cast<const ulonglong2*>(p)[0], b = reinterpret_cast<const ulonglong2*>(p)[1];
+  x[0] = a.x; x[1] = a.y; x[2] = b.x; x[3] = b.y;
+}
+
 struct WkSmem {
   float w[kWkB * kWkF];
   float r[kWkB * kWkF];
@@ -174,21 +200,26 @@ __global__ void __launch_bounds__(kWkThreads, 2) wkv_tc_kernel(const WkvTcParams
 #pragma unroll
         for (int q = 0; q < 8; ++q) diag = fmaf(rj[q] * u[q], e[q], diag);
       }
+      unsigned long long e2[4];
+#pragma unroll
+      for (int q = 0; q < 4; ++q) e2[q] = wk_pair(e[2 * q], e[2 * q + 1]);
       float* dst = sm.part[asub][warp & 3];
       const float* rb = sm.r + asub * 16 * kWkF + ac;
       const float* wb = sm.w + asub * 16 * kWkF + ac;
 #pragma unroll
       for (int t = 0; t < 16; ++t) {
-        float x[8], wv[8], a0 = 0.f, a1 = 0.f;
-        load8(rb + t * kWkF, x);
-        load8(wb + t * kWkF, wv);
-#pragma unroll
-        for (int q = 0; q < 8; q += 2) { a0 = fmaf(x[q], e[q], a0); a1 = fmaf(x[q + 1], e[q + 1], a1); }
+        unsigned long long x[4], wv[4];
+        wk_load4(x, rb + t * kWkF);
+        wk_load4(wv, wb + t * kWkF);
+        unsigned long long s0 = wk_mul2(x[0], e2[0]), s1 = wk_mul2(x[1], e2[1]);
+        s0 = wk_fma2(x[2], e2[2], s0);
+        s1 = wk_fma2(x[3], e2[3], s1);
         if (t > aj) {
 #pragma unroll
-          for (int q = 0; q < 8; ++q) e[q] *= wv[q];
+          for (int q = 0; q < 4; ++q) e2[q] = wk_mul2(e2[q], wv[q]);
         }
-        float a = t > aj ? a0 + a1 : (t == aj ? diag : 0.f);
+        const float2 f0 = wk_unpair(s0), f1 = wk_unpair(s1);
+        float a = t > aj ? (f0.x + f0.y) + (f1.x + f1.y) : (t == aj ? diag : 0.f);
         a += __shfl_xor_sync(0xffffffffu, a, 16);
         if (lane < 16) dst[t * 17 + aj] = a;
       }

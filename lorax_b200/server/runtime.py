@@ -342,8 +342,8 @@ class ShardRuntime:
         for bid in ids:
             for rid in self.batches.pop(bid, []):
                 self._drop(rid)
-        if not req.HasField("id") and self.kv.state_slots is not None:
-            for rid in [r for r in self.kv.state_slots.of_request if r not in self.seqs]:
+        if not req.HasField("id") and self.state_slots is not None:
+            for rid in [r for r in self.state_slots.of_request if r not in self.seqs]:
                 self._release_state(rid)
         if self.seqs:
             self._resort()
@@ -356,13 +356,20 @@ class ShardRuntime:
             self.runner.state.drop_row(s.row)
         self._release_state(rid)
 
+    kv = None                                                # (runtimes whose state lives with the request build no cache)
+
+    @property
+    def state_slots(self):
+        """Slots of the per-request recurrent state, or None."""
+        return self.kv.state_slots if self.kv is not None else None
+
     def _release_state(self, rid: int):
-        if self.kv.state_slots is not None:
-            self.kv.state_slots.release(rid)
+        if self.state_slots is not None:
+            self.state_slots.release(rid)
 
     def _state_slot(self, rid: int, cache_len: int, batch_ids) -> int:
         """The state slot of a request whose prompt (or the portion from `cache_len` on) is about to run; 0 for models without."""
-        slots = self.kv.state_slots
+        slots = self.state_slots
         if slots is None:
             return 0
         if cache_len > 0 and rid not in slots.of_request:

@@ -27,16 +27,40 @@ DECODER_MODEL_TYPES = (
 
 
 # Designs whose config.json lists its layers one by one, each with a mixer of its own (models/mixers.py).
-MIXER_MODEL_TYPES = ("vabunex",)
+MIXER_MODEL_TYPES = ("vabunex", "sapudra")
+
+
+@dataclass
+class MoeSpec:
+    """Routed feed-forward: `experts` of width `ff`, `top` of them per token, chosen within the best `keep` of `groups` groups of
+    neighbours (0: no groups); the chosen scores are normalised and multiplied by `scale`.  `shared_ff`: width of the gated expert
+    that every token takes beside them (0: none)."""
+    experts: int
+    top: int
+    ff: int
+    scale: float = 1.0
+    groups: int = 0
+    keep: int = 0
+    shared_ff: int = 0
+
+    def __post_init__(self):
+        if not 1 <= self.top <= self.experts:
+            raise ValueError(f"{self.top} of {self.experts} experts")
+        if self.groups:
+            if self.experts % self.groups or not 1 <= self.keep <= self.groups:
+                raise ValueError(f"{self.experts} experts in {self.groups} groups of which {self.keep} are kept")
+            if self.keep * (self.experts // self.groups) < self.top:
+                raise ValueError(f"{self.keep} groups of {self.experts // self.groups} experts cannot give {self.top}")
 
 
 @dataclass
 class LayerSpec:
-    """One layer of a design whose layers differ: the kind of mixer, the mixer's sizes and constants, and the width of the
-    gated feed-forward beside it (0: none)."""
+    """One layer of a design whose layers differ: the kind of mixer, the mixer's sizes and constants, and its feed-forward: dense of
+    width `ff` (0: none), or routed experts (`moe`)."""
     mixer: str
     params: Dict[str, Any]
     ff: int = 0
+    moe: Optional[MoeSpec] = None
 
 
 @dataclass
@@ -91,6 +115,9 @@ class ModelConfig:
     # layer-by-layer designs: the layers, and (start, stop, times): layers start .. stop-1 run `times` times in a row
     layer_specs: Optional[List[LayerSpec]] = None
     layer_loop: Optional[Tuple[int, int, int]] = None
+    # their residual: "parallel" (mixer and feed-forward read one norm of the stream, both are added to it) or "post" (each sublayer
+    # reads the stream itself, and a norm of its output, times residual_multiplier, is added)
+    layer_style: str = "parallel"
     eos_token_id: Any = None
     bos_token_id: Any = None
     pad_token_id: Any = None
@@ -250,26 +277,52 @@ class ModelConfig:
         return d
 
 
+def _moe_spec(mlp: Dict[str, Any]) -> MoeSpec:
+    r, groups, shared = mlp["router"], mlp["router"].get("groups"), mlp.get("shared")
+    return MoeSpec(experts=int(r["experts"]), top=int(r["top"]), ff=int(mlp["expert"]["ff"]), scale=float(r.get("scale", 1.0)),
+                   groups=int(groups["count"]) if groups else 0, keep=int(groups["keep"]) if groups else 0,
+                   shared_ff=int(shared["ff"]) if shared else 0)
+
+
+# What a layer-by-layer design fixes itself; everything else comes from its config.json.
+def _vabunex_constants(d: Dict[str, Any]) -> Dict[str, Any]:
+    return dict(layer_style="parallel", parallel_residual=True, hidden_act="gelu_tanh", norm_weight_offset=1.0,
+                embedding_multiplier=float(d["embedding"]["scale"]), max_position_embeddings=int(d.get("max_position_embeddings", 1 << 20)))
+
+
+def _sapudra_constants(d: Dict[str, Any]) -> Dict[str, Any]:
+    cap = d.get("logit_softcap")
+    return dict(layer_style="post", norm_type="layernorm", hidden_act="relu2", residual_multiplier=float(d["residual_mult"]),
+                learned_positions=True, max_position_embeddings=int(d["max_positions"]),
+                final_logit_softcapping=float(cap) if cap is not None else None)
+
+
+_MIXER_DESIGNS = {"vabunex": (_vabunex_constants, ("dense",)), "sapudra": (_sapudra_constants, ("dense", "moe"))}
+
+
 def _mixer_model_kwargs(mt: str, d: Dict[str, Any]) -> Dict[str, Any]:
-    """ModelConfig fields of a config.json that lists its layers (`layers`, `loop`, `norm`, `embedding`, `vocab`, `width`)."""
+    """ModelConfig fields of a config.json that lists its layers (`layers`, `loop`, `norm`, `vocab`, `width`)."""
+    constants, kinds = _MIXER_DESIGNS[mt]
     specs = []
     for i, layer in enumerate(d["layers"]):
         mlp = layer.get("mlp")
-        if mlp is not None and mlp.get("kind", "dense") != "dense":
-            raise NotImplementedError(f"layer {i}: feed-forward kind {mlp['kind']!r}")
-        specs.append(LayerSpec(layer["type"], dict(layer["mixer"]), int(mlp["ff"]) if mlp is not None else 0))
+        kind = mlp.get("kind", "dense") if mlp is not None else None
+        if kind is not None and kind not in kinds:
+            raise NotImplementedError(f"layer {i}: feed-forward kind {kind!r}")
+        specs.append(LayerSpec(layer["type"], dict(layer["mixer"]), int(mlp["ff"]) if kind == "dense" else 0,
+                               _moe_spec(mlp) if kind == "moe" else None))
     loop = d.get("loop")
     if loop is not None:
         loop = (int(loop["start"]), int(loop["stop"]), int(loop["times"]))
         if not (0 <= loop[0] <= loop[1] <= len(specs)) or loop[2] < 0:
             raise ValueError(f"loop {loop} does not fit {len(specs)} layers")
     heads = max([int(s.params["heads"]) for s in specs] + [1])
-    return dict(model_type=mt, vocab_size=int(d["vocab"]), hidden_size=int(d["width"]), intermediate_size=max([s.ff for s in specs] + [1]),
-                num_hidden_layers=len(specs), num_attention_heads=heads, head_dim=max([int(s.params["dim"]) for s in specs] + [1]),
-                rms_norm_eps=float(d["norm"]["eps"]), max_position_embeddings=int(d.get("max_position_embeddings", 1 << 20)),
-                hidden_act="gelu_tanh", norm_weight_offset=1.0, embedding_multiplier=float(d["embedding"]["scale"]), parallel_residual=True,
-                layer_specs=specs, layer_loop=loop, eos_token_id=d.get("eos_token_id"), bos_token_id=d.get("bos_token_id"),
-                torch_dtype=d.get("torch_dtype", "bfloat16"), extra={})
+    kv_heads = max([int(s.params.get("kv_heads", s.params["heads"])) for s in specs] + [1])
+    return dict(dict(model_type=mt, vocab_size=int(d["vocab"]), hidden_size=int(d["width"]), intermediate_size=max([s.ff for s in specs] + [1]),
+                     num_hidden_layers=len(specs), num_attention_heads=heads, num_key_value_heads=kv_heads,
+                     head_dim=max([int(s.params["dim"]) for s in specs] + [1]), rms_norm_eps=float(d["norm"]["eps"]), layer_specs=specs,
+                     layer_loop=loop, eos_token_id=d.get("eos_token_id"), bos_token_id=d.get("bos_token_id"),
+                     torch_dtype=d.get("torch_dtype", "bfloat16"), extra={}), **constants(d))
 
 
 def mistral_7b() -> ModelConfig:

@@ -15,6 +15,9 @@
 //                               per-block products O_j come back from TMEM and are folded into fp32 registers with the
 //                               usual rescaling, so nothing in TMEM ever has to be rescaled
 //
+// WIDE: the softmax weights stay fp32 up to the value product: each is split into two bf16 terms, value and remainder, in two operand
+// tiles, and P V is two products into the same accumulator (the layer-by-layer designs ask for it).
+//
 // Plain, chunked and prefix-cached prefill are one path: `cache_lens` says how many keys precede the chunk.  It replaces the
 // flash-attn-2 varlen call of the reference (server/lorax_server/utils/flash_attn.py:180-201) and the mma.sync kernel in
 // attention.cu, which stays for head sizes and group sizes this one does not take (d != 128, odd heads per KV head).
@@ -46,13 +49,14 @@ struct FaParams {
   int* status;
 };
 
+template <bool WIDE>
 struct FaSmem {
   static constexpr int kQBytes = 128 * kFaD * 2;             // two 64-wide halves of [128 rows x 64]
   static constexpr int kKBytes = kFaKeys * kFaD * 2;
   static constexpr int kVBytes = kFaKeys * kFaD * 2;
   static constexpr int kPBytes = 128 * kFaKeys * 2;
   static constexpr int kStage = kKBytes + kVBytes;
-  static constexpr int kTotal = kQBytes + 2 * kStage + kPBytes + 512 + 1024;
+  static constexpr int kTotal = kQBytes + 2 * kStage + (WIDE ? 2 : 1) * kPBytes + 512 + 1024;
 };
 
 // 5-D tiled load: the paged cache {d, slot in page, K|V, kv head, block}.
@@ -102,8 +106,8 @@ LX_DEVICE float fa_block_max(uint32_t ts, int kb0, int lo, int hi, float scale_l
 }
 
 // p = exp2(score - m_new) for the 128 keys of the block -> bf16, written as this row of the K-major, 128-byte-swizzled operand
-// tile; returns the row sum.
-template <bool PLAIN, bool MASK>
+// tile (WIDE: the remainders as the same row of the tile behind it); returns the row sum.
+template <bool PLAIN, bool MASK, bool WIDE>
 LX_DEVICE float fa_block_probs(uint32_t ts, uint8_t* prow, int row, int kb0, int lo, int hi, float m_new, float scale_l2, float softcap,
                                float scale, float slope_l2) {
   float sum = 0.f;
@@ -114,7 +118,7 @@ LX_DEVICE float fa_block_probs(uint32_t ts, uint8_t* prow, int row, int kb0, int
     uint32_t r[32];
     tmem_ld_32x32b_x32(ts + (uint32_t)c, r);
     tc_wait_ld();
-    uint32_t pk[16];
+    uint32_t pk[16], lo_pk[WIDE ? 16 : 1];
 #pragma unroll
     for (int q = 0; q < 32; q += 2) {
       float pv[2];
@@ -130,27 +134,35 @@ LX_DEVICE float fa_block_probs(uint32_t ts, uint8_t* prow, int row, int kb0, int
       }
       sum += pv[0] + pv[1];
       pk[q >> 1] = pack_bf16x2(pv[0], pv[1]);
+      if constexpr (WIDE) {
+        const float2 h = unpack_bf16x2(pk[q >> 1]);
+        lo_pk[q >> 1] = pack_bf16x2(pv[0] - h.x, pv[1] - h.y);
+      }
     }
     uint8_t* half = prow + (c >> 6) * 16384;
 #pragma unroll
     for (int ch = 0; ch < 4; ++ch) {
       const int chunk = ((c & 63) >> 3) + ch;
       *reinterpret_cast<uint4*>(half + ((chunk ^ (row & 7)) << 4)) = make_uint4(pk[4 * ch], pk[4 * ch + 1], pk[4 * ch + 2], pk[4 * ch + 3]);
+      if constexpr (WIDE)
+        *reinterpret_cast<uint4*>(half + 32768 + ((chunk ^ (row & 7)) << 4)) =
+            make_uint4(lo_pk[4 * ch], lo_pk[4 * ch + 1], lo_pk[4 * ch + 2], lo_pk[4 * ch + 3]);
     }
   }
   return sum;
 }
 
+template <bool WIDE>
 __global__ void __launch_bounds__(kFaThreads, 1)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_kv, const FaParams p) {
   pdl_trigger();
-  using S = FaSmem;
+  using S = FaSmem<WIDE>;
   extern __shared__ uint8_t fa_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(fa_raw) + 1023) & ~uintptr_t(1023));
   uint8_t* sq = smem;
   uint8_t* skv = smem + S::kQBytes;
   uint8_t* sp = skv + 2 * S::kStage;
-  uint64_t* bars = reinterpret_cast<uint64_t*>(sp + S::kPBytes);
+  uint64_t* bars = reinterpret_cast<uint64_t*>(sp + (WIDE ? 2 : 1) * S::kPBytes);
   uint64_t* q_full = bars;            // 1
   uint64_t* kv_full = bars + 1;       // 2
   uint64_t* kv_empty = bars + 3;      // 2
@@ -247,6 +259,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_
           const uint64_t da = make_desc_k_sw128(sp_a + (uint32_t)((ks >> 2) * 16384)) + (uint64_t)((ks & 3) * 2);
           const uint64_t db = make_desc_mn_sw128(sv_a + (uint32_t)(ks * 2048), 16384, 1024);
           umma_f16_ss(tmem_o, da, db, idesc_pv, ks > 0 ? 1u : 0u);
+          if constexpr (WIDE) umma_f16_ss(tmem_o, da + (uint64_t)(S::kPBytes >> 4), db, idesc_pv, 1u);
         }
         tc_commit(&pv_full[st]);
         tc_commit(p_empty);
@@ -316,9 +329,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_
       if (!mbar_wait(p_empty, (j & 1) ^ 1, abort_flag)) { report_status(p.status, kTimeoutTmemEmpty, tile); *abort_flag = 1; alive = false; break; }
       // pass 2: probabilities -> bf16 operand tile, row sum
       float sum;
-      if (plain) sum = need_mask ? fa_block_probs<true, true>(ts, prow, row, kb0, lo, hi, m_new, scale_l2, p.softcap, p.scale, slope_l2)
-                                 : fa_block_probs<true, false>(ts, prow, row, kb0, lo, hi, m_new, scale_l2, p.softcap, p.scale, slope_l2);
-      else sum = fa_block_probs<false, true>(ts, prow, row, kb0, lo, hi, m_new, scale_l2, p.softcap, p.scale, slope_l2);
+      if (plain) sum = need_mask ? fa_block_probs<true, true, WIDE>(ts, prow, row, kb0, lo, hi, m_new, scale_l2, p.softcap, p.scale, slope_l2)
+                                 : fa_block_probs<true, false, WIDE>(ts, prow, row, kb0, lo, hi, m_new, scale_l2, p.softcap, p.scale, slope_l2);
+      else sum = fa_block_probs<false, true, WIDE>(ts, prow, row, kb0, lo, hi, m_new, scale_l2, p.softcap, p.scale, slope_l2);
       tc_fence_before();
       mbar_arrive(&s_empty[st]);
       fence_proxy_async_smem();
@@ -394,6 +407,20 @@ static FaEncodeFn fa_encode_fn() {
   return fn;
 }
 
+template <bool WIDE>
+static int launch_fa(const CUtensorMap& tq, const CUtensorMap& tkv, const FaParams& p, int num_tiles, cudaStream_t s) {
+  static bool configured[64] = {false};
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (dev < 0 || dev >= 64 || !configured[dev]) {
+    cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<WIDE>, cudaFuncAttributeMaxDynamicSharedMemorySize, FaSmem<WIDE>::kTotal);
+    if (e != cudaSuccess) return -(int)e;
+    if (dev >= 0 && dev < 64) configured[dev] = true;
+  }
+  launch_pdl(attn_prefill_tc_kernel<WIDE>, dim3(num_tiles, p.nh / 2), dim3(kFaThreads), (size_t)FaSmem<WIDE>::kTotal, s, tq, tkv, p);
+  return -(int)cudaGetLastError();
+}
+
 }  // namespace lx
 
 extern "C" {
@@ -404,10 +431,10 @@ int lx_attn_prefill_tc_supported(int nh, int nkv, int d, long long ldq, long lon
 }
 
 // Same contract as lx_attn_prefill_alibi (64-query tiles listed by tile_seq / tile_q0), plus the number of tokens `T` of the q
-// buffer and the number of blocks of the cache (bounds of the two tensor maps) and the status word.
+// buffer and the number of blocks of the cache (bounds of the two tensor maps) and the status word.  wide: fp32 softmax weights.
 int lx_attn_prefill_tc(const void* q, long long ldq, int T, const void* kv, int num_blocks, const int* block_tables, int max_blocks,
                        const int* cu_q, const int* cache_lens, const int* tile_seq, const int* tile_q0, int num_tiles, void* out, long long ldo,
-                       int nh, int nkv, int d, int window, float scale, float softcap, const float* alibi, int* status, void* stream) {
+                       int nh, int nkv, int d, int window, float scale, float softcap, const float* alibi, int wide, int* status, void* stream) {
   using namespace lx;
   if (num_tiles <= 0) return 0;
   if (!lx_attn_prefill_tc_supported(nh, nkv, d, ldq, ldo)) return -1;
@@ -438,17 +465,8 @@ int lx_attn_prefill_tc(const void* q, long long ldq, int T, const void* kv, int 
   p.tile_seq = tile_seq; p.tile_q0 = tile_q0;
   p.out = reinterpret_cast<__nv_bfloat16*>(out); p.ldo = ldo;
   p.nh = nh; p.nkv = nkv; p.group = nh / nkv; p.window = window; p.scale = scale; p.softcap = softcap; p.alibi = alibi; p.status = status;
-  static bool configured[64] = {false};
-  int dev = 0;
-  cudaGetDevice(&dev);
-  if (dev < 0 || dev >= 64 || !configured[dev]) {
-    cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, FaSmem::kTotal);
-    if (e != cudaSuccess) return -(int)e;
-    if (dev >= 0 && dev < 64) configured[dev] = true;
-  }
-  launch_pdl(attn_prefill_tc_kernel, dim3(num_tiles, nh / 2), dim3(kFaThreads), (size_t)FaSmem::kTotal, reinterpret_cast<cudaStream_t>(stream),
-             tq, tkv, p);
-  return -(int)cudaGetLastError();
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  return wide ? launch_fa<true>(tq, tkv, p, num_tiles, st) : launch_fa<false>(tq, tkv, p, num_tiles, st);
 }
 
 }  // extern "C"

@@ -230,7 +230,7 @@ rope_kvwrite_kernel(__nv_bfloat16* __restrict__ qkv, const int* __restrict__ pos
 // ------------------------------------------------------------------------------------------------
 // out[t, i] = act(gate_up[t, i]) * gate_up[t, I + i]
 // ------------------------------------------------------------------------------------------------
-enum Act : int { kSilu = 0, kGelu = 1, kGeluTanh = 2, kRelu = 3 };
+enum Act : int { kSilu = 0, kGelu = 1, kGeluTanh = 2, kRelu = 3, kRelu2 = 4 };
 template <int ACT>
 LX_DEVICE float act_fn(float x) {
   if (ACT == kSilu) return x / (1.f + __expf(-x));
@@ -239,7 +239,8 @@ LX_DEVICE float act_fn(float x) {
     const float u = 0.7978845608028654f * (x + 0.044715f * x * x * x);
     return 0.5f * x * (1.f + tanhf(u));
   }
-  return fmaxf(x, 0.f);
+  const float r = fmaxf(x, 0.f);
+  return ACT == kRelu2 ? r * r : r;
 }
 template <int ACT, bool GATED>
 __global__ void __launch_bounds__(256)
@@ -478,6 +479,7 @@ int lx_act_mul(const void* in, void* out, int T, int I, long long ldi, long long
     case kSilu: LX_ACT(kSilu); break;
     case kGelu: LX_ACT(kGelu); break;
     case kGeluTanh: LX_ACT(kGeluTanh); break;
+    case kRelu2: LX_ACT(kRelu2); break;
     default: LX_ACT(kRelu); break;
   }
 #undef LX_ACT

@@ -5,21 +5,30 @@
 namespace lx {
 
 // ------------------------------------------------------------------------------------------------
-// Residual stream: x[t] = table[ids[t]] * mult in fp32.
+// Residual stream: x[t] = table[ids[t]] * mult (+ pos[positions[t]]) in fp32; `copy` takes x in the model's dtype.
 // ------------------------------------------------------------------------------------------------
 template <typename T>
 __global__ void __launch_bounds__(128) embed_stream_kernel(const int* __restrict__ ids, const T* __restrict__ table, float* __restrict__ out,
-                                                           int W, int V, float mult) {
+                                                           int W, int V, float mult, const T* __restrict__ pos,
+                                                           const int* __restrict__ positions, int P, T* __restrict__ copy) {
   pdl_trigger();
   pdl_wait();
   const int t = blockIdx.x;
   const int id = min(max(ids[t], 0), V - 1);
+  const int at = pos != nullptr ? min(max(positions[t], 0), P - 1) : 0;
   for (int c = threadIdx.x * 8; c < W; c += blockDim.x * 8) {
     float f[8];
     load8(table + (long long)id * W + c, f);
 #pragma unroll
     for (int q = 0; q < 8; ++q) f[q] *= mult;
+    if (pos != nullptr) {
+      float g[8];
+      load8(pos + (long long)at * W + c, g);
+#pragma unroll
+      for (int q = 0; q < 8; ++q) f[q] += g[q];
+    }
     store8(out + (long long)t * W + c, f);
+    if (copy != nullptr) store8(copy + (long long)t * W + c, f);
   }
 }
 
@@ -65,6 +74,133 @@ __global__ void __launch_bounds__(kNsThreads) norm_stream_kernel(float* __restri
       for (int q = 0; q < 8; ++q) g[q] = v[it][q] * r * (g[q] + w_offset);
       store8(out + row + c, g);
     }
+  }
+}
+
+// ------------------------------------------------------------------------------------------------
+// Norm of a sublayer's output, added to the stream: residual += mult * (norm(y) * w + b), copy = residual in the model's dtype.  One
+// CTA per row.  Columns from n on are padding: they take no part in mean and variance, and w and b are zero there.  PAIRS: y of a
+// token is the weighted sum of the rows pos[t, 0 .. k) (-1: none) of y (the outputs of its experts).
+// ------------------------------------------------------------------------------------------------
+struct NormAddParams {
+  float* residual;
+  const void* y;
+  long long ldy;
+  const float* w;
+  const float* b;              // or null
+  void* copy;                  // or null
+  const int* pos;              // [T, k]
+  const float* weights;        // [T, k]
+  int k, W, n, layernorm;
+  float inv_n, eps, mult;
+};
+
+// In place on a row held as NV vectors of eight columns per thread: v <- norm(v) * w + b.
+template <int NV>
+LX_DEVICE void norm_row(float (&v)[NV][8], const float* __restrict__ w, const float* __restrict__ b, int W, int n, float inv_n, float eps,
+                        int layernorm, float w_offset, float* red) {
+  float mean = 0.f;
+  if (layernorm) {
+    float s = 0.f;
+#pragma unroll
+    for (int it = 0; it < NV; ++it)
+#pragma unroll
+      for (int q = 0; q < 8; ++q) s += v[it][q];                   // (padding holds zeros)
+    mean = block_sum(s, red) * inv_n;
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int it = 0; it < NV; ++it) {
+    const int c = (threadIdx.x + it * blockDim.x) * 8;
+#pragma unroll
+    for (int q = 0; q < 8; ++q) {
+      v[it][q] -= mean;
+      if (c + q < n) ss += v[it][q] * v[it][q];
+    }
+  }
+  const float r = rsqrtf(block_sum(ss, red) * inv_n + eps);
+#pragma unroll
+  for (int it = 0; it < NV; ++it) {
+    const int c = (threadIdx.x + it * blockDim.x) * 8;
+    if (c < W) {
+      float g[8], h[8];
+      load8(w + c, g);
+#pragma unroll
+      for (int q = 0; q < 8; ++q) h[q] = 0.f;
+      if (b != nullptr) load8(b + c, h);
+#pragma unroll
+      for (int q = 0; q < 8; ++q) v[it][q] = v[it][q] * r * (g[q] + w_offset) + h[q];
+    }
+  }
+}
+
+template <typename T, bool PAIRS, int NV>
+__global__ void __launch_bounds__(kNsThreads) norm_add_kernel(const NormAddParams p) {
+  pdl_trigger();
+  pdl_wait();
+  __shared__ float red[kNsThreads / 32];
+  const int t = blockIdx.x;
+  const T* y = reinterpret_cast<const T*>(p.y);
+  float v[NV][8];
+#pragma unroll
+  for (int it = 0; it < NV; ++it) {
+    const int c = (threadIdx.x + it * blockDim.x) * 8;
+#pragma unroll
+    for (int q = 0; q < 8; ++q) v[it][q] = 0.f;
+    if (c >= p.W) continue;
+    if constexpr (PAIRS) {
+      for (int j = 0; j < p.k; ++j) {
+        const int row = p.pos[(long long)t * p.k + j];
+        if (row < 0) continue;
+        const float wj = p.weights[(long long)t * p.k + j];
+        float f[8];
+        load8(y + (long long)row * p.ldy + c, f);
+#pragma unroll
+        for (int q = 0; q < 8; ++q) v[it][q] = fmaf(wj, f[q], v[it][q]);
+      }
+    } else {
+      load8(y + (long long)t * p.ldy + c, v[it]);
+    }
+  }
+  norm_row<NV>(v, p.w, p.b, p.W, p.n, p.inv_n, p.eps, p.layernorm, 0.f, red);
+  float* res = p.residual + (long long)t * p.W;
+  T* copy = reinterpret_cast<T*>(p.copy);
+#pragma unroll
+  for (int it = 0; it < NV; ++it) {
+    const int c = (threadIdx.x + it * blockDim.x) * 8;
+    if (c < p.W) {
+      float x[8];
+      load8(res + c, x);
+#pragma unroll
+      for (int q = 0; q < 8; ++q) x[q] = fmaf(p.mult, v[it][q], x[q]);
+      store8(res + c, x);
+      if (copy != nullptr) store8(copy + (long long)t * p.W + c, x);
+    }
+  }
+}
+
+// out[i] = norm(residual[rows[i]]) (rows null: every row)
+template <typename T>
+__global__ void __launch_bounds__(kNsThreads) norm_rows_kernel(const float* __restrict__ residual, const int* __restrict__ rows,
+                                                               const float* __restrict__ w, const float* __restrict__ b, T* __restrict__ out,
+                                                               int W, int n, float inv_n, float eps, float w_offset, int layernorm) {
+  pdl_trigger();
+  pdl_wait();
+  __shared__ float red[kNsThreads / 32];
+  const float* res = residual + (long long)(rows != nullptr ? rows[blockIdx.x] : (int)blockIdx.x) * W;
+  float v[kNsMaxVec][8];
+#pragma unroll
+  for (int it = 0; it < kNsMaxVec; ++it) {
+    const int c = (threadIdx.x + it * blockDim.x) * 8;
+#pragma unroll
+    for (int q = 0; q < 8; ++q) v[it][q] = 0.f;
+    if (c < W) load8(res + c, v[it]);
+  }
+  norm_row<kNsMaxVec>(v, w, b, W, n, inv_n, eps, layernorm, w_offset, red);
+#pragma unroll
+  for (int it = 0; it < kNsMaxVec; ++it) {
+    const int c = (threadIdx.x + it * blockDim.x) * 8;
+    if (c < W) store8(out + (long long)blockIdx.x * W + c, v[it]);
   }
 }
 
@@ -119,7 +255,7 @@ __global__ void __launch_bounds__(256) tanh_kernel(T* __restrict__ x, long long 
   }
 }
 
-// out[t, i] = gelu_tanh(x[t, i]) * x[t, I + i] (or silu) for fp32 rows
+// out[t, i] = act(x[t, i]) (* x[t, I + i]) for fp32 rows
 __global__ void __launch_bounds__(256) act_mul_f32_kernel(const float* __restrict__ x, float* __restrict__ out, int I, long long ldx,
                                                           long long ldo, long long total4, int act, int gated) {
   pdl_trigger();
@@ -136,7 +272,7 @@ __global__ void __launch_bounds__(256) act_mul_f32_kernel(const float* __restric
       if (act == 0) e[q] = silu_f(z);
       else if (act == 1) e[q] = 0.5f * z * (1.f + erff(z * 0.70710678118654752f));
       else if (act == 2) e[q] = 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
-      else e[q] = fmaxf(z, 0.f);
+      else { const float r = fmaxf(z, 0.f); e[q] = act == 4 ? r * r : r; }
     }
     if (gated) {
       const float4 u = load4(x + t * ldx + I + c);
@@ -316,14 +452,54 @@ __global__ void __launch_bounds__(128) gemm_heads_kernel(const BatchedGemmParams
 extern "C" {
 
 // `f32` selects the element type of activations and weights everywhere below (0: bf16, 1: fp32).
-int lx_embed_stream(const int* ids, const void* table, void* out, int T, int W, int V, float mult, int f32, void* stream) {
+int lx_embed_stream(const int* ids, const void* table, void* out, int T, int W, int V, float mult, const void* pos, const int* positions, int P,
+                    void* copy, int f32, void* stream) {
   using namespace lx;
   if (T <= 0) return 0;
-  if (W % 8 != 0 || V <= 0) return -1;
+  if (W % 8 != 0 || V <= 0 || (pos != nullptr && P <= 0)) return -1;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   float* o = reinterpret_cast<float*>(out);
-  if (f32) launch_pdl(embed_stream_kernel<float>, dim3(T), dim3(128), 0, s, ids, reinterpret_cast<const float*>(table), o, W, V, mult);
-  else launch_pdl(embed_stream_kernel<__nv_bfloat16>, dim3(T), dim3(128), 0, s, ids, reinterpret_cast<const __nv_bfloat16*>(table), o, W, V, mult);
+#define LX_ES(TY)                                                                                                                        \
+  launch_pdl(embed_stream_kernel<TY>, dim3(T), dim3(128), 0, s, ids, reinterpret_cast<const TY*>(table), o, W, V, mult,                     \
+             reinterpret_cast<const TY*>(pos), positions, P, reinterpret_cast<TY*>(copy))
+  if (f32) LX_ES(float); else LX_ES(__nv_bfloat16);
+#undef LX_ES
+  return -(int)cudaGetLastError();
+}
+
+int lx_norm_add_bytes() { return (int)sizeof(lx::NormAddParams); }
+
+int lx_norm_add(const void* params, int T, int f32, void* stream) {
+  using namespace lx;
+  const NormAddParams& p = *reinterpret_cast<const NormAddParams*>(params);
+  if (T <= 0) return 0;
+  if (p.W % 8 != 0 || p.W > kNsThreads * kNsMaxVec * 8 || p.n <= 0 || p.n > p.W || p.ldy % 8 != 0 || p.ldy < p.W) return -1;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  const int threads = p.W / 8 >= kNsThreads ? kNsThreads : (p.W / 8 + 31) / 32 * 32;
+  const int nv = (p.W / 8 + threads - 1) / threads;
+#define LX_NA(TY, PR)                                                                                   \
+  if (nv <= 1) launch_pdl(norm_add_kernel<TY, PR, 1>, dim3(T), dim3(threads), 0, s, p);                   \
+  else if (nv <= 2) launch_pdl(norm_add_kernel<TY, PR, 2>, dim3(T), dim3(threads), 0, s, p);              \
+  else if (nv <= 4) launch_pdl(norm_add_kernel<TY, PR, 4>, dim3(T), dim3(threads), 0, s, p);              \
+  else launch_pdl(norm_add_kernel<TY, PR, kNsMaxVec>, dim3(T), dim3(threads), 0, s, p);
+  if (f32) { if (p.pos != nullptr) { LX_NA(float, true) } else { LX_NA(float, false) } }
+  else { if (p.pos != nullptr) { LX_NA(__nv_bfloat16, true) } else { LX_NA(__nv_bfloat16, false) } }
+#undef LX_NA
+  return -(int)cudaGetLastError();
+}
+
+int lx_norm_rows(const void* residual, const int* rows, const void* w, const void* b, void* out, int T, int W, int n, float eps, float w_offset,
+                 int layernorm, int f32, void* stream) {
+  using namespace lx;
+  if (T <= 0) return 0;
+  if (W % 8 != 0 || W > kNsThreads * kNsMaxVec * 8 || n <= 0 || n > W) return -1;
+  const int threads = W / 8 >= kNsThreads ? kNsThreads : (W / 8 + 31) / 32 * 32;
+#define LX_NR(TY)                                                                                                                       \
+  launch_pdl(norm_rows_kernel<TY>, dim3(T), dim3(threads), 0, reinterpret_cast<cudaStream_t>(stream), reinterpret_cast<const float*>(residual), \
+             rows, reinterpret_cast<const float*>(w), reinterpret_cast<const float*>(b), reinterpret_cast<TY*>(out), W, n, 1.f / n, eps, w_offset, \
+             layernorm)
+  if (f32) LX_NR(float); else LX_NR(__nv_bfloat16);
+#undef LX_NR
   return -(int)cudaGetLastError();
 }
 

@@ -516,6 +516,8 @@ class DecoderModel:
         """-> logits [n_out, vocab] (full vocabulary on every rank)."""
         c, ops = self.config, self.ops
         if self.mixed:
+            if c.layer_style == "post":
+                return self._forward_post(inp, kv_cache)
             # fp32 residual stream; every layer hands its contribution to the norm that reads the stream next
             residual, pending = ops.embed_stream(inp.input_ids, self.embed, c.embedding_multiplier), None
             for run, li in enumerate(self.schedule):
@@ -564,9 +566,22 @@ class DecoderModel:
         hidden = self._norm(pending, residual, self.final_norm, self.final_norm_b, x_scale=rm)
         return self._score(hidden, inp)
 
-    def _score(self, hidden: torch.Tensor, inp: StepInputs) -> torch.Tensor:
-        """Logits of the rows the step asks for."""
-        if inp.lm_head_indices is not None:
+    def _forward_post(self, inp: StepInputs, kv_cache) -> torch.Tensor:
+        """Layers that read the fp32 stream itself: every addition to the stream also leaves its copy in the model's dtype."""
+        c, ops = self.config, self.ops
+        T = inp.input_ids.shape[0]
+        h = torch.empty(T, self.embed.shape[1], dtype=self.dtype, device=self.device) if self.dtype != torch.float32 else None
+        residual = ops.embed_stream(inp.input_ids, self.embed, c.embedding_multiplier, pos=self.pos_embed, positions=inp.positions, copy=h)
+        h = residual if h is None else h
+        for run, li in enumerate(self.schedule):
+            h = self.layers[li].forward(self, residual, h, inp, kv_cache[run])
+        hidden = ops.norm_stream(residual, None, self.final_norm, self.eps, c.norm_weight_offset, self.hidden, self.dtype, bias=self.final_norm_b,
+                                 layernorm=c.norm_type == "layernorm", rows=inp.lm_head_indices)
+        return self._score(hidden, inp, selected=True)
+
+    def _score(self, hidden: torch.Tensor, inp: StepInputs, selected: bool = False) -> torch.Tensor:
+        """Logits of the rows the step asks for (`selected`: `hidden` holds only those)."""
+        if inp.lm_head_indices is not None and not selected:
             hidden = hidden.index_select(0, inp.lm_head_indices.long()) if hidden.device.type == "cpu" else hidden[inp.lm_head_indices.long()]
         if self.keep_hidden:
             self.last_hidden = hidden          # rows match the returned logits (Medusa heads read them)

@@ -1,9 +1,13 @@
-"""Layers of designs that list their layers one by one: a token mixer and an optional gated feed-forward in parallel, both reading
-one RMS norm of the fp32 residual stream.
+"""Layers of designs that list their layers one by one, over an fp32 residual stream.  Two styles:
+
+  parallel   a token mixer and an optional gated feed-forward side by side, both reading one RMS norm of the stream (`MixerLayer`)
+  post       the mixer, then the feed-forward (dense or routed experts), each reading the stream itself; the norm of its output is
+             added to the stream (`PostNormLayer`)
 
 A mixer declares its tensors (`shapes`), what it keeps per token or per request (`cache_shape`), which of its projections read the
-layer's norm (`in_parts`, fused with the feed-forward's gate and up projections into one GEMM) and its output projection (`out_parts`,
-fused with the down projection into one GEMM: the sum of both sublayers is formed in the accumulator).  All sizes are padded to
+layer's input (`in_parts`, one GEMM; in a parallel layer together with the feed-forward's gate and up projections) and its output
+projection (`out_part`; in a parallel layer fused with the down projection into one GEMM: the sum of both sublayers is formed in the
+accumulator).  All sizes are padded to
 multiples of 16 with zero weights when the layer is loaded, so the kernels see aligned heads whatever the configuration says; a padded
 channel stays exactly zero through every operation.
 
@@ -11,6 +15,7 @@ channel stays exactly zero through every operation.
   wkv               token-shifted linear recurrence with a data-dependent decay per key channel, state [heads, dim, dim] per request
                     plus the previous token's input
   latent_attention  softmax attention over a low-rank latent and one shared rotated key part per token, both paged
+  attention         grouped-query softmax attention over paged keys and values, normed queries and keys, a sliding window of its own
 """
 
 from __future__ import annotations
@@ -74,7 +79,7 @@ class Mixer:
         raise NotImplementedError
 
     def cache_shape(self, model) -> dict:
-        """{"paged": width per token} or {"state": {name: (shape per request, dtype)}}."""
+        """{"paged": width per token}, {"kv": (heads, key width, value width)} or {"state": {name: (shape per request, dtype)}}."""
         raise NotImplementedError
 
     def run(self, model, h, proj, y, inp, cache):
@@ -232,7 +237,54 @@ class LatentAttentionMixer(Mixer):
         ops.gemm_heads(o_lat, self.uv, y, self.kvp, gate=gate)
 
 
-MIXERS = {"lightning": LightningMixer, "wkv": WkvMixer, "latent_attention": LatentAttentionMixer}
+class AttentionMixer(Mixer):
+    """Grouped-query attention.  Queries and keys are divided by their root mean square per head (weights shared by the heads); no
+    rotation; token i sees the last `mask.size` tokens including itself."""
+
+    HEAD_SIZES = (64, 128, 256)                              # of the attention kernels; a head is padded to the next one
+
+    def __init__(self, params: dict, width: int):
+        super().__init__(params, width)
+        self.H, self.G, self.d, self.dv = (int(params[n]) for n in ("heads", "kv_heads", "dim", "vdim"))
+        if self.H % self.G:
+            raise ValueError(f"{self.H} query heads over {self.G} key/value heads")
+        self.scale, self.window = float(params["scale"]), int(params["mask"]["size"])
+        if self.window < 1:
+            raise ValueError(f"a window of {self.window} tokens")
+        self.dp, self.dvp = self._padded(self.d), self._padded(self.dv)
+        self.out_dim = self.H * self.dvp
+
+    def _padded(self, n: int) -> int:
+        for size in self.HEAD_SIZES:
+            if n <= size:
+                return size
+        raise NotImplementedError(f"attention heads of {n} (up to {self.HEAD_SIZES[-1]})")
+
+    def shapes(self):
+        H, G, d, dv, w = self.H, self.G, self.d, self.dv, self.width
+        return {"q": (H * d, w), "k": (G * d, w), "v": (G * dv, w), "q.norm": (d,), "k.norm": (d,), "o": (w, H * dv)}
+
+    def in_parts(self, get):
+        rows = lambda n, heads, d, dp: _pad_to(get(n).view(heads, d, -1), heads, dp, self.W).reshape(heads * dp, self.W)
+        return [("qkv", torch.cat([rows("q", self.H, self.d, self.dp), rows("k", self.G, self.d, self.dp), rows("v", self.G, self.dv, self.dvp)]))]
+
+    def out_part(self, get):
+        o = get("o")
+        return _pad_to(o.view(o.shape[0], self.H, self.dv), self.W, self.H, self.dvp).reshape(self.W, self.out_dim)
+
+    def load(self, get, fin, vec, model):
+        self.q_norm, self.k_norm = (vec(_pad_to(get(n), self.dp)) for n in ("q.norm", "k.norm"))
+
+    def cache_shape(self, model):
+        return {"kv": (self.G, self.dp, self.dvp)}
+
+    def run(self, model, h, proj, y, inp, cache):
+        qkv = proj["qkv"]
+        model.ops.qk_norm_kvwrite(qkv, self.H, self.G, self.dp, self.dvp, self.d, self.q_norm, self.k_norm, model.eps, cache, inp.slots)
+        model.ops.gqa_attn(qkv, cache, self.H, self.G, self.dp, self.dvp, self.scale, self.window, inp, y)
+
+
+MIXERS = {"lightning": LightningMixer, "wkv": WkvMixer, "latent_attention": LatentAttentionMixer, "attention": AttentionMixer}
 
 
 def make_mixer(spec, width: int) -> Mixer:
@@ -266,9 +318,122 @@ class MixerLayer:
         return ops.gemm(y, self.out_w)
 
 
+class DenseMlp:
+    """down(act(up(h))), no gate."""
+
+    def __init__(self, ff: int, width: int):
+        self.ff, self.width, self.W = ff, width, pad16(width)
+        self.fp = pad16(ff)
+
+    def shapes(self):
+        return {"up": (self.ff, self.width), "down": (self.width, self.ff)}
+
+    def load(self, get, fin, vec, model):
+        self.up, self.down = fin(_pad_to(get("up"), self.fp, self.W)), fin(_pad_to(get("down"), self.W, self.fp))
+
+    def run(self, model, h):
+        """-> (rows, None): one row per token."""
+        ops = model.ops
+        return ops.gemm(ops.act_mul(ops.gemm(h, self.up), self.fp, model.config.hidden_act, gated=False), self.down), None
+
+
+class MoeMlp:
+    """Routed experts down(act(up(h))) with sigmoid scores, a correction that takes part in the choice only, and groups of neighbours.
+
+    The shared expert is cut into slices of an expert's (padded) width; every token takes each slice with the weight
+    sigmoid(sg . h), so the slices ride in the grouped products as further experts, and `sg` is one more row of the router."""
+
+    TILE = 128                                               # features per work item of the grouped products
+
+    def __init__(self, spec, width: int):
+        self.spec, self.width, self.W = spec, width, pad16(width)
+        up = lambda n: (n + self.TILE - 1) // self.TILE * self.TILE
+        self.fp, self.Wp = up(spec.ff), up(self.W)
+        self.slices = (spec.shared_ff + self.fp - 1) // self.fp
+        if spec.experts > 256 or spec.top > 32 or self.slices > 32:      # tables of the routing kernels
+            raise NotImplementedError(f"{spec.experts} experts, {spec.top} per token, a shared expert of {self.slices} expert widths")
+
+    def shapes(self):
+        s, w = self.spec, self.width
+        out = {"router": (s.experts, w), "correction": (s.experts,)}
+        for e in range(s.experts):
+            out.update({f"e{e}.up": (s.ff, w), f"e{e}.down": (w, s.ff)})
+        if s.shared_ff:
+            out.update({"shared.up": (s.shared_ff, w), "shared.down": (w, s.shared_ff), "shared.sg": (1, w)})
+        return out
+
+    def load(self, get, fin, vec, model):
+        s, n = self.spec, self.spec.experts + self.slices
+        new = lambda *shape: torch.zeros(*shape, dtype=model.dtype, device=model.device)
+        self.up, self.down = new(n, self.fp, self.W), new(n, self.Wp, self.fp)
+        for e in range(s.experts):
+            self.up[e, : s.ff, : self.width] = fin(get(f"e{e}.up"))
+            self.down[e, : self.width, : s.ff] = fin(get(f"e{e}.down"))
+        router = [get("router")]
+        if s.shared_ff:
+            up, down = fin(get("shared.up")), fin(get("shared.down"))
+            for i in range(self.slices):
+                a, b = i * self.fp, min((i + 1) * self.fp, s.shared_ff)
+                self.up[s.experts + i, : b - a, : self.width] = up[a:b]
+                self.down[s.experts + i, : self.width, : b - a] = down[:, a:b]
+            router.append(get("shared.sg"))
+        self.router = fin(_pad_to(torch.cat(router), pad16(s.experts + 1), self.W))
+        self.correction = vec(get("correction"))
+
+    def run(self, model, h):
+        """-> (rows of every (token, expert) pair, (row, weight) of each token's pairs)."""
+        s, ops = self.spec, model.ops
+        r = ops.moe_route(h, self.router, s.top, 0, s.experts, experts=s.experts, score="sigmoid", correction=self.correction, groups=s.groups,
+                          keep=s.keep, scale=s.scale, shared=self.slices)
+        avg = max(1, (h.shape[0] * s.top + s.experts - 1) // s.experts)
+        a = ops.moe_grouped_gemm(r.xg, self.up, r.seg, avg, shared=self.slices, tokens=h.shape[0], act=model.config.hidden_act)
+        return ops.moe_grouped_gemm(a, self.down, r.seg, avg), (r.pos, r.topk_w)
+
+
+@dataclass
+class PostNormLayer:
+    """x += mult * norm1(mixer(x)), then x += mult * norm2(ff(x)).  The stream is fp32; `h` is its copy in the model's dtype that the
+    products read, written by whoever last added to the stream."""
+    mixer: Mixer
+    mlp: Optional[object]                                    # DenseMlp, MoeMlp or None
+    norm1: Tuple[torch.Tensor, torch.Tensor] = None          # weight, bias: fp32 [W]
+    norm2: Optional[Tuple[torch.Tensor, torch.Tensor]] = None
+    in_w: Optional[torch.Tensor] = None
+    out_w: Optional[torch.Tensor] = None
+    parts: Dict[str, Tuple[int, int]] = field(default_factory=dict)
+
+    def forward(self, model, residual, h, inp, cache):
+        """Adds both sublayers to `residual`; -> its new copy."""
+        ops, m, c = model.ops, self.mixer, model.config
+        proj = ops.gemm(h, self.in_w)
+        y = torch.empty(h.shape[0], m.out_dim, dtype=h.dtype, device=h.device)
+        m.run(model, h, {n: proj[:, a:b] for n, (a, b) in self.parts.items()}, y, inp, cache)
+        add = lambda rows, norm, pairs=None: ops.norm_add(residual, rows, norm[0], norm[1], c.residual_multiplier, model.eps, model.hidden,
+                                                          model.dtype, layernorm=True, pairs=pairs)
+        h = add(ops.gemm(y, self.out_w), self.norm1)
+        if self.mlp is not None:
+            rows, pairs = self.mlp.run(model, h)
+            h = add(rows, self.norm2, pairs)
+        return h
+
+
+def make_mlp(spec, width: int):
+    if spec.moe is not None:
+        return MoeMlp(spec.moe, width)
+    return DenseMlp(spec.ff, width) if spec.ff else None
+
+
+def _parts(layer, rows):
+    """Row ranges of the fused input projection -> layer.parts."""
+    o = 0
+    for name, t in rows:
+        layer.parts[name] = (o, o + t.shape[0])
+        o += t.shape[0]
+
+
 def load_mixer_layers(m, w):
-    """Tensors of a layer-by-layer checkpoint -> `m` (a DecoderModel): `embed`, `l<i>.norm1`, `l<i>.mix.*`, `l<i>.mlp.*`,
-    `final.norm`, `head`."""
+    """Tensors of a layer-by-layer checkpoint -> `m` (a DecoderModel): `embed`, `pos`, `l<i>.norm1`, `l<i>.norm2`, `l<i>.mix.*`,
+    `l<i>.mlp.*`, `final.norm`, `head`; a layer norm's bias is called like its weight with `.b` added."""
     c, dt, dev = m.config, m.dtype, m.device
     if m.tp.world_size > 1:
         raise ValueError(f"{c.model_type} is served on one shard")
@@ -286,7 +451,25 @@ def load_mixer_layers(m, w):
     m.embed = fin(_pad_to(get("embed"), c.vocab_size, W))
     m.lm_head = fin(_pad_to(get("head"), pad16(c.vocab_size), W))
     m.final_norm = vec(_pad_to(get("final.norm"), W))
+    if c.learned_positions:
+        m.pos_embed = fin(_pad_to(get("pos"), c.max_position_embeddings, W))
+    if c.norm_type == "layernorm":
+        m.final_norm_b = vec(_pad_to(get("final.norm.b"), W))
     m.layers = []
+    if c.layer_style == "post":
+        norm = lambda name: (vec(_pad_to(get(name), W)), vec(_pad_to(get(name + ".b"), W)))
+        for i, spec in enumerate(c.layer_specs):
+            layer = PostNormLayer(make_mixer(spec, c.hidden_size), make_mlp(spec, c.hidden_size), norm(f"l{i}.norm1"))
+            sub = lambda name, i=i: get(f"l{i}.mix.{name}")
+            rows = layer.mixer.in_parts(sub)
+            _parts(layer, rows)
+            layer.in_w, layer.out_w = fin(torch.cat([t for _, t in rows])), fin(layer.mixer.out_part(sub))
+            layer.mixer.load(sub, fin, vec, m)
+            if layer.mlp is not None:
+                layer.norm2 = norm(f"l{i}.norm2")
+                layer.mlp.load(lambda name, i=i: get(f"l{i}.mlp.{name}"), fin, vec, m)
+            m.layers.append(layer)
+        return
     for i, spec in enumerate(c.layer_specs):
         mx = make_mixer(spec, c.hidden_size)
         ff = pad16(spec.ff) if spec.ff else 0
@@ -297,10 +480,7 @@ def load_mixer_layers(m, w):
         if ff:
             rows.append(("mlp", torch.cat([_pad_to(get(f"l{i}.mlp.{n}"), ff, W) for n in ("gate", "up")])))
             out.append(_pad_to(get(f"l{i}.mlp.down"), W, ff))
-        o = 0
-        for name, t in rows:
-            layer.parts[name] = (o, o + t.shape[0])
-            o += t.shape[0]
+        _parts(layer, rows)
         layer.in_w = fin(torch.cat([t for _, t in rows])) if rows else None
         layer.out_w = fin(torch.cat(out, 1))
         mx.load(sub, fin, vec, m)
@@ -311,6 +491,15 @@ def tensor_shapes(c) -> Dict[str, Tuple[int, ...]]:
     """Name -> shape of every tensor of a layer-by-layer checkpoint of this configuration."""
     w = c.hidden_size
     out = {"embed": (c.vocab_size, w), "head": (c.vocab_size, w), "final.norm": (w,)}
+    if c.layer_style == "post":
+        out.update({"pos": (c.max_position_embeddings, w), "final.norm.b": (w,)})
+        for i, spec in enumerate(c.layer_specs):
+            mlp = make_mlp(spec, w)
+            for norm in ("norm1",) + (("norm2",) if mlp is not None else ()):
+                out.update({f"l{i}.{norm}": (w,), f"l{i}.{norm}.b": (w,)})
+            out.update({f"l{i}.mix.{n}": s for n, s in make_mixer(spec, w).shapes().items()})
+            out.update({f"l{i}.mlp.{n}": s for n, s in (mlp.shapes() if mlp is not None else {}).items()})
+        return out
     for i, spec in enumerate(c.layer_specs):
         out[f"l{i}.norm1"] = (w,)
         out.update({f"l{i}.mix.{n}": s for n, s in make_mixer(spec, w).shapes().items()})
@@ -326,6 +515,7 @@ class RandomWeights:
     def __init__(self, c, device="cpu", seed: int = 0):
         self.shapes, self.device, self.seed = tensor_shapes(c), device, seed
         self.order = {n: i for i, n in enumerate(self.shapes)}
+        self.plain_norm = 1.0 - c.norm_weight_offset         # a norm weight that scales by one
 
     def has_tensor(self, name):
         return name in self.shapes
@@ -341,8 +531,12 @@ class RandomWeights:
             return 1.0 + 0.1 * t
         if leaf == "w0":
             return -2.0 + 1.5 * t
-        if leaf in ("norm1", "norm"):
+        if leaf in ("norm1", "norm2", "norm"):
+            return self.plain_norm + 0.1 * t
+        if leaf == "b":
             return 0.1 * t
+        if leaf == "correction":
+            return 0.2 * t
         if leaf == "u":
             return 0.5 * t
-        return t if name == "embed" else t * shape[-1] ** -0.5
+        return t if name in ("embed", "pos") else t * shape[-1] ** -0.5

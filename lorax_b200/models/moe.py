@@ -43,7 +43,7 @@ def moe_forward(model, x: torch.Tensor, lw, li: int, inp) -> torch.Tensor:
     T = x.shape[0]
     if (x.is_cuda and x.dtype == torch.bfloat16 and isinstance(lw.experts_w13, torch.Tensor) and isinstance(lw.experts_w2, torch.Tensor)
             and lw.experts_w13.dtype == torch.bfloat16 and lw.experts_w13.shape[1] % 128 == 0 and lw.experts_w2.shape[1] % 128 == 0
-            and model.hidden % 8 == 0 and c.intermediate_size % 8 == 0 and E <= 64 and c.num_experts_per_tok <= 8 and hasattr(ops, "moe_ffn")):
+            and model.hidden % 8 == 0 and c.intermediate_size % 8 == 0 and E <= 256 and c.num_experts_per_tok <= 32 and hasattr(ops, "moe_ffn")):
         out = ops.moe_ffn(x, lw.router_w.to(torch.bfloat16) if lw.router_w.dtype != torch.bfloat16 else lw.router_w, lw.experts_w13,
                           lw.experts_w2, c.num_experts_per_tok, e0, c.hidden_act)
         if ws > 1 and e_local < E:

@@ -17,6 +17,8 @@ from typing import NamedTuple, Optional
 
 import torch
 
+from .reference import MoeRouting
+
 _PKG = Path(__file__).resolve().parent.parent
 _LIB_PATH = _PKG / "_lx_kernels.so"
 _lib: Optional[ctypes.CDLL] = None
@@ -96,12 +98,14 @@ def load() -> ctypes.CDLL:
         "lx_wq4_gemm_ex": ([P, L, P, P, P, P, L, I, I, I, I, I, P], I),
         "lx_lora_expand_tiled": ([P, I, L, I, P, I, I, P, P, P, I, L, P, L, I, I, I, I, P, P], I),
         "lx_attn_prefill_tc_supported": ([I, I, I, L, L], I),
-        "lx_attn_prefill_tc": ([P, L, I, P, I, P, I, P, P, P, P, I, P, L, I, I, I, I, F, F, P, P, P], I),
-        "lx_moe_router_logits": ([P, L, P, L, P, I, I, I, P], I),
-        "lx_moe_route": ([P, I, I, I, I, I, P, P, P, P, P, P], I),
-        "lx_moe_gather": ([P, L, P, P, I, P, L, I, I, P], I),
+        "lx_attn_prefill_tc": ([P, L, I, P, I, P, I, P, P, P, P, I, P, L, I, I, I, I, F, F, P, I, P, P], I),
+        "lx_moe_router_logits": ([P, L, P, L, P, I, I, I, P, I, P], I),
+        "lx_moe_select_bytes": ([], I),
+        "lx_moe_select": ([P, P], I),
+        "lx_moe_place_bytes": ([], I),
+        "lx_moe_place": ([P, P], I),
         "lx_moe_combine": ([P, L, P, P, I, P, L, I, I, P], I),
-        "lx_moe_grouped_gemm": ([P, L, P, L, P, L, P, I, I, I, I, I, P, I, P], I),
+        "lx_moe_grouped_gemm": ([P, L, P, L, P, L, P, I, I, I, I, I, I, I, I, I, I, P, I, P], I),
     }
     from . import native_mixers
     sigs.update(native_mixers.SIGNATURES)
@@ -114,6 +118,9 @@ def load() -> ctypes.CDLL:
         fn.argtypes = argtypes
         fn.restype = restype
     native_mixers.check_layouts(lib)
+    for name, st in (("lx_moe_select_bytes", MoeSelectParams), ("lx_moe_place_bytes", MoePlaceParams)):
+        if getattr(lib, name)() != ctypes.sizeof(st):
+            raise NativeError(f"{name}: C++ says {getattr(lib, name)()} bytes, ctypes says {ctypes.sizeof(st)}")
     _lib = lib
     return lib
 
@@ -312,63 +319,85 @@ def gemm_lora_fused(x: torch.Tensor, w: torch.Tensor, lf: LoraFused, bias: Optio
 
 
 # ------------------------------------------------------------------------------------------------ mixture of experts
-class MoeRouting(NamedTuple):
-    topk_ids: torch.Tensor     # [T, k] int32
-    topk_w: torch.Tensor       # [T, k] fp32, renormalised over the kept experts
-    seg: torch.Tensor          # [e_local + 1] int32: rows of every local expert in the sorted order
-    pos: torch.Tensor          # [T, k] int32: sorted row of (token, choice), -1 when the expert lives on another rank
-    sorted_tok: torch.Tensor   # [T * k] int32
+class MoeSelectParams(ctypes.Structure):
+    """Mirror of the C struct of the same name (csrc/kernels/moe.cu)."""
+    _fields_ = [("logits", c_void_p), ("correction", c_void_p), ("topk_ids", c_void_p), ("topk_w", c_void_p), ("rank", c_void_p),
+                ("counts", c_void_p), ("ldl", c_longlong), ("T", c_int), ("E", c_int), ("k", c_int), ("e0", c_int), ("e_local", c_int),
+                ("sigmoid", c_int), ("groups", c_int), ("keep", c_int), ("shared", c_int), ("scale", c_float)]
 
 
-def moe_route(x: torch.Tensor, router_w: torch.Tensor, k: int, e0: int, e_local: int) -> MoeRouting:
-    """Router logits (fp32), softmax over all experts, top-k, renormalise, and the sorted order of the rows routed to the
-    experts [e0, e0 + e_local) this rank owns: two launches, everything stays on the device."""
+class MoePlaceParams(ctypes.Structure):
+    """Mirror of the C struct of the same name (csrc/kernels/moe.cu)."""
+    _fields_ = [("x", c_void_p), ("xg", c_void_p), ("ldx", c_longlong), ("ldg", c_longlong), ("row_bytes", c_int), ("counts", c_void_p),
+                ("topk_ids", c_void_p), ("pos", c_void_p), ("seg", c_void_p), ("T", c_int), ("k", c_int), ("e0", c_int), ("e_local", c_int),
+                ("shared", c_int), ("rows_cap", c_int)]
+
+
+def moe_route(x: torch.Tensor, router_w: torch.Tensor, k: int, e0: int, e_local: int, experts: Optional[int] = None, score: str = "softmax",
+              correction: Optional[torch.Tensor] = None, groups: int = 0, keep: int = 0, scale: float = 1.0, shared: int = 0) -> MoeRouting:
+    """Router logits (fp32), choice of `k` experts per token (`reference.moe_route` states the rules), and the sorted order of the rows
+    routed to the experts [e0, e0 + e_local) this rank owns with those rows gathered: three launches, everything stays on the device."""
     T, H = x.shape
-    E = router_w.shape[0]
+    rows = router_w.shape[0]
+    E = experts or rows
     dev = x.device
-    logits = torch.empty(T, E, dtype=torch.float32, device=dev)
     lib = load()
-    _check(lib.lx_moe_router_logits(_ptr(x), x.stride(0), _ptr(router_w), router_w.stride(0), _ptr(logits), T, E, H, _stream()), "lx_moe_router_logits")
-    r = MoeRouting(torch.empty(T, k, dtype=torch.int32, device=dev), torch.empty(T, k, dtype=torch.float32, device=dev),
-                   torch.empty(e_local + 1, dtype=torch.int32, device=dev), torch.empty(T, k, dtype=torch.int32, device=dev),
-                   torch.empty(T * k, dtype=torch.int32, device=dev))
-    _check(lib.lx_moe_route(_ptr(logits), T, E, k, e0, e_local, _ptr(r.topk_ids), _ptr(r.topk_w), _ptr(r.seg), _ptr(r.pos), _ptr(r.sorted_tok),
-                            _stream()), "lx_moe_route")
+    counts = torch.empty(e_local, dtype=torch.int32, device=dev)
+    if x.dtype == torch.float32:
+        logits = gemm_f32(x, router_w)
+        counts.zero_()
+    else:
+        logits = torch.empty(T, rows, dtype=torch.float32, device=dev)
+        _check(lib.lx_moe_router_logits(_ptr(x), x.stride(0), _ptr(router_w), router_w.stride(0), _ptr(logits), T, rows, H, _ptr(counts), e_local,
+                                        _stream()), "lx_moe_router_logits")
+    kw = k + shared
+    r = MoeRouting(torch.empty(T, k, dtype=torch.int32, device=dev), torch.empty(T, kw, dtype=torch.float32, device=dev),
+                   torch.empty(e_local + shared + 1, dtype=torch.int32, device=dev), torch.empty(T, kw, dtype=torch.int32, device=dev),
+                   torch.empty(T * (k + (1 if shared else 0)), H, dtype=x.dtype, device=dev))
+    p = MoeSelectParams(_ptr(logits), _ptr(correction), _ptr(r.topk_ids), _ptr(r.topk_w), _ptr(r.pos), _ptr(counts), logits.stride(0), T, E, k,
+                        e0, e_local, int(score == "sigmoid"), groups, keep, shared, scale)
+    _check(lib.lx_moe_select(ctypes.byref(p), _stream()), "lx_moe_select")
+    size = x.element_size()
+    q = MoePlaceParams(_ptr(x), _ptr(r.xg), x.stride(0) * size, r.xg.stride(0) * size, H * size, _ptr(counts), _ptr(r.topk_ids), _ptr(r.pos),
+                       _ptr(r.seg), T, k, e0, e_local, shared, r.xg.shape[0])
+    _check(lib.lx_moe_place(ctypes.byref(q), _stream()), "lx_moe_place")
     return r
 
 
-def moe_grouped_gemm(xg: torch.Tensor, w: torch.Tensor, seg: torch.Tensor, avg_rows: int, out: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """out[q] = xg[q] @ w[e(q)]^T for every sorted row q (e(q): the expert whose run [seg[e], seg[e+1]) holds q).
-    w: [e_local, n_w, K] bf16, n_w a multiple of 128."""
-    e_local, n_w, K = w.shape
-    rows = xg.shape[0]
-    assert w.is_contiguous() and xg.stride(1) == 1 and xg.shape[1] == K
+_MOE_ACTS = {"": 0, "relu2": 1}
+
+
+def moe_grouped_gemm(xg: torch.Tensor, w: torch.Tensor, seg: torch.Tensor, avg_rows: int, out: Optional[torch.Tensor] = None, shared: int = 0,
+                     tokens: int = 0, act: str = "") -> torch.Tensor:
+    """out[q] = act(xg[q] @ w[e(q)]^T) for every sorted row q (e(q): the expert whose run [seg[e], seg[e+1]) holds q).
+    w: [experts, n_w, K], n_w a multiple of 128.  The last `shared` experts all read the one set of `tokens` rows that stands where
+    the first of them begins; the result has rows of its own for each."""
+    runs, n_w, K = w.shape
+    rows = xg.shape[0] + max(shared - 1, 0) * tokens
+    assert w.is_contiguous() and xg.stride(1) == 1 and xg.shape[1] == K and xg.dtype == w.dtype
     if out is None:
-        out = torch.empty(rows, n_w, dtype=torch.bfloat16, device=xg.device)
+        out = torch.empty(rows, n_w, dtype=xg.dtype, device=xg.device)
     ws = workspace(xg.device)
-    rc = load().lx_moe_grouped_gemm(_ptr(xg), xg.stride(0), _ptr(w), K, _ptr(out), out.stride(0), _ptr(seg), e_local, rows, n_w, K, avg_rows,
-                                    _ptr(ws.status), ws.num_sms, _stream())
+    rc = load().lx_moe_grouped_gemm(_ptr(xg), xg.stride(0), _ptr(w), K, _ptr(out), out.stride(0), _ptr(seg), runs, xg.shape[0], rows, n_w, K,
+                                    avg_rows, shared, tokens, _MOE_ACTS[act], int(xg.dtype == torch.float32), _ptr(ws.status), ws.num_sms,
+                                    _stream())
     _check(rc, "lx_moe_grouped_gemm")
     return out
 
 
 def moe_ffn(x: torch.Tensor, router_w: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, k: int, e0: int, act: str = "silu") -> torch.Tensor:
-    """Top-k mixture-of-experts feed-forward of this rank's experts: route, gather, grouped w1|w3 GEMM, act * up, grouped w2
+    """Top-k mixture-of-experts feed-forward of this rank's experts: route and gather, grouped w1|w3 GEMM, act * up, grouped w2
     GEMM, weighted combine.  w13: [e_local, 2I, H], w2: [e_local, H, I].  Returns [T, H] (a partial sum under expert parallelism)."""
     T, H = x.shape
     e_local, two_i, _ = w13.shape
     E = router_w.shape[0]
     r = moe_route(x, router_w, k, e0, e_local)
-    rows = T * k
-    lib = load()
-    xg = torch.empty(rows, H, dtype=torch.bfloat16, device=x.device)
-    _check(lib.lx_moe_gather(_ptr(x), x.stride(0), _ptr(r.sorted_tok), _ptr(r.seg), e_local, _ptr(xg), xg.stride(0), rows, H, _stream()), "lx_moe_gather")
-    avg = max(1, (rows + E - 1) // E)
-    gu = moe_grouped_gemm(xg, w13, r.seg, avg)
+    avg = max(1, (T * k + E - 1) // E)
+    gu = moe_grouped_gemm(r.xg, w13, r.seg, avg)
     a = act_mul(gu, two_i // 2, act, gated=True)
     y = moe_grouped_gemm(a, w2, r.seg, avg)
     out = torch.empty(T, H, dtype=torch.bfloat16, device=x.device)
-    _check(lib.lx_moe_combine(_ptr(y), y.stride(0), _ptr(r.pos), _ptr(r.topk_w), k, _ptr(out), out.stride(0), T, H, _stream()), "lx_moe_combine")
+    _check(load().lx_moe_combine(_ptr(y), y.stride(0), _ptr(r.pos), _ptr(r.topk_w), k, _ptr(out), out.stride(0), T, H, _stream()), "lx_moe_combine")
     return out
 
 
@@ -491,7 +520,7 @@ def rope_kvwrite(qkv: torch.Tensor, positions: torch.Tensor, cos_sin: torch.Tens
     _check(rc, "lx_rope_kvwrite")
 
 
-_ACTS = {"silu": 0, "swish": 0, "gelu": 1, "gelu_new": 2, "gelu_pytorch_tanh": 2, "gelu_fast": 2, "gelu_tanh": 2, "relu": 3}
+_ACTS = {"silu": 0, "swish": 0, "gelu": 1, "gelu_new": 2, "gelu_pytorch_tanh": 2, "gelu_fast": 2, "gelu_tanh": 2, "relu": 3, "relu2": 4}
 
 
 def act_mul(x: torch.Tensor, inter: int, act: str = "silu", gated: bool = True, out: Optional[torch.Tensor] = None) -> torch.Tensor:
@@ -600,7 +629,7 @@ def attn_prefill(q: torch.Tensor, kv_cache: torch.Tensor, block_tables: torch.Te
         # tcgen05 flash kernel: two query heads of a KV group per CTA, K / V pages by TMA from the paged cache
         rc = lib.lx_attn_prefill_tc(_ptr(q), q.stride(0), T, _ptr(kv_cache), kv_cache.shape[0], _ptr(block_tables), block_tables.shape[1],
                                     _ptr(cu_q), _ptr(cache_lens), _ptr(tile_seq), _ptr(tile_q0), tile_seq.shape[0], _ptr(out), out.stride(0),
-                                    nh, nkv, d, window, scale, softcap, _ptr(alibi), _ptr(workspace(q.device).status), _stream())
+                                    nh, nkv, d, window, scale, softcap, _ptr(alibi), 0, _ptr(workspace(q.device).status), _stream())
         _check(rc, "lx_attn_prefill_tc")
         return out
     rc = lib.lx_attn_prefill_alibi(_ptr(q), q.stride(0), _ptr(kv_cache), _ptr(block_tables), block_tables.shape[1], _ptr(cu_q),
@@ -684,14 +713,14 @@ def lora_expand_tiles(v, tiles: torch.Tensor, num_tiles: int, max_tile_rows: int
 
 
 # ------------------------------------------------------------------------------------------------ layer-by-layer designs
-from .native_mixers import (embed_stream, gemm_f32, gemm_heads, gemm_stack, latent_attn, latent_prep, linear_attn, norm_gate,  # noqa: E402
-                            latent_prefill, norm_stream, rope_pairs, tanh_, token_shift, wkv)
+from .native_mixers import (embed_stream, gemm_f32, gemm_heads, gemm_stack, gqa_attn, latent_attn, latent_prep, linear_attn,  # noqa: E402
+                            latent_prefill, norm_add, norm_gate, norm_stream, qk_norm_kvwrite, rope_pairs, tanh_, token_shift, wkv)
 
 # ------------------------------------------------------------------------------------------------ per-op timing
 _TIMED_OPS = ("gemm", "gemm_fp8", "norm_residual", "rope_kvwrite", "act_mul", "embed", "argmax_logprob", "advance_decode", "attn_decode",
               "attn_prefill", "lora_shrink", "lora_expand", "lora_shrink_tiles", "lora_expand_tiles",
               "embed_stream", "norm_stream", "norm_gate", "tanh_", "gemm_heads", "linear_attn", "wkv", "token_shift", "latent_prep", "rope_pairs",
-              "latent_attn", "latent_prefill")
+              "latent_attn", "latent_prefill", "norm_add", "qk_norm_kvwrite", "gqa_attn", "moe_route", "moe_grouped_gemm")
 _timing_records = None
 _timing_originals = {}
 

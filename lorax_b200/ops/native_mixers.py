@@ -1,5 +1,5 @@
-"""Bindings of the kernels of the layer-by-layer designs (`models/mixers.py`): `csrc/kernels/stream.cu`, `recurrent.cu` and
-`latent_attn.cu`.  Every operator exists for bf16 and for fp32 activations.  Imported into :mod:`lorax_b200.ops.native`."""
+"""Bindings of the kernels of the layer-by-layer designs (`models/mixers.py`): `csrc/kernels/stream.cu`, `recurrent.cu`,
+`latent_attn.cu` and `gqa.cu`.  Every operator exists for bf16 and for fp32 activations.  Imported into :mod:`lorax_b200.ops.native`."""
 
 from __future__ import annotations
 
@@ -51,8 +51,33 @@ class LatentDecodeParams(Structure):
                 ("rows", StepRows), ("H", I), ("R", I), ("page", I), ("nsplit", I), ("scale", F), ("part_o", P), ("part_ml", P)]
 
 
+class NormAddParams(Structure):
+    _fields_ = [("residual", P), ("y", P), ("ldy", L), ("w", P), ("b", P), ("copy", P), ("pos", P), ("weights", P), ("k", I), ("W", I), ("n", I),
+                ("layernorm", I), ("inv_n", F), ("eps", F), ("mult", F)]
+
+
+class QkNormParams(Structure):
+    _fields_ = [("qkv", P), ("ld", L), ("cache", P), ("slots", P), ("q_norm", P), ("k_norm", P), ("T", I), ("H", I), ("G", I), ("DK", I),
+                ("DV", I), ("page", I), ("inv_n", F), ("eps", F)]
+
+
+class GqaF32Params(Structure):
+    _fields_ = [("q", P), ("ldq", L), ("cache", P), ("out", P), ("ldo", L), ("rows", StepRows), ("T", I), ("H", I), ("G", I), ("DK", I),
+                ("DV", I), ("page", I), ("window", I), ("scale", F)]
+
+
 SIGNATURES = {
-    "lx_embed_stream": ([P, P, P, I, I, I, F, I, P], I),
+    "lx_embed_stream": ([P, P, P, I, I, I, F, P, P, I, P, I, P], I),
+    "lx_norm_add_bytes": ([], I),
+    "lx_norm_add": ([P, I, I, P], I),
+    "lx_norm_rows": ([P, P, P, P, P, I, I, I, F, F, I, I, P], I),
+    "lx_gqa_page_size": ([], I),
+    "lx_qk_norm_bytes": ([], I),
+    "lx_qk_norm_kvwrite": ([P, I, P], I),
+    "lx_gqa_f32_bytes": ([], I),
+    "lx_gqa_attn_f32": ([P, P], I),
+    "lx_gqa_decode": ([P, L, P, P, I, P, P, L, P, P, I, I, I, I, I, I, F, I, P], I),
+    "lx_gqa_prefill": ([P, L, P, P, I, P, P, P, P, I, P, L, I, I, I, I, I, F, P], I),
     "lx_norm_stream": ([P, P, P, P, I, I, I, F, F, I, P], I),
     "lx_norm_gate": ([P, P, P, L, P, L, I, I, I, I, F, I, I, P], I),
     "lx_tanh": ([P, L, I, P], I),
@@ -87,7 +112,8 @@ SIGNATURES = {
 def check_layouts(lib):
     for name, st in (("lx_step_rows_bytes", StepRows), ("lx_rec_params_bytes", RecParams), ("lx_latent_prep_bytes", LatentPrepParams),
                      ("lx_latent_attn_bytes", LatentAttnParams), ("lx_latent_decode_bytes", LatentDecodeParams),
-                     ("lx_linear_attn_tc_bytes", LinTcParams), ("lx_wkv_tc_bytes", WkvTcParams)):
+                     ("lx_linear_attn_tc_bytes", LinTcParams), ("lx_wkv_tc_bytes", WkvTcParams),
+                     ("lx_norm_add_bytes", NormAddParams), ("lx_qk_norm_bytes", QkNormParams), ("lx_gqa_f32_bytes", GqaF32Params)):
         if getattr(lib, name)() != ctypes.sizeof(st):
             raise nv.NativeError(f"{name}: C++ says {getattr(lib, name)()} bytes, ctypes says {ctypes.sizeof(st)}")
 
@@ -112,20 +138,40 @@ def step_rows(inp, T: int) -> StepRows:
     return r
 
 
-def embed_stream(ids, table, mult: float = 1.0):
+def embed_stream(ids, table, mult: float = 1.0, pos=None, positions=None, copy=None):
     T, W = ids.shape[0], table.shape[1]
     out = torch.empty(T, W, dtype=torch.float32, device=table.device)
-    nv._check(nv.load().lx_embed_stream(_p(ids), _p(table), _p(out), T, W, table.shape[0], mult, _f32(table), nv._stream()), "lx_embed_stream")
+    nv._check(nv.load().lx_embed_stream(_p(ids), _p(table), _p(out), T, W, table.shape[0], mult, _p(pos), _p(positions) if pos is not None else None,
+                                        pos.shape[0] if pos is not None else 0, _p(copy), _f32(table), nv._stream()), "lx_embed_stream")
     return out
 
 
-def norm_stream(residual, pending, weight, eps: float, weight_offset: float, n: int, dtype):
+def norm_stream(residual, pending, weight, eps: float, weight_offset: float, n: int, dtype, bias=None, layernorm: bool = False, rows=None):
     T, W = residual.shape
+    if layernorm or rows is not None:
+        assert pending is None
+        if rows is not None:
+            T = rows.shape[0]
+        out = torch.empty(T, W, dtype=dtype, device=residual.device)
+        if T:
+            nv._check(nv.load().lx_norm_rows(_p(residual), _p(rows), _p(weight), _p(bias), _p(out), T, W, n, eps, weight_offset, int(layernorm),
+                                             _f32(out), nv._stream()), "lx_norm_rows")
+        return out
     out = torch.empty(T, W, dtype=dtype, device=residual.device)
     assert pending is None or pending.is_contiguous()
     nv._check(nv.load().lx_norm_stream(_p(residual), _p(pending), _p(weight), _p(out), T, W, n, eps, weight_offset, _f32(out), nv._stream()),
               "lx_norm_stream")
     return out
+
+
+def norm_add(residual, y, weight, bias, mult: float, eps: float, n: int, dtype, layernorm: bool = True, pairs=None):
+    T, W = residual.shape
+    copy = torch.empty(T, W, dtype=dtype, device=residual.device) if dtype != torch.float32 else None
+    pos, w = pairs if pairs is not None else (None, None)
+    p = NormAddParams(_p(residual), _p(y), y.stride(0), _p(weight), _p(bias), _p(copy), _p(pos), _p(w), pos.shape[1] if pos is not None else 0, W,
+                      n, int(layernorm), 1.0 / n, eps, mult)
+    nv._check(nv.load().lx_norm_add(ctypes.byref(p), T, _f32(y), nv._stream()), "lx_norm_add")
+    return residual if copy is None else copy
 
 
 def norm_gate(x, group: int, n: int, weight, gate, act: str, eps: float, out):
@@ -325,3 +371,48 @@ def latent_prefill(q, cache, w_ukv, gate, out, H: int, dk: int, rot: int, dv: in
                                     _p(inp.q128_seq), _p(inp.q128_q0), inp.q128_seq.shape[0], _p(g), g.stride(0), _p(y), y.stride(0), H, dk, rot,
                                     dv, scale, _p(nv.workspace(dev).status), nv._stream()), "lx_latent_prefill")
     return True
+
+
+def qk_norm_kvwrite(qkv, H: int, G: int, dk: int, dv: int, n: int, q_norm, k_norm, eps: float, cache, slots):
+    p = QkNormParams(_p(qkv), qkv.stride(0), _p(cache), _p(slots), _p(q_norm), _p(k_norm), qkv.shape[0], H, G, dk, dv,
+                     cache.shape[2] // (dk + dv), 1.0 / n, eps)
+    nv._check(nv.load().lx_qk_norm_kvwrite(ctypes.byref(p), _f32(qkv), nv._stream()), "lx_qk_norm_kvwrite")
+
+
+def _gqa_splits(T: int, units: int, window: int, max_blocks: int, page: int, num_sms: int) -> int:
+    """CTAs that share the keys of one row and head group: enough for two per SM, but at least four pages each."""
+    pages = min(max_blocks, (window + page - 1) // page + 1 if window > 0 else max_blocks)
+    return max(1, min(8, 2 * num_sms // max(1, T * units), pages // 4))
+
+
+def gqa_attn(q, cache, H: int, G: int, dk: int, dv: int, scale: float, window: int, inp, out):
+    T = q.shape[0]
+    lib, ws = nv.load(), nv.workspace(q.device)
+    page = cache.shape[2] // (dk + dv)
+    if q.dtype == torch.float32:
+        p = GqaF32Params(_p(q), q.stride(0), _p(cache), _p(out), out.stride(0), step_rows(inp, T), T, H, G, dk, dv, page, window, scale)
+        nv._check(lib.lx_gqa_attn_f32(ctypes.byref(p), nv._stream()), "lx_gqa_attn_f32")
+        return out
+    if page != lib.lx_gqa_page_size():
+        raise ValueError(f"the attention kernels take pages of {lib.lx_gqa_page_size()} tokens, not {page}")
+    nd, dbt, _, ctx = inp.decode_view(T)
+    if nd:
+        nsplit = _gqa_splits(nd, G * ((H // G + 15) // 16), window, dbt.shape[1], page, ws.num_sms)
+        part_o = part_lse = None
+        if nsplit > 1:
+            part_o = torch.empty(nd * H * nsplit * (dv + 1), dtype=torch.float32, device=q.device)
+            part_lse = part_o[nd * H * nsplit * dv:]
+        nv._check(lib.lx_gqa_decode(_p(q), q.stride(0), _p(cache), _p(dbt), dbt.shape[1], _p(ctx), _p(out), out.stride(0), _p(part_o), _p(part_lse),
+                                    nd, H, G, dk, dv, window, scale, nsplit, nv._stream()), "lx_gqa_decode")
+        nv.launch_count += int(nsplit > 1)
+    if inp.is_prefill:
+        qp, op, tiles = q[nd:], out[nd:], inp.tile_seq.shape[0]
+        if nv.TC_PREFILL and dk == dv and lib.lx_attn_prefill_tc_supported(H, G, dk, q.stride(0), out.stride(0)):
+            nv._check(lib.lx_attn_prefill_tc(_p(qp), q.stride(0), T - nd, _p(cache), cache.shape[0], _p(inp.block_tables), inp.block_tables.shape[1],
+                                             _p(inp.cu_q), _p(inp.cache_lens), _p(inp.tile_seq), _p(inp.tile_q0), tiles, _p(op), out.stride(0), H, G,
+                                             dk, window, scale, 0.0, None, 1, _p(ws.status), nv._stream()), "lx_attn_prefill_tc")
+        else:
+            nv._check(lib.lx_gqa_prefill(_p(qp), q.stride(0), _p(cache), _p(inp.block_tables), inp.block_tables.shape[1], _p(inp.cu_q),
+                                         _p(inp.cache_lens), _p(inp.tile_seq), _p(inp.tile_q0), tiles, _p(op), out.stride(0), H, G, dk, dv, window,
+                                         scale, nv._stream()), "lx_gqa_prefill")
+    return out

@@ -8,7 +8,7 @@ function) and the compute path of the engine on a machine without a GPU.  Signat
 from __future__ import annotations
 
 import math
-from typing import Optional
+from typing import NamedTuple, Optional
 
 import torch
 import torch.nn.functional as F
@@ -163,6 +163,8 @@ def _act(x, act):
         return F.gelu(x, approximate="tanh")
     if act == "relu":
         return F.relu(x)
+    if act == "relu2":
+        return F.relu(x).square()
     raise ValueError(act)
 
 
@@ -466,14 +468,51 @@ def rope_table(rot: int, max_pos: int, base: float, device="cpu") -> torch.Tenso
     return torch.cat([a.cos(), a.sin()], -1).float().to(device)
 
 
-def embed_stream(ids, table, mult=1.0):
-    return table[ids.long().clamp(0, table.shape[0] - 1)].float() * mult
+def embed_stream(ids, table, mult=1.0, pos=None, positions=None, copy=None):
+    """table[ids] * mult (+ pos[positions]) in fp32; `copy` takes the same values in its own dtype."""
+    x = table[ids.long().clamp(0, table.shape[0] - 1)].float() * mult
+    if pos is not None:
+        x = x + pos[positions.long().clamp(0, pos.shape[0] - 1)].float()
+    if copy is not None:
+        copy.copy_(x)
+    return x
 
 
-def norm_stream(residual, pending, weight, eps, weight_offset: float, n: int, dtype):
-    """residual (fp32, in place) += pending; returns its RMS norm (mean over the first `n` columns) in `dtype`."""
+def _layer_norm(x, weight, bias, eps, n: int):
+    """Layer norm over the first `n` columns; the padding behind them stays zero when weight and bias are zero there."""
+    d = x - x[:, :n].mean(-1, keepdim=True)
+    y = d * torch.rsqrt(d[:, :n].square().mean(-1, keepdim=True) + eps) * weight
+    return y if bias is None else y + bias
+
+
+def norm_add(residual, y, weight, bias, mult: float, eps, n: int, dtype, layernorm: bool = True, pairs=None):
+    """residual (fp32, in place) += mult * norm(y) over the first `n` columns; returns the new residual in `dtype`.  With `pairs` =
+    (pos [T, k], w [T, k]) a token's y is the weighted sum of its rows pos (-1: none) of `y`."""
+    W = residual.shape[1]
+    if pairs is None:
+        x = y[:, :W].float()
+    else:
+        pos, w = pairs
+        x = torch.einsum("tk,tkw->tw", torch.where(pos >= 0, w, torch.zeros_like(w)), y[pos.long().clamp(min=0)][:, :, :W].float())
+    if layernorm:
+        x = _layer_norm(x, weight, bias, eps, n)
+    else:
+        x = x * torch.rsqrt((x * x).sum(-1, keepdim=True) / n + eps) * weight
+        if bias is not None:
+            x = x + bias
+    residual += mult * x
+    return residual if dtype == torch.float32 else residual.to(dtype)
+
+
+def norm_stream(residual, pending, weight, eps, weight_offset: float, n: int, dtype, bias=None, layernorm: bool = False, rows=None):
+    """residual (fp32, in place) += pending; returns its RMS or layer norm (mean over the first `n` columns) in `dtype`, of `rows` only
+    when given."""
     if pending is not None:
         residual += pending.float()
+    if rows is not None:
+        residual = residual[rows.long()]
+    if layernorm:
+        return _layer_norm(residual, weight + weight_offset, bias, eps, n).to(dtype)
     y = residual * torch.rsqrt((residual * residual).sum(-1, keepdim=True) / n + eps)
     return (y * (weight + weight_offset)).to(dtype)
 
@@ -636,3 +675,118 @@ def latent_attn(q_lat, q, cache, H: int, kv_rank: int, head: int, rot_off: int, 
         s = (s * scale).masked_fill(torch.arange(keys, device=q.device)[None, None, :] > pos[None, :, None], float("-inf"))
         out[r0: r0 + n] = torch.einsum("hts,sc->thc", torch.softmax(s, -1), rows[:, :kv_rank]).to(q.dtype)
     return out.view(T, H * kv_rank)
+
+
+def _kv_planes(cache, blocks, dk: int, dv: int, keys: int):
+    """Pages of a sequence -> K [keys, heads, dk], V [keys, heads, dv] (fp32)."""
+    page = cache.shape[2] // (dk + dv)
+    x = cache[blocks.long()].float()
+    k = x[:, :, : page * dk].reshape(-1, cache.shape[1], page, dk).transpose(1, 2).reshape(-1, cache.shape[1], dk)
+    v = x[:, :, page * dk:].reshape(-1, cache.shape[1], page, dv).transpose(1, 2).reshape(-1, cache.shape[1], dv)
+    return k[:keys], v[:keys]
+
+
+def qk_norm_kvwrite(qkv, H: int, G: int, dk: int, dv: int, n: int, q_norm, k_norm, eps, cache, slots):
+    """Rows [q (H heads) | k (G) | v (G)] of padded widths dk, dk, dv: q (in place) and k are divided by their root mean square over
+    the first `n` columns of each head and multiplied by the norm's weight; k and v go to the cache."""
+    T = qkv.shape[0]
+
+    def rms(x, heads, w):
+        x = x.reshape(T, heads, dk).float()
+        return (x * torch.rsqrt((x * x).sum(-1, keepdim=True) / n + eps) * w).to(qkv.dtype)
+    q = rms(qkv[:, : H * dk], H, q_norm)
+    qkv[:, : H * dk] = q.reshape(T, -1)
+    k = rms(qkv[:, H * dk: (H + G) * dk], G, k_norm)
+    v = qkv[:, (H + G) * dk: (H + G) * dk + G * dv].reshape(T, G, dv)
+    page = cache.shape[2] // (dk + dv)
+    ok = slots >= 0
+    s = slots[ok].long()
+    blk, off = s // page, s % page
+    cache[:, :, : page * dk].view(cache.shape[0], G, page, dk)[blk, :, off] = k[ok]
+    cache[:, :, page * dk:].view(cache.shape[0], G, page, dv)[blk, :, off] = v[ok]
+
+
+def gqa_attn(q, cache, H: int, G: int, dk: int, dv: int, scale: float, window: int, inp, out):
+    """Softmax attention of a step's rows (queries in the first H * dk columns of q) over the cached keys and values; a token sees the
+    last `window` tokens (0: all) including itself.  -> out [T, H * dv]"""
+    T = q.shape[0]
+    page = cache.shape[2] // (dk + dv)
+    nd, dbt, _, ctx = inp.decode_view(T)
+    spans = [(i, 1, dbt[i], int(ctx[i]) - 1) for i in range(nd) if int(ctx[i]) > 0]
+    if inp.is_prefill:
+        cu = [int(c) for c in inp.cu_q]
+        spans += [(nd + cu[b], cu[b + 1] - cu[b], inp.block_tables[b], int(inp.cache_lens[b])) for b in range(len(cu) - 1) if cu[b + 1] > cu[b]]
+    out[:, : H * dv] = 0
+    for r0, n, bt, before in spans:
+        keys = before + n
+        k, v = _kv_planes(cache, bt[: (keys + page - 1) // page], dk, dv, keys)
+        pos, kp = torch.arange(before, keys, device=q.device)[:, None], torch.arange(keys, device=q.device)[None, :]
+        hidden = kp > pos
+        if window > 0:
+            hidden |= kp <= pos - window
+        qs = q[r0: r0 + n, : H * dk].reshape(n, G, H // G, dk).float()
+        s = (torch.einsum("tghd,sgd->ghts", qs, k) * scale).masked_fill(hidden, float("-inf"))
+        out[r0: r0 + n, : H * dv] = torch.einsum("ghts,sgd->tghd", torch.softmax(s, -1), v).reshape(n, H * dv).to(out.dtype)
+    return out
+
+
+class MoeRouting(NamedTuple):
+    topk_ids: torch.Tensor     # [T, k] int32
+    topk_w: torch.Tensor       # [T, k + shared] fp32
+    seg: torch.Tensor          # [experts + shared + 1] int32: rows of every expert in the sorted order
+    pos: torch.Tensor          # [T, k + shared] int32: sorted row of (token, choice), -1 when the expert lives on another rank
+    xg: torch.Tensor           # the tokens' rows in the sorted order; the rows of the shared experts are the same ones, held once
+
+
+def moe_route(x, router_w, k: int, e0: int, e_local: int, experts=None, score: str = "softmax", correction=None, groups: int = 0,
+              keep: int = 0, scale: float = 1.0, shared: int = 0) -> MoeRouting:
+    """Routing of every token to `k` of the router's first `experts` rows.  softmax: the largest logits, weights renormalised.
+    sigmoid: the largest sigmoid + correction within the best `keep` of `groups` groups (by the sum of a group's two largest), weights
+    are the sigmoids divided by their sum and times `scale`.  `shared` experts more take every token, with the weight
+    sigmoid(router row `experts`)."""
+    T, E = x.shape[0], experts or router_w.shape[0]
+    z = x.float() @ router_w.float().t()
+    logits = z[:, :E]
+    if score == "softmax":
+        p, ids = torch.softmax(logits, -1).topk(k, -1)
+        w = p / p.sum(-1, keepdim=True)
+    else:
+        s = torch.sigmoid(logits)
+        choice = s if correction is None else s + correction
+        if groups:
+            g = choice.view(T, groups, E // groups)
+            best = g.topk(min(2, E // groups), -1).values.sum(-1).topk(keep, -1).indices
+            kept = torch.zeros(T, groups, dtype=torch.bool, device=x.device).scatter_(1, best, True)
+            choice = g.masked_fill(~kept[:, :, None], float("-inf")).reshape(T, E)
+        ids = choice.topk(k, -1).indices
+        w = s.gather(1, ids)
+        w = w / (w.sum(-1, keepdim=True) + 1e-20) * scale
+    local = ids - e0
+    flat = torch.where((local >= 0) & (local < e_local), local, torch.full_like(local, e_local)).reshape(-1)
+    order = torch.argsort(flat, stable=True)
+    count = torch.bincount(flat, minlength=e_local + 1)[:e_local]
+    total = int(count.sum())
+    seg = [0] + torch.cumsum(count, 0).tolist() + [total + (i + 1) * T for i in range(shared)]
+    pos = torch.empty_like(flat)
+    pos[order] = torch.arange(flat.shape[0], device=x.device)
+    pos = torch.where(flat < e_local, pos, torch.full_like(pos, -1)).view(T, k)
+    xg = x[torch.div(order[:total], k, rounding_mode="floor")]
+    if shared:
+        t = torch.arange(T, device=x.device)
+        pos = torch.cat([pos] + [(total + i * T + t)[:, None] for i in range(shared)], 1)
+        w = torch.cat([w] + [torch.sigmoid(z[:, E: E + 1])] * shared, 1)
+        xg = torch.cat([xg, x])
+    return MoeRouting(ids.to(torch.int32), w, torch.tensor(seg, dtype=torch.int32), pos.to(torch.int32), xg)
+
+
+def moe_grouped_gemm(xg, w, seg, avg_rows: int, out=None, shared: int = 0, tokens: int = 0, act: str = ""):
+    """out[q] = act(xg[q] @ w[e(q)]^T) for every sorted row q (e(q): the expert whose run [seg[e], seg[e + 1]) holds q).  The last
+    `shared` experts all read the one set of `tokens` rows that stands where the first of them begins."""
+    s = [int(v) for v in seg]
+    n = len(s) - 1
+    y = torch.zeros(s[-1], w.shape[1], dtype=xg.dtype, device=xg.device)
+    for e in range(n):
+        back = max(0, e - (n - shared)) * tokens if shared else 0
+        z = xg[s[e] - back: s[e + 1] - back].float() @ w[e].float().t()
+        y[s[e]: s[e + 1]] = (_act(z, act) if act else z).to(xg.dtype)
+    return y

@@ -76,8 +76,9 @@ class StateSlots:
 
 class LayeredCache:
     """Cache of a model whose layer runs keep different things (`DecoderModel.cache_shapes`): a run's entry in `layers` is either a
-    paged tensor [num_blocks, page, width] in the model's dtype, addressed by the requests' block tables like a key/value cache, or a
-    dict of state tensors [slots, ...], addressed by the requests' state slot."""
+    paged tensor in the model's dtype, addressed by the requests' block tables ([num_blocks, page, width], or for attention layers with
+    head counts and sizes of their own [num_blocks, kv heads, page * (key width + value width)]: a page of one head is its key plane,
+    then its value plane), or a dict of state tensors [slots, ...], addressed by the requests' state slot."""
 
     def __init__(self, shapes: List[dict], num_blocks: int, num_slots: int, dtype, device, page: int = PAGE_SIZE):
         self.page = page
@@ -86,6 +87,9 @@ class LayeredCache:
         for sh in shapes:
             if "paged" in sh:
                 self.layers.append(torch.zeros(num_blocks, page, sh["paged"], dtype=dtype, device=device))
+            elif "kv" in sh:
+                heads, dk, dv = sh["kv"]
+                self.layers.append(torch.zeros(num_blocks, heads, page * (dk + dv), dtype=dtype, device=device))
             else:
                 self.layers.append({n: torch.zeros(num_slots, *dims, dtype=dt, device=device) for n, (dims, dt) in sh["state"].items()})
         self.state_slots = StateSlots(num_slots) if any("state" in sh for sh in shapes) else None
@@ -116,7 +120,8 @@ def cache_bytes(model, cfg, max_batch: int, page: int = PAGE_SIZE):
     if shapes is None:
         return KVCache.bytes_per_block(model.config.num_hidden_layers, model.nkv, model.d, kv_dtype_of(model, cfg), page), 0
     size = lambda dt: torch.empty(0, dtype=dt).element_size()
-    paged = sum(sh["paged"] for sh in shapes if "paged" in sh) * page * size(model.dtype)
+    width = lambda sh: sh.get("paged", 0) + (sh["kv"][0] * (sh["kv"][1] + sh["kv"][2]) if "kv" in sh else 0)
+    paged = sum(width(sh) for sh in shapes) * page * size(model.dtype)
     fixed = 0
     for sh in shapes:
         for dims, dt in sh.get("state", {}).values():

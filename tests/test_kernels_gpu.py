@@ -542,9 +542,8 @@ def test_moe_ffn_on_the_device(nat, T, E, k, H, I, e0, e_local):
     pos = r.pos.long()
     local = (ids >= e0) & (ids < e0 + e_local)
     assert (pos[~local] == -1).all() and (pos[local] >= 0).all()
-    st = r.sorted_tok.long()
     tok = torch.arange(T, device="cuda")[:, None].expand(T, k)
-    assert torch.equal(st[pos[local]], tok[local])
+    assert torch.equal(r.xg[pos[local]], x[tok[local]])
     out = nat.moe_ffn(x, wr, w13, w2, k, e0, "silu")
     torch.cuda.synchronize()
     nat.workspace().check_status()

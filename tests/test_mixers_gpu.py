@@ -38,10 +38,11 @@ def make_step(dec, pre, slots=None, seg_len=64, seed=0, pages_per_seq=None):
             off.append(off[-1] + b + n)
         ss, s0 = reference.prefill_tiles(q, seg_len)
         ts, t0 = reference.prefill_tiles(q, 128)
+        t64s, t64q = reference.prefill_tiles(q)
         inp = StepInputs(is_prefill=True, block_tables=blocks[nd:].contiguous(), cu_q=i32(cu), cache_lens=i32([b for b, _ in pre]),
                          state_slots=sl[nd:].contiguous(), n_decode=nd, dec_block_tables=blocks[:nd].contiguous(), ctx_lens=i32(dec),
                          dec_state_slots=sl[:nd].contiguous(), seg_seq=i32(ss), seg_q0=i32(s0), seg_len=seg_len, q128_seq=i32(ts),
-                         q128_q0=i32(t0), ctx_off=i32(off), ctx_total=off[-1], **kw)
+                         q128_q0=i32(t0), tile_seq=i32(t64s), tile_q0=i32(t64q), ctx_off=i32(off), ctx_total=off[-1], **kw)
     return inp, width * len(spans) + 1, len(spans) + 1
 
 
@@ -257,3 +258,154 @@ def test_32_bit_products_and_head(T, N, K):
     assert torch.equal(ids.cpu(), ri) and torch.allclose(lps.cpu(), rl, atol=1e-4)
     t = torch.randn(8, 16, generator=g)
     assert torch.allclose(native.tanh_(t.cuda()).cpu(), torch.tanh(t), atol=1e-6)
+
+
+# ---------------------------------------------------------------------------------------------- grouped-query attention
+def gqa_case(H, G, dk, dv, window, inp, nb, dtype, peak, seed=11):
+    """Random queries over a random cache.  `peak`: every query matches one key of its own context far better than all others: the
+    oldest that the window holds, the newest that it does not, the first token, itself, one at a page's edge, in turn."""
+    g = torch.Generator().manual_seed(seed)
+    T = inp.positions.shape[0]
+    q = torch.randn(T, H * dk, generator=g).to(dtype)
+    cache = torch.randn(nb, G, PAGE * (dk + dv), generator=g).to(dtype)
+    if peak:
+        nd, dbt, _, ctx = inp.decode_view(T)
+        keys = cache[:, :, : PAGE * dk].view(nb, G, PAGE, dk).float()
+        for t in range(T):
+            if t < nd:
+                bt, n = dbt[t], int(ctx[t])
+            else:
+                b = int(torch.searchsorted(inp.cu_q[1:], torch.tensor(t - nd), right=True))
+                bt, n = inp.block_tables[b], int(inp.cache_lens[b]) + (t - nd - int(inp.cu_q[b])) + 1
+            if n <= 0:
+                continue
+            w = window or n
+            j = (n - w, n - w - 1, 0, n - 1, n // PAGE * PAGE, n // PAGE * PAGE - 1)[t % 6]
+            j = min(max(j, 0), n - 1)
+            for h in range(H):
+                kr = keys[int(bt[j // PAGE]), h // (H // G), j % PAGE]
+                q.view(T, H, dk)[t, h] = (kr * 3.0).to(dtype)
+    return q, cache
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("peak", [False, True])
+@pytest.mark.parametrize("step", list(STEPS) + ["long"])
+@pytest.mark.parametrize("H,G,dk,dv,window", [(4, 2, 64, 64, 33), (6, 2, 128, 64, 1), (8, 2, 128, 128, 200), (3, 3, 128, 128, 64), (40, 2, 64, 128, 31),
+                                              (2, 1, 256, 256, 100), (4, 1, 64, 256, 257), (2, 2, 256, 64, 0), (4, 1, 128, 256, 32),
+                                              (4, 4, 256, 128, 5000), (16, 4, 128, 128, 128)])
+def test_grouped_query_attention(dtype, peak, step, H, G, dk, dv, window):
+    from lorax_b200.ops import native, reference
+    dec, pre = STEPS[step] if step in STEPS else ([1000, 1500], [(1000, 300), (0, 500), (129, 40)])
+    inp, nb, _ = make_step(dec, pre, seed=12)
+    T = inp.positions.shape[0]
+    q, cache = gqa_case(H, G, dk, dv, window, inp, nb, dtype, peak)
+    want = torch.empty(T, H * dv)
+    reference.gqa_attn(q.float(), cache.float(), H, G, dk, dv, dk ** -0.5, window, inp, want)
+    out = torch.full((T, H * dv + 8), 3.0, dtype=dtype, device="cuda")
+    native.gqa_attn(q.cuda(), cache.cuda(), H, G, dk, dv, dk ** -0.5, window, to_dev(inp), out)
+    native.workspace(out.device).check_status()
+    live = [i for i in range(T) if i >= len(dec) or dec[i] > 0]
+    close(out[:, : H * dv], want, dtype, live, tol16=5e-3)
+    assert (out[:, H * dv:] == 3.0).all()
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("H,G,dk,dv,n", [(4, 2, 64, 64, 64), (6, 2, 128, 64, 80), (1, 1, 64, 256, 3), (5, 5, 256, 128, 200)])
+def test_query_and_key_norms_with_cache_write(dtype, H, G, dk, dv, n):
+    from lorax_b200.ops import native, reference
+    inp, nb, _ = make_step([7, 0, 40], [(0, 50), (33, 5)], seed=8)
+    T = inp.positions.shape[0]
+    g = torch.Generator().manual_seed(3)
+    x = torch.randn(T, (H + G) * dk + G * dv, generator=g)
+    heads = x[:, : (H + G) * dk].view(T, H + G, dk)
+    heads[:, :, n:] = 0
+    x = x.to(dtype)
+    wq, wk = torch.rand(dk, generator=g) + 0.5, torch.rand(dk, generator=g) + 0.5
+    cache = torch.zeros(nb, G, PAGE * (dk + dv))
+    xf, xd, cd = x.float(), x.cuda(), torch.zeros(nb, G, PAGE * (dk + dv), dtype=dtype, device="cuda")
+    reference.qk_norm_kvwrite(xf, H, G, dk, dv, n, wq, wk, 1e-3, cache, inp.slots)
+    native.qk_norm_kvwrite(xd, H, G, dk, dv, n, wq.cuda(), wk.cuda(), 1e-3, cd, inp.slots.cuda())
+    close(xd[:, : H * dk], xf[:, : H * dk], dtype, tol16=5e-3)
+    close(cd, cache, dtype, tol16=5e-3)
+
+
+# ---------------------------------------------------------------------------------------------- norms of sublayer outputs, experts
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("layernorm", [True, False])
+@pytest.mark.parametrize("T,W,n,k", [(1, 16, 9, 0), (5, 208, 200, 3), (67, 4096, 4096, 0), (3, 5120, 5100, 9), (9, 2048, 2048, 2)])
+def test_norm_added_to_the_stream(dtype, layernorm, T, W, n, k):
+    from lorax_b200.ops import native, reference
+    g = torch.Generator().manual_seed(T)
+    pad = lambda t: torch.cat([t[..., :n], torch.zeros(*t.shape[:-1], W - n)], -1)
+    res, w, b = pad(torch.randn(T, W, generator=g)), pad(1 + 0.2 * torch.randn(W, generator=g)), pad(torch.randn(W, generator=g))
+    rows = max(T * k, T)
+    y = torch.zeros(rows, W + 128)
+    y[:, :W] = pad(torch.randn(rows, W, generator=g) + 0.7)
+    y = y.to(dtype)
+    pairs = None
+    if k:
+        pos = torch.randperm(T * k, generator=g).view(T, k).to(torch.int32)
+        pos[0, 0] = -1
+        pairs = (pos, torch.randn(T, k, generator=g))
+    rf, rd = res.clone(), res.cuda()
+    reference.norm_add(rf, y.float(), w, b, 0.3, 1e-5, n, torch.float32, layernorm, pairs)
+    got = native.norm_add(rd, y.cuda(), w.cuda(), b.cuda(), 0.3, 1e-5, n, dtype, layernorm, tuple(p.cuda() for p in pairs) if k else None)
+    close(rd, rf, torch.float32, tol32=1e-5)
+    close(got, rf, dtype, tol16=4e-3)
+    rows = torch.randint(0, T, (4,), generator=g, dtype=torch.int32)
+    want = reference.norm_stream(rf, None, w, 1e-5, 0.0, n, torch.float32, bias=b, layernorm=layernorm, rows=rows) if layernorm else None
+    if layernorm:
+        close(native.norm_stream(rd, None, w.cuda(), 1e-5, 0.0, n, dtype, bias=b.cuda(), layernorm=True, rows=rows.cuda()), want, dtype, tol16=4e-3)
+    table, pt = torch.randn(50, W, generator=g).to(dtype), torch.randn(20, W, generator=g).to(dtype)
+    ids, at = torch.randint(0, 50, (T,), generator=g, dtype=torch.int32), torch.randint(0, 20, (T,), generator=g, dtype=torch.int32)
+    c, cd = torch.empty(T, W, dtype=dtype), torch.empty(T, W, dtype=dtype, device="cuda")
+    assert torch.equal(native.embed_stream(ids.cuda(), table.cuda(), 1.0, pos=pt.cuda(), positions=at.cuda(), copy=cd).cpu(),
+                       reference.embed_stream(ids, table, 1.0, pos=pt, positions=at, copy=c))
+    assert torch.equal(cd.cpu(), c)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("T,E,k,groups,keep,shared,W,ff", [(1, 8, 2, 0, 0, 0, 64, 128), (7, 12, 3, 4, 2, 1, 208, 128), (300, 40, 6, 8, 3, 2, 64, 256),
+                                                           (65, 256, 8, 8, 4, 1, 128, 128), (2000, 64, 4, 64, 9, 3, 96, 128), (33, 6, 6, 2, 2, 1, 64, 128),
+                                                           (40, 5, 1, 1, 1, 0, 48, 128), (700, 33, 32, 0, 0, 1, 64, 128)])
+def test_experts_chosen_by_corrected_sigmoids_in_groups(dtype, T, E, k, groups, keep, shared, W, ff):
+    """Choice, weights, sorted rows and the two grouped products; corrections so large that choice scores are negative and that score
+    and choice order differ."""
+    from lorax_b200.ops import native, reference
+    g = torch.Generator().manual_seed(T + E)
+    x = torch.randn(T, W, generator=g).to(dtype)
+    rows = (E + 1 + 15) // 16 * 16
+    wr = torch.zeros(rows, W)
+    wr[: E + 1] = torch.randn(E + 1, W, generator=g) * W ** -0.5 * 2
+    wr = wr.to(dtype)
+    corr = torch.randn(E, generator=g) * 0.7 - 0.6
+    up = (torch.randn(E + shared, ff, W, generator=g) * W ** -0.5).to(dtype)
+    down = (torch.randn(E + shared, 128, ff, generator=g) * ff ** -0.5).to(dtype)
+    kw = dict(experts=E, score="sigmoid", groups=groups, keep=keep, scale=1.7, shared=shared)
+    want = reference.moe_route(x.float(), wr.float(), k, 0, E, correction=corr, **kw)
+    r = native.moe_route(x.cuda(), wr.cuda(), k, 0, E, correction=corr.cuda(), **kw)
+    ids = r.topk_ids.cpu().long()
+    # rows whose choice hangs on a difference below rounding are left out of the comparison of the choice
+    clear = (ids.sort(-1).values == want.topk_ids.long().sort(-1).values).all(-1)
+    assert clear.float().mean() > 0.99
+    dense = lambda r: torch.zeros(T, E).scatter_(1, r.topk_ids.cpu().long(), r.topk_w.cpu()[:, :k])
+    assert torch.allclose(dense(r)[clear], dense(want)[clear], atol=1e-5)
+    if shared:
+        assert torch.allclose(r.topk_w.cpu()[:, k:], want.topk_w[:, k:], atol=1e-5)
+    seg, pos = r.seg.tolist(), r.pos.cpu().long()
+    assert seg[0] == 0 and seg[E] == T * k and [seg[E + 1 + i] for i in range(shared)] == [T * k + (i + 1) * T for i in range(shared)]
+    for j in range(k):
+        assert all(seg[e] <= p < seg[e + 1] for e, p in zip(ids[:, j].tolist(), pos[:, j].tolist()))
+    assert sorted(pos.flatten().tolist()) == list(range(T * (k + shared)))
+    assert torch.equal(r.xg.cpu()[pos[:, :k]], x[:, None].expand(T, k, W))
+    for i in range(shared):
+        assert torch.equal(pos[:, k + i], T * k + i * T + torch.arange(T))
+    avg = max(1, T * k // E)
+    a = native.moe_grouped_gemm(r.xg, up.cuda(), r.seg, avg, shared=shared, tokens=T, act="relu2")
+    y = native.moe_grouped_gemm(a, down.cuda(), r.seg, avg)
+    native.workspace(y.device).check_status()
+    # the reference products on the kernel's own order of rows
+    af = reference.moe_grouped_gemm(r.xg.cpu().float(), up.float(), r.seg.cpu(), avg, shared=shared, tokens=T, act="relu2")
+    close(a, af, dtype, tol16=5e-3)
+    close(y, reference.moe_grouped_gemm(a.cpu().float(), down.float(), r.seg.cpu(), avg), dtype, tol16=5e-3)

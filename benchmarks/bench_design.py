@@ -1,9 +1,12 @@
 """Prefill and decode throughput of a layer-by-layer design (random weights, layers of a real model's size) beside the closest
 uniform decoder of this framework at equal size, and the device time of every kernel of both with its share of the roofline.
 
-    python bench.py --design vabunex [--design-size small,base] [--steps K] [--warmup W]
+    python bench.py --design vabunex|sapudra [--design-size small,base] [--steps K] [--warmup W]
 
-"Equal size": a llama-style decoder with the same width, feed-forward width, number of layer runs and attention heads of 128.
+"Equal size": for Vabunex a llama-style decoder with the same width, feed-forward width, number of layer runs and attention heads of
+128; for Sapudra a Mixtral-style decoder with the same width, heads, window, layers and experts, whose gated experts (three matrices)
+have two thirds of the width, and which takes one expert more per token in place of the shared one; where the size has no experts, a
+Mistral-style decoder likewise.
 Throughput: prefill is one eager forward pass over ragged prompts, decode one CUDA-graph replay per token, both through
 `ModelRunner`, timed with CUDA events.  Kernel times: CUDA events around every operator of an eager pass, L2 flushed in front of it,
 median of the passes.  Rooflines: the measured copy bandwidth and bf16 rate of MEASURED_PEAKS.json, whichever bounds the operator.
@@ -17,10 +20,17 @@ import statistics
 
 REPO = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 
-SIZES = {
+VABUNEX_SIZES = {
     # width, ff, recurrent heads x dim, wkv heads x dim, latent heads, q rank, kv rank, rot
     "small": dict(width=2048, ff=8192, lin=(16, 128), wkv=(32, 64), heads=16, q_rank=1024, kv_rank=512, rot=64),
     "base": dict(width=4096, ff=14336, lin=(32, 128), wkv=(64, 64), heads=32, q_rank=1536, kv_rank=512, rot=64),
+}
+SAPUDRA_SIZES = {
+    # width, layers, heads and key/value heads of 128, window; experts, per token, groups and groups kept, width of an expert (or of the
+    # dense feed-forward)
+    "small": dict(width=2048, layers=4, heads=16, kv=4, window=1024, experts=64, top=6, groups=(8, 4), ff=1536),
+    "base": dict(width=4096, layers=4, heads=32, kv=8, window=1024, experts=32, top=4, groups=(4, 2), ff=6144),
+    "dense": dict(width=4096, layers=4, heads=32, kv=8, window=1024, experts=0, ff=21504),
 }
 PREFILL = [(1, 4096), (4, 2048), (1, 16384)]           # (prompts, tokens each)
 DECODE = [(16, 2048), (64, 2048), (256, 2048)]         # (rows, tokens of context)
@@ -44,6 +54,30 @@ def llama_like(s, runs, vocab=32000):
     heads = s["width"] // 128
     return ModelConfig(model_type="llama", vocab_size=vocab, hidden_size=s["width"], intermediate_size=s["ff"], num_hidden_layers=runs,
                        num_attention_heads=heads, num_key_value_heads=max(heads // 4, 1), head_dim=128, max_position_embeddings=32768)
+
+
+def sapudra_config(s, vocab=32000):
+    if s["experts"]:
+        mlp = dict(kind="moe", expert=dict(ff=s["ff"]), shared=dict(ff=s["ff"]),
+                   router=dict(experts=s["experts"], top=s["top"], scale=2.5, groups=dict(count=s["groups"][0], keep=s["groups"][1])))
+    else:
+        mlp = dict(kind="dense", ff=s["ff"])
+    layer = dict(type="attention", mlp=mlp, mixer=dict(heads=s["heads"], kv_heads=s["kv"], dim=128, vdim=128, scale=128 ** -0.5,
+                                                       mask=dict(size=s["window"])))
+    return dict(architecture="Sapudra", vocab=vocab, width=s["width"], norm=dict(eps=1e-5), residual_mult=0.3, logit_softcap=30.0,
+                max_positions=20000, layers=[layer] * s["layers"])
+
+
+def mixtral_like(s, runs, vocab=32000):
+    from lorax_b200.config import ModelConfig
+    moe = dict(num_local_experts=s["experts"], num_experts_per_tok=s["top"] + 1) if s["experts"] else {}
+    return ModelConfig(model_type="mixtral" if moe else "mistral", vocab_size=vocab, hidden_size=s["width"], intermediate_size=s["ff"] * 2 // 3,
+                       num_hidden_layers=runs, num_attention_heads=s["heads"], num_key_value_heads=s["kv"], head_dim=128,
+                       max_position_embeddings=32768, sliding_window=s["window"], **moe)
+
+
+DESIGNS = {"vabunex": (VABUNEX_SIZES, vabunex_config, llama_like, "llama-like"),
+           "sapudra": (SAPUDRA_SIZES, sapudra_config, mixtral_like, "mixtral-like")}
 
 
 def peaks():
@@ -132,6 +166,30 @@ class OpTimer:
         if name == "attn_prefill":
             nh, d = a[7], a[9]
             return (name, 0, 4 * q["pairs"] * nh * d)
+        if name == "gqa_attn":
+            H, G, dk, dv = a[2:6]
+            if q["decode"]:
+                return (name, q["ctx"] * G * (dk + dv) * 2 + a[0].shape[0] * H * (dk + dv) * 2, 2 * q["ctx"] * H * (dk + dv))
+            return (name, 0, 2 * q["pairs"] * H * (dk + dv))
+        if name == "qk_norm_kvwrite":
+            T, H, G, dk, dv = a[0].shape[0], *a[1:5]
+            return (name, T * 2 * (H * dk + G * (dk + dv)) * 2, 0)
+        if name == "norm_add":
+            r, y = a[0], a[1]
+            return ("norm_add" + (" of experts" if kw.get("pairs") is not None else ""), nb(r) * 2 + y.shape[0] * r.shape[1] * 2 + r.numel() * 2, 0)
+        if name == "moe_route":
+            x, w, k = a[:3]
+            rows = k + (1 if kw.get("shared") else 0)
+            return (name, nb(x, w) + nb(x) * rows, 2 * x.shape[0] * w.numel())
+        if name == "moe_grouped_gemm":
+            xg, w, seg = a[:3]
+            sizes = seg.diff()
+            rows = int(sizes.sum())
+            return (f"moe_grouped_gemm {w.shape[1]}x{w.shape[2]}", nb(xg) + int((sizes > 0).sum()) * w[0].numel() * 2 + rows * w.shape[1] * 2,
+                    2 * rows * w[0].numel())
+        if name == "moe_combine":
+            y, k, out = a[0], a[3], a[4]
+            return (name, nb(out) * (k + 1), 0)
         if name == "norm_stream":
             r, pend = a[0], a[1]
             return (name, nb(r) * (2 if pend is not None else 1) + nb(pend) + r.numel() * 2, 0)
@@ -169,7 +227,8 @@ class OpTimer:
 
 
 OPS = ("gemm", "norm_residual", "rope_kvwrite", "act_mul", "embed", "attn_decode", "attn_prefill", "embed_stream", "norm_stream", "norm_gate",
-       "tanh_", "gemm_heads", "gemm_stack", "linear_attn", "wkv", "token_shift", "latent_prep", "rope_pairs", "latent_attn", "latent_prefill", "argmax_logprob")
+       "tanh_", "gemm_heads", "gemm_stack", "linear_attn", "wkv", "token_shift", "latent_prep", "rope_pairs", "latent_attn", "latent_prefill", "argmax_logprob", "gqa_attn",
+       "qk_norm_kvwrite", "norm_add", "moe_route", "moe_grouped_gemm", "moe_combine")
 
 
 def main(args):
@@ -187,11 +246,13 @@ def main(args):
     steps, warm = min(args.steps, 50), max(3, min(args.warmup, 10))
     from bench import ClockSampler
     results = []
+    sizes, config_of, like, like_name = DESIGNS[args.design]
     with torch.inference_mode():
         for size in args.design_size.split(","):
-            s = SIZES[size]
-            ours = ModelConfig.from_dict(vabunex_config(s))
-            for name, cfg in ((args.design, ours), ("llama-like", llama_like(s, len(ours.layer_schedule)))):
+            s = sizes[size]
+            ours = ModelConfig.from_dict(config_of(s))
+            window = s.get("window", 1 << 30)
+            for name, cfg in ((args.design, ours), (like_name, like(s, len(ours.layer_schedule)))):
                 model = DecoderModel.random_init_on_device(cfg, dev, torch.bfloat16, seed=0, max_positions=20000)
                 model.use_native_layers = True
                 for kind, cases in (("prefill", PREFILL), ("decode", DECODE)):
@@ -210,12 +271,13 @@ def main(args):
                             run.install(rows, [5] * n, [length] * n, blocks, [0] * n, list(range(1, n + 1)))
                             run.resort()
                             step = lambda: run.decode()
-                            info = dict(decode=True, seqs=n, ctx=n * length, pairs=n * length)
+                            info = dict(decode=True, seqs=n, ctx=n * min(length, window), pairs=n * min(length, window))
                             toks = n
                         else:
                             inp, _ = run._prefill_inputs(items)
                             step = lambda: model.forward(inp, kv.layers)
-                            info = dict(decode=False, seqs=n, ctx=n * length, pairs=n * length * (length + 1) // 2)
+                            info = dict(decode=False, seqs=n, ctx=n * length,
+                                        pairs=n * (length * (length + 1) // 2 - max(0, length - window) * (max(0, length - window) + 1) // 2))
                             toks = n * length
                         for _ in range(warm):
                             step()

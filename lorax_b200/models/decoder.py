@@ -207,6 +207,11 @@ class DecoderModel:
             self._rope_tables[key] = reference.rope_table(rot, self.max_positions, base, self.device)
         return self._rope_tables[key]
 
+    def check_positions(self, tokens: int):
+        """Refuses sequences longer than a layer-by-layer design's table of learned positions."""
+        if self.mixed and self.config.learned_positions and tokens > self.config.max_position_embeddings:
+            raise ValueError(f"{self.config.model_type} has {self.config.max_position_embeddings} positions: max_total_tokens={tokens} is too long")
+
     @property
     def state_parallelism(self) -> int:
         """Thread blocks one sequence gives the recurrence kernels (the least of the layers)."""

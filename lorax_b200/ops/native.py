@@ -385,6 +385,13 @@ def moe_grouped_gemm(xg: torch.Tensor, w: torch.Tensor, seg: torch.Tensor, avg_r
     return out
 
 
+def moe_combine(y: torch.Tensor, pos: torch.Tensor, weights: torch.Tensor, k: int, out: torch.Tensor) -> torch.Tensor:
+    """out[t] = sum over the token's k pairs of weights * y[pos] (pos < 0: the pair belongs to another rank)."""
+    T, H = out.shape
+    _check(load().lx_moe_combine(_ptr(y), y.stride(0), _ptr(pos), _ptr(weights), k, _ptr(out), out.stride(0), T, H, _stream()), "lx_moe_combine")
+    return out
+
+
 def moe_ffn(x: torch.Tensor, router_w: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, k: int, e0: int, act: str = "silu") -> torch.Tensor:
     """Top-k mixture-of-experts feed-forward of this rank's experts: route and gather, grouped w1|w3 GEMM, act * up, grouped w2
     GEMM, weighted combine.  w13: [e_local, 2I, H], w2: [e_local, H, I].  Returns [T, H] (a partial sum under expert parallelism)."""
@@ -396,9 +403,7 @@ def moe_ffn(x: torch.Tensor, router_w: torch.Tensor, w13: torch.Tensor, w2: torc
     gu = moe_grouped_gemm(r.xg, w13, r.seg, avg)
     a = act_mul(gu, two_i // 2, act, gated=True)
     y = moe_grouped_gemm(a, w2, r.seg, avg)
-    out = torch.empty(T, H, dtype=torch.bfloat16, device=x.device)
-    _check(load().lx_moe_combine(_ptr(y), y.stride(0), _ptr(r.pos), _ptr(r.topk_w), k, _ptr(out), out.stride(0), T, H, _stream()), "lx_moe_combine")
-    return out
+    return moe_combine(y, r.pos, r.topk_w, k, torch.empty(T, H, dtype=torch.bfloat16, device=x.device))
 
 
 def quant_act_fp8(x: torch.Tensor):
@@ -720,7 +725,7 @@ from .native_mixers import (embed_stream, gemm_f32, gemm_heads, gemm_stack, gqa_
 _TIMED_OPS = ("gemm", "gemm_fp8", "norm_residual", "rope_kvwrite", "act_mul", "embed", "argmax_logprob", "advance_decode", "attn_decode",
               "attn_prefill", "lora_shrink", "lora_expand", "lora_shrink_tiles", "lora_expand_tiles",
               "embed_stream", "norm_stream", "norm_gate", "tanh_", "gemm_heads", "linear_attn", "wkv", "token_shift", "latent_prep", "rope_pairs",
-              "latent_attn", "latent_prefill", "norm_add", "qk_norm_kvwrite", "gqa_attn", "moe_route", "moe_grouped_gemm")
+              "latent_attn", "latent_prefill", "norm_add", "qk_norm_kvwrite", "gqa_attn", "moe_route", "moe_grouped_gemm", "moe_combine")
 _timing_records = None
 _timing_originals = {}
 

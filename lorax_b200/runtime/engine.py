@@ -79,6 +79,7 @@ class Engine:
         self.model = model
         self.cfg = cfg or EngineConfig()
         c = model.config
+        model.check_positions(self.cfg.max_total_tokens)
         page = self.cfg.block_size
         self._max_batch = max_batch
         if num_blocks is None:

@@ -92,6 +92,7 @@ class ShardRuntime:
         self.tp = model.tp
         c = model.config
         dev = model.device
+        model.check_positions(self.cfg.max_total_tokens)
         if adapter_arena_bytes is None and model.mixed:
             adapter_arena_bytes = 0                          # its projections take no adapters
         if adapter_arena_bytes is None:

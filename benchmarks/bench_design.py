@@ -191,7 +191,7 @@ class OpTimer:
             y, k, out = a[0], a[3], a[4]
             return (name, nb(out) * (k + 1), 0)
         if name == "norm_stream":
-            r, pend = a[0], a[1]
+            r, pend = a[0] if kw.get("rows") is None else a[0][: kw["rows"].shape[0]], a[1]
             return (name, nb(r) * (2 if pend is not None else 1) + nb(pend) + r.numel() * 2, 0)
         if name == "norm_residual":
             return (name, nb(a[0]) * 2 + nb(a[1]) * 2, 0)
@@ -200,7 +200,7 @@ class OpTimer:
         if name == "token_shift":
             return (name, nb(a[0]) * (1 + a[1].shape[0]), 0)
         if name == "act_mul":
-            return (name, a[0].shape[0] * a[1] * 6, 0)
+            return (name, a[0].shape[0] * a[1] * (6 if kw.get("gated", True) else 4), 0)
         if name == "rope_kvwrite":
             T, nh, nkv, d = a[0].shape[0], a[5], a[6], a[7]
             return (name, T * (2 * (nh + nkv) * d + 3 * nkv * d) * 2, 0)
@@ -268,7 +268,7 @@ def main(args):
                         if kind == "decode":
                             # (the contents of caches and states do not matter for the time: no prompt is run)
                             rows = [run.state.take_row(i) for i in range(n)]
-                            run.install(rows, [5] * n, [length] * n, blocks, [0] * n, list(range(1, n + 1)))
+                            run.install(rows, torch.randint(0, cfg.vocab_size, (n,), generator=g).tolist(), [length] * n, blocks, [0] * n, list(range(1, n + 1)))
                             run.resort()
                             step = lambda: run.decode()
                             info = dict(decode=True, seqs=n, ctx=n * min(length, window), pairs=n * min(length, window))

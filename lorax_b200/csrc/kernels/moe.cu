@@ -39,7 +39,7 @@ LX_DEVICE void moe_mma(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uin
                : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }
 
-template <int MT, int NT>
+template <int MT, int NT, int UNROLL>
 __global__ void __launch_bounds__(32 * kRouterWarps) moe_router_logits_kernel(const __nv_bfloat16* __restrict__ x, long long ldx,
                                                                               const __nv_bfloat16* __restrict__ wr, long long ldw,
                                                                               float* __restrict__ logits, int T, int E, int H, int* counts,
@@ -56,27 +56,36 @@ __global__ void __launch_bounds__(32 * kRouterWarps) moe_router_logits_kernel(co
 #pragma unroll
     for (int n = 0; n < NT; ++n) acc[m][n][0] = acc[m][n][1] = acc[m][n][2] = acc[m][n][3] = 0.f;
   const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
-#pragma unroll 2
-  for (int kc = warp; kc * 32 < H; kc += kRouterWarps) {
-    const int k = kc * 32 + c * 8;
-    const bool ok = k < H;
-    uint4 b[NT];
+  for (int k0 = warp * 32; k0 < H; k0 += kRouterWarps * 32 * UNROLL) {
+    uint4 b[UNROLL][NT], xa[UNROLL][MT][2];
 #pragma unroll
-    for (int n = 0; n < NT; ++n) {
-      const int e = n0 + n * 8 + r;
-      b[n] = (ok && e < E) ? __ldg(reinterpret_cast<const uint4*>(wr + (long long)e * ldw + k)) : zero;
-    }
-#pragma unroll
-    for (int m = 0; m < MT; ++m) {
-      const int ta = t0 + m * 16 + r, tb = ta + 8;
-      const uint4 a = (ok && ta < T) ? *reinterpret_cast<const uint4*>(x + (long long)ta * ldx + k) : zero;
-      const uint4 d = (ok && tb < T) ? *reinterpret_cast<const uint4*>(x + (long long)tb * ldx + k) : zero;
+    for (int u = 0; u < UNROLL; ++u) {
+      const int k = k0 + u * kRouterWarps * 32 + c * 8;
+      const bool ok = k < H;
 #pragma unroll
       for (int n = 0; n < NT; ++n) {
-        moe_mma(acc[m][n], a.x, d.x, a.y, d.y, b[n].x, b[n].y);
-        moe_mma(acc[m][n], a.z, d.z, a.w, d.w, b[n].z, b[n].w);
+        const int e = n0 + n * 8 + r;
+        b[u][n] = (ok && e < E) ? __ldg(reinterpret_cast<const uint4*>(wr + (long long)e * ldw + k)) : zero;
       }
+#pragma unroll
+      for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+          const int t = t0 + m * 16 + h * 8 + r;
+          xa[u][m][h] = (ok && t < T) ? *reinterpret_cast<const uint4*>(x + (long long)t * ldx + k) : zero;
+        }
     }
+#pragma unroll
+    for (int u = 0; u < UNROLL; ++u)
+#pragma unroll
+      for (int m = 0; m < MT; ++m) {
+        const uint4 &p = xa[u][m][0], &q = xa[u][m][1];
+#pragma unroll
+        for (int n = 0; n < NT; ++n) {
+          moe_mma(acc[m][n], p.x, q.x, p.y, q.y, b[u][n].x, b[u][n].y);
+          moe_mma(acc[m][n], p.z, q.z, p.w, q.w, b[u][n].z, b[u][n].w);
+        }
+      }
   }
 #pragma unroll
   for (int m = 0; m < MT; ++m) {
@@ -124,21 +133,22 @@ LX_DEVICE void warp_argmax(float& v, int& i) {
   }
 }
 
-constexpr int kSelWarps = 8, kSelPer = kMoeMaxExperts / 32;
+constexpr int kSelWarps = 8;
 
 // The order of rows inside a run depends on the order of the atomics; every row's result is independent of it and the combine sums
-// a token's contributions in index order.
+// a token's contributions in index order.  PER: experts per lane.
+template <int PER>
 __global__ void __launch_bounds__(32 * kSelWarps) moe_select_kernel(const MoeSelectParams p) {
   pdl_wait();
-  __shared__ float choice_s[kSelWarps][kMoeMaxExperts];
-  __shared__ uint8_t kept_s[kSelWarps][kMoeMaxExperts];
+  __shared__ float choice_s[kSelWarps][32 * PER];
+  __shared__ uint8_t kept_s[kSelWarps][32 * PER];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * kSelWarps + warp;
   if (t >= p.T) return;
   const float* l = p.logits + (long long)t * p.ldl;
-  float choice[kSelPer];
+  float choice[PER];
 #pragma unroll
-  for (int i = 0; i < kSelPer; ++i) {
+  for (int i = 0; i < PER; ++i) {
     const int e = lane + 32 * i;
     float v = -INFINITY;
     if (e < p.E) {
@@ -150,12 +160,12 @@ __global__ void __launch_bounds__(32 * kSelWarps) moe_select_kernel(const MoeSel
   if (p.groups > 0) {
     const int gs = p.E / p.groups;
 #pragma unroll
-    for (int i = 0; i < kSelPer; ++i)
+    for (int i = 0; i < PER; ++i)
       if (lane + 32 * i < p.E) choice_s[warp][lane + 32 * i] = choice[i];
     __syncwarp();
-    float score[kSelPer];
+    float score[PER];
 #pragma unroll
-    for (int i = 0; i < kSelPer; ++i) {
+    for (int i = 0; i < PER; ++i) {
       const int g = lane + 32 * i;
       score[i] = -INFINITY;
       if (g < p.groups) {
@@ -173,20 +183,20 @@ __global__ void __launch_bounds__(32 * kSelWarps) moe_select_kernel(const MoeSel
       float bv = -INFINITY;
       int bi = 0x7fffffff;
 #pragma unroll
-      for (int i = 0; i < kSelPer; ++i)
+      for (int i = 0; i < PER; ++i)
         if (score[i] > bv) { bv = score[i]; bi = lane + 32 * i; }
       warp_argmax(bv, bi);
       if (bi >= p.groups) bi = j;                                  // (scores that are not numbers: any group)
       if (lane == (bi & 31)) {
         kept_s[warp][bi] = 1;
 #pragma unroll
-        for (int i = 0; i < kSelPer; ++i)
+        for (int i = 0; i < PER; ++i)
           if (i == (bi >> 5)) score[i] = -INFINITY;
       }
     }
     __syncwarp();
 #pragma unroll
-    for (int i = 0; i < kSelPer; ++i) {
+    for (int i = 0; i < PER; ++i) {
       const int e = lane + 32 * i;
       if (e < p.E && !kept_s[warp][e / gs]) choice[i] = -INFINITY;
     }
@@ -197,13 +207,13 @@ __global__ void __launch_bounds__(32 * kSelWarps) moe_select_kernel(const MoeSel
     float bv = -INFINITY;
     int bi = 0x7fffffff;
 #pragma unroll
-    for (int i = 0; i < kSelPer; ++i)
+    for (int i = 0; i < PER; ++i)
       if (choice[i] > bv) { bv = choice[i]; bi = lane + 32 * i; }
     warp_argmax(bv, bi);
     if (bi >= p.E) bi = j;
     if (lane == (bi & 31)) {
 #pragma unroll
-      for (int i = 0; i < kSelPer; ++i)
+      for (int i = 0; i < PER; ++i)
         if (i == (bi >> 5)) choice[i] = -INFINITY;
     }
     if (lane == j) id = bi;
@@ -226,8 +236,8 @@ __global__ void __launch_bounds__(32 * kSelWarps) moe_select_kernel(const MoeSel
 }
 
 // ------------------------------------------------------------------------------------------------ place, gather, combine
-// Every CTA sums the counts up by itself; one warp per (token, choice) turns the rank into the sorted row and copies the token's row
-// there, 16 bytes per lane and pass.  Pairs past T * k are the tokens' rows for the shared experts.
+// Every CTA sums the counts up by itself; one warp per (token, 2 KB of its row) turns the ranks of the token's choices into sorted rows
+// and writes its part of the row to each of them (and to the shared experts' rows, which are the tokens in order).
 struct MoePlaceParams {
   const uint8_t* x;
   uint8_t* xg;
@@ -235,7 +245,8 @@ struct MoePlaceParams {
   int row_bytes;
   const int* counts;
   const int* topk_ids;
-  int* pos;                // [T, k + shared]: rank on entry, sorted row (or -1) on exit
+  const int* rank;         // [T, k + shared] of lx_moe_select
+  int* pos;                // [T, k + shared]: sorted row (or -1)
   int* seg;                // [e_local + shared + 1]
   int T, k, e0, e_local, shared, rows_cap;
 };
@@ -265,27 +276,36 @@ __global__ void __launch_bounds__(256) moe_place_kernel(const MoePlaceParams p) 
     for (int e = threadIdx.x; e <= p.e_local; e += blockDim.x) p.seg[e] = start[e];
     for (int i = threadIdx.x; i < p.shared; i += blockDim.x) p.seg[p.e_local + 1 + i] = total + (i + 1) * p.T;
   }
-  const long long items = (long long)p.T * (p.k + (p.shared > 0 ? 1 : 0));
-  for (long long it = (blockIdx.x * (long long)blockDim.x + threadIdx.x) >> 5; it < items; it += ((long long)gridDim.x * blockDim.x) >> 5) {
-    int t, q;
-    if (it < (long long)p.T * p.k) {
-      t = (int)(it / p.k);
-      const int j = (int)(it % p.k);
-      int rank = 0;
-      if (lane == 0) rank = p.pos[(long long)t * kw + j];
-      rank = __shfl_sync(0xffffffffu, rank, 0);
-      if (rank < 0) continue;
-      q = start[p.topk_ids[it] - p.e0] + rank;
-      if (lane == 0) p.pos[(long long)t * kw + j] = q;
-    } else {
-      t = (int)(it - (long long)p.T * p.k);
-      q = total + t;
-      for (int i = lane; i < p.shared; i += 32) p.pos[(long long)t * kw + p.k + i] = q + i * p.T;
+  constexpr int kPart = 2048;
+  const int parts = (p.row_bytes + kPart - 1) / kPart;
+  for (long long it = (blockIdx.x * (long long)blockDim.x + threadIdx.x) >> 5; it < (long long)p.T * parts;
+       it += ((long long)gridDim.x * blockDim.x) >> 5) {
+    const int t = (int)(it / parts), part = (int)(it % parts);
+    uint4 v[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int b = part * kPart + i * 512 + lane * 16;
+      if (b < p.row_bytes) v[i] = *reinterpret_cast<const uint4*>(p.x + (long long)t * p.ldx + b);
     }
-    if (q >= p.rows_cap) continue;
-    const uint8_t* src = p.x + (long long)t * p.ldx;
-    uint8_t* dst = p.xg + (long long)q * p.ldg;
-    for (int b = lane * 16; b < p.row_bytes; b += 512) *reinterpret_cast<uint4*>(dst + b) = *reinterpret_cast<const uint4*>(src + b);
+    int q = -1;
+    if (lane < p.k) {
+      const int rank = p.rank[(long long)t * kw + lane];
+      if (rank >= 0) q = start[p.topk_ids[(long long)t * p.k + lane] - p.e0] + rank;
+      if (part == 0) p.pos[(long long)t * kw + lane] = q;
+    }
+    if (part == 0)
+      for (int i = lane; i < p.shared; i += 32) p.pos[(long long)t * kw + p.k + i] = total + i * p.T + t;
+    const int rows = p.k + (p.shared > 0 ? 1 : 0);
+    for (int j = 0; j < rows; ++j) {
+      const int row = j < p.k ? __shfl_sync(0xffffffffu, q, j) : total + t;
+      if (row < 0 || row >= p.rows_cap) continue;
+      uint8_t* dst = p.xg + (long long)row * p.ldg;
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int b = part * kPart + i * 512 + lane * 16;
+        if (b < p.row_bytes) *reinterpret_cast<uint4*>(dst + b) = v[i];
+      }
+    }
   }
 }
 
@@ -618,13 +638,17 @@ int lx_moe_router_logits(const void* x, long long ldx, const void* wr, long long
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const __nv_bfloat16* xp = reinterpret_cast<const __nv_bfloat16*>(x);
   const __nv_bfloat16* wp = reinterpret_cast<const __nv_bfloat16*>(wr);
-#define LX_RL(MT, NT)                                                                                                                    \
-  launch_pdl(moe_router_logits_kernel<MT, NT>, dim3((T + 16 * MT - 1) / (16 * MT), (E + 8 * NT - 1) / (8 * NT)), dim3(32 * kRouterWarps), 0, s, \
+#define LX_RL(MT, NT, UN)                                                                                                                    \
+  launch_pdl(moe_router_logits_kernel<MT, NT, UN>, dim3((T + 16 * MT - 1) / (16 * MT), (E + 8 * NT - 1) / (8 * NT)), dim3(32 * kRouterWarps), 0, s, \
              xp, ldx, wp, ldw, logits, T, E, H, counts, ncounts)
-  if (E <= 8) { if (T >= 4096) LX_RL(2, 1); else LX_RL(1, 1); }
-  else if (T <= 512) LX_RL(1, 2);                                  // few tokens: the experts' rows are spread over the CTAs
-  else if (E <= 32) LX_RL(2, 4);
-  else LX_RL(2, 8);
+  const int tiles = (E + 7) / 8;
+  if (tiles == 1) { if (T >= 4096) LX_RL(2, 1, 4); else LX_RL(1, 1, 8); }
+  else if (T <= 512) LX_RL(1, 2, 8);                               // few tokens: the experts' rows are spread over the CTAs
+  else if (tiles == 2) LX_RL(2, 2, 4);
+  else if (tiles == 3) LX_RL(2, 3, 4);
+  else if (tiles <= 5) LX_RL(2, 5, 2);
+  else if (tiles <= 8) LX_RL(2, 8, 2);
+  else LX_RL(2, 9, 2);
 #undef LX_RL
   return -(int)cudaGetLastError();
 }
@@ -639,7 +663,12 @@ int lx_moe_select(const void* params, void* stream) {
   if (p.E > kMoeMaxExperts || p.E < 1 || p.k > kMoeMaxK || p.k > p.E || p.k < 1 || p.e_local > kMoeMaxExperts || p.shared > kMoeMaxShared) return -1;
   if (p.ldl < p.E + (p.shared > 0 ? 1 : 0)) return -2;
   if (p.groups > 0 && (p.E % p.groups != 0 || p.keep < 1 || p.keep > p.groups || p.keep * (p.E / p.groups) < p.k)) return -3;
-  launch_pdl(moe_select_kernel, dim3((p.T + kSelWarps - 1) / kSelWarps), dim3(32 * kSelWarps), 0, reinterpret_cast<cudaStream_t>(stream), p);
+  const dim3 grid((p.T + kSelWarps - 1) / kSelWarps), block(32 * kSelWarps);
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  if (p.E <= 32) launch_pdl(moe_select_kernel<1>, grid, block, 0, s, p);
+  else if (p.E <= 64) launch_pdl(moe_select_kernel<2>, grid, block, 0, s, p);
+  else if (p.E <= 128) launch_pdl(moe_select_kernel<4>, grid, block, 0, s, p);
+  else launch_pdl(moe_select_kernel<8>, grid, block, 0, s, p);
   return -(int)cudaGetLastError();
 }
 
@@ -648,7 +677,7 @@ int lx_moe_place(const void* params, void* stream) {
   const MoePlaceParams& p = *reinterpret_cast<const MoePlaceParams*>(params);
   if (p.T <= 0) return 0;
   if (p.row_bytes % 16 != 0 || p.ldx % 16 != 0 || p.ldg % 16 != 0 || p.e_local > kMoeMaxExperts || p.e_local < 1) return -1;
-  const long long items = (long long)p.T * (p.k + (p.shared > 0 ? 1 : 0));
+  const long long items = (long long)p.T * ((p.row_bytes + 2047) / 2048);
   const int blocks = (int)(items / 8 + 1 < 148 * 8 ? items / 8 + 1 : 148 * 8);
   launch_pdl(moe_place_kernel, dim3(blocks), dim3(256), 0, reinterpret_cast<cudaStream_t>(stream), p);
   return -(int)cudaGetLastError();
@@ -683,7 +712,8 @@ int lx_moe_grouped_gemm(const void* xg, long long ldx, const void* w, long long 
                reinterpret_cast<const float*>(w), ldw, reinterpret_cast<float*>(out), p);
     return -(int)cudaGetLastError();
   }
-  int bn = (avg_rows + 15) / 16 * 16;
+  // few rows per expert: a tile twice the average holds most runs whole (a second tile would read the weights again)
+  int bn = ((avg_rows < 128 ? 2 * avg_rows : avg_rows) + 15) / 16 * 16;
   if (bn < 16) bn = 16;
   if (bn > 256) bn = 256;
   const int tbn = bn <= 16 ? 16 : bn <= 32 ? 32 : bn <= 64 ? 64 : bn <= 128 ? 128 : 256;

@@ -377,7 +377,7 @@ class MoeMlp:
                 self.up[s.experts + i, : b - a, : self.width] = up[a:b]
                 self.down[s.experts + i, : self.width, : b - a] = down[:, a:b]
             router.append(get("shared.sg"))
-        self.router = fin(_pad_to(torch.cat(router), pad16(s.experts + 1), self.W))
+        self.router = fin(_pad_to(torch.cat(router), (s.experts + 8) // 8 * 8, self.W))      # (whole tiles of the router kernel)
         self.correction = vec(get("correction"))
 
     def run(self, model, h):

@@ -329,7 +329,7 @@ class MoeSelectParams(ctypes.Structure):
 class MoePlaceParams(ctypes.Structure):
     """Mirror of the C struct of the same name (csrc/kernels/moe.cu)."""
     _fields_ = [("x", c_void_p), ("xg", c_void_p), ("ldx", c_longlong), ("ldg", c_longlong), ("row_bytes", c_int), ("counts", c_void_p),
-                ("topk_ids", c_void_p), ("pos", c_void_p), ("seg", c_void_p), ("T", c_int), ("k", c_int), ("e0", c_int), ("e_local", c_int),
+                ("topk_ids", c_void_p), ("rank", c_void_p), ("pos", c_void_p), ("seg", c_void_p), ("T", c_int), ("k", c_int), ("e0", c_int), ("e_local", c_int),
                 ("shared", c_int), ("rows_cap", c_int)]
 
 
@@ -351,15 +351,16 @@ def moe_route(x: torch.Tensor, router_w: torch.Tensor, k: int, e0: int, e_local:
         _check(lib.lx_moe_router_logits(_ptr(x), x.stride(0), _ptr(router_w), router_w.stride(0), _ptr(logits), T, rows, H, _ptr(counts), e_local,
                                         _stream()), "lx_moe_router_logits")
     kw = k + shared
+    rank = torch.empty(T, kw, dtype=torch.int32, device=dev)
     r = MoeRouting(torch.empty(T, k, dtype=torch.int32, device=dev), torch.empty(T, kw, dtype=torch.float32, device=dev),
                    torch.empty(e_local + shared + 1, dtype=torch.int32, device=dev), torch.empty(T, kw, dtype=torch.int32, device=dev),
                    torch.empty(T * (k + (1 if shared else 0)), H, dtype=x.dtype, device=dev))
-    p = MoeSelectParams(_ptr(logits), _ptr(correction), _ptr(r.topk_ids), _ptr(r.topk_w), _ptr(r.pos), _ptr(counts), logits.stride(0), T, E, k,
+    p = MoeSelectParams(_ptr(logits), _ptr(correction), _ptr(r.topk_ids), _ptr(r.topk_w), _ptr(rank), _ptr(counts), logits.stride(0), T, E, k,
                         e0, e_local, int(score == "sigmoid"), groups, keep, shared, scale)
     _check(lib.lx_moe_select(ctypes.byref(p), _stream()), "lx_moe_select")
     size = x.element_size()
-    q = MoePlaceParams(_ptr(x), _ptr(r.xg), x.stride(0) * size, r.xg.stride(0) * size, H * size, _ptr(counts), _ptr(r.topk_ids), _ptr(r.pos),
-                       _ptr(r.seg), T, k, e0, e_local, shared, r.xg.shape[0])
+    q = MoePlaceParams(_ptr(x), _ptr(r.xg), x.stride(0) * size, r.xg.stride(0) * size, H * size, _ptr(counts), _ptr(r.topk_ids), _ptr(rank),
+                       _ptr(r.pos), _ptr(r.seg), T, k, e0, e_local, shared, r.xg.shape[0])
     _check(lib.lx_moe_place(ctypes.byref(q), _stream()), "lx_moe_place")
     return r
 

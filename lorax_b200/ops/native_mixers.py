@@ -379,10 +379,13 @@ def qk_norm_kvwrite(qkv, H: int, G: int, dk: int, dv: int, n: int, q_norm, k_nor
     nv._check(nv.load().lx_qk_norm_kvwrite(ctypes.byref(p), _f32(qkv), nv._stream()), "lx_qk_norm_kvwrite")
 
 
-def _gqa_splits(T: int, units: int, window: int, max_blocks: int, page: int, num_sms: int) -> int:
-    """CTAs that share the keys of one row and head group: enough for two per SM, but at least four pages each."""
+def _gqa_splits(ctas: int, window: int, max_blocks: int, page: int) -> int:
+    """Parts the keys of one row and head group are cut into: one when the rows fill the GPU, else enough to do so with at least four
+    pages each."""
+    if ctas >= 96:
+        return 1
     pages = min(max_blocks, (window + page - 1) // page + 1 if window > 0 else max_blocks)
-    return max(1, min(8, 2 * num_sms // max(1, T * units), pages // 4))
+    return max(1, min(8, 192 // max(1, ctas), pages // 4))
 
 
 def gqa_attn(q, cache, H: int, G: int, dk: int, dv: int, scale: float, window: int, inp, out):
@@ -397,7 +400,7 @@ def gqa_attn(q, cache, H: int, G: int, dk: int, dv: int, scale: float, window: i
         raise ValueError(f"the attention kernels take pages of {lib.lx_gqa_page_size()} tokens, not {page}")
     nd, dbt, _, ctx = inp.decode_view(T)
     if nd:
-        nsplit = _gqa_splits(nd, G * ((H // G + 15) // 16), window, dbt.shape[1], page, ws.num_sms)
+        nsplit = _gqa_splits(nd * G * ((H // G + 15) // 16), window, dbt.shape[1], page)
         part_o = part_lse = None
         if nsplit > 1:
             part_o = torch.empty(nd * H * nsplit * (dv + 1), dtype=torch.float32, device=q.device)

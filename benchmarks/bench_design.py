@@ -17,6 +17,7 @@ from __future__ import annotations
 import json
 import os
 import statistics
+import time
 
 REPO = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 
@@ -209,7 +210,8 @@ class OpTimer:
         if name == "rope_pairs":
             return (name, a[0].shape[0] * a[3] * a[6] * 4, 0)
         if name in ("embed", "embed_stream"):
-            return (name, a[0].shape[0] * a[1].shape[1] * (6 if name == "embed_stream" else 4), 0)
+            per = 4 if name == "embed" else 6 + (2 if kw.get("pos") is not None else 0) + (2 if kw.get("copy") is not None else 0)
+            return (name, a[0].shape[0] * a[1].shape[1] * per, 0)
         return (name, nb(*[t for t in a if hasattr(t, "numel")]), 0)
 
     def report(self, bw, fl):
@@ -279,6 +281,7 @@ def main(args):
                             info = dict(decode=False, seqs=n, ctx=n * length,
                                         pairs=n * (length * (length + 1) // 2 - max(0, length - window) * (max(0, length - window) + 1) // 2))
                             toks = n * length
+                        time.sleep(1.0)                      # no case inherits the heat of the one before
                         for _ in range(warm):
                             step()
                         torch.cuda.synchronize()

@@ -31,11 +31,12 @@ __global__ void __launch_bounds__(256) qk_norm_kvwrite_kernel(const QkNormParams
   pdl_trigger();
   pdl_wait();
   const bool values = blockIdx.y == 1;
-  const int width = values ? p.DV : p.DK, lanes = width / 8, heads = values ? p.G : p.H + p.G;
-  const long long item = (blockIdx.x * (long long)blockDim.x + threadIdx.x) / lanes;
-  const int c = (int)(threadIdx.x % lanes) * 8;
-  const bool live = item < (long long)p.T * heads;
-  const int t = live ? (int)(item / heads) : 0, h = live ? (int)(item % heads) : 0;
+  const int width = values ? p.DV : p.DK, lanes = width / 8;                      // 8, 16 or 32 threads
+  const unsigned heads = values ? p.G : p.H + p.G;
+  const unsigned item = (blockIdx.x * blockDim.x + threadIdx.x) >> (31 - __clz(lanes));
+  const int c = (int)(threadIdx.x & (lanes - 1)) * 8;
+  const bool live = item < (unsigned)p.T * heads;
+  const int t = live ? (int)(item / heads) : 0, h = live ? (int)(item - t * heads) : 0;
   T* src = reinterpret_cast<T*>(p.qkv) + t * p.ld + (values ? (long long)(p.H + p.G) * p.DK : 0) + (long long)h * width + c;
   float f[8];
   load8(src, f);
@@ -179,6 +180,7 @@ int lx_qk_norm_kvwrite(const void* params, int f32, void* stream) {
   if (p.T <= 0) return 0;
   if (!gqa_width(p.DK) || !gqa_width(p.DV) || p.ld % 8 != 0) return -1;
   const long long threads = (long long)p.T * ((p.H + p.G) * (p.DK / 8) > p.G * (p.DV / 8) ? (p.H + p.G) * (p.DK / 8) : p.G * (p.DV / 8));
+  if (threads >= 1ll << 31) return -2;
   const dim3 grid((unsigned)((threads + 255) / 256), 2);
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   if (f32) launch_pdl(qk_norm_kvwrite_kernel<float>, grid, dim3(256), 0, s, p);

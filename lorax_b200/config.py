@@ -16,7 +16,7 @@ import dataclasses
 import json
 import os
 from dataclasses import dataclass, field
-from typing import Any, Dict, List, Optional, Tuple
+from typing import Any, Callable, Dict, List, Optional, Tuple
 
 # Architectures handled by the single config-driven decoder (models/decoder.py).
 DECODER_MODEL_TYPES = (
@@ -27,14 +27,16 @@ DECODER_MODEL_TYPES = (
 
 
 # Designs whose config.json lists its layers one by one, each with a mixer of its own (models/mixers.py).
-MIXER_MODEL_TYPES = ("vabunex", "sapudra")
+MIXER_MODEL_TYPES = ("vabunex", "sapudra", "saredra")
 
 
 @dataclass
 class MoeSpec:
     """Routed feed-forward: `experts` of width `ff`, `top` of them per token, chosen within the best `keep` of `groups` groups of
-    neighbours (0: no groups); the chosen scores are normalised and multiplied by `scale`.  `shared_ff`: width of the gated expert
-    that every token takes beside them (0: none)."""
+    neighbours (0: no groups), a group counting by the sum of its `group_top` largest scores.  `score`: "sigmoid" (plus a correction
+    that takes part in the choice only) or "softmax" over all experts.  The weights are the chosen scores, normalised if `renorm`, times
+    `scale`.  `gated`: an expert is down(act(gate) * up) instead of down(act(up)).  `shared_ff`: width of the expert that every token
+    takes beside them, with a weight of its own (0: none)."""
     experts: int
     top: int
     ff: int
@@ -42,6 +44,10 @@ class MoeSpec:
     groups: int = 0
     keep: int = 0
     shared_ff: int = 0
+    score: str = "sigmoid"
+    renorm: bool = True
+    group_top: int = 2
+    gated: bool = False
 
     def __post_init__(self):
         if not 1 <= self.top <= self.experts:
@@ -56,11 +62,12 @@ class MoeSpec:
 @dataclass
 class LayerSpec:
     """One layer of a design whose layers differ: the kind of mixer, the mixer's sizes and constants, and its feed-forward: dense of
-    width `ff` (0: none), or routed experts (`moe`)."""
+    width `ff` (0: none; `gated`: act(gate) * up), or routed experts (`moe`)."""
     mixer: str
     params: Dict[str, Any]
     ff: int = 0
     moe: Optional[MoeSpec] = None
+    gated: bool = False
 
 
 @dataclass
@@ -115,8 +122,9 @@ class ModelConfig:
     # layer-by-layer designs: the layers, and (start, stop, times): layers start .. stop-1 run `times` times in a row
     layer_specs: Optional[List[LayerSpec]] = None
     layer_loop: Optional[Tuple[int, int, int]] = None
-    # their residual: "parallel" (mixer and feed-forward read one norm of the stream, both are added to it) or "post" (each sublayer
-    # reads the stream itself, and a norm of its output, times residual_multiplier, is added)
+    # their residual: "parallel" (mixer and feed-forward read one norm of the stream, both are added to it), "pre" (the mixer, then the
+    # feed-forward, each reading a norm of its own) or "post" (each sublayer reads the stream itself, and a norm of its output, times
+    # residual_multiplier, is added)
     layer_style: str = "parallel"
     eos_token_id: Any = None
     bos_token_id: Any = None
@@ -277,14 +285,17 @@ class ModelConfig:
         return d
 
 
-def _moe_spec(mlp: Dict[str, Any]) -> MoeSpec:
-    r, groups, shared = mlp["router"], mlp["router"].get("groups"), mlp.get("shared")
-    return MoeSpec(experts=int(r["experts"]), top=int(r["top"]), ff=int(mlp["expert"]["ff"]), scale=float(r.get("scale", 1.0)),
-                   groups=int(groups["count"]) if groups else 0, keep=int(groups["keep"]) if groups else 0,
-                   shared_ff=int(shared["ff"]) if shared else 0)
+@dataclass
+class MixerDesign:
+    """What a layer-by-layer design fixes itself; everything else comes from its config.json.  `constants` gives ModelConfig fields from
+    the config; `mixers` holds what a kind of mixer has in this design, under the sizes that the config gives."""
+    constants: Callable[[Dict[str, Any]], Dict[str, Any]]
+    feed_forwards: Tuple[str, ...]
+    gated: bool = True
+    moe: Dict[str, Any] = field(default_factory=dict)
+    mixers: Dict[str, Dict[str, Any]] = field(default_factory=dict)
 
 
-# What a layer-by-layer design fixes itself; everything else comes from its config.json.
 def _vabunex_constants(d: Dict[str, Any]) -> Dict[str, Any]:
     return dict(layer_style="parallel", parallel_residual=True, hidden_act="gelu_tanh", norm_weight_offset=1.0,
                 embedding_multiplier=float(d["embedding"]["scale"]), max_position_embeddings=int(d.get("max_position_embeddings", 1 << 20)))
@@ -297,32 +308,55 @@ def _sapudra_constants(d: Dict[str, Any]) -> Dict[str, Any]:
                 final_logit_softcapping=float(cap) if cap is not None else None)
 
 
-_MIXER_DESIGNS = {"vabunex": (_vabunex_constants, ("dense",)), "sapudra": (_sapudra_constants, ("dense", "moe"))}
+def _saredra_constants(d: Dict[str, Any]) -> Dict[str, Any]:
+    return dict(layer_style="pre", hidden_act="silu", max_position_embeddings=int(d.get("max_position_embeddings", 1 << 20)))
+
+
+_MIXER_DESIGNS = {
+    "vabunex": MixerDesign(_vabunex_constants, ("dense",)),
+    "sapudra": MixerDesign(_sapudra_constants, ("dense", "moe"), gated=False, mixers={"attention": dict(qk_norm=True)}),
+    "saredra": MixerDesign(_saredra_constants, ("dense", "moe"), moe=dict(score="softmax", renorm=False, group_top=1),
+                           mixers={"attention": dict(sink="unit", gate=True),
+                                   "parallel": dict(left=dict(type="attention", bias=True, sink="learned"), right=dict(type="mamba2"))}),
+}
+
+
+def _moe_spec(mlp: Dict[str, Any], design: MixerDesign) -> MoeSpec:
+    r, groups, shared = mlp["router"], mlp["router"].get("groups"), mlp.get("shared")
+    return MoeSpec(experts=int(r["experts"]), top=int(r["top"]), ff=int(mlp["expert"]["ff"]), scale=float(r.get("scale", 1.0)),
+                   groups=int(groups["count"]) if groups else 0, keep=int(groups["keep"]) if groups else 0,
+                   shared_ff=int(shared["ff"]) if shared else 0, gated=design.gated, **design.moe)
+
+
+def _mixer_params(own: Dict[str, Any], fixed: Dict[str, Any]) -> Dict[str, Any]:
+    """A mixer's sizes from the config over what the design fixes; mixers within a mixer likewise."""
+    return {**{k: v for k, v in fixed.items() if not isinstance(v, dict)}, **own,
+            **{k: _mixer_params(own[k], v) for k, v in fixed.items() if isinstance(v, dict)}}
 
 
 def _mixer_model_kwargs(mt: str, d: Dict[str, Any]) -> Dict[str, Any]:
     """ModelConfig fields of a config.json that lists its layers (`layers`, `loop`, `norm`, `vocab`, `width`)."""
-    constants, kinds = _MIXER_DESIGNS[mt]
+    design = _MIXER_DESIGNS[mt]
     specs = []
     for i, layer in enumerate(d["layers"]):
         mlp = layer.get("mlp")
         kind = mlp.get("kind", "dense") if mlp is not None else None
-        if kind is not None and kind not in kinds:
+        if kind is not None and kind not in design.feed_forwards:
             raise NotImplementedError(f"layer {i}: feed-forward kind {kind!r}")
-        specs.append(LayerSpec(layer["type"], dict(layer["mixer"]), int(mlp["ff"]) if kind == "dense" else 0,
-                               _moe_spec(mlp) if kind == "moe" else None))
+        specs.append(LayerSpec(layer["type"], _mixer_params(layer["mixer"], design.mixers.get(layer["type"], {})),
+                               int(mlp["ff"]) if kind == "dense" else 0, _moe_spec(mlp, design) if kind == "moe" else None, design.gated))
     loop = d.get("loop")
     if loop is not None:
         loop = (int(loop["start"]), int(loop["stop"]), int(loop["times"]))
         if not (0 <= loop[0] <= loop[1] <= len(specs)) or loop[2] < 0:
             raise ValueError(f"loop {loop} does not fit {len(specs)} layers")
-    heads = max([int(s.params["heads"]) for s in specs] + [1])
-    kv_heads = max([int(s.params.get("kv_heads", s.params["heads"])) for s in specs] + [1])
+    flat = [p for s in specs for p in ([s.params] if "heads" in s.params else [v for v in s.params.values() if isinstance(v, dict)])]
+    most = lambda *names: max([int(next(p[n] for n in names if n in p)) for p in flat if any(n in p for n in names)] + [1])
     return dict(dict(model_type=mt, vocab_size=int(d["vocab"]), hidden_size=int(d["width"]), intermediate_size=max([s.ff for s in specs] + [1]),
-                     num_hidden_layers=len(specs), num_attention_heads=heads, num_key_value_heads=kv_heads,
-                     head_dim=max([int(s.params["dim"]) for s in specs] + [1]), rms_norm_eps=float(d["norm"]["eps"]), layer_specs=specs,
+                     num_hidden_layers=len(specs), num_attention_heads=most("heads"), num_key_value_heads=most("kv_heads", "heads"),
+                     head_dim=most("dim"), rms_norm_eps=float(d["norm"]["eps"]), layer_specs=specs,
                      layer_loop=loop, eos_token_id=d.get("eos_token_id"), bos_token_id=d.get("bos_token_id"),
-                     torch_dtype=d.get("torch_dtype", "bfloat16"), extra={}), **constants(d))
+                     torch_dtype=d.get("torch_dtype", "bfloat16"), extra={}), **design.constants(d))
 
 
 def mistral_7b() -> ModelConfig:

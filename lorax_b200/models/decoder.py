@@ -155,8 +155,8 @@ class DecoderModel:
         self.mixed = c.layer_specs is not None   # layers with mixers of their own (models/mixers.py) on an fp32 residual stream
         self.recurrent = False
         if self.mixed:
-            from .mixers import MIXERS
-            self.recurrent = any(getattr(MIXERS.get(sp.mixer), "recurrent", False) for sp in c.layer_specs)
+            from .mixers import make_mixer
+            self.recurrent = any(make_mixer(sp, c.hidden_size).recurrent for sp in c.layer_specs)
         self.inter = c.intermediate_size // ws if not c.is_moe else c.intermediate_size
         self.hidden = c.hidden_size
         self.vocab = c.vocab_size
@@ -200,17 +200,19 @@ class DecoderModel:
             full = alibi_slopes(c.num_attention_heads, c.alibi_bias_max, interleave=c.model_type == "mpt")
             self.alibi_slopes = full[self.tp.rank * self.nh:(self.tp.rank + 1) * self.nh].to(self.device).contiguous()
 
-    def rope_table(self, rot: int, base: float) -> torch.Tensor:
+    def rope_table(self, rot: int, base: float, scaling: Optional[dict] = None) -> torch.Tensor:
         """cos / sin of a layer's own rotation, shared by the layers that have the same one."""
-        key = (rot, base)
+        key = (rot, base, tuple(sorted(scaling.items())) if scaling else None)
         if key not in self._rope_tables:
-            self._rope_tables[key] = reference.rope_table(rot, self.max_positions, base, self.device)
+            self._rope_tables[key] = reference.rope_table(rot, self.max_positions, base, self.device, scaling)
         return self._rope_tables[key]
 
     def check_positions(self, tokens: int):
-        """Refuses sequences longer than a layer-by-layer design's table of learned positions."""
+        """Refuses sequences longer than a layer-by-layer design's tables of positions."""
         if self.mixed and self.config.learned_positions and tokens > self.config.max_position_embeddings:
             raise ValueError(f"{self.config.model_type} has {self.config.max_position_embeddings} positions: max_total_tokens={tokens} is too long")
+        if self._rope_tables and tokens > self.max_positions:
+            raise ValueError(f"the rotation tables were made for {self.max_positions} positions: max_total_tokens={tokens} is too long")
 
     @property
     def state_parallelism(self) -> int:
@@ -219,7 +221,14 @@ class DecoderModel:
 
     def cache_shapes(self) -> Optional[List[dict]]:
         """What every layer run keeps (`Mixer.cache_shape`), or None for the uniform key/value cache."""
-        return [self.layers[li].mixer.cache_shape(self) for li in self.schedule] if self.mixed else None
+        if not self.mixed:
+            return None
+        shapes, run_of = [], {}
+        for run, li in enumerate(self.schedule):
+            shape = self.layers[li].mixer.cache_shape(self)
+            shapes.append({"share": run_of[shape["share_layer"]]} if "share_layer" in shape else shape)      # (its latest run so far)
+            run_of[li] = run
+        return shapes
 
     # ------------------------------------------------------------------ shapes
     @property
@@ -523,6 +532,8 @@ class DecoderModel:
         if self.mixed:
             if c.layer_style == "post":
                 return self._forward_post(inp, kv_cache)
+            if c.layer_style == "pre":
+                return self._forward_pre(inp, kv_cache)
             # fp32 residual stream; every layer hands its contribution to the norm that reads the stream next
             residual, pending = ops.embed_stream(inp.input_ids, self.embed, c.embedding_multiplier), None
             for run, li in enumerate(self.schedule):
@@ -582,6 +593,16 @@ class DecoderModel:
             h = self.layers[li].forward(self, residual, h, inp, kv_cache[run])
         hidden = ops.norm_stream(residual, None, self.final_norm, self.eps, c.norm_weight_offset, self.hidden, self.dtype, bias=self.final_norm_b,
                                  layernorm=c.norm_type == "layernorm", rows=inp.lm_head_indices)
+        return self._score(hidden, inp, selected=True)
+
+    def _forward_pre(self, inp: StepInputs, kv_cache) -> torch.Tensor:
+        """Mixer and feed-forward in turn, each behind a norm of its own that also adds what the sublayer before it contributed."""
+        c, ops = self.config, self.ops
+        residual, pending = ops.embed_stream(inp.input_ids, self.embed, c.embedding_multiplier), (None, None)
+        for run, li in enumerate(self.schedule):
+            pending = self.layers[li].forward(self, residual, pending, inp, kv_cache[run])
+        hidden = ops.norm_stream(residual, pending[0], self.final_norm, self.eps, c.norm_weight_offset, self.hidden, self.dtype, pairs=pending[1],
+                                 rows=inp.lm_head_indices)
         return self._score(hidden, inp, selected=True)
 
     def _score(self, hidden: torch.Tensor, inp: StepInputs, selected: bool = False) -> torch.Tensor:

@@ -1,6 +1,8 @@
-"""Layers of designs that list their layers one by one, over an fp32 residual stream.  Two styles:
+"""Layers of designs that list their layers one by one, over an fp32 residual stream.  Three styles:
 
   parallel   a token mixer and an optional gated feed-forward side by side, both reading one RMS norm of the stream (`MixerLayer`)
+  pre        the mixer, then the feed-forward (dense or routed experts), each reading an RMS norm of the stream of its own
+             (`PreNormLayer`)
   post       the mixer, then the feed-forward (dense or routed experts), each reading the stream itself; the norm of its output is
              added to the stream (`PostNormLayer`)
 
@@ -15,7 +17,10 @@ channel stays exactly zero through every operation.
   wkv               token-shifted linear recurrence with a data-dependent decay per key channel, state [heads, dim, dim] per request
                     plus the previous token's input
   latent_attention  softmax attention over a low-rank latent and one shared rotated key part per token, both paged
-  attention         grouped-query softmax attention over paged keys and values, normed queries and keys, a sliding window of its own
+  attention         grouped-query softmax attention over paged keys and values, with a choice of normed queries and keys, short
+                    convolutions, rotation, capped scores, sliding window, sink, output gate, keys and values of another layer
+  mamba2            selective state space recurrence behind a short convolution, state [heads, state, vdim] per request, gated norm
+  parallel          two mixers that read the same rows, their outputs weighted and added
 """
 
 from __future__ import annotations
@@ -59,7 +64,8 @@ class Mixer:
     """Common part.  `get(name)` passed to `load` returns the checkpoint tensor of this mixer in fp32; `fin` brings a matrix to the
     model's dtype and device, `vec` a vector to fp32 on the device."""
 
-    recurrent = False
+    recurrent = False                                        # keeps something per request
+    parallelism = 1 << 20                                    # thread blocks that one sequence gives the recurrence kernels
 
     def __init__(self, params: dict, width: int):
         self.width, self.W = width, pad16(width)
@@ -71,6 +77,10 @@ class Mixer:
         """(name, [rows, W]) of the projections that read the layer's norm."""
         raise NotImplementedError
 
+    def in_bias(self, get) -> Dict[str, torch.Tensor]:
+        """Bias vectors [rows] of those that have one."""
+        return {}
+
     def out_part(self, get) -> torch.Tensor:
         """Output projection [W, out_dim]."""
         raise NotImplementedError
@@ -79,7 +89,8 @@ class Mixer:
         raise NotImplementedError
 
     def cache_shape(self, model) -> dict:
-        """{"paged": width per token}, {"kv": (heads, key width, value width)} or {"state": {name: (shape per request, dtype)}}."""
+        """{"paged": width per token}, {"kv": (heads, key width, value width)} and / or {"state": {name: (shape per request, dtype)}},
+        {"share_layer": the layer whose entry this one reads}, or {"parts": {name: one of these}}."""
         raise NotImplementedError
 
     def run(self, model, h, proj, y, inp, cache):
@@ -238,21 +249,51 @@ class LatentAttentionMixer(Mixer):
 
 
 class AttentionMixer(Mixer):
-    """Grouped-query attention.  Queries and keys are divided by their root mean square per head (weights shared by the heads); no
-    rotation; token i sees the last `mask.size` tokens including itself."""
+    """Grouped-query attention over paged keys and values.  What a design or layer has of the following is a parameter:
+
+      mask.size   token i sees the last `size` tokens including itself (no mask: all before it)
+      qk_norm     queries and keys divided by their root mean square per head (weights shared by the heads)
+      bias        biases of the projections
+      conv        short causal convolution of this many taps on every channel of q, k and v, in front of the rotation
+      rot         rotation of the first `dims` dimensions of q and k, interleaved pairs, `base`, optionally YaRN `scaling`
+      softcap     scores s become softcap * tanh(s / softcap)
+      sink        "learned": a score per head that only the denominator contains; "unit": the denominator plus one
+      gate        the heads times sigmoid of a projection of the same input
+      out_scale   factor of the output
+      kv_from     the layer whose keys and values it uses in place of its own"""
 
     HEAD_SIZES = (64, 128, 256)                              # of the attention kernels; a head is padded to the next one
+    MAX_TAPS = 9                                             # of the convolution kernel
 
     def __init__(self, params: dict, width: int):
         super().__init__(params, width)
         self.H, self.G, self.d, self.dv = (int(params[n]) for n in ("heads", "kv_heads", "dim", "vdim"))
         if self.H % self.G:
             raise ValueError(f"{self.H} query heads over {self.G} key/value heads")
-        self.scale, self.window = float(params["scale"]), int(params["mask"]["size"])
-        if self.window < 1:
+        mask, self.rot, self.sink = params.get("mask"), params.get("rot"), params.get("sink")
+        self.scale, self.window = float(params["scale"]), int(mask["size"]) if mask else 0
+        if mask and self.window < 1:
             raise ValueError(f"a window of {self.window} tokens")
+        if self.scale <= 0:
+            raise ValueError(f"a score scale of {self.scale}")
+        self.softcap, self.out_scale = float(params.get("softcap") or 0.0), float(params.get("out_scale", 1.0))
+        self.qk_norm, self.bias, self.gate = (bool(params.get(n)) for n in ("qk_norm", "bias", "gate"))
+        self.taps, self.kv_from = int(params.get("conv") or 0), params.get("kv_from")
+        self.rot_dims = int(self.rot["dims"]) if self.rot else 0
+        if self.rot_dims % 2 or self.rot_dims > self.d:
+            raise ValueError(f"rotation of {self.rot_dims} of {self.d} dimensions")
+        if self.taps > self.MAX_TAPS:
+            raise NotImplementedError(f"convolutions of {self.taps} taps (up to {self.MAX_TAPS})")
+        if self.qk_norm and (self.taps or self.rot_dims or self.kv_from is not None):
+            raise NotImplementedError("normed queries and keys with a convolution, a rotation or another layer's keys")
+        if self.kv_from is not None and self.taps:
+            raise NotImplementedError("another layer's keys with a convolution")
+        self.recurrent = self.taps > 1
         self.dp, self.dvp = self._padded(self.d), self._padded(self.dv)
         self.out_dim = self.H * self.dvp
+        # projections: name, heads, width of a head, padded width
+        own = [("k", self.G, self.d, self.dp), ("v", self.G, self.dv, self.dvp)] if self.kv_from is None else []
+        self.projections = [("q", self.H, self.d, self.dp)] + own
 
     def _padded(self, n: int) -> int:
         for size in self.HEAD_SIZES:
@@ -261,37 +302,195 @@ class AttentionMixer(Mixer):
         raise NotImplementedError(f"attention heads of {n} (up to {self.HEAD_SIZES[-1]})")
 
     def shapes(self):
-        H, G, d, dv, w = self.H, self.G, self.d, self.dv, self.width
-        return {"q": (H * d, w), "k": (G * d, w), "v": (G * dv, w), "q.norm": (d,), "k.norm": (d,), "o": (w, H * dv)}
+        w, out = self.width, {}
+        for n, heads, d, _ in self.projections:
+            out[n] = (heads * d, w)
+            if self.bias:
+                out[n + ".b"] = (heads * d,)
+            if self.taps:
+                out[n + ".conv"] = (heads * d, self.taps)
+        if self.qk_norm:
+            out.update({"q.norm": (self.d,), "k.norm": (self.d,)})
+        if self.sink == "learned":
+            out["sink"] = (self.H,)
+        if self.gate:
+            out["g"] = (self.H * self.dv, w)
+        out["o"] = (w, self.H * self.dv)
+        return out
+
+    def _rows(self, t, heads, d, dp, cols):
+        return _pad_to(t.view(heads, d, -1), heads, dp, cols).reshape(heads * dp, cols)
 
     def in_parts(self, get):
-        rows = lambda n, heads, d, dp: _pad_to(get(n).view(heads, d, -1), heads, dp, self.W).reshape(heads * dp, self.W)
-        return [("qkv", torch.cat([rows("q", self.H, self.d, self.dp), rows("k", self.G, self.d, self.dp), rows("v", self.G, self.dv, self.dvp)]))]
+        out = [("qkv", torch.cat([self._rows(get(n), heads, d, dp, self.W) for n, heads, d, dp in self.projections]))]
+        return out + ([("g", self._rows(get("g"), self.H, self.dv, self.dvp, self.W))] if self.gate else [])
+
+    def in_bias(self, get):
+        if not self.bias:
+            return {}
+        return {"qkv": torch.cat([self._rows(get(n + ".b"), heads, d, dp, 1)[:, 0] for n, heads, d, dp in self.projections])}
 
     def out_part(self, get):
         o = get("o")
         return _pad_to(o.view(o.shape[0], self.H, self.dv), self.W, self.H, self.dvp).reshape(self.W, self.out_dim)
 
     def load(self, get, fin, vec, model):
-        self.q_norm, self.k_norm = (vec(_pad_to(get(n), self.dp)) for n in ("q.norm", "k.norm"))
+        if self.qk_norm:
+            self.q_norm, self.k_norm = (vec(_pad_to(get(n), self.dp)) for n in ("q.norm", "k.norm"))
+        self.sinks = vec(get("sink")) if self.sink == "learned" else vec(torch.zeros(self.H)) if self.sink == "unit" else None
+        self.conv_w = None
+        if self.taps:                                        # [taps, channels]
+            self.conv_w = vec(torch.cat([self._rows(get(n + ".conv"), heads, d, dp, self.taps) for n, heads, d, dp in self.projections]).t())
+        self.cos_sin = model.rope_table(self.rot_dims, float(self.rot["base"]), self.rot.get("scaling")) if self.rot_dims else None
+        if self.kv_from is not None:
+            self._check_source(model)
+
+    def _check_source(self, model):
+        """The layers in front of this one are there already."""
+        src = model.layers[self.kv_from].mixer if 0 <= self.kv_from < len(model.layers) else None
+        src = getattr(src, "kv_mixer", src)
+        if not isinstance(src, AttentionMixer) or src.kv_from is not None:
+            raise ValueError(f"layer {self.kv_from} has no keys and values of its own in front of the layer that uses them")
+        if (src.G, src.d, src.dv) != (self.G, self.d, self.dv):
+            raise ValueError(f"layer {self.kv_from} has other key/value heads than the layer that uses them")
 
     def cache_shape(self, model):
-        return {"kv": (self.G, self.dp, self.dvp)}
+        if self.kv_from is not None:
+            return {"share_layer": self.kv_from}
+        out = {"kv": (self.G, self.dp, self.dvp)}
+        if self.recurrent:
+            out["state"] = {"conv": ((self.taps - 1, self.conv_w.shape[1]), model.dtype)}
+        return out
 
     def run(self, model, h, proj, y, inp, cache):
-        qkv = proj["qkv"]
-        model.ops.qk_norm_kvwrite(qkv, self.H, self.G, self.dp, self.dvp, self.d, self.q_norm, self.k_norm, model.eps, cache, inp.slots)
-        model.ops.gqa_attn(qkv, cache, self.H, self.G, self.dp, self.dvp, self.scale, self.window, inp, y)
+        qkv, ops, conv = proj["qkv"], model.ops, None
+        while isinstance(cache, dict):                       # pages beside a state, or those of a mixer within a layer
+            conv, cache = cache.get("conv"), cache["kv"] if "kv" in cache else cache["left"]
+        if self.qk_norm:
+            q = qkv
+            ops.qk_norm_kvwrite(qkv, self.H, self.G, self.dp, self.dvp, self.d, self.q_norm, self.k_norm, model.eps, cache, inp.slots)
+        else:
+            own = self.G if self.kv_from is None else 0
+            q = ops.conv_rope_kvwrite(qkv, self.H, own, self.dp, self.dvp, self.cos_sin, self.rot_dims, inp.positions, cache, inp, self.conv_w, conv)
+        ops.gqa_attn(q, cache, self.H, self.G, self.dp, self.dvp, self.scale, self.window, inp, y, softcap=self.softcap, sink=self.sinks,
+                     gate=proj.get("g"), out_scale=self.out_scale)
 
 
-MIXERS = {"lightning": LightningMixer, "wkv": WkvMixer, "latent_attention": LatentAttentionMixer, "attention": AttentionMixer}
+class Mamba2Mixer(Mixer):
+    """Selective state space recurrence: x, B and C through a short causal convolution and silu, a decay and a step size per token and
+    head, the state [state, vdim] of a head, then the gate and an RMS norm of `norm_groups` equal parts."""
+
+    recurrent = True
+    MAX_STATE = 256                                          # of the recurrence kernels
+
+    def __init__(self, params: dict, width: int):
+        super().__init__(params, width)
+        self.H, self.dv, self.n, self.G = (int(params[k]) for k in ("heads", "vdim", "state", "groups"))
+        self.taps, self.parts, self.out_scale = int(params["conv"]), int(params["norm_groups"]), float(params.get("out_scale", 1.0))
+        self.inner = self.H * self.dv
+        if self.H % self.G or self.inner % self.parts:
+            raise ValueError(f"{self.H} heads of {self.dv} in {self.G} groups, normed in {self.parts} parts")
+        if not 1 <= self.taps <= AttentionMixer.MAX_TAPS or self.n > self.MAX_STATE:
+            raise NotImplementedError(f"a state of {self.n} (up to {self.MAX_STATE}) behind {self.taps} taps (1 to {AttentionMixer.MAX_TAPS})")
+        self.np, self.dvp = pad16(self.n), pad16(self.dv)
+        self.out_dim = pad16(self.inner)
+        self.channels = self.H * self.dvp + 2 * self.G * self.np
+        self.parallelism = self.H * ((self.dvp + 63) // 64)
+
+    def shapes(self):
+        c = self.inner + 2 * self.G * self.n
+        return {"in": (self.inner + c + self.H, self.width), "conv": (c, self.taps), "conv.b": (c,), "dt_bias": (self.H,), "A_log": (self.H,),
+                "D": (self.H,), "norm": (self.inner,), "o": (self.width, self.inner)}
+
+    def _channels(self, t, cols):
+        """Rows [x | B | C], every head and group padded on its own."""
+        x, b, c = torch.split(t.reshape(t.shape[0], -1), [self.inner, self.G * self.n, self.G * self.n])
+        pad = lambda u, heads, d: _pad_to(u.reshape(heads, d, -1), heads, pad16(d), cols).reshape(heads * pad16(d), cols)
+        return torch.cat([pad(x, self.H, self.dv), pad(b, self.G, self.n), pad(c, self.G, self.n)])
+
+    def in_parts(self, get):
+        z, xbc, dt = torch.split(get("in"), [self.inner, self.inner + 2 * self.G * self.n, self.H])
+        return [("z", pad_heads_rows(z, self.H, self.dv, self.W)), ("xbc", self._channels(xbc, self.W)), ("dt", _pad_to(dt, pad16(self.H), self.W))]
+
+    def out_part(self, get):
+        return _pad_to(get("o"), self.W, self.out_dim)
+
+    def load(self, get, fin, vec, model):
+        self.conv_w = vec(self._channels(get("conv"), self.taps).t())              # [taps, channels]
+        self.conv_b = vec(self._channels(get("conv.b"), 1)[:, 0])
+        self.dt_bias, self.D = vec(get("dt_bias")), vec(get("D"))
+        self.A = vec(-torch.exp(get("A_log")))
+        self.norm = vec(get("norm") * self.out_scale)
+
+    def cache_shape(self, model):
+        return {"state": {"S": ((self.H, self.np, self.dvp), torch.float32), "conv": ((self.taps - 1, self.channels), model.dtype)}}
+
+    def run(self, model, h, proj, y, inp, cache):
+        ops = model.ops
+        xbc = ops.causal_conv(proj["xbc"], self.conv_w, self.conv_b, "silu", cache["conv"], inp)
+        o = ops.ssd(xbc, proj["dt"], self.H, self.G, self.np, self.dvp, self.dt_bias, self.A, self.D, cache["S"], inp)
+        ops.gate_norm(o, proj["z"], self.H, self.dv, self.parts, self.norm, model.eps, y)
+
+
+class ParallelMixer(Mixer):
+    """left_scale * left(h) + right_scale * right(h).  Both write side by side into one buffer, already scaled, and their output
+    projections are one product whose K runs over both."""
+
+    SIDES = ("left", "right")
+
+    def __init__(self, params: dict, width: int):
+        super().__init__(params, width)
+        sub = lambda side: dict({k: v for k, v in params[side].items() if k != "type"}, out_scale=float(params.get(side + "_scale", 1.0)))
+        self.sides = {s: _mixer_class(params[s]["type"])(sub(s), width) for s in self.SIDES}
+        for m in self.sides.values():
+            if not hasattr(m, "out_scale"):
+                raise NotImplementedError(f"{type(m).__name__} beside another mixer")
+        self.recurrent = any(m.recurrent for m in self.sides.values())
+        self.parallelism = min(m.parallelism for m in self.sides.values())
+        self.out_dim = sum(m.out_dim for m in self.sides.values())
+        self.kv_mixer = self.sides["left"]
+
+    def _each(self, get):
+        return ((s, m, lambda name, s=s: get(f"{s}.{name}")) for s, m in self.sides.items())
+
+    def shapes(self):
+        return {f"{s}.{n}": shape for s, m in self.sides.items() for n, shape in m.shapes().items()}
+
+    def in_parts(self, get):
+        return [(f"{s}.{n}", t) for s, m, sub in self._each(get) for n, t in m.in_parts(sub)]
+
+    def in_bias(self, get):
+        return {f"{s}.{n}": t for s, m, sub in self._each(get) for n, t in m.in_bias(sub).items()}
+
+    def out_part(self, get):
+        return torch.cat([m.out_part(sub) for _, m, sub in self._each(get)], 1)
+
+    def load(self, get, fin, vec, model):
+        for _, m, sub in self._each(get):
+            m.load(sub, fin, vec, model)
+
+    def cache_shape(self, model):
+        return {"parts": {s: m.cache_shape(model) for s, m in self.sides.items()}}
+
+    def run(self, model, h, proj, y, inp, cache):
+        at = 0
+        for s, m in self.sides.items():
+            m.run(model, h, {n[len(s) + 1:]: v for n, v in proj.items() if n.startswith(s + ".")}, y[:, at: at + m.out_dim], inp, cache[s])
+            at += m.out_dim
+
+
+MIXERS = {"lightning": LightningMixer, "wkv": WkvMixer, "latent_attention": LatentAttentionMixer, "attention": AttentionMixer,
+          "mamba2": Mamba2Mixer, "parallel": ParallelMixer}
+
+
+def _mixer_class(name: str):
+    if name not in MIXERS:
+        raise NotImplementedError(f"no mixer {name!r}; known: {sorted(MIXERS)}")
+    return MIXERS[name]
 
 
 def make_mixer(spec, width: int) -> Mixer:
-    cls = MIXERS.get(spec.mixer)
-    if cls is None:
-        raise NotImplementedError(f"no mixer {spec.mixer!r}; known: {sorted(MIXERS)}")
-    return cls(spec.params, width)
+    return _mixer_class(spec.mixer)(spec.params, width)
 
 
 @dataclass
@@ -319,26 +518,29 @@ class MixerLayer:
 
 
 class DenseMlp:
-    """down(act(up(h))), no gate."""
+    """down(act(up(h))), or gated: down(act(gate(h)) * up(h))."""
 
-    def __init__(self, ff: int, width: int):
-        self.ff, self.width, self.W = ff, width, pad16(width)
+    def __init__(self, ff: int, width: int, gated: bool):
+        self.ff, self.width, self.W, self.gated = ff, width, pad16(width), gated
         self.fp = pad16(ff)
+        self.names = ("gate", "up") if gated else ("up",)
 
     def shapes(self):
-        return {"up": (self.ff, self.width), "down": (self.width, self.ff)}
+        return dict({n: (self.ff, self.width) for n in self.names}, down=(self.width, self.ff))
 
     def load(self, get, fin, vec, model):
-        self.up, self.down = fin(_pad_to(get("up"), self.fp, self.W)), fin(_pad_to(get("down"), self.W, self.fp))
+        self.up = fin(torch.cat([_pad_to(get(n), self.fp, self.W) for n in self.names]))
+        self.down = fin(_pad_to(get("down"), self.W, self.fp))
 
     def run(self, model, h):
         """-> (rows, None): one row per token."""
         ops = model.ops
-        return ops.gemm(ops.act_mul(ops.gemm(h, self.up), self.fp, model.config.hidden_act, gated=False), self.down), None
+        return ops.gemm(ops.act_mul(ops.gemm(h, self.up), self.fp, model.config.hidden_act, gated=self.gated), self.down), None
 
 
 class MoeMlp:
-    """Routed experts down(act(up(h))) with sigmoid scores, a correction that takes part in the choice only, and groups of neighbours.
+    """Routed experts down(act(up(h))), or gated: down(silu(gate(h)) * up(h)), with the rows of gate and up taking turns in one matrix, so
+    that the product's epilogue has both.  How the experts are chosen and weighted is in the MoeSpec.
 
     The shared expert is cut into slices of an expert's (padded) width; every token takes each slice with the weight
     sigmoid(sg . h), so the slices ride in the grouped products as further experts, and `sg` is one more row of the router."""
@@ -347,47 +549,83 @@ class MoeMlp:
 
     def __init__(self, spec, width: int):
         self.spec, self.width, self.W = spec, width, pad16(width)
-        up = lambda n: (n + self.TILE - 1) // self.TILE * self.TILE
-        self.fp, self.Wp = up(spec.ff), up(self.W)
+        self.names = ("gate", "up") if spec.gated else ("up",)
+        up = lambda n, tile=self.TILE: (n + tile - 1) // tile * tile
+        self.fp, self.Wp = up(spec.ff, self.TILE // len(self.names)), up(self.W)
         self.slices = (spec.shared_ff + self.fp - 1) // self.fp
         if spec.experts > 256 or spec.top > 32 or self.slices > 32:      # tables of the routing kernels
             raise NotImplementedError(f"{spec.experts} experts, {spec.top} per token, a shared expert of {self.slices} expert widths")
+        if spec.score == "softmax" and (spec.group_top != 1 and spec.groups):
+            raise NotImplementedError("groups of softmax scores by more than their largest")
 
     def shapes(self):
         s, w = self.spec, self.width
-        out = {"router": (s.experts, w), "correction": (s.experts,)}
+        out = {"router": (s.experts, w)}
+        if s.score == "sigmoid":
+            out["correction"] = (s.experts,)
         for e in range(s.experts):
-            out.update({f"e{e}.up": (s.ff, w), f"e{e}.down": (w, s.ff)})
+            out.update({f"e{e}.{n}": (s.ff, w) for n in self.names})
+            out[f"e{e}.down"] = (w, s.ff)
         if s.shared_ff:
-            out.update({"shared.up": (s.shared_ff, w), "shared.down": (w, s.shared_ff), "shared.sg": (1, w)})
+            out.update({f"shared.{n}": (s.shared_ff, w) for n in self.names})
+            out.update({"shared.down": (w, s.shared_ff), "shared.sg": (1, w)})
         return out
 
     def load(self, get, fin, vec, model):
-        s, n = self.spec, self.spec.experts + self.slices
+        s, n, step = self.spec, self.spec.experts + self.slices, len(self.names)
+        if s.gated and model.config.hidden_act != "silu":
+            raise NotImplementedError(f"gated experts with {model.config.hidden_act}")
         new = lambda *shape: torch.zeros(*shape, dtype=model.dtype, device=model.device)
-        self.up, self.down = new(n, self.fp, self.W), new(n, self.Wp, self.fp)
+        self.up, self.down = new(n, step * self.fp, self.W), new(n, self.Wp, self.fp)
         for e in range(s.experts):
-            self.up[e, : s.ff, : self.width] = fin(get(f"e{e}.up"))
+            for i, name in enumerate(self.names):
+                self.up[e, i: step * s.ff: step, : self.width] = fin(get(f"e{e}.{name}"))
             self.down[e, : self.width, : s.ff] = fin(get(f"e{e}.down"))
         router = [get("router")]
         if s.shared_ff:
-            up, down = fin(get("shared.up")), fin(get("shared.down"))
+            ups, down = [fin(get("shared." + name)) for name in self.names], fin(get("shared.down"))
             for i in range(self.slices):
                 a, b = i * self.fp, min((i + 1) * self.fp, s.shared_ff)
-                self.up[s.experts + i, : b - a, : self.width] = up[a:b]
+                for j, up in enumerate(ups):
+                    self.up[s.experts + i, j: step * (b - a): step, : self.width] = up[a:b]
                 self.down[s.experts + i, : self.width, : b - a] = down[:, a:b]
             router.append(get("shared.sg"))
         self.router = fin(_pad_to(torch.cat(router), (s.experts + 8) // 8 * 8, self.W))      # (whole tiles of the router kernel)
-        self.correction = vec(get("correction"))
+        self.correction = vec(get("correction")) if s.score == "sigmoid" else None
 
     def run(self, model, h):
         """-> (rows of every (token, expert) pair, (row, weight) of each token's pairs)."""
         s, ops = self.spec, model.ops
-        r = ops.moe_route(h, self.router, s.top, 0, s.experts, experts=s.experts, score="sigmoid", correction=self.correction, groups=s.groups,
-                          keep=s.keep, scale=s.scale, shared=self.slices)
+        r = ops.moe_route(h, self.router, s.top, 0, s.experts, experts=s.experts, score=s.score, correction=self.correction, groups=s.groups,
+                          keep=s.keep, scale=s.scale, shared=self.slices, group_top=s.group_top, renorm=s.renorm)
         avg = max(1, (h.shape[0] * s.top + s.experts - 1) // s.experts)
-        a = ops.moe_grouped_gemm(r.xg, self.up, r.seg, avg, shared=self.slices, tokens=h.shape[0], act=model.config.hidden_act)
+        a = ops.moe_grouped_gemm(r.xg, self.up, r.seg, avg, shared=self.slices, tokens=h.shape[0],
+                                 act="swiglu" if s.gated else model.config.hidden_act)
         return ops.moe_grouped_gemm(a, self.down, r.seg, avg), (r.pos, r.topk_w)
+
+
+@dataclass
+class PreNormLayer:
+    """x += mixer(norm1(x)), then x += ff(norm2(x)).  The stream is fp32; what a sublayer adds (`pending`: rows, and with experts the
+    (row, weight) pairs of every token) is added by the norm that reads the stream next."""
+    mixer: Mixer
+    mlp: Optional[object]                                    # DenseMlp, MoeMlp or None
+    norm1: torch.Tensor = None                               # fp32 [W]
+    norm2: Optional[torch.Tensor] = None
+    in_w: Optional[torch.Tensor] = None                      # [rows, W]
+    in_b: Optional[torch.Tensor] = None                      # [rows]
+    out_w: Optional[torch.Tensor] = None                     # [W, mixer out_dim]
+    parts: Dict[str, Tuple[int, int]] = field(default_factory=dict)
+
+    def forward(self, model, residual, pending, inp, cache):
+        ops, m, c = model.ops, self.mixer, model.config
+        norm = lambda pending, w: ops.norm_stream(residual, pending[0], w, model.eps, c.norm_weight_offset, model.hidden, model.dtype, pairs=pending[1])
+        h = norm(pending, self.norm1)
+        proj = ops.gemm(h, self.in_w, bias=self.in_b)
+        y = torch.empty(h.shape[0], m.out_dim, dtype=h.dtype, device=h.device)
+        m.run(model, h, {n: proj[:, a:b] for n, (a, b) in self.parts.items()}, y, inp, cache)
+        pending = ops.gemm(y, self.out_w), None
+        return pending if self.mlp is None else self.mlp.run(model, norm(pending, self.norm2))
 
 
 @dataclass
@@ -420,7 +658,7 @@ class PostNormLayer:
 def make_mlp(spec, width: int):
     if spec.moe is not None:
         return MoeMlp(spec.moe, width)
-    return DenseMlp(spec.ff, width) if spec.ff else None
+    return DenseMlp(spec.ff, width, spec.gated) if spec.ff else None
 
 
 def _parts(layer, rows):
@@ -456,14 +694,19 @@ def load_mixer_layers(m, w):
     if c.norm_type == "layernorm":
         m.final_norm_b = vec(_pad_to(get("final.norm.b"), W))
     m.layers = []
-    if c.layer_style == "post":
-        norm = lambda name: (vec(_pad_to(get(name), W)), vec(_pad_to(get(name + ".b"), W)))
+    if c.layer_style in ("pre", "post"):
+        norm = lambda name: vec(_pad_to(get(name), W))
+        if c.layer_style == "post":
+            norm = lambda name: (vec(_pad_to(get(name), W)), vec(_pad_to(get(name + ".b"), W)))
         for i, spec in enumerate(c.layer_specs):
-            layer = PostNormLayer(make_mixer(spec, c.hidden_size), make_mlp(spec, c.hidden_size), norm(f"l{i}.norm1"))
+            kind = PreNormLayer if c.layer_style == "pre" else PostNormLayer
+            layer = kind(make_mixer(spec, c.hidden_size), make_mlp(spec, c.hidden_size), norm(f"l{i}.norm1"))
             sub = lambda name, i=i: get(f"l{i}.mix.{name}")
-            rows = layer.mixer.in_parts(sub)
+            rows, bias = layer.mixer.in_parts(sub), layer.mixer.in_bias(sub)
             _parts(layer, rows)
             layer.in_w, layer.out_w = fin(torch.cat([t for _, t in rows])), fin(layer.mixer.out_part(sub))
+            if bias:
+                layer.in_b = fin(torch.cat([bias[n] if n in bias else torch.zeros_like(t[:, 0]) for n, t in rows]))
             layer.mixer.load(sub, fin, vec, m)
             if layer.mlp is not None:
                 layer.norm2 = norm(f"l{i}.norm2")
@@ -491,12 +734,17 @@ def tensor_shapes(c) -> Dict[str, Tuple[int, ...]]:
     """Name -> shape of every tensor of a layer-by-layer checkpoint of this configuration."""
     w = c.hidden_size
     out = {"embed": (c.vocab_size, w), "head": (c.vocab_size, w), "final.norm": (w,)}
-    if c.layer_style == "post":
-        out.update({"pos": (c.max_position_embeddings, w), "final.norm.b": (w,)})
+    if c.layer_style in ("pre", "post"):
+        if c.learned_positions:
+            out["pos"] = (c.max_position_embeddings, w)
+        if c.norm_type == "layernorm":
+            out["final.norm.b"] = (w,)
         for i, spec in enumerate(c.layer_specs):
             mlp = make_mlp(spec, w)
             for norm in ("norm1",) + (("norm2",) if mlp is not None else ()):
-                out.update({f"l{i}.{norm}": (w,), f"l{i}.{norm}.b": (w,)})
+                out[f"l{i}.{norm}"] = (w,)
+                if c.norm_type == "layernorm":
+                    out[f"l{i}.{norm}.b"] = (w,)
             out.update({f"l{i}.mix.{n}": s for n, s in make_mixer(spec, w).shapes().items()})
             out.update({f"l{i}.mlp.{n}": s for n, s in (mlp.shapes() if mlp is not None else {}).items()})
         return out
@@ -537,6 +785,12 @@ class RandomWeights:
             return 0.1 * t
         if leaf == "correction":
             return 0.2 * t
-        if leaf == "u":
+        if leaf in ("u", "A_log"):
             return 0.5 * t
+        if leaf == "D":
+            return 1.0 + 0.1 * t
+        if leaf == "dt_bias":
+            return -1.5 + t
+        if leaf == "sink":
+            return t
         return t if name in ("embed", "pos") else t * shape[-1] ** -0.5

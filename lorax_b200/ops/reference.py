@@ -461,11 +461,22 @@ def rope_cache(rot: int, max_pos: int, theta: float, scaling: Optional[dict] = N
 # Layer-by-layer designs (models/mixers.py): fp32 residual stream, linear recurrences with per-request state, latent attention.
 # `inp` is the StepInputs of the step: rows [0, nd) are decode rows, the rows after them ragged prompt tokens.
 # ------------------------------------------------------------------------------------------------
-def rope_table(rot: int, max_pos: int, base: float, device="cpu") -> torch.Tensor:
-    """[max_pos, rot] fp32: cos of position * base^(-2i / rot) in the first half, sin in the second; angles formed in fp64."""
+def rope_table(rot: int, max_pos: int, base: float, device="cpu", scaling=None) -> torch.Tensor:
+    """[max_pos, rot] fp32: cos of position * base^(-2i / rot) in the first half, sin in the second; angles formed in fp64.  `scaling`
+    (factor, original, fast, slow): YaRN, which divides the frequencies of pairs that turn less than `slow` times over `original`
+    positions by `factor`, leaves those that turn more than `fast` times, goes linearly between, and multiplies cos and sin by
+    0.1 ln(factor) + 1."""
     f = torch.pow(torch.tensor(float(base), dtype=torch.float64), -torch.arange(0, rot, 2, dtype=torch.float64) / rot)
+    mult = 1.0
+    if scaling:
+        factor, original = float(scaling["factor"]), float(scaling["original"])
+        pair = lambda turns: rot * math.log(original / (2 * math.pi * turns)) / (2 * math.log(base))
+        lo, hi = max(math.floor(pair(scaling["fast"])), 0), min(math.ceil(pair(scaling["slow"])), rot - 1)
+        ramp = ((torch.arange(rot // 2, dtype=torch.float64) - lo) / max(hi - lo, 0.001)).clamp(0, 1)
+        f = f / factor * ramp + f * (1 - ramp)
+        mult = 0.1 * math.log(factor) + 1.0
     a = torch.outer(torch.arange(max_pos, dtype=torch.float64), f)
-    return torch.cat([a.cos(), a.sin()], -1).float().to(device)
+    return (torch.cat([a.cos(), a.sin()], -1) * mult).float().to(device)
 
 
 def embed_stream(ids, table, mult=1.0, pos=None, positions=None, copy=None):
@@ -485,15 +496,17 @@ def _layer_norm(x, weight, bias, eps, n: int):
     return y if bias is None else y + bias
 
 
+def _weighted_rows(y, pairs, W: int):
+    """Sum of every token's rows pos [T, k] (-1: none) of `y` with the weights w [T, k], in fp32."""
+    pos, w = pairs
+    return torch.einsum("tk,tkw->tw", torch.where(pos >= 0, w, torch.zeros_like(w)), y[pos.long().clamp(min=0)][:, :, :W].float())
+
+
 def norm_add(residual, y, weight, bias, mult: float, eps, n: int, dtype, layernorm: bool = True, pairs=None):
     """residual (fp32, in place) += mult * norm(y) over the first `n` columns; returns the new residual in `dtype`.  With `pairs` =
     (pos [T, k], w [T, k]) a token's y is the weighted sum of its rows pos (-1: none) of `y`."""
     W = residual.shape[1]
-    if pairs is None:
-        x = y[:, :W].float()
-    else:
-        pos, w = pairs
-        x = torch.einsum("tk,tkw->tw", torch.where(pos >= 0, w, torch.zeros_like(w)), y[pos.long().clamp(min=0)][:, :, :W].float())
+    x = y[:, :W].float() if pairs is None else _weighted_rows(y, pairs, W)
     if layernorm:
         x = _layer_norm(x, weight, bias, eps, n)
     else:
@@ -504,11 +517,12 @@ def norm_add(residual, y, weight, bias, mult: float, eps, n: int, dtype, layerno
     return residual if dtype == torch.float32 else residual.to(dtype)
 
 
-def norm_stream(residual, pending, weight, eps, weight_offset: float, n: int, dtype, bias=None, layernorm: bool = False, rows=None):
-    """residual (fp32, in place) += pending; returns its RMS or layer norm (mean over the first `n` columns) in `dtype`, of `rows` only
-    when given."""
+def norm_stream(residual, pending, weight, eps, weight_offset: float, n: int, dtype, bias=None, layernorm: bool = False, rows=None, pairs=None):
+    """residual (fp32, in place) += pending, with `pairs` a weighted sum of its rows as in `norm_add`; returns its RMS or layer norm (mean
+    over the first `n` columns) in `dtype`, of `rows` only when given (whether the residual's other rows still take the addition is
+    open: only the last norm of a pass takes `rows`)."""
     if pending is not None:
-        residual += pending.float()
+        residual += pending.float() if pairs is None else _weighted_rows(pending, pairs, residual.shape[1])
     if rows is not None:
         residual = residual[rows.long()]
     if layernorm:
@@ -677,6 +691,84 @@ def latent_attn(q_lat, q, cache, H: int, kv_rank: int, head: int, rot_off: int, 
     return out.view(T, H * kv_rank)
 
 
+def _conv_rows(x, w, state, inp):
+    """Depthwise causal convolution of the step's rows: y_t = sum_j w[j] * u_(t - taps + 1 + j), u the rows of the sequence, zeros in
+    front of it.  w [taps, C]; `state` [slots, taps - 1, C] holds the sequences' last rows and takes the new ones.  -> fp32 [T, C]"""
+    T, taps = x.shape[0], w.shape[0]
+    out = torch.zeros(T, x.shape[1], dtype=torch.float32, device=x.device)
+    for r0, n, slot, before in _sequences(inp, T):
+        u = x[r0: r0 + n]
+        if taps > 1:
+            old = state[slot] if before > 0 else torch.zeros_like(state[slot])
+            u = torch.cat([old, u])
+            state[slot] = u[u.shape[0] - (taps - 1):].clone()
+        for j in range(taps):
+            out[r0: r0 + n] += w[j] * u[j: j + n].float()
+    return out
+
+
+def causal_conv(x, w, b, act: str, state, inp):
+    """act(convolution + b) of x [T, C] in x's dtype, in memory of its own."""
+    y = _conv_rows(x, w, state, inp)
+    if b is not None:
+        y = y + b
+    return (_act(y, act) if act else y).to(x.dtype)
+
+
+def conv_rope_kvwrite(qkv, H: int, G: int, dk: int, dv: int, cos_sin, rot: int, positions, cache, inp, conv_w=None, conv_state=None):
+    """Rows [q (H heads) | k (G) | v (G)] of padded widths dk, dk, dv (G 0: queries only), through the convolution when there is one:
+    the first `rot` columns of every q and k head rotated in interleaved pairs, k and v to the cache.  -> q [T, H * dk], which without
+    convolution is the front of `qkv` itself."""
+    T = qkv.shape[0]
+    x = qkv[:, : (H + G) * dk + G * dv].float() if conv_w is None else _conv_rows(qkv, conv_w, conv_state, inp)
+    qk = x[:, : (H + G) * dk].reshape(T, H + G, dk).clone()
+    if rot:
+        cs = cos_sin[positions.long()]
+        qk[:, :, :rot] = _rotate_pairs(qk[:, :, :rot], cs[:, None, : rot // 2], cs[:, None, rot // 2:])
+    qk = qk.to(qkv.dtype)
+    if G:
+        page = cache.shape[2] // (dk + dv)
+        ok = inp.slots >= 0
+        s = inp.slots[ok].long()
+        blk, off = s // page, s % page
+        cache[:, :, : page * dk].view(cache.shape[0], G, page, dk)[blk, :, off] = qk[ok][:, H:]
+        cache[:, :, page * dk:].view(cache.shape[0], G, page, dv)[blk, :, off] = x[ok][:, (H + G) * dk:].reshape(-1, G, dv).to(qkv.dtype)
+    q = qk[:, :H].reshape(T, H * dk)
+    if conv_w is None:
+        qkv[:, : H * dk] = q
+        return qkv[:, : H * dk]
+    return q
+
+
+def ssd(xbc, dt, H: int, G: int, n: int, p: int, dt_bias, A, D, state, inp):
+    """Selective state space recurrence (Mamba-2) over rows [x (H heads of p) | B (G groups of n) | C (G)]: with s = softplus(dt + dt_bias)
+    per token and head, S <- exp(A s) S + s B x^T, y = S^T C + D x.  `state` [slots, H, n, p] fp32 is read and updated.
+    -> y [T, H * p] fp32"""
+    T = xbc.shape[0]
+    x = xbc[:, : H * p].float().reshape(T, H, p)
+    B, C = (xbc[:, H * p + i * G * n: H * p + (i + 1) * G * n].float().reshape(T, G, n).repeat_interleave(H // G, 1) for i in (0, 1))
+    s = F.softplus(dt[:, :H].float() + dt_bias)
+    out = torch.zeros(T, H * p, dtype=torch.float32, device=xbc.device)
+    for r0, rows, slot, before in _sequences(inp, T):
+        S = state[slot].clone() if before > 0 else torch.zeros_like(state[slot])
+        for t in range(r0, r0 + rows):
+            S = torch.exp(A * s[t])[:, None, None] * S + (s[t][:, None] * B[t])[:, :, None] * x[t][:, None, :]
+            out[t] = (torch.einsum("hnp,hn->hp", S, C[t]) + D[:, None] * x[t]).reshape(-1)
+        state[slot] = S
+    return out
+
+
+def gate_norm(y, z, H: int, p: int, parts: int, weight, eps, out):
+    """y [T, H * p padded] fp32 times silu(z) (the same layout), the heads' real columns closed up to [T, H * p], every one of `parts`
+    equal parts of a row divided by its root mean square, times `weight` [H * p]; columns of `out` behind them are zeroed."""
+    T, pp = y.shape[0], y.shape[1] // H
+    g = (y * F.silu(z[:, : H * pp].float())).view(T, H, pp)[:, :, :p].reshape(T, parts, -1)
+    g = (g * torch.rsqrt(g.square().mean(-1, keepdim=True) + eps)).reshape(T, H * p) * weight
+    out[:, : H * p] = g.to(out.dtype)
+    out[:, H * p:] = 0
+    return out
+
+
 def _kv_planes(cache, blocks, dk: int, dv: int, keys: int):
     """Pages of a sequence -> K [keys, heads, dk], V [keys, heads, dv] (fp32)."""
     page = cache.shape[2] // (dk + dv)
@@ -706,9 +798,11 @@ def qk_norm_kvwrite(qkv, H: int, G: int, dk: int, dv: int, n: int, q_norm, k_nor
     cache[:, :, page * dk:].view(cache.shape[0], G, page, dv)[blk, :, off] = v[ok]
 
 
-def gqa_attn(q, cache, H: int, G: int, dk: int, dv: int, scale: float, window: int, inp, out):
+def gqa_attn(q, cache, H: int, G: int, dk: int, dv: int, scale: float, window: int, inp, out, softcap: float = 0.0, sink=None, gate=None,
+             out_scale: float = 1.0):
     """Softmax attention of a step's rows (queries in the first H * dk columns of q) over the cached keys and values; a token sees the
-    last `window` tokens (0: all) including itself.  -> out [T, H * dv]"""
+    last `window` tokens (0: all) including itself.  softcap: scores become cap * tanh(score / cap).  sink [H]: a score that counts in
+    the denominator only.  The result is multiplied by `out_scale` and by sigmoid(gate) [T, H * dv].  -> out [T, H * dv]"""
     T = q.shape[0]
     page = cache.shape[2] // (dk + dv)
     nd, dbt, _, ctx = inp.decode_view(T)
@@ -725,8 +819,16 @@ def gqa_attn(q, cache, H: int, G: int, dk: int, dv: int, scale: float, window: i
         if window > 0:
             hidden |= kp <= pos - window
         qs = q[r0: r0 + n, : H * dk].reshape(n, G, H // G, dk).float()
-        s = (torch.einsum("tghd,sgd->ghts", qs, k) * scale).masked_fill(hidden, float("-inf"))
-        out[r0: r0 + n, : H * dv] = torch.einsum("ghts,sgd->tghd", torch.softmax(s, -1), v).reshape(n, H * dv).to(out.dtype)
+        s = torch.einsum("tghd,sgd->ghts", qs, k) * scale
+        if softcap > 0:
+            s = softcap * torch.tanh(s / softcap)
+        s = s.masked_fill(hidden, float("-inf"))
+        if sink is not None:
+            s = torch.cat([s, sink.view(G, H // G, 1, 1).expand(-1, -1, n, 1)], -1)
+        y = torch.einsum("ghts,sgd->tghd", torch.softmax(s, -1)[..., :keys], v).reshape(n, H * dv) * out_scale
+        if gate is not None:
+            y = y * torch.sigmoid(gate[r0: r0 + n, : H * dv].float())
+        out[r0: r0 + n, : H * dv] = y.to(out.dtype)
     return out
 
 
@@ -739,28 +841,25 @@ class MoeRouting(NamedTuple):
 
 
 def moe_route(x, router_w, k: int, e0: int, e_local: int, experts=None, score: str = "softmax", correction=None, groups: int = 0,
-              keep: int = 0, scale: float = 1.0, shared: int = 0) -> MoeRouting:
-    """Routing of every token to `k` of the router's first `experts` rows.  softmax: the largest logits, weights renormalised.
-    sigmoid: the largest sigmoid + correction within the best `keep` of `groups` groups (by the sum of a group's two largest), weights
-    are the sigmoids divided by their sum and times `scale`.  `shared` experts more take every token, with the weight
-    sigmoid(router row `experts`)."""
+              keep: int = 0, scale: float = 1.0, shared: int = 0, group_top: int = 2, renorm: bool = True) -> MoeRouting:
+    """Routing of every token to `k` of the router's first `experts` rows by its scores, softmax over all of them or sigmoid (plus a
+    correction that takes part in the choice only), within the best `keep` of `groups` groups (by the sum of a group's `group_top`
+    largest; softmax: 1).  The weights are the scores, divided by their sum if `renorm`, times `scale`.  `shared` experts more take every
+    token, with the weight sigmoid(router row `experts`)."""
     T, E = x.shape[0], experts or router_w.shape[0]
     z = x.float() @ router_w.float().t()
-    logits = z[:, :E]
-    if score == "softmax":
-        p, ids = torch.softmax(logits, -1).topk(k, -1)
-        w = p / p.sum(-1, keepdim=True)
-    else:
-        s = torch.sigmoid(logits)
-        choice = s if correction is None else s + correction
-        if groups:
-            g = choice.view(T, groups, E // groups)
-            best = g.topk(min(2, E // groups), -1).values.sum(-1).topk(keep, -1).indices
-            kept = torch.zeros(T, groups, dtype=torch.bool, device=x.device).scatter_(1, best, True)
-            choice = g.masked_fill(~kept[:, :, None], float("-inf")).reshape(T, E)
-        ids = choice.topk(k, -1).indices
-        w = s.gather(1, ids)
-        w = w / (w.sum(-1, keepdim=True) + 1e-20) * scale
+    s = torch.softmax(z[:, :E], -1) if score == "softmax" else torch.sigmoid(z[:, :E])
+    choice = s if correction is None else s + correction
+    if groups:
+        g = choice.view(T, groups, E // groups)
+        best = g.topk(min(group_top, E // groups), -1).values.sum(-1).topk(keep, -1).indices
+        kept = torch.zeros(T, groups, dtype=torch.bool, device=x.device).scatter_(1, best, True)
+        choice = g.masked_fill(~kept[:, :, None], float("-inf")).reshape(T, E)
+    ids = choice.topk(k, -1).indices
+    w = s.gather(1, ids)
+    if renorm:
+        w = w / (w.sum(-1, keepdim=True) + (0.0 if score == "softmax" else 1e-20))
+    w = w * scale
     local = ids - e0
     flat = torch.where((local >= 0) & (local < e_local), local, torch.full_like(local, e_local)).reshape(-1)
     order = torch.argsort(flat, stable=True)
@@ -781,12 +880,13 @@ def moe_route(x, router_w, k: int, e0: int, e_local: int, experts=None, score: s
 
 def moe_grouped_gemm(xg, w, seg, avg_rows: int, out=None, shared: int = 0, tokens: int = 0, act: str = ""):
     """out[q] = act(xg[q] @ w[e(q)]^T) for every sorted row q (e(q): the expert whose run [seg[e], seg[e + 1]) holds q).  The last
-    `shared` experts all read the one set of `tokens` rows that stands where the first of them begins."""
+    `shared` experts all read the one set of `tokens` rows that stands where the first of them begins.  act "swiglu": the rows of w are
+    gate and up in turn, and column i of the result is silu(column 2i) * column 2i + 1."""
     s = [int(v) for v in seg]
     n = len(s) - 1
-    y = torch.zeros(s[-1], w.shape[1], dtype=xg.dtype, device=xg.device)
+    y = torch.zeros(s[-1], w.shape[1] // (2 if act == "swiglu" else 1), dtype=xg.dtype, device=xg.device)
     for e in range(n):
         back = max(0, e - (n - shared)) * tokens if shared else 0
         z = xg[s[e] - back: s[e + 1] - back].float() @ w[e].float().t()
-        y[s[e]: s[e + 1]] = (_act(z, act) if act else z).to(xg.dtype)
+        y[s[e]: s[e + 1]] = (F.silu(z[:, 0::2]) * z[:, 1::2] if act == "swiglu" else _act(z, act) if act else z).to(xg.dtype)
     return y

@@ -75,28 +75,52 @@ class StateSlots:
 
 
 class LayeredCache:
-    """Cache of a model whose layer runs keep different things (`DecoderModel.cache_shapes`): a run's entry in `layers` is either a
-    paged tensor in the model's dtype, addressed by the requests' block tables ([num_blocks, page, width], or for attention layers with
-    head counts and sizes of their own [num_blocks, kv heads, page * (key width + value width)]: a page of one head is its key plane,
-    then its value plane), or a dict of state tensors [slots, ...], addressed by the requests' state slot."""
+    """Cache of a model whose layer runs keep different things (`DecoderModel.cache_shapes`).  A run's entry in `layers` is one of
+
+      a paged tensor in the model's dtype, addressed by the requests' block tables: [num_blocks, page, width], or for attention layers
+      with head counts and sizes of their own [num_blocks, kv heads, page * (key width + value width)] (a page of one head is its key
+      plane, then its value plane);
+      a dict of state tensors [slots, ...], addressed by the requests' state slot, with the pages under "kv" where there are both;
+      a dict of entries, one per mixer of a layer that has several;
+      the very entry of an earlier run whose keys and values it reads."""
 
     def __init__(self, shapes: List[dict], num_blocks: int, num_slots: int, dtype, device, page: int = PAGE_SIZE):
         self.page = page
         self.num_blocks = num_blocks
         self.layers: List[object] = []
-        for sh in shapes:
+
+        def make(sh):
+            if "share" in sh:
+                return self.layers[sh["share"]]
+            if "parts" in sh:
+                return {n: make(part) for n, part in sh["parts"].items()}
             if "paged" in sh:
-                self.layers.append(torch.zeros(num_blocks, page, sh["paged"], dtype=dtype, device=device))
-            elif "kv" in sh:
+                return torch.zeros(num_blocks, page, sh["paged"], dtype=dtype, device=device)
+            pages = None
+            if "kv" in sh:
                 heads, dk, dv = sh["kv"]
-                self.layers.append(torch.zeros(num_blocks, heads, page * (dk + dv), dtype=dtype, device=device))
-            else:
-                self.layers.append({n: torch.zeros(num_slots, *dims, dtype=dt, device=device) for n, (dims, dt) in sh["state"].items()})
-        self.state_slots = StateSlots(num_slots) if any("state" in sh for sh in shapes) else None
+                pages = torch.zeros(num_blocks, heads, page * (dk + dv), dtype=dtype, device=device)
+                if "state" not in sh:
+                    return pages
+            entry = {n: torch.zeros(num_slots, *dims, dtype=dt, device=device) for n, (dims, dt) in sh["state"].items()}
+            if pages is not None:
+                entry["kv"] = pages
+            return entry
+        for sh in shapes:
+            self.layers.append(make(sh))
+        self.state_slots = StateSlots(num_slots) if any("state" in sh for sh in _leaves(shapes)) else None
 
     @property
     def max_tokens(self) -> int:
         return (self.num_blocks - 1) * self.page
+
+
+def _leaves(shapes) -> List[dict]:
+    """The shapes that take memory of their own, those of mixers within a layer one by one."""
+    out = []
+    for sh in shapes:
+        out += _leaves(sh["parts"].values()) if "parts" in sh else [] if "share" in sh else [sh]
+    return out
 
 
 def num_state_slots(max_batch: int) -> int:
@@ -121,6 +145,7 @@ def cache_bytes(model, cfg, max_batch: int, page: int = PAGE_SIZE):
         return KVCache.bytes_per_block(model.config.num_hidden_layers, model.nkv, model.d, kv_dtype_of(model, cfg), page), 0
     size = lambda dt: torch.empty(0, dtype=dt).element_size()
     width = lambda sh: sh.get("paged", 0) + (sh["kv"][0] * (sh["kv"][1] + sh["kv"][2]) if "kv" in sh else 0)
+    shapes = _leaves(shapes)
     paged = sum(width(sh) for sh in shapes) * page * size(model.dtype)
     fixed = 0
     for sh in shapes:

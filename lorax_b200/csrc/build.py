@@ -66,7 +66,7 @@ def _run(cmd, verbose: bool, log_path: Path | None = None, quiet: bool = False) 
 
 # Sources a program needs that only ever runs one kind of model (`ops.native.use_subset`).
 SUBSETS = {"mixers": ("gemm_bf16", "moe", "elementwise", "stream", "recurrent", "latent_attn", "latent_prefill_tc", "latent_decode_tc", "linear_attn_tc",
-                      "wkv_tc", "gqa", "attn_prefill_tc")}
+                      "wkv_tc", "gqa", "attn_prefill_tc", "conv_rope")}
 
 
 def build_kernels(force: bool = False, verbose: bool = False, subset: str | None = None) -> Path:

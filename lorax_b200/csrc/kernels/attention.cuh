@@ -3,7 +3,7 @@
 
 #include <cuda_fp8.h>
 
-#include "common.cuh"
+#include "attn_tail.cuh"
 
 namespace lx {
 
@@ -131,6 +131,7 @@ LX_DEVICE void softmax_tile(float (&sacc)[NKEYS / 8][4], float (&oacc)[D / 8][4]
                             int lo0, int hi0, int lo1, int hi1, float scale, float softcap, int lane, float slope0 = 0.f,
                             float slope1 = 0.f) {
   float mx[2] = {-INFINITY, -INFINITY};
+  const float cap_k = softcap > 0.f ? 2.f * kLog2e / softcap : 0.f;
 #pragma unroll
   for (int nt = 0; nt < NKEYS / 8; ++nt) {
 #pragma unroll
@@ -138,7 +139,7 @@ LX_DEVICE void softmax_tile(float (&sacc)[NKEYS / 8][4], float (&oacc)[D / 8][4]
       const int key = key0 + nt * 8 + 2 * (lane & 3) + (q & 1);
       const int r = q >> 1;
       float s = sacc[nt][q] * scale;
-      if (softcap > 0.f) s = softcap * tanhf(s / softcap);
+      if (softcap > 0.f) s = softcap_score(s, softcap, cap_k);
       // ALiBi: the bias -slope * (query position - key position) differs from slope * key position by a per-row constant,
       // which the softmax does not see
       s += (r == 0 ? slope0 : slope1) * (float)key;
@@ -198,6 +199,7 @@ struct DecodeParams {
   int nsplit;
   const float* alibi;         // [nh] ALiBi slopes, or null
   float v_scale;              // fp8 cache: multiplies the output (the K scale is folded into `scale` by the host)
+  AttnTail tail;
 };
 
 // NW warps per CTA split the pages of a (row, KV head): four for long contexts; two, so that two CTAs fit an SM and one streams
@@ -340,11 +342,12 @@ __global__ void __launch_bounds__(32 * NW) attn_decode_kernel(const DecodeParams
       num += wgt * so[(w * 16 + g) * DV + d];
       den += wgt * sl[w * 16 + g];
     }
-    const float o = (den > 0.f ? num / den : 0.f) * (KV8 ? p.v_scale : 1.f);
     const int head = head0 + g;
-    if (p.nsplit == 1) {
-      p.out[(long long)t * p.ldo + (long long)head * DV + d] = __float2bfloat16(o);
+    if (p.nsplit == 1) {                         // (of several splits the sink joins where they are combined)
+      const float o = (den > 0.f ? num * attn_denominator(p.tail, head, M * kLog2e, den) : 0.f) * (KV8 ? p.v_scale : 1.f);
+      p.out[(long long)t * p.ldo + (long long)head * DV + d] = __float2bfloat16(attn_tail(p.tail, o, t, head * DV + d));
     } else {
+      const float o = (den > 0.f ? num / den : 0.f) * (KV8 ? p.v_scale : 1.f);
       const long long pi = ((long long)t * p.nh + head) * p.nsplit + split;
       p.part_o[pi * DV + d] = o;
       if (d == 0) p.part_lse[pi] = den > 0.f ? M + __logf(den) : -INFINITY;
@@ -354,21 +357,24 @@ __global__ void __launch_bounds__(32 * NW) attn_decode_kernel(const DecodeParams
 
 template <int D>
 __global__ void __launch_bounds__(D) attn_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_lse,
-                                                         __nv_bfloat16* __restrict__ out, long long ldo, int nh, int nsplit) {
+                                                         __nv_bfloat16* __restrict__ out, long long ldo, int nh, int nsplit,
+                                                         const AttnTail tail) {
   pdl_trigger();
   pdl_wait();      // every block waits, also those that return early below
   const int t = blockIdx.x, h = blockIdx.y, d = threadIdx.x;
   const long long base = ((long long)t * nh + h) * nsplit;
   float M = -INFINITY;
   for (int s = 0; s < nsplit; ++s) M = fmaxf(M, part_lse[base + s]);
-  float num = 0.f, den = 0.f;
+  const bool any = M > -INFINITY;
+  if (tail.sink != nullptr) M = fmaxf(M, tail.sink[h]);
+  float num = 0.f, den = tail.sink != nullptr ? __expf(tail.sink[h] - M) : 0.f;
   for (int s = 0; s < nsplit; ++s) {
     const float ls = part_lse[base + s];
     const float w = (ls == -INFINITY) ? 0.f : __expf(ls - M);
     num += w * part_o[(base + s) * D + d];
     den += w;
   }
-  out[(long long)t * ldo + (long long)h * D + d] = __float2bfloat16(den > 0.f ? num / den : 0.f);
+  out[(long long)t * ldo + (long long)h * D + d] = __float2bfloat16(any ? attn_tail(tail, num / den, t, h * D + d) : 0.f);
 }
 
 // ------------------------------------------------------------------------------------------------
@@ -391,6 +397,7 @@ struct PrefillParams {
   float scale, softcap;
   const float* alibi;         // [nh] ALiBi slopes, or null
   float v_scale;              // fp8 cache: multiplies the output
+  AttnTail tail;
 };
 
 template <int DK, int DV, bool KV8, bool WIDE = false>
@@ -501,14 +508,15 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(const PrefillParams p
     l[r] += __shfl_xor_sync(0xffffffffu, l[r], 2);
   }
   const float vs = KV8 ? p.v_scale : 1.f;
-  const float inv0 = l[0] > 0.f ? vs / l[0] : 0.f, inv1 = l[1] > 0.f ? vs / l[1] : 0.f;
+  const float inv0 = l[0] > 0.f ? vs * attn_denominator(p.tail, head, m[0] * kLog2e, l[0]) : 0.f;
+  const float inv1 = l[1] > 0.f ? vs * attn_denominator(p.tail, head, m[1] * kLog2e, l[1]) : 0.f;
 #pragma unroll
   for (int nd = 0; nd < DV / 8; ++nd) {
-    const int c = nd * 8 + 2 * (lane & 3);
+    const int c = nd * 8 + 2 * (lane & 3), col = head * DV + c;
     if (qr0 < qlen)
-      *reinterpret_cast<uint32_t*>(p.out + tok0 * p.ldo + (long long)head * DV + c) = pack_bf16x2(oacc[nd][0] * inv0, oacc[nd][1] * inv0);
+      *reinterpret_cast<uint32_t*>(p.out + tok0 * p.ldo + (long long)head * DV + c) = pack_bf16x2(attn_tail(p.tail, oacc[nd][0] * inv0, tok0, col), attn_tail(p.tail, oacc[nd][1] * inv0, tok0, col + 1));
     if (qr1 < qlen)
-      *reinterpret_cast<uint32_t*>(p.out + tok1 * p.ldo + (long long)head * DV + c) = pack_bf16x2(oacc[nd][2] * inv1, oacc[nd][3] * inv1);
+      *reinterpret_cast<uint32_t*>(p.out + tok1 * p.ldo + (long long)head * DV + c) = pack_bf16x2(attn_tail(p.tail, oacc[nd][2] * inv1, tok1, col), attn_tail(p.tail, oacc[nd][3] * inv1, tok1, col + 1));
   }
 }
 
@@ -535,7 +543,7 @@ static int launch_decode_nw(const DecodeParams& p, int T, cudaStream_t s) {
   launch_pdl(attn_decode_kernel<DK, DV, STAGES, KV8, NW, WIDE>, grid, dim3(32 * NW), (size_t)SMEM, s, p);
   if (p.nsplit > 1) {
     dim3 g2(T, p.nh);
-    launch_pdl(attn_combine_kernel<DV>, g2, dim3(DV), 0, s, p.part_o, p.part_lse, p.out, p.ldo, p.nh, p.nsplit);
+    launch_pdl(attn_combine_kernel<DV>, g2, dim3(DV), 0, s, p.part_o, p.part_lse, p.out, p.ldo, p.nh, p.nsplit, p.tail);
   }
   return -(int)cudaGetLastError();
 }

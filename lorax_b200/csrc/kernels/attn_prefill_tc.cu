@@ -22,7 +22,7 @@
 // flash-attn-2 varlen call of the reference (server/lorax_server/utils/flash_attn.py:180-201) and the mma.sync kernel in
 // attention.cu, which stays for head sizes and group sizes this one does not take (d != 128, odd heads per KV head).
 // Every wait is bounded and reports through the status word.
-#include "common.cuh"
+#include "attn_tail.cuh"
 
 namespace lx {
 
@@ -47,6 +47,7 @@ struct FaParams {
   float scale, softcap;
   const float* alibi;
   int* status;
+  AttnTail tail;
 };
 
 template <bool WIDE>
@@ -74,18 +75,22 @@ LX_DEVICE float fa_ex2(float x) {
   return y;
 }
 
-// One score: scale, optional tanh cap, optional ALiBi bias, in the log2 domain (the softmax uses exp2).
-LX_DEVICE float fa_score(float s, float scale_l2, float softcap, float scale, float slope_l2, int key) {
-  float t;
-  if (softcap > 0.f) t = softcap * tanhf(s * scale / softcap) * kFaLog2e;
-  else t = s * scale_l2;
-  return fmaf(slope_l2, (float)key, t);
-}
+// How a raw product becomes a score in the log2 domain (the softmax uses exp2): scaled; scaled and capped; also with an ALiBi bias.
+enum FaScores : int { kFaPlain = 0, kFaCap = 1, kFaBias = 2 };
+struct FaScore {
+  float scale_l2, cap_l2, cap_k, slope_l2;       // scale * log2(e), cap * log2(e) (0: none), 2 scale log2(e) / cap, slope * log2(e)
+  template <int MODE>
+  LX_DEVICE float of(float s, int key) const {
+    if (MODE == kFaPlain) return s * scale_l2;
+    if (MODE == kFaCap) return softcap_score(s, cap_l2, cap_k);
+    return fmaf(slope_l2, (float)key, cap_l2 > 0.f ? softcap_score(s, cap_l2, cap_k) : s * scale_l2);
+  }
+};
 
-// Maximum over the 128 scores of a row (log2 domain).  PLAIN: no cap, no bias, so max(s) * scale is the maximum; MASK: keys
-// outside [lo, hi) do not count.
-template <bool PLAIN, bool MASK>
-LX_DEVICE float fa_block_max(uint32_t ts, int kb0, int lo, int hi, float scale_l2, float softcap, float scale, float slope_l2) {
+// Maximum over the 128 scores of a row (log2 domain).  Without a bias the scores grow with the products (scale > 0), so the largest product
+// gives it; MASK: keys outside [lo, hi) do not count.
+template <int MODE, bool MASK>
+LX_DEVICE float fa_block_max(uint32_t ts, int kb0, int lo, int hi, const FaScore& sc) {
   float bm = -INFINITY;
 #pragma unroll 1
   for (int c = 0; c < kFaKeys; c += 32) {
@@ -94,22 +99,19 @@ LX_DEVICE float fa_block_max(uint32_t ts, int kb0, int lo, int hi, float scale_l
     tc_wait_ld();
 #pragma unroll
     for (int q = 0; q < 32; ++q) {
-      float t = PLAIN ? __uint_as_float(r[q]) : fa_score(__uint_as_float(r[q]), scale_l2, softcap, scale, slope_l2, kb0 + c + q);
-      if (MASK) {
-        const int key = kb0 + c + q;
-        t = (key >= lo && key < hi) ? t : -INFINITY;
-      }
+      const int key = kb0 + c + q;
+      float t = MODE == kFaBias ? sc.of<MODE>(__uint_as_float(r[q]), key) : __uint_as_float(r[q]);
+      if (MASK) t = (key >= lo && key < hi) ? t : -INFINITY;
       bm = fmaxf(bm, t);
     }
   }
-  return PLAIN ? bm * scale_l2 : bm;
+  return MODE == kFaBias || bm == -INFINITY ? bm : sc.of<MODE>(bm, 0);
 }
 
 // p = exp2(score - m_new) for the 128 keys of the block -> bf16, written as this row of the K-major, 128-byte-swizzled operand
 // tile (WIDE: the remainders as the same row of the tile behind it); returns the row sum.
-template <bool PLAIN, bool MASK, bool WIDE>
-LX_DEVICE float fa_block_probs(uint32_t ts, uint8_t* prow, int row, int kb0, int lo, int hi, float m_new, float scale_l2, float softcap,
-                               float scale, float slope_l2) {
+template <int MODE, bool MASK, bool WIDE>
+LX_DEVICE float fa_block_probs(uint32_t ts, uint8_t* prow, int row, int kb0, int lo, int hi, float m_new, const FaScore& sc) {
   float sum = 0.f;
   const float neg_m = (m_new == -INFINITY) ? 0.f : -m_new;
   const bool dead = (m_new == -INFINITY);
@@ -125,11 +127,9 @@ LX_DEVICE float fa_block_probs(uint32_t ts, uint8_t* prow, int row, int kb0, int
 #pragma unroll
       for (int u = 0; u < 2; ++u) {
         const float sraw = __uint_as_float(r[q + u]);
-        float e = PLAIN ? fa_ex2(fmaf(sraw, scale_l2, neg_m)) : fa_ex2(fa_score(sraw, scale_l2, softcap, scale, slope_l2, kb0 + c + q + u) + neg_m);
-        if (MASK) {
-          const int key = kb0 + c + q + u;
-          e = (key >= lo && key < hi && !dead) ? e : 0.f;
-        }
+        const int key = kb0 + c + q + u;
+        float e = MODE == kFaPlain ? fa_ex2(fmaf(sraw, sc.scale_l2, neg_m)) : fa_ex2(sc.of<MODE>(sraw, key) + neg_m);
+        if (MASK) e = (key >= lo && key < hi && !dead) ? e : 0.f;
         pv[u] = e;
       }
       sum += pv[0] + pv[1];
@@ -299,9 +299,12 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_
     const int hi_min = cache + q0 + 1;
     const int lo_max = (p.window > 0 && key_hi > p.window) ? key_hi - p.window : 0;
     const bool rows_all_valid = (q0 + kFaQ <= qlen);
-    const float scale_l2 = p.scale * kFaLog2e;
-    const float slope_l2 = p.alibi != nullptr ? p.alibi[head] * kFaLog2e : 0.f;
-    const bool plain = p.softcap <= 0.f && p.alibi == nullptr;       // scores are s * scale: the maximum can be taken before scaling
+    FaScore sc;
+    sc.scale_l2 = p.scale * kFaLog2e;
+    sc.cap_l2 = p.softcap > 0.f ? p.softcap * kFaLog2e : 0.f;
+    sc.cap_k = p.softcap > 0.f ? 2.f * sc.scale_l2 / p.softcap : 0.f;
+    sc.slope_l2 = p.alibi != nullptr ? p.alibi[head] * kFaLog2e : 0.f;
+    const int mode = p.alibi != nullptr ? kFaBias : p.softcap > 0.f ? kFaCap : kFaPlain;
     const uint32_t trow = tmem_base + ((uint32_t)(quad * 32) << 16);
     uint8_t* prow = sp + row * 128;
 
@@ -320,18 +323,20 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_
       const uint32_t ts = trow + (uint32_t)(st * 128);
       // pass 1: block maximum of this row (log2 domain)
       float bm;
-      if (plain) bm = need_mask ? fa_block_max<true, true>(ts, kb0, lo, hi, scale_l2, p.softcap, p.scale, slope_l2)
-                                : fa_block_max<true, false>(ts, kb0, lo, hi, scale_l2, p.softcap, p.scale, slope_l2);
-      else bm = fa_block_max<false, true>(ts, kb0, lo, hi, scale_l2, p.softcap, p.scale, slope_l2);
+      if (mode == kFaPlain) bm = need_mask ? fa_block_max<kFaPlain, true>(ts, kb0, lo, hi, sc) : fa_block_max<kFaPlain, false>(ts, kb0, lo, hi, sc);
+      else if (mode == kFaCap) bm = need_mask ? fa_block_max<kFaCap, true>(ts, kb0, lo, hi, sc) : fa_block_max<kFaCap, false>(ts, kb0, lo, hi, sc);
+      else bm = fa_block_max<kFaBias, true>(ts, kb0, lo, hi, sc);
       const float m_new = fmaxf(m, bm);
       const float alpha = (m_new == -INFINITY) ? 1.f : fa_ex2(m - m_new);
       // the P tile is free once the MMAs of the previous block have read it
       if (!mbar_wait(p_empty, (j & 1) ^ 1, abort_flag)) { report_status(p.status, kTimeoutTmemEmpty, tile); *abort_flag = 1; alive = false; break; }
       // pass 2: probabilities -> bf16 operand tile, row sum
       float sum;
-      if (plain) sum = need_mask ? fa_block_probs<true, true, WIDE>(ts, prow, row, kb0, lo, hi, m_new, scale_l2, p.softcap, p.scale, slope_l2)
-                                 : fa_block_probs<true, false, WIDE>(ts, prow, row, kb0, lo, hi, m_new, scale_l2, p.softcap, p.scale, slope_l2);
-      else sum = fa_block_probs<false, true, WIDE>(ts, prow, row, kb0, lo, hi, m_new, scale_l2, p.softcap, p.scale, slope_l2);
+      if (mode == kFaPlain) sum = need_mask ? fa_block_probs<kFaPlain, true, WIDE>(ts, prow, row, kb0, lo, hi, m_new, sc)
+                                            : fa_block_probs<kFaPlain, false, WIDE>(ts, prow, row, kb0, lo, hi, m_new, sc);
+      else if (mode == kFaCap) sum = need_mask ? fa_block_probs<kFaCap, true, WIDE>(ts, prow, row, kb0, lo, hi, m_new, sc)
+                                               : fa_block_probs<kFaCap, false, WIDE>(ts, prow, row, kb0, lo, hi, m_new, sc);
+      else sum = fa_block_probs<kFaBias, true, WIDE>(ts, prow, row, kb0, lo, hi, m_new, sc);
       tc_fence_before();
       mbar_arrive(&s_empty[st]);
       fence_proxy_async_smem();
@@ -365,7 +370,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_
       const int ps = (nblk - 1) & 1;
       if (mbar_wait(&pv_full[ps], ((nblk - 1) >> 1) & 1, abort_flag)) {
         tc_fence_after();
-        const float inv = l > 0.f ? 1.f / l : 0.f;
+        const float inv = l > 0.f ? attn_denominator(p.tail, head, m, l) * p.tail.scale : 0.f;
+        const __nv_bfloat16* grow = p.tail.gate != nullptr ? p.tail.gate + (long long)(tok_base + qi) * p.tail.ldg + (long long)head * kFaD : nullptr;
         __nv_bfloat16* orow = p.out + (long long)(tok_base + qi) * p.ldo + (long long)head * kFaD;
 #pragma unroll
         for (int c = 0; c < kFaD; c += 32) {
@@ -376,9 +382,21 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_
 #pragma unroll
             for (int q = 0; q < 32; q += 8) {
               uint32_t w[4];
+              float v[8];
 #pragma unroll
-              for (int u = 0; u < 4; ++u)
-                w[u] = pack_bf16x2((o[c + q + 2 * u] + __uint_as_float(r[q + 2 * u])) * inv, (o[c + q + 2 * u + 1] + __uint_as_float(r[q + 2 * u + 1])) * inv);
+              for (int u = 0; u < 8; ++u) v[u] = (o[c + q + u] + __uint_as_float(r[q + u])) * inv;
+              if (grow != nullptr) {
+                const uint4 g = *reinterpret_cast<const uint4*>(grow + c + q);
+                const uint32_t gw[4] = {g.x, g.y, g.z, g.w};
+#pragma unroll
+                for (int u = 0; u < 4; ++u) {
+                  const float2 z = unpack_bf16x2(gw[u]);
+                  v[2 * u] = __fdividef(v[2 * u], 1.f + __expf(-z.x));
+                  v[2 * u + 1] = __fdividef(v[2 * u + 1], 1.f + __expf(-z.y));
+                }
+              }
+#pragma unroll
+              for (int u = 0; u < 4; ++u) w[u] = pack_bf16x2(v[2 * u], v[2 * u + 1]);
               *reinterpret_cast<uint4*>(orow + c + q) = make_uint4(w[0], w[1], w[2], w[3]);
             }
           }
@@ -421,23 +439,11 @@ static int launch_fa(const CUtensorMap& tq, const CUtensorMap& tkv, const FaPara
   return -(int)cudaGetLastError();
 }
 
-}  // namespace lx
-
-extern "C" {
-
-// 1: the tensor-core kernel takes this shape (d = 128, an even number of query heads per KV head, 16-byte aligned strides).
-int lx_attn_prefill_tc_supported(int nh, int nkv, int d, long long ldq, long long ldo) {
-  return (d == 128 && nkv > 0 && nh % nkv == 0 && ((nh / nkv) % 2) == 0 && ldq % 8 == 0 && ldo % 8 == 0) ? 1 : 0;
-}
-
-// Same contract as lx_attn_prefill_alibi (64-query tiles listed by tile_seq / tile_q0), plus the number of tokens `T` of the q
-// buffer and the number of blocks of the cache (bounds of the two tensor maps) and the status word.  wide: fp32 softmax weights.
-int lx_attn_prefill_tc(const void* q, long long ldq, int T, const void* kv, int num_blocks, const int* block_tables, int max_blocks,
-                       const int* cu_q, const int* cache_lens, const int* tile_seq, const int* tile_q0, int num_tiles, void* out, long long ldo,
-                       int nh, int nkv, int d, int window, float scale, float softcap, const float* alibi, int wide, int* status, void* stream) {
-  using namespace lx;
+static int attn_prefill_tc(const void* q, long long ldq, int T, const void* kv, int num_blocks, const int* block_tables, int max_blocks,
+                           const int* cu_q, const int* cache_lens, const int* tile_seq, const int* tile_q0, int num_tiles, void* out,
+                           long long ldo, int nh, int nkv, int window, float scale, float softcap, const float* alibi, int wide,
+                           const AttnTail& tail, int* status, void* stream) {
   if (num_tiles <= 0) return 0;
-  if (!lx_attn_prefill_tc_supported(nh, nkv, d, ldq, ldo)) return -1;
   FaEncodeFn fn = fa_encode_fn();
   if (fn == nullptr) return -2;
   CUtensorMap tq, tkv;
@@ -464,9 +470,39 @@ int lx_attn_prefill_tc(const void* q, long long ldq, int T, const void* kv, int 
   p.block_tables = block_tables; p.max_blocks = max_blocks; p.cu_q = cu_q; p.cache_lens = cache_lens;
   p.tile_seq = tile_seq; p.tile_q0 = tile_q0;
   p.out = reinterpret_cast<__nv_bfloat16*>(out); p.ldo = ldo;
-  p.nh = nh; p.nkv = nkv; p.group = nh / nkv; p.window = window; p.scale = scale; p.softcap = softcap; p.alibi = alibi; p.status = status;
+  p.nh = nh; p.nkv = nkv; p.group = nh / nkv; p.window = window; p.scale = scale; p.softcap = softcap; p.alibi = alibi; p.status = status; p.tail = tail;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   return wide ? launch_fa<true>(tq, tkv, p, num_tiles, st) : launch_fa<false>(tq, tkv, p, num_tiles, st);
+}
+
+}  // namespace lx
+
+extern "C" {
+
+// 1: the tensor-core kernel takes this shape (d = 128, an even number of query heads per KV head, 16-byte aligned strides).
+int lx_attn_prefill_tc_supported(int nh, int nkv, int d, long long ldq, long long ldo) {
+  return (d == 128 && nkv > 0 && nh % nkv == 0 && ((nh / nkv) % 2) == 0 && ldq % 8 == 0 && ldo % 8 == 0) ? 1 : 0;
+}
+
+// Same contract as lx_attn_prefill_alibi (64-query tiles listed by tile_seq / tile_q0), plus the number of tokens `T` of the q
+// buffer and the number of blocks of the cache (bounds of the two tensor maps) and the status word.  wide: fp32 softmax weights.
+int lx_attn_prefill_tc(const void* q, long long ldq, int T, const void* kv, int num_blocks, const int* block_tables, int max_blocks,
+                       const int* cu_q, const int* cache_lens, const int* tile_seq, const int* tile_q0, int num_tiles, void* out, long long ldo,
+                       int nh, int nkv, int d, int window, float scale, float softcap, const float* alibi, int wide, int* status, void* stream) {
+  if (!lx_attn_prefill_tc_supported(nh, nkv, d, ldq, ldo)) return -1;
+  return lx::attn_prefill_tc(q, ldq, T, kv, num_blocks, block_tables, max_blocks, cu_q, cache_lens, tile_seq, tile_q0, num_tiles, out, ldo, nh, nkv,
+                             window, scale, softcap, alibi, wide, lx::AttnTail{}, status, stream);
+}
+
+// The same with fp32 softmax weights, a sink per head, a gate [T, ldg] and a factor on the output (gqa.cu has the contract).
+int lx_gqa_prefill_tc(const void* q, long long ldq, int T, const void* kv, int num_blocks, const int* block_tables, int max_blocks,
+                      const int* cu_q, const int* cache_lens, const int* tile_seq, const int* tile_q0, int num_tiles, void* out, long long ldo,
+                      int nh, int nkv, int d, int window, float scale, float softcap, const float* sink, const void* gate, long long ldg,
+                      float out_scale, int* status, void* stream) {
+  if (!lx_attn_prefill_tc_supported(nh, nkv, d, ldq, ldo) || (gate != nullptr && ldg % 8 != 0)) return -1;
+  return lx::attn_prefill_tc(q, ldq, T, kv, num_blocks, block_tables, max_blocks, cu_q, cache_lens, tile_seq, tile_q0, num_tiles, out, ldo, nh, nkv,
+                             window, scale, softcap, nullptr, 1, lx::AttnTail{sink, reinterpret_cast<const __nv_bfloat16*>(gate), ldg, out_scale},
+                             status, stream);
 }
 
 }  // extern "C"

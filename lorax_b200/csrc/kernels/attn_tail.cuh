@@ -1,0 +1,39 @@
+// What the attention kernels share around the softmax: capped scores, sinks, and the last step of an output element.
+#pragma once
+
+#include "common.cuh"
+
+namespace lx {
+
+// cap * tanh(s / cap) by tanh(x) = 1 - 2 / (exp(2x) + 1); k = 2 log2(e) / cap.  The absolute error is a few 2^-24 of the cap.
+LX_DEVICE float softcap_score(float s, float cap, float k) {
+  float e, r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(s * k));
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(e + 1.f));
+  return fmaf(-2.f * cap, r, cap);
+}
+
+// What may follow the softmax: a sink per head, a score that only the denominator contains; a factor; a gate, sigmoid(gate[t, column]).
+struct AttnTail {
+  const float* sink = nullptr;            // [nh]
+  const __nv_bfloat16* gate = nullptr;    // [T, ldg]
+  long long ldg = 0;
+  float scale = 1.f;                      // of the output
+};
+
+// 1 / denominator of a row whose weights were formed with the maximum m and sum to l > 0 (both in the log2 domain): the sink joins, and
+// the maximum moves up to it when it is the larger one.
+LX_DEVICE float attn_denominator(const AttnTail& tail, int head, float m, float l) {
+  if (tail.sink == nullptr) return 1.f / l;
+  const float sink = tail.sink[head] * 1.4426950408889634f, top = fmaxf(m, sink), keep = exp2f(m - top);
+  return keep / (l * keep + exp2f(sink - top));
+}
+
+// One finished output element.
+LX_DEVICE float attn_tail(const AttnTail& tail, float o, long long t, int col) {
+  o *= tail.scale;
+  if (tail.gate != nullptr) o = __fdividef(o, 1.f + __expf(-__bfloat162float(tail.gate[t * tail.ldg + col])));
+  return o;
+}
+
+}  // namespace lx

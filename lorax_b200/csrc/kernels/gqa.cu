@@ -77,7 +77,10 @@ struct GqaF32Params {
   long long ldo;
   StepRows rows;
   int T, H, G, DK, DV, page, window;
-  float scale;
+  float scale, softcap, out_scale;
+  const float* sink;            // [H] or null
+  const float* gate;            // [T, ldg] or null
+  long long ldg;
 };
 
 __global__ void __launch_bounds__(32 * kGqaWarps) gqa_attn_f32_kernel(const GqaF32Params p) {
@@ -117,6 +120,7 @@ __global__ void __launch_bounds__(32 * kGqaWarps) gqa_attn_f32_kernel(const GqaF
         acc = fmaf(a.x, b.x, acc); acc = fmaf(a.y, b.y, acc); acc = fmaf(a.z, b.z, acc); acc = fmaf(a.w, b.w, acc);
       }
       s = acc * p.scale;
+      if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
       base += p.page * p.DK + (key % p.page) * p.DV;
     }
     const float mn = fmaxf(m, warp_max(s));
@@ -134,10 +138,19 @@ __global__ void __launch_bounds__(32 * kGqaWarps) gqa_attn_f32_kernel(const GqaF
         if (i * 32 < p.DV) o[i] = fmaf(wj, vr[i * 32 + lane], o[i]);
     }
   }
-  const float inv = l > 0.f ? 1.f / l : 0.f;
+  float inv = 0.f;
+  if (l > 0.f) {
+    const float sink = p.sink != nullptr ? p.sink[h] : -INFINITY, top = fmaxf(m, sink), keep = expf(m - top);
+    inv = keep / (l * keep + expf(sink - top)) * p.out_scale;
+  }
 #pragma unroll
-  for (int i = 0; i < kGqaMaxWidth / 32; ++i)
-    if (i * 32 < p.DV) p.out[(long long)t * p.ldo + (long long)h * p.DV + i * 32 + lane] = o[i] * inv;
+  for (int i = 0; i < kGqaMaxWidth / 32; ++i) {
+    if (i * 32 >= p.DV) continue;
+    const int col = h * p.DV + i * 32 + lane;
+    float y = o[i] * inv;
+    if (p.gate != nullptr) y *= sigmoid_f(p.gate[(long long)t * p.ldg + col]);
+    p.out[(long long)t * p.ldo + col] = y;
+  }
 }
 
 template <int DK, int DV>
@@ -188,10 +201,13 @@ int lx_qk_norm_kvwrite(const void* params, int f32, void* stream) {
   return -(int)cudaGetLastError();
 }
 
+// softcap > 0: scores become softcap * tanh(score / softcap).  sink [nh] (or null): a score that only the denominator contains.  The outputs
+// are multiplied by out_scale and by sigmoid(gate[t, column]) (gate [T, ldg] or null).
+//
 // Decode rows (bf16).  part_o / part_lse: T * nh * nsplit * dv and T * nh * nsplit floats, touched when nsplit > 1.
 int lx_gqa_decode(const void* q, long long ldq, const void* cache, const int* block_tables, int max_blocks, const int* ctx_lens, void* out,
                   long long ldo, float* part_o, float* part_lse, int T, int nh, int nkv, int dk, int dv, int window, float scale, int nsplit,
-                  void* stream) {
+                  float softcap, const float* sink, const void* gate, long long ldg, float out_scale, void* stream) {
   using namespace lx;
   if (T <= 0) return 0;
   if (nkv <= 0 || nh % nkv != 0 || ldq % 2 != 0) return -1;
@@ -202,7 +218,8 @@ int lx_gqa_decode(const void* q, long long ldq, const void* cache, const int* bl
   p.out = reinterpret_cast<__nv_bfloat16*>(out); p.ldo = ldo;
   p.part_o = part_o; p.part_lse = part_lse;
   p.nh = nh; p.nkv = nkv; p.group = nh / nkv; p.gchunks = (p.group + 15) / 16;
-  p.window = window; p.scale = scale; p.softcap = 0.f; p.v_scale = 1.f;
+  p.window = window; p.scale = scale; p.softcap = softcap; p.v_scale = 1.f;
+  p.tail = AttnTail{sink, reinterpret_cast<const __nv_bfloat16*>(gate), ldg, out_scale};
   p.nsplit = nsplit < 1 ? 1 : nsplit;
   if (p.nsplit > 1 && (part_o == nullptr || part_lse == nullptr)) return -2;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
@@ -214,7 +231,8 @@ int lx_gqa_decode(const void* q, long long ldq, const void* cache, const int* bl
 // Prompt rows (bf16): 64-query tiles listed by tile_seq / tile_q0.
 int lx_gqa_prefill(const void* q, long long ldq, const void* cache, const int* block_tables, int max_blocks, const int* cu_q,
                    const int* cache_lens, const int* tile_seq, const int* tile_q0, int num_tiles, void* out, long long ldo, int nh, int nkv,
-                   int dk, int dv, int window, float scale, void* stream) {
+                   int dk, int dv, int window, float scale, float softcap, const float* sink, const void* gate, long long ldg, float out_scale,
+                   void* stream) {
   using namespace lx;
   if (num_tiles <= 0) return 0;
   if (nkv <= 0 || nh % nkv != 0 || ldq % 2 != 0 || ldo % 2 != 0) return -1;
@@ -224,7 +242,8 @@ int lx_gqa_prefill(const void* q, long long ldq, const void* cache, const int* b
   p.block_tables = block_tables; p.max_blocks = max_blocks; p.cu_q = cu_q; p.cache_lens = cache_lens;
   p.tile_seq = tile_seq; p.tile_q0 = tile_q0;
   p.out = reinterpret_cast<__nv_bfloat16*>(out); p.ldo = ldo;
-  p.nh = nh; p.nkv = nkv; p.window = window; p.scale = scale; p.softcap = 0.f; p.v_scale = 1.f;
+  p.nh = nh; p.nkv = nkv; p.window = window; p.scale = scale; p.softcap = softcap; p.v_scale = 1.f;
+  p.tail = AttnTail{sink, reinterpret_cast<const __nv_bfloat16*>(gate), ldg, out_scale};
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
 #define LX_CALL(DK, DV) launch_prefill<DK, DV, false, true>(p, num_tiles, s)
   LX_GQA_DISPATCH(LX_CALL)

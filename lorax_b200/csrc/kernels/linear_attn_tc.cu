@@ -8,6 +8,10 @@
 // split into two bf16 terms, value and remainder, and multiplied as two operands; q, k and v arrive as bf16 with their silu applied
 // (silu_cols_kernel: they are read by two passes and two column halves).
 // STATES: the segment's own contribution to the state only (each group of four warps takes half of the columns).
+//
+// SSD (Mamba-2): q, k, v are C, B, x, which hpg heads share for C and B; a token has a step size s = softplus(z + w0) and the decay
+// exp(A s).  With the running sum L of A s within a chunk, c^(i+1) becomes exp(L_i), c^(i-j) becomes exp(L_i - L_j) s_j, c^(n-1-j) becomes
+// exp(L_(n-1) - L_j) s_j (no exponent is positive), and D x is added to the outputs.
 #include "stream.cuh"
 
 namespace lx {
@@ -22,7 +26,11 @@ struct LinTcParams {
   int H, dv;
   StepRows rows;
   const int* seg_seq; const int* seg_q0;
-  int seg_len;
+  int seg_len, hpg;
+  const __nv_bfloat16* z;  // SSD: [T, ldz], head h at column h
+  long long ldz;
+  const float* w0; const float* A; const float* skip;      // [H]
+  float* seg_decay;        // [nseg, H]
 };
 
 constexpr int kLtC = 64;                        // tokens per chunk
@@ -77,10 +85,10 @@ struct LtSmem {
   static constexpr int kK = kLtC * (D + 8) * 2;
   static constexpr int kV = kLtC * kLtVLd * 2;
   static constexpr int kS = STATES ? 0 : 2 * D * kLtVLd * 2;
-  static constexpr int kTotal = kQ + kK + kV + kS + (kLtC + 1) * 4 + 16;
+  static constexpr int kTotal = kQ + kK + kV + kS + 2 * (kLtC + 1) * 4 + 16;
 };
 
-template <int D, bool STATES>
+template <int D, bool STATES, bool SSD>
 __global__ void __launch_bounds__(kLtThreads, 2) linear_attn_tc_kernel(const LinTcParams p) {
   pdl_trigger();
   pdl_wait();
@@ -91,7 +99,8 @@ __global__ void __launch_bounds__(kLtThreads, 2) linear_attn_tc_kernel(const Lin
   __nv_bfloat16* sk = reinterpret_cast<__nv_bfloat16*>(lt_sm + M::kQ);
   __nv_bfloat16* sv = reinterpret_cast<__nv_bfloat16*>(lt_sm + M::kQ + M::kK);
   __nv_bfloat16* ss = reinterpret_cast<__nv_bfloat16*>(lt_sm + M::kQ + M::kK + M::kV);      // [2 terms][D][kLtVLd]
-  float* pw = reinterpret_cast<float*>(lt_sm + M::kQ + M::kK + M::kV + M::kS);             // decay^e, e = 0 .. 64
+  float* pw = reinterpret_cast<float*>(lt_sm + M::kQ + M::kK + M::kV + M::kS);             // decay^e, e = 0 .. 64; SSD: L of the chunk
+  float* sz = pw + kLtC + 1;                                                              // SSD: step sizes (zero behind the last token)
   const int seg = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * kLtV;
   const int b = p.seg_seq[seg], q0 = p.seg_q0[seg];
   const int r0 = p.rows.cu_q[b], qlen = p.rows.cu_q[b + 1] - r0;
@@ -102,8 +111,12 @@ __global__ void __launch_bounds__(kLtThreads, 2) linear_attn_tc_kernel(const Lin
   const bool for_state = STATES || group == 1;
   constexpr int NS = STATES ? 4 : 8;             // 8-wide column tiles of a state warp
   const int cs = STATES ? group * 32 : 0;        // its first column
-  const float lam = p.decay[h];
-  for (int e = threadIdx.x; e <= kLtC; e += kLtThreads) pw[e] = powf(lam, (float)e);
+  const int hk = SSD ? h / p.hpg : h;
+  if (!SSD) {
+    const float lam = p.decay[h];
+    for (int e = threadIdx.x; e <= kLtC; e += kLtThreads) pw[e] = powf(lam, (float)e);
+  }
+  float total = 0.f;                             // SSD: sum of L over the chunks so far
 
   // state warps: rows warp * D / 4 + m * 16 + lane / 4 (+ 8), columns c0 + cs + nt * 8 + 2 (lane % 4)
   float S[MT][NS][4];
@@ -134,10 +147,28 @@ __global__ void __launch_bounds__(kLtThreads, 2) linear_attn_tc_kernel(const Lin
   for (int t0 = 0; t0 < n; t0 += kLtC) {
     const int m_tok = min(kLtC, n - t0);
     __syncthreads();
-    if (!STATES) lt_fetch<D>(sq, p.q + (tok0 + t0) * p.ldq + h * D, p.ldq, m_tok);
-    lt_fetch<D>(sk, p.k + (tok0 + t0) * p.ldk + h * D, p.ldk, m_tok);
+    if (!STATES) lt_fetch<D>(sq, p.q + (tok0 + t0) * p.ldq + hk * D, p.ldq, m_tok);
+    lt_fetch<D>(sk, p.k + (tok0 + t0) * p.ldk + hk * D, p.ldk, m_tok);
     lt_fetch<kLtV>(sv, p.v + (tok0 + t0) * p.ldv + h * p.dv + c0, p.ldv, m_tok);
     cp_async_commit();
+    if (SSD && threadIdx.x < 32) {                 // the first warp, two tokens per lane
+      float a[2];
+#pragma unroll
+      for (int u = 0; u < 2; ++u) {
+        const int j = 2 * lane + u;
+        const float size = j < m_tok ? softplus_f(__bfloat162float(p.z[(tok0 + t0 + j) * p.ldz + h]) + p.w0[h]) : 0.f;
+        sz[j] = size;
+        a[u] = p.A[h] * size;
+      }
+      float sum = a[0] + a[1];
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const float up = __shfl_up_sync(0xffffffffu, sum, o);
+        if (lane >= o) sum += up;
+      }
+      pw[2 * lane] = sum - a[1];
+      pw[2 * lane + 1] = sum;
+    }
     if (!STATES && for_state) {
 #pragma unroll
       for (int m = 0; m < MT; ++m)
@@ -183,7 +214,9 @@ __global__ void __launch_bounds__(kLtThreads, 2) linear_attn_tc_kernel(const Lin
         }
       }
       const int i0 = warp * 16 + (lane >> 2), i1 = i0 + 8;
-      const float f0 = pw[i0 + 1], f1 = pw[i1 + 1];
+      const float f0 = SSD ? __expf(pw[i0]) : pw[i0 + 1], f1 = SSD ? __expf(pw[i1]) : pw[i1 + 1];
+      // weight of key j for the query row i, j <= i
+      auto weight = [&](int i, int j) { return SSD ? __expf(pw[i] - pw[j]) * sz[j] : pw[i - j]; };
 #pragma unroll
       for (int nt = 0; nt < 8; ++nt) { o[nt][0] *= f0; o[nt][1] *= f0; o[nt][2] *= f1; o[nt][3] *= f1; }
 #pragma unroll
@@ -194,8 +227,8 @@ __global__ void __launch_bounds__(kLtThreads, 2) linear_attn_tc_kernel(const Lin
         for (int u = 0; u < 2; ++u) {
           const int j = kk * 16 + u * 8 + (lane & 3) * 2;
           const float* x = s[2 * kk + u];
-          lt_split(j <= i0 ? x[0] * pw[i0 - j] : 0.f, j + 1 <= i0 ? x[1] * pw[i0 - j - 1] : 0.f, ph[2 * u], pl[2 * u]);
-          lt_split(j <= i1 ? x[2] * pw[i1 - j] : 0.f, j + 1 <= i1 ? x[3] * pw[i1 - j - 1] : 0.f, ph[2 * u + 1], pl[2 * u + 1]);
+          lt_split(j <= i0 ? x[0] * weight(i0, j) : 0.f, j + 1 <= i0 ? x[1] * weight(i0, j + 1) : 0.f, ph[2 * u], pl[2 * u]);
+          lt_split(j <= i1 ? x[2] * weight(i1, j) : 0.f, j + 1 <= i1 ? x[3] * weight(i1, j + 1) : 0.f, ph[2 * u + 1], pl[2 * u + 1]);
         }
 #pragma unroll
         for (int n2 = 0; n2 < 4; ++n2) {
@@ -209,6 +242,17 @@ __global__ void __launch_bounds__(kLtThreads, 2) linear_attn_tc_kernel(const Lin
       }
       const long long ldo = (long long)p.H * p.dv;
       float* orow = p.out + (tok0 + t0 + i0) * ldo + (long long)h * p.dv + c0 + cs + (lane & 3) * 2;
+      if constexpr (SSD) {
+        const float skip = p.skip[h];
+        const __nv_bfloat16* x0 = sv + i0 * kLtVLd + (lane & 3) * 2;
+#pragma unroll
+        for (int nt = 0; nt < 8; ++nt) {
+          const float2 a = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(x0 + nt * 8));
+          const float2 b = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(x0 + 8 * kLtVLd + nt * 8));
+          o[nt][0] = fmaf(skip, a.x, o[nt][0]); o[nt][1] = fmaf(skip, a.y, o[nt][1]);
+          o[nt][2] = fmaf(skip, b.x, o[nt][2]); o[nt][3] = fmaf(skip, b.y, o[nt][3]);
+        }
+      }
 #pragma unroll
       for (int nt = 0; nt < 8; ++nt) {
         if (i0 < m_tok) *reinterpret_cast<float2*>(orow + nt * 8) = make_float2(o[nt][0], o[nt][1]);
@@ -217,7 +261,8 @@ __global__ void __launch_bounds__(kLtThreads, 2) linear_attn_tc_kernel(const Lin
     }
     if (!for_state) continue;
     // ---- state
-    const float fs = pw[m_tok];
+    const float fs = SSD ? __expf(pw[kLtC - 1]) : pw[m_tok];
+    if (SSD) total += pw[kLtC - 1];
 #pragma unroll
     for (int m = 0; m < MT; ++m)
 #pragma unroll
@@ -227,7 +272,8 @@ __global__ void __launch_bounds__(kLtThreads, 2) linear_attn_tc_kernel(const Lin
       uint32_t kh[MT][4], kl[MT][4];
       const int j = kk * 16 + (lane & 3) * 2;
       // (rows behind the chunk's last token are zero: their factor only has to exist)
-      const float g0 = pw[max(m_tok - 1 - j, 0)], g1 = pw[max(m_tok - 2 - j, 0)], g8 = pw[max(m_tok - 9 - j, 0)], g9 = pw[max(m_tok - 10 - j, 0)];
+      auto factor = [&](int t) { return SSD ? __expf(pw[kLtC - 1] - pw[t]) * sz[t] : pw[max(m_tok - 1 - t, 0)]; };
+      const float g0 = factor(j), g1 = factor(j + 1), g8 = factor(j + 8), g9 = factor(j + 9);
 #pragma unroll
       for (int m = 0; m < MT; ++m) {
         uint32_t a[4];
@@ -252,6 +298,7 @@ __global__ void __launch_bounds__(kLtThreads, 2) linear_attn_tc_kernel(const Lin
       }
     }
   }
+  if (SSD && STATES && blockIdx.z == 0 && threadIdx.x == 0) p.seg_decay[(long long)seg * p.H + h] = expf(total);
   float* dst = nullptr;
   if (STATES) dst = p.seg_state + ((long long)seg * p.H + h) * D * p.dv;
   else if (last) dst = p.state + ((long long)p.rows.slots[b] * p.H + h) * D * p.dv;
@@ -266,16 +313,10 @@ __global__ void __launch_bounds__(kLtThreads, 2) linear_attn_tc_kernel(const Lin
   }
 }
 
-template <int D>
-static int lt_launch(const LinTcParams& p, int nseg, bool states, cudaStream_t s) {
-  const dim3 grid(nseg, p.H, p.dv / kLtV);
-  if (states) {
-    cudaFuncSetAttribute(linear_attn_tc_kernel<D, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, LtSmem<D, true>::kTotal);
-    launch_pdl(linear_attn_tc_kernel<D, true>, grid, dim3(kLtThreads), (size_t)LtSmem<D, true>::kTotal, s, p);
-  } else {
-    cudaFuncSetAttribute(linear_attn_tc_kernel<D, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, LtSmem<D, false>::kTotal);
-    launch_pdl(linear_attn_tc_kernel<D, false>, grid, dim3(kLtThreads), (size_t)LtSmem<D, false>::kTotal, s, p);
-  }
+template <int D, bool STATES, bool SSD>
+static int lt_launch(const LinTcParams& p, int nseg, cudaStream_t s) {
+  cudaFuncSetAttribute(linear_attn_tc_kernel<D, STATES, SSD>, cudaFuncAttributeMaxDynamicSharedMemorySize, LtSmem<D, STATES>::kTotal);
+  launch_pdl(linear_attn_tc_kernel<D, STATES, SSD>, dim3(nseg, p.H, p.dv / kLtV), dim3(kLtThreads), (size_t)LtSmem<D, STATES>::kTotal, s, p);
   return -(int)cudaGetLastError();
 }
 
@@ -297,15 +338,21 @@ int lx_silu_cols(void* x, long long ld, int T, int cols, void* stream) {
   return -(int)cudaGetLastError();
 }
 
-// q, k, v with their silu applied.  One pass over the segments: states != 0 the segments' contributions, else outputs and final states (the carry pass in between is
-// lx_recurrence's).
-int lx_linear_attn_tc(const void* params, int d, int nseg, int states, void* stream) {
+// q, k, v with their silu applied (ssd: the inputs of the state space recurrence, and z, w0, A, skip, hpg).  One pass over the segments:
+// states != 0 the segments' contributions, else outputs and final states (the carry pass in between is lx_recurrence's).
+int lx_linear_attn_tc(const void* params, int d, int nseg, int states, int ssd, void* stream) {
   using namespace lx;
   if (nseg <= 0) return 0;
   const LinTcParams& p = *reinterpret_cast<const LinTcParams*>(params);
   if (!lx_linear_attn_tc_supported(d, p.dv) || p.ldq % 8 != 0 || p.ldk % 8 != 0 || p.ldv % 8 != 0) return -1;
+  if (ssd && (p.hpg <= 0 || p.H % p.hpg != 0 || (states && p.seg_decay == nullptr))) return -2;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  return d == 64 ? lt_launch<64>(p, nseg, states != 0, s) : lt_launch<128>(p, nseg, states != 0, s);
+  if (ssd) {
+    if (states) return d == 64 ? lt_launch<64, true, true>(p, nseg, s) : lt_launch<128, true, true>(p, nseg, s);
+    return d == 64 ? lt_launch<64, false, true>(p, nseg, s) : lt_launch<128, false, true>(p, nseg, s);
+  }
+  if (states) return d == 64 ? lt_launch<64, true, false>(p, nseg, s) : lt_launch<128, true, false>(p, nseg, s);
+  return d == 64 ? lt_launch<64, false, false>(p, nseg, s) : lt_launch<128, false, false>(p, nseg, s);
 }
 
 }  // extern "C"

@@ -1,10 +1,11 @@
 // Mixture-of-experts feed-forward on the device: routing, dispatch, grouped expert GEMMs, combine.
 //
 //   router logits   logits[t, e] = x[t, :] . Wr[e, :]: bf16 products, fp32 sums (mma.sync; K over the warps of a CTA)
-//   select          one warp per token.  softmax: top-k of the logits, kept weights renormalised (the reference's routing math,
-//                   server/lorax_server/models/custom_modeling/flash_mixtral_modeling.py:449-459).  sigmoid: the choice goes by
-//                   score + correction, within the best groups of neighbouring experts (by the sum of a group's two largest); the
-//                   weights are the scores without the correction, normalised, times a constant
+//   select          one warp per token.  softmax: top-k of the logits, the weights renormalised over the chosen (the reference's routing
+//                   math, server/lorax_server/models/custom_modeling/flash_mixtral_modeling.py:449-459) or over all experts.  sigmoid: the
+//                   choice goes by score + correction; the weights are the scores without the correction, normalised or not.  Both: the
+//                   choice may be limited to the best groups of neighbouring experts (by the largest of a group or its two largest), and
+//                   the weights are multiplied by a constant
 //   place, gather   the rows routed to each expert this rank owns become one contiguous run seg[e] .. seg[e+1] of a sorted order, and
 //                   xg[p, :] = x[token of sorted row p, :]
 //   grouped GEMM    work items (expert, 128 features of its weight, token tile of its run) on tcgen05: weights on the UMMA M
@@ -119,7 +120,7 @@ struct MoeSelectParams {
   int* counts;             // [e_local], zero on entry
   long long ldl;
   int T, E, k, e0, e_local;
-  int sigmoid, groups, keep, shared;
+  int sigmoid, groups, keep, shared, group_top, renorm;
   float scale;
 };
 
@@ -175,7 +176,7 @@ __global__ void __launch_bounds__(32 * kSelWarps) moe_select_kernel(const MoeSel
           const float v = choice_s[warp][g * gs + q];
           if (v > a) { b = a; a = v; } else if (v > b) { b = v; }
         }
-        score[i] = gs > 1 ? a + b : a;
+        score[i] = gs > 1 && p.group_top > 1 ? a + b : a;
       }
     }
     __syncwarp();
@@ -221,7 +222,14 @@ __global__ void __launch_bounds__(32 * kSelWarps) moe_select_kernel(const MoeSel
   }
   float w = 0.f;
   if (lane < p.k) w = p.sigmoid ? 1.f / (1.f + expf(-l[id])) : expf(l[id] - top);
-  const float sum = warp_sum(w) + (p.sigmoid ? 1e-20f : 0.f);
+  float sum = 1.f;
+  if (p.renorm) {
+    sum = warp_sum(w) + (p.sigmoid ? 1e-20f : 0.f);
+  } else if (!p.sigmoid) {                       // (the first chosen logit is the largest of all)
+    float own = 0.f;
+    for (int e = lane; e < p.E; e += 32) own += expf(l[e] - top);
+    sum = warp_sum(own);
+  }
   const int kw = p.k + p.shared;
   if (lane < p.k) {
     const int le = id - p.e0;
@@ -344,7 +352,8 @@ constexpr int kMgBM = 128;
 constexpr int kMgBK = 64;
 constexpr int kMgThreads = 192;
 
-enum MoeAct : int { kMoeActNone = 0, kMoeActRelu2 = 1 };
+// swiglu: the weight's rows are gate and up in turn, output column i is silu(row 2i) * row 2i + 1.
+enum MoeAct : int { kMoeActNone = 0, kMoeActRelu2 = 1, kMoeActSwiglu = 2 };
 LX_DEVICE float moe_act(float v, int act) {
   if (act == kMoeActRelu2) { v = fmaxf(v, 0.f); v *= v; }
   return v;
@@ -353,7 +362,7 @@ LX_DEVICE float moe_act(float v, int act) {
 struct MoeGemmParams {
   int K, n_w, runs;               // runs: routed experts of this rank, then the shared ones
   const int* seg;                 // [runs + 1] rows of every run in the sorted order
-  __nv_bfloat16* out;             // [rows, n_w]
+  __nv_bfloat16* out;             // [rows, n_w], swiglu: [rows, n_w / 2]
   long long ldo;
   int bn;                         // token tile = UMMA N (multiple of 16, <= BN)
   int rows_cap;                   // rows the output holds
@@ -533,7 +542,17 @@ moe_grouped_gemm_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid
 #pragma unroll
           for (int q = 0; q < 16; ++q) v[q] = __uint_as_float(r[q]);
         }
-        if (i < p.n_w) {
+        if (p.act == kMoeActSwiglu) {
+          // gate and up of a column sit in neighbouring lanes: each lane of the pair finishes half of the tokens
+          const bool odd = lane & 1;
+#pragma unroll
+          for (int q = 0; q < CH / 2; ++q) {
+            const float other = __shfl_xor_sync(0xffffffffu, odd ? v[q] : v[q + CH / 2], 1);
+            const float g = odd ? other : v[q], up = odd ? v[q + CH / 2] : other;
+            const int tok = c + q + (odd ? CH / 2 : 0);
+            if (tok < nrows) p.out[(long long)(row0 + tok) * p.ldo + (i >> 1)] = __float2bfloat16(__fdividef(g, 1.f + __expf(-g)) * up);
+          }
+        } else if (i < p.n_w) {
 #pragma unroll
           for (int q = 0; q < CH; ++q) {
             if (c + q < nrows) p.out[(long long)(row0 + c + q) * p.ldo + i] = __float2bfloat16(moe_act(v[q], p.act));
@@ -599,6 +618,14 @@ __global__ void __launch_bounds__(256) moe_grouped_gemm_f32_kernel(const float* 
   for (int i = 0; i < 4; ++i) {
     const int r = ty * 4 + i;
     if (r >= nrows) continue;
+    if (p.act == kMoeActSwiglu) {
+#pragma unroll
+      for (int j = 0; j < 4; j += 2) {
+        const int n = n0 + tx * 4 + j;
+        if (n < p.n_w) out[(long long)(row0 + r) * p.ldo + (n >> 1)] = acc[i][j] / (1.f + expf(-acc[i][j])) * acc[i][j + 1];
+      }
+      continue;
+    }
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx * 4 + j;
@@ -662,6 +689,7 @@ int lx_moe_select(const void* params, void* stream) {
   if (p.T <= 0) return 0;
   if (p.E > kMoeMaxExperts || p.E < 1 || p.k > kMoeMaxK || p.k > p.E || p.k < 1 || p.e_local > kMoeMaxExperts || p.shared > kMoeMaxShared) return -1;
   if (p.ldl < p.E + (p.shared > 0 ? 1 : 0)) return -2;
+  if (p.group_top < 1 || p.group_top > 2 || (!p.sigmoid && p.groups > 0 && p.group_top != 1)) return -4;
   if (p.groups > 0 && (p.E % p.groups != 0 || p.keep < 1 || p.keep > p.groups || p.keep * (p.E / p.groups) < p.k)) return -3;
   const dim3 grid((p.T + kSelWarps - 1) / kSelWarps), block(32 * kSelWarps);
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);

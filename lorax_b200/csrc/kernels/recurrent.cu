@@ -2,6 +2,8 @@
 //
 //   linear attention  S <- decay_h S + k v^T,        o = S^T q            (q, k, v pass through silu; decay constant per head)
 //   WKV               o = (S + diag(u) k v^T)^T r,   S <- diag(w) S + k v^T   (w = exp(-exp(z + w0)) per token and key channel)
+//   SSD               S <- exp(A_h s) S + s k v^T,   o = S^T q + D_h v        (Mamba-2: s = softplus(z + w0) per token and head; q, k, v
+//                     are C, B, x, and hpg heads share q and k)
 //
 // Decode rows take one step each: the state streams through once (read, update, write).  Prompt tokens are cut into segments.  A first
 // pass computes every segment's own contribution to the state and its total decay, a second one carries the state over the segments of
@@ -11,27 +13,28 @@
 
 namespace lx {
 
-enum RecMode : int { kLinAttn = 0, kWkv = 1 };
+enum RecMode : int { kLinAttn = 0, kWkv = 1, kSsd = 2 };
 
 struct RecParams {
-  const void* q;            // [T, ldq] q (linear attention) or r (WKV), head h at column h * d
+  const void* q;            // [T, ldq] q (linear attention) or r (WKV), head h at column (h / hpg) * d
   const void* k;
   const void* v;            // head h at column h * dv
-  const void* z;            // WKV: decay logits [T, ldz]
+  const void* z;            // WKV: decay logits [T, ldz]; SSD: step sizes before the softplus, head h at column h
   long long ldq, ldk, ldv, ldz;
   const float* decay;       // linear attention: [H]
-  const float* w0;          // WKV: [H * d]
-  const float* u;           // WKV: [H * d]
+  const float* w0;          // WKV: [H * d]; SSD: [H]
+  const float* u;           // WKV: [H * d]; SSD: A [H], negative
+  const float* skip;        // SSD: D [H]
   float* state;             // [slots, H, d, dv]
   float* out;               // [T, H * dv]
-  int H, d, dv;
+  int H, d, dv, hpg;
   StepRows rows;
   // prefill segments
   const int* seg_seq;       // [nseg]
   const int* seg_q0;        // [nseg] first token of the segment within its sequence
   int nseg, seg_len;
   float* seg_state;         // [nseg, H, d, dv]: contribution of the segment, then the state in front of it
-  float* seg_decay;         // WKV: [nseg, H, d] product of the segment's decays
+  float* seg_decay;         // product of the segment's decays: WKV [nseg, H, d], SSD [nseg, H]
 };
 
 // ------------------------------------------------------------------------------------------------
@@ -57,15 +60,23 @@ __global__ void __launch_bounds__(kRecStepThreads) rec_step_kernel(const RecPara
     for (int c = threadIdx.x; c < dv; c += blockDim.x) out[c] = 0.f;
     return;
   }
-  const T* q = reinterpret_cast<const T*>(p.q) + (long long)t * p.ldq + h * d;
-  const T* k = reinterpret_cast<const T*>(p.k) + (long long)t * p.ldk + h * d;
+  const int hk = MODE == kSsd ? h / p.hpg : h;
+  const T* q = reinterpret_cast<const T*>(p.q) + (long long)t * p.ldq + hk * d;
+  const T* k = reinterpret_cast<const T*>(p.k) + (long long)t * p.ldk + hk * d;
   const T* v = reinterpret_cast<const T*>(p.v) + (long long)t * p.ldv + h * dv;
-  float bonus = 0.f;
+  float bonus = 0.f, size = 1.f, lam = 1.f;
+  if (MODE == kSsd) {
+    size = softplus_f(to_f(reinterpret_cast<const T*>(p.z)[(long long)t * p.ldz + h]) + p.w0[h]);
+    lam = expf(p.u[h] * size);
+  }
   for (int i = threadIdx.x; i < d; i += blockDim.x) {
     float a = to_f(q[i]), b = to_f(k[i]);
     if (MODE == kLinAttn) {
       a = silu_f(a); b = silu_f(b);
       sw[i] = p.decay[h];
+    } else if (MODE == kSsd) {
+      b *= size;
+      sw[i] = lam;
     } else {
       const T* z = reinterpret_cast<const T*>(p.z) + (long long)t * p.ldz + h * d;
       sw[i] = expf(-expf(to_f(z[i]) + p.w0[h * d + i]));
@@ -100,7 +111,7 @@ __global__ void __launch_bounds__(kRecStepThreads) rec_step_kernel(const RecPara
           if (MODE == kWkv) { o.x += a * s[j].x; o.y += a * s[j].y; o.z += a * s[j].z; o.w += a * s[j].w; }
           s[j].x = w * s[j].x + kk * vv.x; s[j].y = w * s[j].y + kk * vv.y;
           s[j].z = w * s[j].z + kk * vv.z; s[j].w = w * s[j].w + kk * vv.w;
-          if (MODE == kLinAttn) { o.x += a * s[j].x; o.y += a * s[j].y; o.z += a * s[j].z; o.w += a * s[j].w; }
+          if (MODE != kWkv) { o.x += a * s[j].x; o.y += a * s[j].y; o.z += a * s[j].z; o.w += a * s[j].w; }
           *reinterpret_cast<float4*>(S + (long long)i * dv + c4 * 4) = s[j];
         }
       }
@@ -109,7 +120,7 @@ __global__ void __launch_bounds__(kRecStepThreads) rec_step_kernel(const RecPara
   }
   __syncthreads();
   for (int c = threadIdx.x; c < dv; c += blockDim.x) {
-    float s = MODE == kWkv ? bonus * sv[c] : 0.f;
+    float s = MODE == kWkv ? bonus * sv[c] : MODE == kSsd ? p.skip[h] * sv[c] : 0.f;
     for (int g = 0; g < rg_n; ++g) s += part[g * dv + c];
     out[c] = s;
   }
@@ -140,8 +151,10 @@ __global__ void __launch_bounds__(256) rec_scan_kernel(const RecParams p, int tc
   float* sw = sk + tc * d;                         // WKV only
   float* sv = sw + (MODE == kWkv ? tc * d : 0);    // [tc][64]
   float* part = sv + tc * 64;                      // [tc][warps][64]
-  float* bonus = part + (STATES ? 0 : tc * nw * 64);   // [tc]
-  const float lam = MODE == kLinAttn ? p.decay[h] : 0.f;
+  float* bonus = part + (STATES ? 0 : tc * nw * 64);   // [tc]; SSD: the tokens' decays
+  float* ssize = bonus + tc;                       // SSD: the tokens' step sizes
+  float lam = MODE == kLinAttn ? p.decay[h] : 0.f;
+  const int hk = MODE == kSsd ? h / p.hpg : h;
 
   float2 S[RPT];
   // (a sequence of several segments reads its first state from the carry pass too: its last segment overwrites the slot meanwhile)
@@ -160,13 +173,25 @@ __global__ void __launch_bounds__(256) rec_scan_kernel(const RecParams p, int tc
   for (int t0 = 0; t0 < n; t0 += tc) {
     const int m = min(tc, n - t0);
     __syncthreads();
+    if (MODE == kSsd) {
+      if ((int)threadIdx.x < m) {
+        const float z = to_f(reinterpret_cast<const T*>(p.z)[(tok0 + t0 + threadIdx.x) * p.ldz + h]);
+        const float size = softplus_f(z + p.w0[h]);
+        ssize[threadIdx.x] = size;
+        bonus[threadIdx.x] = expf(p.u[h] * size);
+      }
+      __syncthreads();
+    }
     for (int e = threadIdx.x * 4; e < m * d; e += blockDim.x * 4) {
       const int tt = e / d, i = e % d;
       const long long tok = tok0 + t0 + tt;
-      float4 kk = load4(reinterpret_cast<const T*>(p.k) + tok * p.ldk + h * d + i);
+      float4 kk = load4(reinterpret_cast<const T*>(p.k) + tok * p.ldk + hk * d + i);
       float4 qq = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (!STATES) qq = load4(reinterpret_cast<const T*>(p.q) + tok * p.ldq + h * d + i);
-      if (MODE == kLinAttn) {
+      if (!STATES) qq = load4(reinterpret_cast<const T*>(p.q) + tok * p.ldq + hk * d + i);
+      if (MODE == kSsd) {
+        const float size = ssize[tt];
+        kk = make_float4(kk.x * size, kk.y * size, kk.z * size, kk.w * size);
+      } else if (MODE == kLinAttn) {
         kk = make_float4(silu_f(kk.x), silu_f(kk.y), silu_f(kk.z), silu_f(kk.w));
         if (!STATES) qq = make_float4(silu_f(qq.x), silu_f(qq.y), silu_f(qq.z), silu_f(qq.w));
       } else {
@@ -186,6 +211,10 @@ __global__ void __launch_bounds__(256) rec_scan_kernel(const RecParams p, int tc
       *reinterpret_cast<float4*>(sv + e) = v;
     }
     __syncthreads();
+    if (MODE == kSsd) {
+      if (STATES && threadIdx.x == 0)
+        for (int tt = 0; tt < m; ++tt) dprod[0] *= bonus[tt];
+    }
     if (MODE == kWkv) {
       if (STATES) {
         if (blockIdx.z == 0) {
@@ -208,6 +237,7 @@ __global__ void __launch_bounds__(256) rec_scan_kernel(const RecParams p, int tc
     for (int tt = 0; tt < m; ++tt) {
       const float2 v = *reinterpret_cast<const float2*>(sv + tt * 64 + 2 * lane);
       float ox = 0.f, oy = 0.f;
+      if (MODE == kSsd) lam = bonus[tt];
 #pragma unroll
       for (int i = 0; i < RPT; i += 4) {
         if (row0 + i < d) {
@@ -221,7 +251,7 @@ __global__ void __launch_bounds__(256) rec_scan_kernel(const RecParams p, int tc
             if (MODE == kWkv && !STATES) { ox = fmaf(qa[j], S[i + j].x, ox); oy = fmaf(qa[j], S[i + j].y, oy); }
             S[i + j].x = fmaf(wa[j], S[i + j].x, ka[j] * v.x);
             S[i + j].y = fmaf(wa[j], S[i + j].y, ka[j] * v.y);
-            if (MODE == kLinAttn && !STATES) { ox = fmaf(qa[j], S[i + j].x, ox); oy = fmaf(qa[j], S[i + j].y, oy); }
+            if (MODE != kWkv && !STATES) { ox = fmaf(qa[j], S[i + j].x, ox); oy = fmaf(qa[j], S[i + j].y, oy); }
           }
         }
       }
@@ -232,7 +262,7 @@ __global__ void __launch_bounds__(256) rec_scan_kernel(const RecParams p, int tc
       for (int e = threadIdx.x; e < m * 64; e += blockDim.x) {
         const int tt = e >> 6, c = e & 63;
         if (c0 + c < dv) {
-          float s = MODE == kWkv ? bonus[tt] * sv[e] : 0.f;
+          float s = MODE == kWkv ? bonus[tt] * sv[e] : MODE == kSsd ? p.skip[h] * sv[e] : 0.f;
           for (int g = 0; g < nw; ++g) s += part[(tt * nw + g) * 64 + c];
           p.out[(tok0 + t0 + tt) * (long long)p.H * dv + (long long)h * dv + c0 + c] = s;
         }
@@ -247,6 +277,7 @@ __global__ void __launch_bounds__(256) rec_scan_kernel(const RecParams p, int tc
     for (int i = 0; i < RPT; ++i)
       if (row0 + i < d) *reinterpret_cast<float2*>(dst + (long long)(row0 + i) * dv + ca) = S[i];
   }
+  if (STATES && MODE == kSsd && blockIdx.z == 0 && threadIdx.x == 0) p.seg_decay[(long long)seg * p.H + h] = dprod[0];
   if (STATES && MODE == kWkv && blockIdx.z == 0) {
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
@@ -288,6 +319,7 @@ __global__ void __launch_bounds__(256) rec_carry_kernel(const RecParams p) {
       if (j0 + u + 1 < ns) {
         own[u] = load4(p.seg_state + at * dd + e);
         if (MODE == kWkv) w[u] = p.seg_decay[at * p.d + row];
+        if (MODE == kSsd) w[u] = p.seg_decay[at];
       }
     }
 #pragma unroll
@@ -313,7 +345,7 @@ static int rec_launch(const RecParams& p, int what, cudaStream_t s) {
     const int rpt = p.d <= 128 ? 16 : 32;
     const int nw = (p.d + rpt - 1) / rpt;
     const int tc = p.d <= 128 ? 16 : 8;
-    const size_t smem = sizeof(float) * ((MODE == kWkv ? 3 : 2) * tc * p.d + tc * 64 + tc * nw * 64 + tc);
+    const size_t smem = sizeof(float) * ((MODE == kWkv ? 3 : 2) * tc * p.d + tc * 64 + tc * nw * 64 + 2 * tc);
     const dim3 grid(p.nseg, p.H, (p.dv + 63) / 64), block(32 * nw);
     if (what & kRecStates) {
       if (rpt == 16) {
@@ -402,15 +434,19 @@ extern "C" {
 int lx_step_rows_bytes() { return (int)sizeof(lx::StepRows); }
 int lx_rec_params_bytes() { return (int)sizeof(lx::RecParams); }
 
-// mode 0: linear attention, 1: WKV.  what: the passes to launch (1 decode rows, 2 the segments' contributions, 4 the carry over the
+// mode 0: linear attention, 1: WKV, 2: SSD.  what: the passes to launch (1 decode rows, 2 the segments' contributions, 4 the carry over the
 // segments, 8 outputs and final states); 2 and 4 are needed, with seg_state / seg_decay, when some sequence has more than one segment.
 int lx_recurrence(const void* params, int mode, int what, int f32, void* stream) {
   using namespace lx;
   const RecParams& p = *reinterpret_cast<const RecParams*>(params);
   if (p.d % 16 != 0 || p.dv % 16 != 0 || p.d > 256 || p.dv > 1024 || p.H <= 0) return -1;
   if (p.ldq % 4 != 0 || p.ldk % 4 != 0 || p.ldv % 4 != 0 || (mode == kWkv && p.ldz % 4 != 0)) return -2;
-  if ((what & (kRecStates | kRecCarry)) && (p.seg_state == nullptr || (mode == kWkv && p.seg_decay == nullptr))) return -3;
+  if ((what & (kRecStates | kRecCarry)) && (p.seg_state == nullptr || (mode != kLinAttn && p.seg_decay == nullptr))) return -3;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  if (mode == kSsd) {
+    if (p.hpg <= 0 || p.H % p.hpg != 0) return -4;
+    return f32 ? rec_launch<float, kSsd>(p, what, s) : rec_launch<__nv_bfloat16, kSsd>(p, what, s);
+  }
   if (f32) return mode == kLinAttn ? rec_launch<float, kLinAttn>(p, what, s) : rec_launch<float, kWkv>(p, what, s);
   return mode == kLinAttn ? rec_launch<__nv_bfloat16, kLinAttn>(p, what, s) : rec_launch<__nv_bfloat16, kWkv>(p, what, s);
 }

@@ -33,46 +33,79 @@ __global__ void __launch_bounds__(128) embed_stream_kernel(const int* __restrict
 }
 
 // ------------------------------------------------------------------------------------------------
-// residual += pending (fp32); out = residual / sqrt(sum / n + eps) * (w + w_offset).  One CTA per row.
+// residual += pending (fp32); out = residual / sqrt(sum / n + eps) * (w + w_offset).  One CTA per row.  PAIRS: what is added to a token is
+// the weighted sum of the rows pos[t, 0 .. k) (-1: none) of pending (the outputs of its experts).  rows: only these rows, and the
+// residual stays as it is.
 // ------------------------------------------------------------------------------------------------
 constexpr int kNsThreads = 256, kNsMaxVec = 8;      // 16384 columns at most
 
-template <typename T>
-__global__ void __launch_bounds__(kNsThreads) norm_stream_kernel(float* __restrict__ residual, const T* __restrict__ pending,
-                                                                 const float* __restrict__ w, T* __restrict__ out, int W, float inv_n,
-                                                                 float eps, float w_offset) {
+struct NormStreamParams {
+  float* residual;
+  const void* pending;         // [T or pairs, ldp] or null
+  long long ldp;
+  const float* w;
+  void* out;
+  const int* pos;              // [T, k]
+  const float* weights;        // [T, k]
+  const int* rows;             // or null
+  int k, W;
+  float inv_n, eps, w_offset;
+};
+
+template <typename T, bool PAIRS, int NV>
+__global__ void __launch_bounds__(kNsThreads) norm_stream_kernel(const NormStreamParams p) {
   pdl_trigger();
   pdl_wait();
   __shared__ float red[kNsThreads / 32];
-  const long long row = (long long)blockIdx.x * W;
-  float v[kNsMaxVec][8];
+  const int t = p.rows != nullptr ? p.rows[blockIdx.x] : (int)blockIdx.x;
+  float* res = p.residual + (long long)t * p.W;
+  const T* pending = reinterpret_cast<const T*>(p.pending);
+  float v[NV][8];
   float ss = 0.f;
 #pragma unroll
-  for (int it = 0; it < kNsMaxVec; ++it) {
+  for (int it = 0; it < NV; ++it) {
     const int c = (threadIdx.x + it * blockDim.x) * 8;
-    if (c < W) {
-      load8(residual + row + c, v[it]);
+    if (c < p.W) {
+      load8(res + c, v[it]);
       if (pending != nullptr) {
-        float p[8];
-        load8(pending + row + c, p);
+        if constexpr (PAIRS) {
+          float sum[8];
 #pragma unroll
-        for (int q = 0; q < 8; ++q) v[it][q] += p[q];
-        store8(residual + row + c, v[it]);
+          for (int q = 0; q < 8; ++q) sum[q] = 0.f;
+          for (int j = 0; j < p.k; ++j) {
+            const int row = p.pos[(long long)t * p.k + j];
+            if (row < 0) continue;
+            const float wj = p.weights[(long long)t * p.k + j];
+            float f[8];
+            load8(pending + (long long)row * p.ldp + c, f);
+#pragma unroll
+            for (int q = 0; q < 8; ++q) sum[q] = fmaf(wj, f[q], sum[q]);
+          }
+#pragma unroll
+          for (int q = 0; q < 8; ++q) v[it][q] += sum[q];
+        } else {
+          float f[8];
+          load8(pending + (long long)t * p.ldp + c, f);
+#pragma unroll
+          for (int q = 0; q < 8; ++q) v[it][q] += f[q];
+        }
+        if (p.rows == nullptr) store8(res + c, v[it]);
       }
 #pragma unroll
       for (int q = 0; q < 8; ++q) ss += v[it][q] * v[it][q];
     }
   }
-  const float r = rsqrtf(block_sum(ss, red) * inv_n + eps);
+  const float r = rsqrtf(block_sum(ss, red) * p.inv_n + p.eps);
+  T* out = reinterpret_cast<T*>(p.out) + (long long)blockIdx.x * p.W;
 #pragma unroll
-  for (int it = 0; it < kNsMaxVec; ++it) {
+  for (int it = 0; it < NV; ++it) {
     const int c = (threadIdx.x + it * blockDim.x) * 8;
-    if (c < W) {
+    if (c < p.W) {
       float g[8];
-      load8(w + c, g);
+      load8(p.w + c, g);
 #pragma unroll
-      for (int q = 0; q < 8; ++q) g[q] = v[it][q] * r * (g[q] + w_offset);
-      store8(out + row + c, g);
+      for (int q = 0; q < 8; ++q) g[q] = v[it][q] * r * (g[q] + p.w_offset);
+      store8(out + c, g);
     }
   }
 }
@@ -242,6 +275,68 @@ __global__ void __launch_bounds__(256) norm_gate_kernel(const float* __restrict_
   }
 }
 
+// ------------------------------------------------------------------------------------------------
+// The gate first, then the norm: rows of H heads of vd columns (PP apart) of y (fp32) and z, u = y * silu(z) closed up to [H * vd], every
+// `part` columns divided by their own root mean square, times w; zeros in the columns behind them up to ncols.  One CTA per (row, part).
+// VEC: four columns per access.
+// ------------------------------------------------------------------------------------------------
+struct GateNormParams {
+  const float* y;              // [T, H * PP]
+  const void* z;               // [T, ldz]
+  const float* w;              // [H * vd]
+  void* out;                   // [T, ldo]
+  long long ldz, ldo;
+  int H, vd, PP, part, ncols;
+  float eps;
+};
+constexpr int kGnThreads = 256, kGnVec = 8;
+
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(kGnThreads) gate_norm_kernel(const GateNormParams p) {
+  pdl_trigger();
+  pdl_wait();
+  __shared__ float red[kGnThreads / 32];
+  const int t = blockIdx.x, first = blockIdx.y * p.part;
+  const float* y = p.y + (long long)t * p.H * p.PP;
+  const T* z = reinterpret_cast<const T*>(p.z) + (long long)t * p.ldz;
+  T* out = reinterpret_cast<T*>(p.out) + (long long)t * p.ldo;
+  float ss = 0.f;
+  if constexpr (VEC) {
+    float4 v[kGnVec];                            // (part is at most kGnVec * 4 * kGnThreads)
+#pragma unroll
+    for (int it = 0; it < kGnVec; ++it) {
+      const int c = (threadIdx.x + it * kGnThreads) * 4;
+      v[it] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (c >= p.part) continue;
+      const int col = first + c, at = col / p.vd * p.PP + col % p.vd;
+      const float4 a = load4(y + at), g = load4(z + at);
+      v[it] = make_float4(a.x * silu_f(g.x), a.y * silu_f(g.y), a.z * silu_f(g.z), a.w * silu_f(g.w));
+      ss += v[it].x * v[it].x + v[it].y * v[it].y + v[it].z * v[it].z + v[it].w * v[it].w;
+    }
+    const float r = rsqrtf(block_sum(ss, red) / p.part + p.eps);
+#pragma unroll
+    for (int it = 0; it < kGnVec; ++it) {
+      const int c = (threadIdx.x + it * kGnThreads) * 4;
+      if (c >= p.part) continue;
+      const float4 w = load4(p.w + first + c);
+      store4(out + first + c, make_float4(v[it].x * r * w.x, v[it].y * r * w.y, v[it].z * r * w.z, v[it].w * r * w.w));
+    }
+  } else {
+    auto value = [&](int col) {
+      const int at = col / p.vd * p.PP + col % p.vd;
+      return y[at] * silu_f(to_f(z[at]));
+    };
+    for (int c = threadIdx.x; c < p.part; c += kGnThreads) {
+      const float v = value(first + c);
+      ss += v * v;
+    }
+    const float r = rsqrtf(block_sum(ss, red) / p.part + p.eps);
+    for (int c = threadIdx.x; c < p.part; c += kGnThreads) put(out + first + c, value(first + c) * r * p.w[first + c]);
+  }
+  if (blockIdx.y == 0)
+    for (int c = p.H * p.vd + threadIdx.x; c < p.ncols; c += kGnThreads) put(out + c, 0.f);
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256) tanh_kernel(T* __restrict__ x, long long n8) {
   pdl_trigger();
@@ -329,6 +424,7 @@ struct BatchedGemmParams {
   long long ldx, sx, ldw, sw, ldo, so, ldg;
   int T, N, K;
   float out_scale;
+  const float* bias;           // fp32 product: [N] or null
 };
 
 __global__ void __launch_bounds__(256) gemm_f32_kernel(const BatchedGemmParams p) {
@@ -370,7 +466,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const BatchedGemmParams p
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx * 4 + j;
-      if (n < p.N) out[(long long)t * p.ldo + n] = acc[i][j] * s;
+      if (n < p.N) out[(long long)t * p.ldo + n] = acc[i][j] * s + (p.bias != nullptr ? p.bias[n] : 0.f);
     }
   }
 }
@@ -503,21 +599,40 @@ int lx_norm_rows(const void* residual, const int* rows, const void* w, const voi
   return -(int)cudaGetLastError();
 }
 
-int lx_norm_stream(void* residual, const void* pending, const void* w, void* out, int T, int W, int n, float eps, float w_offset, int f32,
-                   void* stream) {
+int lx_norm_stream_bytes() { return (int)sizeof(lx::NormStreamParams); }
+
+// T: rows of the result (p.rows null: of the residual too).
+int lx_norm_stream(const void* params, int T, int f32, void* stream) {
   using namespace lx;
+  const NormStreamParams& p = *reinterpret_cast<const NormStreamParams*>(params);
   if (T <= 0) return 0;
-  if (W % 8 != 0 || W > kNsThreads * kNsMaxVec * 8 || n <= 0) return -1;
+  if (p.W % 8 != 0 || p.W > kNsThreads * kNsMaxVec * 8 || p.ldp % 8 != 0) return -1;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  const int threads = W / 8 >= kNsThreads ? kNsThreads : (W / 8 + 31) / 32 * 32;
-  float* r = reinterpret_cast<float*>(residual);
-  const float* wp = reinterpret_cast<const float*>(w);
-  if (f32)
-    launch_pdl(norm_stream_kernel<float>, dim3(T), dim3(threads), 0, s, r, reinterpret_cast<const float*>(pending), wp, reinterpret_cast<float*>(out), W,
-               1.f / n, eps, w_offset);
-  else
-    launch_pdl(norm_stream_kernel<__nv_bfloat16>, dim3(T), dim3(threads), 0, s, r, reinterpret_cast<const __nv_bfloat16*>(pending), wp,
-               reinterpret_cast<__nv_bfloat16*>(out), W, 1.f / n, eps, w_offset);
+  const int threads = p.W / 8 >= kNsThreads ? kNsThreads : (p.W / 8 + 31) / 32 * 32;
+  const int nv = (p.W / 8 + threads - 1) / threads;
+#define LX_NS(TY, PR)                                                                                   \
+  if (nv <= 1) launch_pdl(norm_stream_kernel<TY, PR, 1>, dim3(T), dim3(threads), 0, s, p);                \
+  else if (nv <= 2) launch_pdl(norm_stream_kernel<TY, PR, 2>, dim3(T), dim3(threads), 0, s, p);           \
+  else if (nv <= 4) launch_pdl(norm_stream_kernel<TY, PR, 4>, dim3(T), dim3(threads), 0, s, p);           \
+  else launch_pdl(norm_stream_kernel<TY, PR, kNsMaxVec>, dim3(T), dim3(threads), 0, s, p);
+  if (f32) { if (p.pos != nullptr) { LX_NS(float, true) } else { LX_NS(float, false) } }
+  else { if (p.pos != nullptr) { LX_NS(__nv_bfloat16, true) } else { LX_NS(__nv_bfloat16, false) } }
+#undef LX_NS
+  return -(int)cudaGetLastError();
+}
+
+int lx_gate_norm_bytes() { return (int)sizeof(lx::GateNormParams); }
+
+int lx_gate_norm(const void* params, int T, int f32, void* stream) {
+  using namespace lx;
+  const GateNormParams& p = *reinterpret_cast<const GateNormParams*>(params);
+  if (T <= 0) return 0;
+  if (p.part <= 0 || p.vd <= 0 || p.vd > p.PP || p.H * p.vd % p.part != 0 || p.ncols < p.H * p.vd) return -1;
+  const bool vec = p.vd % 4 == 0 && p.PP % 4 == 0 && p.part % 4 == 0 && p.ldz % 4 == 0 && p.ldo % 4 == 0 && p.part <= kGnVec * 4 * kGnThreads;
+  const dim3 grid(T, p.H * p.vd / p.part), block(kGnThreads);
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  if (f32) { if (vec) launch_pdl(gate_norm_kernel<float, true>, grid, block, 0, s, p); else launch_pdl(gate_norm_kernel<float, false>, grid, block, 0, s, p); }
+  else { if (vec) launch_pdl(gate_norm_kernel<__nv_bfloat16, true>, grid, block, 0, s, p); else launch_pdl(gate_norm_kernel<__nv_bfloat16, false>, grid, block, 0, s, p); }
   return -(int)cudaGetLastError();
 }
 
@@ -572,14 +687,16 @@ int lx_argmax_f32(const void* logits, long long ld, int T, int V, int* ids, floa
   return -(int)cudaGetLastError();
 }
 
-// out[b][t, n] = x[b][t, :] . w[b][n, :] over `batch` products with element strides sx / sw / so; gate [T, ldg]: column b.
+// out[b][t, n] = x[b][t, :] . w[b][n, :] over `batch` products with element strides sx / sw / so; gate [T, ldg]: column b.  bias [N]: fp32 only.
 int lx_gemm_batched(const void* x, long long ldx, long long sx, const void* w, long long ldw, long long sw, void* out, long long ldo,
-                    long long so, const void* gate, long long ldg, int T, int N, int K, int batch, float out_scale, int f32, void* stream) {
+                    long long so, const void* gate, long long ldg, int T, int N, int K, int batch, float out_scale, const float* bias, int f32,
+                    void* stream) {
   using namespace lx;
   if (T <= 0 || N <= 0 || batch <= 0) return 0;
-  BatchedGemmParams p{x, w, out, gate, ldx, sx, ldw, sw, ldo, so, ldg, T, N, K, out_scale};
+  BatchedGemmParams p{x, w, out, gate, ldx, sx, ldw, sw, ldo, so, ldg, T, N, K, out_scale, bias};
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const dim3 grid((N + 63) / 64, (T + 63) / 64, batch);
+  if (bias != nullptr && !f32) return -2;
   if (f32) {
     launch_pdl(gemm_f32_kernel, grid, dim3(256), 0, s, p);
   } else {

@@ -44,6 +44,7 @@ LX_DEVICE void put(float* p, float v) { *p = v; }
 
 LX_DEVICE float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
 LX_DEVICE float silu_f(float z) { return z / (1.f + expf(-z)); }
+LX_DEVICE float softplus_f(float z) { return z > 20.f ? z : log1pf(expf(z)); }
 
 // Sum over the block, the same value in every thread; `red` holds one float per warp.
 LX_DEVICE float block_sum(float v, float* red) {

@@ -273,8 +273,8 @@ def lora_fused_desc(ws: "Workspace", lf: LoraFused, K: int) -> LxLoraFused:
 def gemm(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None,
          out_scale: float = 1.0, mode: int = 0, force_split: int = 0) -> torch.Tensor:
     """out[T, N] = x[T, K] @ w[N, K]^T (+ bias).  bf16 in, fp32 accumulate on tcgen05, bf16 out (fp32 in: true fp32 throughout)."""
-    if x.dtype == torch.float32 and bias is None:
-        return gemm_f32(x, w, out=out, out_scale=out_scale)
+    if x.dtype == torch.float32:
+        return gemm_f32(x, w, out=out, out_scale=out_scale, bias=bias)
     assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and x.dim() == 2 and w.dim() == 2
     assert x.stride(1) == 1 and w.stride(1) == 1
     T, K = x.shape
@@ -323,7 +323,8 @@ class MoeSelectParams(ctypes.Structure):
     """Mirror of the C struct of the same name (csrc/kernels/moe.cu)."""
     _fields_ = [("logits", c_void_p), ("correction", c_void_p), ("topk_ids", c_void_p), ("topk_w", c_void_p), ("rank", c_void_p),
                 ("counts", c_void_p), ("ldl", c_longlong), ("T", c_int), ("E", c_int), ("k", c_int), ("e0", c_int), ("e_local", c_int),
-                ("sigmoid", c_int), ("groups", c_int), ("keep", c_int), ("shared", c_int), ("scale", c_float)]
+                ("sigmoid", c_int), ("groups", c_int), ("keep", c_int), ("shared", c_int), ("group_top", c_int),
+                ("renorm", c_int), ("scale", c_float)]
 
 
 class MoePlaceParams(ctypes.Structure):
@@ -334,7 +335,8 @@ class MoePlaceParams(ctypes.Structure):
 
 
 def moe_route(x: torch.Tensor, router_w: torch.Tensor, k: int, e0: int, e_local: int, experts: Optional[int] = None, score: str = "softmax",
-              correction: Optional[torch.Tensor] = None, groups: int = 0, keep: int = 0, scale: float = 1.0, shared: int = 0) -> MoeRouting:
+              correction: Optional[torch.Tensor] = None, groups: int = 0, keep: int = 0, scale: float = 1.0, shared: int = 0, group_top: int = 2,
+              renorm: bool = True) -> MoeRouting:
     """Router logits (fp32), choice of `k` experts per token (`reference.moe_route` states the rules), and the sorted order of the rows
     routed to the experts [e0, e0 + e_local) this rank owns with those rows gathered: three launches, everything stays on the device."""
     T, H = x.shape
@@ -356,7 +358,7 @@ def moe_route(x: torch.Tensor, router_w: torch.Tensor, k: int, e0: int, e_local:
                    torch.empty(e_local + shared + 1, dtype=torch.int32, device=dev), torch.empty(T, kw, dtype=torch.int32, device=dev),
                    torch.empty(T * (k + (1 if shared else 0)), H, dtype=x.dtype, device=dev))
     p = MoeSelectParams(_ptr(logits), _ptr(correction), _ptr(r.topk_ids), _ptr(r.topk_w), _ptr(rank), _ptr(counts), logits.stride(0), T, E, k,
-                        e0, e_local, int(score == "sigmoid"), groups, keep, shared, scale)
+                        e0, e_local, int(score == "sigmoid"), groups, keep, shared, group_top, int(renorm), scale)
     _check(lib.lx_moe_select(ctypes.byref(p), _stream()), "lx_moe_select")
     size = x.element_size()
     q = MoePlaceParams(_ptr(x), _ptr(r.xg), x.stride(0) * size, r.xg.stride(0) * size, H * size, _ptr(counts), _ptr(r.topk_ids), _ptr(rank),
@@ -365,19 +367,20 @@ def moe_route(x: torch.Tensor, router_w: torch.Tensor, k: int, e0: int, e_local:
     return r
 
 
-_MOE_ACTS = {"": 0, "relu2": 1}
+_MOE_ACTS = {"": 0, "relu2": 1, "swiglu": 2}
 
 
 def moe_grouped_gemm(xg: torch.Tensor, w: torch.Tensor, seg: torch.Tensor, avg_rows: int, out: Optional[torch.Tensor] = None, shared: int = 0,
                      tokens: int = 0, act: str = "") -> torch.Tensor:
     """out[q] = act(xg[q] @ w[e(q)]^T) for every sorted row q (e(q): the expert whose run [seg[e], seg[e+1]) holds q).
     w: [experts, n_w, K], n_w a multiple of 128.  The last `shared` experts all read the one set of `tokens` rows that stands where
-    the first of them begins; the result has rows of its own for each."""
+    the first of them begins; the result has rows of its own for each.  act "swiglu": the rows of w are gate and up in turn, and column i
+    of the result is silu(column 2i) * column 2i + 1."""
     runs, n_w, K = w.shape
     rows = xg.shape[0] + max(shared - 1, 0) * tokens
     assert w.is_contiguous() and xg.stride(1) == 1 and xg.shape[1] == K and xg.dtype == w.dtype
     if out is None:
-        out = torch.empty(rows, n_w, dtype=xg.dtype, device=xg.device)
+        out = torch.empty(rows, n_w // (2 if act == "swiglu" else 1), dtype=xg.dtype, device=xg.device)
     ws = workspace(xg.device)
     rc = load().lx_moe_grouped_gemm(_ptr(xg), xg.stride(0), _ptr(w), K, _ptr(out), out.stride(0), _ptr(seg), runs, xg.shape[0], rows, n_w, K,
                                     avg_rows, shared, tokens, _MOE_ACTS[act], int(xg.dtype == torch.float32), _ptr(ws.status), ws.num_sms,
@@ -719,14 +722,16 @@ def lora_expand_tiles(v, tiles: torch.Tensor, num_tiles: int, max_tile_rows: int
 
 
 # ------------------------------------------------------------------------------------------------ layer-by-layer designs
-from .native_mixers import (embed_stream, gemm_f32, gemm_heads, gemm_stack, gqa_attn, latent_attn, latent_prep, linear_attn,  # noqa: E402
-                            latent_prefill, norm_add, norm_gate, norm_stream, qk_norm_kvwrite, rope_pairs, tanh_, token_shift, wkv)
+from .native_mixers import (causal_conv, conv_rope_kvwrite, embed_stream, gate_norm, gemm_f32, gemm_heads, gemm_stack, gqa_attn,  # noqa: E402
+                            latent_attn, latent_prefill, latent_prep, linear_attn, norm_add, norm_gate, norm_stream, qk_norm_kvwrite, rope_pairs,
+                            ssd, tanh_, token_shift, wkv)
 
 # ------------------------------------------------------------------------------------------------ per-op timing
 _TIMED_OPS = ("gemm", "gemm_fp8", "norm_residual", "rope_kvwrite", "act_mul", "embed", "argmax_logprob", "advance_decode", "attn_decode",
               "attn_prefill", "lora_shrink", "lora_expand", "lora_shrink_tiles", "lora_expand_tiles",
               "embed_stream", "norm_stream", "norm_gate", "tanh_", "gemm_heads", "linear_attn", "wkv", "token_shift", "latent_prep", "rope_pairs",
-              "latent_attn", "latent_prefill", "norm_add", "qk_norm_kvwrite", "gqa_attn", "moe_route", "moe_grouped_gemm", "moe_combine")
+              "latent_attn", "latent_prefill", "norm_add", "qk_norm_kvwrite", "conv_rope_kvwrite", "causal_conv", "ssd",
+              "gate_norm", "gqa_attn", "moe_route", "moe_grouped_gemm", "moe_combine")
 _timing_records = None
 _timing_originals = {}
 

@@ -1,5 +1,5 @@
 """Bindings of the kernels of the layer-by-layer designs (`models/mixers.py`): `csrc/kernels/stream.cu`, `recurrent.cu`,
-`latent_attn.cu` and `gqa.cu`.  Every operator exists for bf16 and for fp32 activations.  Imported into :mod:`lorax_b200.ops.native`."""
+`conv_rope.cu`, `latent_attn.cu` and `gqa.cu`.  Every operator exists for bf16 and for fp32 activations.  Imported into :mod:`lorax_b200.ops.native`."""
 
 from __future__ import annotations
 
@@ -20,14 +20,15 @@ class StepRows(Structure):
 
 
 class RecParams(Structure):
-    _fields_ = [("q", P), ("k", P), ("v", P), ("z", P), ("ldq", L), ("ldk", L), ("ldv", L), ("ldz", L), ("decay", P), ("w0", P), ("u", P),
-                ("state", P), ("out", P), ("H", I), ("d", I), ("dv", I), ("rows", StepRows), ("seg_seq", P), ("seg_q0", P), ("nseg", I),
+    _fields_ = [("q", P), ("k", P), ("v", P), ("z", P), ("ldq", L), ("ldk", L), ("ldv", L), ("ldz", L), ("decay", P), ("w0", P), ("u", P), ("skip", P),
+                ("state", P), ("out", P), ("H", I), ("d", I), ("dv", I), ("hpg", I), ("rows", StepRows), ("seg_seq", P), ("seg_q0", P), ("nseg", I),
                 ("seg_len", I), ("seg_state", P), ("seg_decay", P)]
 
 
 class LinTcParams(Structure):
     _fields_ = [("q", P), ("k", P), ("v", P), ("ldq", L), ("ldk", L), ("ldv", L), ("decay", P), ("state", P), ("seg_state", P), ("out", P),
-                ("H", I), ("dv", I), ("rows", StepRows), ("seg_seq", P), ("seg_q0", P), ("seg_len", I)]
+                ("H", I), ("dv", I), ("rows", StepRows), ("seg_seq", P), ("seg_q0", P), ("seg_len", I), ("hpg", I), ("z", P), ("ldz", L), ("w0", P),
+                ("A", P), ("skip", P), ("seg_decay", P)]
 
 
 class WkvTcParams(Structure):
@@ -63,7 +64,22 @@ class QkNormParams(Structure):
 
 class GqaF32Params(Structure):
     _fields_ = [("q", P), ("ldq", L), ("cache", P), ("out", P), ("ldo", L), ("rows", StepRows), ("T", I), ("H", I), ("G", I), ("DK", I),
-                ("DV", I), ("page", I), ("window", I), ("scale", F)]
+                ("DV", I), ("page", I), ("window", I), ("scale", F), ("softcap", F), ("out_scale", F), ("sink", P), ("gate", P), ("ldg", L)]
+
+
+class NormStreamParams(Structure):
+    _fields_ = [("residual", P), ("pending", P), ("ldp", L), ("w", P), ("out", P), ("pos", P), ("weights", P), ("rows", P), ("k", I), ("W", I),
+                ("inv_n", F), ("eps", F), ("w_offset", F)]
+
+
+class GateNormParams(Structure):
+    _fields_ = [("y", P), ("z", P), ("w", P), ("out", P), ("ldz", L), ("ldo", L), ("H", I), ("vd", I), ("PP", I), ("part", I), ("ncols", I), ("eps", F)]
+
+
+class ConvParams(Structure):
+    _fields_ = [("x", P), ("ldx", L), ("out", P), ("ldo", L), ("w", P), ("b", P), ("state", P), ("rows", StepRows), ("tile_seq", P), ("tile_q0", P),
+                ("C", I), ("taps", I), ("silu", I), ("dec_ctas", I), ("cache", P), ("slots", P), ("positions", P), ("cos_sin", P), ("P", I),
+                ("rot", I), ("H", I), ("G", I), ("DK", I), ("DV", I), ("page", I)]
 
 
 SIGNATURES = {
@@ -76,20 +92,26 @@ SIGNATURES = {
     "lx_qk_norm_kvwrite": ([P, I, P], I),
     "lx_gqa_f32_bytes": ([], I),
     "lx_gqa_attn_f32": ([P, P], I),
-    "lx_gqa_decode": ([P, L, P, P, I, P, P, L, P, P, I, I, I, I, I, I, F, I, P], I),
-    "lx_gqa_prefill": ([P, L, P, P, I, P, P, P, P, I, P, L, I, I, I, I, I, F, P], I),
-    "lx_norm_stream": ([P, P, P, P, I, I, I, F, F, I, P], I),
+    "lx_gqa_decode": ([P, L, P, P, I, P, P, L, P, P, I, I, I, I, I, I, F, I, F, P, P, L, F, P], I),
+    "lx_gqa_prefill": ([P, L, P, P, I, P, P, P, P, I, P, L, I, I, I, I, I, F, F, P, P, L, F, P], I),
+    "lx_gqa_prefill_tc": ([P, L, I, P, I, P, I, P, P, P, P, I, P, L, I, I, I, I, F, F, P, P, L, F, P, P], I),
+    "lx_norm_stream_bytes": ([], I),
+    "lx_norm_stream": ([P, I, I, P], I),
+    "lx_gate_norm_bytes": ([], I),
+    "lx_gate_norm": ([P, I, I, P], I),
+    "lx_conv_bytes": ([], I),
+    "lx_conv": ([P, I, I, I, P], I),
     "lx_norm_gate": ([P, P, P, L, P, L, I, I, I, I, F, I, I, P], I),
     "lx_tanh": ([P, L, I, P], I),
     "lx_act_mul_f32": ([P, P, I, I, L, L, I, I, P], I),
     "lx_argmax_f32": ([P, L, I, I, P, P, F, P], I),
-    "lx_gemm_batched": ([P, L, L, P, L, L, P, L, L, P, L, I, I, I, I, F, I, P], I),
+    "lx_gemm_batched": ([P, L, L, P, L, L, P, L, L, P, L, I, I, I, I, F, P, I, P], I),
     "lx_step_rows_bytes": ([], I),
     "lx_rec_params_bytes": ([], I),
     "lx_recurrence": ([P, I, I, I, P], I),
     "lx_linear_attn_tc_bytes": ([], I),
     "lx_linear_attn_tc_supported": ([I, I], I),
-    "lx_linear_attn_tc": ([P, I, I, I, P], I),
+    "lx_linear_attn_tc": ([P, I, I, I, I, P], I),
     "lx_wkv_tc_bytes": ([], I),
     "lx_wkv_tc_supported": ([I], I),
     "lx_wkv_tc": ([P, I, I, P], I),
@@ -113,7 +135,8 @@ def check_layouts(lib):
     for name, st in (("lx_step_rows_bytes", StepRows), ("lx_rec_params_bytes", RecParams), ("lx_latent_prep_bytes", LatentPrepParams),
                      ("lx_latent_attn_bytes", LatentAttnParams), ("lx_latent_decode_bytes", LatentDecodeParams),
                      ("lx_linear_attn_tc_bytes", LinTcParams), ("lx_wkv_tc_bytes", WkvTcParams),
-                     ("lx_norm_add_bytes", NormAddParams), ("lx_qk_norm_bytes", QkNormParams), ("lx_gqa_f32_bytes", GqaF32Params)):
+                     ("lx_norm_add_bytes", NormAddParams), ("lx_qk_norm_bytes", QkNormParams), ("lx_gqa_f32_bytes", GqaF32Params),
+                     ("lx_norm_stream_bytes", NormStreamParams), ("lx_gate_norm_bytes", GateNormParams), ("lx_conv_bytes", ConvParams)):
         if getattr(lib, name)() != ctypes.sizeof(st):
             raise nv.NativeError(f"{name}: C++ says {getattr(lib, name)()} bytes, ctypes says {ctypes.sizeof(st)}")
 
@@ -146,21 +169,24 @@ def embed_stream(ids, table, mult: float = 1.0, pos=None, positions=None, copy=N
     return out
 
 
-def norm_stream(residual, pending, weight, eps: float, weight_offset: float, n: int, dtype, bias=None, layernorm: bool = False, rows=None):
+def norm_stream(residual, pending, weight, eps: float, weight_offset: float, n: int, dtype, bias=None, layernorm: bool = False, rows=None,
+                pairs=None):
+    """(with `rows`, pending is added to the rows it takes on the way and `residual` stays as it is)"""
     T, W = residual.shape
-    if layernorm or rows is not None:
-        assert pending is None
-        if rows is not None:
-            T = rows.shape[0]
-        out = torch.empty(T, W, dtype=dtype, device=residual.device)
-        if T:
-            nv._check(nv.load().lx_norm_rows(_p(residual), _p(rows), _p(weight), _p(bias), _p(out), T, W, n, eps, weight_offset, int(layernorm),
-                                             _f32(out), nv._stream()), "lx_norm_rows")
-        return out
+    if rows is not None:
+        T = rows.shape[0]
     out = torch.empty(T, W, dtype=dtype, device=residual.device)
-    assert pending is None or pending.is_contiguous()
-    nv._check(nv.load().lx_norm_stream(_p(residual), _p(pending), _p(weight), _p(out), T, W, n, eps, weight_offset, _f32(out), nv._stream()),
-              "lx_norm_stream")
+    if T == 0:
+        return out
+    if layernorm or (rows is not None and pending is None):
+        assert pending is None
+        nv._check(nv.load().lx_norm_rows(_p(residual), _p(rows), _p(weight), _p(bias), _p(out), T, W, n, eps, weight_offset, int(layernorm),
+                                         _f32(out), nv._stream()), "lx_norm_rows")
+        return out
+    pos, w = pairs if pairs is not None else (None, None)
+    p = NormStreamParams(_p(residual), _p(pending), pending.stride(0) if pending is not None else 0, _p(weight), _p(out), _p(pos), _p(w), _p(rows),
+                         pos.shape[1] if pos is not None else 0, W, 1.0 / n, eps, weight_offset)
+    nv._check(nv.load().lx_norm_stream(ctypes.byref(p), T, _f32(out), nv._stream()), "lx_norm_stream")
     return out
 
 
@@ -187,13 +213,20 @@ def tanh_(x):
     return x
 
 
-def gemm_f32(x, w, out=None, out_scale: float = 1.0):
+def gate_norm(y, z, H: int, p: int, parts: int, weight, eps: float, out):
+    T, C = y.shape
+    a = GateNormParams(_p(y), _p(z), _p(weight), _p(out), z.stride(0), out.stride(0), H, p, C // H, H * p // parts, out.shape[1], eps)
+    nv._check(nv.load().lx_gate_norm(ctypes.byref(a), T, _f32(out), nv._stream()), "lx_gate_norm")
+    return out
+
+
+def gemm_f32(x, w, out=None, out_scale: float = 1.0, bias=None):
     T, K = x.shape
     N = w.shape[0]
     if out is None:
         out = torch.empty(T, N, dtype=torch.float32, device=x.device)
-    nv._check(nv.load().lx_gemm_batched(_p(x), x.stride(0), 0, _p(w), w.stride(0), 0, _p(out), out.stride(0), 0, None, 0, T, N, K, 1, out_scale, 1,
-                                        nv._stream()), "lx_gemm_batched")
+    nv._check(nv.load().lx_gemm_batched(_p(x), x.stride(0), 0, _p(w), w.stride(0), 0, _p(out), out.stride(0), 0, None, 0, T, N, K, 1, out_scale,
+                                        _p(bias), 1, nv._stream()), "lx_gemm_batched")
     return out
 
 
@@ -227,18 +260,19 @@ def gemm_heads(x, w, out, x_head: int, gate=None):
     H, N, K = w.shape
     T = x.shape[0]
     nv._check(nv.load().lx_gemm_batched(_p(x), x.stride(0), x_head, _p(w), K, N * K, _p(out), out.stride(0), N, _p(gate),
-                                        gate.stride(0) if gate is not None else 0, T, N, K, H, 1.0, _f32(x), nv._stream()), "lx_gemm_batched")
+                                        gate.stride(0) if gate is not None else 0, T, N, K, H, 1.0, None, _f32(x), nv._stream()),
+              "lx_gemm_batched")
     return out
 
 
-def _recurrence(mode: int, q, k, v, z, decay, w0, u, H: int, d: int, dv: int, state, inp):
+def _recurrence(mode: int, q, k, v, z, decay, w0, u, H: int, d: int, dv: int, state, inp, skip=None, hpg: int = 1):
     T = q.shape[0]
     out = torch.empty(T, H * dv, dtype=torch.float32, device=q.device)
     p = RecParams()
     p.q, p.k, p.v, p.z = _p(q), _p(k), _p(v), _p(z)
     p.ldq, p.ldk, p.ldv, p.ldz = q.stride(0), k.stride(0), v.stride(0), z.stride(0) if z is not None else 0
-    p.decay, p.w0, p.u, p.state, p.out = _p(decay), _p(w0), _p(u), _p(state), _p(out)
-    p.H, p.d, p.dv, p.rows = H, d, dv, step_rows(inp, T)
+    p.decay, p.w0, p.u, p.skip, p.state, p.out = _p(decay), _p(w0), _p(u), _p(skip), _p(state), _p(out)
+    p.H, p.d, p.dv, p.hpg, p.rows = H, d, dv, hpg, step_rows(inp, T)
     multi = 0
     hold = None
     if inp.is_prefill:
@@ -255,14 +289,15 @@ def _recurrence(mode: int, q, k, v, z, decay, w0, u, H: int, d: int, dv: int, st
             nv._check(lib.lx_recurrence(ctypes.byref(p), mode, what, _f32(q), nv._stream()), "lx_recurrence")
             nv.launch_count += bin(what).count("1") - 1
 
-    if mode == 0 and prompts and q.dtype == torch.bfloat16 and lib.lx_linear_attn_tc_supported(d, dv):
-        t = LinTcParams(p.q, p.k, p.v, p.ldq, p.ldk, p.ldv, p.decay, p.state, p.seg_state, p.out, H, dv, p.rows, p.seg_seq, p.seg_q0, p.seg_len)
+    if mode in (0, 2) and prompts and q.dtype == torch.bfloat16 and lib.lx_linear_attn_tc_supported(d, dv):
+        t = LinTcParams(p.q, p.k, p.v, p.ldq, p.ldk, p.ldv, p.decay, p.state, p.seg_state, p.out, H, dv, p.rows, p.seg_seq, p.seg_q0, p.seg_len,
+                        hpg, p.z, p.ldz, p.w0, p.u, p.skip, p.seg_decay)
 
         def chunks(states):
-            nv._check(lib.lx_linear_attn_tc(ctypes.byref(t), d, p.nseg, states, nv._stream()), "lx_linear_attn_tc")
+            nv._check(lib.lx_linear_attn_tc(ctypes.byref(t), d, p.nseg, states, int(mode == 2), nv._stream()), "lx_linear_attn_tc")
         passes(step)
         nd = p.rows.nd
-        for x, cols in (((q, 2 * H * d + H * dv),) if k.data_ptr() == q.data_ptr() + 2 * H * d and v.data_ptr() == k.data_ptr() + 2 * H * d
+        for x, cols in () if mode == 2 else (((q, 2 * H * d + H * dv),) if k.data_ptr() == q.data_ptr() + 2 * H * d and v.data_ptr() == k.data_ptr() + 2 * H * d
                         else ((q, H * d), (k, H * d), (v, H * dv))):
             nv._check(lib.lx_silu_cols(_p(x[nd:]), x.stride(0), T - nd, cols, nv._stream()), "lx_silu_cols")
         if multi:
@@ -293,6 +328,38 @@ def linear_attn(q, k, v, H: int, d: int, dv: int, decay, state, inp):
 
 def wkv(r, k, v, z, w0, u, H: int, d: int, state, inp):
     return _recurrence(1, r, k, v, z, None, w0, u, H, d, d, state, inp)
+
+
+def ssd(xbc, dt, H: int, G: int, n: int, p: int, dt_bias, A, D, state, inp):
+    x, B, C = xbc[:, : H * p], xbc[:, H * p: H * p + G * n], xbc[:, H * p + G * n:]
+    return _recurrence(2, C, B, x, dt, None, dt_bias, A, H, n, p, state, inp, skip=D, hpg=H // G)
+
+
+def _conv(x, C: int, taps: int, w, b, state, inp, out, attn: bool, **more):
+    T = x.shape[0]
+    p = ConvParams()
+    p.x, p.ldx, p.out, p.ldo, p.w, p.b, p.state = _p(x), x.stride(0), _p(out), out.stride(0), _p(w), _p(b), _p(state)
+    p.rows, p.C, p.taps = step_rows(inp, T), C, taps
+    tiles = 0
+    if inp.is_prefill:
+        p.tile_seq, p.tile_q0, tiles = _p(inp.tile_seq), _p(inp.tile_q0), inp.tile_seq.shape[0]
+    for k, v in more.items():
+        setattr(p, k, v)
+    nv._check(nv.load().lx_conv(ctypes.byref(p), tiles, int(attn), _f32(x), nv._stream()), "lx_conv")
+    return out
+
+
+def causal_conv(x, w, b, act: str, state, inp):
+    taps, C = w.shape
+    return _conv(x, C, taps, w, b, state, inp, torch.empty(x.shape[0], C, dtype=x.dtype, device=x.device), False, silu={"": 0, "silu": 1}[act])
+
+
+def conv_rope_kvwrite(qkv, H: int, G: int, dk: int, dv: int, cos_sin, rot: int, positions, cache, inp, conv_w=None, conv_state=None):
+    out = qkv if conv_w is None else torch.empty(qkv.shape[0], H * dk, dtype=qkv.dtype, device=qkv.device)
+    more = dict(rot=rot, H=H, G=G, DK=dk, DV=dv, page=cache.shape[2] // (dk + dv), cache=_p(cache), slots=_p(inp.slots), positions=_p(positions))
+    if rot:
+        more.update(cos_sin=_p(cos_sin), P=cos_sin.shape[0])
+    return _conv(qkv, (H + G) * dk + G * dv, 0 if conv_w is None else conv_w.shape[0], conv_w, None, conv_state, inp, out, True, **more)
 
 
 def token_shift(h, mu, shift, inp):
@@ -388,12 +455,15 @@ def _gqa_splits(ctas: int, window: int, max_blocks: int, page: int) -> int:
     return max(1, min(8, 192 // max(1, ctas), pages // 4))
 
 
-def gqa_attn(q, cache, H: int, G: int, dk: int, dv: int, scale: float, window: int, inp, out):
+def gqa_attn(q, cache, H: int, G: int, dk: int, dv: int, scale: float, window: int, inp, out, softcap: float = 0.0, sink=None, gate=None,
+             out_scale: float = 1.0):
     T = q.shape[0]
     lib, ws = nv.load(), nv.workspace(q.device)
     page = cache.shape[2] // (dk + dv)
+    ldg = gate.stride(0) if gate is not None else 0
     if q.dtype == torch.float32:
-        p = GqaF32Params(_p(q), q.stride(0), _p(cache), _p(out), out.stride(0), step_rows(inp, T), T, H, G, dk, dv, page, window, scale)
+        p = GqaF32Params(_p(q), q.stride(0), _p(cache), _p(out), out.stride(0), step_rows(inp, T), T, H, G, dk, dv, page, window, scale, softcap,
+                         out_scale, _p(sink), _p(gate), ldg)
         nv._check(lib.lx_gqa_attn_f32(ctypes.byref(p), nv._stream()), "lx_gqa_attn_f32")
         return out
     if page != lib.lx_gqa_page_size():
@@ -406,16 +476,19 @@ def gqa_attn(q, cache, H: int, G: int, dk: int, dv: int, scale: float, window: i
             part_o = torch.empty(nd * H * nsplit * (dv + 1), dtype=torch.float32, device=q.device)
             part_lse = part_o[nd * H * nsplit * dv:]
         nv._check(lib.lx_gqa_decode(_p(q), q.stride(0), _p(cache), _p(dbt), dbt.shape[1], _p(ctx), _p(out), out.stride(0), _p(part_o), _p(part_lse),
-                                    nd, H, G, dk, dv, window, scale, nsplit, nv._stream()), "lx_gqa_decode")
+                                    nd, H, G, dk, dv, window, scale, nsplit, softcap, _p(sink), _p(gate), ldg, out_scale, nv._stream()),
+                  "lx_gqa_decode")
         nv.launch_count += int(nsplit > 1)
     if inp.is_prefill:
         qp, op, tiles = q[nd:], out[nd:], inp.tile_seq.shape[0]
+        gp = gate[nd:] if gate is not None else None
         if nv.TC_PREFILL and dk == dv and lib.lx_attn_prefill_tc_supported(H, G, dk, q.stride(0), out.stride(0)):
-            nv._check(lib.lx_attn_prefill_tc(_p(qp), q.stride(0), T - nd, _p(cache), cache.shape[0], _p(inp.block_tables), inp.block_tables.shape[1],
-                                             _p(inp.cu_q), _p(inp.cache_lens), _p(inp.tile_seq), _p(inp.tile_q0), tiles, _p(op), out.stride(0), H, G,
-                                             dk, window, scale, 0.0, None, 1, _p(ws.status), nv._stream()), "lx_attn_prefill_tc")
+            nv._check(lib.lx_gqa_prefill_tc(_p(qp), q.stride(0), T - nd, _p(cache), cache.shape[0], _p(inp.block_tables), inp.block_tables.shape[1],
+                                            _p(inp.cu_q), _p(inp.cache_lens), _p(inp.tile_seq), _p(inp.tile_q0), tiles, _p(op), out.stride(0), H, G,
+                                            dk, window, scale, softcap, _p(sink), _p(gp), ldg, out_scale, _p(ws.status), nv._stream()),
+                      "lx_gqa_prefill_tc")
         else:
             nv._check(lib.lx_gqa_prefill(_p(qp), q.stride(0), _p(cache), _p(inp.block_tables), inp.block_tables.shape[1], _p(inp.cu_q),
                                          _p(inp.cache_lens), _p(inp.tile_seq), _p(inp.tile_q0), tiles, _p(op), out.stride(0), H, G, dk, dv, window,
-                                         scale, nv._stream()), "lx_gqa_prefill")
+                                         scale, softcap, _p(sink), _p(gp), ldg, out_scale, nv._stream()), "lx_gqa_prefill")
     return out

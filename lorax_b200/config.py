@@ -351,9 +351,10 @@ def _mixer_model_kwargs(mt: str, d: Dict[str, Any]) -> Dict[str, Any]:
         if not (0 <= loop[0] <= loop[1] <= len(specs)) or loop[2] < 0:
             raise ValueError(f"loop {loop} does not fit {len(specs)} layers")
     flat = [p for s in specs for p in ([s.params] if "heads" in s.params else [v for v in s.params.values() if isinstance(v, dict)])]
-    most = lambda *names: max([int(next(p[n] for n in names if n in p)) for p in flat if any(n in p for n in names)] + [1])
+    most = lambda name: max([int(p[name]) for p in flat if name in p] + [1])
     return dict(dict(model_type=mt, vocab_size=int(d["vocab"]), hidden_size=int(d["width"]), intermediate_size=max([s.ff for s in specs] + [1]),
-                     num_hidden_layers=len(specs), num_attention_heads=most("heads"), num_key_value_heads=most("kv_heads", "heads"),
+                     num_hidden_layers=len(specs), num_attention_heads=most("heads"),
+                     num_key_value_heads=most("kv_heads" if any("kv_heads" in p for p in flat) else "heads"),
                      head_dim=most("dim"), rms_norm_eps=float(d["norm"]["eps"]), layer_specs=specs,
                      layer_loop=loop, eos_token_id=d.get("eos_token_id"), bos_token_id=d.get("bos_token_id"),
                      torch_dtype=d.get("torch_dtype", "bfloat16"), extra={}), **design.constants(d))

@@ -274,8 +274,7 @@ class AttentionMixer(Mixer):
         self.scale, self.window = float(params["scale"]), int(mask["size"]) if mask else 0
         if mask and self.window < 1:
             raise ValueError(f"a window of {self.window} tokens")
-        if self.scale <= 0:
-            raise ValueError(f"a score scale of {self.scale}")
+        self.sign, self.scale = (-1.0 if self.scale < 0 else 1.0), abs(self.scale)      # (the kernels take scores that grow with the products)
         self.softcap, self.out_scale = float(params.get("softcap") or 0.0), float(params.get("out_scale", 1.0))
         self.qk_norm, self.bias, self.gate = (bool(params.get(n)) for n in ("qk_norm", "bias", "gate"))
         self.taps, self.kv_from = int(params.get("conv") or 0), params.get("kv_from")
@@ -318,17 +317,20 @@ class AttentionMixer(Mixer):
         out["o"] = (w, self.H * self.dv)
         return out
 
+    def _q_sign(self, name):
+        return self.sign if name == "q" else 1.0
+
     def _rows(self, t, heads, d, dp, cols):
         return _pad_to(t.view(heads, d, -1), heads, dp, cols).reshape(heads * dp, cols)
 
     def in_parts(self, get):
-        out = [("qkv", torch.cat([self._rows(get(n), heads, d, dp, self.W) for n, heads, d, dp in self.projections]))]
+        out = [("qkv", torch.cat([self._q_sign(n) * self._rows(get(n), heads, d, dp, self.W) for n, heads, d, dp in self.projections]))]
         return out + ([("g", self._rows(get("g"), self.H, self.dv, self.dvp, self.W))] if self.gate else [])
 
     def in_bias(self, get):
         if not self.bias:
             return {}
-        return {"qkv": torch.cat([self._rows(get(n + ".b"), heads, d, dp, 1)[:, 0] for n, heads, d, dp in self.projections])}
+        return {"qkv": torch.cat([self._q_sign(n) * self._rows(get(n + ".b"), heads, d, dp, 1)[:, 0] for n, heads, d, dp in self.projections])}
 
     def out_part(self, get):
         o = get("o")
@@ -336,7 +338,7 @@ class AttentionMixer(Mixer):
 
     def load(self, get, fin, vec, model):
         if self.qk_norm:
-            self.q_norm, self.k_norm = (vec(_pad_to(get(n), self.dp)) for n in ("q.norm", "k.norm"))
+            self.q_norm, self.k_norm = (vec(_pad_to(get(n), self.dp)) for n in ("q.norm", "k.norm"))      # (the norm keeps the sign of q)
         self.sinks = vec(get("sink")) if self.sink == "learned" else vec(torch.zeros(self.H)) if self.sink == "unit" else None
         self.conv_w = None
         if self.taps:                                        # [taps, channels]

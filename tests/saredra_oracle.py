@@ -118,14 +118,12 @@ def window_attention(h, W, p, m, kv=None):
 def ssd(x, B, C, dt, A_log, D):
     """x [T, H, P], B, C [T, G, N], dt [T, H] (after softplus): the recurrence token by token.  -> y [T, H, P]"""
     T, H, P = x.shape
-    per = H // B.shape[1]
-    y = torch.zeros_like(x)
-    for h in range(H):
-        S = torch.zeros(B.shape[2], P, dtype=F64)
-        g = h // per
-        for t in range(T):
-            S = torch.exp(-torch.exp(A_log[h]) * dt[t, h]) * S + dt[t, h] * B[t, g][:, None] * x[t, h][None, :]
-            y[t, h] = S.t() @ C[t, g] + D[h] * x[t, h]
+    group = [h // (H // B.shape[1]) for h in range(H)]
+    y, S = torch.zeros_like(x), torch.zeros(H, B.shape[2], P, dtype=F64)
+    for t in range(T):
+        decay = torch.exp(-torch.exp(A_log) * dt[t])
+        S = decay[:, None, None] * S + (dt[t][:, None] * B[t, group])[:, :, None] * x[t][:, None, :]
+        y[t] = (S * C[t, group][:, :, None]).sum(1) + D[:, None] * x[t]
     return y
 
 
@@ -207,8 +205,7 @@ def forward(cfg, weights, tokens, layers_out=None):
     return linear(W["head"], rms_norm(x, W["final.norm"], eps))
 
 
-def greedy(cfg, weights, prompt, n):
-    ids = list(prompt)
-    for _ in range(n):
-        ids.append(int(forward(cfg, weights, ids)[-1].argmax()))
-    return ids[len(prompt):]
+def is_greedy(cfg, weights, prompt, out):
+    """Whether every token of `out` is the arg-max behind the prompt and the tokens before it."""
+    best = forward(cfg, weights, list(prompt) + list(out[:-1])).argmax(-1)[len(prompt) - 1:]
+    return best.tolist() == list(out)

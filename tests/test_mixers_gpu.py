@@ -409,3 +409,170 @@ def test_experts_chosen_by_corrected_sigmoids_in_groups(dtype, T, E, k, groups, 
     af = reference.moe_grouped_gemm(r.xg.cpu().float(), up.float(), r.seg.cpu(), avg, shared=shared, tokens=T, act="relu2")
     close(a, af, dtype, tol16=5e-3)
     close(y, reference.moe_grouped_gemm(a.cpu().float(), down.float(), r.seg.cpu(), avg), dtype, tol16=5e-3)
+
+
+# ---------------------------------------------------------------------------------------------- convolutions, state space recurrence, gated experts
+SHORT = {"portions": ([3, 0, 1, 40], [(0, 1), (5, 1), (0, 2), (9, 2), (33, 7), (0, 9), (64, 8), (2, 70), (0, 200)])}
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("step", list(STEPS) + ["portions"])
+@pytest.mark.parametrize("taps,C", [(1, 16), (2, 272), (3, 48), (4, 528), (5, 40), (9, 256)])
+def test_causal_convolution(dtype, step, taps, C):
+    from lorax_b200.ops import native, reference
+    dec, pre = {**STEPS, **SHORT}[step]
+    inp, _, ns = make_step(dec, pre)
+    T = inp.positions.shape[0]
+    g = torch.Generator().manual_seed(taps)
+    x = torch.randn(T, C + 24, generator=g).to(dtype)
+    w, b, state = torch.randn(taps, C, generator=g), torch.randn(C, generator=g), torch.randn(ns, taps - 1, C, generator=g).to(dtype)
+    live = [i for i in range(T) if i >= len(dec) or dec[i] > 0]
+    for bias, act in ((b, "silu"), (None, "")):
+        st, sd = state.float(), state.cuda()
+        want = reference.causal_conv(x[:, 8: 8 + C].float(), w, bias, act, st, inp)
+        got = native.causal_conv(x.cuda()[:, 8: 8 + C], w.cuda(), bias.cuda() if bias is not None else None, act, sd, to_dev(inp))
+        close(got, want, dtype, live, tol16=4e-3, tol32=2e-6)
+        assert torch.equal(sd.float().cpu(), st)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("step", list(STEPS) + ["portions"])
+@pytest.mark.parametrize("H,G,dk,dv,rot,taps", [(4, 2, 64, 64, 12, 0), (6, 2, 128, 64, 128, 3), (3, 0, 64, 128, 30, 0), (1, 1, 256, 128, 2, 4), (5, 5, 64, 256, 0, 7),
+                                                (2, 2, 128, 128, 64, 1)])
+def test_convolution_rotation_and_cache_write(dtype, step, H, G, dk, dv, rot, taps):
+    from lorax_b200.ops import native, reference
+    dec, pre = {**STEPS, **SHORT}[step]
+    inp, nb, ns = make_step(dec, pre)
+    T, C = inp.positions.shape[0], (H + G) * dk + G * dv
+    g = torch.Generator().manual_seed(taps)
+    x = torch.randn(T, C + 16, generator=g).to(dtype)
+    table = reference.rope_table(rot, 1024, 500.0) if rot else None
+    cache = torch.randn(nb, max(G, 1), PAGE * (dk + dv), generator=g).to(dtype)
+    w = torch.randn(taps, C, generator=g) if taps else None
+    state = torch.randn(ns, max(taps - 1, 0), C, generator=g).to(dtype)
+    xf, cf, st = x.float(), cache.float(), state.float()
+    want = reference.conv_rope_kvwrite(xf, H, G, dk, dv, table, rot, inp.positions, cf, inp, w, st)
+    xd, cd, sd = x.cuda(), cache.cuda(), state.cuda()
+    di = to_dev(inp)
+    got = native.conv_rope_kvwrite(xd, H, G, dk, dv, table.cuda() if rot else None, rot, di.positions, cd, di, w.cuda() if taps else None, sd)
+    live = [i for i in range(T) if i >= len(dec) or dec[i] > 0]
+    close(got[:, : H * dk], want[:, : H * dk], dtype, live, tol16=4e-3, tol32=3e-6)
+    close(cd, cf, dtype, tol16=4e-3, tol32=3e-6)
+    assert torch.equal(sd.float().cpu(), st)
+    if not taps:
+        assert got.data_ptr() == xd.data_ptr() and torch.equal(xd[:, H * dk:].cpu(), x[:, H * dk:])
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("step", list(STEPS) + ["portions", "long"])
+@pytest.mark.parametrize("H,G,n,p,strong", [(6, 3, 16, 48, False), (4, 1, 128, 64, False), (4, 2, 64, 128, True), (3, 3, 128, 64, True), (2, 1, 48, 16, False),
+                                            (2, 2, 256, 64, True), (1, 1, 16, 16, False), (6, 2, 64, 32, False)])
+def test_state_space_recurrence(dtype, step, H, G, n, p, strong):
+    """Decays from almost none to almost everything within one token."""
+    from lorax_b200.ops import native, reference
+    dec, pre = {**STEPS, **SHORT, "long": ([700], [(100, 333), (0, 640)])}[step]
+    inp, _, ns = make_step(dec, pre, seg_len=128 if step == "long" else 64)
+    T = inp.positions.shape[0]
+    g = torch.Generator().manual_seed(H)
+    xbc = torch.randn(T, H * p + 2 * G * n, generator=g).to(dtype)
+    dt = torch.randn(T, 16, generator=g).to(dtype)
+    bias = torch.linspace(-9.0, 3.0 if strong else -1.0, H)
+    A, D = -torch.exp(torch.linspace(-1.0, 3.0 if strong else 0.5, H)), torch.randn(H, generator=g)
+    state = torch.randn(ns, H, n, p, generator=g)
+    st, sd = state.clone(), state.cuda()
+    want = reference.ssd(xbc.float(), dt.float(), H, G, n, p, bias, A, D, st, inp)
+    got = native.ssd(xbc.cuda(), dt.cuda(), H, G, n, p, bias.cuda(), A.cuda(), D.cuda(), sd, to_dev(inp))
+    live = [i for i in range(T) if i >= len(dec) or dec[i] > 0]
+    close(got, want, dtype, live, tol16=1e-3)
+    close(sd, st, dtype, tol16=1e-3)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("T,H,vd,parts", [(1, 6, 12, 4), (5, 1, 1, 1), (70, 4, 64, 2), (3, 64, 64, 1), (9, 128, 80, 1), (4, 3, 7, 7), (6, 8, 128, 8)])
+def test_gated_group_norm(dtype, T, H, vd, parts):
+    from lorax_b200.ops import native, reference
+    g = torch.Generator().manual_seed(T)
+    pp, out_dim = (vd + 15) // 16 * 16, (H * vd + 15) // 16 * 16
+    y, z, w = torch.randn(T, H * pp, generator=g) * 3, torch.randn(T, H * pp + 32, generator=g).to(dtype), torch.randn(H * vd, generator=g)
+    want = reference.gate_norm(y, z[:, 16:].float(), H, vd, parts, w, 1e-4, torch.empty(T, out_dim))
+    out = torch.full((T, out_dim + 48), 5.0, dtype=dtype, device="cuda")
+    native.gate_norm(y.cuda(), z.cuda()[:, 16:], H, vd, parts, w.cuda(), 1e-4, out[:, 32: 32 + out_dim])
+    close(out[:, 32: 32 + out_dim], want, dtype, tol16=4e-3)
+    assert (out[:, :32] == 5.0).all() and (out[:, 32 + out_dim:] == 5.0).all()
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("sinks", ["none", "zero", "high", "low"])
+@pytest.mark.parametrize("step", list(STEPS) + ["long"])
+@pytest.mark.parametrize("H,G,dk,dv,window,cap", [(4, 2, 64, 64, 33, 5.0), (8, 2, 128, 128, 200, 30.0), (3, 3, 128, 128, 64, 0.0), (34, 2, 64, 128, 0, 2.0),
+                                                  (2, 1, 256, 256, 100, 50.0), (4, 1, 128, 256, 1, 1.0), (16, 4, 128, 128, 128, 15.0)])
+def test_attention_with_caps_sinks_and_gates(dtype, sinks, step, H, G, dk, dv, window, cap):
+    from lorax_b200.ops import native, reference
+    dec, pre = STEPS[step] if step in STEPS else ([1000, 1500], [(1000, 300), (0, 500), (129, 40)])
+    inp, nb, _ = make_step(dec, pre, seed=12)
+    T = inp.positions.shape[0]
+    q, cache = gqa_case(H, G, dk, dv, window, inp, nb, dtype, True)
+    g = torch.Generator().manual_seed(1)
+    sink = {"none": None, "zero": torch.zeros(H), "high": torch.randn(H, generator=g) + 25.0, "low": torch.randn(H, generator=g) - 90.0}[sinks]
+    gate = torch.randn(T, H * dv + 16, generator=g).to(dtype) * 2 if sinks != "low" else None
+    scale = 0.02 if sinks == "zero" else dk ** -0.5
+    want = torch.empty(T, H * dv)
+    reference.gqa_attn(q.float(), cache.float(), H, G, dk, dv, scale, window, inp, want, softcap=cap, sink=sink,
+                       gate=gate[:, 8: 8 + H * dv].float() if gate is not None else None, out_scale=0.7)
+    out = torch.full((T, H * dv + 8), 3.0, dtype=dtype, device="cuda")
+    native.gqa_attn(q.cuda(), cache.cuda(), H, G, dk, dv, scale, window, to_dev(inp), out, softcap=cap, sink=sink.cuda() if sink is not None else None,
+                    gate=gate.cuda()[:, 8: 8 + H * dv] if gate is not None else None, out_scale=0.7)
+    native.workspace(out.device).check_status()
+    live = [i for i in range(T) if i >= len(dec) or dec[i] > 0]
+    close(out[:, : H * dv], want, dtype, live, tol16=5e-3, tol32=4e-5)
+    assert (out[:, H * dv:] == 3.0).all()
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("T,E,k,groups,keep,W,ff", [(1, 8, 2, 0, 0, 64, 64), (7, 12, 3, 4, 2, 208, 128), (300, 40, 6, 8, 3, 64, 192), (65, 256, 8, 8, 4, 128, 64),
+                                                    (33, 6, 6, 2, 2, 64, 64), (40, 5, 1, 1, 1, 48, 64), (700, 33, 32, 0, 0, 64, 64)])
+def test_gated_experts_chosen_by_softmax_in_groups(dtype, T, E, k, groups, keep, W, ff):
+    """Groups by their largest score, weights over all experts that are not renormalised, silu(gate) * up in the product's epilogue."""
+    from lorax_b200.ops import native, reference
+    g = torch.Generator().manual_seed(T + E)
+    x = torch.randn(T, W, generator=g).to(dtype)
+    wr = torch.zeros((E + 15) // 16 * 16, W)
+    wr[:E] = torch.randn(E, W, generator=g) * W ** -0.5 * 2
+    wr = wr.to(dtype)
+    up, down = (torch.randn(E, 2 * ff, W, generator=g) * W ** -0.5).to(dtype), (torch.randn(E, 128, ff, generator=g) * ff ** -0.5).to(dtype)
+    kw = dict(experts=E, score="softmax", groups=groups, keep=keep, group_top=1, renorm=False)
+    want = reference.moe_route(x.float(), wr.float(), k, 0, E, **kw)
+    r = native.moe_route(x.cuda(), wr.cuda(), k, 0, E, **kw)
+    ids = r.topk_ids.cpu().long()
+    clear = (ids.sort(-1).values == want.topk_ids.long().sort(-1).values).all(-1)
+    assert clear.float().mean() > 0.99
+    dense = lambda r: torch.zeros(T, E).scatter_(1, r.topk_ids.cpu().long(), r.topk_w.cpu())
+    assert torch.allclose(dense(r)[clear], dense(want)[clear], atol=1e-5)
+    avg = max(1, T * k // E)
+    a = native.moe_grouped_gemm(r.xg, up.cuda(), r.seg, avg, act="swiglu")
+    y = native.moe_grouped_gemm(a, down.cuda(), r.seg, avg)
+    native.workspace(y.device).check_status()
+    assert a.shape == (T * k, ff)
+    close(a, reference.moe_grouped_gemm(r.xg.cpu().float(), up.float(), r.seg.cpu(), avg, act="swiglu"), dtype, tol16=5e-3)
+    close(y, reference.moe_grouped_gemm(a.cpu().float(), down.float(), r.seg.cpu(), avg), dtype, tol16=5e-3)
+    # the norm that reads the stream next forms the weighted sums
+    res, w = torch.randn(T, 128, generator=g), torch.randn(128, generator=g)
+    rows = torch.randint(0, T, (3,), generator=g, dtype=torch.int32)
+    pairs = (r.pos.cpu(), r.topk_w.cpu())
+    for at in (None, rows):
+        rf, rd = res.clone(), res.cuda()
+        wn = reference.norm_stream(rf, y.cpu().float(), w, 1e-5, 0.0, 120, torch.float32, pairs=pairs, rows=at)
+        gn = native.norm_stream(rd, y, w.cuda(), 1e-5, 0.0, 120, dtype, pairs=(r.pos, r.topk_w), rows=at.cuda() if at is not None else None)
+        close(gn, wn, dtype, tol16=4e-3)
+        if at is None:
+            close(rd, rf, torch.float32, tol32=1e-5)
+        plain = reference.norm_stream(res.clone(), y[:T].cpu().float(), w, 1e-5, 0.0, 120, torch.float32, rows=at)
+        close(native.norm_stream(res.cuda(), y[:T], w.cuda(), 1e-5, 0.0, 120, dtype, rows=at.cuda() if at is not None else None), plain, dtype, tol16=4e-3)
+
+
+@pytest.mark.parametrize("T,N,K", [(1, 48, 16), (70, 200, 96)])
+def test_32_bit_product_with_bias(T, N, K):
+    from lorax_b200.ops import native
+    g = torch.Generator().manual_seed(T)
+    x, w, b = torch.randn(T, K, generator=g), torch.randn(N, K, generator=g), torch.randn(N, generator=g)
+    close(native.gemm(x.cuda(), w.cuda(), bias=b.cuda()), (x.double() @ w.double().t() + b).float(), torch.float32, tol32=2e-6)

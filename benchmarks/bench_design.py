@@ -1,12 +1,14 @@
 """Prefill and decode throughput of a layer-by-layer design (random weights, layers of a real model's size) beside the closest
 uniform decoder of this framework at equal size, and the device time of every kernel of both with its share of the roofline.
 
-    python bench.py --design vabunex|sapudra [--design-size small,base] [--steps K] [--warmup W]
+    python bench.py --design vabunex|sapudra|saredra [--design-size small,base] [--steps K] [--warmup W]
 
 "Equal size": for Vabunex a llama-style decoder with the same width, feed-forward width, number of layer runs and attention heads of
 128; for Sapudra a Mixtral-style decoder with the same width, heads, window, layers and experts, whose gated experts (three matrices)
 have two thirds of the width, and which takes one expert more per token in place of the shared one; where the size has no experts, a
-Mistral-style decoder likewise.
+Mistral-style decoder likewise; for Saredra two designs whose kernels are its kernels' closest relatives: Sapudra with the same width,
+heads, window, layers and experts (not gated, of 3/2 the width: the same bytes), and Vabunex with as many layers of linear attention
+whose state has the size of the state space mixer's.
 Throughput: prefill is one eager forward pass over ragged prompts, decode one CUDA-graph replay per token, both through
 `ModelRunner`, timed with CUDA events.  Kernel times: CUDA events around every operator of an eager pass, L2 flushed in front of it,
 median of the passes.  Rooflines: the measured copy bandwidth and bf16 rate of MEASURED_PEAKS.json, whichever bounds the operator.
@@ -32,6 +34,14 @@ SAPUDRA_SIZES = {
     "small": dict(width=2048, layers=4, heads=16, kv=4, window=1024, experts=64, top=6, groups=(8, 4), ff=1536),
     "base": dict(width=4096, layers=4, heads=32, kv=8, window=1024, experts=32, top=4, groups=(4, 2), ff=6144),
     "dense": dict(width=4096, layers=4, heads=32, kv=8, window=1024, experts=0, ff=21504),
+}
+SAREDRA_SIZES = {
+    # width, layer triples (parallel, attention, attention over the keys of the one before), heads and key/value heads of 128, window;
+    # state space heads of 64, their groups and parts of the norm, state; experts, per token, groups and groups kept, width of an expert
+    # (or of the dense feed-forward)
+    "small": dict(width=2048, triples=2, heads=16, kv=4, window=1024, ssm=64, ssm_groups=1, parts=1, state=128, experts=64, top=6, groups=(8, 4), ff=1024),
+    "base": dict(width=4096, triples=1, heads=32, kv=8, window=1024, ssm=128, ssm_groups=8, parts=8, state=128, experts=32, top=4, groups=(4, 2), ff=4096),
+    "dense": dict(width=4096, triples=1, heads=32, kv=8, window=1024, ssm=128, ssm_groups=8, parts=8, state=128, experts=0, ff=14336),
 }
 PREFILL = [(1, 4096), (4, 2048), (1, 16384)]           # (prompts, tokens each)
 DECODE = [(16, 2048), (64, 2048), (256, 2048)]         # (rows, tokens of context)
@@ -77,8 +87,45 @@ def mixtral_like(s, runs, vocab=32000):
                        max_position_embeddings=32768, sliding_window=s["window"], **moe)
 
 
-DESIGNS = {"vabunex": (VABUNEX_SIZES, vabunex_config, llama_like, "llama-like"),
-           "sapudra": (SAPUDRA_SIZES, sapudra_config, mixtral_like, "mixtral-like")}
+def saredra_config(s, vocab=32000):
+    if s["experts"]:
+        mlp = dict(kind="moe", expert=dict(ff=s["ff"]),
+                   router=dict(experts=s["experts"], top=s["top"], groups=dict(count=s["groups"][0], keep=s["groups"][1])))
+    else:
+        mlp = dict(kind="dense", ff=s["ff"])
+    heads = lambda **rot: dict(heads=s["heads"], kv_heads=s["kv"], dim=128, vdim=128, scale=128 ** -0.5, softcap=50.0, mask=dict(size=s["window"]),
+                               rot=dict(base=500000.0, dims=64, **rot))
+    yarn = dict(factor=4.0, original=8192, fast=32.0, slow=1.0)
+    right = dict(heads=s["ssm"], vdim=64, state=s["state"], groups=s["ssm_groups"], norm_groups=s["parts"], conv=4)
+    layers = []
+    for i in range(s["triples"]):
+        layers.append(dict(type="parallel", mlp=mlp, mixer=dict(left=dict(heads(scaling=yarn), conv=4), right=right, left_scale=0.7, right_scale=0.7)))
+        layers.append(dict(type="attention", mlp=mlp, mixer=heads()))
+        layers.append(dict(type="attention", mlp=mlp, mixer=dict(heads(), kv_from=3 * i + 1)))
+    return dict(architecture="Saredra", vocab=vocab, width=s["width"], norm=dict(eps=1e-5), layers=layers)
+
+
+def sapudra_of_that_size(s, runs, vocab=32000):
+    from lorax_b200.config import ModelConfig
+    d = sapudra_config(dict(s, layers=runs, ff=s["ff"] * 3 // 2), vocab)
+    for layer in d["layers"]:
+        layer["mlp"].pop("shared", None)
+    return ModelConfig.from_dict(d)
+
+
+def linear_attention_of_that_size(s, runs, vocab=32000):
+    from lorax_b200.config import ModelConfig
+    H, d = s["ssm"], s["state"]
+    lin = dict(type="lightning", mixer=dict(heads=H, dim=d, vdim=64, decay=[1.0 - 2.0 ** (-3 - 7 * h / max(H - 1, 1)) for h in range(H)]),
+               mlp=dict(kind="dense", ff=2 * s["width"]))
+    return ModelConfig.from_dict(dict(architecture="Vabunex", vocab=vocab, width=s["width"], norm=dict(eps=1e-5), embedding=dict(scale=1.0),
+                                      layers=[lin] * runs))
+
+
+# sizes, configuration of the design, and what runs beside it
+DESIGNS = {"vabunex": (VABUNEX_SIZES, vabunex_config, [("llama-like", llama_like)]),
+           "sapudra": (SAPUDRA_SIZES, sapudra_config, [("mixtral-like", mixtral_like)]),
+           "saredra": (SAREDRA_SIZES, saredra_config, [("sapudra", sapudra_of_that_size), ("linear-attention", linear_attention_of_that_size)])}
 
 
 def peaks():
@@ -152,6 +199,18 @@ class OpTimer:
             io = T * H * (2 * d + dv) * 2 + T * H * dv * 4 + (T * H * d * 2 if name == "wkv" else 0)
             st = q["seqs"] * H * d * dv * 4 * (2 if q["decode"] else 1)
             return (name, io + st, 0)
+        if name == "ssd":
+            T, H, G, n, p = a[0].shape[0], *a[2:6]
+            st = q["seqs"] * H * n * p * 4 * (2 if q["decode"] else 1)
+            return (name, T * (H * p + 2 * G * n + H) * 2 + T * H * p * 4 + st, 0)
+        if name == "causal_conv":
+            return (name, a[0].shape[0] * a[1].shape[1] * 4, 0)
+        if name == "conv_rope_kvwrite":
+            T, H, G, dk, dv = a[0].shape[0], *a[1:5]
+            return (name + (" with conv" if len(a) > 10 and a[10] is not None else ""), T * 2 * (H * dk + G * (dk + dv)) * 2, 0)
+        if name == "gate_norm":
+            T, H, p = a[0].shape[0], a[2], a[3]
+            return (name, T * H * p * (4 + 2 + 2), 0)
         if name == "latent_attn":
             H, kv, rot = a[3], a[4], a[7]
             T = a[0].shape[0]
@@ -186,14 +245,17 @@ class OpTimer:
             xg, w, seg = a[:3]
             sizes = seg.diff()
             rows = int(sizes.sum())
-            return (f"moe_grouped_gemm {w.shape[1]}x{w.shape[2]}", nb(xg) + int((sizes > 0).sum()) * w[0].numel() * 2 + rows * w.shape[1] * 2,
+            cols = w.shape[1] // (2 if kw.get("act") == "swiglu" else 1)
+            return (f"moe_grouped_gemm {w.shape[1]}x{w.shape[2]}", nb(xg) + int((sizes > 0).sum()) * w[0].numel() * 2 + rows * cols * 2,
                     2 * rows * w[0].numel())
         if name == "moe_combine":
             y, k, out = a[0], a[3], a[4]
             return (name, nb(out) * (k + 1), 0)
         if name == "norm_stream":
             r, pend = a[0] if kw.get("rows") is None else a[0][: kw["rows"].shape[0]], a[1]
-            return (name, nb(r) * (2 if pend is not None else 1) + nb(pend) + r.numel() * 2, 0)
+            pairs = kw.get("pairs")
+            more = 0 if pend is None else r.numel() * pend.element_size() * (pairs[0].shape[1] if pairs is not None else 1)
+            return (name + (" of experts" if pairs is not None else ""), nb(r) * (2 if pend is not None else 1) + more + r.numel() * 2, 0)
         if name == "norm_residual":
             return (name, nb(a[0]) * 2 + nb(a[1]) * 2, 0)
         if name == "norm_gate":
@@ -230,7 +292,7 @@ class OpTimer:
 
 OPS = ("gemm", "norm_residual", "rope_kvwrite", "act_mul", "embed", "attn_decode", "attn_prefill", "embed_stream", "norm_stream", "norm_gate",
        "tanh_", "gemm_heads", "gemm_stack", "linear_attn", "wkv", "token_shift", "latent_prep", "rope_pairs", "latent_attn", "latent_prefill", "argmax_logprob", "gqa_attn",
-       "qk_norm_kvwrite", "norm_add", "moe_route", "moe_grouped_gemm", "moe_combine")
+       "qk_norm_kvwrite", "conv_rope_kvwrite", "causal_conv", "ssd", "gate_norm", "norm_add", "moe_route", "moe_grouped_gemm", "moe_combine")
 
 
 def main(args):
@@ -248,13 +310,13 @@ def main(args):
     steps, warm = min(args.steps, 50), max(3, min(args.warmup, 10))
     from bench import ClockSampler
     results = []
-    sizes, config_of, like, like_name = DESIGNS[args.design]
+    sizes, config_of, likes = DESIGNS[args.design]
     with torch.inference_mode():
         for size in args.design_size.split(","):
             s = sizes[size]
             ours = ModelConfig.from_dict(config_of(s))
             window = s.get("window", 1 << 30)
-            for name, cfg in ((args.design, ours), (like_name, like(s, len(ours.layer_schedule)))):
+            for name, cfg in [(args.design, ours)] + [(n, like(s, len(ours.layer_schedule))) for n, like in likes]:
                 model = DecoderModel.random_init_on_device(cfg, dev, torch.bfloat16, seed=0, max_positions=20000)
                 model.use_native_layers = True
                 for kind, cases in (("prefill", PREFILL), ("decode", DECODE)):

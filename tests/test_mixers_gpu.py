@@ -428,7 +428,7 @@ def test_causal_convolution(dtype, step, taps, C):
     w, b, state = torch.randn(taps, C, generator=g), torch.randn(C, generator=g), torch.randn(ns, taps - 1, C, generator=g).to(dtype)
     live = [i for i in range(T) if i >= len(dec) or dec[i] > 0]
     for bias, act in ((b, "silu"), (None, "")):
-        st, sd = state.float(), state.cuda()
+        st, sd = state.float().clone(), state.cuda()
         want = reference.causal_conv(x[:, 8: 8 + C].float(), w, bias, act, st, inp)
         got = native.causal_conv(x.cuda()[:, 8: 8 + C], w.cuda(), bias.cuda() if bias is not None else None, act, sd, to_dev(inp))
         close(got, want, dtype, live, tol16=4e-3, tol32=2e-6)
@@ -450,7 +450,7 @@ def test_convolution_rotation_and_cache_write(dtype, step, H, G, dk, dv, rot, ta
     cache = torch.randn(nb, max(G, 1), PAGE * (dk + dv), generator=g).to(dtype)
     w = torch.randn(taps, C, generator=g) if taps else None
     state = torch.randn(ns, max(taps - 1, 0), C, generator=g).to(dtype)
-    xf, cf, st = x.float(), cache.float(), state.float()
+    xf, cf, st = x[:, :C].float().clone(), cache.float().clone(), state.float().clone()
     want = reference.conv_rope_kvwrite(xf, H, G, dk, dv, table, rot, inp.positions, cf, inp, w, st)
     xd, cd, sd = x.cuda(), cache.cuda(), state.cuda()
     di = to_dev(inp)

@@ -204,10 +204,13 @@ class OpTimer:
             st = q["seqs"] * H * n * p * 4 * (2 if q["decode"] else 1)
             return (name, T * (H * p + 2 * G * n + H) * 2 + T * H * p * 4 + st, 0)
         if name == "causal_conv":
-            return (name, a[0].shape[0] * a[1].shape[1] * 4, 0)
+            taps, C = a[1].shape
+            return (name, a[0].shape[0] * C * 4 + q["seqs"] * (taps - 1) * C * (4 if q["decode"] else 2), 0)
         if name == "conv_rope_kvwrite":
             T, H, G, dk, dv = a[0].shape[0], *a[1:5]
-            return (name + (" with conv" if len(a) > 10 and a[10] is not None else ""), T * 2 * (H * dk + G * (dk + dv)) * 2, 0)
+            w = a[10] if len(a) > 10 else None
+            kept = q["seqs"] * (w.shape[0] - 1) * w.shape[1] * (4 if q["decode"] else 2) if w is not None else 0
+            return (name + (" with conv" if w is not None else ""), T * 2 * (H * dk + G * (dk + dv)) * 2 + kept, 0)
         if name == "gate_norm":
             T, H, p = a[0].shape[0], a[2], a[3]
             return (name, T * H * p * (4 + 2 + 2), 0)

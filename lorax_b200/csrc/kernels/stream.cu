@@ -278,7 +278,7 @@ __global__ void __launch_bounds__(256) norm_gate_kernel(const float* __restrict_
 // ------------------------------------------------------------------------------------------------
 // The gate first, then the norm: rows of H heads of vd columns (PP apart) of y (fp32) and z, u = y * silu(z) closed up to [H * vd], every
 // `part` columns divided by their own root mean square, times w; zeros in the columns behind them up to ncols.  One CTA per (row, part).
-// VEC: four columns per access.
+// VEC: four columns per access; parts of up to kGnWarpPart columns then take a warp each.
 // ------------------------------------------------------------------------------------------------
 struct GateNormParams {
   const float* y;              // [T, H * PP]
@@ -289,52 +289,63 @@ struct GateNormParams {
   int H, vd, PP, part, ncols;
   float eps;
 };
-constexpr int kGnThreads = 256, kGnVec = 8;
+constexpr int kGnThreads = 256, kGnVec = 8, kGnWarpPart = 32 * 4 * kGnVec;
 
-template <typename T, bool VEC>
+template <typename T>
+LX_DEVICE float gn_gate(float y, float z) {
+  return sizeof(T) == 2 ? __fdividef(y * z, 1.f + __expf(-z)) : y * silu_f(z);
+}
+
+template <typename T, bool VEC, bool WARP>
 __global__ void __launch_bounds__(kGnThreads) gate_norm_kernel(const GateNormParams p) {
   pdl_trigger();
   pdl_wait();
   __shared__ float red[kGnThreads / 32];
-  const int t = blockIdx.x, first = blockIdx.y * p.part;
+  const int t = blockIdx.x, lane = WARP ? threadIdx.x & 31 : threadIdx.x;
+  constexpr int width = WARP ? 32 : kGnThreads;
+  const int first = (WARP ? blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5) : blockIdx.y) * p.part;
+  const int inner = p.H * p.vd;
   const float* y = p.y + (long long)t * p.H * p.PP;
   const T* z = reinterpret_cast<const T*>(p.z) + (long long)t * p.ldz;
   T* out = reinterpret_cast<T*>(p.out) + (long long)t * p.ldo;
+  if (blockIdx.y == 0)
+    for (int c = inner + threadIdx.x; c < p.ncols; c += blockDim.x) put(out + c, 0.f);
+  if (WARP && first >= inner) return;
   float ss = 0.f;
   if constexpr (VEC) {
-    float4 v[kGnVec];                            // (part is at most kGnVec * 4 * kGnThreads)
+    float4 v[kGnVec];                            // (part is at most kGnVec * 4 * width)
 #pragma unroll
     for (int it = 0; it < kGnVec; ++it) {
-      const int c = (threadIdx.x + it * kGnThreads) * 4;
+      const int c = (lane + it * width) * 4;
       v[it] = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (c >= p.part) continue;
-      const int col = first + c, at = col / p.vd * p.PP + col % p.vd;
-      const float4 a = load4(y + at), g = load4(z + at);
-      v[it] = make_float4(a.x * silu_f(g.x), a.y * silu_f(g.y), a.z * silu_f(g.z), a.w * silu_f(g.w));
+      if (c < p.part) {
+        const int col = first + c, at = p.vd == p.PP ? col : col / p.vd * p.PP + col % p.vd;
+        const float4 a = load4(y + at), g = load4(z + at);
+        v[it] = make_float4(gn_gate<T>(a.x, g.x), gn_gate<T>(a.y, g.y), gn_gate<T>(a.z, g.z), gn_gate<T>(a.w, g.w));
+      }
       ss += v[it].x * v[it].x + v[it].y * v[it].y + v[it].z * v[it].z + v[it].w * v[it].w;
     }
-    const float r = rsqrtf(block_sum(ss, red) / p.part + p.eps);
+    const float r = rsqrtf((WARP ? warp_sum(ss) : block_sum(ss, red)) / p.part + p.eps);
 #pragma unroll
     for (int it = 0; it < kGnVec; ++it) {
-      const int c = (threadIdx.x + it * kGnThreads) * 4;
-      if (c >= p.part) continue;
-      const float4 w = load4(p.w + first + c);
-      store4(out + first + c, make_float4(v[it].x * r * w.x, v[it].y * r * w.y, v[it].z * r * w.z, v[it].w * r * w.w));
+      const int c = (lane + it * width) * 4;
+      if (c < p.part) {
+        const float4 w = load4(p.w + first + c);
+        store4(out + first + c, make_float4(v[it].x * r * w.x, v[it].y * r * w.y, v[it].z * r * w.z, v[it].w * r * w.w));
+      }
     }
   } else {
     auto value = [&](int col) {
       const int at = col / p.vd * p.PP + col % p.vd;
-      return y[at] * silu_f(to_f(z[at]));
+      return gn_gate<T>(y[at], to_f(z[at]));
     };
-    for (int c = threadIdx.x; c < p.part; c += kGnThreads) {
+    for (int c = lane; c < p.part; c += width) {
       const float v = value(first + c);
       ss += v * v;
     }
     const float r = rsqrtf(block_sum(ss, red) / p.part + p.eps);
-    for (int c = threadIdx.x; c < p.part; c += kGnThreads) put(out + first + c, value(first + c) * r * p.w[first + c]);
+    for (int c = lane; c < p.part; c += width) put(out + first + c, value(first + c) * r * p.w[first + c]);
   }
-  if (blockIdx.y == 0)
-    for (int c = p.H * p.vd + threadIdx.x; c < p.ncols; c += kGnThreads) put(out + c, 0.f);
 }
 
 template <typename T>
@@ -629,10 +640,16 @@ int lx_gate_norm(const void* params, int T, int f32, void* stream) {
   if (T <= 0) return 0;
   if (p.part <= 0 || p.vd <= 0 || p.vd > p.PP || p.H * p.vd % p.part != 0 || p.ncols < p.H * p.vd) return -1;
   const bool vec = p.vd % 4 == 0 && p.PP % 4 == 0 && p.part % 4 == 0 && p.ldz % 4 == 0 && p.ldo % 4 == 0 && p.part <= kGnVec * 4 * kGnThreads;
-  const dim3 grid(T, p.H * p.vd / p.part), block(kGnThreads);
+  const bool warp = vec && p.part <= kGnWarpPart;
+  const int parts = p.H * p.vd / p.part, per = parts < 4 ? parts : 4;          // parts per CTA of warps
+  const dim3 grid(T, warp ? (parts + per - 1) / per : parts), block(warp ? 32 * per : kGnThreads);
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  if (f32) { if (vec) launch_pdl(gate_norm_kernel<float, true>, grid, block, 0, s, p); else launch_pdl(gate_norm_kernel<float, false>, grid, block, 0, s, p); }
-  else { if (vec) launch_pdl(gate_norm_kernel<__nv_bfloat16, true>, grid, block, 0, s, p); else launch_pdl(gate_norm_kernel<__nv_bfloat16, false>, grid, block, 0, s, p); }
+#define LX_GN(TY)                                                                              \
+  if (warp) launch_pdl(gate_norm_kernel<TY, true, true>, grid, block, 0, s, p);                  \
+  else if (vec) launch_pdl(gate_norm_kernel<TY, true, false>, grid, block, 0, s, p);             \
+  else launch_pdl(gate_norm_kernel<TY, false, false>, grid, block, 0, s, p);
+  if (f32) { LX_GN(float) } else { LX_GN(__nv_bfloat16) }
+#undef LX_GN
   return -(int)cudaGetLastError();
 }
 

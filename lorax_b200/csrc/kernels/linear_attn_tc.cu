@@ -64,6 +64,17 @@ LX_DEVICE void lt_fetch(__nv_bfloat16* dst, const __nv_bfloat16* src, long long 
   }
 }
 
+// rows [0, n) of a tile of COLS columns on their way to L2, for the chunk after this one
+template <int COLS>
+LX_DEVICE void lt_prefetch(const __nv_bfloat16* src, long long ld, int n) {
+  constexpr int LINES = COLS / 64;
+  for (int e = threadIdx.x; e < n * LINES; e += kLtThreads)
+    asm volatile("prefetch.global.L2 [%0];" ::"l"(src + (e / LINES) * ld + (e % LINES) * 64));
+}
+
+// Barrier over the whole CTA from the two loops of the kernel (outputs, state), which pass it equally often.
+LX_DEVICE void lt_sync() { asm volatile("bar.sync 0;" ::: "memory"); }
+
 // silu in place over the columns [0, cols) of a row-strided matrix (the projections of prompt rows, read several times below)
 __global__ void __launch_bounds__(256) silu_cols_kernel(__nv_bfloat16* __restrict__ x, long long ld, int cols, long long total) {
   pdl_trigger();
@@ -108,7 +119,6 @@ __global__ void __launch_bounds__(kLtThreads, 2) linear_attn_tc_kernel(const Lin
   const bool last = q0 + p.seg_len >= qlen;
   if (STATES && last) return;
   const int warp = (threadIdx.x >> 5) & 3, group = threadIdx.x >> 7, lane = threadIdx.x & 31;
-  const bool for_state = STATES || group == 1;
   constexpr int NS = STATES ? 4 : 8;             // 8-wide column tiles of a state warp
   const int cs = STATES ? group * 32 : 0;        // its first column
   const int hk = SSD ? h / p.hpg : h;
@@ -116,41 +126,22 @@ __global__ void __launch_bounds__(kLtThreads, 2) linear_attn_tc_kernel(const Lin
     const float lam = p.decay[h];
     for (int e = threadIdx.x; e <= kLtC; e += kLtThreads) pw[e] = powf(lam, (float)e);
   }
-  float total = 0.f;                             // SSD: sum of L over the chunks so far
-
-  // state warps: rows warp * D / 4 + m * 16 + lane / 4 (+ 8), columns c0 + cs + nt * 8 + 2 (lane % 4)
-  float S[MT][NS][4];
-  const float* init = nullptr;
-  if (!STATES) {
-    if (qlen > p.seg_len) init = p.seg_state + ((long long)seg * p.H + h) * D * p.dv;
-    else if (p.rows.cache_lens[b] > 0) init = p.state + ((long long)p.rows.slots[b] * p.H + h) * D * p.dv;
-  }
-  const long long s_at = (long long)(warp * (D / 4) + (lane >> 2)) * p.dv + c0 + cs + (lane & 3) * 2;
-#pragma unroll
-  for (int m = 0; m < MT; ++m)
-#pragma unroll
-    for (int nt = 0; nt < NS; ++nt)
-#pragma unroll
-      for (int hr = 0; hr < 2; ++hr) {
-        float2 v = make_float2(0.f, 0.f);
-        if (init != nullptr && for_state) v = *reinterpret_cast<const float2*>(init + s_at + (long long)(m * 16 + hr * 8) * p.dv + nt * 8);
-        S[m][nt][2 * hr] = v.x;
-        S[m][nt][2 * hr + 1] = v.y;
-      }
   const long long tok0 = (long long)p.rows.nd + r0 + q0;
-  const uint32_t q_a = smem_u32(sq) + ((warp * 16 + (lane & 15)) * LD + (lane >> 4) * 8) * 2;
-  const uint32_t k_b = smem_u32(sk) + (((lane & 7) + (lane >> 4) * 8) * LD + ((lane >> 3) & 1) * 8) * 2;
-  const uint32_t kt_a = smem_u32(sk) + (((lane & 7) + (lane >> 4) * 8) * LD + warp * (D / 4) + ((lane >> 3) & 1) * 8) * 2;
-  const uint32_t v_b = smem_u32(sv) + (((lane & 7) + ((lane >> 3) & 1) * 8) * kLtVLd + (lane >> 4) * 8) * 2;
-  const uint32_t s_b = smem_u32(ss) + (((lane & 7) + ((lane >> 3) & 1) * 8) * kLtVLd + (lane >> 4) * 8) * 2;
 
-  for (int t0 = 0; t0 < n; t0 += kLtC) {
-    const int m_tok = min(kLtC, n - t0);
-    __syncthreads();
+  // every thread: the chunk's rows on their way, and for SSD its decays
+  auto fetch = [&](int t0, int m_tok) {
+    lt_sync();
     if (!STATES) lt_fetch<D>(sq, p.q + (tok0 + t0) * p.ldq + hk * D, p.ldq, m_tok);
     lt_fetch<D>(sk, p.k + (tok0 + t0) * p.ldk + hk * D, p.ldk, m_tok);
     lt_fetch<kLtV>(sv, p.v + (tok0 + t0) * p.ldv + h * p.dv + c0, p.ldv, m_tok);
     cp_async_commit();
+    if (t0 + kLtC < n) {
+      const int ahead = min(kLtC, n - t0 - kLtC);
+      const long long tok = tok0 + t0 + kLtC;
+      if (!STATES) lt_prefetch<D>(p.q + tok * p.ldq + hk * D, p.ldq, ahead);
+      lt_prefetch<D>(p.k + tok * p.ldk + hk * D, p.ldk, ahead);
+      lt_prefetch<kLtV>(p.v + tok * p.ldv + h * p.dv + c0, p.ldv, ahead);
+    }
     if (SSD && threadIdx.x < 32) {                 // the first warp, two tokens per lane
       float a[2];
 #pragma unroll
@@ -169,51 +160,50 @@ __global__ void __launch_bounds__(kLtThreads, 2) linear_attn_tc_kernel(const Lin
       pw[2 * lane] = sum - a[1];
       pw[2 * lane + 1] = sum;
     }
-    if (!STATES && for_state) {
-#pragma unroll
-      for (int m = 0; m < MT; ++m)
-#pragma unroll
-        for (int nt = 0; nt < NS; ++nt)
-#pragma unroll
-          for (int hr = 0; hr < 2; ++hr) {
-            uint32_t hi, lo;
-            lt_split(S[m][nt][2 * hr], S[m][nt][2 * hr + 1], hi, lo);
-            __nv_bfloat16* d = ss + (warp * (D / 4) + m * 16 + (lane >> 2) + hr * 8) * kLtVLd + nt * 8 + (lane & 3) * 2;
-            *reinterpret_cast<uint32_t*>(d) = hi;
-            *reinterpret_cast<uint32_t*>(d + D * kLtVLd) = lo;
-          }
-    }
+  };
+  auto ready = [&]() {
     cp_async_wait<0>();
-    __syncthreads();
-    if (!for_state && warp * 16 < m_tok) {
+    lt_sync();
+  };
+
+  if (!STATES && group == 0) {
+    // ---- outputs
+    const uint32_t q_a = smem_u32(sq) + ((warp * 16 + (lane & 15)) * LD + (lane >> 4) * 8) * 2;
+    const uint32_t k_b = smem_u32(sk) + (((lane & 7) + (lane >> 4) * 8) * LD + ((lane >> 3) & 1) * 8) * 2;
+    const uint32_t v_b = smem_u32(sv) + (((lane & 7) + ((lane >> 3) & 1) * 8) * kLtVLd + (lane >> 4) * 8) * 2;
+    const uint32_t s_b = smem_u32(ss) + (((lane & 7) + ((lane >> 3) & 1) * 8) * kLtVLd + (lane >> 4) * 8) * 2;
+    const int i0 = warp * 16 + (lane >> 2), i1 = i0 + 8;
+    const float skip = SSD ? p.skip[h] : 0.f;
+    for (int t0 = 0; t0 < n; t0 += kLtC) {
+      const int m_tok = min(kLtC, n - t0);
+      fetch(t0, m_tok);
+      ready();
+      if (warp * 16 >= m_tok) continue;
       float o[8][4], s[8][4];
 #pragma unroll
       for (int nt = 0; nt < 8; ++nt) {
         o[nt][0] = o[nt][1] = o[nt][2] = o[nt][3] = 0.f;
         s[nt][0] = s[nt][1] = s[nt][2] = s[nt][3] = 0.f;
       }
+      // (keys behind the rows of this warp are multiplied too, which keeps the loop free of branches; their weights are zero)
 #pragma unroll
       for (int ks = 0; ks < D / 16; ++ks) {
         uint32_t a[4];
         lt_ldsm(a, q_a + ks * 32);
 #pragma unroll
         for (int n2 = 0; n2 < 4; ++n2) {
-          if (n2 <= warp) {                        // keys behind the rows of this warp do not count
-            uint32_t kb[4];
-            lt_ldsm(kb, k_b + n2 * 16 * LD * 2 + ks * 32);
-            lt_mma(s[2 * n2], a, kb[0], kb[1]);
-            lt_mma(s[2 * n2 + 1], a, kb[2], kb[3]);
-          }
-          uint32_t sb[4];
+          uint32_t kb[4], sb[4], sl[4];
+          lt_ldsm(kb, k_b + n2 * 16 * LD * 2 + ks * 32);
           lt_ldsm_t(sb, s_b + ks * 16 * kLtVLd * 2 + n2 * 32);
+          lt_ldsm_t(sl, s_b + (D + ks * 16) * kLtVLd * 2 + n2 * 32);
+          lt_mma(s[2 * n2], a, kb[0], kb[1]);
+          lt_mma(s[2 * n2 + 1], a, kb[2], kb[3]);
           lt_mma(o[2 * n2], a, sb[0], sb[1]);
           lt_mma(o[2 * n2 + 1], a, sb[2], sb[3]);
-          lt_ldsm_t(sb, s_b + (D + ks * 16) * kLtVLd * 2 + n2 * 32);
-          lt_mma(o[2 * n2], a, sb[0], sb[1]);
-          lt_mma(o[2 * n2 + 1], a, sb[2], sb[3]);
+          lt_mma(o[2 * n2], a, sl[0], sl[1]);
+          lt_mma(o[2 * n2 + 1], a, sl[2], sl[3]);
         }
       }
-      const int i0 = warp * 16 + (lane >> 2), i1 = i0 + 8;
       const float f0 = SSD ? __expf(pw[i0]) : pw[i0 + 1], f1 = SSD ? __expf(pw[i1]) : pw[i1 + 1];
       // weight of key j for the query row i, j <= i
       auto weight = [&](int i, int j) { return SSD ? __expf(pw[i] - pw[j]) * sz[j] : pw[i - j]; };
@@ -240,10 +230,7 @@ __global__ void __launch_bounds__(kLtThreads, 2) linear_attn_tc_kernel(const Lin
           lt_mma(o[2 * n2 + 1], pl, vb[2], vb[3]);
         }
       }
-      const long long ldo = (long long)p.H * p.dv;
-      float* orow = p.out + (tok0 + t0 + i0) * ldo + (long long)h * p.dv + c0 + cs + (lane & 3) * 2;
       if constexpr (SSD) {
-        const float skip = p.skip[h];
         const __nv_bfloat16* x0 = sv + i0 * kLtVLd + (lane & 3) * 2;
 #pragma unroll
         for (int nt = 0; nt < 8; ++nt) {
@@ -253,14 +240,57 @@ __global__ void __launch_bounds__(kLtThreads, 2) linear_attn_tc_kernel(const Lin
           o[nt][2] = fmaf(skip, b.x, o[nt][2]); o[nt][3] = fmaf(skip, b.y, o[nt][3]);
         }
       }
+      const long long ldo = (long long)p.H * p.dv;
+      float* orow = p.out + (tok0 + t0 + i0) * ldo + (long long)h * p.dv + c0 + (lane & 3) * 2;
 #pragma unroll
       for (int nt = 0; nt < 8; ++nt) {
         if (i0 < m_tok) *reinterpret_cast<float2*>(orow + nt * 8) = make_float2(o[nt][0], o[nt][1]);
         if (i1 < m_tok) *reinterpret_cast<float2*>(orow + 8 * ldo + nt * 8) = make_float2(o[nt][2], o[nt][3]);
       }
     }
-    if (!for_state) continue;
-    // ---- state
+    return;
+  }
+
+  // ---- state: rows warp * D / 4 + m * 16 + lane / 4 (+ 8), columns c0 + cs + nt * 8 + 2 (lane % 4)
+  float S[MT][NS][4];
+  const float* init = nullptr;
+  if (!STATES) {
+    if (qlen > p.seg_len) init = p.seg_state + ((long long)seg * p.H + h) * D * p.dv;
+    else if (p.rows.cache_lens[b] > 0) init = p.state + ((long long)p.rows.slots[b] * p.H + h) * D * p.dv;
+  }
+  const long long s_at = (long long)(warp * (D / 4) + (lane >> 2)) * p.dv + c0 + cs + (lane & 3) * 2;
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int nt = 0; nt < NS; ++nt)
+#pragma unroll
+      for (int hr = 0; hr < 2; ++hr) {
+        float2 v = make_float2(0.f, 0.f);
+        if (init != nullptr) v = *reinterpret_cast<const float2*>(init + s_at + (long long)(m * 16 + hr * 8) * p.dv + nt * 8);
+        S[m][nt][2 * hr] = v.x;
+        S[m][nt][2 * hr + 1] = v.y;
+      }
+  const uint32_t kt_a = smem_u32(sk) + (((lane & 7) + (lane >> 4) * 8) * LD + warp * (D / 4) + ((lane >> 3) & 1) * 8) * 2;
+  const uint32_t v_b = smem_u32(sv) + (((lane & 7) + ((lane >> 3) & 1) * 8) * kLtVLd + (lane >> 4) * 8) * 2;
+  float total = 0.f;                             // SSD: sum of L over the chunks so far
+  for (int t0 = 0; t0 < n; t0 += kLtC) {
+    const int m_tok = min(kLtC, n - t0);
+    fetch(t0, m_tok);
+    if (!STATES) {
+#pragma unroll
+      for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int nt = 0; nt < NS; ++nt)
+#pragma unroll
+          for (int hr = 0; hr < 2; ++hr) {
+            uint32_t hi, lo;
+            lt_split(S[m][nt][2 * hr], S[m][nt][2 * hr + 1], hi, lo);
+            __nv_bfloat16* d = ss + (warp * (D / 4) + m * 16 + (lane >> 2) + hr * 8) * kLtVLd + nt * 8 + (lane & 3) * 2;
+            *reinterpret_cast<uint32_t*>(d) = hi;
+            *reinterpret_cast<uint32_t*>(d + D * kLtVLd) = lo;
+          }
+    }
+    ready();
     const float fs = SSD ? __expf(pw[kLtC - 1]) : pw[m_tok];
     if (SSD) total += pw[kLtC - 1];
 #pragma unroll
@@ -302,7 +332,7 @@ __global__ void __launch_bounds__(kLtThreads, 2) linear_attn_tc_kernel(const Lin
   float* dst = nullptr;
   if (STATES) dst = p.seg_state + ((long long)seg * p.H + h) * D * p.dv;
   else if (last) dst = p.state + ((long long)p.rows.slots[b] * p.H + h) * D * p.dv;
-  if (dst != nullptr && for_state) {
+  if (dst != nullptr) {
 #pragma unroll
     for (int m = 0; m < MT; ++m)
 #pragma unroll

@@ -27,7 +27,7 @@ DECODER_MODEL_TYPES = (
 
 
 # Designs whose config.json lists its layers one by one, each with a mixer of its own (models/mixers.py).
-MIXER_MODEL_TYPES = ("vabunex", "sapudra", "saredra")
+MIXER_MODEL_TYPES = ("vabunex", "sapudra", "saredra", "fegolorn")
 
 
 @dataclass
@@ -36,7 +36,7 @@ class MoeSpec:
     neighbours (0: no groups), a group counting by the sum of its `group_top` largest scores.  `score`: "sigmoid" (plus a correction
     that takes part in the choice only) or "softmax" over all experts.  The weights are the chosen scores, normalised if `renorm`, times
     `scale`.  `gated`: an expert is down(act(gate) * up) instead of down(act(up)).  `shared_ff`: width of the expert that every token
-    takes beside them, with a weight of its own (0: none)."""
+    takes beside them (0: none), with a weight of its own (`shared_gate`) or with weight one.  `bias`: the router's logits have one."""
     experts: int
     top: int
     ff: int
@@ -48,6 +48,8 @@ class MoeSpec:
     renorm: bool = True
     group_top: int = 2
     gated: bool = False
+    bias: bool = False
+    shared_gate: bool = True
 
     def __post_init__(self):
         if not 1 <= self.top <= self.experts:
@@ -62,12 +64,16 @@ class MoeSpec:
 @dataclass
 class LayerSpec:
     """One layer of a design whose layers differ: the kind of mixer, the mixer's sizes and constants, and its feed-forward: dense of
-    width `ff` (0: none; `gated`: act(gate) * up), or routed experts (`moe`)."""
+    width `ff` (0: none; `gated`: act(gate) * up), or routed experts (`moe`).  `act`: activation of the dense one (empty: the model's), with
+    its `limit` where it has one.  `weights_of`: the layer whose tensors it uses (its cache or state is its own)."""
     mixer: str
     params: Dict[str, Any]
     ff: int = 0
     moe: Optional[MoeSpec] = None
     gated: bool = False
+    act: str = ""
+    limit: float = 0.0
+    weights_of: Optional[int] = None
 
 
 @dataclass
@@ -123,9 +129,15 @@ class ModelConfig:
     layer_specs: Optional[List[LayerSpec]] = None
     layer_loop: Optional[Tuple[int, int, int]] = None
     # their residual: "parallel" (mixer and feed-forward read one norm of the stream, both are added to it), "pre" (the mixer, then the
-    # feed-forward, each reading a norm of its own) or "post" (each sublayer reads the stream itself, and a norm of its output, times
-    # residual_multiplier, is added)
+    # feed-forward, each reading a norm of its own), "post" (each sublayer reads the stream itself, and a norm of its output, times
+    # residual_multiplier, is added) or "sandwich" (each reads a norm of its own, and a second norm of its output is added)
     layer_style: str = "parallel"
+    # "sandwich": each sublayer's output is multiplied by the sigmoid of a projection of its input before its norm, and by a vector after it
+    residual_gate: bool = False
+    layer_scale: bool = False
+    norm_scalar: bool = False                # the norms of the stream have one number for all coordinates
+    # vectors looked up by (previous token * mul_prev + token * mul_cur) mod buckets, added to the token's: (buckets, mul_prev, mul_cur)
+    bigram: Optional[Tuple[int, int, int]] = None
     eos_token_id: Any = None
     bos_token_id: Any = None
     pad_token_id: Any = None
@@ -294,6 +306,7 @@ class MixerDesign:
     gated: bool = True
     moe: Dict[str, Any] = field(default_factory=dict)
     mixers: Dict[str, Dict[str, Any]] = field(default_factory=dict)
+    dense_act: str = ""
 
 
 def _vabunex_constants(d: Dict[str, Any]) -> Dict[str, Any]:
@@ -312,12 +325,23 @@ def _saredra_constants(d: Dict[str, Any]) -> Dict[str, Any]:
     return dict(layer_style="pre", hidden_act="silu", max_position_embeddings=int(d.get("max_position_embeddings", 1 << 20)))
 
 
+def _fegolorn_constants(d: Dict[str, Any]) -> Dict[str, Any]:
+    cap, bigram = d.get("logit_softcap"), d["embedding"].get("bigram")
+    return dict(layer_style="sandwich", residual_gate=True, layer_scale=True, norm_scalar=True, hidden_act="silu",
+                embedding_multiplier=float(d["embedding"]["scale"]), final_logit_softcapping=float(cap) if cap is not None else None,
+                bigram=tuple(int(bigram[n]) for n in ("buckets", "mul_prev", "mul_cur")) if bigram else None,
+                max_position_embeddings=int(d.get("max_position_embeddings", 1 << 20)))
+
+
 _MIXER_DESIGNS = {
     "vabunex": MixerDesign(_vabunex_constants, ("dense",)),
     "sapudra": MixerDesign(_sapudra_constants, ("dense", "moe"), gated=False, mixers={"attention": dict(qk_norm=True)}),
     "saredra": MixerDesign(_saredra_constants, ("dense", "moe"), moe=dict(score="softmax", renorm=False, group_top=1),
                            mixers={"attention": dict(sink="unit", gate=True),
                                    "parallel": dict(left=dict(type="attention", bias=True, sink="learned"), right=dict(type="mamba2"))}),
+    "fegolorn": MixerDesign(_fegolorn_constants, ("dense", "moe"), moe=dict(score="softmax", bias=True, shared_gate=False), dense_act="clamped_swiglu",
+                            mixers={"attention": dict(qk_norm=True, rot_values=True),
+                                    "latent_attention": dict(gate="element", rot_layout="halves")}),
 }
 
 
@@ -334,6 +358,19 @@ def _mixer_params(own: Dict[str, Any], fixed: Dict[str, Any]) -> Dict[str, Any]:
             **{k: _mixer_params(own[k], v) for k, v in fixed.items() if isinstance(v, dict)}}
 
 
+def _owner(i: int, specs: List[LayerSpec]) -> int:
+    """The layer whose tensors layer i uses, through others that have none of their own."""
+    j, seen = i, set()
+    while specs[j].weights_of is not None:
+        seen.add(j)
+        j = specs[j].weights_of
+        if not 0 <= j < len(specs) or j in seen:
+            raise ValueError(f"layer {i} uses the weights of layer {j}, which has none of its own")
+    if dataclasses.replace(specs[i], weights_of=None) != specs[j]:
+        raise ValueError(f"layer {i} uses the weights of layer {j}, which is of another kind or size")
+    return j
+
+
 def _mixer_model_kwargs(mt: str, d: Dict[str, Any]) -> Dict[str, Any]:
     """ModelConfig fields of a config.json that lists its layers (`layers`, `loop`, `norm`, `vocab`, `width`)."""
     design = _MIXER_DESIGNS[mt]
@@ -344,7 +381,12 @@ def _mixer_model_kwargs(mt: str, d: Dict[str, Any]) -> Dict[str, Any]:
         if kind is not None and kind not in design.feed_forwards:
             raise NotImplementedError(f"layer {i}: feed-forward kind {kind!r}")
         specs.append(LayerSpec(layer["type"], _mixer_params(layer["mixer"], design.mixers.get(layer["type"], {})),
-                               int(mlp["ff"]) if kind == "dense" else 0, _moe_spec(mlp, design) if kind == "moe" else None, design.gated))
+                               int(mlp["ff"]) if kind == "dense" else 0, _moe_spec(mlp, design) if kind == "moe" else None, design.gated,
+                               design.dense_act if kind == "dense" else "", float(mlp["limit"]) if kind == "dense" and design.dense_act else 0.0,
+                               int(layer["weights_of"]) if layer.get("weights_of") is not None else None))
+    owners = [_owner(i, specs) for i in range(len(specs))]
+    for i, j in enumerate(owners):
+        specs[i].weights_of = j if j != i else None
     loop = d.get("loop")
     if loop is not None:
         loop = (int(loop["start"]), int(loop["stop"]), int(loop["times"]))

@@ -114,11 +114,11 @@ class StepInputs:
     seg_seq: Optional[torch.Tensor] = None
     seg_q0: Optional[torch.Tensor] = None
     seg_len: int = 0
-    # latent attention over prompts: 128-query tiles (sequence, first query), and the contexts of the prefill sequences laid end to end
+    # latent attention over prompts: 128-query tiles (sequence, first query), and per window of the model's layers (0: none) the contexts
+    # that the prefill sequences can see laid end to end: ([B + 1] first row of every sequence, rows)
     q128_seq: Optional[torch.Tensor] = None
     q128_q0: Optional[torch.Tensor] = None
-    ctx_off: Optional[torch.Tensor] = None           # [B + 1]
-    ctx_total: int = 0
+    contexts: Optional[Dict[int, tuple]] = None
 
     def decode_view(self, T: int):
         """(decode rows, their block tables, state slots, context lengths) of a step over T rows."""
@@ -154,9 +154,12 @@ class DecoderModel:
         self.schedule = c.layer_schedule         # layer of every run (a looped layer runs several times, each with its own cache)
         self.mixed = c.layer_specs is not None   # layers with mixers of their own (models/mixers.py) on an fp32 residual stream
         self.recurrent = False
+        self.context_windows: List[int] = []     # of the latent attention layers
         if self.mixed:
             from .mixers import make_mixer
-            self.recurrent = any(make_mixer(sp, c.hidden_size).recurrent for sp in c.layer_specs)
+            mixers = [make_mixer(sp, c.hidden_size) for sp in c.layer_specs]
+            self.recurrent = any(m.recurrent for m in mixers)
+            self.context_windows = sorted({m.window for m in mixers if m.gathers_context})
         self.inter = c.intermediate_size // ws if not c.is_moe else c.intermediate_size
         self.hidden = c.hidden_size
         self.vocab = c.vocab_size
@@ -166,6 +169,7 @@ class DecoderModel:
         self.layers: List[LayerWeights] = []
         self.embed: Optional[torch.Tensor] = None
         self.pos_embed: Optional[torch.Tensor] = None
+        self.bigram_embed: Optional[torch.Tensor] = None        # [buckets + 1, hidden], the last row for a sequence's first token
         self.embed_norm: Optional[torch.Tensor] = None          # BLOOM normalises the embeddings
         self.embed_norm_b: Optional[torch.Tensor] = None
         self.alibi_slopes: Optional[torch.Tensor] = None        # [local heads] fp32 (BLOOM, MPT)
@@ -220,7 +224,7 @@ class DecoderModel:
         return min([lw.mixer.parallelism for lw in self.layers if lw.mixer.recurrent] + [1 << 20])
 
     def cache_shapes(self) -> Optional[List[dict]]:
-        """What every layer run keeps (`Mixer.cache_shape`), or None for the uniform key/value cache."""
+        """What every layer run keeps (`Mixer.cache_shape`), behind them what the embedding keeps; None for the uniform key/value cache."""
         if not self.mixed:
             return None
         shapes, run_of = [], {}
@@ -228,7 +232,7 @@ class DecoderModel:
             shape = self.layers[li].mixer.cache_shape(self)
             shapes.append({"share": run_of[shape["share_layer"]]} if "share_layer" in shape else shape)      # (its latest run so far)
             run_of[li] = run
-        return shapes
+        return shapes + ([{"ids": True}] if self.config.bigram else [])
 
     # ------------------------------------------------------------------ shapes
     @property
@@ -534,6 +538,8 @@ class DecoderModel:
                 return self._forward_post(inp, kv_cache)
             if c.layer_style == "pre":
                 return self._forward_pre(inp, kv_cache)
+            if c.layer_style == "sandwich":
+                return self._forward_sandwich(inp, kv_cache)
             # fp32 residual stream; every layer hands its contribution to the norm that reads the stream next
             residual, pending = ops.embed_stream(inp.input_ids, self.embed, c.embedding_multiplier), None
             for run, li in enumerate(self.schedule):
@@ -604,6 +610,18 @@ class DecoderModel:
         hidden = ops.norm_stream(residual, pending[0], self.final_norm, self.eps, c.norm_weight_offset, self.hidden, self.dtype, pairs=pending[1],
                                  rows=inp.lm_head_indices)
         return self._score(hidden, inp, selected=True)
+
+    def _forward_sandwich(self, inp: StepInputs, kv_cache) -> torch.Tensor:
+        """Norms on both sides of every sublayer: what a sublayer adds is normed, added and the stream normed for the next one in one pass."""
+        c, ops = self.config, self.ops
+        bigram = (self.bigram_embed, c.bigram, kv_cache[len(self.schedule)], inp) if c.bigram else None
+        residual = ops.embed_stream(inp.input_ids, self.embed, c.embedding_multiplier, bigram=bigram)
+        norms = [self.layers[li].norm1 for li in self.schedule] + [self.final_norm]
+        h = ops.norm_stream(residual, None, norms[0], self.eps, c.norm_weight_offset, self.hidden, self.dtype)
+        for run, li in enumerate(self.schedule):
+            rows = inp.lm_head_indices if run + 1 == len(self.schedule) else None
+            h = self.layers[li].forward(self, residual, h, inp, kv_cache[run], norms[run + 1], rows)
+        return self._score(h, inp, selected=True)
 
     def _score(self, hidden: torch.Tensor, inp: StepInputs, selected: bool = False) -> torch.Tensor:
         """Logits of the rows the step asks for (`selected`: `hidden` holds only those)."""

@@ -1,10 +1,12 @@
-"""Layers of designs that list their layers one by one, over an fp32 residual stream.  Three styles:
+"""Layers of designs that list their layers one by one, over an fp32 residual stream.  Four styles:
 
   parallel   a token mixer and an optional gated feed-forward side by side, both reading one RMS norm of the stream (`MixerLayer`)
   pre        the mixer, then the feed-forward (dense or routed experts), each reading an RMS norm of the stream of its own
              (`PreNormLayer`)
   post       the mixer, then the feed-forward (dense or routed experts), each reading the stream itself; the norm of its output is
              added to the stream (`PostNormLayer`)
+  sandwich   the mixer, then the feed-forward, each reading an RMS norm of the stream of its own; its output, times the sigmoid of a
+             projection of its input, goes through a second norm and is added (`SandwichLayer`)
 
 A mixer declares its tensors (`shapes`), what it keeps per token or per request (`cache_shape`), which of its projections read the
 layer's input (`in_parts`, one GEMM; in a parallel layer together with the feed-forward's gate and up projections) and its output
@@ -16,9 +18,11 @@ channel stays exactly zero through every operation.
   lightning         linear attention, one constant decay per head, state [heads, dim, vdim] per request
   wkv               token-shifted linear recurrence with a data-dependent decay per key channel, state [heads, dim, dim] per request
                     plus the previous token's input
-  latent_attention  softmax attention over a low-rank latent and one shared rotated key part per token, both paged
+  latent_attention  softmax attention over a low-rank latent and one shared rotated key part per token, both paged; with or without a
+                    low-rank query, a sliding window, an output gate per head or per element
   attention         grouped-query softmax attention over paged keys and values, with a choice of normed queries and keys, short
-                    convolutions, rotation, capped scores, sliding window, sink, output gate, keys and values of another layer
+                    convolutions, rotation, rotated values, capped scores, sliding window, sink, output gate, keys and values of another
+                    layer
   mamba2            selective state space recurrence behind a short convolution, state [heads, state, vdim] per request, gated norm
   parallel          two mixers that read the same rows, their outputs weighted and added
 """
@@ -65,6 +69,8 @@ class Mixer:
     model's dtype and device, `vec` a vector to fp32 on the device."""
 
     recurrent = False                                        # keeps something per request
+    window = 0                                               # tokens that attention sees (0: all)
+    gathers_context = False                                  # prompts are attended to over their contexts laid end to end
     parallelism = 1 << 20                                    # thread blocks that one sequence gives the recurrence kernels
 
     def __init__(self, params: dict, width: int):
@@ -185,67 +191,99 @@ class WkvMixer(Mixer):
 
 
 class LatentAttentionMixer(Mixer):
+    """What a design has of the following is a parameter:
+
+      q_rank      queries come from a normed latent of this rank of their own (none: from the layer's input)
+      mask.size   token i sees the last `size` tokens including itself (no mask: all before it)
+      rot_layout  "interleaved": pairs of neighbours; "halves": dimension i with i + rot_dim / 2.  Scores do not change when the rotated
+                  dimensions of queries and keys are put in another order, so halves are brought to pairs when the weights are loaded
+      gate        the heads times sigmoid of a projection of the input: one number per "head" or one per "element" """
+
+    gathers_context = True
+
     def __init__(self, params: dict, width: int):
         super().__init__(params, width)
         p = params
         self.H, self.d, self.rot, self.dv = int(p["heads"]), int(p["dim"]), int(p["rot_dim"]), int(p["vdim"])
-        self.q_rank, self.kv_rank, self.scale = int(p["q_rank"]), int(p["kv_rank"]), float(p["scale"])
-        self.rot_base = float(p["rot"]["base"])
-        if int(p["rot"].get("dims", self.rot)) != self.rot:
+        self.q_rank, self.kv_rank, self.scale = int(p.get("q_rank") or 0), int(p["kv_rank"]), float(p["scale"])
+        self.rot_spec, mask = p["rot"], p.get("mask")
+        if int(self.rot_spec.get("dims", self.rot)) != self.rot:
             raise NotImplementedError("latent attention rotates the whole rotated key part")
+        if self.rot % 2:
+            raise ValueError(f"rotation of {self.rot} dimensions")
+        self.window = int(mask["size"]) if mask else 0
+        if mask and self.window < 1:
+            raise ValueError(f"a window of {self.window} tokens")
+        self.gate, self.layout = p.get("gate", "head"), p.get("rot_layout", "interleaved")
         self.dp, self.rp, self.dvp = pad16(self.d), pad16(self.rot), pad16(self.dv)
         self.qrp, self.kvp, self.gp = pad16(self.q_rank), pad16(self.kv_rank), pad16(self.H)
+        self.head = self.dp + self.rp
         self.out_dim = self.H * self.dvp
 
     def shapes(self):
         H, d, r, dv, w = self.H, self.d, self.rot, self.dv, self.width
-        return {"dq": (self.q_rank, w), "dq.norm": (self.q_rank,), "uq": (H * (d + r), self.q_rank), "dkv": (self.kv_rank + r, w),
-                "dkv.norm": (self.kv_rank,), "uk": (H * d, self.kv_rank), "uv": (H * dv, self.kv_rank), "g": (H, w), "o": (w, H * dv)}
+        q = ({"dq": (self.q_rank, w), "dq.norm": (self.q_rank,), "uq": (H * (d + r), self.q_rank)} if self.q_rank else {"q": (H * (d + r), w)})
+        return {**q, "dkv": (self.kv_rank + r, w), "dkv.norm": (self.kv_rank,), "uk": (H * d, self.kv_rank), "uv": (H * dv, self.kv_rank),
+                "g": (H if self.gate == "head" else H * dv, w), "o": (w, H * dv)}
+
+    def _pairs(self, t):
+        """Rows of a rotated part [..., rot, n] in the order of interleaved pairs."""
+        return t if self.layout == "interleaved" else t[..., torch.arange(self.rot).view(2, -1).t().reshape(-1), :]
+
+    def _q_rows(self, t, cols):
+        """Rows of every query head, unrotated and rotated part padded on their own."""
+        t = t.view(self.H, self.d + self.rot, -1)
+        return torch.cat([_pad_to(t[:, : self.d], self.H, self.dp, cols), _pad_to(self._pairs(t[:, self.d:]), self.H, self.rp, cols)],
+                         1).reshape(self.H * self.head, cols)
 
     def in_parts(self, get):
         dkv, W = get("dkv"), self.W
-        dkv = torch.cat([_pad_to(dkv[: self.kv_rank], self.kvp, W), _pad_to(dkv[self.kv_rank:], self.rp, W)])
-        return [("dq", _pad_to(get("dq"), self.qrp, W)), ("dkv", dkv), ("g", _pad_to(get("g"), self.gp, W))]
+        dkv = torch.cat([_pad_to(dkv[: self.kv_rank], self.kvp, W), _pad_to(self._pairs(dkv[self.kv_rank:]), self.rp, W)])
+        g = _pad_to(get("g"), self.gp, W) if self.gate == "head" else pad_heads_rows(get("g"), self.H, self.dv, W)
+        q = ("dq", _pad_to(get("dq"), self.qrp, W)) if self.q_rank else ("q", self._q_rows(get("q"), W))
+        return [q, ("dkv", dkv), ("g", g)]
 
     def out_part(self, get):
         return pad_heads_cols(get("o"), self.H, self.dv, self.W)
 
     def load(self, get, fin, vec, model):
-        H, d, r, dv = self.H, self.d, self.rot, self.dv
-        uq = get("uq").view(H, d + r, self.q_rank)
-        self.uq = fin(torch.cat([_pad_to(uq[:, :d], H, self.dp, self.qrp), _pad_to(uq[:, d:], H, self.rp, self.qrp)], 1)
-                      .reshape(H * (self.dp + self.rp), self.qrp))
+        H, d, dv = self.H, self.d, self.dv
+        if self.q_rank:
+            self.uq, self.dq_norm = fin(self._q_rows(get("uq"), self.qrp)), vec(_pad_to(get("dq.norm"), self.qrp))
         self.uk_t = fin(_pad_to(get("uk").view(H, d, self.kv_rank).transpose(1, 2), H, self.kvp, self.dp))     # [H, kv_rank, dim]
         self.uv = fin(_pad_to(get("uv").view(H, dv, self.kv_rank), H, self.dvp, self.kvp))                     # [H, vdim, kv_rank]
         # the expansion of prompts: every head's key rows, then its value rows
         self.ukv = fin(torch.cat([_pad_to(get("uk").view(H, d, self.kv_rank), H, self.dp, self.kvp),
                                   _pad_to(get("uv").view(H, dv, self.kv_rank), H, self.dvp, self.kvp)], 1)
                        .reshape(H * (self.dp + self.dvp), self.kvp))
-        self.dq_norm = vec(_pad_to(get("dq.norm"), self.qrp))
         self.dkv_norm = vec(_pad_to(get("dkv.norm"), self.kvp))
-        self.cos_sin = model.rope_table(self.rot, self.rot_base)
+        self.cos_sin = model.rope_table(self.rot, float(self.rot_spec["base"]), self.rot_spec.get("scaling"))
 
     def cache_shape(self, model):
         return {"paged": self.kvp + self.rp}
 
     def run(self, model, h, proj, y, inp, cache):
         ops = model.ops
-        head = self.dp + self.rp
-        cq = ops.latent_prep(proj["dq"], proj["dkv"], self.dq_norm, self.dkv_norm, self.q_rank, self.kv_rank, self.rot, model.eps,
-                             self.cos_sin, inp.positions, inp.slots, cache)
-        q = ops.gemm(cq, self.uq)
-        ops.rope_pairs(q, inp.positions, self.cos_sin, self.H, head, self.dp, self.rot)
-        gate = proj["g"]
-        if inp.is_prefill and ops.latent_prefill(q, cache, self.ukv, gate, y, self.H, self.dp, self.rp, self.dvp, self.scale, inp, inp.n_decode):
+        prep = lambda dq, norm, **q: ops.latent_prep(dq, proj["dkv"], norm, self.dkv_norm, self.q_rank, self.kv_rank, self.rot, model.eps, self.cos_sin,
+                                                     inp.positions, inp.slots, cache, **q)
+        if self.q_rank:
+            q = ops.gemm(prep(proj["dq"], self.dq_norm), self.uq)
+            ops.rope_pairs(q, inp.positions, self.cos_sin, self.H, self.head, self.dp, self.rot)
+        else:
+            q = proj["q"]
+            prep(None, None, q=q, heads=self.H, head=self.head, off=self.dp)
+        gate, wide = proj["g"], self.gate == "element"
+        if inp.is_prefill and ops.latent_prefill(q, cache, self.ukv, gate, y, self.H, self.dp, self.rp, self.dvp, self.scale, inp, inp.n_decode,
+                                                 window=self.window, wide_gate=wide):
             if inp.n_decode == 0:
                 return
             inp = inp.decode_rows()                          # the decode rows of a mixed step are left
             n = inp.input_ids.shape[0]
             q, gate, y = q[:n], gate[:n], y[:n]
         q_lat = torch.empty(q.shape[0], self.H * self.kvp, dtype=q.dtype, device=q.device)
-        ops.gemm_heads(q, self.uk_t, q_lat, head)
-        o_lat = ops.latent_attn(q_lat, q, cache, self.H, self.kvp, head, self.dp, self.rp, self.scale, inp)
-        ops.gemm_heads(o_lat, self.uv, y, self.kvp, gate=gate)
+        ops.gemm_heads(q, self.uk_t, q_lat, self.head)
+        o_lat = ops.latent_attn(q_lat, q, cache, self.H, self.kvp, self.head, self.dp, self.rp, self.scale, inp, window=self.window)
+        ops.gemm_heads(o_lat, self.uv, y, self.kvp, gate=gate, wide_gate=wide)
 
 
 class AttentionMixer(Mixer):
@@ -255,7 +293,8 @@ class AttentionMixer(Mixer):
       qk_norm     queries and keys divided by their root mean square per head (weights shared by the heads)
       bias        biases of the projections
       conv        short causal convolution of this many taps on every channel of q, k and v, in front of the rotation
-      rot         rotation of the first `dims` dimensions of q and k, interleaved pairs, `base`, optionally YaRN `scaling`
+      rot         rotation of the first `dims` dimensions of q and k, interleaved pairs, `base`, optionally `scaling` of the frequencies
+      rot_values  values rotated by their position over all `vdim` dimensions (`base`, no scaling), the result back by the query's
       softcap     scores s become softcap * tanh(s / softcap)
       sink        "learned": a score per head that only the denominator contains; "unit": the denominator plus one
       gate        the heads times sigmoid of a projection of the same input
@@ -276,15 +315,19 @@ class AttentionMixer(Mixer):
             raise ValueError(f"a window of {self.window} tokens")
         self.sign, self.scale = (-1.0 if self.scale < 0 else 1.0), abs(self.scale)      # (the kernels take scores that grow with the products)
         self.softcap, self.out_scale = float(params.get("softcap") or 0.0), float(params.get("out_scale", 1.0))
-        self.qk_norm, self.bias, self.gate = (bool(params.get(n)) for n in ("qk_norm", "bias", "gate"))
+        self.qk_norm, self.bias, self.gate, self.rot_values = (bool(params.get(n)) for n in ("qk_norm", "bias", "gate", "rot_values"))
         self.taps, self.kv_from = int(params.get("conv") or 0), params.get("kv_from")
         self.rot_dims = int(self.rot["dims"]) if self.rot else 0
         if self.rot_dims % 2 or self.rot_dims > self.d:
             raise ValueError(f"rotation of {self.rot_dims} of {self.d} dimensions")
         if self.taps > self.MAX_TAPS:
             raise NotImplementedError(f"convolutions of {self.taps} taps (up to {self.MAX_TAPS})")
-        if self.qk_norm and (self.taps or self.rot_dims or self.kv_from is not None):
-            raise NotImplementedError("normed queries and keys with a convolution, a rotation or another layer's keys")
+        if self.qk_norm and (self.taps or self.kv_from is not None):
+            raise NotImplementedError("normed queries and keys with a convolution or another layer's keys")
+        if self.rot_values and not self.qk_norm:
+            raise NotImplementedError("rotated values without normed queries and keys")
+        if self.rot_values and self.dv % 2:
+            raise ValueError(f"rotation of {self.dv} dimensions")
         if self.kv_from is not None and self.taps:
             raise NotImplementedError("another layer's keys with a convolution")
         self.recurrent = self.taps > 1
@@ -344,6 +387,7 @@ class AttentionMixer(Mixer):
         if self.taps:                                        # [taps, channels]
             self.conv_w = vec(torch.cat([self._rows(get(n + ".conv"), heads, d, dp, self.taps) for n, heads, d, dp in self.projections]).t())
         self.cos_sin = model.rope_table(self.rot_dims, float(self.rot["base"]), self.rot.get("scaling")) if self.rot_dims else None
+        self.v_cos_sin = model.rope_table(self.dv, float(self.rot["base"])) if self.rot_values else None
         if self.kv_from is not None:
             self._check_source(model)
 
@@ -370,12 +414,13 @@ class AttentionMixer(Mixer):
             conv, cache = cache.get("conv"), cache["kv"] if "kv" in cache else cache["left"]
         if self.qk_norm:
             q = qkv
-            ops.qk_norm_kvwrite(qkv, self.H, self.G, self.dp, self.dvp, self.d, self.q_norm, self.k_norm, model.eps, cache, inp.slots)
+            ops.qk_norm_kvwrite(qkv, self.H, self.G, self.dp, self.dvp, self.d, self.q_norm, self.k_norm, model.eps, cache, inp.slots,
+                                positions=inp.positions, cos_sin=self.cos_sin, v_cos_sin=self.v_cos_sin)
         else:
             own = self.G if self.kv_from is None else 0
             q = ops.conv_rope_kvwrite(qkv, self.H, own, self.dp, self.dvp, self.cos_sin, self.rot_dims, inp.positions, cache, inp, self.conv_w, conv)
         ops.gqa_attn(q, cache, self.H, self.G, self.dp, self.dvp, self.scale, self.window, inp, y, softcap=self.softcap, sink=self.sinks,
-                     gate=proj.get("g"), out_scale=self.out_scale)
+                     gate=proj.get("g"), out_scale=self.out_scale, turn_back=self.v_cos_sin)
 
 
 class Mamba2Mixer(Mixer):
@@ -520,24 +565,36 @@ class MixerLayer:
 
 
 class DenseMlp:
-    """down(act(up(h))), or gated: down(act(gate(h)) * up(h))."""
+    """down(act(up(h))), or gated: down(act(gate(h)) * up(h)).  `act`: an activation of its own in place of the model's, with its limit."""
 
-    def __init__(self, ff: int, width: int, gated: bool):
+    def __init__(self, ff: int, width: int, gated: bool, act: str = "", limit: float = 0.0):
         self.ff, self.width, self.W, self.gated = ff, width, pad16(width), gated
         self.fp = pad16(ff)
         self.names = ("gate", "up") if gated else ("up",)
+        self.act, self.act_args = act, dict(limit=limit) if act else {}
 
     def shapes(self):
         return dict({n: (self.ff, self.width) for n in self.names}, down=(self.width, self.ff))
 
-    def load(self, get, fin, vec, model):
-        self.up = fin(torch.cat([_pad_to(get(n), self.fp, self.W) for n in self.names]))
+    def load(self, get, fin, vec, model, beside=None):
+        """`beside`: (weight [n, W], bias [n]) of a further projection of the same input, which rides in the first product."""
+        rows, self.up_b = [_pad_to(get(n), self.fp, self.W) for n in self.names], None
+        if beside is not None:
+            self.up_b = fin(torch.cat([torch.zeros(len(rows) * self.fp, device=beside[1].device), beside[1]]))
+            rows.append(beside[0])
+        self.up = fin(torch.cat(rows))
         self.down = fin(_pad_to(get("down"), self.W, self.fp))
 
     def run(self, model, h):
         """-> (rows, None): one row per token."""
-        ops = model.ops
-        return ops.gemm(ops.act_mul(ops.gemm(h, self.up), self.fp, model.config.hidden_act, gated=self.gated), self.down), None
+        return self.run_beside(model, h)[:2]
+
+    def run_beside(self, model, h):
+        """-> the same and the projection beside (or None)."""
+        ops, n = model.ops, len(self.names) * self.fp
+        u = ops.gemm(h, self.up, bias=self.up_b)
+        a = ops.act_mul(u, self.fp, self.act or model.config.hidden_act, gated=self.gated, **self.act_args)
+        return ops.gemm(a, self.down), None, u[:, n:] if self.up_b is not None else None
 
 
 class MoeMlp:
@@ -545,7 +602,7 @@ class MoeMlp:
     that the product's epilogue has both.  How the experts are chosen and weighted is in the MoeSpec.
 
     The shared expert is cut into slices of an expert's (padded) width; every token takes each slice with the weight
-    sigmoid(sg . h), so the slices ride in the grouped products as further experts, and `sg` is one more row of the router."""
+    sigmoid(sg . h), or one, so the slices ride in the grouped products as further experts, and `sg` is one more row of the router."""
 
     TILE = 128                                               # features per work item of the grouped products
 
@@ -565,15 +622,19 @@ class MoeMlp:
         out = {"router": (s.experts, w)}
         if s.score == "sigmoid":
             out["correction"] = (s.experts,)
+        if s.bias:
+            out["router.b"] = (s.experts,)
         for e in range(s.experts):
             out.update({f"e{e}.{n}": (s.ff, w) for n in self.names})
             out[f"e{e}.down"] = (w, s.ff)
         if s.shared_ff:
             out.update({f"shared.{n}": (s.shared_ff, w) for n in self.names})
-            out.update({"shared.down": (w, s.shared_ff), "shared.sg": (1, w)})
+            out["shared.down"] = (w, s.shared_ff)
+            if s.shared_gate:
+                out["shared.sg"] = (1, w)
         return out
 
-    def load(self, get, fin, vec, model):
+    def load(self, get, fin, vec, model, beside=None):
         s, n, step = self.spec, self.spec.experts + self.slices, len(self.names)
         if s.gated and model.config.hidden_act != "silu":
             raise NotImplementedError(f"gated experts with {model.config.hidden_act}")
@@ -591,19 +652,28 @@ class MoeMlp:
                 for j, up in enumerate(ups):
                     self.up[s.experts + i, j: step * (b - a): step, : self.width] = up[a:b]
                 self.down[s.experts + i, : self.width, : b - a] = down[:, a:b]
-            router.append(get("shared.sg"))
+            if s.shared_gate:
+                router.append(get("shared.sg"))
         self.router = fin(_pad_to(torch.cat(router), (s.experts + 8) // 8 * 8, self.W))      # (whole tiles of the router kernel)
         self.correction = vec(get("correction")) if s.score == "sigmoid" else None
+        self.router_b = vec(get("router.b")) if s.bias else None
+        self.beside = (fin(beside[0]), fin(beside[1])) if beside is not None else None
 
     def run(self, model, h):
         """-> (rows of every (token, expert) pair, (row, weight) of each token's pairs)."""
+        return self.run_beside(model, h)[:2]
+
+    def run_beside(self, model, h):
+        """-> the same and the projection beside (or None)."""
         s, ops = self.spec, model.ops
         r = ops.moe_route(h, self.router, s.top, 0, s.experts, experts=s.experts, score=s.score, correction=self.correction, groups=s.groups,
-                          keep=s.keep, scale=s.scale, shared=self.slices, group_top=s.group_top, renorm=s.renorm)
+                          keep=s.keep, scale=s.scale, shared=self.slices, group_top=s.group_top, renorm=s.renorm, bias=self.router_b,
+                          shared_gate=s.shared_gate)
         avg = max(1, (h.shape[0] * s.top + s.experts - 1) // s.experts)
         a = ops.moe_grouped_gemm(r.xg, self.up, r.seg, avg, shared=self.slices, tokens=h.shape[0],
                                  act="swiglu" if s.gated else model.config.hidden_act)
-        return ops.moe_grouped_gemm(a, self.down, r.seg, avg), (r.pos, r.topk_w)
+        beside = ops.gemm(h, self.beside[0], bias=self.beside[1]) if self.beside is not None else None
+        return ops.moe_grouped_gemm(a, self.down, r.seg, avg), (r.pos, r.topk_w), beside
 
 
 @dataclass
@@ -657,10 +727,47 @@ class PostNormLayer:
         return h
 
 
+@dataclass
+class SandwichLayer:
+    """x += scale1 * norm1b(mixer(norm1(x)) * gate1), then x += scale2 * norm2b(ff(norm2(x)) * gate2), a gate being the sigmoid of a
+    projection (with bias) of what its sublayer reads.  The gates' projections ride in the products that read the same rows.  The stream
+    is fp32; `h` is its norm that the next sublayer reads, written by whoever last added to the stream."""
+    mixer: Mixer
+    mlp: Optional[object]                                    # DenseMlp, MoeMlp or None
+    norm1: torch.Tensor = None                               # fp32 [W]
+    norm2: Optional[torch.Tensor] = None
+    add1: torch.Tensor = None                                # fp32 [W]: weight of the output's norm times the layer scale
+    add2: Optional[torch.Tensor] = None
+    in_w: Optional[torch.Tensor] = None                      # [rows, W]
+    in_b: Optional[torch.Tensor] = None                      # [rows]
+    out_w: Optional[torch.Tensor] = None                     # [W, mixer out_dim]
+    parts: Dict[str, Tuple[int, int]] = field(default_factory=dict)
+
+    def forward(self, model, residual, h, inp, cache, next_norm, rows=None):
+        """Adds both sublayers to `residual`; -> its norm by `next_norm` (of `rows` only when given: the stream's other rows are then
+        not needed any more)."""
+        ops, m, c = model.ops, self.mixer, model.config
+        add = lambda y, w, gate, nxt, rows, pairs=None: ops.norm_add(residual, y, w, None, c.residual_multiplier, model.eps, model.hidden, model.dtype,
+                                                                     layernorm=False, pairs=pairs, gate=gate, next_weight=nxt, rows=rows)
+        proj = ops.gemm(h, self.in_w, bias=self.in_b)
+        views = {n: proj[:, a:b] for n, (a, b) in self.parts.items()}
+        y = torch.empty(h.shape[0], m.out_dim, dtype=h.dtype, device=h.device)
+        m.run(model, h, views, y, inp, cache)
+        y, gate = ops.gemm(y, self.out_w), views.get("residual_gate")
+        if self.mlp is None:
+            return add(y, self.add1, gate, next_norm, rows)
+        h = add(y, self.add1, gate, self.norm2, None)
+        y, pairs, gate = self.mlp.run_beside(model, h)
+        return add(y, self.add2, gate, next_norm, rows, pairs)
+
+
+LAYER_KINDS = {"pre": PreNormLayer, "post": PostNormLayer, "sandwich": SandwichLayer}
+
+
 def make_mlp(spec, width: int):
     if spec.moe is not None:
         return MoeMlp(spec.moe, width)
-    return DenseMlp(spec.ff, width, spec.gated) if spec.ff else None
+    return DenseMlp(spec.ff, width, spec.gated, spec.act, spec.limit) if spec.ff else None
 
 
 def _parts(layer, rows):
@@ -673,7 +780,9 @@ def _parts(layer, rows):
 
 def load_mixer_layers(m, w):
     """Tensors of a layer-by-layer checkpoint -> `m` (a DecoderModel): `embed`, `pos`, `l<i>.norm1`, `l<i>.norm2`, `l<i>.mix.*`,
-    `l<i>.mlp.*`, `final.norm`, `head`; a layer norm's bias is called like its weight with `.b` added."""
+    `l<i>.mlp.*`, `final.norm`, `head`; a layer norm's bias is called like its weight with `.b` added.  Also, where the design has them:
+    `bigram`; `l<i>.norm1b`, `l<i>.norm2b` (norms of the sublayers' outputs), `l<i>.ls1`, `l<i>.ls2` (their scale) and `l<i>.rg1`, `l<i>.rg2`
+    with `.b` (their gate)."""
     c, dt, dev = m.config, m.dtype, m.device
     if m.tp.world_size > 1:
         raise ValueError(f"{c.model_type} is served on one shard")
@@ -690,21 +799,36 @@ def load_mixer_layers(m, w):
 
     m.embed = fin(_pad_to(get("embed"), c.vocab_size, W))
     m.lm_head = fin(_pad_to(get("head"), pad16(c.vocab_size), W))
-    m.final_norm = vec(_pad_to(get("final.norm"), W))
+    stream_vec = lambda t: vec(_pad_to(t.expand(c.hidden_size), W))          # (a single number counts for every column)
+    m.final_norm = stream_vec(get("final.norm"))
+    if c.bigram:
+        m.bigram_embed = fin(_pad_to(get("bigram"), c.bigram[0] + 1, W))
     if c.learned_positions:
         m.pos_embed = fin(_pad_to(get("pos"), c.max_position_embeddings, W))
     if c.norm_type == "layernorm":
         m.final_norm_b = vec(_pad_to(get("final.norm.b"), W))
     m.layers = []
-    if c.layer_style in ("pre", "post"):
-        norm = lambda name: vec(_pad_to(get(name), W))
+    if c.layer_style in LAYER_KINDS:
+        norm = lambda name: stream_vec(get(name))
         if c.layer_style == "post":
             norm = lambda name: (vec(_pad_to(get(name), W)), vec(_pad_to(get(name + ".b"), W)))
         for i, spec in enumerate(c.layer_specs):
-            kind = PreNormLayer if c.layer_style == "pre" else PostNormLayer
-            layer = kind(make_mixer(spec, c.hidden_size), make_mlp(spec, c.hidden_size), norm(f"l{i}.norm1"))
+            if spec.weights_of is not None:
+                m.layers.append(None)
+                continue
+            layer = LAYER_KINDS[c.layer_style](make_mixer(spec, c.hidden_size), make_mlp(spec, c.hidden_size), norm(f"l{i}.norm1"))
             sub = lambda name, i=i: get(f"l{i}.mix.{name}")
             rows, bias = layer.mixer.in_parts(sub), layer.mixer.in_bias(sub)
+            beside = None
+            if c.layer_style == "sandwich":
+                out_norm = lambda n, i=i: stream_vec(get(f"l{i}.norm{n}b") * (get(f"l{i}.ls{n}") if c.layer_scale else 1.0))
+                layer.add1 = out_norm(1)
+                if c.residual_gate:
+                    gate = lambda n, i=i: (_pad_to(get(f"l{i}.rg{n}"), W, W), _pad_to(get(f"l{i}.rg{n}.b"), W))
+                    w_gate, bias["residual_gate"] = gate(1)
+                    rows.append(("residual_gate", w_gate))
+                if layer.mlp is not None:
+                    layer.add2, beside = out_norm(2), gate(2) if c.residual_gate else None
             _parts(layer, rows)
             layer.in_w, layer.out_w = fin(torch.cat([t for _, t in rows])), fin(layer.mixer.out_part(sub))
             if bias:
@@ -712,8 +836,11 @@ def load_mixer_layers(m, w):
             layer.mixer.load(sub, fin, vec, m)
             if layer.mlp is not None:
                 layer.norm2 = norm(f"l{i}.norm2")
-                layer.mlp.load(lambda name, i=i: get(f"l{i}.mlp.{name}"), fin, vec, m)
+                layer.mlp.load(lambda name, i=i: get(f"l{i}.mlp.{name}"), fin, vec, m, **(dict(beside=beside) if beside is not None else {}))
             m.layers.append(layer)
+        for i, spec in enumerate(c.layer_specs):
+            if spec.weights_of is not None:
+                m.layers[i] = m.layers[spec.weights_of]
         return
     for i, spec in enumerate(c.layer_specs):
         mx = make_mixer(spec, c.hidden_size)
@@ -735,18 +862,27 @@ def load_mixer_layers(m, w):
 def tensor_shapes(c) -> Dict[str, Tuple[int, ...]]:
     """Name -> shape of every tensor of a layer-by-layer checkpoint of this configuration."""
     w = c.hidden_size
-    out = {"embed": (c.vocab_size, w), "head": (c.vocab_size, w), "final.norm": (w,)}
-    if c.layer_style in ("pre", "post"):
+    stream = () if c.norm_scalar else (w,)
+    out = {"embed": (c.vocab_size, w), "head": (c.vocab_size, w), "final.norm": stream}
+    if c.bigram:
+        out["bigram"] = (c.bigram[0] + 1, w)
+    if c.layer_style in LAYER_KINDS:
         if c.learned_positions:
             out["pos"] = (c.max_position_embeddings, w)
         if c.norm_type == "layernorm":
             out["final.norm.b"] = (w,)
         for i, spec in enumerate(c.layer_specs):
+            if spec.weights_of is not None:
+                continue
             mlp = make_mlp(spec, w)
-            for norm in ("norm1",) + (("norm2",) if mlp is not None else ()):
-                out[f"l{i}.{norm}"] = (w,)
+            for n in (1, 2) if mlp is not None else (1,):
+                out[f"l{i}.norm{n}"] = stream
                 if c.norm_type == "layernorm":
-                    out[f"l{i}.{norm}.b"] = (w,)
+                    out[f"l{i}.norm{n}.b"] = (w,)
+                if c.layer_style == "sandwich":
+                    out[f"l{i}.norm{n}b"] = stream
+                    out.update({f"l{i}.ls{n}": (w,)} if c.layer_scale else {})
+                    out.update({f"l{i}.rg{n}": (w, w), f"l{i}.rg{n}.b": (w,)} if c.residual_gate else {})
             out.update({f"l{i}.mix.{n}": s for n, s in make_mixer(spec, w).shapes().items()})
             out.update({f"l{i}.mlp.{n}": s for n, s in (mlp.shapes() if mlp is not None else {}).items()})
         return out
@@ -781,7 +917,7 @@ class RandomWeights:
             return 1.0 + 0.1 * t
         if leaf == "w0":
             return -2.0 + 1.5 * t
-        if leaf in ("norm1", "norm2", "norm"):
+        if leaf in ("norm1", "norm2", "norm", "norm1b", "norm2b", "ls1", "ls2"):
             return self.plain_norm + 0.1 * t
         if leaf == "b":
             return 0.1 * t
@@ -795,4 +931,4 @@ class RandomWeights:
             return -1.5 + t
         if leaf == "sink":
             return t
-        return t if name in ("embed", "pos") else t * shape[-1] ** -0.5
+        return t if name in ("embed", "pos", "bigram") else t * shape[-1] ** -0.5

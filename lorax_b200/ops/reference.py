@@ -168,10 +168,20 @@ def _act(x, act):
     raise ValueError(act)
 
 
-def act_mul(x, inter, act="silu", gated=True, out=None):
-    g = _act(x[:, :inter].float(), act)
-    if gated:
-        g = g * x[:, inter: 2 * inter].float()
+CLAMPED_SWIGLU_ALPHA = 1.702
+
+
+def act_mul(x, inter, act="silu", gated=True, out=None, limit: float = 0.0):
+    """act(gate) * up of rows [gate | up], or act(gate).  "clamped_swiglu" (gated): gate at most `limit`, up within +-limit,
+    gate * sigmoid(1.702 gate) * (up + 1)."""
+    g = x[:, :inter].float()
+    if act == "clamped_swiglu":
+        g = g.clamp(max=limit)
+        g = g * torch.sigmoid(CLAMPED_SWIGLU_ALPHA * g) * (x[:, inter: 2 * inter].float().clamp(-limit, limit) + 1.0)
+    else:
+        g = _act(g, act)
+        if gated:
+            g = g * x[:, inter: 2 * inter].float()
     g = g.to(x.dtype)
     if out is not None:
         out.copy_(g)
@@ -317,6 +327,15 @@ def prefill_tiles(q_lens, tile: int = 64):
             seq.append(b)
             q0.append(s)
     return seq, q0
+
+
+def context_offsets(cache_lens, q_lens, window: int = 0):
+    """First rows of the sequences' contexts laid end to end, and their total: what precedes a portion of q tokens and can be seen from
+    it, then the portion (window: at most window - 1 tokens precede it)."""
+    off = [0]
+    for c, n in zip(cache_lens, q_lens):
+        off.append(off[-1] + (min(c, window - 1) if window else c) + n)
+    return off
 
 
 def lora_shrink(x, tok_slot, arena, slot_base, slot_rank, unit_off, nparts, max_rank, v=None):
@@ -465,10 +484,16 @@ def rope_table(rot: int, max_pos: int, base: float, device="cpu", scaling=None) 
     """[max_pos, rot] fp32: cos of position * base^(-2i / rot) in the first half, sin in the second; angles formed in fp64.  `scaling`
     (factor, original, fast, slow): YaRN, which divides the frequencies of pairs that turn less than `slow` times over `original`
     positions by `factor`, leaves those that turn more than `fast` times, goes linearly between, and multiplies cos and sin by
-    0.1 ln(factor) + 1."""
+    0.1 ln(factor) + 1.  `scaling` (factor, original, low, high): bands as in Llama 3.1, which divides the frequencies of pairs that turn less
+    than `low` times over `original` positions by `factor`, leaves those that turn more than `high` times, and blends between."""
     f = torch.pow(torch.tensor(float(base), dtype=torch.float64), -torch.arange(0, rot, 2, dtype=torch.float64) / rot)
     mult = 1.0
-    if scaling:
+    if scaling and "high" in scaling:
+        factor, low, high = float(scaling["factor"]), float(scaling["low"]), float(scaling["high"])
+        turns = float(scaling["original"]) * f / (2 * math.pi)
+        keep = ((turns - low) / (high - low)).clamp(0, 1) if high != low else (turns >= low).double()
+        f = torch.where(turns > high, f, torch.where(turns < low, f / factor, (1 - keep) * f / factor + keep * f))
+    elif scaling:
         factor, original = float(scaling["factor"]), float(scaling["original"])
         pair = lambda turns: rot * math.log(original / (2 * math.pi * turns)) / (2 * math.log(base))
         lo, hi = max(math.floor(pair(scaling["fast"])), 0), min(math.ceil(pair(scaling["slow"])), rot - 1)
@@ -479,11 +504,37 @@ def rope_table(rot: int, max_pos: int, base: float, device="cpu", scaling=None) 
     return (torch.cat([a.cos(), a.sin()], -1) * mult).float().to(device)
 
 
-def embed_stream(ids, table, mult=1.0, pos=None, positions=None, copy=None):
-    """table[ids] * mult (+ pos[positions]) in fp32; `copy` takes the same values in its own dtype."""
+def _tokens_before(ids, pages, inp):
+    """The token in front of every row's (-1: none), from the step itself or, in front of a sequence's first row, from the pages of token
+    ids [blocks, page]; the step's own ids are left there."""
+    T, page = ids.shape[0], pages.shape[1]
+    prev = torch.full((T,), -1, dtype=torch.int64, device=ids.device)
+    nd, dbt, _, ctx = inp.decode_view(T)
+    spans = [(i, 1, dbt[i], int(ctx[i]) - 1) for i in range(nd) if int(ctx[i]) > 0]
+    if inp.is_prefill:
+        cu = [int(c) for c in inp.cu_q]
+        spans += [(nd + cu[b], cu[b + 1] - cu[b], inp.block_tables[b], int(inp.cache_lens[b])) for b in range(len(cu) - 1) if cu[b + 1] > cu[b]]
+    for r0, n, bt, before in spans:
+        prev[r0 + 1: r0 + n] = ids[r0: r0 + n - 1].long()
+        if before > 0:
+            prev[r0] = pages[int(bt[(before - 1) // page]), (before - 1) % page].long()
+    ok = inp.slots >= 0
+    pages.view(-1)[inp.slots[ok].long()] = ids[ok].to(pages.dtype)
+    return prev
+
+
+def embed_stream(ids, table, mult=1.0, pos=None, positions=None, copy=None, bigram=None):
+    """table[ids] * mult (+ pos[positions]) in fp32; `copy` takes the same values in its own dtype.  bigram = (vectors [buckets + 1, W],
+    (buckets, mul_prev, mul_cur), pages of token ids, inp) adds the vector of (token before, token), the last one where none is before."""
+    ids = ids.clamp(0, table.shape[0] - 1)
     x = table[ids.long().clamp(0, table.shape[0] - 1)].float() * mult
     if pos is not None:
         x = x + pos[positions.long().clamp(0, pos.shape[0] - 1)].float()
+    if bigram is not None:
+        vectors, (buckets, mul_prev, mul_cur), pages, inp = bigram
+        prev = _tokens_before(ids, pages, inp)
+        row = (prev * mul_prev + ids.long() * mul_cur) % buckets
+        x = x + vectors[torch.where(prev < 0, torch.full_like(row, buckets), row)].float()
     if copy is not None:
         copy.copy_(x)
     return x
@@ -502,11 +553,16 @@ def _weighted_rows(y, pairs, W: int):
     return torch.einsum("tk,tkw->tw", torch.where(pos >= 0, w, torch.zeros_like(w)), y[pos.long().clamp(min=0)][:, :, :W].float())
 
 
-def norm_add(residual, y, weight, bias, mult: float, eps, n: int, dtype, layernorm: bool = True, pairs=None):
+def norm_add(residual, y, weight, bias, mult: float, eps, n: int, dtype, layernorm: bool = True, pairs=None, gate=None, next_weight=None,
+             rows=None):
     """residual (fp32, in place) += mult * norm(y) over the first `n` columns; returns the new residual in `dtype`.  With `pairs` =
-    (pos [T, k], w [T, k]) a token's y is the weighted sum of its rows pos (-1: none) of `y`."""
+    (pos [T, k], w [T, k]) a token's y is the weighted sum of its rows pos (-1: none) of `y`.  gate [T, W]: y times its sigmoid.
+    next_weight [W]: returns the new residual's RMS norm with this weight instead, of `rows` only when given (whether the residual's other
+    rows still take the addition is open)."""
     W = residual.shape[1]
     x = y[:, :W].float() if pairs is None else _weighted_rows(y, pairs, W)
+    if gate is not None:
+        x = x * torch.sigmoid(gate[:, :W].float())
     if layernorm:
         x = _layer_norm(x, weight, bias, eps, n)
     else:
@@ -514,6 +570,8 @@ def norm_add(residual, y, weight, bias, mult: float, eps, n: int, dtype, layerno
         if bias is not None:
             x = x + bias
     residual += mult * x
+    if next_weight is not None:
+        return norm_stream(residual, None, next_weight, eps, 0.0, n, dtype, rows=rows)
     return residual if dtype == torch.float32 else residual.to(dtype)
 
 
@@ -622,18 +680,22 @@ def _rotate_pairs(x, cos, sin):
     return torch.stack([u * cos - v * sin, v * cos + u * sin], -1).flatten(-2)
 
 
-def latent_prep(dq, dkv, dq_norm, dkv_norm, q_rank: int, kv_rank: int, rot: int, eps, cos_sin, positions, slots, cache):
+def latent_prep(dq, dkv, dq_norm, dkv_norm, q_rank: int, kv_rank: int, rot: int, eps, cos_sin, positions, slots, cache, q=None, heads: int = 0,
+                head: int = 0, off: int = 0):
     """Down-projections of latent attention -> normalised query latent [T, q_rank padded] (returned) and cache rows
-    [normalised key/value latent | rotated key part] (scattered into `cache` [blocks, page, kv_rank padded + rot padded])."""
-    dt = dq.dtype
-    qr, kr = dq_norm.shape[0], dkv_norm.shape[0]
+    [normalised key/value latent | rotated key part] (scattered into `cache` [blocks, page, kv_rank padded + rot padded]).  Without a query
+    latent (dq None) the columns [off, off + rot) of every head of q [T, heads * head] are rotated in place."""
+    dt = dkv.dtype
+    kr = dkv_norm.shape[0]
     page = cache.shape[1]
 
     def rms(x, n, w):
         x = x.float()
         return (x * torch.rsqrt((x * x).sum(-1, keepdim=True) / n + eps) * w).to(dt)
-    cq = rms(dq[:, :qr], q_rank, dq_norm)
-    row = torch.zeros(dq.shape[0], cache.shape[2], dtype=dt, device=dq.device)
+    cq = rms(dq[:, : dq_norm.shape[0]], q_rank, dq_norm) if dq is not None else None
+    if q is not None:
+        rope_pairs(q, positions, cos_sin, heads, head, off, rot)
+    row = torch.zeros(dkv.shape[0], cache.shape[2], dtype=dt, device=dkv.device)
     row[:, :kr] = rms(dkv[:, :kr], kv_rank, dkv_norm)
     cs = cos_sin[positions.long()]
     row[:, kr: kr + rot] = _rotate_pairs(dkv[:, kr: kr + rot], cs[:, : rot // 2], cs[:, rot // 2:]).to(dt)
@@ -647,35 +709,37 @@ def rope_pairs(x, positions, cos_sin, H: int, head: int, off: int, rot: int):
     """Rotates columns [off, off + rot) of every head (width `head`) of x [T, H * head] in place, interleaved pairs."""
     T = x.shape[0]
     cs = cos_sin[positions.long()]
-    part = x.view(T, H, head)[:, :, off: off + rot]
+    part = x[:, : H * head].unflatten(1, (H, head))[:, :, off: off + rot]
     part.copy_(_rotate_pairs(part, cs[:, None, : rot // 2], cs[:, None, rot // 2:]).to(x.dtype))
 
 
-def gemm_heads(x, w, out, x_head: int, gate=None):
+def gemm_heads(x, w, out, x_head: int, gate=None, wide_gate: bool = False):
     """Per-head products: head h of `out` (width N) = columns [h * x_head, h * x_head + K) of x times w[h]^T (w [H, N, K]),
-    optionally times sigmoid(gate[:, h])."""
+    optionally times sigmoid(gate[:, h]), or (wide_gate) times sigmoid of the gate column of every output column."""
     H, N, K = w.shape
     T = x.shape[0]
     xs = torch.stack([x[:, h * x_head: h * x_head + K] for h in range(H)], 1).float()
     y = torch.einsum("thk,hnk->thn", xs, w.float())
     if gate is not None:
-        y = y * torch.sigmoid(gate[:, :H].float())[:, :, None]
+        z = torch.sigmoid(gate[:, : H * N if wide_gate else H].float())
+        y = y * (z.view(T, H, N) if wide_gate else z[:, :, None])
     out[:, : H * N] = y.reshape(T, H * N).to(out.dtype)
     return out
 
 
-def latent_prefill(q, cache, w_ukv, gate, out, H: int, dk: int, rot: int, dv: int, scale: float, inp, nd: int) -> bool:
+def latent_prefill(q, cache, w_ukv, gate, out, H: int, dk: int, rot: int, dv: int, scale: float, inp, nd: int, window: int = 0,
+                   wide_gate: bool = False) -> bool:
     """The expanded form of prompt attention exists on the device only; False sends the rows through `latent_attn`."""
     return False
 
 
-def latent_attn(q_lat, q, cache, H: int, kv_rank: int, head: int, rot_off: int, rot: int, scale: float, inp):
+def latent_attn(q_lat, q, cache, H: int, kv_rank: int, head: int, rot_off: int, rot: int, scale: float, inp, window: int = 0):
     """Causal softmax attention in the latent space: head h's query is [q_lat[h] | q[h, rot_off : rot_off + rot]] against the
-    cached rows [latent | rotated key].  -> weighted latents [T, H * kv_rank]."""
+    cached rows [latent | rotated key], the last `window` of them (0: all).  -> weighted latents [T, H * kv_rank]."""
     T = q.shape[0]
     page = cache.shape[1]
     nd, dbt, _, ctx = inp.decode_view(T)
-    ql, qr = q_lat.view(T, H, kv_rank).float(), q.view(T, H, head)[:, :, rot_off: rot_off + rot].float()
+    ql, qr = q_lat.view(T, H, kv_rank).float(), q[:, : H * head].unflatten(1, (H, head))[:, :, rot_off: rot_off + rot].float()
     out = torch.zeros(T, H, kv_rank, dtype=q.dtype, device=q.device)
     spans = [(i, 1, dbt[i], int(ctx[i]) - 1) for i in range(nd) if int(ctx[i]) > 0]
     if inp.is_prefill:
@@ -685,8 +749,11 @@ def latent_attn(q_lat, q, cache, H: int, kv_rank: int, head: int, rot_off: int, 
         keys = before + n
         rows = cache[bt[: (keys + page - 1) // page].long()].reshape(-1, cache.shape[2])[:keys].float()
         s = torch.einsum("thc,sc->hts", ql[r0: r0 + n], rows[:, :kv_rank]) + torch.einsum("thc,sc->hts", qr[r0: r0 + n], rows[:, kv_rank: kv_rank + rot])
-        pos = torch.arange(before, keys, device=q.device)
-        s = (s * scale).masked_fill(torch.arange(keys, device=q.device)[None, None, :] > pos[None, :, None], float("-inf"))
+        pos, kp = torch.arange(before, keys, device=q.device)[:, None], torch.arange(keys, device=q.device)[None, :]
+        hidden = kp > pos
+        if window > 0:
+            hidden |= kp <= pos - window
+        s = (s * scale).masked_fill(hidden, float("-inf"))
         out[r0: r0 + n] = torch.einsum("hts,sc->thc", torch.softmax(s, -1), rows[:, :kv_rank]).to(q.dtype)
     return out.view(T, H * kv_rank)
 
@@ -778,18 +845,25 @@ def _kv_planes(cache, blocks, dk: int, dv: int, keys: int):
     return k[:keys], v[:keys]
 
 
-def qk_norm_kvwrite(qkv, H: int, G: int, dk: int, dv: int, n: int, q_norm, k_norm, eps, cache, slots):
+def qk_norm_kvwrite(qkv, H: int, G: int, dk: int, dv: int, n: int, q_norm, k_norm, eps, cache, slots, positions=None, cos_sin=None, v_cos_sin=None):
     """Rows [q (H heads) | k (G) | v (G)] of padded widths dk, dk, dv: q (in place) and k are divided by their root mean square over
-    the first `n` columns of each head and multiplied by the norm's weight; k and v go to the cache."""
+    the first `n` columns of each head and multiplied by the norm's weight, and with cos_sin [P, rot] rotated in their first `rot` columns
+    (interleaved pairs); with v_cos_sin v is rotated likewise.  k and v go to the cache."""
     T = qkv.shape[0]
+
+    def turn(x, table):
+        if table is None:
+            return x
+        rot, cs = table.shape[1], table[positions.long()][:, None]
+        return torch.cat([_rotate_pairs(x[..., :rot], cs[..., : rot // 2], cs[..., rot // 2:]), x[..., rot:].float()], -1)
 
     def rms(x, heads, w):
         x = x.reshape(T, heads, dk).float()
-        return (x * torch.rsqrt((x * x).sum(-1, keepdim=True) / n + eps) * w).to(qkv.dtype)
+        return turn(x * torch.rsqrt((x * x).sum(-1, keepdim=True) / n + eps) * w, cos_sin).to(qkv.dtype)
     q = rms(qkv[:, : H * dk], H, q_norm)
     qkv[:, : H * dk] = q.reshape(T, -1)
     k = rms(qkv[:, H * dk: (H + G) * dk], G, k_norm)
-    v = qkv[:, (H + G) * dk: (H + G) * dk + G * dv].reshape(T, G, dv)
+    v = turn(qkv[:, (H + G) * dk: (H + G) * dk + G * dv].reshape(T, G, dv), v_cos_sin).to(qkv.dtype)
     page = cache.shape[2] // (dk + dv)
     ok = slots >= 0
     s = slots[ok].long()
@@ -799,10 +873,11 @@ def qk_norm_kvwrite(qkv, H: int, G: int, dk: int, dv: int, n: int, q_norm, k_nor
 
 
 def gqa_attn(q, cache, H: int, G: int, dk: int, dv: int, scale: float, window: int, inp, out, softcap: float = 0.0, sink=None, gate=None,
-             out_scale: float = 1.0):
+             out_scale: float = 1.0, turn_back=None):
     """Softmax attention of a step's rows (queries in the first H * dk columns of q) over the cached keys and values; a token sees the
     last `window` tokens (0: all) including itself.  softcap: scores become cap * tanh(score / cap).  sink [H]: a score that counts in
-    the denominator only.  The result is multiplied by `out_scale` and by sigmoid(gate) [T, H * dv].  -> out [T, H * dv]"""
+    the denominator only.  turn_back [P, rot]: the first `rot` columns of every head's result are rotated back by the token's position
+    (interleaved pairs).  The result is multiplied by `out_scale` and by sigmoid(gate) [T, H * dv].  -> out [T, H * dv]"""
     T = q.shape[0]
     page = cache.shape[2] // (dk + dv)
     nd, dbt, _, ctx = inp.decode_view(T)
@@ -825,7 +900,11 @@ def gqa_attn(q, cache, H: int, G: int, dk: int, dv: int, scale: float, window: i
         s = s.masked_fill(hidden, float("-inf"))
         if sink is not None:
             s = torch.cat([s, sink.view(G, H // G, 1, 1).expand(-1, -1, n, 1)], -1)
-        y = torch.einsum("ghts,sgd->tghd", torch.softmax(s, -1)[..., :keys], v).reshape(n, H * dv) * out_scale
+        y = torch.einsum("ghts,sgd->tghd", torch.softmax(s, -1)[..., :keys], v).reshape(n, H, dv)
+        if turn_back is not None:
+            rot, cs = turn_back.shape[1], turn_back[before: keys][:, None]
+            y = torch.cat([_rotate_pairs(y[..., :rot], cs[..., : rot // 2], -cs[..., rot // 2:]), y[..., rot:]], -1)
+        y = y.reshape(n, H * dv) * out_scale
         if gate is not None:
             y = y * torch.sigmoid(gate[r0: r0 + n, : H * dv].float())
         out[r0: r0 + n, : H * dv] = y.to(out.dtype)
@@ -841,13 +920,16 @@ class MoeRouting(NamedTuple):
 
 
 def moe_route(x, router_w, k: int, e0: int, e_local: int, experts=None, score: str = "softmax", correction=None, groups: int = 0,
-              keep: int = 0, scale: float = 1.0, shared: int = 0, group_top: int = 2, renorm: bool = True) -> MoeRouting:
+              keep: int = 0, scale: float = 1.0, shared: int = 0, group_top: int = 2, renorm: bool = True, bias=None,
+              shared_gate: bool = True) -> MoeRouting:
     """Routing of every token to `k` of the router's first `experts` rows by its scores, softmax over all of them or sigmoid (plus a
     correction that takes part in the choice only), within the best `keep` of `groups` groups (by the sum of a group's `group_top`
-    largest; softmax: 1).  The weights are the scores, divided by their sum if `renorm`, times `scale`.  `shared` experts more take every
-    token, with the weight sigmoid(router row `experts`)."""
+    largest; softmax: 1).  The weights are the scores, divided by their sum if `renorm`, times `scale`.  `bias` [experts] is added to the
+    logits.  `shared` experts more take every token, with the weight sigmoid(router row `experts`), or without shared_gate one."""
     T, E = x.shape[0], experts or router_w.shape[0]
     z = x.float() @ router_w.float().t()
+    if bias is not None:
+        z[:, :E] += bias
     s = torch.softmax(z[:, :E], -1) if score == "softmax" else torch.sigmoid(z[:, :E])
     choice = s if correction is None else s + correction
     if groups:
@@ -873,7 +955,7 @@ def moe_route(x, router_w, k: int, e0: int, e_local: int, experts=None, score: s
     if shared:
         t = torch.arange(T, device=x.device)
         pos = torch.cat([pos] + [(total + i * T + t)[:, None] for i in range(shared)], 1)
-        w = torch.cat([w] + [torch.sigmoid(z[:, E: E + 1])] * shared, 1)
+        w = torch.cat([w] + [torch.sigmoid(z[:, E: E + 1]) if shared_gate else torch.ones_like(w[:, :1])] * shared, 1)
         xg = torch.cat([xg, x])
     return MoeRouting(ids.to(torch.int32), w, torch.tensor(seg, dtype=torch.int32), pos.to(torch.int32), xg)
 

@@ -82,6 +82,7 @@ class LayeredCache:
       plane, then its value plane);
       a dict of state tensors [slots, ...], addressed by the requests' state slot, with the pages under "kv" where there are both;
       a dict of entries, one per mixer of a layer that has several;
+      int32 pages [num_blocks, page] of token ids (embeddings that look at the token before);
       the very entry of an earlier run whose keys and values it reads."""
 
     def __init__(self, shapes: List[dict], num_blocks: int, num_slots: int, dtype, device, page: int = PAGE_SIZE):
@@ -94,6 +95,8 @@ class LayeredCache:
                 return self.layers[sh["share"]]
             if "parts" in sh:
                 return {n: make(part) for n, part in sh["parts"].items()}
+            if "ids" in sh:
+                return torch.zeros(num_blocks, page, dtype=torch.int32, device=device)
             if "paged" in sh:
                 return torch.zeros(num_blocks, page, sh["paged"], dtype=dtype, device=device)
             pages = None
@@ -146,7 +149,7 @@ def cache_bytes(model, cfg, max_batch: int, page: int = PAGE_SIZE):
     size = lambda dt: torch.empty(0, dtype=dt).element_size()
     width = lambda sh: sh.get("paged", 0) + (sh["kv"][0] * (sh["kv"][1] + sh["kv"][2]) if "kv" in sh else 0)
     shapes = _leaves(shapes)
-    paged = sum(width(sh) for sh in shapes) * page * size(model.dtype)
+    paged = sum(width(sh) * size(model.dtype) + (4 if "ids" in sh else 0) for sh in shapes) * page
     fixed = 0
     for sh in shapes:
         for dims, dt in sh.get("state", {}).values():

@@ -220,11 +220,10 @@ class ModelRunner:
         if not any_lora:
             tl = list(lead_tiles)
         seg_len, sgs, sgq = 0, [], []
-        q8s, q8q, ctx_off = [], [], [0]
-        if self.model.mixed:
+        q8s, q8q, ctx_offs = [], [], {}
+        if self.model.context_windows:
             q8s, q8q = reference.prefill_tiles(q_lens, 128)
-            for c, n in zip(cache_lens, q_lens):
-                ctx_off.append(ctx_off[-1] + c + n)
+            ctx_offs = {w: reference.context_offsets(cache_lens, q_lens, w) for w in self.model.context_windows}
         if self.model.recurrent:
             # the recurrence kernels carry the state through segments of this many tokens: long enough that the states between
             # segments stay a small part of the traffic, short enough that a lone prompt fills the GPU.  Prompts that fill it by
@@ -236,8 +235,8 @@ class ModelRunner:
             sgs, sgq = reference.prefill_tiles(q_lens, seg_len)
         i32 = lambda v: np.asarray(v, dtype=np.int32).reshape(-1)
         segs = [np.concatenate(id_parts) if id_parts else i32([]), i32(cu), i32(cache_lens), i32(seq_slot), i32(ts), i32(tq), i32(head_idx),
-                i32(head_slot), i32(tl), i32(tables), i32(state_slots), i32(sgs), i32(sgq), i32(q8s), i32(q8q),
-                i32(ctx_off)]
+                i32(head_slot), i32(tl), i32(tables), i32(state_slots), i32(sgs), i32(sgq), i32(q8s), i32(q8q)] + \
+            [i32(o) for o in ctx_offs.values()]
         flat = torch.from_numpy(np.concatenate(segs))
         if self.is_cuda:
             flat = flat.pin_memory().to(self.device, non_blocking=True)
@@ -246,7 +245,7 @@ class ModelRunner:
         for sgm in segs:
             views.append(flat[o:o + sgm.shape[0]])
             o += sgm.shape[0]
-        d_ids, d_cu, d_cl, d_seqslot, d_ts, d_tq, d_head, d_headslot, d_tiles, d_bt, d_state, d_sgs, d_sgq, d_q8s, d_q8q, d_off = views
+        d_ids, d_cu, d_cl, d_seqslot, d_ts, d_tq, d_head, d_headslot, d_tiles, d_bt, d_state, d_sgs, d_sgq, d_q8s, d_q8q, *d_off = views
         bt = d_bt.view(len(items), self.max_blocks)
         d_pos, d_slots, d_tokslot = self.model.ops.prefill_metadata(d_cu, d_cl, d_seqslot, bt, page, T)
         if any_lora and self.model.adapters is not None:
@@ -256,7 +255,7 @@ class ModelRunner:
                          cache_lens=d_cl, tile_seq=d_ts, tile_q0=d_tq, lm_head_indices=d_head if len(head_idx) else d_ids[:0],
                          tok_slot=d_tokslot if any_lora else None, head_tok_slot=d_headslot if any_lora else None,
                          lora_tiles=tiles, state_slots=d_state, seg_seq=d_sgs, seg_q0=d_sgq, seg_len=seg_len,
-                         q128_seq=d_q8s, q128_q0=d_q8q, ctx_off=d_off, ctx_total=ctx_off[-1])
+                         q128_seq=d_q8s, q128_q0=d_q8q, contexts={w: (t, o[-1]) for (w, o), t in zip(ctx_offs.items(), d_off)})
         if over_rows:
             inp.embed_rows = torch.tensor(over_rows, dtype=torch.long, device=self.model.device)
             inp.embed_values = torch.cat(over_vals, 0).to(self.model.dtype).to(self.model.device)
@@ -321,7 +320,7 @@ class ModelRunner:
                          dec_block_tables=st.block_tables[:nd], ctx_lens=st.ctx_lens[:nd], embed_rows=pin.embed_rows,
                          embed_values=pin.embed_values, state_slots=pin.state_slots, dec_state_slots=st.state_slots[:nd],
                          seg_seq=pin.seg_seq, seg_q0=pin.seg_q0, seg_len=pin.seg_len,
-                         q128_seq=pin.q128_seq, q128_q0=pin.q128_q0, ctx_off=pin.ctx_off, ctx_total=pin.ctx_total)
+                         q128_seq=pin.q128_seq, q128_q0=pin.q128_q0, contexts=pin.contexts)
         logits = self.model.forward(inp, self.kv.layers)
         self.last_logits = self._cap(logits) if self.keep_logits else None
         ids, lps = self.model.ops.argmax_logprob(logits, softcap=self.model.config.final_logit_softcapping or 0.0)

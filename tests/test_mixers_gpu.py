@@ -8,7 +8,7 @@ PAGE = 32
 DTYPES = (torch.bfloat16, torch.float32)
 
 
-def make_step(dec, pre, slots=None, seg_len=64, seed=0, pages_per_seq=None):
+def make_step(dec, pre, slots=None, seg_len=64, seed=0, pages_per_seq=None, windows=(0,)):
     """StepInputs (on the CPU) of decode rows with contexts `dec` and prompt portions `pre` = [(tokens before, tokens)], over shuffled
     pages and state slots.  -> (inp, number of blocks, number of state slots)"""
     from lorax_b200.models.decoder import StepInputs
@@ -32,17 +32,17 @@ def make_step(dec, pre, slots=None, seg_len=64, seed=0, pages_per_seq=None):
         inp = StepInputs(is_prefill=False, block_tables=blocks, ctx_lens=i32(dec), state_slots=sl, **kw)
     else:
         q = [n for _, n in pre]
-        cu, off = [0], [0]
-        for b, n in pre:
+        cu = [0]
+        for _, n in pre:
             cu.append(cu[-1] + n)
-            off.append(off[-1] + b + n)
+        contexts = {w: reference.context_offsets([b for b, _ in pre], q, w) for w in windows}
         ss, s0 = reference.prefill_tiles(q, seg_len)
         ts, t0 = reference.prefill_tiles(q, 128)
         t64s, t64q = reference.prefill_tiles(q)
         inp = StepInputs(is_prefill=True, block_tables=blocks[nd:].contiguous(), cu_q=i32(cu), cache_lens=i32([b for b, _ in pre]),
                          state_slots=sl[nd:].contiguous(), n_decode=nd, dec_block_tables=blocks[:nd].contiguous(), ctx_lens=i32(dec),
                          dec_state_slots=sl[:nd].contiguous(), seg_seq=i32(ss), seg_q0=i32(s0), seg_len=seg_len, q128_seq=i32(ts),
-                         q128_q0=i32(t0), tile_seq=i32(t64s), tile_q0=i32(t64q), ctx_off=i32(off), ctx_total=off[-1], **kw)
+                         q128_q0=i32(t0), tile_seq=i32(t64s), tile_q0=i32(t64q), contexts={w: (i32(o), o[-1]) for w, o in contexts.items()}, **kw)
     return inp, width * len(spans) + 1, len(spans) + 1
 
 
@@ -50,8 +50,10 @@ def to_dev(x):
     import dataclasses
     if isinstance(x, torch.Tensor):
         return x.cuda()
-    return dataclasses.replace(x, **{f.name: getattr(x, f.name).cuda() for f in dataclasses.fields(x)
-                                     if isinstance(getattr(x, f.name), torch.Tensor)})
+    moved = {f.name: getattr(x, f.name).cuda() for f in dataclasses.fields(x) if isinstance(getattr(x, f.name), torch.Tensor)}
+    if x.contexts is not None:
+        moved["contexts"] = {w: (t.cuda(), n) for w, (t, n) in x.contexts.items()}
+    return dataclasses.replace(x, **moved)
 
 
 def close(got, want, dtype, rows=None, tol16=2e-2, tol32=2e-5):

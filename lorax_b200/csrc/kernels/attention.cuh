@@ -329,27 +329,34 @@ __global__ void __launch_bounds__(32 * NW) attn_decode_kernel(const DecodeParams
     }
   }
   __syncthreads();
-  for (int idx = threadIdx.x; idx < grows * DV; idx += 32 * NW) {
+  for (int idx = threadIdx.x * 2; idx < grows * DV; idx += 64 * NW) {
     const int g = idx / DV, d = idx % DV;
     float M = -INFINITY;
 #pragma unroll
     for (int w = 0; w < NW; ++w) M = fmaxf(M, sm[w * 16 + g]);
-    float num = 0.f, den = 0.f;
+    float2 num = make_float2(0.f, 0.f);
+    float den = 0.f;
 #pragma unroll
     for (int w = 0; w < NW; ++w) {
       const float mw = sm[w * 16 + g];
       const float wgt = (mw == -INFINITY) ? 0.f : exp2f((mw - M) * kLog2e);
-      num += wgt * so[(w * 16 + g) * DV + d];
+      const float2 v = *reinterpret_cast<const float2*>(so + (w * 16 + g) * DV + d);
+      num.x += wgt * v.x;
+      num.y += wgt * v.y;
       den += wgt * sl[w * 16 + g];
     }
     const int head = head0 + g;
-    if (p.nsplit == 1) {                         // (of several splits the sink joins where they are combined)
-      const float o = (den > 0.f ? num * attn_denominator(p.tail, head, M * kLog2e, den) : 0.f) * (KV8 ? p.v_scale : 1.f);
-      p.out[(long long)t * p.ldo + (long long)head * DV + d] = __float2bfloat16(attn_tail(p.tail, o, t, head * DV + d));
+    if (p.nsplit == 1) {                         // (of several splits the tail joins where they are combined)
+      const float f = (den > 0.f ? attn_denominator(p.tail, head, M * kLog2e, den) : 0.f) * (KV8 ? p.v_scale : 1.f);
+      const float2 o = attn_turn_back(p.tail, make_float2(num.x * f, num.y * f), d, ctx - 1);
+      const int col = head * DV + d;
+      __nv_bfloat16* dst = p.out + (long long)t * p.ldo + col;
+      dst[0] = __float2bfloat16(attn_tail(p.tail, o.x, t, col));
+      dst[1] = __float2bfloat16(attn_tail(p.tail, o.y, t, col + 1));
     } else {
-      const float o = (den > 0.f ? num / den : 0.f) * (KV8 ? p.v_scale : 1.f);
+      const float f = (den > 0.f ? 1.f / den : 0.f) * (KV8 ? p.v_scale : 1.f);
       const long long pi = ((long long)t * p.nh + head) * p.nsplit + split;
-      p.part_o[pi * DV + d] = o;
+      *reinterpret_cast<float2*>(p.part_o + pi * DV + d) = make_float2(num.x * f, num.y * f);
       if (d == 0) p.part_lse[pi] = den > 0.f ? M + __logf(den) : -INFINITY;
     }
   }
@@ -358,7 +365,7 @@ __global__ void __launch_bounds__(32 * NW) attn_decode_kernel(const DecodeParams
 template <int D>
 __global__ void __launch_bounds__(D) attn_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_lse,
                                                          __nv_bfloat16* __restrict__ out, long long ldo, int nh, int nsplit,
-                                                         const AttnTail tail) {
+                                                         const AttnTail tail, const int* __restrict__ ctx_lens) {
   pdl_trigger();
   pdl_wait();      // every block waits, also those that return early below
   const int t = blockIdx.x, h = blockIdx.y, d = threadIdx.x;
@@ -374,7 +381,13 @@ __global__ void __launch_bounds__(D) attn_combine_kernel(const float* __restrict
     num += w * part_o[(base + s) * D + d];
     den += w;
   }
-  out[(long long)t * ldo + (long long)h * D + d] = __float2bfloat16(any ? attn_tail(tail, num / den, t, h * D + d) : 0.f);
+  float o = any ? num / den : 0.f;
+  if (tail.turn != nullptr && any) {             // (the whole block takes this branch or none of it)
+    const float other = __shfl_xor_sync(0xffffffffu, o, 1);
+    const float2 both = attn_turn_back(tail, d & 1 ? make_float2(other, o) : make_float2(o, other), d & ~1, ctx_lens[t] - 1);
+    o = d & 1 ? both.y : both.x;
+  }
+  out[(long long)t * ldo + (long long)h * D + d] = __float2bfloat16(any ? attn_tail(tail, o, t, h * D + d) : 0.f);
 }
 
 // ------------------------------------------------------------------------------------------------
@@ -513,10 +526,14 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(const PrefillParams p
 #pragma unroll
   for (int nd = 0; nd < DV / 8; ++nd) {
     const int c = nd * 8 + 2 * (lane & 3), col = head * DV + c;
-    if (qr0 < qlen)
-      *reinterpret_cast<uint32_t*>(p.out + tok0 * p.ldo + (long long)head * DV + c) = pack_bf16x2(attn_tail(p.tail, oacc[nd][0] * inv0, tok0, col), attn_tail(p.tail, oacc[nd][1] * inv0, tok0, col + 1));
-    if (qr1 < qlen)
-      *reinterpret_cast<uint32_t*>(p.out + tok1 * p.ldo + (long long)head * DV + c) = pack_bf16x2(attn_tail(p.tail, oacc[nd][2] * inv1, tok1, col), attn_tail(p.tail, oacc[nd][3] * inv1, tok1, col + 1));
+    if (qr0 < qlen) {
+      const float2 o = attn_turn_back(p.tail, make_float2(oacc[nd][0] * inv0, oacc[nd][1] * inv0), c, pos0);
+      *reinterpret_cast<uint32_t*>(p.out + tok0 * p.ldo + (long long)head * DV + c) = pack_bf16x2(attn_tail(p.tail, o.x, tok0, col), attn_tail(p.tail, o.y, tok0, col + 1));
+    }
+    if (qr1 < qlen) {
+      const float2 o = attn_turn_back(p.tail, make_float2(oacc[nd][2] * inv1, oacc[nd][3] * inv1), c, pos1);
+      *reinterpret_cast<uint32_t*>(p.out + tok1 * p.ldo + (long long)head * DV + c) = pack_bf16x2(attn_tail(p.tail, o.x, tok1, col), attn_tail(p.tail, o.y, tok1, col + 1));
+    }
   }
 }
 
@@ -543,7 +560,7 @@ static int launch_decode_nw(const DecodeParams& p, int T, cudaStream_t s) {
   launch_pdl(attn_decode_kernel<DK, DV, STAGES, KV8, NW, WIDE>, grid, dim3(32 * NW), (size_t)SMEM, s, p);
   if (p.nsplit > 1) {
     dim3 g2(T, p.nh);
-    launch_pdl(attn_combine_kernel<DV>, g2, dim3(DV), 0, s, p.part_o, p.part_lse, p.out, p.ldo, p.nh, p.nsplit, p.tail);
+    launch_pdl(attn_combine_kernel<DV>, g2, dim3(DV), 0, s, p.part_o, p.part_lse, p.out, p.ldo, p.nh, p.nsplit, p.tail, p.ctx_lens);
   }
   return -(int)cudaGetLastError();
 }

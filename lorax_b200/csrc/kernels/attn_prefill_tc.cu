@@ -385,6 +385,14 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_
               float v[8];
 #pragma unroll
               for (int u = 0; u < 8; ++u) v[u] = (o[c + q + u] + __uint_as_float(r[q + u])) * inv;
+              if (p.tail.turn != nullptr) {
+#pragma unroll
+                for (int u = 0; u < 8; u += 2) {
+                  const float2 back = attn_turn_back(p.tail, make_float2(v[u], v[u + 1]), c + q + u, cache + qi);
+                  v[u] = back.x;
+                  v[u + 1] = back.y;
+                }
+              }
               if (grow != nullptr) {
                 const uint4 g = *reinterpret_cast<const uint4*>(grow + c + q);
                 const uint32_t gw[4] = {g.x, g.y, g.z, g.w};
@@ -494,15 +502,15 @@ int lx_attn_prefill_tc(const void* q, long long ldq, int T, const void* kv, int 
                              window, scale, softcap, alibi, wide, lx::AttnTail{}, status, stream);
 }
 
-// The same with fp32 softmax weights, a sink per head, a gate [T, ldg] and a factor on the output (gqa.cu has the contract).
+// The same with fp32 softmax weights, a sink per head, outputs turned back, a gate [T, ldg] and a factor on them (gqa.cu has the contract).
 int lx_gqa_prefill_tc(const void* q, long long ldq, int T, const void* kv, int num_blocks, const int* block_tables, int max_blocks,
                       const int* cu_q, const int* cache_lens, const int* tile_seq, const int* tile_q0, int num_tiles, void* out, long long ldo,
                       int nh, int nkv, int d, int window, float scale, float softcap, const float* sink, const void* gate, long long ldg,
-                      float out_scale, int* status, void* stream) {
-  if (!lx_attn_prefill_tc_supported(nh, nkv, d, ldq, ldo) || (gate != nullptr && ldg % 8 != 0)) return -1;
+                      float out_scale, const float* turn, int turn_dims, int turn_rows, int* status, void* stream) {
+  if (!lx_attn_prefill_tc_supported(nh, nkv, d, ldq, ldo) || turn_dims % 2 != 0 || turn_dims > d || (gate != nullptr && ldg % 8 != 0)) return -1;
   return lx::attn_prefill_tc(q, ldq, T, kv, num_blocks, block_tables, max_blocks, cu_q, cache_lens, tile_seq, tile_q0, num_tiles, out, ldo, nh, nkv,
-                             window, scale, softcap, nullptr, 1, lx::AttnTail{sink, reinterpret_cast<const __nv_bfloat16*>(gate), ldg, out_scale},
-                             status, stream);
+                             window, scale, softcap, nullptr, 1,
+                             lx::AttnTail{sink, reinterpret_cast<const __nv_bfloat16*>(gate), ldg, out_scale, turn, turn_dims, turn_rows}, status, stream);
 }
 
 }  // extern "C"

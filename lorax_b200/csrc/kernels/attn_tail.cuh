@@ -13,12 +13,15 @@ LX_DEVICE float softcap_score(float s, float cap, float k) {
   return fmaf(-2.f * cap, r, cap);
 }
 
-// What may follow the softmax: a sink per head, a score that only the denominator contains; a factor; a gate, sigmoid(gate[t, column]).
+// What may follow the softmax: a sink per head, a score that only the denominator contains; the first turn_dims columns of a head turned
+// back by the token's position (pairs of neighbours); a factor; a gate, sigmoid(gate[t, column]).
 struct AttnTail {
   const float* sink = nullptr;            // [nh]
   const __nv_bfloat16* gate = nullptr;    // [T, ldg]
   long long ldg = 0;
   float scale = 1.f;                      // of the output
+  const float* turn = nullptr;            // [turn_rows, turn_dims] cos, then sin of every position's angles
+  int turn_dims = 0, turn_rows = 0;
 };
 
 // 1 / denominator of a row whose weights were formed with the maximum m and sum to l > 0 (both in the log2 domain): the sink joins, and
@@ -27,6 +30,14 @@ LX_DEVICE float attn_denominator(const AttnTail& tail, int head, float m, float 
   if (tail.sink == nullptr) return 1.f / l;
   const float sink = tail.sink[head] * 1.4426950408889634f, top = fmaxf(m, sink), keep = exp2f(m - top);
   return keep / (l * keep + exp2f(sink - top));
+}
+
+// Columns d (even) and d + 1 of a head, turned back by the angles of position pos.
+LX_DEVICE float2 attn_turn_back(const AttnTail& tail, float2 o, int d, int pos) {
+  if (tail.turn == nullptr || d >= tail.turn_dims) return o;
+  const float* cs = tail.turn + (long long)min(pos, tail.turn_rows - 1) * tail.turn_dims + (d >> 1);
+  const float c = __ldg(cs), s = __ldg(cs + (tail.turn_dims >> 1));
+  return make_float2(o.x * c + o.y * s, o.y * c - o.x * s);
 }
 
 // One finished output element.

@@ -1,7 +1,8 @@
 // Grouped-query attention of the layer-by-layer designs: per-head norms of queries and keys fused with the cache write, and softmax
 // attention with head counts, widths of keys and values, and a window that belong to the layer.
 //
-//   qk_norm_kvwrite   q and k divided by their root mean square per head (fp32), times a weight; k and v to the paged cache
+//   qk_norm_kvwrite   q and k divided by their root mean square per head (fp32), times a weight; where asked for, their first columns
+//                     rotated, and the values by a table of their own (pairs of neighbours); k and v to the paged cache
 //   bf16              the kernels of attention.cuh with the fp32 softmax weights carried into the value product as two bf16 terms
 //                     (widths 64, 128, 256); prompts with keys and values of 128 run on attn_prefill_tc.cu
 //   fp32              one warp per (token, head)
@@ -24,7 +25,35 @@ struct QkNormParams {
   const float* k_norm;
   int T, H, G, DK, DV, page;
   float inv_n, eps;
+  const int* positions;        // [T] (with a table)
+  const float* cos_sin;        // [P, rot] cos, then sin; null: no rotation of q and k
+  const float* v_cos_sin;      // [P, v_rot]; null: none of v
+  int rot, v_rot, P;
 };
+
+// Columns [c, c + 8) of a head turned by row `pos` of the table.
+LX_DEVICE void turn8(float (&f)[8], const float* __restrict__ table, int rot, int pos, int c) {
+  const float* cs = table + (long long)pos * rot + (c >> 1);
+  float co[4], si[4];
+  if (rot % 8 == 0) {
+    const float4 a = __ldg(reinterpret_cast<const float4*>(cs)), b = __ldg(reinterpret_cast<const float4*>(cs + (rot >> 1)));
+    co[0] = a.x; co[1] = a.y; co[2] = a.z; co[3] = a.w;
+    si[0] = b.x; si[1] = b.y; si[2] = b.z; si[3] = b.w;
+  } else {
+#pragma unroll
+    for (int q = 0; q < 4; ++q) {
+      const bool on = c + 2 * q < rot;
+      co[q] = on ? __ldg(cs + q) : 1.f;
+      si[q] = on ? __ldg(cs + (rot >> 1) + q) : 0.f;
+    }
+  }
+#pragma unroll
+  for (int q = 0; q < 4; ++q) {
+    const float u = f[2 * q], v = f[2 * q + 1];
+    f[2 * q] = u * co[q] - v * si[q];
+    f[2 * q + 1] = v * co[q] + u * si[q];
+  }
+}
 
 template <typename T>
 __global__ void __launch_bounds__(256) qk_norm_kvwrite_kernel(const QkNormParams p) {
@@ -52,6 +81,9 @@ __global__ void __launch_bounds__(256) qk_norm_kvwrite_kernel(const QkNormParams
     for (int q = 0; q < 8; ++q) f[q] *= r * g[q];
   }
   if (!live) return;
+  const float* table = values ? p.v_cos_sin : p.cos_sin;
+  const int rot = values ? p.v_rot : p.rot;
+  if (table != nullptr && c < rot) turn8(f, table, rot, min(max(p.positions[t], 0), p.P - 1), c);
   if (!values && h < p.H) {
     store8(src, f);
     return;
@@ -81,6 +113,8 @@ struct GqaF32Params {
   const float* sink;            // [H] or null
   const float* gate;            // [T, ldg] or null
   long long ldg;
+  const float* turn;            // [turn_rows, turn_dims] or null
+  int turn_dims, turn_rows;
 };
 
 __global__ void __launch_bounds__(32 * kGqaWarps) gqa_attn_f32_kernel(const GqaF32Params p) {
@@ -148,6 +182,12 @@ __global__ void __launch_bounds__(32 * kGqaWarps) gqa_attn_f32_kernel(const GqaF
     if (i * 32 >= p.DV) continue;
     const int col = h * p.DV + i * 32 + lane;
     float y = o[i] * inv;
+    const float other = __shfl_xor_sync(0xffffffffu, y, 1);
+    if (p.turn != nullptr && i * 32 + lane < p.turn_dims) {
+      const float* cs = p.turn + (long long)min(max(ctx - 1, 0), p.turn_rows - 1) * p.turn_dims + ((i * 32 + lane) >> 1);
+      const float c = cs[0], s = cs[p.turn_dims >> 1];
+      y = lane & 1 ? y * c - other * s : y * c + other * s;
+    }
     if (p.gate != nullptr) y *= sigmoid_f(p.gate[(long long)t * p.ldg + col]);
     p.out[(long long)t * p.ldo + col] = y;
   }
@@ -192,6 +232,8 @@ int lx_qk_norm_kvwrite(const void* params, int f32, void* stream) {
   const QkNormParams& p = *reinterpret_cast<const QkNormParams*>(params);
   if (p.T <= 0) return 0;
   if (!gqa_width(p.DK) || !gqa_width(p.DV) || p.ld % 8 != 0) return -1;
+  if ((p.cos_sin != nullptr || p.v_cos_sin != nullptr) && (p.positions == nullptr || p.P <= 0)) return -3;
+  if ((p.cos_sin != nullptr && (p.rot % 2 != 0 || p.rot > p.DK)) || (p.v_cos_sin != nullptr && (p.v_rot % 2 != 0 || p.v_rot > p.DV))) return -4;
   const long long threads = (long long)p.T * ((p.H + p.G) * (p.DK / 8) > p.G * (p.DV / 8) ? (p.H + p.G) * (p.DK / 8) : p.G * (p.DV / 8));
   if (threads >= 1ll << 31) return -2;
   const dim3 grid((unsigned)((threads + 255) / 256), 2);
@@ -201,16 +243,18 @@ int lx_qk_norm_kvwrite(const void* params, int f32, void* stream) {
   return -(int)cudaGetLastError();
 }
 
-// softcap > 0: scores become softcap * tanh(score / softcap).  sink [nh] (or null): a score that only the denominator contains.  The outputs
-// are multiplied by out_scale and by sigmoid(gate[t, column]) (gate [T, ldg] or null).
+// softcap > 0: scores become softcap * tanh(score / softcap).  sink [nh] (or null): a score that only the denominator contains.  The outputs'
+// first turn_dims columns of a head are turned back by the token's row of turn [turn_rows, turn_dims] (or null); then they are multiplied
+// by out_scale and by sigmoid(gate[t, column]) (gate [T, ldg] or null).
 //
 // Decode rows (bf16).  part_o / part_lse: T * nh * nsplit * dv and T * nh * nsplit floats, touched when nsplit > 1.
 int lx_gqa_decode(const void* q, long long ldq, const void* cache, const int* block_tables, int max_blocks, const int* ctx_lens, void* out,
                   long long ldo, float* part_o, float* part_lse, int T, int nh, int nkv, int dk, int dv, int window, float scale, int nsplit,
-                  float softcap, const float* sink, const void* gate, long long ldg, float out_scale, void* stream) {
+                  float softcap, const float* sink, const void* gate, long long ldg, float out_scale, const float* turn, int turn_dims,
+                  int turn_rows, void* stream) {
   using namespace lx;
   if (T <= 0) return 0;
-  if (nkv <= 0 || nh % nkv != 0 || ldq % 2 != 0) return -1;
+  if (nkv <= 0 || nh % nkv != 0 || ldq % 2 != 0 || turn_dims % 2 != 0 || turn_dims > dv) return -1;
   DecodeParams p{};
   p.q = reinterpret_cast<const __nv_bfloat16*>(q); p.ldq = ldq;
   p.kv = reinterpret_cast<const __nv_bfloat16*>(cache);
@@ -219,7 +263,7 @@ int lx_gqa_decode(const void* q, long long ldq, const void* cache, const int* bl
   p.part_o = part_o; p.part_lse = part_lse;
   p.nh = nh; p.nkv = nkv; p.group = nh / nkv; p.gchunks = (p.group + 15) / 16;
   p.window = window; p.scale = scale; p.softcap = softcap; p.v_scale = 1.f;
-  p.tail = AttnTail{sink, reinterpret_cast<const __nv_bfloat16*>(gate), ldg, out_scale};
+  p.tail = AttnTail{sink, reinterpret_cast<const __nv_bfloat16*>(gate), ldg, out_scale, turn, turn_dims, turn_rows};
   p.nsplit = nsplit < 1 ? 1 : nsplit;
   if (p.nsplit > 1 && (part_o == nullptr || part_lse == nullptr)) return -2;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
@@ -232,10 +276,10 @@ int lx_gqa_decode(const void* q, long long ldq, const void* cache, const int* bl
 int lx_gqa_prefill(const void* q, long long ldq, const void* cache, const int* block_tables, int max_blocks, const int* cu_q,
                    const int* cache_lens, const int* tile_seq, const int* tile_q0, int num_tiles, void* out, long long ldo, int nh, int nkv,
                    int dk, int dv, int window, float scale, float softcap, const float* sink, const void* gate, long long ldg, float out_scale,
-                   void* stream) {
+                   const float* turn, int turn_dims, int turn_rows, void* stream) {
   using namespace lx;
   if (num_tiles <= 0) return 0;
-  if (nkv <= 0 || nh % nkv != 0 || ldq % 2 != 0 || ldo % 2 != 0) return -1;
+  if (nkv <= 0 || nh % nkv != 0 || ldq % 2 != 0 || ldo % 2 != 0 || turn_dims % 2 != 0 || turn_dims > dv) return -1;
   PrefillParams p{};
   p.q = reinterpret_cast<const __nv_bfloat16*>(q); p.ldq = ldq;
   p.kv = reinterpret_cast<const __nv_bfloat16*>(cache);
@@ -243,7 +287,7 @@ int lx_gqa_prefill(const void* q, long long ldq, const void* cache, const int* b
   p.tile_seq = tile_seq; p.tile_q0 = tile_q0;
   p.out = reinterpret_cast<__nv_bfloat16*>(out); p.ldo = ldo;
   p.nh = nh; p.nkv = nkv; p.window = window; p.scale = scale; p.softcap = softcap; p.v_scale = 1.f;
-  p.tail = AttnTail{sink, reinterpret_cast<const __nv_bfloat16*>(gate), ldg, out_scale};
+  p.tail = AttnTail{sink, reinterpret_cast<const __nv_bfloat16*>(gate), ldg, out_scale, turn, turn_dims, turn_rows};
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
 #define LX_CALL(DK, DV) launch_prefill<DK, DV, false, true>(p, num_tiles, s)
   LX_GQA_DISPATCH(LX_CALL)
@@ -254,7 +298,7 @@ int lx_gqa_attn_f32(const void* params, void* stream) {
   using namespace lx;
   const GqaF32Params& p = *reinterpret_cast<const GqaF32Params*>(params);
   if (p.T <= 0) return 0;
-  if (!gqa_width(p.DK) || !gqa_width(p.DV) || p.G <= 0 || p.H % p.G != 0) return -1;
+  if (!gqa_width(p.DK) || !gqa_width(p.DV) || p.G <= 0 || p.H % p.G != 0 || p.turn_dims % 2 != 0 || p.turn_dims > p.DV) return -1;
   launch_pdl(gqa_attn_f32_kernel, dim3(p.T, (p.H + kGqaWarps - 1) / kGqaWarps), dim3(32 * kGqaWarps), 0, reinterpret_cast<cudaStream_t>(stream), p);
   return -(int)cudaGetLastError();
 }

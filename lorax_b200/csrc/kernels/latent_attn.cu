@@ -6,11 +6,11 @@
 namespace lx {
 
 // ------------------------------------------------------------------------------------------------
-// Preparation of a token: RMS norm of the query down-projection (-> cq), RMS norm of the key/value latent and interleaved rotation of
-// the shared key part (-> cache row).  One CTA per token.
+// Preparation of a token: RMS norm of the query down-projection (-> cq) or, without one, interleaved rotation of the queries in place; RMS
+// norm of the key/value latent and interleaved rotation of the shared key part (-> cache row).  One CTA per token.
 // ------------------------------------------------------------------------------------------------
 struct LatentPrepParams {
-  const void* dq; const void* dkv;      // [T, ld] rows of the fused projection
+  const void* dq; const void* dkv;      // [T, ld] rows of the fused projection; dq null (QR 0): no query latent
   long long ld_dq, ld_dkv;
   const float* dq_norm;                 // [QR] padded with zeros
   const float* dkv_norm;                // [KR]
@@ -20,6 +20,9 @@ struct LatentPrepParams {
   const float* cos_sin;                 // [max_pos, rot]
   int QR, KR, R, q_rank, kv_rank, rot;
   float eps;
+  void* q;                              // [T, ldq] or null: columns [off, off + rot) of every head are rotated
+  long long ldq;
+  int H, head, off;
 };
 
 template <typename T>
@@ -43,7 +46,33 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(const LatentPrepParams
 #pragma unroll
     for (int q = 0; q < 8; ++q) sk += f[q] * f[q];
   }
-  const float rq = rsqrtf(block_sum(sq, red) / p.q_rank + p.eps);
+  const float* cs = p.cos_sin + (long long)p.positions[t] * p.rot;
+  const int half = p.rot / 2;
+  if (p.q != nullptr) {
+    T* x = reinterpret_cast<T*>(p.q) + (long long)t * p.ldq + p.off;
+    if (p.rot % 8 == 0) {
+      const int per = p.rot / 8;
+      for (int e = threadIdx.x; e < p.H * per; e += blockDim.x) {
+        const int h = e / per, i = (e - h * per) * 4;
+        const float4 c = __ldg(reinterpret_cast<const float4*>(cs + i)), s = __ldg(reinterpret_cast<const float4*>(cs + half + i));
+        T* at = x + (long long)h * p.head + 2 * i;
+        float f[8];
+        load8(at, f);
+        const float g[8] = {f[0] * c.x - f[1] * s.x, f[1] * c.x + f[0] * s.x, f[2] * c.y - f[3] * s.y, f[3] * c.y + f[2] * s.y,
+                            f[4] * c.z - f[5] * s.z, f[5] * c.z + f[4] * s.z, f[6] * c.w - f[7] * s.w, f[7] * c.w + f[6] * s.w};
+        store8(at, g);
+      }
+    } else {
+      for (int e = threadIdx.x; e < p.H * half; e += blockDim.x) {
+        const int h = e / half, i = e - h * half;
+        T* at = x + (long long)h * p.head + 2 * i;
+        const float u = to_f(at[0]), v = to_f(at[1]), c = cs[i], s = cs[half + i];
+        put(at, u * c - v * s);
+        put(at + 1, v * c + u * s);
+      }
+    }
+  }
+  const float rq = p.QR > 0 ? rsqrtf(block_sum(sq, red) / p.q_rank + p.eps) : 0.f;
   const float rk = rsqrtf(block_sum(sk, red) / p.kv_rank + p.eps);
   T* cq = reinterpret_cast<T*>(p.cq) + (long long)t * p.QR;
   for (int c = threadIdx.x * 8; c < p.QR; c += blockDim.x * 8) {
@@ -65,8 +94,6 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(const LatentPrepParams
     for (int q = 0; q < 8; ++q) f[q] *= rk * w[q];
     store8(row + c, f);
   }
-  const float* cs = p.cos_sin + (long long)p.positions[t] * p.rot;
-  const int half = p.rot / 2;
   for (int i = threadIdx.x; i < (p.R - p.KR) / 2; i += blockDim.x) {
     float a = 0.f, b = 0.f;
     if (i < half) {
@@ -110,6 +137,7 @@ struct LatentAttnParams {
   StepRows rows;
   int H, KR, R, page;
   float scale;
+  int window;                            // <= 0: none
 };
 
 constexpr int kLaMaxVec = 5;             // R <= 32 * 8 * 5
@@ -145,7 +173,7 @@ __global__ void __launch_bounds__(128) latent_attn_kernel(const LatentAttnParams
     for (int e = 0; e < 8; ++e) q[i][e] *= p.scale;
   }
   float m = -INFINITY, l = 0.f;
-  for (int j = warp; j < keys; j += 4) {
+  for (int j = (p.window > 0 ? max(keys - p.window, 0) : 0) + warp; j < keys; j += 4) {
     const T* row = reinterpret_cast<const T*>(p.cache) + ((long long)bt[j / p.page] * p.page + j % p.page) * p.R;
     float k[kLaMaxVec][8], s = 0.f;
 #pragma unroll
@@ -201,6 +229,7 @@ int lx_latent_prep(const void* params, int T, int f32, void* stream) {
   if (T <= 0) return 0;
   const LatentPrepParams& p = *reinterpret_cast<const LatentPrepParams*>(params);
   if (p.QR % 8 != 0 || p.KR % 8 != 0 || p.R % 8 != 0 || p.ld_dq % 8 != 0 || p.ld_dkv % 8 != 0 || p.rot % 2 != 0 || p.rot > p.R - p.KR) return -1;
+  if (p.q != nullptr && (p.head % 8 != 0 || p.off % 8 != 0 || p.ldq % 8 != 0 || p.off + p.rot > p.head)) return -2;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   if (f32) launch_pdl(latent_prep_kernel<float>, dim3(T), dim3(128), 0, s, p);
   else launch_pdl(latent_prep_kernel<__nv_bfloat16>, dim3(T), dim3(128), 0, s, p);

@@ -23,6 +23,7 @@ struct LatentDecodeParams {
   float scale;
   float* part_o;                                  // [T, H, nsplit, KR]
   float* part_ml;                                 // [T, H, nsplit, 2] maximum (log2 domain), sum
+  int window;                                     // <= 0: none
 };
 
 LX_DEVICE void ld_mma(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
@@ -83,9 +84,10 @@ __global__ void __launch_bounds__(32 * WARPS, OCC) latent_decode_kernel(const La
     bt = p.rows.bt + (long long)b * p.rows.max_blocks;
   }
   keys = max(keys, 0);
-  const int tiles = (keys + KEYS - 1) / KEYS;
-  const int per = (tiles + p.nsplit - 1) / p.nsplit;
-  const int t_lo = split * per, t_hi = min(t_lo + per, tiles);
+  const int lo = p.window > 0 ? max(keys - p.window, 0) : 0;
+  const int first = lo / KEYS, tiles = (keys + KEYS - 1) / KEYS;
+  const int per = (tiles - first + p.nsplit - 1) / p.nsplit;
+  const int t_lo = first + split * per, t_hi = min(t_lo + per, tiles);
 
   const int kg = warp % KG, kh = warp / KG;         // K slice, key half of the score products
   const int nk = p.R / 16;
@@ -186,7 +188,8 @@ __global__ void __launch_bounds__(32 * WARPS, OCC) latent_decode_kernel(const La
       }
 #pragma unroll
       for (int q = 0; q < KPT; ++q) {
-        s[q] = (i * KEYS + sk0 + q < keys) ? s[q] * scale_l2 : -INFINITY;
+        const int key = i * KEYS + sk0 + q;
+        s[q] = (key >= lo && key < keys) ? s[q] * scale_l2 : -INFINITY;
         bm = fmaxf(bm, s[q]);
       }
 #pragma unroll

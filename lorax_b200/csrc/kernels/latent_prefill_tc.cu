@@ -1,6 +1,6 @@
 // Prompt attention of the latent mixer on the tensor cores (tcgen05): the latents of the sequences of a step are gathered from their
-// pages, expanded to per-head keys and values by one GEMM, and attended to here as plain multi-head attention with a key part that all
-// heads share.  (The absorbed form in latent_attn.cu reads the latents once per query row instead: right for single tokens, three to
+// pages (with a window: what a portion's first query sees), expanded to per-head keys and values by one GEMM, and attended to here as
+// plain multi-head attention with a key part that all heads share.  (The absorbed form in latent_attn.cu reads the latents once per query row instead: right for single tokens, three to
 // four times the products for a prompt.)
 //
 // One CTA = 128 queries of one sequence x one head.  Keys are walked in blocks of 64:
@@ -10,7 +10,7 @@
 //   softmax (warps 2..5)        one thread per query: 64 scores in registers, exp2 against a reference maximum.  The weights stay fp32:
 //                               they are split into two bf16 terms (value + remainder) and multiplied as two operands.  O is rescaled in
 //                               TMEM only when a row's maximum grew by more than 2^8 over its reference.
-// The head's output gate multiplies the result on its way out.  Every wait is bounded and reports through the status word.
+// The output gate, one number per head or per element, multiplies the result on its way out.  Every wait is bounded and reports through the status word.
 #include "stream.cuh"
 
 namespace lx {
@@ -23,12 +23,13 @@ struct LatentPrefillParams {
   const int* tile_seq; const int* tile_q0;         // 128-query tiles
   const int* cu_q; const int* cache_lens;
   const int* ctx_off;                              // [B + 1] first gathered row of every sequence
-  const __nv_bfloat16* gate; long long ldg;        // [T, ldg]
+  const __nv_bfloat16* gate; long long ldg;        // [T, ldg]; column h, or (gate_wide) the output's column
   __nv_bfloat16* out; long long ldo;               // rows of the prompt tokens
   int kv_head;                                     // columns of one head in the expansion (key part, then value)
   int q_head;                                      // columns of one head in q
   float scale;
   int* status;
+  int window, gate_wide;                           // window <= 0: none
 };
 
 LX_DEVICE float lp_ex2(float x) {
@@ -112,10 +113,12 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
   const int q0 = p.tile_q0[tile];
   const int tok0 = p.cu_q[b];
   const int qlen = p.cu_q[b + 1] - tok0;
-  const int cache = p.cache_lens[b];
-  const int row_base = p.ctx_off[b];
-  const int key_hi = cache + min(q0 + kLpQ, qlen);             // keys of the tile: [0, key_hi)
-  const int nblk = (key_hi + kLpKeys - 1) / kLpKeys;
+  const int cache = p.window > 0 ? min(p.cache_lens[b], p.window - 1) : p.cache_lens[b];       // gathered rows in front of the portion
+  const int key_hi = cache + min(q0 + kLpQ, qlen);             // keys of the tile, in gathered rows: [key_lo, key_hi)
+  const int key_lo = p.window > 0 ? max(cache + q0 + 1 - p.window, 0) : 0;
+  const int first = key_lo / kLpKeys;                          // (block 0 below holds the rows from first * kLpKeys on)
+  const int row_base = p.ctx_off[b] + first * kLpKeys;
+  const int nblk = (key_hi + kLpKeys - 1) / kLpKeys - first;
 
   if (warp == 0) {
     if (lane == 0) {
@@ -188,7 +191,9 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
     const int qi = q0 + row;
     const bool row_ok = qi < qlen;
     const int hi = row_ok ? cache + qi + 1 : 0;                // keys this row sees
+    const int lo = p.window > 0 ? max(hi - p.window, 0) : 0;
     const int hi_min = (q0 + kLpQ <= qlen) ? cache + q0 + 1 : 0;
+    const int lo_max = p.window > 0 ? max(key_hi - p.window, 0) : 0;
     const float scale_l2 = p.scale * kLpLog2e;
     const uint32_t trow = tmem_base + ((uint32_t)(quad * 32) << 16);
     float m = -INFINITY, l = 0.f;                              // reference maximum (log2 domain), sum against it
@@ -206,10 +211,10 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
       float s[64];
 #pragma unroll
       for (int i = 0; i < 32; ++i) { s[i] = __uint_as_float(r0[i]); s[32 + i] = __uint_as_float(r1[i]); }
-      const int kb0 = j * kLpKeys;
-      if (kb0 + kLpKeys > hi_min) {
+      const int kb0 = (first + j) * kLpKeys;
+      if (kb0 + kLpKeys > hi_min || kb0 < lo_max) {
 #pragma unroll
-        for (int i = 0; i < 64; ++i) s[i] = kb0 + i < hi ? s[i] : -INFINITY;
+        for (int i = 0; i < 64; ++i) s[i] = kb0 + i < hi && kb0 + i >= lo ? s[i] : -INFINITY;
       }
       float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
@@ -278,13 +283,23 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
         tc_fence_after();
         const long long tok = (long long)tok0 + qi;
         float f = 0.f;
-        if (row_ok) f = (l > 0.f ? 1.f / l : 0.f) * (p.gate ? sigmoid_f(to_f(p.gate[tok * p.ldg + h])) : 1.f);
+        if (row_ok) f = (l > 0.f ? 1.f / l : 0.f) * (p.gate && !p.gate_wide ? sigmoid_f(to_f(p.gate[tok * p.ldg + h])) : 1.f);
+        const __nv_bfloat16* grow = p.gate && p.gate_wide && row_ok ? p.gate + tok * p.ldg + (long long)h * NV * 64 : nullptr;
         __nv_bfloat16* orow = p.out + tok * p.ldo + (long long)h * NV * 64;
 #pragma unroll
         for (int c = 0; c < NV * 64; c += 32) {
           uint32_t o[32];
           tmem_ld_32x32b_x32(trow + (uint32_t)(128 + c), o);
           tc_wait_ld();
+          if (grow != nullptr) {
+#pragma unroll
+            for (int q = 0; q < 32; q += 8) {
+              float z[8];
+              load8(grow + c + q, z);
+#pragma unroll
+              for (int u = 0; u < 8; ++u) o[q + u] = __float_as_uint(__fdividef(__uint_as_float(o[q + u]), 1.f + __expf(-z[u])));
+            }
+          }
           if (row_ok) {
 #pragma unroll
             for (int q = 0; q < 32; q += 8)
@@ -306,9 +321,11 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
   if (warp == 1) { tc_fence_after(); tmem_dealloc(tmem_base, 256); }
 }
 
-// Rows of the sequences' pages, in order, as one contiguous matrix: latents [N, KR] and shared key parts [N, RR].
+// Rows of the sequences' pages, in order, as one contiguous matrix: latents [N, KR] and shared key parts [N, RR].  With a window a
+// sequence's rows begin window - 1 in front of its portion.
 __global__ void __launch_bounds__(128) latent_gather_kernel(const __nv_bfloat16* __restrict__ cache, const int* __restrict__ bt, int max_blocks,
-                                                            const int* __restrict__ ctx_off, int B, int page, int KR, int RR,
+                                                            const int* __restrict__ ctx_off, const int* __restrict__ cache_lens, int window,
+                                                            int B, int page, int KR, int RR,
                                                             __nv_bfloat16* __restrict__ lat, __nv_bfloat16* __restrict__ rot) {
   pdl_trigger();
   pdl_wait();
@@ -318,7 +335,7 @@ __global__ void __launch_bounds__(128) latent_gather_kernel(const __nv_bfloat16*
     const int mid = (lo + hi) >> 1;
     if (ctx_off[mid] <= r) lo = mid; else hi = mid;
   }
-  const int pos = r - ctx_off[lo];
+  const int pos = r - ctx_off[lo] + (window > 0 ? max(cache_lens[lo] - (window - 1), 0) : 0);
   const __nv_bfloat16* src = cache + ((long long)bt[(long long)lo * max_blocks + pos / page] * page + pos % page) * (KR + RR);
   for (int c = threadIdx.x * 8; c < KR + RR; c += blockDim.x * 8) {
     const uint4 v = *reinterpret_cast<const uint4*>(src + c);
@@ -360,28 +377,29 @@ static int lp_launch(const CUtensorMap& tq, const CUtensorMap& tkv, const CUtens
 
 extern "C" {
 
-int lx_latent_gather(const void* cache, const int* bt, int max_blocks, const int* ctx_off, int B, int rows, int page, int KR, int RR, void* lat,
-                     void* rot, void* stream) {
+int lx_latent_gather(const void* cache, const int* bt, int max_blocks, const int* ctx_off, const int* cache_lens, int window, int B, int rows,
+                     int page, int KR, int RR, void* lat, void* rot, void* stream) {
   using namespace lx;
   if (rows <= 0) return 0;
   if (KR % 8 != 0 || RR % 8 != 0) return -1;
   launch_pdl(latent_gather_kernel, dim3(rows), dim3(128), 0, reinterpret_cast<cudaStream_t>(stream), reinterpret_cast<const __nv_bfloat16*>(cache), bt,
-             max_blocks, ctx_off, B, page, KR, RR, reinterpret_cast<__nv_bfloat16*>(lat), reinterpret_cast<__nv_bfloat16*>(rot));
+             max_blocks, ctx_off, cache_lens, window, B, page, KR, RR, reinterpret_cast<__nv_bfloat16*>(lat), reinterpret_cast<__nv_bfloat16*>(rot));
   return -(int)cudaGetLastError();
 }
 
-// 1: head sizes (per-head key part, shared key part, value) the kernel takes.
+// 1: head sizes (per-head key part, shared key part, value) the kernel takes.  A shared part of less than 64 columns is a panel whose tail
+// the tensor map fills with zeros on the keys' side (the queries' side reads the columns behind the head's, which then count nothing).
 int lx_latent_prefill_supported(int dk, int rot, int dv) {
-  return ((dk == 128 && rot == 64 && dv == 128) || (dk == 64 && rot == 64 && (dv == 64 || dv == 128))) ? 1 : 0;
+  return rot > 0 && rot <= 64 && rot % 16 == 0 && ((dk == 128 && dv == 128) || (dk == 64 && (dv == 64 || dv == 128))) ? 1 : 0;
 }
 
 // q [T, ldq]: head h at column h * (dk + rot), per-head part first.  kv [rows, H * (dk + dv)] the expansion, rot_keys [rows, rot].
 int lx_latent_prefill(const void* q, long long ldq, int T, const void* kv, const void* rot_keys, int rows, const int* ctx_off, const int* cu_q,
                       const int* cache_lens, const int* tile_seq, const int* tile_q0, int tiles, const void* gate, long long ldg, void* out,
-                      long long ldo, int H, int dk, int rot, int dv, float scale, int* status, void* stream) {
+                      long long ldo, int H, int dk, int rot, int dv, float scale, int window, int gate_wide, int* status, void* stream) {
   using namespace lx;
   if (tiles <= 0) return 0;
-  if (!lx_latent_prefill_supported(dk, rot, dv) || ldq % 8 != 0 || ldo % 8 != 0) return -1;
+  if (!lx_latent_prefill_supported(dk, rot, dv) || ldq % 8 != 0 || ldo % 8 != 0 || (gate_wide && ldg % 8 != 0)) return -1;
   CUtensorMap tq, tkv, tr;
   if (lp_map(&tq, q, (long long)H * (dk + rot), T, ldq, kLpQ) || lp_map(&tkv, kv, (long long)H * (dk + dv), rows, (long long)H * (dk + dv), kLpKeys) ||
       lp_map(&tr, rot_keys, rot, rows, rot, kLpKeys))
@@ -390,6 +408,7 @@ int lx_latent_prefill(const void* q, long long ldq, int T, const void* kv, const
   p.tile_seq = tile_seq; p.tile_q0 = tile_q0; p.cu_q = cu_q; p.cache_lens = cache_lens; p.ctx_off = ctx_off;
   p.gate = reinterpret_cast<const __nv_bfloat16*>(gate); p.ldg = ldg;
   p.out = reinterpret_cast<__nv_bfloat16*>(out); p.ldo = ldo;
+  p.window = window; p.gate_wide = gate_wide;
   p.kv_head = dk + dv; p.q_head = dk + rot; p.scale = scale; p.status = status;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   if (dk == 128) return lp_launch<2, 1, 2>(tq, tkv, tr, p, tiles, H, s);

@@ -13,7 +13,7 @@
 //                   a token tile that runs past its expert's rows computes a few columns nobody stores
 //   combine         out[t, :] = sum_j w[t, j] * y[pos[t, j], :]
 //
-// Shared experts (every token, weight sigmoid(one more router row)) are further runs of the same grouped products; their input rows
+// Shared experts (every token, weight one or sigmoid(one more router row)) are further runs of the same grouped products; their input rows
 // are the tokens themselves and stand in xg once.
 //
 // Only the k experts a token was routed to do work for it (the reference gets that from megablocks' block-sparse kernels,
@@ -122,6 +122,8 @@ struct MoeSelectParams {
   int T, E, k, e0, e_local;
   int sigmoid, groups, keep, shared, group_top, renorm;
   float scale;
+  int shared_one;          // the shared experts' weight is one (else the sigmoid of router row E)
+  const float* bias;       // [E], added to the logits, or null
 };
 
 // Largest value of the warp and its index; the lower index on ties.
@@ -146,14 +148,15 @@ __global__ void __launch_bounds__(32 * kSelWarps) moe_select_kernel(const MoeSel
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * kSelWarps + warp;
   if (t >= p.T) return;
-  const float* l = p.logits + (long long)t * p.ldl;
+  const float* row = p.logits + (long long)t * p.ldl;
+  auto logit = [&](int e) { return p.bias != nullptr ? row[e] + p.bias[e] : row[e]; };
   float choice[PER];
 #pragma unroll
   for (int i = 0; i < PER; ++i) {
     const int e = lane + 32 * i;
     float v = -INFINITY;
     if (e < p.E) {
-      v = l[e];
+      v = logit(e);
       if (p.sigmoid) v = 1.f / (1.f + expf(-v)) + (p.correction != nullptr ? p.correction[e] : 0.f);
     }
     choice[i] = v;
@@ -218,16 +221,16 @@ __global__ void __launch_bounds__(32 * kSelWarps) moe_select_kernel(const MoeSel
         if (i == (bi >> 5)) choice[i] = -INFINITY;
     }
     if (lane == j) id = bi;
-    if (j == 0) top = l[bi];
+    if (j == 0) top = logit(bi);
   }
   float w = 0.f;
-  if (lane < p.k) w = p.sigmoid ? 1.f / (1.f + expf(-l[id])) : expf(l[id] - top);
+  if (lane < p.k) w = p.sigmoid ? 1.f / (1.f + expf(-logit(id))) : expf(logit(id) - top);
   float sum = 1.f;
   if (p.renorm) {
     sum = warp_sum(w) + (p.sigmoid ? 1e-20f : 0.f);
   } else if (!p.sigmoid) {                       // (the first chosen logit is the largest of all)
     float own = 0.f;
-    for (int e = lane; e < p.E; e += 32) own += expf(l[e] - top);
+    for (int e = lane; e < p.E; e += 32) own += expf(logit(e) - top);
     sum = warp_sum(own);
   }
   const int kw = p.k + p.shared;
@@ -238,7 +241,7 @@ __global__ void __launch_bounds__(32 * kSelWarps) moe_select_kernel(const MoeSel
     p.rank[(long long)t * kw + lane] = (le >= 0 && le < p.e_local) ? atomicAdd(&p.counts[le], 1) : -1;
   }
   if (p.shared > 0) {
-    const float g = 1.f / (1.f + expf(-l[p.E]));
+    const float g = p.shared_one ? 1.f : 1.f / (1.f + expf(-row[p.E]));
     for (int j = lane; j < p.shared; j += 32) p.topk_w[(long long)t * kw + p.k + j] = g;
   }
 }
@@ -688,7 +691,7 @@ int lx_moe_select(const void* params, void* stream) {
   const MoeSelectParams& p = *reinterpret_cast<const MoeSelectParams*>(params);
   if (p.T <= 0) return 0;
   if (p.E > kMoeMaxExperts || p.E < 1 || p.k > kMoeMaxK || p.k > p.E || p.k < 1 || p.e_local > kMoeMaxExperts || p.shared > kMoeMaxShared) return -1;
-  if (p.ldl < p.E + (p.shared > 0 ? 1 : 0)) return -2;
+  if (p.ldl < p.E + (p.shared > 0 && !p.shared_one ? 1 : 0)) return -2;
   if (p.group_top < 1 || p.group_top > 2 || (!p.sigmoid && p.groups > 0 && p.group_top != 1)) return -4;
   if (p.groups > 0 && (p.E % p.groups != 0 || p.keep < 1 || p.keep > p.groups || p.keep * (p.E / p.groups) < p.k)) return -3;
   const dim3 grid((p.T + kSelWarps - 1) / kSelWarps), block(32 * kSelWarps);

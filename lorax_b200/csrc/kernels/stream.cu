@@ -6,16 +6,52 @@ namespace lx {
 
 // ------------------------------------------------------------------------------------------------
 // Residual stream: x[t] = table[ids[t]] * mult (+ pos[positions[t]]) in fp32; `copy` takes x in the model's dtype.
+// Pairs: the vector of (token before, token) is added too.  The token before a row is the row before it or, for a sequence's first row of
+// the step, stands in the paged token ids, where every row leaves its own (a page's slot is written once per token, and read by the
+// steps behind it only).
 // ------------------------------------------------------------------------------------------------
+struct EmbedPairs {
+  const void* vectors;         // [buckets + 1, W], the last row for a sequence's first token; null: no pairs
+  int* pages;                  // [blocks * page] token ids
+  const int* slots;            // [T] slot of the row's token, < 0: none
+  long long mul_prev, mul_cur;
+  int buckets, page;
+  StepRows rows;
+};
+
+// Token in front of row t, or -1.
+LX_DEVICE int token_before(const EmbedPairs& e, const int* ids, int t) {
+  int before;
+  const int* bt;
+  if (t < e.rows.nd) {
+    before = e.rows.ctx_lens[t] - 1;
+    bt = e.rows.dec_bt + (long long)t * e.rows.dec_max_blocks;
+  } else {
+    const int b = seq_of(e.rows, t - e.rows.nd), i = t - e.rows.nd - e.rows.cu_q[b];
+    if (i > 0) return ids[t - 1];
+    before = e.rows.cache_lens[b];
+    bt = e.rows.bt + (long long)b * e.rows.max_blocks;
+  }
+  return before > 0 ? e.pages[(long long)bt[(before - 1) / e.page] * e.page + (before - 1) % e.page] : -1;
+}
+
 template <typename T>
 __global__ void __launch_bounds__(128) embed_stream_kernel(const int* __restrict__ ids, const T* __restrict__ table, float* __restrict__ out,
                                                            int W, int V, float mult, const T* __restrict__ pos,
-                                                           const int* __restrict__ positions, int P, T* __restrict__ copy) {
+                                                           const int* __restrict__ positions, int P, T* __restrict__ copy,
+                                                           const EmbedPairs pairs) {
   pdl_trigger();
   pdl_wait();
   const int t = blockIdx.x;
   const int id = min(max(ids[t], 0), V - 1);
   const int at = pos != nullptr ? min(max(positions[t], 0), P - 1) : 0;
+  const T* pair = nullptr;
+  if (pairs.vectors != nullptr) {
+    const int prev = token_before(pairs, ids, t);
+    const long long row = prev < 0 ? pairs.buckets : (min(prev, V - 1) * pairs.mul_prev + id * pairs.mul_cur) % pairs.buckets;
+    pair = reinterpret_cast<const T*>(pairs.vectors) + row * W;
+    if (threadIdx.x == 0 && pairs.slots[t] >= 0) pairs.pages[pairs.slots[t]] = id;
+  }
   for (int c = threadIdx.x * 8; c < W; c += blockDim.x * 8) {
     float f[8];
     load8(table + (long long)id * W + c, f);
@@ -24,6 +60,12 @@ __global__ void __launch_bounds__(128) embed_stream_kernel(const int* __restrict
     if (pos != nullptr) {
       float g[8];
       load8(pos + (long long)at * W + c, g);
+#pragma unroll
+      for (int q = 0; q < 8; ++q) f[q] += g[q];
+    }
+    if (pair != nullptr) {
+      float g[8];
+      load8(pair + c, g);
 #pragma unroll
       for (int q = 0; q < 8; ++q) f[q] += g[q];
     }
@@ -113,7 +155,8 @@ __global__ void __launch_bounds__(kNsThreads) norm_stream_kernel(const NormStrea
 // ------------------------------------------------------------------------------------------------
 // Norm of a sublayer's output, added to the stream: residual += mult * (norm(y) * w + b), copy = residual in the model's dtype.  One
 // CTA per row.  Columns from n on are padding: they take no part in mean and variance, and w and b are zero there.  PAIRS: y of a
-// token is the weighted sum of the rows pos[t, 0 .. k) (-1: none) of y (the outputs of its experts).
+// token is the weighted sum of the rows pos[t, 0 .. k) (-1: none) of y (the outputs of its experts).  NEXT: y is multiplied by
+// sigmoid(gate) first when there is one, and copy = norm(residual) * next_w, of `rows` only when given (the residual then stays as it is).
 // ------------------------------------------------------------------------------------------------
 struct NormAddParams {
   float* residual;
@@ -126,6 +169,10 @@ struct NormAddParams {
   const float* weights;        // [T, k]
   int k, W, n, layernorm;
   float inv_n, eps, mult;
+  const void* gate;            // [T, ldg] or null
+  long long ldg;
+  const float* next_w;         // [W] (NEXT)
+  const int* rows;             // or null
 };
 
 // In place on a row held as NV vectors of eight columns per thread: v <- norm(v) * w + b.
@@ -167,12 +214,17 @@ LX_DEVICE void norm_row(float (&v)[NV][8], const float* __restrict__ w, const fl
   }
 }
 
-template <typename T, bool PAIRS, int NV>
+template <typename T>
+LX_DEVICE float gate_f(float z) {
+  return sizeof(T) == 2 ? __fdividef(1.f, 1.f + __expf(-z)) : sigmoid_f(z);
+}
+
+template <typename T, bool PAIRS, int NV, bool NEXT>
 __global__ void __launch_bounds__(kNsThreads) norm_add_kernel(const NormAddParams p) {
   pdl_trigger();
   pdl_wait();
   __shared__ float red[kNsThreads / 32];
-  const int t = blockIdx.x;
+  const int t = NEXT && p.rows != nullptr ? p.rows[blockIdx.x] : (int)blockIdx.x;
   const T* y = reinterpret_cast<const T*>(p.y);
   float v[NV][8];
 #pragma unroll
@@ -194,10 +246,36 @@ __global__ void __launch_bounds__(kNsThreads) norm_add_kernel(const NormAddParam
     } else {
       load8(y + (long long)t * p.ldy + c, v[it]);
     }
+    if (NEXT && p.gate != nullptr) {
+      float g[8];
+      load8(reinterpret_cast<const T*>(p.gate) + (long long)t * p.ldg + c, g);
+#pragma unroll
+      for (int q = 0; q < 8; ++q) v[it][q] *= gate_f<T>(g[q]);
+    }
   }
   norm_row<NV>(v, p.w, p.b, p.W, p.n, p.inv_n, p.eps, p.layernorm, 0.f, red);
   float* res = p.residual + (long long)t * p.W;
   T* copy = reinterpret_cast<T*>(p.copy);
+  if constexpr (NEXT) {
+#pragma unroll
+    for (int it = 0; it < NV; ++it) {
+      const int c = (threadIdx.x + it * blockDim.x) * 8;
+      if (c < p.W) {
+        float x[8];
+        load8(res + c, x);
+#pragma unroll
+        for (int q = 0; q < 8; ++q) v[it][q] = fmaf(p.mult, v[it][q], x[q]);
+        if (p.rows == nullptr) store8(res + c, v[it]);
+      }
+    }
+    norm_row<NV>(v, p.next_w, nullptr, p.W, p.n, p.inv_n, p.eps, 0, 0.f, red);
+#pragma unroll
+    for (int it = 0; it < NV; ++it) {
+      const int c = (threadIdx.x + it * blockDim.x) * 8;
+      if (c < p.W) store8(copy + (long long)blockIdx.x * p.W + c, v[it]);
+    }
+    return;
+  }
 #pragma unroll
   for (int it = 0; it < NV; ++it) {
     const int c = (threadIdx.x + it * blockDim.x) * 8;
@@ -388,6 +466,28 @@ __global__ void __launch_bounds__(256) act_mul_f32_kernel(const float* __restric
   }
 }
 
+// out[t, i] = g * sigmoid(alpha g) * (u + 1), g = min(x[t, i], limit), u = x[t, I + i] within +-limit.
+template <typename T>
+__global__ void __launch_bounds__(256) clamped_swiglu_kernel(const T* __restrict__ x, T* __restrict__ out, int I, long long ldx, long long ldo,
+                                                             long long total, float alpha, float limit) {
+  pdl_trigger();
+  pdl_wait();
+  const int per_row = I / 8;
+  for (long long v = blockIdx.x * (long long)blockDim.x + threadIdx.x; v < total; v += (long long)gridDim.x * blockDim.x) {
+    const long long t = v / per_row;
+    const int c = (int)(v - t * per_row) * 8;
+    float g[8], u[8];
+    load8(x + t * ldx + c, g);
+    load8(x + t * ldx + I + c, u);
+#pragma unroll
+    for (int q = 0; q < 8; ++q) {
+      const float a = fminf(g[q], limit), b = fminf(fmaxf(u[q], -limit), limit);
+      g[q] = a * gate_f<T>(alpha * a) * (b + 1.f);
+    }
+    store8(out + t * ldo + c, g);
+  }
+}
+
 // Greedy head over fp32 logits: arg-max (lowest index on ties) and its log-probability.
 __global__ void __launch_bounds__(512) argmax_f32_kernel(const float* __restrict__ logits, long long ld, int V, int* __restrict__ ids,
                                                          float* __restrict__ lps, float softcap) {
@@ -428,7 +528,8 @@ __global__ void __launch_bounds__(512) argmax_f32_kernel(const float* __restrict
 }
 
 // ------------------------------------------------------------------------------------------------
-// Batched product in true fp32: out[b][t, n] = sum_k x[b][t, k] * w[b][n, k] (* sigmoid(gate[t, b])).  64 x 64 tiles.
+// Batched product in true fp32: out[b][t, n] = sum_k x[b][t, k] * w[b][n, k] (* sigmoid(gate[t, b]), or of gate[t, b * N + n]).
+// 64 x 64 tiles.
 // ------------------------------------------------------------------------------------------------
 struct BatchedGemmParams {
   const void* x; const void* w; void* out; const void* gate;
@@ -436,6 +537,7 @@ struct BatchedGemmParams {
   int T, N, K;
   float out_scale;
   const float* bias;           // fp32 product: [N] or null
+  int gate_wide;               // the gate has a column for every output column: b * N + n
 };
 
 __global__ void __launch_bounds__(256) gemm_f32_kernel(const BatchedGemmParams p) {
@@ -473,10 +575,12 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const BatchedGemmParams p
   for (int i = 0; i < 4; ++i) {
     const int t = t0 + ty * 4 + i;
     if (t >= p.T) continue;
-    const float s = p.gate ? p.out_scale * sigmoid_f(reinterpret_cast<const float*>(p.gate)[(long long)t * p.ldg + b]) : p.out_scale;
+    const float* gate = p.gate ? reinterpret_cast<const float*>(p.gate) + (long long)t * p.ldg : nullptr;
+    float s = gate && !p.gate_wide ? p.out_scale * sigmoid_f(gate[b]) : p.out_scale;
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx * 4 + j;
+      if (gate && p.gate_wide && n < p.N) s = p.out_scale * sigmoid_f(gate[(long long)b * p.N + n]);
       if (n < p.N) out[(long long)t * p.ldo + n] = acc[i][j] * s + (p.bias != nullptr ? p.bias[n] : 0.f);
     }
   }
@@ -545,11 +649,18 @@ __global__ void __launch_bounds__(128) gemm_heads_kernel(const BatchedGemmParams
   for (int hr = 0; hr < 2; ++hr) {
     const int t = t0 + warp * 16 + (lane >> 2) + hr * 8;
     if (t >= p.T) continue;
-    const float s = p.gate ? sigmoid_f(to_f(reinterpret_cast<const __nv_bfloat16*>(p.gate)[(long long)t * p.ldg + b])) : 1.f;
+    const __nv_bfloat16* gate = p.gate ? reinterpret_cast<const __nv_bfloat16*>(p.gate) + (long long)t * p.ldg : nullptr;
+    float2 s = make_float2(1.f, 1.f);
+    if (gate && !p.gate_wide) s.x = s.y = sigmoid_f(to_f(gate[b]));
 #pragma unroll
     for (int nt = 0; nt < 8; ++nt) {
       const int n = n0 + nt * 8 + (lane & 3) * 2;
-      if (n < p.N) *reinterpret_cast<uint32_t*>(out + (long long)t * p.ldo + n) = pack_bf16x2(acc[nt][2 * hr] * s, acc[nt][2 * hr + 1] * s);
+      if (n >= p.N) continue;
+      if (gate && p.gate_wide) {
+        const float2 z = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(gate + (long long)b * p.N + n));
+        s = make_float2(gate_f<__nv_bfloat16>(z.x), gate_f<__nv_bfloat16>(z.y));
+      }
+      *reinterpret_cast<uint32_t*>(out + (long long)t * p.ldo + n) = pack_bf16x2(acc[nt][2 * hr] * s.x, acc[nt][2 * hr + 1] * s.y);
     }
   }
 }
@@ -558,17 +669,21 @@ __global__ void __launch_bounds__(128) gemm_heads_kernel(const BatchedGemmParams
 
 extern "C" {
 
+int lx_embed_pairs_bytes() { return (int)sizeof(lx::EmbedPairs); }
+
 // `f32` selects the element type of activations and weights everywhere below (0: bf16, 1: fp32).
 int lx_embed_stream(const int* ids, const void* table, void* out, int T, int W, int V, float mult, const void* pos, const int* positions, int P,
-                    void* copy, int f32, void* stream) {
+                    void* copy, const void* pairs, int f32, void* stream) {
   using namespace lx;
   if (T <= 0) return 0;
   if (W % 8 != 0 || V <= 0 || (pos != nullptr && P <= 0)) return -1;
+  const EmbedPairs e = pairs != nullptr ? *reinterpret_cast<const EmbedPairs*>(pairs) : EmbedPairs{};
+  if (e.vectors != nullptr && (e.buckets <= 0 || e.page <= 0 || e.mul_prev < 0 || e.mul_cur < 0 || e.slots == nullptr || e.pages == nullptr)) return -2;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   float* o = reinterpret_cast<float*>(out);
 #define LX_ES(TY)                                                                                                                        \
   launch_pdl(embed_stream_kernel<TY>, dim3(T), dim3(128), 0, s, ids, reinterpret_cast<const TY*>(table), o, W, V, mult,                     \
-             reinterpret_cast<const TY*>(pos), positions, P, reinterpret_cast<TY*>(copy))
+             reinterpret_cast<const TY*>(pos), positions, P, reinterpret_cast<TY*>(copy), e)
   if (f32) LX_ES(float); else LX_ES(__nv_bfloat16);
 #undef LX_ES
   return -(int)cudaGetLastError();
@@ -576,21 +691,26 @@ int lx_embed_stream(const int* ids, const void* table, void* out, int T, int W, 
 
 int lx_norm_add_bytes() { return (int)sizeof(lx::NormAddParams); }
 
+// T: rows of y (with p.rows: of the result).
 int lx_norm_add(const void* params, int T, int f32, void* stream) {
   using namespace lx;
   const NormAddParams& p = *reinterpret_cast<const NormAddParams*>(params);
   if (T <= 0) return 0;
   if (p.W % 8 != 0 || p.W > kNsThreads * kNsMaxVec * 8 || p.n <= 0 || p.n > p.W || p.ldy % 8 != 0 || p.ldy < p.W) return -1;
+  if (p.next_w != nullptr ? p.copy == nullptr || (p.gate != nullptr && p.ldg % 8 != 0) : p.gate != nullptr || p.rows != nullptr) return -2;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const int threads = p.W / 8 >= kNsThreads ? kNsThreads : (p.W / 8 + 31) / 32 * 32;
   const int nv = (p.W / 8 + threads - 1) / threads;
-#define LX_NA(TY, PR)                                                                                   \
-  if (nv <= 1) launch_pdl(norm_add_kernel<TY, PR, 1>, dim3(T), dim3(threads), 0, s, p);                   \
-  else if (nv <= 2) launch_pdl(norm_add_kernel<TY, PR, 2>, dim3(T), dim3(threads), 0, s, p);              \
-  else if (nv <= 4) launch_pdl(norm_add_kernel<TY, PR, 4>, dim3(T), dim3(threads), 0, s, p);              \
-  else launch_pdl(norm_add_kernel<TY, PR, kNsMaxVec>, dim3(T), dim3(threads), 0, s, p);
-  if (f32) { if (p.pos != nullptr) { LX_NA(float, true) } else { LX_NA(float, false) } }
-  else { if (p.pos != nullptr) { LX_NA(__nv_bfloat16, true) } else { LX_NA(__nv_bfloat16, false) } }
+#define LX_NA(TY, PR, NX)                                                                                   \
+  if (nv <= 1) launch_pdl(norm_add_kernel<TY, PR, 1, NX>, dim3(T), dim3(threads), 0, s, p);                   \
+  else if (nv <= 2) launch_pdl(norm_add_kernel<TY, PR, 2, NX>, dim3(T), dim3(threads), 0, s, p);              \
+  else if (nv <= 4) launch_pdl(norm_add_kernel<TY, PR, 4, NX>, dim3(T), dim3(threads), 0, s, p);              \
+  else launch_pdl(norm_add_kernel<TY, PR, kNsMaxVec, NX>, dim3(T), dim3(threads), 0, s, p);
+#define LX_NAP(TY, NX)  \
+  if (p.pos != nullptr) { LX_NA(TY, true, NX) } else { LX_NA(TY, false, NX) }
+  if (f32) { if (p.next_w != nullptr) { LX_NAP(float, true) } else { LX_NAP(float, false) } }
+  else { if (p.next_w != nullptr) { LX_NAP(__nv_bfloat16, true) } else { LX_NAP(__nv_bfloat16, false) } }
+#undef LX_NAP
 #undef LX_NA
   return -(int)cudaGetLastError();
 }
@@ -696,6 +816,20 @@ int lx_act_mul_f32(const void* x, void* out, int T, int I, long long ldx, long l
   return -(int)cudaGetLastError();
 }
 
+int lx_clamped_swiglu(const void* x, void* out, int T, int I, long long ldx, long long ldo, float alpha, float limit, int f32, void* stream) {
+  using namespace lx;
+  if (T <= 0) return 0;
+  if (I % 8 != 0 || ldx % 8 != 0 || ldo % 8 != 0) return -1;
+  const long long total = (long long)T * (I / 8);
+  const int grid = (int)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16);
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+#define LX_CS(TY) \
+  launch_pdl(clamped_swiglu_kernel<TY>, dim3(grid), dim3(256), 0, s, reinterpret_cast<const TY*>(x), reinterpret_cast<TY*>(out), I, ldx, ldo, total, alpha, limit)
+  if (f32) LX_CS(float); else LX_CS(__nv_bfloat16);
+#undef LX_CS
+  return -(int)cudaGetLastError();
+}
+
 int lx_argmax_f32(const void* logits, long long ld, int T, int V, int* ids, float* logprobs, float softcap, void* stream) {
   using namespace lx;
   if (T <= 0) return 0;
@@ -704,13 +838,14 @@ int lx_argmax_f32(const void* logits, long long ld, int T, int V, int* ids, floa
   return -(int)cudaGetLastError();
 }
 
-// out[b][t, n] = x[b][t, :] . w[b][n, :] over `batch` products with element strides sx / sw / so; gate [T, ldg]: column b.  bias [N]: fp32 only.
+// out[b][t, n] = x[b][t, :] . w[b][n, :] over `batch` products with element strides sx / sw / so; gate [T, ldg]: column b, or
+// (gate_wide) column b * N + n.  bias [N]: fp32 only.
 int lx_gemm_batched(const void* x, long long ldx, long long sx, const void* w, long long ldw, long long sw, void* out, long long ldo,
-                    long long so, const void* gate, long long ldg, int T, int N, int K, int batch, float out_scale, const float* bias, int f32,
-                    void* stream) {
+                    long long so, const void* gate, long long ldg, int T, int N, int K, int batch, float out_scale, const float* bias, int gate_wide,
+                    int f32, void* stream) {
   using namespace lx;
   if (T <= 0 || N <= 0 || batch <= 0) return 0;
-  BatchedGemmParams p{x, w, out, gate, ldx, sx, ldw, sw, ldo, so, ldg, T, N, K, out_scale, bias};
+  BatchedGemmParams p{x, w, out, gate, ldx, sx, ldw, sw, ldo, so, ldg, T, N, K, out_scale, bias, gate_wide};
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const dim3 grid((N + 63) / 64, (T + 63) / 64, batch);
   if (bias != nullptr && !f32) return -2;
@@ -718,6 +853,7 @@ int lx_gemm_batched(const void* x, long long ldx, long long sx, const void* w, l
     launch_pdl(gemm_f32_kernel, grid, dim3(256), 0, s, p);
   } else {
     if (K % 8 != 0 || N % 2 != 0 || ldx % 8 != 0 || sx % 8 != 0 || ldw % 8 != 0 || sw % 8 != 0 || ldo % 2 != 0 || so % 2 != 0) return -1;
+    if (gate_wide && ldg % 2 != 0) return -3;
     launch_pdl(gemm_heads_kernel, grid, dim3(128), 0, s, p);
   }
   return -(int)cudaGetLastError();

@@ -17,7 +17,7 @@ from typing import NamedTuple, Optional
 
 import torch
 
-from .reference import MoeRouting
+from .reference import CLAMPED_SWIGLU_ALPHA, MoeRouting
 
 _PKG = Path(__file__).resolve().parent.parent
 _LIB_PATH = _PKG / "_lx_kernels.so"
@@ -324,7 +324,7 @@ class MoeSelectParams(ctypes.Structure):
     _fields_ = [("logits", c_void_p), ("correction", c_void_p), ("topk_ids", c_void_p), ("topk_w", c_void_p), ("rank", c_void_p),
                 ("counts", c_void_p), ("ldl", c_longlong), ("T", c_int), ("E", c_int), ("k", c_int), ("e0", c_int), ("e_local", c_int),
                 ("sigmoid", c_int), ("groups", c_int), ("keep", c_int), ("shared", c_int), ("group_top", c_int),
-                ("renorm", c_int), ("scale", c_float)]
+                ("renorm", c_int), ("scale", c_float), ("shared_one", c_int), ("bias", c_void_p)]
 
 
 class MoePlaceParams(ctypes.Structure):
@@ -336,7 +336,7 @@ class MoePlaceParams(ctypes.Structure):
 
 def moe_route(x: torch.Tensor, router_w: torch.Tensor, k: int, e0: int, e_local: int, experts: Optional[int] = None, score: str = "softmax",
               correction: Optional[torch.Tensor] = None, groups: int = 0, keep: int = 0, scale: float = 1.0, shared: int = 0, group_top: int = 2,
-              renorm: bool = True) -> MoeRouting:
+              renorm: bool = True, bias: Optional[torch.Tensor] = None, shared_gate: bool = True) -> MoeRouting:
     """Router logits (fp32), choice of `k` experts per token (`reference.moe_route` states the rules), and the sorted order of the rows
     routed to the experts [e0, e0 + e_local) this rank owns with those rows gathered: three launches, everything stays on the device."""
     T, H = x.shape
@@ -358,7 +358,7 @@ def moe_route(x: torch.Tensor, router_w: torch.Tensor, k: int, e0: int, e_local:
                    torch.empty(e_local + shared + 1, dtype=torch.int32, device=dev), torch.empty(T, kw, dtype=torch.int32, device=dev),
                    torch.empty(T * (k + (1 if shared else 0)), H, dtype=x.dtype, device=dev))
     p = MoeSelectParams(_ptr(logits), _ptr(correction), _ptr(r.topk_ids), _ptr(r.topk_w), _ptr(rank), _ptr(counts), logits.stride(0), T, E, k,
-                        e0, e_local, int(score == "sigmoid"), groups, keep, shared, group_top, int(renorm), scale)
+                        e0, e_local, int(score == "sigmoid"), groups, keep, shared, group_top, int(renorm), scale, int(not shared_gate), _ptr(bias))
     _check(lib.lx_moe_select(ctypes.byref(p), _stream()), "lx_moe_select")
     size = x.element_size()
     q = MoePlaceParams(_ptr(x), _ptr(r.xg), x.stride(0) * size, r.xg.stride(0) * size, H * size, _ptr(counts), _ptr(r.topk_ids), _ptr(rank),
@@ -532,10 +532,15 @@ def rope_kvwrite(qkv: torch.Tensor, positions: torch.Tensor, cos_sin: torch.Tens
 _ACTS = {"silu": 0, "swish": 0, "gelu": 1, "gelu_new": 2, "gelu_pytorch_tanh": 2, "gelu_fast": 2, "gelu_tanh": 2, "relu": 3, "relu2": 4}
 
 
-def act_mul(x: torch.Tensor, inter: int, act: str = "silu", gated: bool = True, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+def act_mul(x: torch.Tensor, inter: int, act: str = "silu", gated: bool = True, out: Optional[torch.Tensor] = None,
+            limit: float = 0.0) -> torch.Tensor:
     T = x.shape[0]
     if out is None:
         out = torch.empty(T, inter, dtype=x.dtype, device=x.device)
+    if act == "clamped_swiglu":
+        _check(load().lx_clamped_swiglu(_ptr(x), _ptr(out), T, inter, x.stride(0), out.stride(0), CLAMPED_SWIGLU_ALPHA, limit,
+                                        int(x.dtype == torch.float32), _stream()), "lx_clamped_swiglu")
+        return out
     if x.dtype == torch.float32:
         _check(load().lx_act_mul_f32(_ptr(x), _ptr(out), T, inter, x.stride(0), out.stride(0), _ACTS[act], int(gated), _stream()), "lx_act_mul_f32")
         return out

@@ -19,6 +19,10 @@ class StepRows(Structure):
                 ("bt", P), ("max_blocks", I), ("dec_max_blocks", I)]
 
 
+class EmbedPairs(Structure):
+    _fields_ = [("vectors", P), ("pages", P), ("slots", P), ("mul_prev", L), ("mul_cur", L), ("buckets", I), ("page", I), ("rows", StepRows)]
+
+
 class RecParams(Structure):
     _fields_ = [("q", P), ("k", P), ("v", P), ("z", P), ("ldq", L), ("ldk", L), ("ldv", L), ("ldz", L), ("decay", P), ("w0", P), ("u", P), ("skip", P),
                 ("state", P), ("out", P), ("H", I), ("d", I), ("dv", I), ("hpg", I), ("rows", StepRows), ("seg_seq", P), ("seg_q0", P), ("nseg", I),
@@ -39,32 +43,33 @@ class WkvTcParams(Structure):
 class LatentPrepParams(Structure):
     _fields_ = [("dq", P), ("dkv", P), ("ld_dq", L), ("ld_dkv", L), ("dq_norm", P), ("dkv_norm", P), ("cq", P), ("cache", P),
                 ("positions", P), ("slots", P), ("cos_sin", P), ("QR", I), ("KR", I), ("R", I), ("q_rank", I), ("kv_rank", I), ("rot", I),
-                ("eps", F)]
+                ("eps", F), ("q", P), ("ldq", L), ("H", I), ("head", I), ("off", I)]
 
 
 class LatentAttnParams(Structure):
     _fields_ = [("q_lat", P), ("ld_ql", L), ("q", P), ("ldq", L), ("head", I), ("rot_off", I), ("cache", P), ("out", P), ("ldo", L),
-                ("rows", StepRows), ("H", I), ("KR", I), ("R", I), ("page", I), ("scale", F)]
+                ("rows", StepRows), ("H", I), ("KR", I), ("R", I), ("page", I), ("scale", F), ("window", I)]
 
 
 class LatentDecodeParams(Structure):
     _fields_ = [("q_lat", P), ("ld_ql", L), ("q", P), ("ldq", L), ("head", I), ("rot_off", I), ("cache", P), ("out", P), ("ldo", L),
-                ("rows", StepRows), ("H", I), ("R", I), ("page", I), ("nsplit", I), ("scale", F), ("part_o", P), ("part_ml", P)]
+                ("rows", StepRows), ("H", I), ("R", I), ("page", I), ("nsplit", I), ("scale", F), ("part_o", P), ("part_ml", P), ("window", I)]
 
 
 class NormAddParams(Structure):
     _fields_ = [("residual", P), ("y", P), ("ldy", L), ("w", P), ("b", P), ("copy", P), ("pos", P), ("weights", P), ("k", I), ("W", I), ("n", I),
-                ("layernorm", I), ("inv_n", F), ("eps", F), ("mult", F)]
+                ("layernorm", I), ("inv_n", F), ("eps", F), ("mult", F), ("gate", P), ("ldg", L), ("next_w", P), ("rows", P)]
 
 
 class QkNormParams(Structure):
     _fields_ = [("qkv", P), ("ld", L), ("cache", P), ("slots", P), ("q_norm", P), ("k_norm", P), ("T", I), ("H", I), ("G", I), ("DK", I),
-                ("DV", I), ("page", I), ("inv_n", F), ("eps", F)]
+                ("DV", I), ("page", I), ("inv_n", F), ("eps", F), ("positions", P), ("cos_sin", P), ("v_cos_sin", P), ("rot", I), ("v_rot", I), ("P", I)]
 
 
 class GqaF32Params(Structure):
     _fields_ = [("q", P), ("ldq", L), ("cache", P), ("out", P), ("ldo", L), ("rows", StepRows), ("T", I), ("H", I), ("G", I), ("DK", I),
-                ("DV", I), ("page", I), ("window", I), ("scale", F), ("softcap", F), ("out_scale", F), ("sink", P), ("gate", P), ("ldg", L)]
+                ("DV", I), ("page", I), ("window", I), ("scale", F), ("softcap", F), ("out_scale", F), ("sink", P), ("gate", P), ("ldg", L), ("turn", P),
+                ("turn_dims", I), ("turn_rows", I)]
 
 
 class NormStreamParams(Structure):
@@ -83,7 +88,8 @@ class ConvParams(Structure):
 
 
 SIGNATURES = {
-    "lx_embed_stream": ([P, P, P, I, I, I, F, P, P, I, P, I, P], I),
+    "lx_embed_pairs_bytes": ([], I),
+    "lx_embed_stream": ([P, P, P, I, I, I, F, P, P, I, P, P, I, P], I),
     "lx_norm_add_bytes": ([], I),
     "lx_norm_add": ([P, I, I, P], I),
     "lx_norm_rows": ([P, P, P, P, P, I, I, I, F, F, I, I, P], I),
@@ -92,9 +98,9 @@ SIGNATURES = {
     "lx_qk_norm_kvwrite": ([P, I, P], I),
     "lx_gqa_f32_bytes": ([], I),
     "lx_gqa_attn_f32": ([P, P], I),
-    "lx_gqa_decode": ([P, L, P, P, I, P, P, L, P, P, I, I, I, I, I, I, F, I, F, P, P, L, F, P], I),
-    "lx_gqa_prefill": ([P, L, P, P, I, P, P, P, P, I, P, L, I, I, I, I, I, F, F, P, P, L, F, P], I),
-    "lx_gqa_prefill_tc": ([P, L, I, P, I, P, I, P, P, P, P, I, P, L, I, I, I, I, F, F, P, P, L, F, P, P], I),
+    "lx_gqa_decode": ([P, L, P, P, I, P, P, L, P, P, I, I, I, I, I, I, F, I, F, P, P, L, F, P, I, I, P], I),
+    "lx_gqa_prefill": ([P, L, P, P, I, P, P, P, P, I, P, L, I, I, I, I, I, F, F, P, P, L, F, P, I, I, P], I),
+    "lx_gqa_prefill_tc": ([P, L, I, P, I, P, I, P, P, P, P, I, P, L, I, I, I, I, F, F, P, P, L, F, P, I, I, P, P], I),
     "lx_norm_stream_bytes": ([], I),
     "lx_norm_stream": ([P, I, I, P], I),
     "lx_gate_norm_bytes": ([], I),
@@ -104,8 +110,9 @@ SIGNATURES = {
     "lx_norm_gate": ([P, P, P, L, P, L, I, I, I, I, F, I, I, P], I),
     "lx_tanh": ([P, L, I, P], I),
     "lx_act_mul_f32": ([P, P, I, I, L, L, I, I, P], I),
+    "lx_clamped_swiglu": ([P, P, I, I, L, L, F, F, I, P], I),
     "lx_argmax_f32": ([P, L, I, I, P, P, F, P], I),
-    "lx_gemm_batched": ([P, L, L, P, L, L, P, L, L, P, L, I, I, I, I, F, P, I, P], I),
+    "lx_gemm_batched": ([P, L, L, P, L, L, P, L, L, P, L, I, I, I, I, F, P, I, I, P], I),
     "lx_step_rows_bytes": ([], I),
     "lx_rec_params_bytes": ([], I),
     "lx_recurrence": ([P, I, I, I, P], I),
@@ -125,14 +132,14 @@ SIGNATURES = {
     "lx_latent_decode_bytes": ([], I),
     "lx_latent_decode_supported": ([I, I], I),
     "lx_latent_decode": ([P, I, I, P], I),
-    "lx_latent_gather": ([P, P, I, P, I, I, I, I, I, P, P, P], I),
+    "lx_latent_gather": ([P, P, I, P, P, I, I, I, I, I, I, P, P, P], I),
     "lx_latent_prefill_supported": ([I, I, I], I),
-    "lx_latent_prefill": ([P, L, I, P, P, I, P, P, P, P, P, I, P, L, P, L, I, I, I, I, F, P, P], I),
+    "lx_latent_prefill": ([P, L, I, P, P, I, P, P, P, P, P, I, P, L, P, L, I, I, I, I, F, I, I, P, P], I),
 }
 
 
 def check_layouts(lib):
-    for name, st in (("lx_step_rows_bytes", StepRows), ("lx_rec_params_bytes", RecParams), ("lx_latent_prep_bytes", LatentPrepParams),
+    for name, st in (("lx_step_rows_bytes", StepRows), ("lx_embed_pairs_bytes", EmbedPairs), ("lx_rec_params_bytes", RecParams), ("lx_latent_prep_bytes", LatentPrepParams),
                      ("lx_latent_attn_bytes", LatentAttnParams), ("lx_latent_decode_bytes", LatentDecodeParams),
                      ("lx_linear_attn_tc_bytes", LinTcParams), ("lx_wkv_tc_bytes", WkvTcParams),
                      ("lx_norm_add_bytes", NormAddParams), ("lx_qk_norm_bytes", QkNormParams), ("lx_gqa_f32_bytes", GqaF32Params),
@@ -161,11 +168,15 @@ def step_rows(inp, T: int) -> StepRows:
     return r
 
 
-def embed_stream(ids, table, mult: float = 1.0, pos=None, positions=None, copy=None):
+def embed_stream(ids, table, mult: float = 1.0, pos=None, positions=None, copy=None, bigram=None):
     T, W = ids.shape[0], table.shape[1]
     out = torch.empty(T, W, dtype=torch.float32, device=table.device)
+    pairs = None
+    if bigram is not None:
+        vectors, (buckets, mul_prev, mul_cur), pages, inp = bigram
+        pairs = ctypes.byref(EmbedPairs(_p(vectors), _p(pages), _p(inp.slots), mul_prev, mul_cur, buckets, pages.shape[1], step_rows(inp, T)))
     nv._check(nv.load().lx_embed_stream(_p(ids), _p(table), _p(out), T, W, table.shape[0], mult, _p(pos), _p(positions) if pos is not None else None,
-                                        pos.shape[0] if pos is not None else 0, _p(copy), _f32(table), nv._stream()), "lx_embed_stream")
+                                        pos.shape[0] if pos is not None else 0, _p(copy), pairs, _f32(table), nv._stream()), "lx_embed_stream")
     return out
 
 
@@ -190,12 +201,15 @@ def norm_stream(residual, pending, weight, eps: float, weight_offset: float, n: 
     return out
 
 
-def norm_add(residual, y, weight, bias, mult: float, eps: float, n: int, dtype, layernorm: bool = True, pairs=None):
+def norm_add(residual, y, weight, bias, mult: float, eps: float, n: int, dtype, layernorm: bool = True, pairs=None, gate=None,
+             next_weight=None, rows=None):
     T, W = residual.shape
-    copy = torch.empty(T, W, dtype=dtype, device=residual.device) if dtype != torch.float32 else None
+    if rows is not None:
+        T = rows.shape[0]
+    copy = torch.empty(T, W, dtype=dtype, device=residual.device) if dtype != torch.float32 or next_weight is not None else None
     pos, w = pairs if pairs is not None else (None, None)
     p = NormAddParams(_p(residual), _p(y), y.stride(0), _p(weight), _p(bias), _p(copy), _p(pos), _p(w), pos.shape[1] if pos is not None else 0, W,
-                      n, int(layernorm), 1.0 / n, eps, mult)
+                      n, int(layernorm), 1.0 / n, eps, mult, _p(gate), gate.stride(0) if gate is not None else 0, _p(next_weight), _p(rows))
     nv._check(nv.load().lx_norm_add(ctypes.byref(p), T, _f32(y), nv._stream()), "lx_norm_add")
     return residual if copy is None else copy
 
@@ -226,7 +240,7 @@ def gemm_f32(x, w, out=None, out_scale: float = 1.0, bias=None):
     if out is None:
         out = torch.empty(T, N, dtype=torch.float32, device=x.device)
     nv._check(nv.load().lx_gemm_batched(_p(x), x.stride(0), 0, _p(w), w.stride(0), 0, _p(out), out.stride(0), 0, None, 0, T, N, K, 1, out_scale,
-                                        _p(bias), 1, nv._stream()), "lx_gemm_batched")
+                                        _p(bias), 0, 1, nv._stream()), "lx_gemm_batched")
     return out
 
 
@@ -255,12 +269,12 @@ def gemm_stack(x, w):
     return out
 
 
-def gemm_heads(x, w, out, x_head: int, gate=None):
-    """out[:, h * N : (h + 1) * N] = x[:, h * x_head : h * x_head + K] @ w[h]^T (* sigmoid(gate[:, h]))."""
+def gemm_heads(x, w, out, x_head: int, gate=None, wide_gate: bool = False):
+    """out[:, h * N : (h + 1) * N] = x[:, h * x_head : h * x_head + K] @ w[h]^T (* sigmoid(gate[:, h]), or of the output's own gate column)."""
     H, N, K = w.shape
     T = x.shape[0]
     nv._check(nv.load().lx_gemm_batched(_p(x), x.stride(0), x_head, _p(w), K, N * K, _p(out), out.stride(0), N, _p(gate),
-                                        gate.stride(0) if gate is not None else 0, T, N, K, H, 1.0, None, _f32(x), nv._stream()),
+                                        gate.stride(0) if gate is not None else 0, T, N, K, H, 1.0, None, int(wide_gate), _f32(x), nv._stream()),
               "lx_gemm_batched")
     return out
 
@@ -372,12 +386,13 @@ def token_shift(h, mu, shift, inp):
     return out
 
 
-def latent_prep(dq, dkv, dq_norm, dkv_norm, q_rank: int, kv_rank: int, rot: int, eps: float, cos_sin, positions, slots, cache):
-    T, QR, KR = dq.shape[0], dq_norm.shape[0], dkv_norm.shape[0]
-    cq = torch.empty(T, QR, dtype=dq.dtype, device=dq.device)
-    p = LatentPrepParams(_p(dq), _p(dkv), dq.stride(0), dkv.stride(0), _p(dq_norm), _p(dkv_norm), _p(cq), _p(cache), _p(positions), _p(slots),
-                         _p(cos_sin), QR, KR, cache.shape[2], q_rank, kv_rank, rot, eps)
-    nv._check(nv.load().lx_latent_prep(ctypes.byref(p), T, _f32(dq), nv._stream()), "lx_latent_prep")
+def latent_prep(dq, dkv, dq_norm, dkv_norm, q_rank: int, kv_rank: int, rot: int, eps: float, cos_sin, positions, slots, cache, q=None,
+                heads: int = 0, head: int = 0, off: int = 0):
+    T, QR, KR = dkv.shape[0], dq_norm.shape[0] if dq is not None else 0, dkv_norm.shape[0]
+    cq = torch.empty(T, QR, dtype=dq.dtype, device=dq.device) if dq is not None else None
+    p = LatentPrepParams(_p(dq), _p(dkv), dq.stride(0) if dq is not None else 0, dkv.stride(0), _p(dq_norm), _p(dkv_norm), _p(cq), _p(cache), _p(positions), _p(slots),
+                         _p(cos_sin), QR, KR, cache.shape[2], q_rank, kv_rank, rot, eps, _p(q), q.stride(0) if q is not None else 0, heads, head, off)
+    nv._check(nv.load().lx_latent_prep(ctypes.byref(p), T, _f32(dkv), nv._stream()), "lx_latent_prep")
     return cq
 
 
@@ -386,7 +401,7 @@ def rope_pairs(x, positions, cos_sin, H: int, head: int, off: int, rot: int):
               "lx_rope_pairs")
 
 
-def latent_attn(q_lat, q, cache, H: int, kv_rank: int, head: int, rot_off: int, rot: int, scale: float, inp):
+def latent_attn(q_lat, q, cache, H: int, kv_rank: int, head: int, rot_off: int, rot: int, scale: float, inp, window: int = 0):
     T = q.shape[0]
     out = torch.empty(T, H * kv_rank, dtype=q.dtype, device=q.device)
     lib = nv.load()
@@ -398,6 +413,9 @@ def latent_attn(q_lat, q, cache, H: int, kv_rank: int, head: int, rot_off: int, 
         # the keys of a row are shared out until the grid fills the GPU once (one CTA per SM, two for up to 16 heads)
         groups, per_sm = ((H + 31) // 32, 1) if H > 16 else (1, 2)
         d.nsplit = max(1, min(32, nv.workspace(q.device).num_sms * per_sm // (T * groups)))
+        d.window = window
+        if window > 0:                                       # (no share without a 64-key tile)
+            d.nsplit = min(d.nsplit, window // 64 + 1)
         hold = None
         if d.nsplit > 1:
             n = T * H * d.nsplit
@@ -409,7 +427,7 @@ def latent_attn(q_lat, q, cache, H: int, kv_rank: int, head: int, rot_off: int, 
     p = LatentAttnParams()
     p.q_lat, p.ld_ql, p.q, p.ldq, p.head, p.rot_off = _p(q_lat), q_lat.stride(0), _p(q), q.stride(0), head, rot_off
     p.cache, p.out, p.ldo, p.rows = _p(cache), _p(out), out.stride(0), step_rows(inp, T)
-    p.H, p.KR, p.R, p.page, p.scale = H, kv_rank, kv_rank + rot, cache.shape[1], scale
+    p.H, p.KR, p.R, p.page, p.scale, p.window = H, kv_rank, kv_rank + rot, cache.shape[1], scale, window
     nv._check(nv.load().lx_latent_attn(ctypes.byref(p), T, _f32(q), nv._stream()), "lx_latent_attn")
     return out
 
@@ -419,30 +437,35 @@ def latent_attn(q_lat, q, cache, H: int, kv_rank: int, head: int, rot_off: int, 
 LATENT_EXPAND_MIN_ROWS = 24
 
 
-def latent_prefill(q, cache, w_ukv, gate, out, H: int, dk: int, rot: int, dv: int, scale: float, inp, nd: int) -> bool:
+def latent_prefill(q, cache, w_ukv, gate, out, H: int, dk: int, rot: int, dv: int, scale: float, inp, nd: int, window: int = 0,
+                   wide_gate: bool = False) -> bool:
     """Gated attention outputs of the prompt rows [nd, T) into out[nd:, : H * dv] on the tensor-core kernel; False when this step is
     better (or only) served by the absorbed form."""
     T, B = q.shape[0] - nd, inp.cache_lens.shape[0]
     lib = nv.load()
     if q.dtype != torch.bfloat16 or T < LATENT_EXPAND_MIN_ROWS * B or not lib.lx_latent_prefill_supported(dk, rot, dv):
         return False
-    rows, KR, dev = inp.ctx_total, cache.shape[2] - rot, q.device
+    ctx_off, rows = inp.contexts[window]
+    KR, dev = cache.shape[2] - rot, q.device
     lat = torch.empty(rows, KR, dtype=q.dtype, device=dev)
     keys = torch.empty(rows, rot, dtype=q.dtype, device=dev)
-    nv._check(lib.lx_latent_gather(_p(cache), _p(inp.block_tables), inp.block_tables.shape[1], _p(inp.ctx_off), B, rows, cache.shape[1], KR, rot,
-                                   _p(lat), _p(keys), nv._stream()), "lx_latent_gather")
+    nv._check(lib.lx_latent_gather(_p(cache), _p(inp.block_tables), inp.block_tables.shape[1], _p(ctx_off), _p(inp.cache_lens), window, B, rows,
+                                   cache.shape[1], KR, rot, _p(lat), _p(keys), nv._stream()), "lx_latent_gather")
     kv = nv.gemm(lat, w_ukv)
     y, g = out[nd:], gate[nd:]
     qp = q[nd:]
-    nv._check(lib.lx_latent_prefill(_p(qp), qp.stride(0), T, _p(kv), _p(keys), rows, _p(inp.ctx_off), _p(inp.cu_q), _p(inp.cache_lens),
+    nv._check(lib.lx_latent_prefill(_p(qp), qp.stride(0), T, _p(kv), _p(keys), rows, _p(ctx_off), _p(inp.cu_q), _p(inp.cache_lens),
                                     _p(inp.q128_seq), _p(inp.q128_q0), inp.q128_seq.shape[0], _p(g), g.stride(0), _p(y), y.stride(0), H, dk, rot,
-                                    dv, scale, _p(nv.workspace(dev).status), nv._stream()), "lx_latent_prefill")
+                                    dv, scale, window, int(wide_gate), _p(nv.workspace(dev).status), nv._stream()), "lx_latent_prefill")
     return True
 
 
-def qk_norm_kvwrite(qkv, H: int, G: int, dk: int, dv: int, n: int, q_norm, k_norm, eps: float, cache, slots):
+def qk_norm_kvwrite(qkv, H: int, G: int, dk: int, dv: int, n: int, q_norm, k_norm, eps: float, cache, slots, positions=None,
+                    cos_sin=None, v_cos_sin=None):
+    width = lambda t: t.shape[1] if t is not None else 0
+    rows = min([t.shape[0] for t in (cos_sin, v_cos_sin) if t is not None] + [1 << 30])
     p = QkNormParams(_p(qkv), qkv.stride(0), _p(cache), _p(slots), _p(q_norm), _p(k_norm), qkv.shape[0], H, G, dk, dv,
-                     cache.shape[2] // (dk + dv), 1.0 / n, eps)
+                     cache.shape[2] // (dk + dv), 1.0 / n, eps, _p(positions), _p(cos_sin), _p(v_cos_sin), width(cos_sin), width(v_cos_sin), rows)
     nv._check(nv.load().lx_qk_norm_kvwrite(ctypes.byref(p), _f32(qkv), nv._stream()), "lx_qk_norm_kvwrite")
 
 
@@ -456,14 +479,15 @@ def _gqa_splits(ctas: int, window: int, max_blocks: int, page: int) -> int:
 
 
 def gqa_attn(q, cache, H: int, G: int, dk: int, dv: int, scale: float, window: int, inp, out, softcap: float = 0.0, sink=None, gate=None,
-             out_scale: float = 1.0):
+             out_scale: float = 1.0, turn_back=None):
     T = q.shape[0]
+    turn = (_p(turn_back), turn_back.shape[1], turn_back.shape[0]) if turn_back is not None else (None, 0, 0)
     lib, ws = nv.load(), nv.workspace(q.device)
     page = cache.shape[2] // (dk + dv)
     ldg = gate.stride(0) if gate is not None else 0
     if q.dtype == torch.float32:
         p = GqaF32Params(_p(q), q.stride(0), _p(cache), _p(out), out.stride(0), step_rows(inp, T), T, H, G, dk, dv, page, window, scale, softcap,
-                         out_scale, _p(sink), _p(gate), ldg)
+                         out_scale, _p(sink), _p(gate), ldg, *turn)
         nv._check(lib.lx_gqa_attn_f32(ctypes.byref(p), nv._stream()), "lx_gqa_attn_f32")
         return out
     if page != lib.lx_gqa_page_size():
@@ -476,7 +500,7 @@ def gqa_attn(q, cache, H: int, G: int, dk: int, dv: int, scale: float, window: i
             part_o = torch.empty(nd * H * nsplit * (dv + 1), dtype=torch.float32, device=q.device)
             part_lse = part_o[nd * H * nsplit * dv:]
         nv._check(lib.lx_gqa_decode(_p(q), q.stride(0), _p(cache), _p(dbt), dbt.shape[1], _p(ctx), _p(out), out.stride(0), _p(part_o), _p(part_lse),
-                                    nd, H, G, dk, dv, window, scale, nsplit, softcap, _p(sink), _p(gate), ldg, out_scale, nv._stream()),
+                                    nd, H, G, dk, dv, window, scale, nsplit, softcap, _p(sink), _p(gate), ldg, out_scale, *turn, nv._stream()),
                   "lx_gqa_decode")
         nv.launch_count += int(nsplit > 1)
     if inp.is_prefill:
@@ -485,10 +509,10 @@ def gqa_attn(q, cache, H: int, G: int, dk: int, dv: int, scale: float, window: i
         if nv.TC_PREFILL and dk == dv and lib.lx_attn_prefill_tc_supported(H, G, dk, q.stride(0), out.stride(0)):
             nv._check(lib.lx_gqa_prefill_tc(_p(qp), q.stride(0), T - nd, _p(cache), cache.shape[0], _p(inp.block_tables), inp.block_tables.shape[1],
                                             _p(inp.cu_q), _p(inp.cache_lens), _p(inp.tile_seq), _p(inp.tile_q0), tiles, _p(op), out.stride(0), H, G,
-                                            dk, window, scale, softcap, _p(sink), _p(gp), ldg, out_scale, _p(ws.status), nv._stream()),
+                                            dk, window, scale, softcap, _p(sink), _p(gp), ldg, out_scale, *turn, _p(ws.status), nv._stream()),
                       "lx_gqa_prefill_tc")
         else:
             nv._check(lib.lx_gqa_prefill(_p(qp), q.stride(0), _p(cache), _p(inp.block_tables), inp.block_tables.shape[1], _p(inp.cu_q),
                                          _p(inp.cache_lens), _p(inp.tile_seq), _p(inp.tile_q0), tiles, _p(op), out.stride(0), H, G, dk, dv, window,
-                                         scale, softcap, _p(sink), _p(gp), ldg, out_scale, nv._stream()), "lx_gqa_prefill")
+                                         scale, softcap, _p(sink), _p(gp), ldg, out_scale, *turn, nv._stream()), "lx_gqa_prefill")
     return out

@@ -909,7 +909,7 @@ class RandomWeights:
     def get_tensor(self, name):
         shape = self.shapes[name]
         g = torch.Generator(device=self.device).manual_seed(self.seed * 100003 + self.order[name])
-        t = torch.randn(*shape, generator=g, device=self.device, dtype=torch.float32)
+        t = torch.randn(shape, generator=g, device=self.device, dtype=torch.float32)
         leaf = name.rsplit(".", 1)[-1]
         if ".mu." in name:
             return torch.sigmoid(t)

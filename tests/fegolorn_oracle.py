@@ -165,7 +165,9 @@ def forward(cfg, weights, tokens, layers_out=None):
     eps = cfg["norm"]["eps"]
     x = embed(tokens, W, cfg["embedding"])
     for i, spec in enumerate(cfg["layers"]):
-        p = f"l{spec['weights_of'] if spec.get('weights_of') is not None else i}."
+        while cfg["layers"][i].get("weights_of") is not None:
+            i = cfg["layers"][i]["weights_of"]
+        p = f"l{i}."
         x = sublayer(x, W, p, 1, lambda h: mixer(h, W, p + "mix.", spec, eps), eps)
         if spec.get("mlp"):
             x = sublayer(x, W, p, 2, lambda h: feed_forward(h, W, p + "mlp.", spec["mlp"]), eps)

@@ -578,3 +578,181 @@ def test_32_bit_product_with_bias(T, N, K):
     g = torch.Generator().manual_seed(T)
     x, w, b = torch.randn(T, K, generator=g), torch.randn(N, K, generator=g), torch.randn(N, generator=g)
     close(native.gemm(x.cuda(), w.cuda(), bias=b.cuda()), (x.double() @ w.double().t() + b).float(), torch.float32, tol32=2e-6)
+
+
+# ---------------------------------------------------------------------------------------------- sandwich norms, turned values, windowed latents
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("step", list(STEPS) + ["long"])
+@pytest.mark.parametrize("window", [1, 33, 64, 200])
+@pytest.mark.parametrize("H,dk,rot,dv,kv", [(3, 32, 16, 48, 80), (2, 128, 64, 128, 512), (5, 64, 48, 64, 256), (17, 64, 16, 128, 128), (4, 128, 32, 128, 128)])
+def test_latent_attention_with_windows_and_element_gates(dtype, window, step, H, dk, rot, dv, kv):
+    """Both forms over queries that each match one key far better than all others: inside the window, at its edges, or just outside."""
+    from lorax_b200.ops import native, reference
+    dec, pre = STEPS[step] if step in STEPS else ([1000, 1500], [(1000, 300), (0, 500), (129, 40)])
+    inp, nb, _ = make_step(dec, pre, seed=6, windows=(window,))
+    T, head = inp.positions.shape[0], dk + rot
+    q, cache, uk, uv = latent_case(H, dk, rot, dv, kv, inp, nb, dtype, False)
+    nd, dbt, _, ctx = inp.decode_view(T)
+    for t in range(T):
+        b = int(torch.searchsorted(inp.cu_q[1:], torch.tensor(t - nd), right=True)) if t >= nd else 0
+        bt, keys = (dbt[t], int(ctx[t])) if t < nd else (inp.block_tables[b], int(inp.cache_lens[b]) + (t - nd - int(inp.cu_q[b])) + 1)
+        j = keys - 1 - (0, window - 1, window, window // 2, 1)[t % 5]
+        if 0 <= j < keys:
+            q.view(T, H, head)[t, :, dk:] = (cache[int(bt[j // PAGE]), j % PAGE, kv:].float() * 2.0).to(dtype)
+    wide = torch.randn(T, H * dv + 32, generator=torch.Generator().manual_seed(9)).to(dtype)
+    gate, scale = wide[:, 16: 16 + H * dv], head ** -0.5
+    ql, want = torch.empty(T, H * kv), torch.zeros(T, H * dv)
+    reference.gemm_heads(q.float(), uk.float().transpose(1, 2).contiguous(), ql, head)
+    o = reference.latent_attn(ql, q.float(), cache.float(), H, kv, head, dk, rot, scale, inp, window=window)
+    reference.gemm_heads(o, uv.float(), want, kv, gate=gate.float(), wide_gate=True)
+    live = [i for i in range(T) if i >= len(dec) or dec[i] > 0]
+
+    d, gd = to_dev(inp), wide.cuda()[:, 16: 16 + H * dv]
+    rows = torch.zeros(T, H * head + 64, dtype=dtype, device="cuda")              # (queries within wider rows)
+    qd, cd = rows[:, : H * head].copy_(q.cuda()), cache.cuda()
+    qld, got = torch.empty(T, H * kv, dtype=dtype, device="cuda"), torch.zeros(T, H * dv, dtype=dtype, device="cuda")
+    native.gemm_heads(qd, uk.transpose(1, 2).contiguous().cuda(), qld, head)
+    od = native.latent_attn(qld, qd, cd, H, kv, head, dk, rot, scale, d, window=window)
+    native.gemm_heads(od, uv.cuda(), got, kv, gate=gd, wide_gate=True)
+    close(got, want, dtype, live)
+    if pre:
+        ukv = torch.cat([uk, uv], 1).reshape(H * (dk + dv), kv).contiguous().cuda()
+        out = torch.zeros(T, H * dv, dtype=dtype, device="cuda")
+        done = native.latent_prefill(qd, cd, ukv, gd, out, H, dk, rot, dv, scale, d, len(dec), window=window, wide_gate=True)
+        assert done == (dtype == torch.bfloat16 and dk != 32 and T - len(dec) >= native.LATENT_EXPAND_MIN_ROWS * len(pre))
+        if done:
+            native.workspace(out.device).check_status()
+            close(out, want, dtype, list(range(len(dec), T)))
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("rot,rp,H,dk", [(10, 16, 3, 32), (64, 64, 5, 128), (16, 16, 9, 48)])
+def test_latent_preparation_without_a_query_latent(dtype, rot, rp, H, dk):
+    from lorax_b200.ops import native, reference
+    inp, nb, _ = make_step([7, 0, 40], [(0, 50), (33, 5)], seed=8)
+    T, kr, head = inp.positions.shape[0], 80, dk + rp
+    g = torch.Generator().manual_seed(rot)
+    x = torch.randn(T, H * head + kr + rp, generator=g).to(dtype)
+    kn, cs = torch.rand(kr, generator=g) + 0.5, reference.rope_table(rot, 128, 10000.0)
+    cache, xf = torch.zeros(nb, PAGE, kr + rp), x.float()
+    assert reference.latent_prep(None, xf[:, H * head:], None, kn, 0, 75, rot, 1e-5, cs, inp.positions, inp.slots, cache, q=xf, heads=H, head=head, off=dk) is None
+    xd, cd = x.cuda(), torch.zeros(nb, PAGE, kr + rp, dtype=dtype, device="cuda")
+    native.latent_prep(None, xd[:, H * head:], None, kn.cuda(), 0, 75, rot, 1e-5, cs.cuda(), inp.positions.cuda(), inp.slots.cuda(), cd, q=xd, heads=H,
+                       head=head, off=dk)
+    close(xd, xf, dtype, tol16=5e-3)
+    close(cd, cache, dtype, tol16=5e-3)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("T,W,n,k,gated", [(7, 80, 76, 0, True), (1, 2048, 2048, 0, True), (33, 4096, 4090, 5, True), (3, 7168, 7168, 0, False), (5, 16384, 16384, 2, True)])
+def test_gated_norm_added_and_the_stream_normed(dtype, T, W, n, k, gated):
+    from lorax_b200.ops import native, reference
+    g = torch.Generator().manual_seed(T)
+    pad = lambda t: torch.cat([t[..., :n], torch.zeros(*t.shape[:-1], W - n)], -1)
+    res, w, nxt = pad(torch.randn(T, W, generator=g)), pad(1 + 0.2 * torch.randn(W, generator=g)), pad(torch.randn(W, generator=g))
+    y = torch.zeros(max(T * k, T), W + 128)
+    y[:, :W] = pad(torch.randn(y.shape[0], W, generator=g))
+    y, z = y.to(dtype), torch.randn(T, W + 16, generator=g).to(dtype)[:, 8: 8 + W] if gated else None
+    pairs = None
+    if k:
+        pos = torch.randperm(T * k, generator=g).view(T, k).to(torch.int32)
+        pos[0, 0] = -1
+        pairs = (pos, torch.randn(T, k, generator=g))
+    on = lambda t: t.cuda() if t is not None else None
+    for rows in (None, torch.randint(0, T, (4,), generator=g, dtype=torch.int32)):
+        rf, rd = res.clone(), res.cuda()
+        want = reference.norm_add(rf, y.float(), w, None, 0.7, 1e-5, n, torch.float32, False, pairs, gate=z.float() if gated else None, next_weight=nxt, rows=rows)
+        got = native.norm_add(rd, y.cuda(), w.cuda(), None, 0.7, 1e-5, n, dtype, False, tuple(p.cuda() for p in pairs) if k else None, gate=on(z),
+                              next_weight=nxt.cuda(), rows=on(rows))
+        close(got, want, dtype, tol16=5e-3)
+        if rows is None:
+            close(rd, rf, torch.float32, tol32=3e-5)
+    none = native.norm_add(res.cuda(), y.cuda(), w.cuda(), None, 0.7, 1e-5, n, dtype, False, next_weight=nxt.cuda(), rows=torch.empty(0, dtype=torch.int32).cuda()) \
+        if not k else torch.empty(0, W)
+    assert none.shape == (0, W)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("limit", [0.3, 1.5, 100.0])
+def test_clamped_gated_activation(dtype, limit):
+    from lorax_b200.ops import native, reference
+    x = (torch.randn(37, 2 * 96 + 40, generator=torch.Generator().manual_seed(1)) * 3).to(dtype)
+    want = reference.act_mul(x.float(), 96, "clamped_swiglu", True, limit=limit)
+    close(native.act_mul(x.cuda(), 96, "clamped_swiglu", True, limit=limit), want, dtype, tol16=4e-3, tol32=1e-6)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("step", list(STEPS))
+@pytest.mark.parametrize("buckets,mul_prev,mul_cur", [(61, 31, 5), (1, 3, 2), (997, 1 << 33, 12345678901)])
+def test_token_pairs(dtype, step, buckets, mul_prev, mul_cur):
+    from lorax_b200.ops import native, reference
+    inp, nb, _ = make_step(*STEPS[step], seed=2)
+    T, V, W = inp.positions.shape[0], 50, 80
+    g = torch.Generator().manual_seed(buckets)
+    table, vectors = torch.randn(V, W, generator=g).to(dtype), torch.randn(buckets + 1, W, generator=g).to(dtype)
+    ids, pages = (torch.randint(0, V, s, generator=g, dtype=torch.int32) for s in ((T,), (nb, PAGE)))
+    pd = pages.cuda()
+    got = native.embed_stream(ids.cuda(), table.cuda(), 0.6, bigram=(vectors.cuda(), (buckets, mul_prev, mul_cur), pd, to_dev(inp)))
+    want = reference.embed_stream(ids, table, 0.6, bigram=(vectors, (buckets, mul_prev, mul_cur), pages, inp))
+    live = [i for i in range(T) if i >= len(STEPS[step][0]) or STEPS[step][0][i] > 0]
+    assert torch.allclose(got.cpu()[live], want[live], atol=1e-6) and torch.equal(pd.cpu(), pages)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("T,E,k,shared", [(1, 8, 2, 1), (70, 16, 4, 3), (300, 40, 6, 0), (33, 200, 9, 1), (9, 1, 1, 2)])
+def test_routing_with_a_bias_and_shared_experts_of_weight_one(dtype, T, E, k, shared):
+    from lorax_b200.ops import native, reference
+    g = torch.Generator().manual_seed(T + E)
+    W = 96
+    x, wr, b = torch.randn(T, W, generator=g).to(dtype), torch.zeros((E + 8) // 8 * 8, W), torch.randn(E, generator=g)
+    wr[:E] = torch.randn(E, W, generator=g) * W ** -0.5
+    wr = wr.to(dtype)
+    kw = dict(experts=E, score="softmax", renorm=True, shared=shared, shared_gate=False)
+    want = reference.moe_route(x.float(), wr.float(), k, 0, E, bias=b, **kw)
+    r = native.moe_route(x.cuda(), wr.cuda(), k, 0, E, bias=b.cuda(), **kw)
+    clear = (r.topk_ids.cpu().long().sort(-1).values == want.topk_ids.long().sort(-1).values).all(-1)
+    assert clear.float().mean() > 0.98
+    dense = lambda r: torch.zeros(T, E).scatter_(1, r.topk_ids.cpu().long(), r.topk_w.cpu()[:, :k])
+    assert torch.allclose(dense(r)[clear], dense(want)[clear], atol=1e-5) and (r.topk_w[:, k:] == 1).all() and r.topk_w.shape[1] == k + shared
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("H,G,dk,dv,n,rot,vd", [(6, 2, 64, 64, 20, 12, 28), (16, 2, 128, 128, 128, 64, 128), (3, 3, 128, 64, 70, 70, 10), (5, 1, 256, 256, 256, 2, 250)])
+def test_normed_heads_and_values_rotated_into_the_cache(dtype, H, G, dk, dv, n, rot, vd):
+    from lorax_b200.ops import native, reference
+    inp, nb, _ = make_step([7, 0, 40], [(0, 50), (33, 5)], seed=8)
+    T = inp.positions.shape[0]
+    g = torch.Generator().manual_seed(n)
+    x = torch.randn(T, (H + G) * dk + G * dv, generator=g)
+    x[:, : (H + G) * dk].view(T, H + G, dk)[:, :, n:] = 0
+    x[:, (H + G) * dk:].view(T, G, dv)[:, :, vd:] = 0
+    x = x.to(dtype)
+    wq, wk = torch.rand(dk, generator=g) + 0.5, torch.rand(dk, generator=g) + 0.5
+    cs, vcs = reference.rope_table(rot, 128, 300.0), reference.rope_table(vd, 128, 300.0)
+    for tables in ((cs, vcs), (cs, None), (None, vcs)):
+        on = [t.cuda() if t is not None else None for t in tables]
+        cache, cd = torch.zeros(nb, G, PAGE * (dk + dv)), torch.zeros(nb, G, PAGE * (dk + dv), dtype=dtype, device="cuda")
+        xf, xd = x.float(), x.cuda()
+        reference.qk_norm_kvwrite(xf, H, G, dk, dv, n, wq, wk, 1e-3, cache, inp.slots, positions=inp.positions, cos_sin=tables[0], v_cos_sin=tables[1])
+        native.qk_norm_kvwrite(xd, H, G, dk, dv, n, wq.cuda(), wk.cuda(), 1e-3, cd, inp.slots.cuda(), positions=inp.positions.cuda(), cos_sin=on[0], v_cos_sin=on[1])
+        close(xd[:, : H * dk], xf[:, : H * dk], dtype, tol16=5e-3)
+        close(cd, cache, dtype, tol16=5e-3)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("step", list(STEPS) + ["long"])
+@pytest.mark.parametrize("H,G,dk,dv,vd,gated", [(6, 2, 64, 64, 28, False), (8, 2, 128, 128, 128, True), (3, 1, 128, 64, 64, False), (17, 1, 64, 256, 250, True), (4, 2, 128, 128, 90, False)])
+def test_attention_outputs_turned_back(dtype, step, H, G, dk, dv, vd, gated):
+    from lorax_b200.ops import native, reference
+    dec, pre = STEPS[step] if step in STEPS else ([1000, 1500], [(1000, 300), (0, 500), (129, 40)])
+    inp, nb, _ = make_step(dec, pre, seed=12)
+    T = inp.positions.shape[0]
+    q, cache = gqa_case(H, G, dk, dv, 0, inp, nb, dtype, True)
+    turn = reference.rope_table(vd, 1600, 300.0)
+    gate = torch.randn(T, H * dv, generator=torch.Generator().manual_seed(1)).to(dtype) if gated else None
+    want = torch.empty(T, H * dv)
+    reference.gqa_attn(q.float(), cache.float(), H, G, dk, dv, dk ** -0.5, 0, inp, want, gate=gate.float() if gated else None, turn_back=turn)
+    out = torch.empty(T, H * dv, dtype=dtype, device="cuda")
+    native.gqa_attn(q.cuda(), cache.cuda(), H, G, dk, dv, dk ** -0.5, 0, to_dev(inp), out, gate=gate.cuda() if gated else None, turn_back=turn.cuda())
+    native.workspace(out.device).check_status()
+    close(out, want, dtype, [i for i in range(T) if i >= len(dec) or dec[i] > 0], tol16=5e-3, tol32=4e-5)

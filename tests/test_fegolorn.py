@@ -386,7 +386,7 @@ def edge_model(kind, size, dim, vdim, width=64):
     """One layer in which the query of token 1 singles out the key of token 2: queries read the first half of the stream, keys (or the
     latent) the second half with the same matrix, and token 1 has in its first half what token 2 has in its second.  The rotated
     dimensions are left out, and the token pairs."""
-    cfg = config([attention(heads=2, kv_heads=1, dim=dim, vdim=vdim, scale=1.0, dims=4, scaling=None) if kind == "attention" else
+    cfg = config([attention(heads=2, kv_heads=1, dim=dim, vdim=vdim, scale=24.0 / dim, dims=4, scaling=None) if kind == "attention" else
                   latent(heads=2, dim=dim, rot_dim=16, vdim=vdim, kv_rank=128, size=size, scale=1.5 * dim ** -0.5)], width=width, vocab=40, scale=1.0)
     w = {k: v.float() for k, v in weights_of(cfg, seed=dim + vdim, sharp=1.0).items()}
     g = torch.Generator().manual_seed(dim)

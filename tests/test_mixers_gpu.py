@@ -587,7 +587,7 @@ def test_32_bit_product_with_bias(T, N, K):
 @pytest.mark.parametrize("H,dk,rot,dv,kv", [(3, 32, 16, 48, 80), (2, 128, 64, 128, 512), (5, 64, 48, 64, 256), (17, 64, 16, 128, 128), (4, 128, 32, 128, 128)])
 def test_latent_attention_with_windows_and_element_gates(dtype, window, step, H, dk, rot, dv, kv):
     """Both forms over queries that each match one key far better than all others: inside the window, at its edges, or just outside."""
-    from lorax_b200.ops import native, reference
+    from lorax_b200.ops import native, native_mixers, reference
     dec, pre = STEPS[step] if step in STEPS else ([1000, 1500], [(1000, 300), (0, 500), (129, 40)])
     inp, nb, _ = make_step(dec, pre, seed=6, windows=(window,))
     T, head = inp.positions.shape[0], dk + rot
@@ -619,7 +619,7 @@ def test_latent_attention_with_windows_and_element_gates(dtype, window, step, H,
         ukv = torch.cat([uk, uv], 1).reshape(H * (dk + dv), kv).contiguous().cuda()
         out = torch.zeros(T, H * dv, dtype=dtype, device="cuda")
         done = native.latent_prefill(qd, cd, ukv, gd, out, H, dk, rot, dv, scale, d, len(dec), window=window, wide_gate=True)
-        assert done == (dtype == torch.bfloat16 and dk != 32 and T - len(dec) >= native.LATENT_EXPAND_MIN_ROWS * len(pre))
+        assert done == (dtype == torch.bfloat16 and dk != 32 and T - len(dec) >= native_mixers.LATENT_EXPAND_MIN_ROWS * len(pre))
         if done:
             native.workspace(out.device).check_status()
             close(out, want, dtype, list(range(len(dec), T)))
@@ -634,7 +634,7 @@ def test_latent_preparation_without_a_query_latent(dtype, rot, rp, H, dk):
     g = torch.Generator().manual_seed(rot)
     x = torch.randn(T, H * head + kr + rp, generator=g).to(dtype)
     kn, cs = torch.rand(kr, generator=g) + 0.5, reference.rope_table(rot, 128, 10000.0)
-    cache, xf = torch.zeros(nb, PAGE, kr + rp), x.float()
+    cache, xf = torch.zeros(nb, PAGE, kr + rp), x.float().clone()
     assert reference.latent_prep(None, xf[:, H * head:], None, kn, 0, 75, rot, 1e-5, cs, inp.positions, inp.slots, cache, q=xf, heads=H, head=head, off=dk) is None
     xd, cd = x.cuda(), torch.zeros(nb, PAGE, kr + rp, dtype=dtype, device="cuda")
     native.latent_prep(None, xd[:, H * head:], None, kn.cuda(), 0, 75, rot, 1e-5, cs.cuda(), inp.positions.cuda(), inp.slots.cuda(), cd, q=xd, heads=H,
@@ -732,7 +732,7 @@ def test_normed_heads_and_values_rotated_into_the_cache(dtype, H, G, dk, dv, n, 
     for tables in ((cs, vcs), (cs, None), (None, vcs)):
         on = [t.cuda() if t is not None else None for t in tables]
         cache, cd = torch.zeros(nb, G, PAGE * (dk + dv)), torch.zeros(nb, G, PAGE * (dk + dv), dtype=dtype, device="cuda")
-        xf, xd = x.float(), x.cuda()
+        xf, xd = x.float().clone(), x.cuda()
         reference.qk_norm_kvwrite(xf, H, G, dk, dv, n, wq, wk, 1e-3, cache, inp.slots, positions=inp.positions, cos_sin=tables[0], v_cos_sin=tables[1])
         native.qk_norm_kvwrite(xd, H, G, dk, dv, n, wq.cuda(), wk.cuda(), 1e-3, cd, inp.slots.cuda(), positions=inp.positions.cuda(), cos_sin=on[0], v_cos_sin=on[1])
         close(xd[:, : H * dk], xf[:, : H * dk], dtype, tol16=5e-3)

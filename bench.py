@@ -200,7 +200,7 @@ def main():
     ap.add_argument("--no-graphs", action="store_true")
     ap.add_argument("--waiting-served-ratio", type=float, default=None, help="scheduler knob (default: the engine's)")
     ap.add_argument("--baseline-mode", action="store_true", help="NCCL collectives instead of the fused NVLink kernels")
-    ap.add_argument("--design", default=None, choices=[None, "vabunex", "sapudra", "saredra"],
+    ap.add_argument("--design", default=None, choices=[None, "vabunex", "sapudra", "saredra", "fegolorn"],
                     help="instead of the serving benchmark: prefill / decode throughput and kernel times of this design beside the closest "
                          "uniform decoder (benchmarks/bench_design.py; one JSON line per case)")
     ap.add_argument("--design-size", default="small,base", help="sizes of that design, with commas between them")

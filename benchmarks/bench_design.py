@@ -1,14 +1,15 @@
 """Prefill and decode throughput of a layer-by-layer design (random weights, layers of a real model's size) beside the closest
 uniform decoder of this framework at equal size, and the device time of every kernel of both with its share of the roofline.
 
-    python bench.py --design vabunex|sapudra|saredra [--design-size small,base] [--steps K] [--warmup W]
+    python bench.py --design vabunex|sapudra|saredra|fegolorn [--design-size small,base] [--steps K] [--warmup W]
 
 "Equal size": for Vabunex a llama-style decoder with the same width, feed-forward width, number of layer runs and attention heads of
 128; for Sapudra a Mixtral-style decoder with the same width, heads, window, layers and experts, whose gated experts (three matrices)
 have two thirds of the width, and which takes one expert more per token in place of the shared one; where the size has no experts, a
 Mistral-style decoder likewise; for Saredra two designs whose kernels are its kernels' closest relatives: Sapudra with the same width,
 heads, window, layers and experts (not gated, of 3/2 the width: the same bytes), and Vabunex with as many layers of linear attention
-whose state has the size of the state space mixer's.
+whose state has the size of the state space mixer's; for Fegolorn likewise Sapudra with the same width, heads (no window), layers and
+experts, and Vabunex with as many layers of latent attention (no window, a low-rank query) and its dense feed-forward.
 Throughput: prefill is one eager forward pass over ragged prompts, decode one CUDA-graph replay per token, both through
 `ModelRunner`, timed with CUDA events.  Kernel times: CUDA events around every operator of an eager pass, L2 flushed in front of it,
 median of the passes.  Rooflines: the measured copy bandwidth and bf16 rate of MEASURED_PEAKS.json, whichever bounds the operator.
@@ -43,6 +44,14 @@ SAREDRA_SIZES = {
     "base": dict(width=4096, triples=1, heads=32, kv=8, window=1024, ssm=128, ssm_groups=8, parts=8, state=128, experts=32, top=4, groups=(4, 2), ff=4096),
     "dense": dict(width=4096, triples=1, heads=32, kv=8, window=1024, ssm=128, ssm_groups=8, parts=8, state=128, experts=0, ff=14336),
 }
+FEGOLORN_SIZES = {
+    # width, layer pairs (latent attention with a dense feed-forward, attention with experts); heads of 128, key/value heads; rank of the
+    # latent, rotated part, window of the latent layers; width of the dense feed-forward; experts, per token, width of an expert and of the
+    # shared one (0 experts: dense in every layer)
+    "small": dict(width=2048, pairs=2, heads=16, kv=4, rank=512, rot=64, latent_window=1024, dense=8192, experts=64, top=6, ff=1024),
+    "base": dict(width=4096, pairs=2, heads=32, kv=8, rank=512, rot=64, latent_window=1024, dense=14336, experts=32, top=4, ff=4096),
+    "dense": dict(width=4096, pairs=2, heads=32, kv=8, rank=512, rot=64, latent_window=1024, dense=14336, experts=0, ff=14336),
+}
 PREFILL = [(1, 4096), (4, 2048), (1, 16384)]           # (prompts, tokens each)
 DECODE = [(16, 2048), (64, 2048), (256, 2048)]         # (rows, tokens of context)
 
@@ -73,8 +82,9 @@ def sapudra_config(s, vocab=32000):
                    router=dict(experts=s["experts"], top=s["top"], scale=2.5, groups=dict(count=s["groups"][0], keep=s["groups"][1])))
     else:
         mlp = dict(kind="dense", ff=s["ff"])
-    layer = dict(type="attention", mlp=mlp, mixer=dict(heads=s["heads"], kv_heads=s["kv"], dim=128, vdim=128, scale=128 ** -0.5,
-                                                       mask=dict(size=s["window"])))
+    layer = dict(type="attention", mlp=mlp, mixer=dict(heads=s["heads"], kv_heads=s["kv"], dim=128, vdim=128, scale=128 ** -0.5))
+    if s.get("window"):
+        layer["mixer"]["mask"] = dict(size=s["window"])
     return dict(architecture="Sapudra", vocab=vocab, width=s["width"], norm=dict(eps=1e-5), residual_mult=0.3, logit_softcap=30.0,
                 max_positions=20000, layers=[layer] * s["layers"])
 
@@ -122,10 +132,38 @@ def linear_attention_of_that_size(s, runs, vocab=32000):
                                       layers=[lin] * runs))
 
 
+def fegolorn_config(s, vocab=32000):
+    dense = dict(kind="dense", ff=s["dense"], limit=7.0)
+    mlp = dict(kind="moe", expert=dict(ff=s["ff"]), shared=dict(ff=s["ff"]), router=dict(experts=s["experts"], top=s["top"])) if s["experts"] else dense
+    bands = dict(factor=8.0, low=1.0, high=4.0, original=8192)
+    lat = dict(type="latent_attention", mlp=dense, mixer=dict(heads=s["heads"], dim=128, rot_dim=s["rot"], vdim=128, kv_rank=s["rank"],
+                                                              scale=(128 + s["rot"]) ** -0.5, mask=dict(size=s["latent_window"]),
+                                                              rot=dict(base=10000.0, dims=s["rot"])))
+    att = dict(type="attention", mlp=mlp, mixer=dict(heads=s["heads"], kv_heads=s["kv"], dim=128, vdim=128, scale=128 ** -0.5,
+                                                     rot=dict(base=500000.0, dims=128, scaling=bands)))
+    return dict(architecture="Fegolorn", vocab=vocab, width=s["width"], norm=dict(eps=1e-5), logit_softcap=30.0, layers=[lat, att] * s["pairs"],
+                embedding=dict(scale=1.0, bigram=dict(buckets=16381, mul_prev=8191, mul_cur=127)))
+
+
+def sapudra_with_those_experts(s, runs, vocab=32000):
+    from lorax_b200.config import ModelConfig
+    return ModelConfig.from_dict(sapudra_config(dict(s, layers=runs, ff=s["ff"] * 3 // 2, groups=(1, 1)), vocab))
+
+
+def latent_attention_of_that_size(s, runs, vocab=32000):
+    from lorax_b200.config import ModelConfig
+    lat = dict(type="latent_attention", mlp=dict(kind="dense", ff=s["dense"]),
+               mixer=dict(heads=s["heads"], dim=128, rot_dim=s["rot"], vdim=128, q_rank=s["width"] // 2, kv_rank=s["rank"],
+                          scale=(128 + s["rot"]) ** -0.5, rot=dict(base=10000.0, dims=s["rot"])))
+    return ModelConfig.from_dict(dict(architecture="Vabunex", vocab=vocab, width=s["width"], norm=dict(eps=1e-5), embedding=dict(scale=1.0),
+                                      layers=[lat] * runs))
+
+
 # sizes, configuration of the design, and what runs beside it
 DESIGNS = {"vabunex": (VABUNEX_SIZES, vabunex_config, [("llama-like", llama_like)]),
            "sapudra": (SAPUDRA_SIZES, sapudra_config, [("mixtral-like", mixtral_like)]),
-           "saredra": (SAREDRA_SIZES, saredra_config, [("sapudra", sapudra_of_that_size), ("linear-attention", linear_attention_of_that_size)])}
+           "saredra": (SAREDRA_SIZES, saredra_config, [("sapudra", sapudra_of_that_size), ("linear-attention", linear_attention_of_that_size)]),
+           "fegolorn": (FEGOLORN_SIZES, fegolorn_config, [("sapudra", sapudra_with_those_experts), ("latent-attention", latent_attention_of_that_size)])}
 
 
 def peaks():
@@ -181,7 +219,15 @@ class OpTimer:
     def cost(self, name, a, kw):
         """(label, bytes, flops) of one call."""
         nb = lambda *ts: sum(t.numel() * t.element_size() for t in ts if t is not None)
-        q = self.info                                       # rows, causal (query, key) pairs, cached tokens read, sequences, decode?
+        q = self.info                                       # sequences, their tokens, decode?, window of a uniform model
+
+        def pairs(window):
+            """(query, key) pairs of the step, a decode row's keys counting once."""
+            n, w = q["length"], window if window and window > 0 else 1 << 30
+            if q["decode"]:
+                return q["seqs"] * min(n, w)
+            out = max(0, n - w)
+            return q["seqs"] * (n * (n + 1) // 2 - out * (out + 1) // 2)
         if name == "gemm":
             x, w = a[0], a[1]
             return (f"gemm [{x.shape[0]}, {w.shape[1]}] x [{w.shape[0]}]", nb(x, w) + x.shape[0] * w.shape[0] * 2, 2 * x.shape[0] * w.numel())
@@ -217,29 +263,34 @@ class OpTimer:
         if name == "latent_attn":
             H, kv, rot = a[3], a[4], a[7]
             T = a[0].shape[0]
+            ctx = pairs(kw.get("window"))
             if q["decode"]:                                 # absorbed: rows of the cache against every head
-                return (name, q["ctx"] * (kv + rot) * 2 + T * H * (2 * kv + rot) * 2, 2 * q["ctx"] * H * (2 * kv + rot))
-            return (name, 0, 2 * q["pairs"] * H * (128 + rot + 128))       # the products of plain multi-head attention
+                return (name, ctx * (kv + rot) * 2 + T * H * (2 * kv + rot) * 2, 2 * ctx * H * (2 * kv + rot))
+            return (name, 0, 2 * ctx * H * (128 + rot + 128))       # the products of plain multi-head attention
         if name == "latent_prefill":                        # expansion of the contexts, then multi-head attention
             w, H, dk, rot, dv = a[2], *a[5:9]
-            return (name, 0, 2 * q["ctx"] * w.numel() + 2 * q["pairs"] * H * (dk + rot + dv))
+            return (name, 0, 2 * q["seqs"] * q["length"] * w.numel() + 2 * pairs(kw.get("window")) * H * (dk + rot + dv))
         if name == "attn_decode":
             nh, nkv, d = a[4], a[5], a[6]
-            return (name, q["ctx"] * nkv * 2 * d * 2 + a[0].shape[0] * nh * d * 4, 4 * q["ctx"] * nh * d)
+            ctx = pairs(q["window"])
+            return (name, ctx * nkv * 2 * d * 2 + a[0].shape[0] * nh * d * 4, 4 * ctx * nh * d)
         if name == "attn_prefill":
             nh, d = a[7], a[9]
-            return (name, 0, 4 * q["pairs"] * nh * d)
+            return (name, 0, 4 * pairs(q["window"]) * nh * d)
         if name == "gqa_attn":
             H, G, dk, dv = a[2:6]
+            ctx = pairs(a[7])
             if q["decode"]:
-                return (name, q["ctx"] * G * (dk + dv) * 2 + a[0].shape[0] * H * (dk + dv) * 2, 2 * q["ctx"] * H * (dk + dv))
-            return (name, 0, 2 * q["pairs"] * H * (dk + dv))
+                return (name, ctx * G * (dk + dv) * 2 + a[0].shape[0] * H * (dk + dv) * 2, 2 * ctx * H * (dk + dv))
+            return (name, 0, 2 * ctx * H * (dk + dv))
         if name == "qk_norm_kvwrite":
             T, H, G, dk, dv = a[0].shape[0], *a[1:5]
             return (name, T * 2 * (H * dk + G * (dk + dv)) * 2, 0)
         if name == "norm_add":
-            r, y = a[0], a[1]
-            return ("norm_add" + (" of experts" if kw.get("pairs") is not None else ""), nb(r) * 2 + y.shape[0] * r.shape[1] * 2 + r.numel() * 2, 0)
+            r, y, pr, z = a[0], a[1], kw.get("pairs"), kw.get("gate")
+            n = (kw["rows"] if kw.get("rows") is not None else r).shape[0] * r.shape[1]
+            per = 2 * (pr[0].shape[1] if pr is not None else 1) + (2 if z is not None else 0) + (4 if kw.get("rows") is not None else 8) + 2
+            return ("norm_add" + (" of experts" if pr is not None else "") + (" with gate and next norm" if z is not None else ""), n * per, 0)
         if name == "moe_route":
             x, w, k = a[:3]
             rows = k + (1 if kw.get("shared") else 0)
@@ -271,11 +322,12 @@ class OpTimer:
             T, nh, nkv, d = a[0].shape[0], a[5], a[6], a[7]
             return (name, T * (2 * (nh + nkv) * d + 3 * nkv * d) * 2, 0)
         if name == "latent_prep":
-            return (name, a[0].shape[0] * (a[2].shape[0] * 2 + a[3].shape[0] * 2) * 2, 0)
+            cq, q_rot = a[2].shape[0] if a[2] is not None else 0, kw.get("heads", 0) * a[6]
+            return (name, a[1].shape[0] * (cq + a[3].shape[0] + a[6] + q_rot) * 4, 0)
         if name == "rope_pairs":
             return (name, a[0].shape[0] * a[3] * a[6] * 4, 0)
         if name in ("embed", "embed_stream"):
-            per = 4 if name == "embed" else 6 + (2 if kw.get("pos") is not None else 0) + (2 if kw.get("copy") is not None else 0)
+            per = 4 if name == "embed" else 6 + (2 if kw.get("pos") is not None else 0) + (2 if kw.get("copy") is not None else 0) + (2 if kw.get("bigram") is not None else 0)
             return (name, a[0].shape[0] * a[1].shape[1] * per, 0)
         return (name, nb(*[t for t in a if hasattr(t, "numel")]), 0)
 
@@ -318,7 +370,7 @@ def main(args):
         for size in args.design_size.split(","):
             s = sizes[size]
             ours = ModelConfig.from_dict(config_of(s))
-            window = s.get("window", 1 << 30)
+            window = s.get("window", 0)
             for name, cfg in [(args.design, ours)] + [(n, like(s, len(ours.layer_schedule))) for n, like in likes]:
                 model = DecoderModel.random_init_on_device(cfg, dev, torch.bfloat16, seed=0, max_positions=20000)
                 model.use_native_layers = True
@@ -338,13 +390,12 @@ def main(args):
                             run.install(rows, torch.randint(0, cfg.vocab_size, (n,), generator=g).tolist(), [length] * n, blocks, [0] * n, list(range(1, n + 1)))
                             run.resort()
                             step = lambda: run.decode()
-                            info = dict(decode=True, seqs=n, ctx=n * min(length, window), pairs=n * min(length, window))
+                            info = dict(decode=True, seqs=n, length=length, window=window)
                             toks = n
                         else:
                             inp, _ = run._prefill_inputs(items)
                             step = lambda: model.forward(inp, kv.layers)
-                            info = dict(decode=False, seqs=n, ctx=n * length,
-                                        pairs=n * (length * (length + 1) // 2 - max(0, length - window) * (max(0, length - window) + 1) // 2))
+                            info = dict(decode=False, seqs=n, length=length, window=window)
                             toks = n * length
                         time.sleep(1.0)                      # no case inherits the heat of the one before
                         for _ in range(warm):

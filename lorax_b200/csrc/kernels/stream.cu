@@ -220,7 +220,7 @@ LX_DEVICE float gate_f(float z) {
 }
 
 template <typename T, bool PAIRS, int NV, bool NEXT>
-__global__ void __launch_bounds__(kNsThreads) norm_add_kernel(const NormAddParams p) {
+__global__ void __launch_bounds__(kNsThreads, NEXT && NV <= 2 ? 4 : 1) norm_add_kernel(const NormAddParams p) {
   pdl_trigger();
   pdl_wait();
   __shared__ float red[kNsThreads / 32];
@@ -253,18 +253,27 @@ __global__ void __launch_bounds__(kNsThreads) norm_add_kernel(const NormAddParam
       for (int q = 0; q < 8; ++q) v[it][q] *= gate_f<T>(g[q]);
     }
   }
-  norm_row<NV>(v, p.w, p.b, p.W, p.n, p.inv_n, p.eps, p.layernorm, 0.f, red);
   float* res = p.residual + (long long)t * p.W;
   T* copy = reinterpret_cast<T*>(p.copy);
   if constexpr (NEXT) {
+    constexpr bool EARLY = NV <= 2;            // the stream's row is on its way while the first norm is formed
+    float x[EARLY ? NV : 1][8];
+    if constexpr (EARLY) {
+#pragma unroll
+      for (int it = 0; it < NV; ++it) {
+        const int c = (threadIdx.x + it * blockDim.x) * 8;
+        if (c < p.W) load8(res + c, x[it]);
+      }
+    }
+    norm_row<NV>(v, p.w, nullptr, p.W, p.n, p.inv_n, p.eps, 0, 0.f, red);
 #pragma unroll
     for (int it = 0; it < NV; ++it) {
       const int c = (threadIdx.x + it * blockDim.x) * 8;
       if (c < p.W) {
-        float x[8];
-        load8(res + c, x);
+        float (&own)[8] = x[EARLY ? it : 0];
+        if constexpr (!EARLY) load8(res + c, own);
 #pragma unroll
-        for (int q = 0; q < 8; ++q) v[it][q] = fmaf(p.mult, v[it][q], x[q]);
+        for (int q = 0; q < 8; ++q) v[it][q] = fmaf(p.mult, v[it][q], own[q]);
         if (p.rows == nullptr) store8(res + c, v[it]);
       }
     }
@@ -276,6 +285,7 @@ __global__ void __launch_bounds__(kNsThreads) norm_add_kernel(const NormAddParam
     }
     return;
   }
+  norm_row<NV>(v, p.w, p.b, p.W, p.n, p.inv_n, p.eps, p.layernorm, 0.f, red);
 #pragma unroll
   for (int it = 0; it < NV; ++it) {
     const int c = (threadIdx.x + it * blockDim.x) * 8;
@@ -697,6 +707,7 @@ int lx_norm_add(const void* params, int T, int f32, void* stream) {
   const NormAddParams& p = *reinterpret_cast<const NormAddParams*>(params);
   if (T <= 0) return 0;
   if (p.W % 8 != 0 || p.W > kNsThreads * kNsMaxVec * 8 || p.n <= 0 || p.n > p.W || p.ldy % 8 != 0 || p.ldy < p.W) return -1;
+  if (p.next_w != nullptr && (p.b != nullptr || p.layernorm)) return -3;
   if (p.next_w != nullptr ? p.copy == nullptr || (p.gate != nullptr && p.ldg % 8 != 0) : p.gate != nullptr || p.rows != nullptr) return -2;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const int threads = p.W / 8 >= kNsThreads ? kNsThreads : (p.W / 8 + 31) / 32 * 32;

@@ -385,14 +385,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_
               float v[8];
 #pragma unroll
               for (int u = 0; u < 8; ++u) v[u] = (o[c + q + u] + __uint_as_float(r[q + u])) * inv;
-              if (p.tail.turn != nullptr) {
-#pragma unroll
-                for (int u = 0; u < 8; u += 2) {
-                  const float2 back = attn_turn_back(p.tail, make_float2(v[u], v[u + 1]), c + q + u, cache + qi);
-                  v[u] = back.x;
-                  v[u + 1] = back.y;
-                }
-              }
+              if (p.tail.turn != nullptr) attn_turn_back8(p.tail, v, c + q, cache + qi);
               if (grow != nullptr) {
                 const uint4 g = *reinterpret_cast<const uint4*>(grow + c + q);
                 const uint32_t gw[4] = {g.x, g.y, g.z, g.w};

@@ -40,6 +40,29 @@ LX_DEVICE float2 attn_turn_back(const AttnTail& tail, float2 o, int d, int pos) 
   return make_float2(o.x * c + o.y * s, o.y * c - o.x * s);
 }
 
+// The same for columns [d, d + 8), d a multiple of eight.
+LX_DEVICE void attn_turn_back8(const AttnTail& tail, float (&v)[8], int d, int pos) {
+  if (tail.turn_dims % 8 == 0) {
+    if (d >= tail.turn_dims) return;
+    const float* cs = tail.turn + (long long)min(pos, tail.turn_rows - 1) * tail.turn_dims + (d >> 1);
+    const float4 c = __ldg(reinterpret_cast<const float4*>(cs)), s = __ldg(reinterpret_cast<const float4*>(cs + (tail.turn_dims >> 1)));
+    const float co[4] = {c.x, c.y, c.z, c.w}, si[4] = {s.x, s.y, s.z, s.w};
+#pragma unroll
+    for (int u = 0; u < 4; ++u) {
+      const float a = v[2 * u], b = v[2 * u + 1];
+      v[2 * u] = a * co[u] + b * si[u];
+      v[2 * u + 1] = b * co[u] - a * si[u];
+    }
+    return;
+  }
+#pragma unroll
+  for (int u = 0; u < 8; u += 2) {
+    const float2 o = attn_turn_back(tail, make_float2(v[u], v[u + 1]), d + u, pos);
+    v[u] = o.x;
+    v[u + 1] = o.y;
+  }
+}
+
 // One finished output element.
 LX_DEVICE float attn_tail(const AttnTail& tail, float o, long long t, int col) {
   o *= tail.scale;

@@ -495,7 +495,7 @@ int lx_attn_prefill_tc(const void* q, long long ldq, int T, const void* kv, int 
                              window, scale, softcap, alibi, wide, lx::AttnTail{}, status, stream);
 }
 
-// The same with fp32 softmax weights, a sink per head, outputs turned back, a gate [T, ldg] and a factor on them (gqa.cu has the contract).
+// The same with fp32 softmax weights, a sink per head, outputs turned back, a gate [T, ldg] and a factor on them (gqa.cu has the details).
 int lx_gqa_prefill_tc(const void* q, long long ldq, int T, const void* kv, int num_blocks, const int* block_tables, int max_blocks,
                       const int* cu_q, const int* cache_lens, const int* tile_seq, const int* tile_q0, int num_tiles, void* out, long long ldo,
                       int nh, int nkv, int d, int window, float scale, float softcap, const float* sink, const void* gate, long long ldg,
